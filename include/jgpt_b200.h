@@ -330,6 +330,73 @@ JGPT_API int32_t jgpt_generate_greedy_rolling(jgpt_model model, jgpt_kvpool pool
 
 
 /* ---------------------------------------------------------------------------------------------
+ * Layered decoders: models described layer by layer instead of by the fixed block above.  The handle is
+ * a jgpt_model: jgpt_forward_prefill[_batch], jgpt_forward_decode[_sample], jgpt_generate_greedy, the
+ * scheduler and jgpt_model_destroy take it; entry points that need the fixed block return
+ * JGPT_ERR_UNSUPPORTED.  The reference has one block design only (J/model/DecoderBlock.java).
+ *
+ * A layer is x += sum over its branches of out_scale * mixer(LN1(x)), then x += ff(LN2(x)) when ff > 0;
+ * norms are layer norms with weight and bias, ff is W_down (gelu_tanh(W_gate h) * (W_up h)).
+ * ------------------------------------------------------------------------------------------- */
+enum {
+    JGPT_MIX_ATTENTION = 1, /* softmax attention over paged K/V, no rotation, positions of the query's chunk only */
+    JGPT_MIX_GLA = 2,       /* gated linear attention: S <- diag(a) S + k v^T, a = sigmoid(W_a2 W_a1 h + bias)^(1/tau) */
+    JGPT_MIX_DELTA = 3      /* gated delta rule with a decay per key channel and short convolutions on q, k, v */
+};
+enum { JGPT_DTYPE_BF16 = 0, /* bf16 products, activations and K/V; norms, scores, recurrences and the residual in fp32 */
+       JGPT_DTYPE_F32 = 1 /* everything in fp32 (no reduced-precision matrix mode) */ };
+#define JGPT_MAX_BRANCHES 2
+typedef struct {
+    int32_t kind;             /* JGPT_MIX_* */
+    int32_t heads, kv_heads;  /* attention: query / key heads; delta: value heads / query-key heads */
+    int32_t dim, vdim;        /* query-key and value head size, up to 256 each */
+    int32_t chunk;            /* attention: position i sees j <= i with i / chunk == j / chunk; 0: every j <= i */
+    int32_t gate;             /* attention: output of head h times sigmoid(W_g h)_h */
+    int32_t taps;             /* delta: columns of the causal convolutions, 1..8 */
+    int32_t rank_a, rank_g;   /* inner sizes of the two-factor decay and output-gate projections */
+    float score_scale;        /* attention */
+    float tau;                /* gla */
+    float out_scale;
+} jgpt_mixer_spec;
+typedef struct {
+    int32_t n_branches;
+    jgpt_mixer_spec branch[JGPT_MAX_BRANCHES];
+    int32_t ff; /* 0: no feed-forward part */
+} jgpt_layer_spec;
+typedef struct {
+    int32_t vocab, width, max_positions, n_layers;
+    int32_t embed_norm; /* layer norm behind the embedding */
+    float eps, embed_scale, logit_scale;
+} jgpt_decoder_spec;
+/* Tensors.  Of the model: layer = branch = -1; of a layer: branch = -1; of a mixer: layer and branch. */
+enum {
+    JGPT_W_EMBED = 0, JGPT_W_POS, JGPT_W_EMBED_NORM, JGPT_W_EMBED_NORM_B, JGPT_W_FINAL_NORM, JGPT_W_FINAL_NORM_B,
+    JGPT_W_NORM1 = 10, JGPT_W_NORM1_B, JGPT_W_NORM2, JGPT_W_NORM2_B, JGPT_W_FF_GATE, JGPT_W_FF_UP, JGPT_W_FF_DOWN,
+    JGPT_W_Q = 20, JGPT_W_K, JGPT_W_V, JGPT_W_O, JGPT_W_G /* output gate */, JGPT_W_B /* step size */, JGPT_W_A1, JGPT_W_A2,
+    JGPT_W_DECAY_BIAS, JGPT_W_A_LOG, JGPT_W_G1, JGPT_W_G2, JGPT_W_HEAD_NORM, JGPT_W_CONV_Q, JGPT_W_CONV_K, JGPT_W_CONV_V
+};
+
+/* max_rows bounds the rows (tokens) of one step. */
+JGPT_API int32_t jgpt_decoder_create(jgpt_ctx ctx, const jgpt_decoder_spec *spec, const jgpt_layer_spec *layers, int32_t dtype,
+                                     int32_t max_rows, jgpt_model *out);
+/* host: fp32 [rows, cols], linear weights [out, in]; vectors have rows = 1.  The library stores what dtype asks for. */
+JGPT_API int32_t jgpt_decoder_set_tensor(jgpt_model model, int32_t layer, int32_t branch, int32_t role, const float *host,
+                                         int32_t rows, int32_t cols);
+/* A pool with the pages the model's attention layers need and a slot of recurrent state per sequence.  Blocks, tables,
+ * sequence slots and eviction are those of jgpt_kvpool_create; a slot's state starts over when its length is 0. */
+JGPT_API int32_t jgpt_decoder_new_pool(jgpt_model model, int32_t n_blocks, int32_t max_seqs, int32_t max_blocks_per_seq,
+                                       jgpt_kvpool *out);
+/* One step over a mixed batch: entry i brings tokens ids[starts[i] .. starts[i+1]) of sequence seq_ids[i] - a whole prompt,
+ * a portion of one, or a decoded token - which continue what the sequence holds (starts has n + 1 entries, starts[0] = 0).
+ * want_rows: rows of ids whose logits are asked for; logits_host [n_want, vocab] and next_tokens_host [n_want] (greedy
+ * argmax, ties -> lowest id) may be NULL.  Blocks are reserved for all entries or for none (JGPT_ERR_POOL_EXHAUSTED). */
+JGPT_API int32_t jgpt_forward_step(jgpt_model model, jgpt_kvpool pool, int32_t n, const int32_t *seq_ids_host,
+                                   const int32_t *starts_host, const int32_t *ids_host, int32_t n_want,
+                                   const int32_t *want_rows_host, float *logits_host, int32_t *next_tokens_host);
+/* Copies the residual after every layer of the NEXT step to host, [layers][rows][width] (inspection; NULL: off). */
+JGPT_API int32_t jgpt_decoder_capture_layers(jgpt_model model, float *host, uint64_t n_floats);
+
+/* ---------------------------------------------------------------------------------------------
  * Continuous-batching scheduler (one model + one pool on one GPU).  The reference generates one
  * sequence per call with a fresh KvCacheGpu (J/model/GptAutoregressiveGenerator.java:108-206); the
  * per-sequence rules are kept (greedy argmax, lowest-index ties, stop on sampled id 0), the batching

@@ -96,6 +96,11 @@ public final class JgptB200 {
     private static final MethodHandle H_SAMPLE_NEXT_TOKEN = bind("jgpt_sample_next_token", FunctionDescriptor.of(JAVA_INT, ADDRESS, JAVA_INT, JAVA_FLOAT, JAVA_INT, JAVA_FLOAT, ADDRESS));
     private static final MethodHandle H_GENERATE_GREEDY = bind("jgpt_generate_greedy", FunctionDescriptor.of(JAVA_INT, JAVA_LONG, JAVA_LONG, ADDRESS, JAVA_INT, JAVA_INT, ADDRESS, ADDRESS));
     private static final MethodHandle H_GENERATE_GREEDY_ROLLING = bind("jgpt_generate_greedy_rolling", FunctionDescriptor.of(JAVA_INT, JAVA_LONG, JAVA_LONG, ADDRESS, JAVA_INT, JAVA_INT, ADDRESS, ADDRESS));
+    private static final MethodHandle H_DECODER_CREATE = bind("jgpt_decoder_create", FunctionDescriptor.of(JAVA_INT, JAVA_LONG, ADDRESS, ADDRESS, JAVA_INT, JAVA_INT, ADDRESS));
+    private static final MethodHandle H_DECODER_SET_TENSOR = bind("jgpt_decoder_set_tensor", FunctionDescriptor.of(JAVA_INT, JAVA_LONG, JAVA_INT, JAVA_INT, JAVA_INT, ADDRESS, JAVA_INT, JAVA_INT));
+    private static final MethodHandle H_DECODER_NEW_POOL = bind("jgpt_decoder_new_pool", FunctionDescriptor.of(JAVA_INT, JAVA_LONG, JAVA_INT, JAVA_INT, JAVA_INT, ADDRESS));
+    private static final MethodHandle H_FORWARD_STEP = bind("jgpt_forward_step", FunctionDescriptor.of(JAVA_INT, JAVA_LONG, JAVA_LONG, JAVA_INT, ADDRESS, ADDRESS, ADDRESS, JAVA_INT, ADDRESS, ADDRESS, ADDRESS));
+    private static final MethodHandle H_DECODER_CAPTURE_LAYERS = bind("jgpt_decoder_capture_layers", FunctionDescriptor.of(JAVA_INT, JAVA_LONG, ADDRESS, JAVA_LONG));
     private static final MethodHandle H_SCHED_CREATE = bind("jgpt_sched_create", FunctionDescriptor.of(JAVA_INT, JAVA_LONG, JAVA_LONG, JAVA_INT, JAVA_INT, JAVA_INT, ADDRESS));
     private static final MethodHandle H_SCHED_DESTROY = bind("jgpt_sched_destroy", FunctionDescriptor.of(JAVA_INT, JAVA_LONG));
     private static final MethodHandle H_SCHED_SUBMIT = bind("jgpt_sched_submit", FunctionDescriptor.of(JAVA_INT, JAVA_LONG, ADDRESS, JAVA_INT, JAVA_INT, ADDRESS));
@@ -430,6 +435,31 @@ public final class JgptB200 {
     /** jgpt_generate_greedy_rolling */
     public static int generateGreedyRolling(long model, long pool, MemorySegment prompt_host, int S, int max_new, MemorySegment out_host, MemorySegment n_sampled_out) {
         try { return (int) H_GENERATE_GREEDY_ROLLING.invokeExact(model, pool, promptHost, S, maxNew, outHost, nSampledOut); } catch (Throwable t) { throw rethrow(t); }
+    }
+
+    /** jgpt_decoder_create */
+    public static int decoderCreate(long ctx, MemorySegment spec, MemorySegment layers, int dtype, int maxRows, MemorySegment out) {
+        try { return (int) H_DECODER_CREATE.invokeExact(ctx, spec, layers, dtype, maxRows, out); } catch (Throwable t) { throw rethrow(t); }
+    }
+
+    /** jgpt_decoder_set_tensor */
+    public static int decoderSetTensor(long model, int layer, int branch, int role, MemorySegment host, int rows, int cols) {
+        try { return (int) H_DECODER_SET_TENSOR.invokeExact(model, layer, branch, role, host, rows, cols); } catch (Throwable t) { throw rethrow(t); }
+    }
+
+    /** jgpt_decoder_new_pool */
+    public static int decoderNewPool(long model, int nBlocks, int maxSeqs, int maxBlocksPerSeq, MemorySegment out) {
+        try { return (int) H_DECODER_NEW_POOL.invokeExact(model, nBlocks, maxSeqs, maxBlocksPerSeq, out); } catch (Throwable t) { throw rethrow(t); }
+    }
+
+    /** jgpt_forward_step */
+    public static int forwardStep(long model, long pool, int n, MemorySegment seqIds, MemorySegment starts, MemorySegment ids, int nWant, MemorySegment wantRows, MemorySegment logits, MemorySegment nextTokens) {
+        try { return (int) H_FORWARD_STEP.invokeExact(model, pool, n, seqIds, starts, ids, nWant, wantRows, logits, nextTokens); } catch (Throwable t) { throw rethrow(t); }
+    }
+
+    /** jgpt_decoder_capture_layers */
+    public static int decoderCaptureLayers(long model, MemorySegment host, long nFloats) {
+        try { return (int) H_DECODER_CAPTURE_LAYERS.invokeExact(model, host, nFloats); } catch (Throwable t) { throw rethrow(t); }
     }
 
     /** jgpt_sched_create */

@@ -9,4 +9,6 @@ from .binding import JgptError, PoolExhausted, load  # noqa: F401
 from .runtime import Context, DeviceBuffer  # noqa: F401
 from .kv_cache import KvPool, KvCacheGpu  # noqa: F401
 from .model import GPTModel  # noqa: F401
+from .decoder import DecoderConfig, DecoderModel, DecoderPool  # noqa: F401
+from .registry import describe, load_model  # noqa: F401
 from .scheduler import ContinuousBatcher, TokenGather, pack_pairs, shard_requests, unpack_pairs  # noqa: F401

@@ -1122,6 +1122,7 @@ static int32_t decode_common(jgpt_kvpool h, int32_t layer0, int32_t n_layers, co
                              float *out, bool fused) {
     Pool *p = pool_registry().get(h);
     JGPT_REQUIRE(p, JGPT_ERR_BAD_HANDLE, "bad kvpool handle");
+    JGPT_REQUIRE(!p->layered, JGPT_ERR_UNSUPPORTED, "not available on a layered decoder's pool");
     JGPT_CUDA_TRY(make_current(p->ctx));
     JGPT_REQUIRE(n_layers >= 1 && layer0 >= 0 && layer0 + n_layers <= p->layers, JGPT_ERR_OUT_OF_RANGE,
                  "layers [%d, %d) outside [0,%d)", layer0, layer0 + n_layers, p->layers);
@@ -1153,6 +1154,7 @@ int32_t jgpt_attn_decode_append_host(jgpt_kvpool pool, int32_t layer0, int32_t n
                                      const int32_t *rope_pos_host, const int32_t *lens_host, int32_t n, float *out_host) {
     Pool *p = pool_registry().get(pool);
     JGPT_REQUIRE(p, JGPT_ERR_BAD_HANDLE, "bad kvpool handle");
+    JGPT_REQUIRE(!p->layered, JGPT_ERR_UNSUPPORTED, "not available on a layered decoder's pool");
     JGPT_CUDA_TRY(make_current(p->ctx));
     if (n == 0) return JGPT_OK;
     JGPT_REQUIRE(n > 0 && n_layers >= 1 && q_host && k_host && v_host && seq_ids_host && rope_pos_host && lens_host && out_host,
@@ -1474,6 +1476,7 @@ extern "C" int32_t jgpt_attn_decode_static_scratch(jgpt_kvpool pool, int32_t lay
                                                    const int32_t *lens_dev, int32_t n, int32_t max_len, float *out_dev) {
     Pool *p = pool_registry().get(pool);
     JGPT_REQUIRE(p, JGPT_ERR_BAD_HANDLE, "bad kvpool handle");
+    JGPT_REQUIRE(!p->layered, JGPT_ERR_UNSUPPORTED, "not available on a layered decoder's pool");
     JGPT_CUDA_TRY(make_current(p->ctx));
     JGPT_REQUIRE(layer >= 0 && layer < p->layers, JGPT_ERR_OUT_OF_RANGE, "layer %d outside [0,%d)", layer, p->layers);
     JGPT_REQUIRE(p->dhead == 4 || p->dhead == 8 || p->dhead == 16 || p->dhead == 32, JGPT_ERR_UNSUPPORTED,

@@ -521,6 +521,7 @@ extern "C" int32_t jgpt_attn_prefill(jgpt_kvpool pool, int32_t layer, const floa
                                      const int32_t *rope_offsets_host, int32_t n_seqs, float *out_dev) {
     Pool *p = pool_registry().get(pool);
     JGPT_REQUIRE(p, JGPT_ERR_BAD_HANDLE, "bad kvpool handle");
+    JGPT_REQUIRE(!p->layered, JGPT_ERR_UNSUPPORTED, "not available on a layered decoder's pool");
     JGPT_CUDA_TRY(make_current(p->ctx));
     JGPT_REQUIRE(layer >= 0 && layer < p->layers, JGPT_ERR_OUT_OF_RANGE, "layer %d outside [0,%d)", layer, p->layers);
     if (n_seqs == 0) return JGPT_OK;

@@ -60,10 +60,17 @@ struct SeqState {
     bool evictable = false;
     int len = 0;
     uint64_t tick = 0;
+    int conv_set = 0;  // which copy of the convolution history is current (layered pools)
     std::vector<int> blocks;
 };
 
 constexpr int kBlockTokens = 16;
+
+// Pages of one attention layer of a layered pool: [n_blocks][heads][K 16 x dim | V 16 x dim] elements at `offset` bytes.
+struct KvLayerGeom {
+    int heads = 0, dim = 0;
+    uint64_t offset = 0, block_bytes = 0;
+};
 
 struct Pool {
     Ctx *ctx = nullptr;
@@ -72,6 +79,14 @@ struct Pool {
     // device
     __half *kv = nullptr;      // [layers][n_blocks][heads][2][16][dhead]
     uint64_t kv_bytes = 0;
+    // Layered pools (decoder.cu): every attention layer has its own geometry, and every sequence slot carries the recurrent
+    // state of its layers.  Blocks, tables and the host allocator are shared with the uniform form; kv is null.
+    bool layered = false;
+    int elem_bytes = 2;
+    std::vector<KvLayerGeom> vlayers;
+    uint8_t *vkv = nullptr;
+    uint8_t *state = nullptr;      // [max_seqs] x state_stride bytes; starts from zeros at position 0, so never cleared
+    uint64_t state_stride = 0;
     int *d_table = nullptr;    // [max_seqs][max_blocks_per_seq], -1 = unmapped
     float2 *d_rope = nullptr;  // [max_positions][dhead/2] (cos, sin)
     float *d_partials = nullptr;  // split-K scratch

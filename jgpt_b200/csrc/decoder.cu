@@ -1,0 +1,713 @@
+// Layered decoder: configuration, weights, step function.
+//
+// A layer is  x <- x + sum of its mixer branches(LN1(x)),  then  x <- x + ff(LN2(x))  when it has a feed-forward part.
+// All branches of a layer read the same normalised rows, so their input projections are ONE product over concatenated
+// weights, and their output projections are ONE product over concatenated (gated, scaled) head outputs that adds to the
+// residual in its epilogue:
+//
+//   LN1 -> proj = h W_in^T -> [z = low-rank second factors] -> mixer kernels -> x += mixed W_out^T -> LN2 -> gelu pair -> x += act W_down^T
+//
+// The residual x is fp32; rows entering a product are bf16 (or fp32 in the exact mode).  Head sizes are padded with zero
+// weights to what the kernels take, so every size of a configuration works; sums over a head use the true size.
+#include "decoder.cuh"
+
+#include <algorithm>
+#include <cmath>
+#include <memory>
+
+#include "gemm_nt.cuh"
+#include "mixers.cuh"
+
+namespace jgpt {
+
+static int up(int n, int m) { return (n + m - 1) / m * m; }
+
+struct DBranch {
+    jgpt_mixer_spec s{};
+    int D = 0, DK = 0, DV = 0;          // padded head sizes (attention: D; recurrent: DK, DV)
+    int q = -1, k = -1, v = -1, g = -1, a1 = -1, b = -1, g1 = -1;  // column offsets inside proj
+    int za = -1, zg = -1;               // column offsets inside z
+    int ra = 0, rg = 0;                 // padded ranks
+    int out = 0;                        // column offset inside mixed
+    int kv_layer = -1;
+    uint64_t state_off = 0, conv_off = 0;
+    void *w_a2 = nullptr, *w_g2 = nullptr;  // [heads * DK, ra], [heads * DV, rg]
+    float *bias = nullptr, *a_log = nullptr, *norm = nullptr, *conv_q = nullptr, *conv_k = nullptr, *conv_v = nullptr;
+    uint64_t have = 0;
+    int cols() const { return s.heads * (s.kind == JGPT_MIX_ATTENTION ? D : DV); }
+};
+
+struct DLayer {
+    std::vector<DBranch> br;
+    int ff = 0, ffp = 0, n_in = 0, n_out = 0, n_z = 0;
+    void *w_in = nullptr, *w_out = nullptr, *w_gu = nullptr, *w_down = nullptr;
+    float *n1w = nullptr, *n1b = nullptr, *n2w = nullptr, *n2b = nullptr;
+    uint64_t have = 0;
+};
+
+struct Decoder {
+    Ctx *ctx = nullptr;
+    jgpt_decoder_spec s{};
+    bool f32 = false;
+    int eb = 2, R = 0, ldw = 0;  // element bytes, rows per step, padded width
+    std::vector<DLayer> L;
+    void *embed = nullptr, *pos = nullptr;
+    float *enw = nullptr, *enb = nullptr, *fnw = nullptr, *fnb = nullptr;
+    uint64_t have = 0;
+    std::vector<KvLayerGeom> kv;
+    uint64_t state_stride = 0;
+    std::vector<void *> allocs;
+    // workspace
+    float *x = nullptr, *raw = nullptr, *logits = nullptr, *partials = nullptr;
+    uint64_t partial_floats = 0;
+    void *h = nullptr, *proj = nullptr, *z = nullptr, *mixed = nullptr, *act = nullptr;
+    int *d_desc = nullptr, *h_desc = nullptr;
+    int *d_next = nullptr, *h_next = nullptr;
+    float *d_u = nullptr, *h_u = nullptr, *samp = nullptr;
+    int logit_rows = 0;
+    float *capture = nullptr;  // host, [layers][rows][width] of the next step
+    uint64_t capture_floats = 0;
+};
+
+Registry<Decoder> &decoder_registry() {
+    static Registry<Decoder> r;
+    return r;
+}
+int decoder_max_rows(const Decoder *d) { return d->R; }
+int decoder_max_positions(const Decoder *d) { return d->s.max_positions; }
+const int *decoder_next_tokens_device(const Decoder *d) { return d->d_next; }
+Ctx *decoder_ctx(const Decoder *d) { return d->ctx; }
+
+static int32_t dalloc(Decoder *d, void **p, uint64_t bytes) {
+    JGPT_CUDA_TRY(cudaMalloc(p, std::max<uint64_t>(bytes, 16)));
+    d->allocs.push_back(*p);
+    JGPT_CUDA_TRY(cudaMemsetAsync(*p, 0, std::max<uint64_t>(bytes, 16), d->ctx->stream));
+    return JGPT_OK;
+}
+#define TRY(expr)                        \
+    do {                                 \
+        const int32_t rc_ = (expr);      \
+        if (rc_) return rc_;             \
+    } while (0)
+
+static void release(Decoder *d) {
+    for (void *p : d->allocs) cudaFree(p);
+    cudaFreeHost(d->h_desc), cudaFreeHost(d->h_next), cudaFreeHost(d->h_u);
+    delete d;
+}
+int32_t decoder_destroy(Decoder *d) {
+    JGPT_CUDA_TRY(make_current(d->ctx));
+    cudaStreamSynchronize(d->ctx->stream);
+    decoder_registry().remove(d);
+    release(d);
+    return JGPT_OK;
+}
+
+static mix::RecArgs rec_args(const DBranch &b) {
+    mix::RecArgs a{};
+    a.kind = b.s.kind == JGPT_MIX_DELTA ? mix::REC_DELTA : mix::REC_GLA;
+    a.q_off = b.q, a.k_off = b.k, a.v_off = b.v, a.b_off = b.b, a.g_off = b.g, a.z_off = b.za, a.zg_off = b.zg;
+    a.heads = b.s.heads, a.kv_heads = b.s.kv_heads, a.DK = b.DK, a.DV = b.DV, a.dim = b.s.dim, a.vdim = b.s.vdim;
+    a.tau = b.s.tau, a.out_scale = b.s.out_scale, a.taps = b.s.kind == JGPT_MIX_DELTA ? b.s.taps : 0;
+    a.conv_q = b.conv_q, a.conv_k = b.conv_k, a.conv_v = b.conv_v, a.decay_bias = b.bias, a.a_log = b.a_log, a.norm_w = b.norm;
+    a.conv_off = b.conv_off, a.out_off = b.out;
+    return a;
+}
+
+// Sizes, column layouts and device memory of one layer.
+static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int index) {
+    JGPT_REQUIRE(ls.n_branches >= 1 && ls.n_branches <= JGPT_MAX_BRANCHES, JGPT_ERR_INVALID_ARGUMENT, "layer %d: %d mixer branches", index,
+                 ls.n_branches);
+    JGPT_REQUIRE(ls.ff >= 0, JGPT_ERR_INVALID_ARGUMENT, "layer %d: feed-forward size %d", index, ls.ff);
+    const int eb = d->eb, W = d->s.width;
+    int in = 0, out = 0, zc = 0;
+    auto seg = [&](int n) {
+        const int o = in;
+        in += up(n, 8);
+        return o;
+    };
+    for (int i = 0; i < ls.n_branches; i++) {
+        DBranch b;
+        b.s = ls.branch[i];
+        const jgpt_mixer_spec &s = b.s;
+        JGPT_REQUIRE(s.heads > 0 && s.kv_heads > 0 && s.heads % s.kv_heads == 0 && s.dim > 0 && s.vdim > 0, JGPT_ERR_INVALID_ARGUMENT,
+                     "layer %d: heads %d / %d, head sizes %d / %d", index, s.heads, s.kv_heads, s.dim, s.vdim);
+        b.out = out;
+        if (s.kind == JGPT_MIX_ATTENTION) {
+            b.D = mix::attn_padded_head(s.dim, s.vdim);
+            JGPT_REQUIRE(b.D > 0, JGPT_ERR_UNSUPPORTED, "layer %d: head sizes %d / %d", index, s.dim, s.vdim);
+            b.q = seg(s.heads * b.D), b.k = seg(s.kv_heads * b.D), b.v = seg(s.kv_heads * b.D);
+            if (s.gate) b.g = seg(s.heads);
+            b.kv_layer = (int)d->kv.size();
+            KvLayerGeom geom;
+            geom.heads = s.kv_heads, geom.dim = b.D;
+            d->kv.push_back(geom);
+        } else if (s.kind == JGPT_MIX_GLA || s.kind == JGPT_MIX_DELTA) {
+            const bool delta = s.kind == JGPT_MIX_DELTA;
+            JGPT_REQUIRE(delta || s.kv_heads == s.heads, JGPT_ERR_UNSUPPORTED, "layer %d: gated linear attention has one key head per head", index);
+            JGPT_REQUIRE(s.rank_a > 0 && (!delta || (s.rank_g > 0 && s.taps >= 1 && s.taps <= 8)) && (delta || s.tau > 0.f), JGPT_ERR_INVALID_ARGUMENT,
+                         "layer %d: ranks %d / %d, %d convolution taps, tau %g", index, s.rank_a, s.rank_g, s.taps, (double)s.tau);
+            b.DK = mix::rec_padded_key(s.dim), b.DV = mix::rec_padded_value(s.vdim);
+            JGPT_REQUIRE(b.DK > 0 && b.DV > 0, JGPT_ERR_UNSUPPORTED, "layer %d: head sizes %d / %d", index, s.dim, s.vdim);
+            b.q = seg(s.kv_heads * b.DK), b.k = seg(s.kv_heads * b.DK), b.v = seg(s.heads * b.DV);
+            b.ra = up(s.rank_a, 8), b.a1 = seg(s.rank_a);
+            b.za = zc, zc += s.heads * b.DK;
+            TRY(dalloc(d, &b.w_a2, (uint64_t)s.heads * b.DK * b.ra * eb));
+            TRY(dalloc(d, (void **)&b.bias, sizeof(float) * (uint64_t)s.heads * b.DK));
+            TRY(dalloc(d, (void **)&b.norm, sizeof(float) * (uint64_t)b.DV));
+            if (delta) {
+                b.b = seg(s.heads);
+                b.rg = up(s.rank_g, 8), b.g1 = seg(s.rank_g);
+                b.zg = zc, zc += s.heads * b.DV;
+                TRY(dalloc(d, &b.w_g2, (uint64_t)s.heads * b.DV * b.rg * eb));
+                TRY(dalloc(d, (void **)&b.a_log, sizeof(float) * (uint64_t)s.heads));
+                TRY(dalloc(d, (void **)&b.conv_q, sizeof(float) * (uint64_t)s.kv_heads * b.DK * s.taps));
+                TRY(dalloc(d, (void **)&b.conv_k, sizeof(float) * (uint64_t)s.kv_heads * b.DK * s.taps));
+                TRY(dalloc(d, (void **)&b.conv_v, sizeof(float) * (uint64_t)s.heads * b.DV * s.taps));
+            } else {
+                b.g = seg(s.heads * b.DV);
+            }
+            b.state_off = d->state_stride;
+            d->state_stride += mix::rec_state_bytes(rec_args(b), eb, &b.conv_off);
+        } else {
+            return fail(JGPT_ERR_UNSUPPORTED, "layer %d: mixer kind %d", index, s.kind);
+        }
+        out += b.cols();
+        y.br.push_back(b);
+    }
+    y.n_in = in, y.n_out = up(out, 8), y.n_z = zc, y.ff = ls.ff, y.ffp = up(ls.ff, 16);
+    TRY(dalloc(d, &y.w_in, (uint64_t)y.n_in * d->ldw * eb));
+    TRY(dalloc(d, &y.w_out, (uint64_t)W * y.n_out * eb));
+    TRY(dalloc(d, (void **)&y.n1w, sizeof(float) * (uint64_t)W));
+    TRY(dalloc(d, (void **)&y.n1b, sizeof(float) * (uint64_t)W));
+    if (y.ff) {
+        TRY(dalloc(d, &y.w_gu, 2ull * y.ffp * d->ldw * eb));
+        TRY(dalloc(d, &y.w_down, (uint64_t)W * y.ffp * eb));
+        TRY(dalloc(d, (void **)&y.n2w, sizeof(float) * (uint64_t)W));
+        TRY(dalloc(d, (void **)&y.n2b, sizeof(float) * (uint64_t)W));
+    }
+    return JGPT_OK;
+}
+
+static size_t desc_ints(const Decoder *d) { return 14 * (size_t)d->R + 64; }
+
+static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
+    const uint64_t R = d->R, W = d->s.width, eb = d->eb;
+    d->L.resize((size_t)d->s.n_layers);
+    int n_in = 8, n_z = 8, n_out = 8, ffp = 16, raw = 0;
+    for (int i = 0; i < d->s.n_layers; i++) {
+        DLayer &y = d->L[(size_t)i];
+        TRY(plan_layer(d, y, layers[i], i));
+        n_in = std::max(n_in, y.n_in), n_z = std::max(n_z, y.n_z), n_out = std::max(n_out, y.n_out), ffp = std::max(ffp, y.ffp);
+        for (const DBranch &b : y.br) {
+            if (b.s.kind != JGPT_MIX_ATTENTION) raw = std::max(raw, b.s.heads * b.DV);
+            else d->partial_floats = std::max(d->partial_floats, mix::attn_partial_floats(d->R, b.s.heads, b.D));
+        }
+    }
+    TRY(dalloc(d, &d->embed, (uint64_t)d->s.vocab * d->ldw * eb));
+    TRY(dalloc(d, &d->pos, (uint64_t)d->s.max_positions * d->ldw * eb));
+    for (float **p : {&d->enw, &d->enb, &d->fnw, &d->fnb}) TRY(dalloc(d, (void **)p, sizeof(float) * W));
+    TRY(dalloc(d, (void **)&d->x, sizeof(float) * R * W));
+    TRY(dalloc(d, (void **)&d->raw, sizeof(float) * R * raw));
+    TRY(dalloc(d, (void **)&d->partials, sizeof(float) * d->partial_floats));
+    TRY(dalloc(d, &d->h, R * d->ldw * eb));
+    TRY(dalloc(d, &d->proj, R * n_in * eb));
+    TRY(dalloc(d, &d->z, R * n_z * eb));
+    TRY(dalloc(d, &d->mixed, R * n_out * eb));
+    TRY(dalloc(d, &d->act, R * ffp * eb));
+    // logits of up to this many rows at a time
+    d->logit_rows = (int)std::max<uint64_t>(1, std::min<uint64_t>(R, (64ull << 20) / (uint64_t)d->s.vocab));
+    TRY(dalloc(d, (void **)&d->logits, sizeof(float) * (uint64_t)d->logit_rows * d->s.vocab));
+    TRY(dalloc(d, (void **)&d->d_next, sizeof(int) * R));
+    TRY(dalloc(d, (void **)&d->d_u, sizeof(float) * R));
+    TRY(dalloc(d, (void **)&d->d_desc, sizeof(int) * desc_ints(d)));
+    JGPT_CUDA_TRY(cudaHostAlloc(&d->h_desc, sizeof(int) * desc_ints(d), cudaHostAllocDefault));
+    JGPT_CUDA_TRY(cudaHostAlloc(&d->h_next, sizeof(int) * R, cudaHostAllocDefault));
+    JGPT_CUDA_TRY(cudaHostAlloc(&d->h_u, sizeof(float) * R, cudaHostAllocDefault));
+    JGPT_CUDA_TRY(cudaStreamSynchronize(d->ctx->stream));
+    return JGPT_OK;
+}
+
+// ------------------------------------------------------------------------------------------------
+// Weights
+// ------------------------------------------------------------------------------------------------
+// Source row i lands in row (i / rgroup) * rpad + i % rgroup, columns likewise: padding per head.
+struct Grouping {
+    int group = 0, pad = 0;  // group == 0: no grouping
+    int at(int i) const { return group ? i / group * pad + i % group : i; }
+};
+
+static int32_t put_matrix(Decoder *d, void *dst, int ld, int row0, int col0, const float *src, int rows, int cols, Grouping rg, Grouping cg) {
+    const int last = rg.at(rows - 1) + 1;
+    const int width = cg.at(cols - 1) + 1;
+    std::vector<uint8_t> buf((size_t)last * width * d->eb, 0);
+    for (int r = 0; r < rows; r++)
+        for (int c = 0; c < cols; c++) {
+            const size_t o = (size_t)rg.at(r) * width + cg.at(c);
+            const float v = src[(size_t)r * cols + c];
+            if (d->f32) reinterpret_cast<float *>(buf.data())[o] = v;
+            else reinterpret_cast<__nv_bfloat16 *>(buf.data())[o] = __float2bfloat16(v);
+        }
+    JGPT_CUDA_TRY(cudaMemcpy2DAsync(reinterpret_cast<uint8_t *>(dst) + ((size_t)row0 * ld + col0) * d->eb, (size_t)ld * d->eb, buf.data(),
+                                    (size_t)width * d->eb, (size_t)width * d->eb, (size_t)last, cudaMemcpyHostToDevice, d->ctx->stream));
+    JGPT_CUDA_TRY(cudaStreamSynchronize(d->ctx->stream));
+    return JGPT_OK;
+}
+static int32_t put_floats(Decoder *d, float *dst, const float *src, int rows, int cols, Grouping rg) {
+    std::vector<float> buf((size_t)(rg.at(rows - 1) + 1) * cols, 0.f);
+    for (int r = 0; r < rows; r++) std::copy(src + (size_t)r * cols, src + (size_t)(r + 1) * cols, buf.begin() + (size_t)rg.at(r) * cols);
+    JGPT_CUDA_TRY(cudaMemcpyAsync(dst, buf.data(), sizeof(float) * buf.size(), cudaMemcpyHostToDevice, d->ctx->stream));
+    JGPT_CUDA_TRY(cudaStreamSynchronize(d->ctx->stream));
+    return JGPT_OK;
+}
+
+static uint64_t bit(int role) { return 1ull << role; }
+
+static uint64_t needed_roles(const jgpt_mixer_spec &s) {
+    uint64_t n = bit(JGPT_W_Q) | bit(JGPT_W_K) | bit(JGPT_W_V) | bit(JGPT_W_O);
+    if (s.kind == JGPT_MIX_ATTENTION) return s.gate ? n | bit(JGPT_W_G) : n;
+    n |= bit(JGPT_W_A1) | bit(JGPT_W_A2) | bit(JGPT_W_DECAY_BIAS) | bit(JGPT_W_HEAD_NORM);
+    if (s.kind == JGPT_MIX_GLA) return n | bit(JGPT_W_G);
+    return n | bit(JGPT_W_B) | bit(JGPT_W_A_LOG) | bit(JGPT_W_G1) | bit(JGPT_W_G2) | bit(JGPT_W_CONV_Q) | bit(JGPT_W_CONV_K) | bit(JGPT_W_CONV_V);
+}
+
+static int32_t missing_weights(const Decoder *d) {
+    const uint64_t top = bit(JGPT_W_EMBED) | bit(JGPT_W_POS) | bit(JGPT_W_FINAL_NORM) | bit(JGPT_W_FINAL_NORM_B) |
+                         (d->s.embed_norm ? bit(JGPT_W_EMBED_NORM) | bit(JGPT_W_EMBED_NORM_B) : 0);
+    JGPT_REQUIRE((d->have & top) == top, JGPT_ERR_ILLEGAL_STATE, "embedding or final norm weights are not set");
+    for (size_t i = 0; i < d->L.size(); i++) {
+        const DLayer &y = d->L[i];
+        uint64_t n = bit(JGPT_W_NORM1) | bit(JGPT_W_NORM1_B);
+        if (y.ff) n |= bit(JGPT_W_NORM2) | bit(JGPT_W_NORM2_B) | bit(JGPT_W_FF_GATE) | bit(JGPT_W_FF_UP) | bit(JGPT_W_FF_DOWN);
+        JGPT_REQUIRE((y.have & n) == n, JGPT_ERR_ILLEGAL_STATE, "norm or feed-forward weights of layer %zu are not set", i);
+        for (const DBranch &b : y.br)
+            JGPT_REQUIRE((b.have & needed_roles(b.s)) == needed_roles(b.s), JGPT_ERR_ILLEGAL_STATE, "mixer weights of layer %zu are not set", i);
+    }
+    return JGPT_OK;
+}
+
+static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const float *src, int rows, int cols) {
+    const int W = d->s.width;
+    auto shape = [&](int r, int c) -> int32_t {
+        JGPT_REQUIRE(rows == r && cols == c, JGPT_ERR_INVALID_ARGUMENT, "layer %d branch %d tensor %d: [%d, %d] expected, got [%d, %d]", layer, branch,
+                     role, r, c, rows, cols);
+        return JGPT_OK;
+    };
+    const Grouping none;
+    if (layer < 0) {
+        switch (role) {
+            case JGPT_W_EMBED: TRY(shape(d->s.vocab, W)); TRY(put_matrix(d, d->embed, d->ldw, 0, 0, src, rows, cols, none, none)); break;
+            case JGPT_W_POS: TRY(shape(d->s.max_positions, W)); TRY(put_matrix(d, d->pos, d->ldw, 0, 0, src, rows, cols, none, none)); break;
+            case JGPT_W_EMBED_NORM: TRY(shape(1, W)); TRY(put_floats(d, d->enw, src, 1, W, none)); break;
+            case JGPT_W_EMBED_NORM_B: TRY(shape(1, W)); TRY(put_floats(d, d->enb, src, 1, W, none)); break;
+            case JGPT_W_FINAL_NORM: TRY(shape(1, W)); TRY(put_floats(d, d->fnw, src, 1, W, none)); break;
+            case JGPT_W_FINAL_NORM_B: TRY(shape(1, W)); TRY(put_floats(d, d->fnb, src, 1, W, none)); break;
+            default: return fail(JGPT_ERR_INVALID_ARGUMENT, "tensor %d does not belong to the model", role);
+        }
+        d->have |= bit(role);
+        return JGPT_OK;
+    }
+    DLayer &y = d->L[(size_t)layer];
+    if (branch < 0) {
+        const Grouping pair{16, 32};
+        const bool ff_role = role == JGPT_W_FF_GATE || role == JGPT_W_FF_UP || role == JGPT_W_FF_DOWN || role == JGPT_W_NORM2 || role == JGPT_W_NORM2_B;
+        JGPT_REQUIRE(!ff_role || y.ff, JGPT_ERR_INVALID_ARGUMENT, "layer %d has no feed-forward part", layer);
+        switch (role) {
+            case JGPT_W_NORM1: TRY(shape(1, W)); TRY(put_floats(d, y.n1w, src, 1, W, none)); break;
+            case JGPT_W_NORM1_B: TRY(shape(1, W)); TRY(put_floats(d, y.n1b, src, 1, W, none)); break;
+            case JGPT_W_NORM2: TRY(shape(1, W)); TRY(put_floats(d, y.n2w, src, 1, W, none)); break;
+            case JGPT_W_NORM2_B: TRY(shape(1, W)); TRY(put_floats(d, y.n2b, src, 1, W, none)); break;
+            case JGPT_W_FF_GATE:
+            case JGPT_W_FF_UP: {
+                // rows in groups of 16: gate, linear, gate, ... (two strided copies would overwrite each other's gaps)
+                TRY(shape(y.ff, W));
+                for (int r = 0; r < rows; r += 16)
+                    TRY(put_matrix(d, y.w_gu, d->ldw, pair.at(r) + (role == JGPT_W_FF_UP ? 16 : 0), 0, src + (size_t)r * W, std::min(16, rows - r), W,
+                                   none, none));
+                break;
+            }
+            case JGPT_W_FF_DOWN: TRY(shape(W, y.ff)); TRY(put_matrix(d, y.w_down, y.ffp, 0, 0, src, rows, cols, none, none)); break;
+            default: return fail(JGPT_ERR_INVALID_ARGUMENT, "tensor %d does not belong to a layer", role);
+        }
+        y.have |= bit(role);
+        return JGPT_OK;
+    }
+    JGPT_REQUIRE(branch < (int)y.br.size(), JGPT_ERR_OUT_OF_RANGE, "layer %d has %zu mixer branches", layer, y.br.size());
+    DBranch &b = y.br[(size_t)branch];
+    const jgpt_mixer_spec &s = b.s;
+    JGPT_REQUIRE(role >= 0 && role < 63 && (needed_roles(s) & bit(role)), JGPT_ERR_INVALID_ARGUMENT, "tensor %d does not belong to mixer kind %d", role,
+                 s.kind);
+    const bool att = s.kind == JGPT_MIX_ATTENTION;
+    const Grouping kg{s.dim, att ? b.D : b.DK}, vg{s.vdim, att ? b.D : b.DV};
+    const int vheads = att ? s.kv_heads : s.heads, qheads = att ? s.heads : s.kv_heads;
+    auto into_proj = [&](int off, int n, Grouping g) -> int32_t {
+        TRY(shape(n, W));
+        return put_matrix(d, y.w_in, d->ldw, off, 0, src, rows, cols, g, none);
+    };
+    switch (role) {
+        case JGPT_W_Q: TRY(into_proj(b.q, qheads * s.dim, kg)); break;
+        case JGPT_W_K: TRY(into_proj(b.k, s.kv_heads * s.dim, kg)); break;
+        case JGPT_W_V: TRY(into_proj(b.v, vheads * s.vdim, vg)); break;
+        case JGPT_W_G:
+            if (att) TRY(into_proj(b.g, s.heads, none));
+            else TRY(into_proj(b.g, s.heads * s.vdim, vg));
+            break;
+        case JGPT_W_B: TRY(into_proj(b.b, s.heads, none)); break;
+        case JGPT_W_A1: TRY(into_proj(b.a1, s.rank_a, none)); break;
+        case JGPT_W_G1: TRY(into_proj(b.g1, s.rank_g, none)); break;
+        case JGPT_W_A2: TRY(shape(s.heads * s.dim, s.rank_a)); TRY(put_matrix(d, b.w_a2, b.ra, 0, 0, src, rows, cols, kg, none)); break;
+        case JGPT_W_G2: TRY(shape(s.heads * s.vdim, s.rank_g)); TRY(put_matrix(d, b.w_g2, b.rg, 0, 0, src, rows, cols, vg, none)); break;
+        case JGPT_W_DECAY_BIAS: TRY(shape(1, s.heads * s.dim)); TRY(put_floats(d, b.bias, src, cols, 1, kg)); break;
+        case JGPT_W_A_LOG: TRY(shape(1, s.heads)); TRY(put_floats(d, b.a_log, src, 1, cols, none)); break;
+        case JGPT_W_HEAD_NORM: TRY(shape(1, s.vdim)); TRY(put_floats(d, b.norm, src, 1, cols, none)); break;
+        case JGPT_W_CONV_Q: TRY(shape(s.kv_heads * s.dim, s.taps)); TRY(put_floats(d, b.conv_q, src, rows, cols, kg)); break;
+        case JGPT_W_CONV_K: TRY(shape(s.kv_heads * s.dim, s.taps)); TRY(put_floats(d, b.conv_k, src, rows, cols, kg)); break;
+        case JGPT_W_CONV_V: TRY(shape(s.heads * s.vdim, s.taps)); TRY(put_floats(d, b.conv_v, src, rows, cols, vg)); break;
+        case JGPT_W_O: TRY(shape(W, s.heads * s.vdim)); TRY(put_matrix(d, y.w_out, y.n_out, 0, b.out, src, rows, cols, none, vg)); break;
+        default: return fail(JGPT_ERR_INVALID_ARGUMENT, "tensor %d", role);
+    }
+    b.have |= bit(role);
+    return JGPT_OK;
+}
+
+// ------------------------------------------------------------------------------------------------
+// The step
+// ------------------------------------------------------------------------------------------------
+int32_t decoder_check_pool(const Decoder *d, const Pool *p) {
+    JGPT_REQUIRE(p, JGPT_ERR_BAD_HANDLE, "bad kvpool handle");
+    JGPT_REQUIRE(p->ctx == d->ctx, JGPT_ERR_INVALID_ARGUMENT, "model and KV pool live on different contexts");
+    bool ok = p->layered && p->elem_bytes == d->eb && p->state_stride == d->state_stride && p->vlayers.size() == d->kv.size();
+    for (size_t i = 0; ok && i < d->kv.size(); i++) ok = p->vlayers[i].heads == d->kv[i].heads && p->vlayers[i].dim == d->kv[i].dim;
+    JGPT_REQUIRE(ok, JGPT_ERR_INVALID_ARGUMENT, "KV pool geometry does not match the model");
+    return JGPT_OK;
+}
+
+static int32_t product(Decoder *d, const nt::Problem *p, int n, nt::Epilogue epi) {
+    return d->f32 ? nt::launch_f32(p, n, epi, d->ctx->stream) : nt::launch_bf16(d->ctx, p, n, epi, 0, d->ctx->stream);
+}
+
+static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, uint64_t capture_rows) {
+    const int W = d->s.width, R = sd.rows, ldw = d->ldw, eb = d->eb;
+    const float eps = d->s.eps;
+    cudaStream_t st = d->ctx->stream;
+    int *status = d->ctx->d_status;
+    for (size_t i = 0; i < d->L.size(); i++) {
+        DLayer &y = d->L[i];
+        if (i == 0)
+            TRY(mix::launch_embed(d->f32, sd, d->embed, ldw, d->pos, ldw, d->s.embed_scale,
+                                  d->s.embed_norm ? mix::NormW{d->enw, d->enb} : mix::NormW{nullptr, nullptr}, mix::NormW{y.n1w, y.n1b}, eps, d->x,
+                                  d->h, W, ldw, d->s.vocab, d->s.max_positions, status, 0, st));
+        else TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n1w, y.n1b}, eps, d->h, R, W, ldw, 0, st));
+        nt::Problem in{d->h, y.w_in, d->proj, nullptr, R, y.n_in, ldw, ldw, ldw, y.n_in, 1.f};
+        TRY(product(d, &in, 1, nt::EPI_STORE));
+        for (DBranch &b : y.br) {
+            if (b.s.kind == JGPT_MIX_ATTENTION) {
+                mix::AttnArgs a{};
+                a.proj = d->proj, a.ldp = y.n_in, a.q_off = b.q, a.k_off = b.k, a.v_off = b.v, a.g_off = b.g;
+                a.heads = b.s.heads, a.kv_heads = b.s.kv_heads, a.D = b.D, a.chunk = b.s.chunk, a.scale = b.s.score_scale, a.out_scale = b.s.out_scale;
+                a.kv = p->vkv + p->vlayers[(size_t)b.kv_layer].offset, a.table = p->d_table, a.n_blocks = p->n_blocks, a.mbs = p->max_blocks_per_seq;
+                a.out = d->mixed, a.ldo = y.n_out, a.out_off = b.out, a.partials = d->partials, a.partial_floats = d->partial_floats;
+                a.sm_count = d->ctx->sm_count, a.status = status;
+                TRY(mix::launch_attention(d->f32, sd, a, 0, st));
+            } else {
+                uint8_t *proj = reinterpret_cast<uint8_t *>(d->proj), *z = reinterpret_cast<uint8_t *>(d->z);
+                nt::Problem zp[2];
+                int nz = 0;
+                zp[nz++] = nt::Problem{proj + (size_t)b.a1 * eb, b.w_a2, z + (size_t)b.za * eb, nullptr, R, b.s.heads * b.DK, b.ra, y.n_in, b.ra, y.n_z, 1.f};
+                if (b.g1 >= 0)
+                    zp[nz++] = nt::Problem{proj + (size_t)b.g1 * eb, b.w_g2, z + (size_t)b.zg * eb, nullptr, R, b.s.heads * b.DV, b.rg, y.n_in, b.rg, y.n_z, 1.f};
+                TRY(product(d, zp, nz, nt::EPI_STORE));
+                mix::RecArgs a = rec_args(b);
+                a.proj = d->proj, a.ldp = y.n_in, a.z = d->z, a.ldz = y.n_z, a.eps = eps;
+                a.state = p->state + b.state_off, a.state_stride = p->state_stride, a.max_seqs = p->max_seqs;
+                a.out = d->mixed, a.ldo = y.n_out, a.raw = d->raw, a.sm_count = d->ctx->sm_count, a.status = status;
+                TRY(mix::launch_recurrent(d->f32, sd, a, 0, st));
+            }
+        }
+        nt::Problem out{d->mixed, y.w_out, d->x, nullptr, R, W, y.n_out, y.n_out, y.n_out, W, 1.f};
+        TRY(product(d, &out, 1, nt::EPI_ADD_F32));
+        if (y.ff) {
+            TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n2w, y.n2b}, eps, d->h, R, W, ldw, 0, st));
+            nt::Problem gu{d->h, y.w_gu, d->act, nullptr, R, 2 * y.ffp, ldw, ldw, ldw, y.ffp, 1.f};
+            TRY(product(d, &gu, 1, nt::EPI_GATE_GELU));
+            nt::Problem down{d->act, y.w_down, d->x, nullptr, R, W, y.ffp, y.ffp, y.ffp, W, 1.f};
+            TRY(product(d, &down, 1, nt::EPI_ADD_F32));
+        }
+        if (capture_rows)
+            JGPT_CUDA_TRY(cudaMemcpyAsync(d->capture + (uint64_t)i * capture_rows * W, d->x, sizeof(float) * capture_rows * W, cudaMemcpyDeviceToHost, st));
+    }
+    return JGPT_OK;
+}
+
+// Final norm, logits and token choice of wanted rows [w0, w0 + n).
+static int32_t enqueue_head(Decoder *d, const mix::StepDesc &sd, int w0, int n, bool pick, const SampleSpec &spec) {
+    cudaStream_t st = d->ctx->stream;
+    TRY(mix::launch_layer_norm(d->f32, d->x, sd.want + w0, mix::NormW{d->fnw, d->fnb}, d->s.eps, d->h, n, d->s.width, d->ldw, 0, st));
+    nt::Problem p{d->h, d->embed, d->logits, nullptr, n, d->s.vocab, d->ldw, d->ldw, d->ldw, d->s.vocab, d->s.logit_scale};
+    TRY(product(d, &p, 1, nt::EPI_SCALE_F32));
+    if (!pick) return JGPT_OK;
+    if (spec.temperature > 0.f) return launch_sample(d->logits, d->samp, n, d->s.vocab, spec, d->d_u + w0, d->d_next + w0, st);
+    return launch_argmax(d->logits, n, d->s.vocab, d->d_next + w0, st);
+}
+
+int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) {
+    TRY(decoder_check_pool(d, p));
+    JGPT_CUDA_TRY(make_current(d->ctx));
+    TRY(missing_weights(d));
+    JGPT_REQUIRE(c.n >= 1 && c.seq_ids && c.starts && c.ids && c.starts[0] == 0, JGPT_ERR_INVALID_ARGUMENT, "null pointer or empty step");
+    const int rows = c.starts[c.n];
+    JGPT_REQUIRE(rows >= c.n && rows <= d->R, JGPT_ERR_INVALID_ARGUMENT, "a step of %d rows; the model's workspace holds %d", rows, d->R);
+    JGPT_REQUIRE(c.n_want >= 0 && (c.n_want == 0 || c.want), JGPT_ERR_INVALID_ARGUMENT, "null list of wanted rows");
+    JGPT_REQUIRE(c.spec.temperature <= 0.f || c.u01 || c.n_want == 0, JGPT_ERR_INVALID_ARGUMENT, "sampling needs one draw per row");
+    for (int i = 0; i < c.n_want; i++)
+        JGPT_REQUIRE(c.want[i] >= 0 && c.want[i] < rows, JGPT_ERR_OUT_OF_RANGE, "wanted row %d of %d", c.want[i], rows);
+    for (int i = 0; i < rows; i++)
+        JGPT_REQUIRE(c.ids[i] >= 0 && c.ids[i] < d->s.vocab, JGPT_ERR_OUT_OF_RANGE, "token id %d outside [0,%d)", c.ids[i], d->s.vocab);
+    std::vector<char> seen((size_t)p->max_seqs, 0);
+    int n_tiles = 0, n_single = 0;
+    for (int i = 0; i < c.n; i++) {
+        const int s = c.seq_ids[i], T = c.starts[i + 1] - c.starts[i];
+        JGPT_REQUIRE(s >= 0 && s < p->max_seqs && p->seqs[(size_t)s].used, JGPT_ERR_OUT_OF_RANGE, "sequence %d is not allocated", s);
+        JGPT_REQUIRE(T >= 1 && !seen[(size_t)s], JGPT_ERR_INVALID_ARGUMENT, "entry %d: no tokens, or its sequence appears twice", i);
+        seen[(size_t)s] = 1;
+        JGPT_REQUIRE(p->seqs[(size_t)s].len + T <= d->s.max_positions, JGPT_ERR_ILLEGAL_STATE, "sequence %d: %d + %d tokens exceed the %d positions", s,
+                     p->seqs[(size_t)s].len, T, d->s.max_positions);
+    }
+    JGPT_REQUIRE(c.n_want <= d->R, JGPT_ERR_INVALID_ARGUMENT, "%d wanted rows; the workspace holds %d", c.n_want, d->R);
+    // blocks for every entry, or none
+    for (int i = 0; i < c.n; i++) {
+        const int s = c.seq_ids[i], T = c.starts[i + 1] - c.starts[i];
+        const int32_t rc = jgpt_seq_reserve(poolh, s, p->seqs[(size_t)s].len + T);
+        if (rc) {
+            const std::string keep = last_error_ref();
+            for (int j = 0; j < i; j++) pool_trim_reservation(p, c.seq_ids[j], p->seqs[(size_t)c.seq_ids[j]].len);
+            last_error_ref() = keep;
+            return rc;
+        }
+    }
+    // ---- descriptors ----
+    int *hd = d->h_desc;
+    size_t at = 0;
+    auto take = [&](size_t n) {
+        const size_t o = at;
+        at += (n + 3) / 4 * 4;
+        return o;
+    };
+    const size_t o_tok = take((size_t)rows), o_pos = take((size_t)rows), o_seq = take((size_t)rows), o_seg = take(6 * (size_t)c.n);
+    const size_t o_single = take((size_t)c.n), o_want = take((size_t)c.n_want), o_tile = at;
+    int max_len = 0;
+    mix::Seg *segs = reinterpret_cast<mix::Seg *>(hd + o_seg);
+    for (int i = 0; i < c.n; i++) {
+        const int s = c.seq_ids[i], r0 = c.starts[i], T = c.starts[i + 1] - r0;
+        const SeqState &ss = p->seqs[(size_t)s];
+        segs[i] = mix::Seg{s, r0, T, ss.len, ss.conv_set, 0};
+        max_len = std::max(max_len, ss.len + T);
+        for (int t = 0; t < T; t++) hd[o_tok + r0 + t] = c.ids[r0 + t], hd[o_pos + r0 + t] = ss.len + t, hd[o_seq + r0 + t] = s;
+        if (T == 1) hd[o_single + n_single++] = i;
+    }
+    for (int i = 0; i < c.n_want; i++) hd[o_want + i] = c.want[i];
+    // query tiles: the same list serves every layer, so tiles hold as many tokens as the layer with the largest groups allows
+    int qt = 64;
+    for (const DLayer &y : d->L)
+        for (const DBranch &b : y.br)
+            if (b.s.kind == JGPT_MIX_ATTENTION) qt = std::min(qt, mix::attn_query_tile(b.s.heads, b.s.kv_heads));
+    for (int i = 0; i < c.n; i++) {
+        const int T = c.starts[i + 1] - c.starts[i];
+        if (T > 1)
+            for (int t = 0; t < T; t += qt) hd[o_tile + 2 * n_tiles] = i, hd[o_tile + 2 * n_tiles + 1] = t, n_tiles++;
+    }
+    at = o_tile + 2 * (size_t)n_tiles;
+    JGPT_REQUIRE(at <= desc_ints(d), JGPT_ERR_INVALID_ARGUMENT, "step descriptors need %zu words, there are %zu", at, desc_ints(d));
+    cudaStream_t st = d->ctx->stream;
+    JGPT_CUDA_TRY(cudaMemcpyAsync(d->d_desc, hd, sizeof(int) * at, cudaMemcpyHostToDevice, st));
+    mix::StepDesc sd{};
+    const int *dd = d->d_desc;
+    sd.tok = dd + o_tok, sd.pos = dd + o_pos, sd.seq = dd + o_seq, sd.segs = reinterpret_cast<const mix::Seg *>(dd + o_seg);
+    sd.tiles = reinterpret_cast<const int2 *>(dd + o_tile), sd.singles = dd + o_single, sd.want = dd + o_want;
+    sd.rows = rows, sd.n_segs = c.n, sd.n_tiles = n_tiles, sd.n_singles = n_single, sd.n_want = c.n_want, sd.max_len = max_len;
+    sd.qt = qt;
+
+    uint64_t cap_rows = 0;
+    if (d->capture) {
+        JGPT_REQUIRE(d->capture_floats >= (uint64_t)d->L.size() * rows * d->s.width, JGPT_ERR_INVALID_ARGUMENT, "capture buffer is too small");
+        cap_rows = (uint64_t)rows;
+    }
+    TRY(enqueue_layers(d, p, sd, cap_rows));
+    d->capture = nullptr;
+    const bool pick = c.next_host != nullptr;
+    if (pick && c.spec.temperature > 0.f && c.n_want) {
+        if (!d->samp) TRY(dalloc(d, (void **)&d->samp, sizeof(float) * (uint64_t)d->logit_rows * d->s.vocab));
+        std::copy(c.u01, c.u01 + c.n_want, d->h_u);
+        JGPT_CUDA_TRY(cudaMemcpyAsync(d->d_u, d->h_u, sizeof(float) * c.n_want, cudaMemcpyHostToDevice, st));
+    }
+    for (int w0 = 0; w0 < c.n_want; w0 += d->logit_rows) {
+        const int n = std::min(d->logit_rows, c.n_want - w0);
+        TRY(enqueue_head(d, sd, w0, n, pick, c.spec));
+        if (c.logits_host)
+            JGPT_CUDA_TRY(cudaMemcpyAsync(c.logits_host + (size_t)w0 * d->s.vocab, d->logits, sizeof(float) * (size_t)n * d->s.vocab, cudaMemcpyDeviceToHost, st));
+    }
+    if (pick && c.n_want) JGPT_CUDA_TRY(cudaMemcpyAsync(d->h_next, d->d_next, sizeof(int) * c.n_want, cudaMemcpyDeviceToHost, st));
+    JGPT_CUDA_TRY(status_enqueue_read(d->ctx));
+    JGPT_CUDA_TRY(cudaStreamSynchronize(st));
+    TRY(status_check_after_sync(d->ctx, p, "forward step"));
+    if (pick) std::copy(d->h_next, d->h_next + c.n_want, c.next_host);
+    for (int i = 0; i < c.n; i++) {
+        SeqState &ss = p->seqs[(size_t)c.seq_ids[i]];
+        ss.len += c.starts[i + 1] - c.starts[i];
+        ss.conv_set ^= 1;
+        ss.tick = ++p->clock;
+    }
+    return JGPT_OK;
+}
+
+// ------------------------------------------------------------------------------------------------
+// The fixed-block model's forms
+// ------------------------------------------------------------------------------------------------
+int32_t decoder_prefill_batch(Decoder *d, jgpt_kvpool poolh, const int *seq_ids, const int *starts, const int *ids, const int *rope_offsets,
+                              int n, float *all_logits, float *last_logits, int *next) {
+    Pool *p = pool_registry().get(poolh);
+    TRY(decoder_check_pool(d, p));
+    JGPT_REQUIRE(n >= 1 && seq_ids && starts && ids && rope_offsets, JGPT_ERR_INVALID_ARGUMENT, "null pointer or empty batch");
+    JGPT_REQUIRE(!all_logits || n == 1, JGPT_ERR_INVALID_ARGUMENT, "all-row logits are available for one sequence at a time");
+    for (int i = 0; i < n; i++) {
+        JGPT_REQUIRE(rope_offsets[i] == 0, JGPT_ERR_UNSUPPORTED, "positions of a layered decoder start at 0");
+        const int s = seq_ids[i];
+        JGPT_REQUIRE(s >= 0 && s < p->max_seqs && p->seqs[(size_t)s].used, JGPT_ERR_OUT_OF_RANGE, "sequence %d is not allocated", s);
+        p->seqs[(size_t)s].len = 0;  // a prefill starts the sequence over
+    }
+    std::vector<int> want;
+    if (all_logits)
+        for (int r = 0; r < starts[n]; r++) want.push_back(r);
+    else
+        for (int i = 0; i < n; i++) want.push_back(starts[i + 1] - 1);
+    StepCall c;
+    c.n = n, c.seq_ids = seq_ids, c.starts = starts, c.ids = ids, c.n_want = (int)want.size(), c.want = want.data();
+    c.logits_host = all_logits ? all_logits : last_logits;
+    std::vector<int> picked(want.size());
+    if (next) c.next_host = picked.data();
+    TRY(decoder_step(d, p, poolh, c));
+    if (all_logits && last_logits) std::copy(all_logits + (size_t)(starts[n] - 1) * d->s.vocab, all_logits + (size_t)starts[n] * d->s.vocab, last_logits);
+    if (next) {
+        if (all_logits) next[0] = picked.back();
+        else std::copy(picked.begin(), picked.end(), next);
+    }
+    return JGPT_OK;
+}
+
+int32_t decoder_decode(Decoder *d, jgpt_kvpool poolh, const int *seq_ids, const int *ids, const int *len_before, const int *rope_pos, int n,
+                       float *logits, int *next, const SampleSpec &spec, const float *u01) {
+    Pool *p = pool_registry().get(poolh);
+    TRY(decoder_check_pool(d, p));
+    JGPT_REQUIRE(n >= 1 && seq_ids && ids && len_before && rope_pos, JGPT_ERR_INVALID_ARGUMENT, "null pointer or empty batch");
+    std::vector<int> starts((size_t)n + 1), want((size_t)n);
+    for (int i = 0; i < n; i++) {
+        const int s = seq_ids[i];
+        JGPT_REQUIRE(s >= 0 && s < p->max_seqs && p->seqs[(size_t)s].used, JGPT_ERR_OUT_OF_RANGE, "sequence %d is not allocated", s);
+        JGPT_REQUIRE(p->seqs[(size_t)s].len == len_before[i], JGPT_ERR_ILLEGAL_STATE, "sequence %d holds %d tokens, the call says %d", s,
+                     p->seqs[(size_t)s].len, len_before[i]);
+        JGPT_REQUIRE(rope_pos[i] == len_before[i], JGPT_ERR_INVALID_ARGUMENT, "positions of a layered decoder follow the length");
+        starts[(size_t)i + 1] = i + 1, want[(size_t)i] = i;
+    }
+    StepCall c;
+    c.n = n, c.seq_ids = seq_ids, c.starts = starts.data(), c.ids = ids, c.n_want = n, c.want = want.data();
+    c.logits_host = logits, c.next_host = next, c.spec = spec, c.u01 = u01;
+    return decoder_step(d, p, poolh, c);
+}
+
+int32_t decoder_generate_greedy(Decoder *d, jgpt_kvpool poolh, const int *prompt, int S, int max_new, int *out, int *n_sampled) {
+    Pool *p = pool_registry().get(poolh);
+    TRY(decoder_check_pool(d, p));
+    JGPT_REQUIRE(prompt && out && S >= 1 && max_new >= 0, JGPT_ERR_INVALID_ARGUMENT, "bad prompt");
+    JGPT_REQUIRE(S + std::max(max_new, 1) - 1 <= d->s.max_positions, JGPT_ERR_INVALID_ARGUMENT, "prompt %d + %d new tokens exceed the %d positions", S,
+                 max_new, d->s.max_positions);
+    std::copy(prompt, prompt + S, out);
+    std::fill(out + S, out + S + max_new, 0);
+    if (n_sampled) *n_sampled = 0;
+    if (max_new == 0) return JGPT_OK;
+    int32_t seq = -1;
+    TRY(jgpt_seq_alloc(poolh, &seq));
+    const int32_t rc = [&]() -> int32_t {
+        int tok = 0;
+        for (int t0 = 0; t0 < S; t0 += d->R) {  // the prompt in portions of the workspace's rows
+            const int T = std::min(d->R, S - t0), starts[2] = {0, T}, last = T - 1;
+            StepCall c;
+            c.n = 1, c.seq_ids = &seq, c.starts = starts, c.ids = prompt + t0;
+            if (t0 + T == S) c.n_want = 1, c.want = &last, c.next_host = &tok;
+            TRY(decoder_step(d, p, poolh, c));
+        }
+        for (int j = 0;; j++) {
+            out[S + j] = tok;
+            if (n_sampled) *n_sampled = j + 1;
+            if (tok == 0 || j + 1 == max_new) return JGPT_OK;
+            const int len = S + j;
+            TRY(decoder_decode(d, poolh, &seq, &tok, &len, &len, 1, nullptr, &tok, SampleSpec(), nullptr));
+        }
+    }();
+    const std::string keep = last_error_ref();
+    jgpt_seq_free(poolh, seq);
+    last_error_ref() = keep;
+    return rc;
+}
+
+}  // namespace jgpt
+
+using namespace jgpt;
+
+#define GET_DECODER(d, h)                                                   \
+    Decoder *d = decoder_registry().get(h);                                 \
+    JGPT_REQUIRE(d, JGPT_ERR_BAD_HANDLE, "not a layered decoder's handle"); \
+    JGPT_CUDA_TRY(make_current(d->ctx))
+
+extern "C" {
+
+int32_t jgpt_decoder_create(jgpt_ctx ctxh, const jgpt_decoder_spec *spec, const jgpt_layer_spec *layers, int32_t dtype, int32_t max_rows,
+                            jgpt_model *out) {
+    Ctx *c = ctx_registry().get(ctxh);
+    JGPT_REQUIRE(c, JGPT_ERR_BAD_HANDLE, "bad context handle");
+    JGPT_REQUIRE(spec && layers && out, JGPT_ERR_INVALID_ARGUMENT, "null pointer");
+    JGPT_REQUIRE(spec->vocab > 0 && spec->width > 0 && spec->max_positions > 0 && spec->n_layers > 0 && max_rows > 0, JGPT_ERR_INVALID_ARGUMENT,
+                 "model dimensions must be positive");
+    JGPT_REQUIRE(dtype == JGPT_DTYPE_BF16 || dtype == JGPT_DTYPE_F32, JGPT_ERR_INVALID_ARGUMENT, "dtype %d", dtype);
+    JGPT_CUDA_TRY(make_current(c));
+    Decoder *d = new Decoder();
+    d->ctx = c, d->s = *spec, d->f32 = dtype == JGPT_DTYPE_F32, d->eb = d->f32 ? 4 : 2, d->R = max_rows, d->ldw = up(spec->width, 8);
+    const int32_t rc = build(d, layers);
+    if (rc) {
+        const std::string keep = last_error_ref();
+        release(d);
+        last_error_ref() = keep;
+        return rc;
+    }
+    *out = decoder_registry().add(d);
+    return JGPT_OK;
+}
+
+int32_t jgpt_decoder_set_tensor(jgpt_model h, int32_t layer, int32_t branch, int32_t role, const float *host, int32_t rows, int32_t cols) {
+    GET_DECODER(d, h);
+    JGPT_REQUIRE(layer >= -1 && layer < (int)d->L.size(), JGPT_ERR_OUT_OF_RANGE, "layer %d outside [-1,%zu)", layer, d->L.size());
+    JGPT_REQUIRE(host && rows >= 1 && cols >= 1, JGPT_ERR_INVALID_ARGUMENT, "null or empty tensor");
+    return set_tensor(d, layer, branch, role, host, rows, cols);
+}
+
+int32_t jgpt_decoder_capture_layers(jgpt_model h, float *host, uint64_t n_floats) {
+    GET_DECODER(d, h);
+    d->capture = host, d->capture_floats = host ? n_floats : 0;
+    return JGPT_OK;
+}
+
+int32_t jgpt_decoder_new_pool(jgpt_model h, int32_t n_blocks, int32_t max_seqs, int32_t max_blocks_per_seq, jgpt_kvpool *out) {
+    GET_DECODER(d, h);
+    JGPT_REQUIRE(out, JGPT_ERR_INVALID_ARGUMENT, "out is null");
+    return pool_create_layered(d->ctx, d->kv, d->eb, n_blocks, max_seqs, max_blocks_per_seq, d->state_stride, out);
+}
+
+int32_t jgpt_forward_step(jgpt_model h, jgpt_kvpool poolh, int32_t n, const int32_t *seq_ids_host, const int32_t *starts_host,
+                          const int32_t *ids_host, int32_t n_want, const int32_t *want_rows_host, float *logits_host, int32_t *next_tokens_host) {
+    GET_DECODER(d, h);
+    StepCall c;
+    c.n = n, c.seq_ids = seq_ids_host, c.starts = starts_host, c.ids = ids_host, c.n_want = n_want, c.want = want_rows_host;
+    c.logits_host = logits_host, c.next_host = next_tokens_host;
+    return decoder_step(d, pool_registry().get(poolh), poolh, c);
+}
+
+}  // extern "C"

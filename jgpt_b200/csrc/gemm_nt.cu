@@ -1,0 +1,331 @@
+// C[M, N] = A[M, K] . W[N, K]^T for decode-sized M (bf16, mma.sync) and in plain fp32.
+//
+// Decode-sized bf16 products are bound by the weight stream and by latency: a CTA owns 32 output columns and up to 64
+// rows, its eight warps split every 128-wide k tile (each warp covers the whole output tile with its own 16-wide
+// slice), tiles arrive through a cp.async ring, and the eight partial tiles are added in warp order through shared
+// memory.  Products with few column tiles run as clusters of CTAs that split the k range; the partial sums meet in the
+// first CTA's shared memory and are added in k order: no atomics, the same bits every time.
+#include "gemm_nt.cuh"
+
+#include <algorithm>
+
+#include "ptx.cuh"
+
+namespace jgpt {
+namespace nt {
+
+// D(16x8, f32) += A(16x16, bf16, row) * B(16x8, bf16, col)
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+constexpr int kBN = 32, kBK = 128, kMaxSplit = 8;
+
+struct SmallArgs {
+    Problem p[2];
+    int tiles[2];   // column tiles of each product
+    int n, k_split, pdl;
+};
+
+template <int MT, int STAGES>
+constexpr size_t small_smem(int k_split) {
+    const size_t ring = (size_t)STAGES * (16 * MT + kBN) * kBK * 2, red = sizeof(float) * 8 * 16 * MT * (kBN + 1);
+    return std::max(ring, red) + sizeof(float) * (size_t)(k_split - 1) * 16 * MT * kBN;
+}
+
+template <int MT, int STAGES, int EPI>
+__global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args) {
+    constexpr int BM = 16 * MT;
+    extern __shared__ __align__(128) uint8_t nt_smem[];
+    __nv_bfloat16 *As = reinterpret_cast<__nv_bfloat16 *>(nt_smem);         // [STAGES][BM][128], 16-byte chunks xor-swizzled by row
+    __nv_bfloat16 *Ws = As + (size_t)STAGES * BM * kBK;                     // [STAGES][32][128]
+    float *red = reinterpret_cast<float *>(nt_smem);                        // [8][BM][33], after the k loop
+    constexpr size_t ring_bytes = (size_t)STAGES * (BM + kBN) * kBK * 2, red_bytes = sizeof(float) * 8 * BM * (kBN + 1);
+    float *xch = reinterpret_cast<float *>(nt_smem + (ring_bytes > red_bytes ? ring_bytes : red_bytes));  // [k_split - 1][BM * 32]
+
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    int tile = blockIdx.x / args.k_split;
+    const int k_part = blockIdx.x % args.k_split;
+    const bool second = args.n > 1 && tile >= args.tiles[0];
+    if (second) tile -= args.tiles[0];
+    const Problem &P = second ? args.p[1] : args.p[0];
+    const int M = P.M, N = P.N, K = P.K, lda = P.lda, ldw = P.ldw;
+    const int m0 = blockIdx.y * BM, n0 = tile * kBN;
+    const __nv_bfloat16 *__restrict__ A = reinterpret_cast<const __nv_bfloat16 *>(P.A);
+    const __nv_bfloat16 *__restrict__ W = reinterpret_cast<const __nv_bfloat16 *>(P.W);
+    const int nk_all = (K + kBK - 1) / kBK;
+    const int kt0 = k_part * nk_all / args.k_split, nk = (k_part + 1) * nk_all / args.k_split - kt0;
+
+    const int r16 = tid >> 4, c16 = tid & 15;  // chunk slot: row r16 (+ 16 i), 16-byte chunk c16 of the 128-wide tile
+    auto load_w = [&](int buf, int k0) {
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int r = r16 + 16 * i, k = k0 + c16 * 8;
+            const bool ok = n0 + r < N && k < K;
+            cp_async16(Ws + ((size_t)buf * kBN + r) * kBK + ((c16 ^ (r & 7)) * 8), ok ? W + (size_t)(n0 + r) * ldw + k : W, ok);
+        }
+    };
+    if (args.pdl & 2) griddep_launch_dependents();
+    // weights do not depend on the previous kernel: the first tiles are requested before the wait
+#pragma unroll
+    for (int s = 0; s < STAGES - 1; s++)
+        if (s < nk) load_w(s, (kt0 + s) * kBK);
+    if (args.pdl & 1) griddep_wait();
+    const __nv_bfloat16 *a_src[MT];
+    bool a_ok[MT];
+#pragma unroll
+    for (int i = 0; i < MT; i++) {
+        const int m = m0 + r16 + 16 * i;
+        a_ok[i] = m < M;
+        a_src[i] = A + (size_t)(a_ok[i] ? (P.rowsel ? P.rowsel[m] : m) : 0) * lda;
+    }
+    auto load_a = [&](int buf, int k0) {
+#pragma unroll
+        for (int i = 0; i < MT; i++) {
+            const int r = r16 + 16 * i, k = k0 + c16 * 8;
+            const bool ok = a_ok[i] && k < K;
+            cp_async16(As + ((size_t)buf * BM + r) * kBK + ((c16 ^ (r & 7)) * 8), ok ? a_src[i] + k : A, ok);
+        }
+    };
+#pragma unroll
+    for (int s = 0; s < STAGES - 1; s++) {
+        if (s < nk) load_a(s, (kt0 + s) * kBK);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    float acc[MT][4][4];
+#pragma unroll
+    for (int i = 0; i < MT; i++)
+#pragma unroll
+        for (int j = 0; j < 4; j++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) acc[i][j][e] = 0.f;
+
+    for (int kt = 0; kt < nk; kt++) {
+        const int buf = kt % STAGES;
+        asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
+        __syncthreads();
+        if (kt + STAGES - 1 < nk) {
+            const int nb = (kt + STAGES - 1) % STAGES, k0 = (kt0 + kt + STAGES - 1) * kBK;
+            load_w(nb, k0);
+            load_a(nb, k0);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        // this warp's slice: chunks 2 * warp and 2 * warp + 1 of every row
+        uint32_t b[2][4];
+#pragma unroll
+        for (int h = 0; h < 2; h++) {  // 16 output columns each
+            const int r = h * 16 + ((lane >> 4) << 3) + (lane & 7), c = 2 * warp + ((lane >> 3) & 1);
+            ldmatrix_x4(b[h], Ws + ((size_t)buf * kBN + r) * kBK + ((c ^ (r & 7)) * 8));
+        }
+#pragma unroll
+        for (int i = 0; i < MT; i++) {
+            uint32_t a[4];
+            const int r = i * 16 + (((lane >> 3) & 1) << 3) + (lane & 7), c = 2 * warp + (lane >> 4);
+            ldmatrix_x4(a, As + ((size_t)buf * BM + r) * kBK + ((c ^ (r & 7)) * 8));
+#pragma unroll
+            for (int j = 0; j < 4; j++) mma_bf16(acc[i][j], a, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
+        }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();  // the ring is free: it becomes the reduction buffer
+    {
+        const int g = lane >> 2, t = lane & 3;
+        float *w = red + (size_t)warp * BM * (kBN + 1);
+#pragma unroll
+        for (int i = 0; i < MT; i++)
+#pragma unroll
+            for (int j = 0; j < 4; j++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) w[(i * 16 + g + (e >> 1) * 8) * (kBN + 1) + j * 8 + 2 * t + (e & 1)] = acc[i][j][e];
+    }
+    __syncthreads();
+    constexpr int PER = BM * kBN / 256;
+    float sum[PER];
+#pragma unroll
+    for (int i = 0; i < PER; i++) {
+        const int e = tid + 256 * i;
+        float s = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; w++) s += red[(size_t)w * BM * (kBN + 1) + (e >> 5) * (kBN + 1) + (e & 31)];
+        sum[i] = s;
+    }
+    if (args.k_split > 1) {
+        cluster_sync();  // every CTA of the cluster runs: its shared memory may be written
+        if (k_part > 0) {
+#pragma unroll
+            for (int i = 0; i < PER; i++) st_cluster_f32(&xch[(size_t)(k_part - 1) * BM * kBN + tid + 256 * i], 0, sum[i]);
+        }
+        cluster_sync();
+        if (k_part > 0) return;
+        for (int s = 0; s + 1 < args.k_split; s++)
+#pragma unroll
+            for (int i = 0; i < PER; i++) sum[i] += xch[(size_t)s * BM * kBN + tid + 256 * i];
+    }
+#pragma unroll
+    for (int i = 0; i < PER; i++) {
+        const int e = tid + 256 * i, m = m0 + (e >> 5), c = e & 31, n = n0 + c;
+        if (EPI == EPI_GATE_GELU) {
+            // lanes 0-15 of a warp hold the gate of a row's 16 outputs, lanes 16-31 the linear part
+            const float up = __shfl_down_sync(0xffffffffu, sum[i], 16);
+            if (c < 16 && m < M && n + 16 < N)
+                reinterpret_cast<__nv_bfloat16 *>(P.C)[(size_t)m * P.ldc + tile * 16 + c] = __float2bfloat16(gelu_tanh(sum[i]) * up);
+        } else if (m < M && n < N) {
+            if (EPI == EPI_STORE) reinterpret_cast<__nv_bfloat16 *>(P.C)[(size_t)m * P.ldc + n] = __float2bfloat16(sum[i]);
+            if (EPI == EPI_ADD_F32) reinterpret_cast<float *>(P.C)[(size_t)m * P.ldc + n] += sum[i];
+            if (EPI == EPI_SCALE_F32) reinterpret_cast<float *>(P.C)[(size_t)m * P.ldc + n] = sum[i] * P.scale;
+        }
+    }
+}
+
+template <int MT, int STAGES, int EPI>
+static int32_t small_launch(const SmallArgs &args, int total_tiles, int M, cudaStream_t st) {
+    auto kern = gemm_nt_small_kernel<MT, STAGES, EPI>;
+    const size_t smem = small_smem<MT, STAGES>(args.k_split);
+    static thread_local int set_for = -1;  // the opt-in to more than 48 KiB, once per device
+    int dev = 0;
+    JGPT_CUDA_TRY(cudaGetDevice(&dev));
+    if (set_for != dev) {
+        JGPT_CUDA_TRY(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(small_smem<MT, STAGES>(kMaxSplit))));
+        set_for = dev;
+    }
+    cudaLaunchConfig_t cfg = {};
+    cudaLaunchAttribute attr[2];
+    int na = 0;
+    if (args.k_split > 1) {
+        attr[na].id = cudaLaunchAttributeClusterDimension;
+        attr[na].val.clusterDim.x = (unsigned)args.k_split, attr[na].val.clusterDim.y = 1, attr[na].val.clusterDim.z = 1;
+        na++;
+    }
+    if (args.pdl & 1) {
+        attr[na].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[na].val.programmaticStreamSerializationAllowed = 1;
+        na++;
+    }
+    cfg.gridDim = dim3((unsigned)(total_tiles * args.k_split), (unsigned)((M + 16 * MT - 1) / (16 * MT)));
+    cfg.blockDim = dim3(256), cfg.dynamicSmemBytes = smem, cfg.stream = st, cfg.attrs = attr, cfg.numAttrs = (unsigned)na;
+    JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, kern, args));
+    return JGPT_OK;
+}
+
+template <int EPI>
+static int32_t small_dispatch(const Ctx *ctx, const Problem *p, int n, int pdl, cudaStream_t st) {
+    SmallArgs a{};
+    a.n = n, a.pdl = pdl;
+    int tiles = 0, K = 0;
+    for (int i = 0; i < n; i++) {
+        a.p[i] = p[i];
+        a.tiles[i] = (p[i].N + kBN - 1) / kBN;
+        tiles += a.tiles[i];
+        K = std::max(K, p[i].K);
+    }
+    const int M = p[0].M, mt = M <= 16 ? 1 : (M <= 32 ? 2 : 4);
+    const int ctas = tiles * ((M + 16 * mt - 1) / (16 * mt)), nk = (K + kBK - 1) / kBK;
+    // split k while the launch leaves SMs idle and every part keeps two tiles
+    a.k_split = 1;
+    while (n == 1 && a.k_split < kMaxSplit && ctas * a.k_split * 2 <= 2 * ctx->sm_count && nk / (a.k_split * 2) >= 2) a.k_split *= 2;
+    switch (mt) {
+        case 1: return small_launch<1, 6, EPI>(a, tiles, M, st);
+        case 2: return small_launch<2, 5, EPI>(a, tiles, M, st);
+        default: return small_launch<4, 4, EPI>(a, tiles, M, st);
+    }
+}
+
+int umma_min_rows() {
+    static const int v = env_int("JGPT_B200_NT_UMMA_MIN_ROWS", 0);
+    return v;
+}
+
+int32_t launch_bf16(const Ctx *ctx, const Problem *p, int n, Epilogue epi, int pdl, cudaStream_t st) {
+    JGPT_REQUIRE(n >= 1 && n <= 2 && p[0].M > 0, JGPT_ERR_INVALID_ARGUMENT, "1 or 2 products per launch");
+    bool big = p[0].M >= umma_min_rows() && umma_min_rows() > 0;
+    for (int i = 0; i < n; i++) big = big && !p[i].rowsel;
+    if (big) {
+        for (int i = 0; i < n; i++)
+            if (int32_t rc = launch_bf16_umma(ctx, p[i], epi, i == 0 ? pdl : 0, st)) return rc;
+        return JGPT_OK;
+    }
+    switch (epi) {
+        case EPI_STORE: return small_dispatch<EPI_STORE>(ctx, p, n, pdl, st);
+        case EPI_ADD_F32: return small_dispatch<EPI_ADD_F32>(ctx, p, n, pdl, st);
+        case EPI_SCALE_F32: return small_dispatch<EPI_SCALE_F32>(ctx, p, n, pdl, st);
+        case EPI_GATE_GELU: return small_dispatch<EPI_GATE_GELU>(ctx, p, n, pdl, st);
+    }
+    return fail(JGPT_ERR_INVALID_ARGUMENT, "unknown epilogue");
+}
+
+// ------------------------------------------------------------------------------------------------
+// Plain fp32: 64 x 64 tiles, fused multiply-add, k in ascending order in one thread.  The exact mode of the forward step.
+// ------------------------------------------------------------------------------------------------
+template <int EPI>
+__global__ void __launch_bounds__(256) gemm_nt_f32_kernel(const Problem P0, const Problem P1) {
+    constexpr int BT = 64, BK = 16;
+    __shared__ float As[BK][BT + 1], Ws[BK][BT + 1];
+    const Problem &P = blockIdx.z == 0 ? P0 : P1;
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    const int m0 = blockIdx.y * BT, n0 = blockIdx.x * BT;
+    if (n0 >= P.N) return;
+    const float *__restrict__ A = reinterpret_cast<const float *>(P.A);
+    const float *__restrict__ W = reinterpret_cast<const float *>(P.W);
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < P.K; k0 += BK) {
+        for (int e = tid; e < BT * BK; e += 256) {
+            const int r = e / BK, k = k0 + e % BK, m = m0 + r, n = n0 + r;
+            As[e % BK][r] = (m < P.M && k < P.K) ? A[(size_t)(P.rowsel ? P.rowsel[m] : m) * P.lda + k] : 0.f;
+            Ws[e % BK][r] = (n < P.N && k < P.K) ? W[(size_t)n * P.ldw + k] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int kk = 0; kk < BK; kk++) {
+            float a[4], w[4];
+#pragma unroll
+            for (int i = 0; i < 4; i++) a[i] = As[kk][ty * 4 + i], w[i] = Ws[kk][tx + 16 * i];
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+#pragma unroll
+                for (int j = 0; j < 4; j++) acc[i][j] = fmaf(a[i], w[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+    float *C = reinterpret_cast<float *>(P.C);
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int m = m0 + ty * 4 + i;
+        if (m >= P.M) continue;
+        if (EPI == EPI_GATE_GELU) {  // columns tx (+ 32) of a group of 32 are the gate, tx + 16 the linear part
+#pragma unroll
+            for (int j = 0; j < 4; j += 2) {
+                const int n = n0 + tx + 16 * j;
+                if (n + 16 < P.N) C[(size_t)m * P.ldc + n / 32 * 16 + tx] = gelu_tanh(acc[i][j]) * acc[i][j + 1];
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const int n = n0 + tx + 16 * j;
+                if (n >= P.N) continue;
+                float *c = C + (size_t)m * P.ldc + n;
+                if (EPI == EPI_STORE) *c = acc[i][j];
+                if (EPI == EPI_ADD_F32) *c += acc[i][j];
+                if (EPI == EPI_SCALE_F32) *c = acc[i][j] * P.scale;
+            }
+        }
+    }
+}
+
+int32_t launch_f32(const Problem *p, int n, Epilogue epi, cudaStream_t st) {
+    JGPT_REQUIRE(n >= 1 && n <= 2 && p[0].M > 0, JGPT_ERR_INVALID_ARGUMENT, "1 or 2 products per launch");
+    const Problem &q = p[n - 1];
+    const dim3 grid((unsigned)((std::max(p[0].N, q.N) + 63) / 64), (unsigned)((p[0].M + 63) / 64), (unsigned)n);
+    switch (epi) {
+        case EPI_STORE: gemm_nt_f32_kernel<EPI_STORE><<<grid, 256, 0, st>>>(p[0], q); break;
+        case EPI_ADD_F32: gemm_nt_f32_kernel<EPI_ADD_F32><<<grid, 256, 0, st>>>(p[0], q); break;
+        case EPI_SCALE_F32: gemm_nt_f32_kernel<EPI_SCALE_F32><<<grid, 256, 0, st>>>(p[0], q); break;
+        case EPI_GATE_GELU: gemm_nt_f32_kernel<EPI_GATE_GELU><<<grid, 256, 0, st>>>(p[0], q); break;
+    }
+    JGPT_CUDA_TRY(cudaGetLastError());
+    return JGPT_OK;
+}
+
+}  // namespace nt
+}  // namespace jgpt

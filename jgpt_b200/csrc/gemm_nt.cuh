@@ -1,0 +1,46 @@
+// Projections with weights in [out, in] layout: C[M, N] = A[M, K] . W[N, K]^T, bf16 operands with fp32 accumulation or
+// plain fp32.  Host-side interface of gemm_nt.cu (small M, and fp32) and gemm_nt_umma.cu (large M, tcgen05).
+#pragma once
+
+#include <cuda_bf16.h>
+
+#include "common.cuh"
+
+namespace jgpt {
+namespace nt {
+
+// What happens to a finished sum.
+enum Epilogue : int {
+    EPI_STORE = 0,     // C (activation type) = sum
+    EPI_ADD_F32 = 1,   // C (fp32) += sum: the residual; every element is read and written by one thread
+    EPI_SCALE_F32 = 2, // C (fp32) = sum * scale
+    EPI_GATE_GELU = 3, // W rows alternate in groups of 16: 16 of the gate, 16 of the linear part; C [M, N / 2] = gelu(gate) * linear
+};
+
+struct Problem {
+    const void *A;     // [M, lda]
+    const void *W;     // [N, ldw]
+    void *C;           // [M, ldc]
+    const int *rowsel; // optional: row m of A is rowsel[m] (not for the large-M kernel)
+    int M, N, K, lda, ldw, ldc;
+    float scale;
+};
+
+// gelu(z) in its tanh form, 0.5 z (1 + tanh(u)) = z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3).
+__device__ __forceinline__ float gelu_tanh(float z) {
+    const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+    return z / (1.f + expf(-2.f * u));
+}
+
+// Runs 1 or 2 independent products (same M) in one launch.  K, lda, ldw and (bf16) the operand addresses must allow
+// 16-byte row chunks: multiples of 8 elements (bf16) or 4 (fp32).  pdl: bit 0 = this launch may start early and waits
+// itself; bit 1 = it lets the next launch in.
+int32_t launch_bf16(const Ctx *ctx, const Problem *p, int n, Epilogue epi, int pdl, cudaStream_t st);
+int32_t launch_f32(const Problem *p, int n, Epilogue epi, cudaStream_t st);
+
+// From this many rows on launch_bf16 takes the tcgen05 kernel.
+int umma_min_rows();
+int32_t launch_bf16_umma(const Ctx *ctx, const Problem &p, Epilogue epi, int pdl, cudaStream_t st);
+
+}  // namespace nt
+}  // namespace jgpt

@@ -28,6 +28,7 @@
 #include "gemm_umma.cuh"
 
 #include "ptx.cuh"
+#include "tcgen05.cuh"
 
 namespace jgpt {
 namespace umma {
@@ -183,18 +184,8 @@ int32_t pack_weight_pair(const float *W1, const float *W3, int K, int F, float *
 }
 
 // ------------------------------------------------------------------------------------------------
-// tcgen05 wrappers
+// tcgen05: descriptors and the TF32 instruction (the wrappers that do not depend on the operand type: tcgen05.cuh)
 // ------------------------------------------------------------------------------------------------
-__device__ __forceinline__ void tmem_alloc(uint32_t *smem_dst, uint32_t cols) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(smem_dst)), "r"(cols) : "memory");
-    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
-}
-__device__ __forceinline__ void tmem_dealloc(uint32_t taddr, uint32_t cols) {
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(taddr), "r"(cols) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-
 // Shared-memory matrix descriptor, no swizzle: start address, leading / stride byte offsets in 16-byte units,
 // descriptor version 1 (bits 46-47), base offset 0, layout type 0.
 __device__ __forceinline__ uint64_t smem_desc(uint32_t saddr) {
@@ -215,33 +206,6 @@ __device__ __forceinline__ void mma_tf32_ss(uint32_t tmem_d, uint64_t adesc, uin
         ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
         : "memory");
 }
-// The mbarrier gets one arrival when every MMA this thread issued so far has completed.
-__device__ __forceinline__ void mma_commit(uint64_t *bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-// 32 lanes x 32 consecutive fp32 columns: thread t of the warp receives lane (base lane + t).
-__device__ __forceinline__ void tmem_ld32_nowait(uint32_t taddr, uint32_t (&v)[32]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-        "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]),
-          "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]), "=r"(v[17]), "=r"(v[18]),
-          "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]),
-          "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
-        : "r"(taddr)
-        : "memory");
-}
-__device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
-
-// 32 columns starting at `col` of this warp's 32 accumulator lanes.
-__device__ __forceinline__ void load_acc32(uint32_t tmem_acc, int quarter, int col, float (&out)[32]) {
-    uint32_t v[32];
-    tmem_ld32_nowait(tmem_acc + ((uint32_t)(quarter * 32) << 16) + (uint32_t)col, v);
-    tmem_ld_wait();
-#pragma unroll
-    for (int j = 0; j < 32; j++) out[j] = __uint_as_float(v[j]);
-}
-
 // ------------------------------------------------------------------------------------------------
 // The GEMM: a persistent CTA per SM walks the output tiles (n fastest, so CTAs running side by side share the
 // A tile through L2).  The accumulator is double-buffered in tensor memory (2 x 256 columns): while the

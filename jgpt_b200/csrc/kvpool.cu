@@ -213,6 +213,13 @@ int32_t launch_kv_scrub(Pool *p, const std::vector<int> &blocks) {
     }
     JGPT_CUDA_TRY(cudaMemcpyAsync(p->d_evict_list, blocks.data(), sizeof(int) * blocks.size(), cudaMemcpyHostToDevice,
                                   p->ctx->stream));
+    if (p->layered) {
+        for (const KvLayerGeom &g : p->vlayers)
+            kv_scrub_kernel<<<dim3((unsigned)blocks.size(), 1), 256, 0, p->ctx->stream>>>(
+                reinterpret_cast<__half *>(p->vkv + g.offset), p->d_evict_list, p->n_blocks, g.block_bytes / sizeof(__half), p->ctx->d_status);
+        JGPT_CUDA_TRY(cudaGetLastError());
+        return JGPT_OK;
+    }
     const size_t block_halfs = (size_t)p->heads * 2 * kBlockTokens * p->dhead;
     dim3 grid((unsigned)blocks.size(), (unsigned)p->layers);
     kv_scrub_kernel<<<grid, 256, 0, p->ctx->stream>>>(p->kv, p->d_evict_list, p->n_blocks, block_halfs, p->ctx->d_status);
@@ -311,6 +318,7 @@ static void free_seq_blocks(Pool *p, SeqState &s, std::vector<int> *freed) {
 
 // Frees everything a pool owns (also a partly built one: null pointers are skipped by the runtime).
 static void release_pool(Pool *p) {
+    cudaFree(p->vkv), cudaFree(p->state);
     cudaFree(p->kv), cudaFree(p->d_table), cudaFree(p->d_rope), cudaFree(p->d_partials), cudaFree(p->d_tickets);
     cudaFree(p->d_evict_list), cudaFree(p->d_stage_f), cudaFree(p->d_stage_i);
     cudaFree(p->d_prefill_desc);
@@ -324,6 +332,49 @@ static void release_pool(Pool *p) {
     delete p;
 }
 
+static uint64_t new_generation() {
+    static std::atomic<uint64_t> next{1};
+    return next.fetch_add(1);
+}
+
+int32_t pool_create_layered(Ctx *c, const std::vector<KvLayerGeom> &layers, int elem_bytes, int n_blocks, int max_seqs, int max_blocks_per_seq,
+                            uint64_t state_stride, jgpt_kvpool *out) {
+    JGPT_REQUIRE(n_blocks > 0 && max_seqs > 0 && max_blocks_per_seq > 0, JGPT_ERR_INVALID_ARGUMENT, "KV pool dimensions must be positive");
+    Pool *p = new Pool();
+    p->ctx = c, p->layered = true, p->elem_bytes = elem_bytes, p->n_blocks = n_blocks, p->max_seqs = max_seqs;
+    p->max_blocks_per_seq = max_blocks_per_seq, p->max_positions = max_blocks_per_seq * kBlockTokens, p->state_stride = state_stride;
+    for (KvLayerGeom g : layers) {
+        g.offset = p->kv_bytes, g.block_bytes = 2ull * kBlockTokens * g.heads * g.dim * elem_bytes;
+        p->kv_bytes += g.block_bytes * (uint64_t)n_blocks;
+        p->vlayers.push_back(g);
+    }
+    const int32_t rc = [&]() -> int32_t {
+        JGPT_CUDA_TRY(cudaMalloc(&p->vkv, std::max<uint64_t>(p->kv_bytes, 16)));
+        JGPT_CUDA_TRY(cudaMemsetAsync(p->vkv, 0, std::max<uint64_t>(p->kv_bytes, 16), c->stream));
+        JGPT_CUDA_TRY(cudaMalloc(&p->state, std::max<uint64_t>(state_stride * max_seqs, 16)));
+        JGPT_CUDA_TRY(cudaMemsetAsync(p->state, 0, std::max<uint64_t>(state_stride * max_seqs, 16), c->stream));
+        const size_t tn = (size_t)max_seqs * max_blocks_per_seq;
+        JGPT_CUDA_TRY(cudaMalloc(&p->d_table, sizeof(int) * tn));
+        JGPT_CUDA_TRY(cudaMemsetAsync(p->d_table, 0xFF, sizeof(int) * tn, c->stream));
+        JGPT_CUDA_TRY(cudaMalloc(&p->d_item_counters, sizeof(int) * 2));
+        JGPT_CUDA_TRY(cudaMemsetAsync(p->d_item_counters, 0, sizeof(int) * 2, c->stream));
+        return JGPT_OK;
+    }();
+    if (rc) {
+        const std::string keep = last_error_ref();
+        release_pool(p);
+        cudaGetLastError();
+        last_error_ref() = keep;
+        return rc;
+    }
+    p->generation = new_generation();
+    p->free_list.resize((size_t)n_blocks);
+    for (int i = 0; i < n_blocks; i++) p->free_list[(size_t)i] = n_blocks - 1 - i;
+    p->seqs.resize((size_t)max_seqs);
+    *out = pool_registry().add(p);
+    return JGPT_OK;
+}
+
 }  // namespace jgpt
 
 using namespace jgpt;
@@ -332,6 +383,8 @@ using namespace jgpt;
     Pool *p = pool_registry().get(h);                                       \
     JGPT_REQUIRE(p, JGPT_ERR_BAD_HANDLE, "bad kvpool handle");              \
     JGPT_CUDA_TRY(make_current(p->ctx))
+
+#define REQUIRE_UNIFORM(p) JGPT_REQUIRE(!(p)->layered, JGPT_ERR_UNSUPPORTED, "not available on a layered decoder's pool")
 
 #define CHECK_SEQ(p, seq)                                                                                  \
     JGPT_REQUIRE((seq) >= 0 && (seq) < (p)->max_seqs, JGPT_ERR_OUT_OF_RANGE, "seq %d outside [0,%d)", (seq), \
@@ -408,8 +461,7 @@ int32_t jgpt_kvpool_create(jgpt_ctx ctxh, int32_t layers, int32_t heads, int32_t
         last_error_ref() = keep;
         return rc_build;
     }
-    static std::atomic<uint64_t> next_generation{1};
-    p->generation = next_generation.fetch_add(1);
+    p->generation = new_generation();
     p->free_list.resize((size_t)n_blocks);
     for (int i = 0; i < n_blocks; i++) p->free_list[(size_t)i] = n_blocks - 1 - i;  // block 0 is handed out first
     p->seqs.resize((size_t)max_seqs);
@@ -434,7 +486,7 @@ int32_t jgpt_kvpool_free_blocks(jgpt_kvpool h, int32_t *n_free_out) {
 
 int32_t jgpt_kvpool_storage(jgpt_kvpool h, void **dev_out, uint64_t *bytes_out) {
     GET_POOL(p, h);
-    if (dev_out) *dev_out = p->kv;
+    if (dev_out) *dev_out = p->layered ? static_cast<void *>(p->vkv) : static_cast<void *>(p->kv);
     if (bytes_out) *bytes_out = p->kv_bytes;
     return JGPT_OK;
 }
@@ -517,6 +569,8 @@ int32_t jgpt_seq_set_length(jgpt_kvpool h, int32_t seq, int32_t len) {
     SeqState &s = p->seqs[(size_t)seq];
     JGPT_REQUIRE(len >= 0 && len <= (int)s.blocks.size() * kBlockTokens, JGPT_ERR_INVALID_ARGUMENT,
                  "length %d outside [0, %d]", len, (int)s.blocks.size() * kBlockTokens);
+    // recurrent state cannot be taken back to an earlier position
+    JGPT_REQUIRE(!p->state_stride || len == s.len || len == 0, JGPT_ERR_ILLEGAL_STATE, "sequence %d carries recurrent state of %d tokens", seq, s.len);
     s.len = len;
     s.tick = ++p->clock;
     return JGPT_OK;
@@ -543,6 +597,7 @@ int32_t jgpt_seq_drop_front(jgpt_kvpool h, int32_t seq, int32_t n_blocks, int32_
     JGPT_REQUIRE(n_blocks >= 0 && n_blocks <= (int)s.blocks.size() && s.len >= n_blocks * kBlockTokens, JGPT_ERR_INVALID_ARGUMENT,
                  "cannot drop %d blocks from a sequence of %d tokens in %d blocks", n_blocks, s.len, (int)s.blocks.size());
     if (n_blocks == 0) return JGPT_OK;
+    REQUIRE_UNIFORM(p);
     std::vector<int> freed(s.blocks.begin(), s.blocks.begin() + n_blocks);
     for (int b : freed) p->free_list.push_back(b);
     s.blocks.erase(s.blocks.begin(), s.blocks.begin() + n_blocks);
@@ -642,6 +697,7 @@ int32_t jgpt_kv_evict_lru(jgpt_kvpool h, int32_t need_free, int32_t zero_fill, i
 int32_t jgpt_kv_append(jgpt_kvpool h, int32_t layer, const float *k_dev, const float *v_dev, const int32_t *seq_ids_dev,
                        const int32_t *slot_pos_dev, const int32_t *rope_pos_dev, int32_t n) {
     GET_POOL(p, h);
+    REQUIRE_UNIFORM(p);
     JGPT_REQUIRE(layer >= 0 && layer < p->layers, JGPT_ERR_OUT_OF_RANGE, "layer %d outside [0,%d)", layer, p->layers);
     if (n == 0) return JGPT_OK;
     JGPT_REQUIRE(n > 0 && k_dev && v_dev && seq_ids_dev && slot_pos_dev && rope_pos_dev, JGPT_ERR_INVALID_ARGUMENT,
@@ -652,6 +708,7 @@ int32_t jgpt_kv_append(jgpt_kvpool h, int32_t layer, const float *k_dev, const f
 int32_t jgpt_kv_gather(jgpt_kvpool h, int32_t layer, int32_t seq, int32_t len, int32_t max_seq_len, float *k_out_dev,
                        float *v_out_dev) {
     GET_POOL(p, h);
+    REQUIRE_UNIFORM(p);
     CHECK_SEQ(p, seq);
     JGPT_REQUIRE(layer >= 0 && layer < p->layers, JGPT_ERR_OUT_OF_RANGE, "layer %d outside [0,%d)", layer, p->layers);
     JGPT_REQUIRE(max_seq_len > 0 && len >= 0 && len <= max_seq_len, JGPT_ERR_INVALID_ARGUMENT, "bad len/max_seq_len");
@@ -665,6 +722,7 @@ int32_t jgpt_kv_gather(jgpt_kvpool h, int32_t layer, int32_t seq, int32_t len, i
 int32_t jgpt_kv_gather_batch(jgpt_kvpool h, int32_t layer, const int32_t *seq_ids_host, const int32_t *lens_host, int32_t n,
                              int32_t max_seq_len, float *k_out_dev, float *v_out_dev) {
     GET_POOL(p, h);
+    REQUIRE_UNIFORM(p);
     JGPT_REQUIRE(layer >= 0 && layer < p->layers, JGPT_ERR_OUT_OF_RANGE, "layer %d outside [0,%d)", layer, p->layers);
     if (n == 0) return JGPT_OK;
     JGPT_REQUIRE(n > 0 && n <= 65535 && seq_ids_host && lens_host && k_out_dev && v_out_dev && max_seq_len > 0, JGPT_ERR_INVALID_ARGUMENT,

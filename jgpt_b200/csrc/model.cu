@@ -10,6 +10,7 @@
 // scalar CPU loop.
 #include "common.cuh"
 #include "ptx.cuh"
+#include "decoder.cuh"
 #include "gemm_umma.cuh"
 
 #include <algorithm>
@@ -787,6 +788,19 @@ __global__ void __launch_bounds__(256) sample_kernel(const float *__restrict__ l
     }
 }
 
+// The token choice for models that run their own forward step (decoder.cu).
+int32_t launch_argmax(const float *logits, int rows, int vocab, int *next_dev, cudaStream_t st) {
+    argmax_kernel<<<rows, 256, 0, st>>>(logits, vocab, next_dev);
+    JGPT_CUDA_TRY(cudaGetLastError());
+    return JGPT_OK;
+}
+int32_t launch_sample(const float *logits, float *work, int rows, int vocab, const SampleSpec &spec, const float *u01_dev, int *next_dev,
+                      cudaStream_t st) {
+    sample_kernel<<<rows, 256, 0, st>>>(logits, work, vocab, spec.temperature, spec.top_k, u01_dev, next_dev);
+    JGPT_CUDA_TRY(cudaGetLastError());
+    return JGPT_OK;
+}
+
 // ------------------------------------------------------------------------------------------------
 // Host side
 // ------------------------------------------------------------------------------------------------
@@ -957,10 +971,6 @@ static int32_t ensure_logits(Model *m, int rows) {
     return JGPT_OK;
 }
 
-struct SampleSpec {
-    float temperature = 0.f;  // <= 0: greedy argmax on the device
-    int top_k = 0;
-};
 static int32_t ensure_sample_work(Model *m, int rows) {
     if (rows <= m->samp_rows) return JGPT_OK;
     JGPT_CUDA_TRY(cudaStreamSynchronize(m->ctx->stream));
@@ -1453,9 +1463,10 @@ extern "C" __attribute__((visibility("default"))) int32_t jgpt_debug_timeline_re
 }
 #endif
 
-#define GET_MODEL(m, h)                                         \
-    Model *m = model_registry().get(h);                         \
-    JGPT_REQUIRE(m, JGPT_ERR_BAD_HANDLE, "bad model handle");   \
+#define GET_MODEL(m, h)                                                                                                      \
+    Model *m = model_registry().get(h);                                                                                      \
+    JGPT_REQUIRE(m || !decoder_registry().get(h), JGPT_ERR_UNSUPPORTED, "%s is not available for a layered decoder", __func__); \
+    JGPT_REQUIRE(m, JGPT_ERR_BAD_HANDLE, "bad model handle");                                                                \
     JGPT_CUDA_TRY(make_current(m->ctx))
 
 static int32_t check_pool(const Model *m, const Pool *p) {
@@ -1604,6 +1615,7 @@ int32_t jgpt_model_create(jgpt_ctx ctxh, int32_t vocab, int32_t max_seq_len, int
 }
 
 int32_t jgpt_model_destroy(jgpt_model h) {
+    if (Decoder *d = decoder_registry().get(h)) return decoder_destroy(d);
     GET_MODEL(m, h);
     cudaStreamSynchronize(m->ctx->stream);
     model_registry().remove(m);
@@ -1781,6 +1793,9 @@ int32_t jgpt_model_save_weights(jgpt_model h, const char *path) {
 int32_t jgpt_forward_prefill_batch(jgpt_model h, jgpt_kvpool poolh, const int32_t *seq_ids_host, const int32_t *seq_starts_host,
                                    const int32_t *ids_host, const int32_t *rope_offsets_host, int32_t n, float *all_logits_host,
                                    float *last_logits_host, int32_t *next_tokens_host) {
+    if (Decoder *d = decoder_registry().get(h)) 
+        return decoder_prefill_batch(d, poolh, seq_ids_host, seq_starts_host, ids_host, rope_offsets_host, n, all_logits_host, last_logits_host,
+                                     next_tokens_host);
     GET_MODEL(m, h);
     Pool *p = pool_registry().get(poolh);
     int32_t rc = check_pool(m, p);
@@ -1876,6 +1891,9 @@ int32_t jgpt_forward_prefill(jgpt_model h, jgpt_kvpool poolh, int32_t seq, const
 static int32_t forward_decode_impl(jgpt_model h, jgpt_kvpool poolh, const int32_t *seq_ids_host, const int32_t *ids_host,
                                    const int32_t *cache_len_before_host, const int32_t *rope_pos_host, int32_t n, float *logits_host,
                                    int32_t *next_tokens_host, const SampleSpec &spec, const float *u01_host) {
+    if (Decoder *d = decoder_registry().get(h))
+        return decoder_decode(d, poolh, seq_ids_host, ids_host, cache_len_before_host, rope_pos_host, n, logits_host, next_tokens_host, spec,
+                              u01_host);
     GET_MODEL(m, h);
     Pool *p = pool_registry().get(poolh);
     int32_t rc = check_pool(m, p);
@@ -2073,6 +2091,11 @@ int32_t jgpt_forward_decode_sample(jgpt_model h, jgpt_kvpool poolh, const int32_
 }
 
 int32_t jgpt_model_next_tokens_device(jgpt_model h, const int32_t **dev_out) {
+    if (Decoder *d = decoder_registry().get(h)) {
+        JGPT_REQUIRE(dev_out, JGPT_ERR_INVALID_ARGUMENT, "null output");
+        *dev_out = decoder_next_tokens_device(d);
+        return JGPT_OK;
+    }
     GET_MODEL(m, h);
     JGPT_REQUIRE(dev_out, JGPT_ERR_INVALID_ARGUMENT, "null output");
     *dev_out = m->d_next;
@@ -2164,6 +2187,8 @@ static bool fused_greedy_steps(Model *m, Pool *p, jgpt_kvpool poolh, int32_t seq
 // GPTModel.generateGpuKv with temperature <= 0 (GptAutoregressiveGenerator.java:108-206).
 int32_t jgpt_generate_greedy(jgpt_model h, jgpt_kvpool poolh, const int32_t *prompt_host, int32_t S, int32_t max_new,
                              int32_t *out_host, int32_t *n_sampled_out) {
+    if (Decoder *d = decoder_registry().get(h)) 
+        return decoder_generate_greedy(d, poolh, prompt_host, S, max_new, out_host, n_sampled_out);
     GET_MODEL(m, h);
     Pool *p = pool_registry().get(poolh);
     int32_t rc = check_pool(m, p);

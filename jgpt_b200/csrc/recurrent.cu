@@ -1,0 +1,423 @@
+// Recurrent mixers of the layered decoder: gated linear attention and the gated delta rule, both with a decay per key
+// channel, as ONE kernel from the layer's projections to the gated, normalised head outputs - for prompts, portions of
+// prompts and single tokens alike, so a token's arithmetic does not depend on how its sequence was cut.
+//
+//   GLA    S <- diag(a) S + k v^T;                       o = S^T q
+//   DELTA  S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q   (o read off as S_decayed^T q + (q.k) u)
+//
+// A CTA owns one (sequence, head); a warp owns 16 value columns with every key row of the state in registers: lane =
+// (row lane 0..7, column lane 0..3), DK / 8 rows x 4 columns, rows in pairs for the packed fp32 instructions
+// (fma.rn.f32x2).  Tokens go through in tiles: the CTA first prepares a tile in shared memory (short convolution + silu,
+// unit vectors, decays, step sizes), then every warp walks the tile's tokens on its own - no barrier inside - and the
+// head outputs are normalised and gated from shared memory.  State and all of this arithmetic are fp32.
+//
+// State of a sequence and layer: S as [head][16-column group][DK][16] floats, then the convolution history
+// [2][taps - 1][channels] of projection outputs.  The history has two copies: a step reads the one its entry names and
+// writes the other, because heads that share query / key channels run in different CTAs.  Nothing is cleared when a slot
+// is handed out: a step that starts at position 0 starts from zeros.
+#include "mixers.cuh"
+
+#include <algorithm>
+
+#include "ptx.cuh"
+
+namespace jgpt {
+namespace mix {
+
+constexpr int kMaxTaps = 8;
+constexpr int kTileTokens = 16;
+
+typedef unsigned long long u64;
+__device__ __forceinline__ u64 pack2(float lo, float hi) {
+    u64 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ float2 unpack2(u64 v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ u64 fma2(u64 a, u64 b, u64 c) {
+    u64 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ u64 mul2(u64 a, u64 b) {
+    u64 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
+__device__ __forceinline__ float2 load2(const __nv_bfloat16 *p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(p)); }
+__device__ __forceinline__ float2 load2(const float *p) { return *reinterpret_cast<const float2 *>(p); }
+__device__ __forceinline__ float load1(const __nv_bfloat16 *p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float load1(const float *p) { return *p; }
+__device__ __forceinline__ void store2(__nv_bfloat16 *p, float2 v) { *reinterpret_cast<__nv_bfloat162 *>(p) = __float22bfloat162_rn(v); }
+__device__ __forceinline__ void store2(float *p, float2 v) { *reinterpret_cast<float2 *>(p) = v; }
+__device__ __forceinline__ void store1(__nv_bfloat16 *p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ void store1(float *p, float v) { *p = v; }
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+    for (int off = 16; off >= 1; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
+    return v;
+}
+
+// Eight sums over the eight row lanes (lane bits 2-4): on return a lane holds the total of value 4 * bit4 + 2 * bit3 + bit2.
+__device__ __forceinline__ float reduce8(const float (&lo)[4], const float (&hi)[4], int lane) {
+    const bool b4 = lane & 16, b3 = lane & 8, b2 = lane & 4;
+    float r[4];
+#pragma unroll
+    for (int c = 0; c < 4; c++) r[c] = (b4 ? hi[c] : lo[c]) + __shfl_xor_sync(0xffffffffu, b4 ? lo[c] : hi[c], 16);
+    float s[2];
+#pragma unroll
+    for (int c = 0; c < 2; c++) s[c] = (b3 ? r[c + 2] : r[c]) + __shfl_xor_sync(0xffffffffu, b3 ? r[c] : r[c + 2], 8);
+    return (b2 ? s[1] : s[0]) + __shfl_xor_sync(0xffffffffu, b2 ? s[0] : s[1], 4);
+}
+
+template <class AT, int KIND, int DK>
+__global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const RecArgs a, const Seg *__restrict__ segs, int col_split, int tt,
+                                                                          int pdl) {
+    constexpr int NI = DK / 32;  // groups of four rows per lane
+    extern __shared__ __align__(16) float rec_smem[];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rl = lane >> 2, cl = lane & 3;
+    const int nthreads = blockDim.x, nw = nthreads >> 5, DVc = nw * 16;
+    const int h = blockIdx.x % a.heads, split = blockIdx.x / a.heads, col0 = split * DVc;
+    float *sq = rec_smem, *sk = sq + tt * DK, *sg = sk + tt * DK, *sv = sg + tt * DK, *so = sv + tt * DVc, *sbeta = so + tt * DVc,
+          *sqk = sbeta + tt;
+
+    if (pdl & 2) griddep_launch_dependents();
+    const Seg sgm = segs[blockIdx.y];
+    if (sgm.seq < 0 || sgm.seq >= a.max_seqs) {
+        if (tid == 0) atomicOr(a.status, DEV_STATUS_BAD_SEQ);
+        return;
+    }
+    uint8_t *part = a.state + (uint64_t)sgm.seq * a.state_stride;
+    float *S = reinterpret_cast<float *>(part) + ((size_t)h * (a.DV / 16) + col0 / 16 + warp) * (DK * 16);
+    // no kernel of this step but this one touches this layer's state, and earlier steps are complete: read before the wait
+    u64 st[NI * 2][4];
+#pragma unroll
+    for (int i = 0; i < NI * 2; i++) {
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
+        if (sgm.pos0 > 0) {
+            const float *row = S + (size_t)((i >> 1) * 32 + rl * 4 + (i & 1) * 2) * 16 + cl * 4;
+            x = *reinterpret_cast<const float4 *>(row), y = *reinterpret_cast<const float4 *>(row + 16);
+        }
+        st[i][0] = pack2(x.x, y.x), st[i][1] = pack2(x.y, y.y), st[i][2] = pack2(x.z, y.z), st[i][3] = pack2(x.w, y.w);
+    }
+    if (pdl & 1) griddep_wait();
+
+    const AT *__restrict__ proj = reinterpret_cast<const AT *>(a.proj) + (size_t)sgm.row0 * a.ldp;
+    const AT *__restrict__ z = reinterpret_cast<const AT *>(a.z) + (size_t)sgm.row0 * a.ldz;
+    const int kvh = h / (a.heads / a.kv_heads);
+    const int nq = a.kv_heads * DK, channels = 2 * nq + a.heads * a.DV;  // convolution channels: q, k, v
+    const AT *hist = reinterpret_cast<const AT *>(part + a.conv_off) + (size_t)sgm.conv_set * (a.taps > 0 ? a.taps - 1 : 0) * channels;
+    const float qscale = rsqrtf((float)a.dim);
+    const float rate = KIND == REC_DELTA ? expf(a.a_log[h]) : 1.f / a.tau;
+    // the input of the convolution at token t of this entry (t < 0: history; before position 0: zero)
+    auto conv_input = [&](int t, int proj_col, int channel) -> float2 {
+        if (t >= 0) return load2(proj + (size_t)t * a.ldp + proj_col);
+        if (sgm.pos0 + t >= 0) return load2(hist + (size_t)(-1 - t) * channels + channel);
+        return make_float2(0.f, 0.f);
+    };
+    // channel pair idx of this CTA: q, then k, then its value columns
+    auto locate = [&](int idx, int &proj_col, int &channel, float *&dst, int &ld, const float *&w) {
+        if (idx < DK / 2) {
+            const int c = kvh * DK + 2 * idx;
+            proj_col = a.q_off + c, channel = c, dst = sq + 2 * idx, ld = DK, w = a.conv_q + (size_t)c * a.taps;
+        } else if (idx < DK) {
+            const int c = kvh * DK + 2 * idx - DK;
+            proj_col = a.k_off + c, channel = nq + c, dst = sk + 2 * idx - DK, ld = DK, w = a.conv_k + (size_t)c * a.taps;
+        } else {
+            const int j = 2 * (idx - DK), c = h * a.DV + col0 + j;
+            proj_col = a.v_off + c, channel = 2 * nq + c, dst = sv + j, ld = DVc, w = a.conv_v + (size_t)c * a.taps;
+        }
+    };
+    const int npairs = DK + DVc / 2;
+
+    for (int t0 = 0; t0 < sgm.T; t0 += tt) {
+        const int tn = min(tt, sgm.T - t0);
+        // ---- prepare the tile ----
+        for (int idx = tid; idx < npairs; idx += nthreads) {
+            int pc, ch, ld;
+            float *dst;
+            const float *w;
+            locate(idx, pc, ch, dst, ld, w);
+            if (KIND == REC_DELTA) {
+                float2 wt[kMaxTaps], win[kMaxTaps];  // right-aligned: entry kMaxTaps - 1 is the current token's
+#pragma unroll
+                for (int i = 0; i < kMaxTaps; i++) {
+                    const int back = kMaxTaps - 1 - i;
+                    const bool on = back < a.taps;
+                    wt[i] = on ? make_float2(w[a.taps - 1 - back], w[2 * a.taps - 1 - back]) : make_float2(0.f, 0.f);
+                    // the window in front of the tile's first token: entry i holds token t0 - back
+                    win[i] = on && back > 0 ? conv_input(t0 - back, pc, ch) : make_float2(0.f, 0.f);
+                }
+#pragma unroll 4
+                for (int t = 0; t < tn; t++) {
+                    win[kMaxTaps - 1] = load2(proj + (size_t)(t0 + t) * a.ldp + pc);
+                    float2 y = make_float2(0.f, 0.f);
+#pragma unroll
+                    for (int i = 0; i < kMaxTaps; i++) y.x = fmaf(wt[i].x, win[i].x, y.x), y.y = fmaf(wt[i].y, win[i].y, y.y);
+                    y.x *= sigmoid_f(y.x), y.y *= sigmoid_f(y.y);
+                    *reinterpret_cast<float2 *>(dst + t * ld) = y;
+#pragma unroll
+                    for (int i = 0; i + 1 < kMaxTaps; i++) win[i] = win[i + 1];
+                }
+            } else {
+                const float f = idx < DK / 2 ? qscale : 1.f;
+#pragma unroll 4
+                for (int t = 0; t < tn; t++) {
+                    float2 y = load2(proj + (size_t)(t0 + t) * a.ldp + pc);
+                    y.x *= f, y.y *= f;
+                    *reinterpret_cast<float2 *>(dst + t * ld) = y;
+                }
+                if (tn & 1) *reinterpret_cast<float2 *>(dst + tn * ld) = make_float2(0.f, 0.f);  // pads the last pair of tokens
+            }
+        }
+        for (int idx = tid; idx < tn * (DK / 2); idx += nthreads) {
+            const int t = idx / (DK / 2), c = 2 * (idx % (DK / 2));
+            float2 y = load2(z + (size_t)(t0 + t) * a.ldz + a.z_off + h * DK + c);
+            const float2 b = *reinterpret_cast<const float2 *>(a.decay_bias + h * DK + c);
+            y.x += b.x, y.y += b.y;
+            if (KIND == REC_DELTA) y.x = expf(-rate * softplus_f(y.x)), y.y = expf(-rate * softplus_f(y.y));
+            else y.x = expf(-rate * softplus_f(-y.x)), y.y = expf(-rate * softplus_f(-y.y));  // sigmoid(z)^(1 / tau)
+            *reinterpret_cast<float2 *>(sg + t * DK + c) = y;
+        }
+        if (KIND == REC_GLA && (tn & 1))
+            for (int c = tid; c < DK; c += nthreads) sg[tn * DK + c] = 1.f;
+        __syncthreads();
+        if (KIND == REC_DELTA) {
+            for (int t = warp; t < tn; t += nw) {
+                float qv[NI], kv[NI], qq = 0.f, kk = 0.f, qk = 0.f;
+#pragma unroll
+                for (int i = 0; i < NI; i++) {
+                    qv[i] = sq[t * DK + lane + 32 * i], kv[i] = sk[t * DK + lane + 32 * i];
+                    qq += qv[i] * qv[i], kk += kv[i] * kv[i], qk += qv[i] * kv[i];
+                }
+                qq = warp_sum(qq), kk = warp_sum(kk), qk = warp_sum(qk);
+                const float fq = qscale / sqrtf(qq + 1e-6f), fk = 1.f / sqrtf(kk + 1e-6f);
+#pragma unroll
+                for (int i = 0; i < NI; i++) sq[t * DK + lane + 32 * i] = qv[i] * fq, sk[t * DK + lane + 32 * i] = kv[i] * fk;
+                if (lane == 0) sqk[t] = qk * fq * fk, sbeta[t] = sigmoid_f(load1(proj + (size_t)(t0 + t) * a.ldp + a.b_off + h));
+            }
+            __syncthreads();
+        }
+        // ---- the recurrence: every warp on its own columns ----
+        const int vcol = warp * 16 + cl * 4;
+        if (KIND == REC_DELTA) {
+            for (int t = 0; t < tn; t++) {
+                u64 ks[4] = {0, 0, 0, 0}, qs[4] = {0, 0, 0, 0};
+                const float *qp = sq + t * DK + rl * 4, *kp = sk + t * DK + rl * 4, *gp = sg + t * DK + rl * 4;
+#pragma unroll
+                for (int i = 0; i < NI; i++) {
+                    const ulonglong2 q2 = *reinterpret_cast<const ulonglong2 *>(qp + 32 * i);
+                    const ulonglong2 k2 = *reinterpret_cast<const ulonglong2 *>(kp + 32 * i);
+                    const ulonglong2 g2 = *reinterpret_cast<const ulonglong2 *>(gp + 32 * i);
+#pragma unroll
+                    for (int c = 0; c < 4; c++) {
+                        st[2 * i][c] = mul2(g2.x, st[2 * i][c]);
+                        st[2 * i + 1][c] = mul2(g2.y, st[2 * i + 1][c]);
+                        ks[c] = fma2(k2.x, st[2 * i][c], ks[c]), ks[c] = fma2(k2.y, st[2 * i + 1][c], ks[c]);
+                        qs[c] = fma2(q2.x, st[2 * i][c], qs[c]), qs[c] = fma2(q2.y, st[2 * i + 1][c], qs[c]);
+                    }
+                }
+                float kf[4], qf[4];
+#pragma unroll
+                for (int c = 0; c < 4; c++) {
+                    const float2 x = unpack2(ks[c]), y = unpack2(qs[c]);
+                    kf[c] = x.x + x.y, qf[c] = y.x + y.y;
+                }
+                const float tot = reduce8(kf, qf, lane);
+                const float4 v4 = *reinterpret_cast<const float4 *>(sv + t * DVc + vcol);
+                const float beta = sbeta[t];
+                float u[4];
+#pragma unroll
+                for (int c = 0; c < 4; c++) {
+                    const float sk_c = __shfl_sync(0xffffffffu, tot, ((c & 2) << 2) | ((c & 1) << 2) | cl);
+                    u[c] = beta * ((c == 0 ? v4.x : c == 1 ? v4.y : c == 2 ? v4.z : v4.w) - sk_c);
+                }
+                if (lane & 16) {
+                    const int c = rl & 3;
+                    const float uc = c == 0 ? u[0] : c == 1 ? u[1] : c == 2 ? u[2] : u[3];
+                    so[t * DVc + vcol + c] = fmaf(sqk[t], uc, tot);
+                }
+#pragma unroll
+                for (int c = 0; c < 4; c++) {
+                    const u64 u2 = pack2(u[c], u[c]);
+#pragma unroll
+                    for (int i = 0; i < NI; i++) {
+                        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2 *>(kp + 32 * i);
+                        st[2 * i][c] = fma2(k2.x, u2, st[2 * i][c]), st[2 * i + 1][c] = fma2(k2.y, u2, st[2 * i + 1][c]);
+                    }
+                }
+            }
+        } else {
+            for (int t = 0; t < tn; t += 2) {
+                float of[2][4];
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    u64 qs[4] = {0, 0, 0, 0}, v2[4];
+                    const float *qp = sq + (t + e) * DK + rl * 4, *kp = sk + (t + e) * DK + rl * 4, *gp = sg + (t + e) * DK + rl * 4;
+                    const float4 v4 = *reinterpret_cast<const float4 *>(sv + (t + e) * DVc + vcol);
+                    v2[0] = pack2(v4.x, v4.x), v2[1] = pack2(v4.y, v4.y), v2[2] = pack2(v4.z, v4.z), v2[3] = pack2(v4.w, v4.w);
+#pragma unroll
+                    for (int i = 0; i < NI; i++) {
+                        const ulonglong2 q2 = *reinterpret_cast<const ulonglong2 *>(qp + 32 * i);
+                        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2 *>(kp + 32 * i);
+                        const ulonglong2 g2 = *reinterpret_cast<const ulonglong2 *>(gp + 32 * i);
+#pragma unroll
+                        for (int c = 0; c < 4; c++) {
+                            st[2 * i][c] = fma2(k2.x, v2[c], mul2(g2.x, st[2 * i][c]));
+                            st[2 * i + 1][c] = fma2(k2.y, v2[c], mul2(g2.y, st[2 * i + 1][c]));
+                            qs[c] = fma2(q2.x, st[2 * i][c], qs[c]), qs[c] = fma2(q2.y, st[2 * i + 1][c], qs[c]);
+                        }
+                    }
+#pragma unroll
+                    for (int c = 0; c < 4; c++) {
+                        const float2 y = unpack2(qs[c]);
+                        of[e][c] = y.x + y.y;
+                    }
+                }
+                const float tot = reduce8(of[0], of[1], lane);
+                so[(t + (lane >> 4)) * DVc + vcol + (rl & 3)] = tot;  // row tn of an odd tile is a spare
+            }
+        }
+        __syncthreads();
+        // ---- head outputs: RMS norm over the value columns, gate ----
+        if (col_split > 1) {
+            for (int idx = tid; idx < tn * DVc; idx += nthreads)
+                a.raw[(size_t)(sgm.row0 + t0 + idx / DVc) * (a.heads * a.DV) + h * a.DV + col0 + idx % DVc] = so[idx];
+        } else {
+            for (int t = warp; t < tn; t += nw) {
+                float ss = 0.f;
+                for (int c = lane; c < DVc; c += 32) {
+                    const float v = so[t * DVc + c];
+                    ss += v * v;
+                }
+                const float inv = a.out_scale / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
+                AT *o = reinterpret_cast<AT *>(a.out) + (size_t)(sgm.row0 + t0 + t) * a.ldo + a.out_off + h * DVc;
+                const AT *gp = KIND == REC_DELTA ? z + (size_t)(t0 + t) * a.ldz + a.zg_off + h * DVc
+                                                 : proj + (size_t)(t0 + t) * a.ldp + a.g_off + h * DVc;
+                for (int c = lane; c < DVc; c += 32) {
+                    const float gt = load1(gp + c), sgt = sigmoid_f(gt);
+                    store1(o + c, so[t * DVc + c] * inv * a.norm_w[c] * (KIND == REC_DELTA ? sgt : gt * sgt));
+                }
+            }
+        }
+    }
+    // ---- leave the state for the next step ----
+#pragma unroll
+    for (int i = 0; i < NI * 2; i++) {
+        float *row = S + (size_t)((i >> 1) * 32 + rl * 4 + (i & 1) * 2) * 16 + cl * 4;
+        const float2 c0 = unpack2(st[i][0]), c1 = unpack2(st[i][1]), c2 = unpack2(st[i][2]), c3 = unpack2(st[i][3]);
+        *reinterpret_cast<float4 *>(row) = make_float4(c0.x, c1.x, c2.x, c3.x);
+        *reinterpret_cast<float4 *>(row + 16) = make_float4(c0.y, c1.y, c2.y, c3.y);
+    }
+    if (KIND == REC_DELTA && a.taps > 1) {
+        AT *next = reinterpret_cast<AT *>(part + a.conv_off) + (size_t)(1 - sgm.conv_set) * (a.taps - 1) * channels;
+        const bool first_of_group = h % (a.heads / a.kv_heads) == 0 && split == 0;
+        for (int idx = tid; idx < npairs; idx += nthreads) {
+            if (idx < DK && !first_of_group) continue;  // shared channels are written once
+            int pc, ch, ld;
+            float *dst;
+            const float *w;
+            locate(idx, pc, ch, dst, ld, w);
+            for (int i = 0; i < a.taps - 1; i++) store2(next + (size_t)i * channels + ch, conv_input(sgm.T - 1 - i, pc, ch));
+        }
+    }
+}
+
+// RMS norm and gate of heads whose columns were cut over several CTAs.  One warp per (row, head).
+template <class AT, int KIND>
+__global__ void __launch_bounds__(256) gated_norm_kernel(const RecArgs a, int rows) {
+    const int item = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (item >= rows * a.heads) return;
+    const int r = item / a.heads, h = item % a.heads;
+    const float *raw = a.raw + (size_t)r * a.heads * a.DV + h * a.DV;
+    float ss = 0.f;
+    for (int c = lane; c < a.DV; c += 32) ss += raw[c] * raw[c];
+    const float inv = a.out_scale / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
+    AT *o = reinterpret_cast<AT *>(a.out) + (size_t)r * a.ldo + a.out_off + h * a.DV;
+    const AT *gp = KIND == REC_DELTA ? reinterpret_cast<const AT *>(a.z) + (size_t)r * a.ldz + a.zg_off + h * a.DV
+                                     : reinterpret_cast<const AT *>(a.proj) + (size_t)r * a.ldp + a.g_off + h * a.DV;
+    for (int c = lane; c < a.DV; c += 32) {
+        const float gt = load1(gp + c), sgt = sigmoid_f(gt);
+        store1(o + c, raw[c] * inv * a.norm_w[c] * (KIND == REC_DELTA ? sgt : gt * sgt));
+    }
+}
+
+int rec_padded_key(int dim) {
+    for (int d : {32, 64, 96, 128, 192, 256})
+        if (dim <= d) return dim > 0 ? d : 0;
+    return 0;
+}
+int rec_padded_value(int vdim) { return vdim > 0 && vdim <= 256 ? (vdim + 15) / 16 * 16 : 0; }
+
+uint64_t rec_state_bytes(const RecArgs &a, int elem_bytes, uint64_t *conv_off) {
+    const uint64_t s = (uint64_t)a.heads * a.DK * a.DV * sizeof(float);
+    *conv_off = s;
+    const uint64_t channels = 2ull * a.kv_heads * a.DK + (uint64_t)a.heads * a.DV;
+    const uint64_t conv = a.taps > 1 ? 2ull * (uint64_t)(a.taps - 1) * channels * (uint64_t)elem_bytes : 0;
+    return (s + conv + 255) / 256 * 256;
+}
+
+template <class AT, int KIND, int DK>
+static int32_t rec_launch(const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st) {
+    const bool single = d.n_tiles == 0;
+    const int tt = single ? 2 : kTileTokens;
+    const int groups = a.DV / 16, max_groups = DK <= 128 ? 16 : 8;
+    int split = 1;
+    auto allowed = [&](int s) { return groups % s == 0; };
+    while (split < groups && (!allowed(split) || groups / split > max_groups)) split++;
+    // a few long entries: more CTAs per head (each prepares the tile's q, k again) and a norm kernel behind them
+    if (!single)
+        while (a.heads * d.n_segs * split * 2 <= a.sm_count && groups / split >= 4 && allowed(split * 2)) split *= 2;
+    const int nw = groups / split, DVc = nw * 16;
+    const size_t smem = sizeof(float) * ((size_t)tt * (3 * DK + 2 * DVc) + 2 * tt);
+    auto kern = recurrent_kernel<AT, KIND, DK>;
+    static thread_local int set_for = -1;
+    int dev = 0;
+    JGPT_CUDA_TRY(cudaGetDevice(&dev));
+    if (set_for != dev) {
+        JGPT_CUDA_TRY(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(float) * (kTileTokens * (3 * DK + 2 * 256) + 2 * kTileTokens))));
+        set_for = dev;
+    }
+    cudaLaunchConfig_t cfg = {};
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.gridDim = dim3((unsigned)(a.heads * split), (unsigned)d.n_segs), cfg.blockDim = dim3((unsigned)(32 * nw));
+    cfg.dynamicSmemBytes = smem, cfg.stream = st, cfg.attrs = attr, cfg.numAttrs = (pdl & 1) ? 1 : 0;
+    JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, kern, a, d.segs, split, tt, pdl));
+    if (split > 1) {
+        gated_norm_kernel<AT, KIND><<<(unsigned)((d.rows * a.heads + 7) / 8), 256, 0, st>>>(a, d.rows);
+        JGPT_CUDA_TRY(cudaGetLastError());
+    }
+    return JGPT_OK;
+}
+
+template <class AT, int KIND>
+static int32_t rec_dispatch(const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st) {
+    switch (a.DK) {
+        case 32: return rec_launch<AT, KIND, 32>(d, a, pdl, st);
+        case 64: return rec_launch<AT, KIND, 64>(d, a, pdl, st);
+        case 96: return rec_launch<AT, KIND, 96>(d, a, pdl, st);
+        case 128: return rec_launch<AT, KIND, 128>(d, a, pdl, st);
+        case 192: return rec_launch<AT, KIND, 192>(d, a, pdl, st);
+        case 256: return rec_launch<AT, KIND, 256>(d, a, pdl, st);
+        default: return fail(JGPT_ERR_UNSUPPORTED, "key size %d", a.DK);
+    }
+}
+
+int32_t launch_recurrent(bool f32, const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st) {
+    JGPT_REQUIRE(a.taps <= kMaxTaps, JGPT_ERR_UNSUPPORTED, "convolutions of up to %d taps", kMaxTaps);
+    if (f32) return a.kind == REC_DELTA ? rec_dispatch<float, REC_DELTA>(d, a, pdl, st) : rec_dispatch<float, REC_GLA>(d, a, pdl, st);
+    return a.kind == REC_DELTA ? rec_dispatch<__nv_bfloat16, REC_DELTA>(d, a, pdl, st) : rec_dispatch<__nv_bfloat16, REC_GLA>(d, a, pdl, st);
+}
+
+}  // namespace mix
+}  // namespace jgpt

@@ -15,9 +15,12 @@
 //     2. all requests admitted in this step are prefilled in one batched call (split when the rows exceed
 //        the model workspace); the argmax of each last row is the request's first new token.
 //     3. every request that was already running takes one batched decode step.
+//     (A layered decoder takes steps that mix portions of prompts with decoded tokens: 2. and 3. are then one step whose
+//     rows are the running requests' tokens followed, in admission order, by as much of the unfinished prompts as the
+//     workspace holds; a prompt may be longer than the workspace and samples its first token when its last row has run.)
 //     4. a request finishes when it has max_new tokens or sampled id 0; its blocks stay in the pool, marked
 //        evictable, until admission needs them.
-#include "common.cuh"
+#include "decoder.cuh"
 
 #include <algorithm>
 #include <deque>
@@ -37,6 +40,7 @@ struct Request {
     std::vector<int> prompt;
     std::vector<int> out;  // sampled tokens
     int max_new = 0, seq = -1, state = REQ_WAITING;
+    int done = 0;  // prompt rows that have run (layered decoders)
 };
 
 struct Sched {
@@ -122,7 +126,7 @@ int32_t jgpt_sched_submit(uint64_t h, const int32_t *prompt_host, int32_t S, int
     // no sliding window while batching: the whole request must fit the context and the per-sequence table
     JGPT_REQUIRE(S + max_new - 1 <= s->max_seq && S + max_new <= s->p->max_blocks_per_seq * kBlockTokens + 1,
                  JGPT_ERR_INVALID_ARGUMENT, "prompt %d + %d new tokens exceed the context of %d", S, max_new, s->max_seq);
-    JGPT_REQUIRE(S <= s->max_rows, JGPT_ERR_INVALID_ARGUMENT, "prompt of %d rows exceeds the per-call workspace of %d", S, s->max_rows);
+    JGPT_REQUIRE(decoder_registry().get(s->model) || S <= s->max_rows, JGPT_ERR_INVALID_ARGUMENT, "prompt of %d rows exceeds the per-call workspace of %d", S, s->max_rows);
     // a reservation larger than the whole pool could never be admitted and would block the queue for ever
     const int need_blocks = (S + max_new - 1 + kBlockTokens - 1) / kBlockTokens;
     JGPT_REQUIRE(need_blocks <= s->p->n_blocks, JGPT_ERR_INVALID_ARGUMENT,
@@ -181,8 +185,41 @@ int32_t jgpt_sched_step(uint64_t h, int32_t *pairs_out, int32_t cap_pairs, int32
         s->events.insert(s->events.end(), {EV_ADMIT, rid, seq});
     }
 
+    // ---- 2. + 3. for models that take mixed steps ----
+    Decoder *dec = decoder_registry().get(s->model);
+    if (dec) {
+        std::vector<int> seqs, starts{0}, ids, want, owner, portion;
+        auto entry = [&](int rid, const int *tok, int T, bool sample) {
+            ids.insert(ids.end(), tok, tok + T);
+            seqs.push_back(s->reqs[(size_t)rid].seq), starts.push_back((int)ids.size());
+            if (sample) want.push_back((int)ids.size() - 1), owner.push_back(rid);
+        };
+        for (int rid : s->running)
+            if (!s->reqs[(size_t)rid].out.empty()) entry(rid, &s->reqs[(size_t)rid].out.back(), 1, true);
+        for (int rid : s->running) {
+            const Request &r = s->reqs[(size_t)rid];
+            const int left = (int)r.prompt.size() - r.done, T = std::min(left, s->max_rows - (int)ids.size());
+            if (!r.out.empty() || T <= 0) continue;
+            entry(rid, r.prompt.data() + r.done, T, T == left);
+            portion.push_back(rid), portion.push_back(T);
+        }
+        if (!seqs.empty()) {
+            std::vector<int> next(want.size());
+            StepCall c;
+            c.n = (int)seqs.size(), c.seq_ids = seqs.data(), c.starts = starts.data(), c.ids = ids.data();
+            c.n_want = (int)want.size(), c.want = want.data(), c.next_host = next.data();
+            const int32_t rc = decoder_step(dec, p, s->pool, c);
+            if (rc) return rc;
+            for (size_t i = 0; i < portion.size(); i += 2) s->reqs[(size_t)portion[i]].done += portion[i + 1];
+            for (size_t i = 0; i < owner.size(); i++) {
+                s->reqs[(size_t)owner[i]].out.push_back(next[i]);
+                produced.push_back(owner[i]), produced.push_back(next[i]);
+            }
+        }
+    }
+
     // ---- 2. batched prefill of the newly admitted requests ----
-    for (size_t a0 = 0; a0 < admitted.size();) {
+    for (size_t a0 = 0; !dec && a0 < admitted.size();) {
         std::vector<int> seqs, starts{0}, ids, ro;
         size_t a1 = a0;
         while (a1 < admitted.size()) {
@@ -207,7 +244,7 @@ int32_t jgpt_sched_step(uint64_t h, int32_t *pairs_out, int32_t cap_pairs, int32
     }
 
     // ---- 3. one decode step for the requests that were already running ----
-    if (!decoding.empty()) {
+    if (!dec && !decoding.empty()) {
         std::vector<int> seqs, toks, lens, rope;
         for (int rid : decoding) {
             const Request &r = s->reqs[(size_t)rid];
@@ -228,7 +265,7 @@ int32_t jgpt_sched_step(uint64_t h, int32_t *pairs_out, int32_t cap_pairs, int32
     std::vector<int> still;
     for (int rid : s->running) {
         Request &r = s->reqs[(size_t)rid];
-        if ((int)r.out.size() >= r.max_new || r.out.back() == 0) finish(s, rid);
+        if (!r.out.empty() && ((int)r.out.size() >= r.max_new || r.out.back() == 0)) finish(s, rid);
         else still.push_back(rid);
     }
     s->running.swap(still);

@@ -1,0 +1,223 @@
+"""Layered decoders: models the library assembles from layer descriptions (``jgpt_decoder_create``).
+
+``DecoderConfig`` is the description (what ``jgpt_layer_spec`` holds) plus the names of the tensors each part is loaded
+from; designs build it from their config.json (``registry.py``).  ``DecoderModel`` has the methods of ``GPTModel`` that do
+not depend on its fixed block, so generation and ``ContinuousBatcher`` take either.
+"""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass, field
+
+import numpy as np
+
+from . import binding as B
+from .kv_cache import KvPool
+from .runtime import Context
+
+MIX_ATTENTION, MIX_GLA, MIX_DELTA = 1, 2, 3
+DTYPES = {"bfloat16": 0, "float32": 1}
+BLOCK_TOKENS = 16
+
+
+class _MixerSpec(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("kind", "heads", "kv_heads", "dim", "vdim", "chunk", "gate", "taps", "rank_a", "rank_g")] + \
+               [(n, C.c_float) for n in ("score_scale", "tau", "out_scale")]
+
+
+class _LayerSpec(C.Structure):
+    _fields_ = [("n_branches", C.c_int32), ("branch", _MixerSpec * 2), ("ff", C.c_int32)]
+
+
+class _DecoderSpec(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("vocab", "width", "max_positions", "n_layers", "embed_norm")] + \
+               [(n, C.c_float) for n in ("eps", "embed_scale", "logit_scale")]
+
+
+# tensor roles (JGPT_W_* of the header)
+W_EMBED, W_POS, W_EMBED_NORM, W_EMBED_NORM_B, W_FINAL_NORM, W_FINAL_NORM_B = range(6)
+W_NORM1, W_NORM1_B, W_NORM2, W_NORM2_B, W_FF_GATE, W_FF_UP, W_FF_DOWN = range(10, 17)
+(W_Q, W_K, W_V, W_O, W_G, W_B, W_A1, W_A2, W_DECAY_BIAS, W_A_LOG, W_G1, W_G2, W_HEAD_NORM, W_CONV_Q, W_CONV_K,
+ W_CONV_V) = range(20, 36)
+
+
+@dataclass
+class Mixer:
+    kind: int
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    chunk: int = 0
+    gate: bool = False
+    taps: int = 0
+    rank_a: int = 0
+    rank_g: int = 0
+    score_scale: float = 1.0
+    tau: float = 1.0
+    out_scale: float = 1.0
+    tensors: dict = field(default_factory=dict)  # role -> tensor name
+
+
+@dataclass
+class Layer:
+    branches: list
+    ff: int = 0
+    tensors: dict = field(default_factory=dict)
+
+
+@dataclass
+class DecoderConfig:
+    vocab: int
+    width: int
+    max_positions: int
+    eps: float
+    layers: list
+    embed_norm: bool = False
+    embed_scale: float = 1.0
+    logit_scale: float = 1.0
+    tensors: dict = field(default_factory=dict)
+
+    def all_tensors(self):
+        """(layer, branch, role, name) of every tensor the model needs."""
+        for role, name in self.tensors.items():
+            yield -1, -1, role, name
+        for i, layer in enumerate(self.layers):
+            for role, name in layer.tensors.items():
+                yield i, -1, role, name
+            for j, m in enumerate(layer.branches):
+                for role, name in m.tensors.items():
+                    yield i, j, role, name
+
+
+class DecoderModel:
+    def __init__(self, ctx: Context, config: DecoderConfig, dtype="bfloat16", maxRows=2048):
+        if dtype not in DTYPES:
+            raise ValueError(f"dtype {dtype}: one of {', '.join(DTYPES)}")
+        self.ctx, self._lib, self.config, self.dtype = ctx, ctx._lib, config, dtype
+        self.vocabSize, self.maxSeqLen, self.dModel = config.vocab, config.max_positions, config.width
+        self.numLayers, self.maxRows = len(config.layers), maxRows
+        layers = (_LayerSpec * len(config.layers))()
+        for spec, layer in zip(layers, config.layers):
+            if not 1 <= len(layer.branches) <= 2:
+                raise ValueError(f"a layer has one or two mixer branches, not {len(layer.branches)}")
+            spec.n_branches, spec.ff = len(layer.branches), layer.ff
+            for b, m in zip(spec.branch, layer.branches):
+                for n, _ in _MixerSpec._fields_:
+                    setattr(b, n, int(m.gate) if n == "gate" else getattr(m, n))
+        top = _DecoderSpec(config.vocab, config.width, config.max_positions, len(config.layers), int(config.embed_norm),
+                           config.eps, config.embed_scale, config.logit_scale)
+        h = C.c_uint64()
+        B.check(self._lib.jgpt_decoder_create(ctx.handle, C.byref(top), layers, DTYPES[dtype], maxRows, C.byref(h)))
+        self.handle = h.value
+
+    # ---- weights -------------------------------------------------------------------------------
+    def setTensor(self, layer, branch, role, array):
+        a = np.ascontiguousarray(array, np.float32)
+        rows, cols = (1, a.size) if a.ndim == 1 else a.shape
+        B.check(self._lib.jgpt_decoder_set_tensor(self.handle, layer, branch, role, a.ctypes.data, rows, cols))
+
+    def loadTensors(self, get):
+        """``get(name)`` returns the array of a tensor name of the configuration."""
+        for layer, branch, role, name in self.config.all_tensors():
+            try:
+                self.setTensor(layer, branch, role, get(name))
+            except ValueError as e:
+                raise ValueError(f"{name}: {e}") from None
+
+    def newPool(self, n_blocks, max_seqs, max_blocks_per_seq=None) -> "DecoderPool":
+        return DecoderPool(self, n_blocks, max_seqs, max_blocks_per_seq or -(-self.maxSeqLen // BLOCK_TOKENS))
+
+    # ---- forward step --------------------------------------------------------------------------
+    def step(self, pool: KvPool, seqs, tokens, want=(), want_logits=True, want_next=False):
+        """One mixed step: ``tokens[i]`` continues sequence ``seqs[i]``; ``want`` = rows of the concatenated tokens.
+        Returns (logits [len(want), vocab] or None, greedy next tokens [len(want)] or None)."""
+        starts = np.zeros(len(seqs) + 1, np.int32)
+        starts[1:] = np.cumsum([len(t) for t in tokens])
+        ids = np.ascontiguousarray(np.concatenate([np.asarray(t, np.int32) for t in tokens]), np.int32)
+        sq, w = np.ascontiguousarray(seqs, np.int32), np.ascontiguousarray(want, np.int32)
+        logits = np.empty((w.size, self.vocabSize), np.float32) if want_logits else None
+        nxt = np.empty(w.size, np.int32) if want_next else None
+        B.check(self._lib.jgpt_forward_step(self.handle, pool.handle, sq.size, sq.ctypes.data, starts.ctypes.data, ids.ctypes.data, w.size,
+                                            w.ctypes.data if w.size else None, logits.ctypes.data if logits is not None else None,
+                                            nxt.ctypes.data if nxt is not None else None))
+        return logits, nxt
+
+    def captureLayers(self, rows) -> np.ndarray:
+        """The residual after every layer of the next step lands in the returned array, [layers, rows, width]."""
+        out = np.empty((self.numLayers, rows, self.dModel), np.float32)
+        B.check(self._lib.jgpt_decoder_capture_layers(self.handle, out.ctypes.data, out.size))
+        return out
+
+    def forwardDecodeBatch(self, pool, seqs, tokens, cacheLenBefore, ropePositions=None, want_logits=True):
+        """One decode step for n independent sequences -> (logits [n, vocab] or None, greedy next tokens [n])."""
+        sq, tk, lb = (np.ascontiguousarray(x, np.int32) for x in (seqs, tokens, cacheLenBefore))
+        rp = lb if ropePositions is None else np.ascontiguousarray(ropePositions, np.int32)
+        logits = np.empty((sq.size, self.vocabSize), np.float32) if want_logits else None
+        nxt = np.empty(sq.size, np.int32)
+        B.check(self._lib.jgpt_forward_decode(self.handle, pool.handle, sq.ctypes.data, tk.ctypes.data, lb.ctypes.data, rp.ctypes.data, sq.size,
+                                              logits.ctypes.data if want_logits else None, nxt.ctypes.data))
+        return logits, nxt
+
+    def forwardDecodeSampleBatch(self, pool, seqs, tokens, cacheLenBefore, temperature, topK, u01):
+        """One decode step + ``sampleNextToken`` per row on the device with the uniform draws ``u01`` -> next tokens [n]."""
+        sq, tk, lb = (np.ascontiguousarray(x, np.int32) for x in (seqs, tokens, cacheLenBefore))
+        u = np.ascontiguousarray(u01, np.float32)
+        if u.size != sq.size:
+            raise ValueError("one uniform draw per row")
+        nxt = np.empty(sq.size, np.int32)
+        B.check(self._lib.jgpt_forward_decode_sample(self.handle, pool.handle, sq.ctypes.data, tk.ctypes.data, lb.ctypes.data, lb.ctypes.data,
+                                                     sq.size, float(temperature), int(topK), u.ctypes.data, nxt.ctypes.data))
+        return nxt
+
+    # ---- generation ----------------------------------------------------------------------------
+    def generateGpuKv(self, inputTokens, maxNewTokens, temperature=0.0, topK=0, pool: KvPool | None = None, rng=None):
+        """Ids [S + maxNewTokens]: the prompt, then the picked tokens, a zero tail after an early stop on id 0 (the rules of
+        ``GPTModel.generateGpuKv``; no sliding window: prompt and new tokens must fit the model's positions)."""
+        prompt = np.ascontiguousarray(inputTokens, np.int32).reshape(-1)
+        own = pool is None
+        if own:
+            pool = self.newPool(-(-min(self.maxSeqLen, prompt.size + maxNewTokens) // BLOCK_TOKENS), 1)
+        try:
+            out = np.zeros(prompt.size + maxNewTokens, np.int32)
+            if temperature <= 0:
+                n = C.c_int32()
+                B.check(self._lib.jgpt_generate_greedy(self.handle, pool.handle, prompt.ctypes.data, prompt.size, maxNewTokens,
+                                                       out.ctypes.data, C.byref(n)))
+                return out
+            rng = rng or np.random.default_rng()
+            out[: prompt.size] = prompt
+            seq = pool.seq_alloc()
+            try:
+                for t0 in range(0, prompt.size - 1, self.maxRows):  # all but the last prompt token, in portions
+                    self.step(pool, [seq], [prompt[t0:min(t0 + self.maxRows, prompt.size - 1)]], want_logits=False)
+                for j in range(maxNewTokens):
+                    at = prompt.size + j
+                    tok = self.forwardDecodeSampleBatch(pool, [seq], [out[at - 1]], [at - 1], temperature, topK, [rng.random()])[0]
+                    out[at] = tok
+                    if tok == 0:
+                        break
+            finally:
+                pool.seq_free(seq)
+            return out
+        finally:
+            if own:
+                pool.close()
+
+    def close(self):
+        if self.handle:
+            self._lib.jgpt_model_destroy(self.handle)
+            self.handle = 0
+
+
+class DecoderPool(KvPool):
+    """The paged store of a layered decoder: the allocator of ``KvPool`` over pages of the model's own geometry, plus a
+    slot of recurrent state per sequence."""
+
+    def __init__(self, model: DecoderModel, n_blocks, max_seqs, max_blocks_per_seq):
+        self.ctx, self._lib = model.ctx, model._lib
+        self.n_blocks, self.max_seqs, self.max_blocks_per_seq = n_blocks, max_seqs, max_blocks_per_seq
+        self.max_positions = max_blocks_per_seq * BLOCK_TOKENS
+        h = C.c_uint64()
+        B.check(self._lib.jgpt_decoder_new_pool(model.handle, n_blocks, max_seqs, max_blocks_per_seq, C.byref(h)))
+        self.handle = h.value
