@@ -585,6 +585,18 @@ def run_secondary(args, rank, world, local_rank):
         pool.close()
     elif args.workload == "fusedphases":
         line.update(W.run_fused_phases(ctx))
+    elif args.workload == "decoder":
+        from jgpt_b200 import decoder_bench
+
+        part = {"prefill": {"batches": ()}, "decode": {"prompts": ()}}.get(args.decoder_part, {})
+        widths = [int(w) for w in args.decoder_widths.split(",")]
+        if args.quick:  # one size, no comparison: what a profiler captures
+            part.update(gpt=False, repeats=1, steps=8)
+            if "batches" not in part:
+                part["batches"] = (args.batch,)
+            if "prompts" not in part:
+                part["prompts"] = ((8, 1024),)
+        line.update(decoder_bench.run_decoder(ctx, widths=widths, **part))
     elif args.workload == "steptimeline":
         line.update(W.run_step_timeline(ctx, batch=args.batch))
     elif args.workload == "contbatch":
@@ -629,8 +641,10 @@ def main():
     ap.add_argument("--per-layer", action="store_true", help="with --quick: one launch per layer instead of one per step")
     ap.add_argument("--launch-overlap", type=int, default=2, help="with --quick --per-layer: 0 ordinary launches, 1 / 2 overlapped")
     ap.add_argument("--batch", type=int, default=64, help="sequences per step for --workload decodestep")
+    ap.add_argument("--decoder-widths", default="1024,2048", help="model widths for --workload decoder")
+    ap.add_argument("--decoder-part", default="all", choices=["all", "prefill", "decode"], help="--workload decoder: what to run")
     ap.add_argument("--gather-depth", type=int, default=4, help="continuous batching: steps a rank may run ahead of the token-id gather")
-    ap.add_argument("--workload", default="microbench", choices=["microbench", "decode35m", "decodestep", "prefill", "contbatch", "longctx", "kvstore", "phases", "fusedphases", "steptimeline"],
+    ap.add_argument("--workload", default="microbench", choices=["microbench", "decode35m", "decodestep", "prefill", "contbatch", "longctx", "kvstore", "phases", "fusedphases", "steptimeline", "decoder"],
                     help="microbench (default) is the headline KV-append + decode-attention step; the others are the "
                          "remaining named configurations (reported, not the contract line)")
     args = ap.parse_args()

@@ -233,7 +233,7 @@ static int32_t small_dispatch(const Ctx *ctx, const Problem *p, int n, int pdl, 
 }
 
 int umma_min_rows() {
-    static const int v = env_int("JGPT_B200_NT_UMMA_MIN_ROWS", 0);
+    static const int v = env_int("JGPT_B200_NT_UMMA_MIN_ROWS", 129);
     return v;
 }
 

@@ -1,0 +1,150 @@
+"""Prefill and decode throughput of a layered decoder (the Somopel design with random weights) beside the fixed-block GPT
+model at equal width, depth, feed-forward size and vocabulary: ``bench.py --workload decoder``."""
+from __future__ import annotations
+
+import time
+
+import numpy as np
+
+from . import decoder as D
+from . import registry
+from .model import GPTModel
+from .runtime import Event
+
+VOCAB, LAYERS, MAX_POS = 32000, 6, 2304
+
+
+def somopel_config(width):
+    h = width // 128
+    par = {"type": "parallel", "mlp": {"kind": "dense", "ff": width * 11 // 4},
+           "mixer": {"left": {"heads": h, "kv_heads": max(h // 4, 1), "dim": 128, "vdim": 128, "mask": {"size": 512}, "scale": 128 ** -0.5},
+                     "right": {"heads": h, "dim": 64, "vdim": 128, "tau": 16.0}, "left_scale": 0.7, "right_scale": 0.9}}
+    delta = {"type": "channel_delta", "mlp": {"kind": "dense", "ff": width * 11 // 4},
+             "mixer": {"heads": h, "kv_heads": h, "dim": 128, "vdim": 128, "conv": 4}}
+    return {"architecture": "Somopel", "width": width, "vocab": VOCAB, "max_positions": MAX_POS, "norm": {"eps": 1e-5},
+            "layers": [delta, par, par] * (LAYERS // 3), "embedding": {"scale": 1.0}, "logit_scale": 0.5}
+
+
+def random_somopel(ctx, width, max_rows, rank=64):
+    cfg = somopel_config(width)
+    rng = np.random.default_rng(0)
+    shapes = {}
+
+    def lin(n, o, i):
+        shapes[n] = (o, i)
+
+    def vec(n, k):
+        shapes[n] = (k,)
+    for n in ("embed.norm", "embed.norm.b", "final.norm", "final.norm.b"):
+        vec(n, width)
+    lin("embed", VOCAB, width), lin("pos", MAX_POS, width)
+    for i, e in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", e["mixer"]
+        for n in ("norm1", "norm1.b", "norm2", "norm2.b"):
+            vec(p + n, width)
+        ff = e["mlp"]["ff"]
+        lin(p + "mlp.gate", ff, width), lin(p + "mlp.up", ff, width), lin(p + "mlp.down", width, ff)
+        if e["type"] == "parallel":
+            a, b = m["left"], m["right"]
+            for n, k in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"]), ("g", a["heads"])):
+                lin(p + "mix.left." + n, k, width)
+            lin(p + "mix.left.o", width, a["heads"] * a["vdim"])
+            q, hk, hv = p + "mix.right.", b["heads"] * b["dim"], b["heads"] * b["vdim"]
+            lin(q + "q", hk, width), lin(q + "k", hk, width), lin(q + "v", hv, width), lin(q + "g", hv, width), lin(q + "o", width, hv)
+            lin(q + "a1", rank, width), lin(q + "a2", hk, rank), vec(q + "a2.b", hk), vec(q + "norm", b["vdim"])
+        else:
+            q, H, G, dk, dv, t = p + "mix.", m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+            for n, k in (("q", G * dk), ("k", G * dk), ("v", H * dv)):
+                lin(q + n, k, width), lin(q + n + ".conv", k, t)
+            lin(q + "b", H, width), vec(q + "A_log", H), vec(q + "dt_bias", H * dk), lin(q + "o", width, H * dv)
+            lin(q + "a1", rank, width), lin(q + "a2", H * dk, rank), lin(q + "g1", rank, width), lin(q + "g2", H * dv, rank), vec(q + "norm", dv)
+    noise = rng.standard_normal(1 << 22, dtype=np.float32)
+
+    def get(n):  # slices of one noise block: making fresh numbers for every weight takes longer than the benchmark
+        s = shapes[n]
+        k = int(np.prod(s))
+        x = np.resize(noise[int(rng.integers(0, 1 << 20)):], k).reshape(s)
+        return x / np.sqrt(s[1]) if len(s) == 2 else 1 + 0.1 * x
+    model = D.DecoderModel(ctx, registry.describe(cfg, shapes.__getitem__), "bfloat16", max_rows)
+    model.loadTensors(get)
+    return model
+
+
+def random_gpt(ctx, width, max_rows):
+    """The fixed-block model of the same width, depth, feed-forward size and vocabulary (head size 16, its tuned case)."""
+    ff, L = width * 11 // 4, LAYERS
+    m = GPTModel(ctx, VOCAB, MAX_POS, width, width // 16, L, ff, maxRows=max_rows)
+    noise = np.random.default_rng(0).standard_normal(VOCAB * width, dtype=np.float32) * np.float32(width ** -0.5)
+    sizes = [VOCAB * width, MAX_POS * width]
+    for _ in range(L):
+        sizes += [width * width] * 4 + [width * ff] * 3 + [width] * 2
+    sizes += [width, VOCAB * width]
+    m.setParameters([np.ones(n, np.float32) if n == width else np.resize(noise, n) for n in sizes])
+    return m
+
+
+def _decode(ctx, model, batch, ctx_len, steps):
+    pool = model.newPool(batch * -(-(ctx_len + steps + 8) // 16), batch)
+    rng = np.random.default_rng(1)
+    seqs = [pool.seq_alloc() for _ in range(batch)]
+    toks, per = np.zeros(batch, np.int32), max(1, model.maxRows // ctx_len)
+    for i in range(0, batch, per):
+        ps = [rng.integers(1, VOCAB, ctx_len).astype(np.int32) for _ in seqs[i:i + per]]
+        if isinstance(model, GPTModel):
+            _, toks[i:i + per] = model.forwardPrefillBatch(pool, seqs[i:i + per], ps)
+        else:
+            ends = np.cumsum([len(p) for p in ps]) - 1
+            _, toks[i:i + per] = model.step(pool, seqs[i:i + per], ps, ends, want_logits=False, want_next=True)
+    lens, ids, ms = np.full(batch, ctx_len, np.int32), np.asarray(seqs, np.int32), []
+    for i in range(steps):
+        t0 = time.perf_counter()
+        _, toks = model.forwardDecodeBatch(pool, ids, toks, lens, lens, want_logits=False)
+        if i >= 4:
+            ms.append((time.perf_counter() - t0) * 1e3)
+        lens += 1
+    pool.close()
+    return float(np.median(ms))
+
+
+def _prefill(ctx, model, batch, seq_len, repeats):
+    pool = model.newPool(batch * -(-seq_len // 16), batch)
+    rng = np.random.default_rng(2)
+    ps = [rng.integers(1, VOCAB, seq_len).astype(np.int32) for _ in range(batch)]
+    seqs, best = [pool.seq_alloc() for _ in range(batch)], []
+    e0, e1 = Event(ctx), Event(ctx)
+    for i in range(repeats + 2):
+        for s in seqs:
+            pool.clear(s, zero_fill=False)
+        ctx.synchronize()
+        e0.record()
+        if isinstance(model, GPTModel):
+            model.forwardPrefillBatch(pool, seqs, ps)
+        else:
+            model.step(pool, seqs, ps, np.arange(1, batch + 1) * seq_len - 1, want_logits=False, want_next=True)
+        e1.record()
+        if i >= 2:
+            best.append(e0.elapsed_ms(e1))
+    pool.close()
+    return float(np.median(best))
+
+
+def run_decoder(ctx, widths=(1024, 2048), batches=(1, 16, 64), prompts=((1, 2048), (8, 1024)), ctx_len=1024, steps=24, repeats=5, gpt=True):
+    out = {"workload": f"{LAYERS} layers, vocabulary {VOCAB}, random weights; prefill = prompts of one call, decode at context {ctx_len}+",
+           "timing": "prefill: CUDA events around the call; decode: host clock around a step that reads its ids back; medians", "sizes": []}
+    for w in widths:
+        row = {"width": w}
+        for name, make in (("somopel", random_somopel), ("gpt", random_gpt)):
+            if name == "gpt" and not gpt:
+                continue
+            m = make(ctx, w, 8192)
+            r = {}
+            for b, n in prompts:
+                ms = _prefill(ctx, m, b, n, repeats)
+                r[f"prefill_{b}x{n}"] = {"ms": ms, "tokens_per_s": b * n / ms * 1e3}
+            for b in batches:
+                ms = _decode(ctx, m, b, ctx_len, steps)
+                r[f"decode_b{b}"] = {"ms": ms, "tokens_per_s": b / ms * 1e3}
+            row[name] = r
+            m.close()
+        out["sizes"].append(row)
+    return out
