@@ -58,8 +58,7 @@ struct Decoder {
     uint64_t state_stride = 0;
     std::vector<void *> allocs;
     // workspace
-    float *x = nullptr, *raw = nullptr, *logits = nullptr, *partials = nullptr;
-    uint64_t partial_floats = 0;
+    float *x = nullptr, *raw = nullptr, *logits = nullptr;
     void *h = nullptr, *proj = nullptr, *z = nullptr, *mixed = nullptr, *act = nullptr;
     int *d_desc = nullptr, *h_desc = nullptr;
     int *d_next = nullptr, *h_next = nullptr;
@@ -201,7 +200,6 @@ static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
         n_in = std::max(n_in, y.n_in), n_z = std::max(n_z, y.n_z), n_out = std::max(n_out, y.n_out), ffp = std::max(ffp, y.ffp);
         for (const DBranch &b : y.br) {
             if (b.s.kind != JGPT_MIX_ATTENTION) raw = std::max(raw, b.s.heads * b.DV);
-            else d->partial_floats = std::max(d->partial_floats, mix::attn_partial_floats(d->R, b.s.heads, b.D));
         }
     }
     TRY(dalloc(d, &d->embed, (uint64_t)d->s.vocab * d->ldw * eb));
@@ -209,7 +207,6 @@ static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
     for (float **p : {&d->enw, &d->enb, &d->fnw, &d->fnb}) TRY(dalloc(d, (void **)p, sizeof(float) * W));
     TRY(dalloc(d, (void **)&d->x, sizeof(float) * R * W));
     TRY(dalloc(d, (void **)&d->raw, sizeof(float) * R * raw));
-    TRY(dalloc(d, (void **)&d->partials, sizeof(float) * d->partial_floats));
     TRY(dalloc(d, &d->h, R * d->ldw * eb));
     TRY(dalloc(d, &d->proj, R * n_in * eb));
     TRY(dalloc(d, &d->z, R * n_z * eb));
@@ -406,7 +403,7 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, uint
                 a.proj = d->proj, a.ldp = y.n_in, a.q_off = b.q, a.k_off = b.k, a.v_off = b.v, a.g_off = b.g;
                 a.heads = b.s.heads, a.kv_heads = b.s.kv_heads, a.D = b.D, a.chunk = b.s.chunk, a.scale = b.s.score_scale, a.out_scale = b.s.out_scale;
                 a.kv = p->vkv + p->vlayers[(size_t)b.kv_layer].offset, a.table = p->d_table, a.n_blocks = p->n_blocks, a.mbs = p->max_blocks_per_seq;
-                a.out = d->mixed, a.ldo = y.n_out, a.out_off = b.out, a.partials = d->partials, a.partial_floats = d->partial_floats;
+                a.out = d->mixed, a.ldo = y.n_out, a.out_off = b.out;
                 a.sm_count = d->ctx->sm_count, a.status = status;
                 TRY(mix::launch_attention(d->f32, sd, a, 0, st));
             } else {

@@ -51,15 +51,12 @@ struct AttnArgs {
     int n_blocks, mbs;
     void *out;          // [rows, ldo], head h at out_off + h * D
     int ldo, out_off;
-    float *partials;    // split-sequence scratch of single-token attention
-    uint64_t partial_floats;
     int sm_count;
     int *status;
 };
 int32_t launch_attention(bool f32, const StepDesc &d, const AttnArgs &a, int pdl, cudaStream_t st);
 int attn_padded_head(int dim, int vdim);          // 0: not supported
 int attn_query_tile(int heads, int kv_heads);     // tokens per query tile of the multi-token kernel
-uint64_t attn_partial_floats(int rows, int heads, int D);
 
 // ---- recurrent.cu ----------------------------------------------------------------------------------
 enum RecKind : int { REC_GLA = 0, REC_DELTA = 1 };
