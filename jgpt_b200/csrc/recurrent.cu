@@ -18,6 +18,7 @@
 #include "mixers.cuh"
 
 #include <algorithm>
+#include <type_traits>
 
 #include "ptx.cuh"
 
@@ -58,7 +59,15 @@ __device__ __forceinline__ void store2(float *p, float2 v) { *reinterpret_cast<f
 __device__ __forceinline__ void store1(__nv_bfloat16 *p, float v) { *p = __float2bfloat16(v); }
 __device__ __forceinline__ void store1(float *p, float v) { *p = v; }
 
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+// exp for the bf16 mode is the fast one (relative error ~2^-21 on the ranges used here), the exact mode takes expf.
+template <class AT>
+__device__ __forceinline__ float exp_f(float x) {
+    return sizeof(AT) == 4 ? expf(x) : __expf(x);
+}
+template <class AT>
+__device__ __forceinline__ float sigmoid_f(float x) {
+    return sizeof(AT) == 4 ? 1.f / (1.f + expf(-x)) : __fdividef(1.f, 1.f + __expf(-x));
+}
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -86,8 +95,12 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rl = lane >> 2, cl = lane & 3;
     const int nthreads = blockDim.x, nw = nthreads >> 5, DVc = nw * 16;
     const int h = blockIdx.x % a.heads, split = blockIdx.x / a.heads, col0 = split * DVc;
+    constexpr int E = 16 / sizeof(AT);  // elements of a 16-byte chunk
+    // a token's raw row: q, k, v, decay logits, output gate, then (delta) the chunk that holds its step size
+    const int RW = 3 * DK + 2 * DVc + (KIND == REC_DELTA ? E : 0), RK = DK, RV = 2 * DK, RZ = RV + DVc, RG = RZ + DK, RB = RG + DVc;
     float *sq = rec_smem, *sk = sq + tt * DK, *sg = sk + tt * DK, *sv = sg + tt * DK, *so = sv + tt * DVc, *sbeta = so + tt * DVc,
           *sqk = sbeta + tt;
+    AT *raw_s = reinterpret_cast<AT *>(sqk + tt);  // [2][tt][RW]; one stage is enough for a single token
 
     if (pdl & 2) griddep_launch_dependents();
     const Seg sgm = segs[blockIdx.y];
@@ -123,55 +136,80 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
         if (sgm.pos0 + t >= 0) return load2(hist + (size_t)(-1 - t) * channels + channel);
         return make_float2(0.f, 0.f);
     };
-    // channel pair idx of this CTA: q, then k, then its value columns
-    auto locate = [&](int idx, int &proj_col, int &channel, float *&dst, int &ld, const float *&w) {
-        if (idx < DK / 2) {
-            const int c = kvh * DK + 2 * idx;
-            proj_col = a.q_off + c, channel = c, dst = sq + 2 * idx, ld = DK, w = a.conv_q + (size_t)c * a.taps;
-        } else if (idx < DK) {
-            const int c = kvh * DK + 2 * idx - DK;
-            proj_col = a.k_off + c, channel = nq + c, dst = sk + 2 * idx - DK, ld = DK, w = a.conv_k + (size_t)c * a.taps;
+    // channel pair idx of this CTA (q, then k, then its value columns): column in proj, convolution channel
+    auto locate = [&](int idx, int &proj_col, int &channel) {
+        if (idx < DK) {
+            const bool is_k = idx >= DK / 2;
+            const int c = kvh * DK + 2 * idx - (is_k ? DK : 0);
+            proj_col = (is_k ? a.k_off : a.q_off) + c, channel = (is_k ? nq : 0) + c;
         } else {
-            const int j = 2 * (idx - DK), c = h * a.DV + col0 + j;
-            proj_col = a.v_off + c, channel = 2 * nq + c, dst = sv + j, ld = DVc, w = a.conv_v + (size_t)c * a.taps;
+            const int c = h * a.DV + col0 + 2 * (idx - DK);
+            proj_col = a.v_off + c, channel = 2 * nq + c;
         }
     };
     const int npairs = DK + DVc / 2;
-
-    for (int t0 = 0; t0 < sgm.T; t0 += tt) {
+    // raw rows of a tile into stage `buf`
+    auto stage = [&](int buf, int t0) {
+        const int tn = min(tt, sgm.T - t0), per = RW / E;
+        for (int e = tid; e < tn * per; e += nthreads) {
+            const int t = e / per, c = (e % per) * E;
+            const AT *row = proj + (size_t)(t0 + t) * a.ldp, *zr = z + (size_t)(t0 + t) * a.ldz, *src;
+            if (c < RK) src = row + a.q_off + kvh * DK + c;
+            else if (c < RV) src = row + a.k_off + kvh * DK + c - RK;
+            else if (c < RZ) src = row + a.v_off + h * a.DV + col0 + c - RV;
+            else if (c < RG) src = zr + a.z_off + h * DK + c - RZ;
+            else if (c < RB) src = (KIND == REC_DELTA ? zr + a.zg_off : row + a.g_off) + h * a.DV + col0 + c - RG;
+            else src = row + a.b_off + h / E * E;
+            cp_async16(raw_s + ((size_t)buf * tt + t) * RW + c, src, true);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    // convolution + silu of one channel pair over the tile
+    auto convolve = [&](auto max_taps, int idx, const AT *raw, const AT *prev, int t0, int tn, float *dst, int ld) {
+        constexpr int MT = decltype(max_taps)::value;
+        int pc, ch;
+        locate(idx, pc, ch);
+        const float *w = (ch < nq ? a.conv_q + (size_t)ch * a.taps
+                                  : (ch < 2 * nq ? a.conv_k + (size_t)(ch - nq) * a.taps : a.conv_v + (size_t)(ch - 2 * nq) * a.taps));
+        float2 wt[MT], win[MT];  // right-aligned: entry MT - 1 is the current token's
+#pragma unroll
+        for (int i = 0; i < MT; i++) {
+            const int back = MT - 1 - i;
+            const bool on = back < a.taps;
+            wt[i] = on ? make_float2(w[a.taps - 1 - back], w[2 * a.taps - 1 - back]) : make_float2(0.f, 0.f);
+            // the window in front of the tile's first token: entry i holds token t0 - back
+            win[i] = !on || back == 0 ? make_float2(0.f, 0.f) : (t0 > 0 ? load2(prev + (size_t)(tt - back) * RW + 2 * idx) : conv_input(-back, pc, ch));
+        }
+#pragma unroll 4
+        for (int t = 0; t < tn; t++) {
+            win[MT - 1] = load2(raw + (size_t)t * RW + 2 * idx);
+            float2 y = make_float2(0.f, 0.f);
+#pragma unroll
+            for (int i = 0; i < MT; i++) y.x = fmaf(wt[i].x, win[i].x, y.x), y.y = fmaf(wt[i].y, win[i].y, y.y);
+            y.x *= sigmoid_f<AT>(y.x), y.y *= sigmoid_f<AT>(y.y);
+            *reinterpret_cast<float2 *>(dst + t * ld) = y;
+#pragma unroll
+            for (int i = 0; i + 1 < MT; i++) win[i] = win[i + 1];
+        }
+    };
+    stage(0, 0);
+    for (int t0 = 0, buf = 0; t0 < sgm.T; t0 += tt, buf ^= 1) {
         const int tn = min(tt, sgm.T - t0);
+        const AT *raw = raw_s + (size_t)buf * tt * RW, *prev = raw_s + (size_t)(buf ^ 1) * tt * RW;
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
         // ---- prepare the tile ----
         for (int idx = tid; idx < npairs; idx += nthreads) {
-            int pc, ch, ld;
-            float *dst;
-            const float *w;
-            locate(idx, pc, ch, dst, ld, w);
+            float *dst = idx < DK / 2 ? sq + 2 * idx : (idx < DK ? sk + 2 * idx - DK : sv + 2 * (idx - DK));
+            const int ld = idx < DK ? DK : DVc;
             if (KIND == REC_DELTA) {
-                float2 wt[kMaxTaps], win[kMaxTaps];  // right-aligned: entry kMaxTaps - 1 is the current token's
-#pragma unroll
-                for (int i = 0; i < kMaxTaps; i++) {
-                    const int back = kMaxTaps - 1 - i;
-                    const bool on = back < a.taps;
-                    wt[i] = on ? make_float2(w[a.taps - 1 - back], w[2 * a.taps - 1 - back]) : make_float2(0.f, 0.f);
-                    // the window in front of the tile's first token: entry i holds token t0 - back
-                    win[i] = on && back > 0 ? conv_input(t0 - back, pc, ch) : make_float2(0.f, 0.f);
-                }
-#pragma unroll 4
-                for (int t = 0; t < tn; t++) {
-                    win[kMaxTaps - 1] = load2(proj + (size_t)(t0 + t) * a.ldp + pc);
-                    float2 y = make_float2(0.f, 0.f);
-#pragma unroll
-                    for (int i = 0; i < kMaxTaps; i++) y.x = fmaf(wt[i].x, win[i].x, y.x), y.y = fmaf(wt[i].y, win[i].y, y.y);
-                    y.x *= sigmoid_f(y.x), y.y *= sigmoid_f(y.y);
-                    *reinterpret_cast<float2 *>(dst + t * ld) = y;
-#pragma unroll
-                    for (int i = 0; i + 1 < kMaxTaps; i++) win[i] = win[i + 1];
-                }
+                if (a.taps <= 4) convolve(std::integral_constant<int, 4>(), idx, raw, prev, t0, tn, dst, ld);
+                else convolve(std::integral_constant<int, kMaxTaps>(), idx, raw, prev, t0, tn, dst, ld);
             } else {
                 const float f = idx < DK / 2 ? qscale : 1.f;
 #pragma unroll 4
                 for (int t = 0; t < tn; t++) {
-                    float2 y = load2(proj + (size_t)(t0 + t) * a.ldp + pc);
+                    float2 y = load2(raw + (size_t)t * RW + 2 * idx);
                     y.x *= f, y.y *= f;
                     *reinterpret_cast<float2 *>(dst + t * ld) = y;
                 }
@@ -180,16 +218,17 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
         }
         for (int idx = tid; idx < tn * (DK / 2); idx += nthreads) {
             const int t = idx / (DK / 2), c = 2 * (idx % (DK / 2));
-            float2 y = load2(z + (size_t)(t0 + t) * a.ldz + a.z_off + h * DK + c);
+            float2 y = load2(raw + (size_t)t * RW + RZ + c);
             const float2 b = *reinterpret_cast<const float2 *>(a.decay_bias + h * DK + c);
             y.x += b.x, y.y += b.y;
-            if (KIND == REC_DELTA) y.x = expf(-rate * softplus_f(y.x)), y.y = expf(-rate * softplus_f(y.y));
-            else y.x = expf(-rate * softplus_f(-y.x)), y.y = expf(-rate * softplus_f(-y.y));  // sigmoid(z)^(1 / tau)
+            if (KIND == REC_GLA) y.x = -y.x, y.y = -y.y;  // sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau)
+            y.x = exp_f<AT>(-rate * softplus_f(y.x)), y.y = exp_f<AT>(-rate * softplus_f(y.y));
             *reinterpret_cast<float2 *>(sg + t * DK + c) = y;
         }
         if (KIND == REC_GLA && (tn & 1))
             for (int c = tid; c < DK; c += nthreads) sg[tn * DK + c] = 1.f;
         __syncthreads();
+        if (t0 + tt < sgm.T) stage(buf ^ 1, t0 + tt);  // lands while this tile runs; the previous tile's rows are no longer needed
         if (KIND == REC_DELTA) {
             for (int t = warp; t < tn; t += nw) {
                 float qv[NI], kv[NI], qq = 0.f, kk = 0.f, qk = 0.f;
@@ -202,7 +241,7 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
                 const float fq = qscale / sqrtf(qq + 1e-6f), fk = 1.f / sqrtf(kk + 1e-6f);
 #pragma unroll
                 for (int i = 0; i < NI; i++) sq[t * DK + lane + 32 * i] = qv[i] * fq, sk[t * DK + lane + 32 * i] = kv[i] * fk;
-                if (lane == 0) sqk[t] = qk * fq * fk, sbeta[t] = sigmoid_f(load1(proj + (size_t)(t0 + t) * a.ldp + a.b_off + h));
+                if (lane == 0) sqk[t] = qk * fq * fk, sbeta[t] = sigmoid_f<AT>(load1(raw + (size_t)t * RW + RB + h % E));
             }
             __syncthreads();
         }
@@ -300,10 +339,9 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
                 }
                 const float inv = a.out_scale / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
                 AT *o = reinterpret_cast<AT *>(a.out) + (size_t)(sgm.row0 + t0 + t) * a.ldo + a.out_off + h * DVc;
-                const AT *gp = KIND == REC_DELTA ? z + (size_t)(t0 + t) * a.ldz + a.zg_off + h * DVc
-                                                 : proj + (size_t)(t0 + t) * a.ldp + a.g_off + h * DVc;
+                const AT *gp = raw + (size_t)t * RW + RG;
                 for (int c = lane; c < DVc; c += 32) {
-                    const float gt = load1(gp + c), sgt = sigmoid_f(gt);
+                    const float gt = load1(gp + c), sgt = sigmoid_f<AT>(gt);
                     store1(o + c, so[t * DVc + c] * inv * a.norm_w[c] * (KIND == REC_DELTA ? sgt : gt * sgt));
                 }
             }
@@ -322,10 +360,8 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
         const bool first_of_group = h % (a.heads / a.kv_heads) == 0 && split == 0;
         for (int idx = tid; idx < npairs; idx += nthreads) {
             if (idx < DK && !first_of_group) continue;  // shared channels are written once
-            int pc, ch, ld;
-            float *dst;
-            const float *w;
-            locate(idx, pc, ch, dst, ld, w);
+            int pc, ch;
+            locate(idx, pc, ch);
             for (int i = 0; i < a.taps - 1; i++) store2(next + (size_t)i * channels + ch, conv_input(sgm.T - 1 - i, pc, ch));
         }
     }
@@ -345,7 +381,7 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const RecArgs a, int ro
     const AT *gp = KIND == REC_DELTA ? reinterpret_cast<const AT *>(a.z) + (size_t)r * a.ldz + a.zg_off + h * a.DV
                                      : reinterpret_cast<const AT *>(a.proj) + (size_t)r * a.ldp + a.g_off + h * a.DV;
     for (int c = lane; c < a.DV; c += 32) {
-        const float gt = load1(gp + c), sgt = sigmoid_f(gt);
+        const float gt = load1(gp + c), sgt = sigmoid_f<AT>(gt);
         store1(o + c, raw[c] * inv * a.norm_w[c] * (KIND == REC_DELTA ? sgt : gt * sgt));
     }
 }
@@ -377,13 +413,17 @@ static int32_t rec_launch(const StepDesc &d, const RecArgs &a, int pdl, cudaStre
     if (!single)
         while (a.heads * d.n_segs * split * 2 <= a.sm_count && groups / split >= 4 && allowed(split * 2)) split *= 2;
     const int nw = groups / split, DVc = nw * 16;
-    const size_t smem = sizeof(float) * ((size_t)tt * (3 * DK + 2 * DVc) + 2 * tt);
+    auto smem_bytes = [](int tokens, int cols, int stages) {
+        const size_t row = 3 * DK + 2 * (size_t)cols;
+        return sizeof(float) * ((size_t)tokens * row + 2 * tokens) + (size_t)stages * tokens * (row * sizeof(AT) + (KIND == REC_DELTA ? 16 : 0));
+    };
+    const size_t smem = smem_bytes(tt, DVc, single ? 1 : 2);
     auto kern = recurrent_kernel<AT, KIND, DK>;
     static thread_local int set_for = -1;
     int dev = 0;
     JGPT_CUDA_TRY(cudaGetDevice(&dev));
     if (set_for != dev) {
-        JGPT_CUDA_TRY(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(float) * (kTileTokens * (3 * DK + 2 * 256) + 2 * kTileTokens))));
+        JGPT_CUDA_TRY(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_bytes(kTileTokens, 16 * max_groups, 2)));
         set_for = dev;
     }
     cudaLaunchConfig_t cfg = {};
