@@ -58,11 +58,13 @@ struct Decoder {
     uint64_t state_stride = 0;
     std::vector<void *> allocs;
     // workspace
-    float *x = nullptr, *raw = nullptr, *logits = nullptr;
+    float *x = nullptr, *raw = nullptr, *chunk_ws = nullptr, *logits = nullptr;
     void *h = nullptr, *proj = nullptr, *z = nullptr, *mixed = nullptr, *act = nullptr;
     int *d_desc = nullptr, *h_desc = nullptr;
     int *d_next = nullptr, *h_next = nullptr;
     float *d_u = nullptr, *h_u = nullptr, *samp = nullptr;
+    uint64_t chunk_ws_floats = 0;
+    int long_min = 0;  // entries of at least this many tokens run their recurrences in chunks (0: none)
     int logit_rows = 0;
     float *capture = nullptr;  // host, [layers][rows][width] of the next step
     uint64_t capture_floats = 0;
@@ -188,18 +190,23 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
     return JGPT_OK;
 }
 
-static size_t desc_ints(const Decoder *d) { return 14 * (size_t)d->R + 64; }
+static size_t desc_ints(const Decoder *d) { return 18 * (size_t)d->R + 64; }
 
 static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
     const uint64_t R = d->R, W = d->s.width, eb = d->eb;
     d->L.resize((size_t)d->s.n_layers);
+    d->long_min = mix::rec_chunk_min_tokens(d->f32);
     int n_in = 8, n_z = 8, n_out = 8, ffp = 16, raw = 0;
     for (int i = 0; i < d->s.n_layers; i++) {
         DLayer &y = d->L[(size_t)i];
         TRY(plan_layer(d, y, layers[i], i));
         n_in = std::max(n_in, y.n_in), n_z = std::max(n_z, y.n_z), n_out = std::max(n_out, y.n_out), ffp = std::max(ffp, y.ffp);
         for (const DBranch &b : y.br) {
-            if (b.s.kind != JGPT_MIX_ATTENTION) raw = std::max(raw, b.s.heads * b.DV);
+            if (b.s.kind == JGPT_MIX_ATTENTION) continue;
+            raw = std::max(raw, b.s.heads * b.DV);
+            if (const int t = d->long_min)
+                d->chunk_ws_floats = std::max(d->chunk_ws_floats, (uint64_t)(d->R / mix::kRecChunk + d->R / t + 1) * b.s.heads *
+                                                                      mix::rec_chunk_record_floats(rec_args(b).kind, b.DK, b.DV));
         }
     }
     TRY(dalloc(d, &d->embed, (uint64_t)d->s.vocab * d->ldw * eb));
@@ -207,6 +214,7 @@ static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
     for (float **p : {&d->enw, &d->enb, &d->fnw, &d->fnb}) TRY(dalloc(d, (void **)p, sizeof(float) * W));
     TRY(dalloc(d, (void **)&d->x, sizeof(float) * R * W));
     TRY(dalloc(d, (void **)&d->raw, sizeof(float) * R * raw));
+    TRY(dalloc(d, (void **)&d->chunk_ws, sizeof(float) * d->chunk_ws_floats));
     TRY(dalloc(d, &d->h, R * d->ldw * eb));
     TRY(dalloc(d, &d->proj, R * n_in * eb));
     TRY(dalloc(d, &d->z, R * n_z * eb));
@@ -417,7 +425,7 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, uint
                 mix::RecArgs a = rec_args(b);
                 a.proj = d->proj, a.ldp = y.n_in, a.z = d->z, a.ldz = y.n_z, a.eps = eps;
                 a.state = p->state + b.state_off, a.state_stride = p->state_stride, a.max_seqs = p->max_seqs;
-                a.out = d->mixed, a.ldo = y.n_out, a.raw = d->raw, a.sm_count = d->ctx->sm_count, a.status = status;
+                a.out = d->mixed, a.ldo = y.n_out, a.raw = d->raw, a.chunk_ws = d->chunk_ws, a.chunk_ws_floats = d->chunk_ws_floats, a.sm_count = d->ctx->sm_count, a.status = status;
                 TRY(mix::launch_recurrent(d->f32, sd, a, 0, st));
             }
         }
@@ -491,8 +499,9 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
         return o;
     };
     const size_t o_tok = take((size_t)rows), o_pos = take((size_t)rows), o_seq = take((size_t)rows), o_seg = take(6 * (size_t)c.n);
-    const size_t o_single = take((size_t)c.n), o_want = take((size_t)c.n_want), o_tile = at;
-    int max_len = 0;
+    const size_t o_single = take((size_t)c.n), o_short = take((size_t)c.n), o_want = take((size_t)c.n_want), o_long = take(2 * (size_t)c.n);
+    int max_len = 0, n_short = 0, n_long = 0, n_chunks = 0;
+    const int long_min = d->long_min;
     mix::Seg *segs = reinterpret_cast<mix::Seg *>(hd + o_seg);
     for (int i = 0; i < c.n; i++) {
         const int s = c.seq_ids[i], r0 = c.starts[i], T = c.starts[i + 1] - r0;
@@ -501,8 +510,18 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
         max_len = std::max(max_len, ss.len + T);
         for (int t = 0; t < T; t++) hd[o_tok + r0 + t] = c.ids[r0 + t], hd[o_pos + r0 + t] = ss.len + t, hd[o_seq + r0 + t] = s;
         if (T == 1) hd[o_single + n_single++] = i;
+        if (long_min == 0 || T < long_min) hd[o_short + n_short++] = i;
+        else {
+            hd[o_long + 2 * n_long] = i, hd[o_long + 2 * n_long + 1] = n_chunks, n_long++;
+            n_chunks += (T + mix::kRecChunk - 1) / mix::kRecChunk;
+        }
     }
     for (int i = 0; i < c.n_want; i++) hd[o_want + i] = c.want[i];
+    const size_t o_chunk = take(2 * (size_t)n_chunks), o_tile = at;
+    for (int l = 0, k = 0; l < n_long; l++) {
+        const int i = hd[o_long + 2 * l], T = c.starts[i + 1] - c.starts[i];
+        for (int t = 0; t < T; t += mix::kRecChunk, k++) hd[o_chunk + 2 * k] = i, hd[o_chunk + 2 * k + 1] = t;
+    }
     // query tiles: the same list serves every layer, so tiles hold as many tokens as the layer with the largest groups allows
     int qt = 64;
     for (const DLayer &y : d->L)
@@ -523,6 +542,8 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
     sd.tiles = reinterpret_cast<const int2 *>(dd + o_tile), sd.singles = dd + o_single, sd.want = dd + o_want;
     sd.rows = rows, sd.n_segs = c.n, sd.n_tiles = n_tiles, sd.n_singles = n_single, sd.n_want = c.n_want, sd.max_len = max_len;
     sd.qt = qt;
+    sd.short_segs = dd + o_short, sd.long_segs = reinterpret_cast<const int2 *>(dd + o_long), sd.chunks = reinterpret_cast<const int2 *>(dd + o_chunk);
+    sd.n_short = n_short, sd.n_long = n_long, sd.n_chunks = n_chunks;
 
     uint64_t cap_rows = 0;
     if (d->capture) {

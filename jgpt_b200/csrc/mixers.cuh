@@ -21,8 +21,11 @@ struct StepDesc {
     const Seg *segs;
     const int2 *tiles;           // (entry, first token) of every query tile of the entries with more than one token
     const int *singles;          // entries with one token
+    const int *short_segs;       // entries whose recurrences run token by token
+    const int2 *long_segs;       // the others: (entry, index of its first chunk)
+    const int2 *chunks;          // (entry, first token) of the long entries' chunks of kRecChunk tokens
     const int *want;             // rows whose logits are wanted
-    int rows, n_segs, n_tiles, n_singles, n_want;
+    int rows, n_segs, n_tiles, n_singles, n_short, n_long, n_chunks, n_want;
     int qt;                      // tokens per query tile
     int max_len;                 // upper bound of pos0 + T (sizes the split of single-token attention)
 };
@@ -81,9 +84,15 @@ struct RecArgs {
     void *out;          // [rows, ldo]
     int ldo, out_off;
     float *raw;         // [rows, heads * DV] scratch for heads whose columns are cut over several CTAs
+    float *chunk_ws;    // records of the chunked form
+    uint64_t chunk_ws_floats;
     int sm_count;
     int *status;
 };
+constexpr int kRecChunk = 16;
+int rec_chunk_min_tokens(bool f32);  // entries of at least this many tokens take the chunked form (0: none)
+uint64_t rec_chunk_record_floats(int kind, int DK, int DV);
+int32_t launch_recurrent_chunks(bool f32, const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st);
 int32_t launch_recurrent(bool f32, const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st);
 int rec_padded_key(int dim);    // 0: not supported
 int rec_padded_value(int vdim);

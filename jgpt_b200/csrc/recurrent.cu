@@ -1,5 +1,5 @@
-// Recurrent mixers of the layered decoder: gated linear attention and the gated delta rule, both with a decay per key
-// channel, as ONE kernel from the layer's projections to the gated, normalised head outputs - for prompts, portions of
+// Recurrent mixers of the layered decoder, token by token: gated linear attention and the gated delta rule, both with a
+// decay per key channel (long entries of a bf16 step take the chunked form, recurrent_chunk.cu), as ONE kernel from the layer's projections to the gated, normalised head outputs - for prompts, portions of
 // prompts and single tokens alike, so a token's arithmetic does not depend on how its sequence was cut.
 //
 //   GLA    S <- diag(a) S + k v^T;                       o = S^T q
@@ -15,17 +15,14 @@
 // [2][taps - 1][channels] of projection outputs.  The history has two copies: a step reads the one its entry names and
 // writes the other, because heads that share query / key channels run in different CTAs.  Nothing is cleared when a slot
 // is handed out: a step that starts at position 0 starts from zeros.
-#include "mixers.cuh"
+#include "recurrent_math.cuh"
 
 #include <algorithm>
 #include <type_traits>
 
-#include "ptx.cuh"
-
 namespace jgpt {
 namespace mix {
 
-constexpr int kMaxTaps = 8;
 constexpr int kTileTokens = 16;
 
 typedef unsigned long long u64;
@@ -50,31 +47,6 @@ __device__ __forceinline__ u64 mul2(u64 a, u64 b) {
     return r;
 }
 
-__device__ __forceinline__ float2 load2(const __nv_bfloat16 *p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(p)); }
-__device__ __forceinline__ float2 load2(const float *p) { return *reinterpret_cast<const float2 *>(p); }
-__device__ __forceinline__ float load1(const __nv_bfloat16 *p) { return __bfloat162float(*p); }
-__device__ __forceinline__ float load1(const float *p) { return *p; }
-__device__ __forceinline__ void store2(__nv_bfloat16 *p, float2 v) { *reinterpret_cast<__nv_bfloat162 *>(p) = __float22bfloat162_rn(v); }
-__device__ __forceinline__ void store2(float *p, float2 v) { *reinterpret_cast<float2 *>(p) = v; }
-__device__ __forceinline__ void store1(__nv_bfloat16 *p, float v) { *p = __float2bfloat16(v); }
-__device__ __forceinline__ void store1(float *p, float v) { *p = v; }
-
-// exp for the bf16 mode is the fast one (relative error ~2^-21 on the ranges used here), the exact mode takes expf.
-template <class AT>
-__device__ __forceinline__ float exp_f(float x) {
-    return sizeof(AT) == 4 ? expf(x) : __expf(x);
-}
-template <class AT>
-__device__ __forceinline__ float sigmoid_f(float x) {
-    return sizeof(AT) == 4 ? 1.f / (1.f + expf(-x)) : __fdividef(1.f, 1.f + __expf(-x));
-}
-__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-    for (int off = 16; off >= 1; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
-    return v;
-}
-
 // Eight sums over the eight row lanes (lane bits 2-4): on return a lane holds the total of value 4 * bit4 + 2 * bit3 + bit2.
 __device__ __forceinline__ float reduce8(const float (&lo)[4], const float (&hi)[4], int lane) {
     const bool b4 = lane & 16, b3 = lane & 8, b2 = lane & 4;
@@ -88,7 +60,8 @@ __device__ __forceinline__ float reduce8(const float (&lo)[4], const float (&hi)
 }
 
 template <class AT, int KIND, int DK>
-__global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const RecArgs a, const Seg *__restrict__ segs, int col_split, int tt,
+__global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const RecArgs a, const Seg *__restrict__ segs, const int *__restrict__ list,
+                                                                          int col_split, int tt,
                                                                           int pdl) {
     constexpr int NI = DK / 32;  // groups of four rows per lane
     extern __shared__ __align__(16) float rec_smem[];
@@ -103,7 +76,7 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
     AT *raw_s = reinterpret_cast<AT *>(sqk + tt);  // [2][tt][RW]; one stage is enough for a single token
 
     if (pdl & 2) griddep_launch_dependents();
-    const Seg sgm = segs[blockIdx.y];
+    const Seg sgm = segs[list[blockIdx.y]];
     if (sgm.seq < 0 || sgm.seq >= a.max_seqs) {
         if (tid == 0) atomicOr(a.status, DEV_STATUS_BAD_SEQ);
         return;
@@ -372,18 +345,7 @@ template <class AT, int KIND>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const RecArgs a, int rows) {
     const int item = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (item >= rows * a.heads) return;
-    const int r = item / a.heads, h = item % a.heads;
-    const float *raw = a.raw + (size_t)r * a.heads * a.DV + h * a.DV;
-    float ss = 0.f;
-    for (int c = lane; c < a.DV; c += 32) ss += raw[c] * raw[c];
-    const float inv = a.out_scale / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
-    AT *o = reinterpret_cast<AT *>(a.out) + (size_t)r * a.ldo + a.out_off + h * a.DV;
-    const AT *gp = KIND == REC_DELTA ? reinterpret_cast<const AT *>(a.z) + (size_t)r * a.ldz + a.zg_off + h * a.DV
-                                     : reinterpret_cast<const AT *>(a.proj) + (size_t)r * a.ldp + a.g_off + h * a.DV;
-    for (int c = lane; c < a.DV; c += 32) {
-        const float gt = load1(gp + c), sgt = sigmoid_f<AT>(gt);
-        store1(o + c, raw[c] * inv * a.norm_w[c] * (KIND == REC_DELTA ? sgt : gt * sgt));
-    }
+    norm_gate_head<AT, KIND>(a, item / a.heads, item % a.heads, lane);
 }
 
 int rec_padded_key(int dim) {
@@ -402,16 +364,15 @@ uint64_t rec_state_bytes(const RecArgs &a, int elem_bytes, uint64_t *conv_off) {
 }
 
 template <class AT, int KIND, int DK>
-static int32_t rec_launch(const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st) {
+static int32_t rec_launch(const StepDesc &d, const RecArgs &a, int pdl, int *split_out, cudaStream_t st) {
     const bool single = d.n_tiles == 0;
+    if (d.n_short == 0) return JGPT_OK;
     const int tt = single ? 2 : kTileTokens;
     const int groups = a.DV / 16, max_groups = DK <= 128 ? 16 : 8;
     int split = 1;
     auto allowed = [&](int s) { return groups % s == 0; };
     while (split < groups && (!allowed(split) || groups / split > max_groups)) split++;
-    // a few long entries: more CTAs per head (each prepares the tile's q, k again) and a norm kernel behind them
-    if (!single)
-        while (a.heads * d.n_segs * split * 2 <= a.sm_count && groups / split >= 4 && allowed(split * 2)) split *= 2;
+    *split_out = split;
     const int nw = groups / split, DVc = nw * 16;
     auto smem_bytes = [](int tokens, int cols, int stages) {
         const size_t row = 3 * DK + 2 * (size_t)cols;
@@ -430,33 +391,38 @@ static int32_t rec_launch(const StepDesc &d, const RecArgs &a, int pdl, cudaStre
     cudaLaunchAttribute attr[1];
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
     attr[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.gridDim = dim3((unsigned)(a.heads * split), (unsigned)d.n_segs), cfg.blockDim = dim3((unsigned)(32 * nw));
+    cfg.gridDim = dim3((unsigned)(a.heads * split), (unsigned)d.n_short), cfg.blockDim = dim3((unsigned)(32 * nw));
     cfg.dynamicSmemBytes = smem, cfg.stream = st, cfg.attrs = attr, cfg.numAttrs = (pdl & 1) ? 1 : 0;
-    JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, kern, a, d.segs, split, tt, pdl));
-    if (split > 1) {
+    JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, kern, a, d.segs, d.short_segs, split, tt, pdl));
+    return JGPT_OK;
+}
+
+template <class AT, int KIND>
+static int32_t rec_run(const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st) {
+    int split = 1;
+    int32_t rc = launch_recurrent_chunks(sizeof(AT) == 4, d, a, pdl, st);
+    if (!rc)
+        switch (a.DK) {
+            case 32: rc = rec_launch<AT, KIND, 32>(d, a, pdl, &split, st); break;
+            case 64: rc = rec_launch<AT, KIND, 64>(d, a, pdl, &split, st); break;
+            case 96: rc = rec_launch<AT, KIND, 96>(d, a, pdl, &split, st); break;
+            case 128: rc = rec_launch<AT, KIND, 128>(d, a, pdl, &split, st); break;
+            case 192: rc = rec_launch<AT, KIND, 192>(d, a, pdl, &split, st); break;
+            case 256: rc = rec_launch<AT, KIND, 256>(d, a, pdl, &split, st); break;
+            default: return fail(JGPT_ERR_UNSUPPORTED, "key size %d", a.DK);
+        }
+    if (rc) return rc;
+    if (split > 1) {  // raw outputs of every row: the chunked rows are normed here as well (once more, to the same values)
         gated_norm_kernel<AT, KIND><<<(unsigned)((d.rows * a.heads + 7) / 8), 256, 0, st>>>(a, d.rows);
         JGPT_CUDA_TRY(cudaGetLastError());
     }
     return JGPT_OK;
 }
 
-template <class AT, int KIND>
-static int32_t rec_dispatch(const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st) {
-    switch (a.DK) {
-        case 32: return rec_launch<AT, KIND, 32>(d, a, pdl, st);
-        case 64: return rec_launch<AT, KIND, 64>(d, a, pdl, st);
-        case 96: return rec_launch<AT, KIND, 96>(d, a, pdl, st);
-        case 128: return rec_launch<AT, KIND, 128>(d, a, pdl, st);
-        case 192: return rec_launch<AT, KIND, 192>(d, a, pdl, st);
-        case 256: return rec_launch<AT, KIND, 256>(d, a, pdl, st);
-        default: return fail(JGPT_ERR_UNSUPPORTED, "key size %d", a.DK);
-    }
-}
-
 int32_t launch_recurrent(bool f32, const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st) {
     JGPT_REQUIRE(a.taps <= kMaxTaps, JGPT_ERR_UNSUPPORTED, "convolutions of up to %d taps", kMaxTaps);
-    if (f32) return a.kind == REC_DELTA ? rec_dispatch<float, REC_DELTA>(d, a, pdl, st) : rec_dispatch<float, REC_GLA>(d, a, pdl, st);
-    return a.kind == REC_DELTA ? rec_dispatch<__nv_bfloat16, REC_DELTA>(d, a, pdl, st) : rec_dispatch<__nv_bfloat16, REC_GLA>(d, a, pdl, st);
+    if (f32) return a.kind == REC_DELTA ? rec_run<float, REC_DELTA>(d, a, pdl, st) : rec_run<float, REC_GLA>(d, a, pdl, st);
+    return a.kind == REC_DELTA ? rec_run<__nv_bfloat16, REC_DELTA>(d, a, pdl, st) : rec_run<__nv_bfloat16, REC_GLA>(d, a, pdl, st);
 }
 
 }  // namespace mix

@@ -1,0 +1,54 @@
+// Elementwise pieces shared by the token-by-token and the chunked form of the recurrent mixers.
+#pragma once
+
+#include "mixers.cuh"
+#include "ptx.cuh"
+
+namespace jgpt {
+namespace mix {
+
+constexpr int kMaxTaps = 8;
+
+__device__ __forceinline__ float2 load2(const __nv_bfloat16 *p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(p)); }
+__device__ __forceinline__ float2 load2(const float *p) { return *reinterpret_cast<const float2 *>(p); }
+__device__ __forceinline__ float load1(const __nv_bfloat16 *p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float load1(const float *p) { return *p; }
+__device__ __forceinline__ void store2(__nv_bfloat16 *p, float2 v) { *reinterpret_cast<__nv_bfloat162 *>(p) = __float22bfloat162_rn(v); }
+__device__ __forceinline__ void store2(float *p, float2 v) { *reinterpret_cast<float2 *>(p) = v; }
+__device__ __forceinline__ void store1(__nv_bfloat16 *p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ void store1(float *p, float v) { *p = v; }
+
+// exp for the bf16 mode is the fast one (relative error ~2^-21 on the ranges used here), the exact mode takes expf.
+template <class AT>
+__device__ __forceinline__ float exp_f(float x) {
+    return sizeof(AT) == 4 ? expf(x) : __expf(x);
+}
+template <class AT>
+__device__ __forceinline__ float sigmoid_f(float x) {
+    return sizeof(AT) == 4 ? 1.f / (1.f + expf(-x)) : __fdividef(1.f, 1.f + __expf(-x));
+}
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+    for (int off = 16; off >= 1; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
+    return v;
+}
+
+// RMS norm over a head's value columns and its output gate, by one warp: raw fp32 values -> activations.
+template <class AT, int KIND>
+__device__ __forceinline__ void norm_gate_head(const RecArgs &a, int r, int h, int lane) {
+    const float *raw = a.raw + (size_t)r * a.heads * a.DV + h * a.DV;
+    float ss = 0.f;
+    for (int c = lane; c < a.DV; c += 32) ss += raw[c] * raw[c];
+    const float inv = a.out_scale / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
+    AT *o = reinterpret_cast<AT *>(a.out) + (size_t)r * a.ldo + a.out_off + h * a.DV;
+    const AT *gp = KIND == REC_DELTA ? reinterpret_cast<const AT *>(a.z) + (size_t)r * a.ldz + a.zg_off + h * a.DV
+                                     : reinterpret_cast<const AT *>(a.proj) + (size_t)r * a.ldp + a.g_off + h * a.DV;
+    for (int c = lane; c < a.DV; c += 32) {
+        const float gt = load1(gp + c), sgt = sigmoid_f<AT>(gt);
+        store1(o + c, raw[c] * inv * a.norm_w[c] * (KIND == REC_DELTA ? sgt : gt * sgt));
+    }
+}
+
+}  // namespace mix
+}  // namespace jgpt

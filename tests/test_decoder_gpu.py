@@ -147,6 +147,43 @@ def test_portions_equal_the_whole(ctx, cases, sizes, dtype):
         pool.close(), m.close()
 
 
+@pytest.mark.parametrize("name", list(CASES))
+def test_chunked_recurrences_at_full_precision(ctx, cases, name, monkeypatch):
+    """The chunked form of the recurrences (tensor cores, three TF32 products) on fp32 activations: as close to the oracle as
+    the token-by-token form, for whole prompts, for portions around the length from which it is used, and beside short ones."""
+    monkeypatch.setenv("JGPT_B200_REC_CHUNK_EXACT", "1")
+    monkeypatch.setenv("JGPT_B200_REC_CHUNK_MIN", "6")
+    c = cases[name]
+    m = c.model(ctx, "float32")
+    pool = m.newPool(60, 3)
+    for sizes in ([320], [6], [5, 7, 1, 40, 2, 16, 17, 33], [161, 1, 158]):
+        t = dc.tokens(c.cfg, 320, 17)
+        _close(dc.run_steps(m, pool, [[("a", p)] for p in dc.cut(t, sizes)])["a"], c.ref(t), "float32")
+    toks = {f"r{i}": dc.tokens(c.cfg, L, 50 + i) for i, L in enumerate([1, 150, 33, 64, 17, 2])}
+    got = dc.run_steps(m, pool, _mixed_plan(toks, 3))
+    for r, t in toks.items():
+        _close(got[r], c.ref(t), "float32")
+    pool.close(), m.close()
+
+
+def test_chunked_recurrences_with_decays_that_vanish(ctx, monkeypatch):
+    """Channels that forget everything from one token to the next, beside channels that forget nothing."""
+    monkeypatch.setenv("JGPT_B200_REC_CHUNK_EXACT", "1")
+    cfg = dc.config([dc.delta(heads=2, kv_heads=2, dim=32, vdim=16), dc.par(right=dc.gla(heads=2, dim=32, vdim=16, tau=0.1))])
+
+    def edit(W):
+        W["l0.mix.A_log"] = np.array([4.0, -8.0])
+        W["l0.mix.dt_bias"] = W["l0.mix.dt_bias"] * 4
+        W["l1.mix.right.a2.b"] = W["l1.mix.right.a2.b"] * 10 - 20
+    c = dc.Case(cfg, seed=4, edit=edit)
+    t = dc.tokens(cfg, 200, 1)
+    for dtype in ("float32", "bfloat16"):
+        m = c.model(ctx, dtype)
+        pool = m.newPool(16, 1)
+        _close(dc.run_steps(m, pool, [[("a", p)] for p in dc.cut(t, [100, 1, 99])])["a"], c.ref(t), dtype)
+        pool.close(), m.close()
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_long_decoding(ctx, cases, dtype):
     c = cases["both"]
