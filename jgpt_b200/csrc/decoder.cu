@@ -66,6 +66,18 @@ struct Decoder {
     uint64_t chunk_ws_floats = 0;
     int long_min = 0;  // entries of at least this many tokens run their recurrences in chunks (0: none)
     int logit_rows = 0;
+    // Decode steps (one token per entry, the picked ids as the only result) replayed as CUDA graphs from the second step of a
+    // kind on.  The launches depend on the batch size, the length bucket and the pool's addresses: the key.
+    struct Graph {
+        const Pool *pool = nullptr;
+        uint64_t generation = 0, last_use = 0;
+        int n = 0, bucket = 0;
+        cudaGraphExec_t exec = nullptr;
+        bool failed = false;
+    };
+    std::vector<Graph> graphs;
+    uint64_t graph_clock = 0;
+    int use_graphs = 1, overlap = 1;  // JGPT_B200_DECODE_GRAPH, JGPT_B200_STEP_OVERLAP (0: off)
     float *capture = nullptr;  // host, [layers][rows][width] of the next step
     uint64_t capture_floats = 0;
 };
@@ -92,6 +104,8 @@ static int32_t dalloc(Decoder *d, void **p, uint64_t bytes) {
     } while (0)
 
 static void release(Decoder *d) {
+    for (Decoder::Graph &g : d->graphs)
+        if (g.exec) cudaGraphExecDestroy(g.exec);
     for (void *p : d->allocs) cudaFree(p);
     cudaFreeHost(d->h_desc), cudaFreeHost(d->h_next), cudaFreeHost(d->h_u);
     delete d;
@@ -387,8 +401,10 @@ int32_t decoder_check_pool(const Decoder *d, const Pool *p) {
     return JGPT_OK;
 }
 
-static int32_t product(Decoder *d, const nt::Problem *p, int n, nt::Epilogue epi) {
-    return d->f32 ? nt::launch_f32(p, n, epi, d->ctx->stream) : nt::launch_bf16(d->ctx, p, n, epi, 0, d->ctx->stream);
+// pdl (every launch of a step but the first): bit 0 = the kernel may start while its predecessor drains and waits itself
+// before it touches anything a kernel of this step writes; bit 1 = it lets its successor do the same.
+static int32_t product(Decoder *d, const nt::Problem *p, int n, nt::Epilogue epi, int pdl) {
+    return d->f32 ? nt::launch_f32(p, n, epi, d->ctx->stream) : nt::launch_bf16(d->ctx, p, n, epi, pdl, d->ctx->stream);
 }
 
 static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, uint64_t capture_rows) {
@@ -396,15 +412,16 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, uint
     const float eps = d->s.eps;
     cudaStream_t st = d->ctx->stream;
     int *status = d->ctx->d_status;
+    const int pdl = d->overlap && !d->f32 && !capture_rows ? 3 : 0;
     for (size_t i = 0; i < d->L.size(); i++) {
         DLayer &y = d->L[i];
         if (i == 0)
             TRY(mix::launch_embed(d->f32, sd, d->embed, ldw, d->pos, ldw, d->s.embed_scale,
                                   d->s.embed_norm ? mix::NormW{d->enw, d->enb} : mix::NormW{nullptr, nullptr}, mix::NormW{y.n1w, y.n1b}, eps, d->x,
-                                  d->h, W, ldw, d->s.vocab, d->s.max_positions, status, 0, st));
-        else TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n1w, y.n1b}, eps, d->h, R, W, ldw, 0, st));
+                                  d->h, W, ldw, d->s.vocab, d->s.max_positions, status, pdl & 2, st));
+        else TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n1w, y.n1b}, eps, d->h, R, W, ldw, pdl, st));
         nt::Problem in{d->h, y.w_in, d->proj, nullptr, R, y.n_in, ldw, ldw, ldw, y.n_in, 1.f};
-        TRY(product(d, &in, 1, nt::EPI_STORE));
+        TRY(product(d, &in, 1, nt::EPI_STORE, pdl));
         for (DBranch &b : y.br) {
             if (b.s.kind == JGPT_MIX_ATTENTION) {
                 mix::AttnArgs a{};
@@ -413,7 +430,7 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, uint
                 a.kv = p->vkv + p->vlayers[(size_t)b.kv_layer].offset, a.table = p->d_table, a.n_blocks = p->n_blocks, a.mbs = p->max_blocks_per_seq;
                 a.out = d->mixed, a.ldo = y.n_out, a.out_off = b.out;
                 a.sm_count = d->ctx->sm_count, a.status = status;
-                TRY(mix::launch_attention(d->f32, sd, a, 0, st));
+                TRY(mix::launch_attention(d->f32, sd, a, pdl, st));
             } else {
                 uint8_t *proj = reinterpret_cast<uint8_t *>(d->proj), *z = reinterpret_cast<uint8_t *>(d->z);
                 nt::Problem zp[2];
@@ -421,22 +438,22 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, uint
                 zp[nz++] = nt::Problem{proj + (size_t)b.a1 * eb, b.w_a2, z + (size_t)b.za * eb, nullptr, R, b.s.heads * b.DK, b.ra, y.n_in, b.ra, y.n_z, 1.f};
                 if (b.g1 >= 0)
                     zp[nz++] = nt::Problem{proj + (size_t)b.g1 * eb, b.w_g2, z + (size_t)b.zg * eb, nullptr, R, b.s.heads * b.DV, b.rg, y.n_in, b.rg, y.n_z, 1.f};
-                TRY(product(d, zp, nz, nt::EPI_STORE));
+                TRY(product(d, zp, nz, nt::EPI_STORE, pdl));
                 mix::RecArgs a = rec_args(b);
                 a.proj = d->proj, a.ldp = y.n_in, a.z = d->z, a.ldz = y.n_z, a.eps = eps;
                 a.state = p->state + b.state_off, a.state_stride = p->state_stride, a.max_seqs = p->max_seqs;
                 a.out = d->mixed, a.ldo = y.n_out, a.raw = d->raw, a.chunk_ws = d->chunk_ws, a.chunk_ws_floats = d->chunk_ws_floats, a.sm_count = d->ctx->sm_count, a.status = status;
-                TRY(mix::launch_recurrent(d->f32, sd, a, 0, st));
+                TRY(mix::launch_recurrent(d->f32, sd, a, pdl, st));
             }
         }
         nt::Problem out{d->mixed, y.w_out, d->x, nullptr, R, W, y.n_out, y.n_out, y.n_out, W, 1.f};
-        TRY(product(d, &out, 1, nt::EPI_ADD_F32));
+        TRY(product(d, &out, 1, nt::EPI_ADD_F32, pdl));
         if (y.ff) {
-            TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n2w, y.n2b}, eps, d->h, R, W, ldw, 0, st));
+            TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n2w, y.n2b}, eps, d->h, R, W, ldw, pdl, st));
             nt::Problem gu{d->h, y.w_gu, d->act, nullptr, R, 2 * y.ffp, ldw, ldw, ldw, y.ffp, 1.f};
-            TRY(product(d, &gu, 1, nt::EPI_GATE_GELU));
+            TRY(product(d, &gu, 1, nt::EPI_GATE_GELU, pdl));
             nt::Problem down{d->act, y.w_down, d->x, nullptr, R, W, y.ffp, y.ffp, y.ffp, W, 1.f};
-            TRY(product(d, &down, 1, nt::EPI_ADD_F32));
+            TRY(product(d, &down, 1, nt::EPI_ADD_F32, pdl));
         }
         if (capture_rows)
             JGPT_CUDA_TRY(cudaMemcpyAsync(d->capture + (uint64_t)i * capture_rows * W, d->x, sizeof(float) * capture_rows * W, cudaMemcpyDeviceToHost, st));
@@ -447,12 +464,48 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, uint
 // Final norm, logits and token choice of wanted rows [w0, w0 + n).
 static int32_t enqueue_head(Decoder *d, const mix::StepDesc &sd, int w0, int n, bool pick, const SampleSpec &spec) {
     cudaStream_t st = d->ctx->stream;
-    TRY(mix::launch_layer_norm(d->f32, d->x, sd.want + w0, mix::NormW{d->fnw, d->fnb}, d->s.eps, d->h, n, d->s.width, d->ldw, 0, st));
+    const int pdl = d->overlap && !d->f32 && w0 == 0 ? 3 : 0;
+    TRY(mix::launch_layer_norm(d->f32, d->x, sd.want + w0, mix::NormW{d->fnw, d->fnb}, d->s.eps, d->h, n, d->s.width, d->ldw, pdl, st));
     nt::Problem p{d->h, d->embed, d->logits, nullptr, n, d->s.vocab, d->ldw, d->ldw, d->ldw, d->s.vocab, d->s.logit_scale};
-    TRY(product(d, &p, 1, nt::EPI_SCALE_F32));
+    TRY(product(d, &p, 1, nt::EPI_SCALE_F32, pdl & 1));
     if (!pick) return JGPT_OK;
     if (spec.temperature > 0.f) return launch_sample(d->logits, d->samp, n, d->s.vocab, spec, d->d_u + w0, d->d_next + w0, st);
     return launch_argmax(d->logits, n, d->s.vocab, d->d_next + w0, st);
+}
+
+// Replays the step's graph, captures it at the second step of its kind, or runs the launches one by one.
+template <class Fn>
+static int32_t run_graph(Decoder *d, const Pool *p, int n, int bucket, Fn &&enqueue) {
+    cudaStream_t st = d->ctx->stream;
+    for (Decoder::Graph &g : d->graphs) {
+        if (g.pool != p || g.generation != p->generation || g.n != n || g.bucket != bucket) continue;
+        g.last_use = ++d->graph_clock;
+        if (!g.exec && !g.failed) {
+            cudaGraph_t graph = nullptr;
+            JGPT_CUDA_TRY(cudaStreamBeginCapture(st, cudaStreamCaptureModeThreadLocal));
+            const int32_t rc = enqueue();
+            const cudaError_t e = cudaStreamEndCapture(st, &graph);
+            if (rc || e != cudaSuccess || cudaGraphInstantiate(&g.exec, graph, 0) != cudaSuccess) g.exec = nullptr, g.failed = true;
+            if (graph) cudaGraphDestroy(graph);
+            cudaGetLastError();
+        }
+        if (!g.exec) break;
+        JGPT_CUDA_TRY(cudaGraphLaunch(g.exec, st));
+        return JGPT_OK;
+    }
+    bool known = false;
+    for (const Decoder::Graph &g : d->graphs) known = known || (g.pool == p && g.generation == p->generation && g.n == n && g.bucket == bucket);
+    if (!known) {
+        if (d->graphs.size() >= 64) {  // forget the one that has not been used for longest
+            auto old = std::min_element(d->graphs.begin(), d->graphs.end(), [](const Decoder::Graph &x, const Decoder::Graph &y) { return x.last_use < y.last_use; });
+            if (old->exec) cudaGraphExecDestroy(old->exec);
+            d->graphs.erase(old);
+        }
+        Decoder::Graph g;
+        g.pool = p, g.generation = p->generation, g.n = n, g.bucket = bucket, g.last_use = ++d->graph_clock;
+        d->graphs.push_back(g);
+    }
+    return enqueue();
 }
 
 int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) {
@@ -535,7 +588,6 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
     at = o_tile + 2 * (size_t)n_tiles;
     JGPT_REQUIRE(at <= desc_ints(d), JGPT_ERR_INVALID_ARGUMENT, "step descriptors need %zu words, there are %zu", at, desc_ints(d));
     cudaStream_t st = d->ctx->stream;
-    JGPT_CUDA_TRY(cudaMemcpyAsync(d->d_desc, hd, sizeof(int) * at, cudaMemcpyHostToDevice, st));
     mix::StepDesc sd{};
     const int *dd = d->d_desc;
     sd.tok = dd + o_tok, sd.pos = dd + o_pos, sd.seq = dd + o_seq, sd.segs = reinterpret_cast<const mix::Seg *>(dd + o_seg);
@@ -545,27 +597,43 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
     sd.short_segs = dd + o_short, sd.long_segs = reinterpret_cast<const int2 *>(dd + o_long), sd.chunks = reinterpret_cast<const int2 *>(dd + o_chunk);
     sd.n_short = n_short, sd.n_long = n_long, sd.n_chunks = n_chunks;
 
+    if (n_tiles == 0) sd.max_len = std::min(up(max_len, 256), d->s.max_positions);  // a bucket: it only shapes the launches
     uint64_t cap_rows = 0;
     if (d->capture) {
         JGPT_REQUIRE(d->capture_floats >= (uint64_t)d->L.size() * rows * d->s.width, JGPT_ERR_INVALID_ARGUMENT, "capture buffer is too small");
         cap_rows = (uint64_t)rows;
     }
-    TRY(enqueue_layers(d, p, sd, cap_rows));
-    d->capture = nullptr;
+    float *capture_to = d->capture;
     const bool pick = c.next_host != nullptr;
     if (pick && c.spec.temperature > 0.f && c.n_want) {
         if (!d->samp) TRY(dalloc(d, (void **)&d->samp, sizeof(float) * (uint64_t)d->logit_rows * d->s.vocab));
         std::copy(c.u01, c.u01 + c.n_want, d->h_u);
         JGPT_CUDA_TRY(cudaMemcpyAsync(d->d_u, d->h_u, sizeof(float) * c.n_want, cudaMemcpyHostToDevice, st));
     }
-    for (int w0 = 0; w0 < c.n_want; w0 += d->logit_rows) {
-        const int n = std::min(d->logit_rows, c.n_want - w0);
-        TRY(enqueue_head(d, sd, w0, n, pick, c.spec));
-        if (c.logits_host)
-            JGPT_CUDA_TRY(cudaMemcpyAsync(c.logits_host + (size_t)w0 * d->s.vocab, d->logits, sizeof(float) * (size_t)n * d->s.vocab, cudaMemcpyDeviceToHost, st));
+    auto enqueue = [&]() -> int32_t {
+        JGPT_CUDA_TRY(cudaMemcpyAsync(d->d_desc, hd, sizeof(int) * at, cudaMemcpyHostToDevice, st));
+        TRY(enqueue_layers(d, p, sd, cap_rows));
+        for (int w0 = 0; w0 < c.n_want; w0 += d->logit_rows) {
+            const int n = std::min(d->logit_rows, c.n_want - w0);
+            TRY(enqueue_head(d, sd, w0, n, pick, c.spec));
+            if (c.logits_host)
+                JGPT_CUDA_TRY(cudaMemcpyAsync(c.logits_host + (size_t)w0 * d->s.vocab, d->logits, sizeof(float) * (size_t)n * d->s.vocab,
+                                              cudaMemcpyDeviceToHost, st));
+        }
+        if (pick && c.n_want) JGPT_CUDA_TRY(cudaMemcpyAsync(d->h_next, d->d_next, sizeof(int) * c.n_want, cudaMemcpyDeviceToHost, st));
+        JGPT_CUDA_TRY(status_enqueue_read(d->ctx));
+        return JGPT_OK;
+    };
+    bool plain = d->use_graphs && n_tiles == 0 && pick && !c.logits_host && !capture_to && c.spec.temperature <= 0.f && c.n_want == c.n;
+    for (int i = 0; plain && i < c.n; i++) plain = c.want[i] == i;
+    d->capture = nullptr;
+    if (plain) TRY(run_graph(d, p, c.n, sd.max_len, enqueue));
+    else {
+        d->capture = capture_to;
+        const int32_t rc = enqueue();
+        d->capture = nullptr;
+        if (rc) return rc;
     }
-    if (pick && c.n_want) JGPT_CUDA_TRY(cudaMemcpyAsync(d->h_next, d->d_next, sizeof(int) * c.n_want, cudaMemcpyDeviceToHost, st));
-    JGPT_CUDA_TRY(status_enqueue_read(d->ctx));
     JGPT_CUDA_TRY(cudaStreamSynchronize(st));
     TRY(status_check_after_sync(d->ctx, p, "forward step"));
     if (pick) std::copy(d->h_next, d->h_next + c.n_want, c.next_host);
@@ -688,6 +756,7 @@ int32_t jgpt_decoder_create(jgpt_ctx ctxh, const jgpt_decoder_spec *spec, const 
     JGPT_REQUIRE(dtype == JGPT_DTYPE_BF16 || dtype == JGPT_DTYPE_F32, JGPT_ERR_INVALID_ARGUMENT, "dtype %d", dtype);
     JGPT_CUDA_TRY(make_current(c));
     Decoder *d = new Decoder();
+    d->use_graphs = env_int("JGPT_B200_DECODE_GRAPH", 1), d->overlap = env_int("JGPT_B200_STEP_OVERLAP", 1);
     d->ctx = c, d->s = *spec, d->f32 = dtype == JGPT_DTYPE_F32, d->eb = d->f32 ? 4 : 2, d->R = max_rows, d->ldw = up(spec->width, 8);
     const int32_t rc = build(d, layers);
     if (rc) {

@@ -19,6 +19,7 @@
 // of its 16 value columns as fp32 accumulators; the accumulator layout IS the A operand layout of the next chunk once channels
 // 2t, 2t+1 of a k step are taken in the order (t, t + 4), so the state never leaves registers.  Records come in by bulk copies.
 #include <algorithm>
+#include <type_traits>
 
 #include "recurrent_math.cuh"
 
@@ -47,6 +48,21 @@ __device__ __forceinline__ int at_16(int x, int j) { return x * 16 + ((((j >> 3)
 __device__ __forceinline__ void store_row16(float *m, int x, const float (&v)[16]) {
 #pragma unroll
     for (int j = 0; j < 16; j += 4) *reinterpret_cast<float4 *>(m + at_16(x, j)) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+}
+
+// Row i of a lower triangular 16 x 16 matrix in shared memory times x (entries past i are not touched).
+__device__ __forceinline__ float lower_dot(const float *T, int i, const float (&x)[16]) {
+    float s = 0.f;
+#pragma unroll
+    for (int j = 0; j < 16; j += 4)
+        if (j <= i) {
+            const float4 q = *reinterpret_cast<const float4 *>(T + i * 16 + j);
+            s = fmaf(q.x, x[j], s);
+            if (j + 1 <= i) s = fmaf(q.y, x[j + 1], s);
+            if (j + 2 <= i) s = fmaf(q.z, x[j + 2], s);
+            if (j + 3 <= i) s = fmaf(q.w, x[j + 3], s);
+        }
+    return s;
 }
 
 // 32 sums over the 32 lanes: lane L returns the total of v[L].
@@ -97,57 +113,70 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
         }
     };
     const int npairs = DK + DV / 2;
+    // decay logits and step sizes are requested first and used last
+    constexpr int ZN = (kC * DK / 2 + 255) / 256;
+    float2 zr[ZN];
+#pragma unroll
+    for (int e = 0; e < ZN; e++) {
+        const int idx = e * 256 + tid, t = idx / (DK / 2), c = 2 * (idx % (DK / 2));
+        zr[e] = t < tn ? load2(z + (size_t)(t0 + t) * a.ldz + a.z_off + h * DK + c) : make_float2(0.f, 0.f);
+    }
+    float bl = 0.f;
+    if (KIND == REC_DELTA && tid < tn) bl = load1(proj + (size_t)(t0 + tid) * a.ldp + a.b_off + h);
     // ---- q, k, v of the chunk ----
+    auto convolve = [&](auto max_taps, int pc, int ch, float *dst, int ld) {
+        constexpr int MT = decltype(max_taps)::value;
+        const float *w = (ch < nq ? a.conv_q + (size_t)ch * a.taps
+                                  : (ch < 2 * nq ? a.conv_k + (size_t)(ch - nq) * a.taps : a.conv_v + (size_t)(ch - 2 * nq) * a.taps));
+        float2 wt[MT], x[kC + MT - 1];  // x[i]: token t0 + i - (MT - 1); every load in flight at once
+#pragma unroll
+        for (int back = 0; back < MT; back++) wt[back] = back < a.taps ? make_float2(w[a.taps - 1 - back], w[2 * a.taps - 1 - back]) : make_float2(0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < kC + MT - 1; i++) {
+            const int t = t0 + i - (MT - 1);
+            x[i] = i < MT - 1 ? (MT - 1 - i < a.taps ? conv_input(t, pc, ch) : make_float2(0.f, 0.f))
+                              : (i - (MT - 1) < tn ? load2(proj + (size_t)t * a.ldp + pc) : make_float2(0.f, 0.f));
+        }
+#pragma unroll
+        for (int t = 0; t < kC; t++) {
+            float2 y = make_float2(0.f, 0.f);
+#pragma unroll
+            for (int back = 0; back < MT; back++) y.x = fmaf(wt[back].x, x[t + MT - 1 - back].x, y.x), y.y = fmaf(wt[back].y, x[t + MT - 1 - back].y, y.y);
+            *reinterpret_cast<float2 *>(dst + t * ld) = t < tn ? make_float2(y.x * sigmoid_f<AT>(y.x), y.y * sigmoid_f<AT>(y.y)) : make_float2(0.f, 0.f);
+        }
+    };
     for (int idx = tid; idx < npairs; idx += 256) {
         int pc, ch;
         locate(idx, pc, ch);
         float *dst = idx < DK / 2 ? sq + 2 * idx : (idx < DK ? sk + 2 * idx - DK : sv + 2 * (idx - DK));
         const int ld = idx < DK ? DK : DV;
-        float2 x[kC];  // every load in flight at once
-#pragma unroll
-        for (int t = 0; t < kC; t++) x[t] = t < tn ? load2(proj + (size_t)(t0 + t) * a.ldp + pc) : make_float2(0.f, 0.f);
         if (KIND == REC_DELTA) {
-            const float *w = (ch < nq ? a.conv_q + (size_t)ch * a.taps
-                                      : (ch < 2 * nq ? a.conv_k + (size_t)(ch - nq) * a.taps : a.conv_v + (size_t)(ch - 2 * nq) * a.taps));
-            float2 y[kC];
-#pragma unroll
-            for (int t = 0; t < kC; t++) y[t] = make_float2(0.f, 0.f);
-#pragma unroll
-            for (int back = 0; back < kMaxTaps; back++) {
-                if (back >= a.taps) break;
-                const float wx = w[a.taps - 1 - back], wy = w[2 * a.taps - 1 - back];
-#pragma unroll
-                for (int t = 0; t < kC; t++) {
-                    const float2 in = t >= back ? x[t - back] : conv_input(t0 + t - back, pc, ch);
-                    y[t].x = fmaf(wx, in.x, y[t].x), y[t].y = fmaf(wy, in.y, y[t].y);
-                }
-            }
-#pragma unroll
-            for (int t = 0; t < kC; t++)
-                *reinterpret_cast<float2 *>(dst + t * ld) =
-                    t < tn ? make_float2(y[t].x * sigmoid_f<AT>(y[t].x), y[t].y * sigmoid_f<AT>(y[t].y)) : make_float2(0.f, 0.f);
+            if (a.taps <= 4) convolve(std::integral_constant<int, 4>(), pc, ch, dst, ld);
+            else convolve(std::integral_constant<int, kMaxTaps>(), pc, ch, dst, ld);
         } else {
+            float2 x[kC];
             const float f = idx < DK / 2 ? qscale : 1.f;
+#pragma unroll
+            for (int t = 0; t < kC; t++) x[t] = t < tn ? load2(proj + (size_t)(t0 + t) * a.ldp + pc) : make_float2(0.f, 0.f);
 #pragma unroll
             for (int t = 0; t < kC; t++) *reinterpret_cast<float2 *>(dst + t * ld) = make_float2(x[t].x * f, x[t].y * f);
         }
     }
     // ---- decays (1 past the end: the state stays) and step sizes ----
 #pragma unroll
-    for (int e = 0; e < kC * DK / 2; e += 256) {
-        const int idx = e + tid, t = idx / (DK / 2), c = 2 * (idx % (DK / 2));
-        if (kC * DK / 2 % 256 != 0 && idx >= kC * DK / 2) break;
+    for (int e = 0; e < ZN; e++) {
+        const int idx = e * 256 + tid, t = idx / (DK / 2), c = 2 * (idx % (DK / 2));
+        if (t >= kC) break;
         float2 y = make_float2(1.f, 1.f);
         if (t < tn) {
-            y = load2(z + (size_t)(t0 + t) * a.ldz + a.z_off + h * DK + c);
             const float2 b = *reinterpret_cast<const float2 *>(a.decay_bias + h * DK + c);
-            y.x += b.x, y.y += b.y;
+            y.x = zr[e].x + b.x, y.y = zr[e].y + b.y;
             if (KIND == REC_GLA) y.x = -y.x, y.y = -y.y;
             y.x = exp_f<AT>(-rate * softplus_f(y.x)), y.y = exp_f<AT>(-rate * softplus_f(y.y));
         }
         *reinterpret_cast<float2 *>(sg + t * DK + c) = y;
     }
-    if (KIND == REC_DELTA && tid < kC) sbeta[tid] = tid < tn ? sigmoid_f<AT>(load1(proj + (size_t)(t0 + tid) * a.ldp + a.b_off + h)) : 0.f;
+    if (KIND == REC_DELTA && tid < kC) sbeta[tid] = tid < tn ? sigmoid_f<AT>(bl) : 0.f;
     __syncthreads();
     if (KIND == REC_DELTA) {
         for (int t = warp; t < kC; t += 8) {
@@ -229,11 +258,7 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
             if (KIND == REC_DELTA) {
 #pragma unroll
                 for (int i = 0; i < kC; i++) {
-                    float w = 0.f;
-#pragma unroll
-                    for (int j = 0; j < kC; j++)
-                        if (j <= i) w = fmaf(sT[i * kC + j], kt[j], w);
-                    rw[at_tok(i, d, DK)] = -w;
+                    rw[at_tok(i, d, DK)] = -lower_dot(sT, i, kt);
                 }
             }
             b = 1.f;
@@ -251,11 +276,7 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
             if (KIND == REC_DELTA) {
 #pragma unroll
                 for (int i = kC - 1; i >= 0; i--) {  // T is lower triangular: row i needs rows up to i only
-                    float u = 0.f;
-#pragma unroll
-                    for (int j = 0; j < kC; j++)
-                        if (j <= i) u = fmaf(sT[i * kC + j], vv[j], u);
-                    vv[i] = u;
+                    vv[i] = lower_dot(sT, i, vv);
                 }
             }
             store_row16(ru, c, vv);
@@ -275,16 +296,22 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
     }
 }
 
+// TF32 high and low part by truncation (the remainder is exact before its own truncation: ~2^-21 together).  Two masks and
+// a subtraction; the rounding conversion would give half a bit more and costs the scan more issue time than its products.
+__device__ __forceinline__ void split_trunc(float x, uint32_t &hi, uint32_t &lo) {
+    hi = __float_as_uint(x) & 0xffffe000u;
+    lo = __float_as_uint(x - __uint_as_float(hi)) & 0xffffe000u;
+}
 // hi / lo TF32 parts of an A fragment held as accumulators (see the order note above) and the three-product update.
 struct SplitA {
     uint32_t hi[4], lo[4];
     __device__ __forceinline__ explicit SplitA(const float (&c)[4]) {
-        split_tf32(c[0], hi[0], lo[0]), split_tf32(c[2], hi[1], lo[1]), split_tf32(c[1], hi[2], lo[2]), split_tf32(c[3], hi[3], lo[3]);
+        split_trunc(c[0], hi[0], lo[0]), split_trunc(c[2], hi[1], lo[1]), split_trunc(c[1], hi[2], lo[2]), split_trunc(c[3], hi[3], lo[3]);
     }
 };
 struct SplitB {
     uint32_t hi[2], lo[2];
-    __device__ __forceinline__ explicit SplitB(const float2 v) { split_tf32(v.x, hi[0], lo[0]), split_tf32(v.y, hi[1], lo[1]); }
+    __device__ __forceinline__ explicit SplitB(const float2 v) { split_trunc(v.x, hi[0], lo[0]), split_trunc(v.y, hi[1], lo[1]); }
 };
 __device__ __forceinline__ void mma3(float (&acc)[4], float (&cor)[4], const SplitA &x, const SplitB &y) {
     mma_tf32(cor, x.lo, y.hi[0], y.hi[1]);
