@@ -1,9 +1,9 @@
 // C[M, N] = A[M, K] . W[N, K]^T for decode-sized M (bf16, mma.sync) and in plain fp32.
 //
-// Decode-sized bf16 products are bound by the weight stream and by latency: a CTA owns 32 output columns and up to 64
-// rows, its eight warps split every 128-wide k tile (each warp covers the whole output tile with its own 16-wide
-// slice), tiles arrive through a cp.async ring, and the eight partial tiles are added in warp order through shared
-// memory.  Products with few column tiles run as clusters of CTAs that split the k range; the partial sums meet in the
+// Decode-sized bf16 products are bound by the weight stream and by latency: a CTA owns 32 output columns (64 from 33 rows
+// on, so that the rows are read half as often) and up to 64 rows; its eight warps split every 128-wide k tile (a warp
+// covers 32 columns with its own k slice), tiles arrive through a cp.async ring, and the partial tiles are added in warp
+// order through shared memory.  Products with few column tiles run as clusters of CTAs that split the k range; the partial sums meet in the
 // first CTA's shared memory and are added in k order: no atomics, the same bits every time.
 #include "gemm_nt.cuh"
 
@@ -21,7 +21,7 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-constexpr int kBN = 32, kBK = 128, kMaxSplit = 8;
+constexpr int kBK = 128, kMaxSplit = 8;
 
 struct SmallArgs {
     Problem p[2];
@@ -29,23 +29,27 @@ struct SmallArgs {
     int n, k_split, pdl;
 };
 
-template <int MT, int STAGES>
+// Warps: NH groups of 32 columns x 8 / NH slices of the k tile.
+template <int MT, int NH>
+__host__ __device__ constexpr size_t small_red_bytes() { return sizeof(float) * (8 / NH) * 16 * MT * (32 * NH + 1); }
+template <int MT, int NH, int STAGES>
+__host__ __device__ constexpr size_t small_ring_bytes() { return (size_t)STAGES * (16 * MT + 32 * NH) * kBK * 2; }
+// The ring, the reduction buffer and the other k parts' sums follow one another in the same memory.
+template <int MT, int NH, int STAGES>
 constexpr size_t small_smem(int k_split) {
-    const size_t ring = (size_t)STAGES * (16 * MT + kBN) * kBK * 2, red = sizeof(float) * 8 * 16 * MT * (kBN + 1);
-    return std::max(ring, red) + sizeof(float) * (size_t)(k_split - 1) * 16 * MT * kBN;
+    return std::max(std::max(small_ring_bytes<MT, NH, STAGES>(), small_red_bytes<MT, NH>()), sizeof(float) * (size_t)(k_split - 1) * 16 * MT * 32 * NH);
 }
 
-template <int MT, int STAGES, int EPI>
+template <int MT, int NH, int STAGES, int EPI>
 __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args) {
-    constexpr int BM = 16 * MT;
+    constexpr int BM = 16 * MT, kBN = 32 * NH, KS = 8 / NH;
     extern __shared__ __align__(128) uint8_t nt_smem[];
     __nv_bfloat16 *As = reinterpret_cast<__nv_bfloat16 *>(nt_smem);         // [STAGES][BM][128], 16-byte chunks xor-swizzled by row
-    __nv_bfloat16 *Ws = As + (size_t)STAGES * BM * kBK;                     // [STAGES][32][128]
-    float *red = reinterpret_cast<float *>(nt_smem);                        // [8][BM][33], after the k loop
-    constexpr size_t ring_bytes = (size_t)STAGES * (BM + kBN) * kBK * 2, red_bytes = sizeof(float) * 8 * BM * (kBN + 1);
-    float *xch = reinterpret_cast<float *>(nt_smem + (ring_bytes > red_bytes ? ring_bytes : red_bytes));  // [k_split - 1][BM * 32]
+    __nv_bfloat16 *Ws = As + (size_t)STAGES * BM * kBK;                     // [STAGES][kBN][128]
+    float *red = reinterpret_cast<float *>(nt_smem);                        // [KS][BM][kBN + 1], after the k loop
+    float *xch = reinterpret_cast<float *>(nt_smem);                        // [k_split - 1][BM * kBN], after the reduction
 
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nh = warp % NH, kslice = warp / NH;
     int tile = blockIdx.x / args.k_split;
     const int k_part = blockIdx.x % args.k_split;
     const bool second = args.n > 1 && tile >= args.tiles[0];
@@ -61,7 +65,7 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
     const int r16 = tid >> 4, c16 = tid & 15;  // chunk slot: row r16 (+ 16 i), 16-byte chunk c16 of the 128-wide tile
     auto load_w = [&](int buf, int k0) {
 #pragma unroll
-        for (int i = 0; i < 2; i++) {
+        for (int i = 0; i < 2 * NH; i++) {
             const int r = r16 + 16 * i, k = k0 + c16 * 8;
             const bool ok = n0 + r < N && k < K;
             cp_async16(Ws + ((size_t)buf * kBN + r) * kBK + ((c16 ^ (r & 7)) * 8), ok ? W + (size_t)(n0 + r) * ldw + k : W, ok);
@@ -112,27 +116,31 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
             load_a(nb, k0);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
-        // this warp's slice: chunks 2 * warp and 2 * warp + 1 of every row
-        uint32_t b[2][4];
+        // this warp's slice: NH k steps of 16 (chunks 2 step and 2 step + 1 of every row), columns [32 nh, + 32)
 #pragma unroll
-        for (int h = 0; h < 2; h++) {  // 16 output columns each
-            const int r = h * 16 + ((lane >> 4) << 3) + (lane & 7), c = 2 * warp + ((lane >> 3) & 1);
-            ldmatrix_x4(b[h], Ws + ((size_t)buf * kBN + r) * kBK + ((c ^ (r & 7)) * 8));
-        }
+        for (int ks = 0; ks < NH; ks++) {
+            const int step = kslice * NH + ks;
+            uint32_t b[2][4];
 #pragma unroll
-        for (int i = 0; i < MT; i++) {
-            uint32_t a[4];
-            const int r = i * 16 + (((lane >> 3) & 1) << 3) + (lane & 7), c = 2 * warp + (lane >> 4);
-            ldmatrix_x4(a, As + ((size_t)buf * BM + r) * kBK + ((c ^ (r & 7)) * 8));
+            for (int h = 0; h < 2; h++) {  // 16 output columns each
+                const int r = nh * 32 + h * 16 + ((lane >> 4) << 3) + (lane & 7), c = 2 * step + ((lane >> 3) & 1);
+                ldmatrix_x4(b[h], Ws + ((size_t)buf * kBN + r) * kBK + ((c ^ (r & 7)) * 8));
+            }
 #pragma unroll
-            for (int j = 0; j < 4; j++) mma_bf16(acc[i][j], a, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
+            for (int i = 0; i < MT; i++) {
+                uint32_t a[4];
+                const int r = i * 16 + (((lane >> 3) & 1) << 3) + (lane & 7), c = 2 * step + (lane >> 4);
+                ldmatrix_x4(a, As + ((size_t)buf * BM + r) * kBK + ((c ^ (r & 7)) * 8));
+#pragma unroll
+                for (int j = 0; j < 4; j++) mma_bf16(acc[i][j], a, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
+            }
         }
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();  // the ring is free: it becomes the reduction buffer
     {
         const int g = lane >> 2, t = lane & 3;
-        float *w = red + (size_t)warp * BM * (kBN + 1);
+        float *w = red + (size_t)kslice * BM * (kBN + 1) + nh * 32;
 #pragma unroll
         for (int i = 0; i < MT; i++)
 #pragma unroll
@@ -148,11 +156,11 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
         const int e = tid + 256 * i;
         float s = 0.f;
 #pragma unroll
-        for (int w = 0; w < 8; w++) s += red[(size_t)w * BM * (kBN + 1) + (e >> 5) * (kBN + 1) + (e & 31)];
+        for (int w = 0; w < KS; w++) s += red[(size_t)w * BM * (kBN + 1) + e / kBN * (kBN + 1) + e % kBN];
         sum[i] = s;
     }
     if (args.k_split > 1) {
-        cluster_sync();  // every CTA of the cluster runs: its shared memory may be written
+        cluster_sync();  // every CTA of the cluster is past its reduction: its shared memory may be written
         if (k_part > 0) {
 #pragma unroll
             for (int i = 0; i < PER; i++) st_cluster_f32(&xch[(size_t)(k_part - 1) * BM * kBN + tid + 256 * i], 0, sum[i]);
@@ -165,12 +173,12 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
     }
 #pragma unroll
     for (int i = 0; i < PER; i++) {
-        const int e = tid + 256 * i, m = m0 + (e >> 5), c = e & 31, n = n0 + c;
+        const int e = tid + 256 * i, m = m0 + e / kBN, c = e % kBN, n = n0 + c;
         if (EPI == EPI_GATE_GELU) {
             // lanes 0-15 of a warp hold the gate of a row's 16 outputs, lanes 16-31 the linear part
             const float up = __shfl_down_sync(0xffffffffu, sum[i], 16);
-            if (c < 16 && m < M && n + 16 < N)
-                reinterpret_cast<__nv_bfloat16 *>(P.C)[(size_t)m * P.ldc + tile * 16 + c] = __float2bfloat16(gelu_tanh(sum[i]) * up);
+            if ((c & 31) < 16 && m < M && n + 16 < N)
+                reinterpret_cast<__nv_bfloat16 *>(P.C)[(size_t)m * P.ldc + n / 32 * 16 + (c & 15)] = __float2bfloat16(gelu_tanh(sum[i]) * up);
         } else if (m < M && n < N) {
             if (EPI == EPI_STORE) reinterpret_cast<__nv_bfloat16 *>(P.C)[(size_t)m * P.ldc + n] = __float2bfloat16(sum[i]);
             if (EPI == EPI_ADD_F32) reinterpret_cast<float *>(P.C)[(size_t)m * P.ldc + n] += sum[i];
@@ -179,15 +187,15 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
     }
 }
 
-template <int MT, int STAGES, int EPI>
+template <int MT, int NH, int STAGES, int EPI>
 static int32_t small_launch(const SmallArgs &args, int total_tiles, int M, cudaStream_t st) {
-    auto kern = gemm_nt_small_kernel<MT, STAGES, EPI>;
-    const size_t smem = small_smem<MT, STAGES>(args.k_split);
+    auto kern = gemm_nt_small_kernel<MT, NH, STAGES, EPI>;
+    const size_t smem = small_smem<MT, NH, STAGES>(args.k_split);
     static thread_local int set_for = -1;  // the opt-in to more than 48 KiB, once per device
     int dev = 0;
     JGPT_CUDA_TRY(cudaGetDevice(&dev));
     if (set_for != dev) {
-        JGPT_CUDA_TRY(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(small_smem<MT, STAGES>(kMaxSplit))));
+        JGPT_CUDA_TRY(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(small_smem<MT, NH, STAGES>(kMaxSplit))));
         set_for = dev;
     }
     cudaLaunchConfig_t cfg = {};
@@ -213,22 +221,22 @@ template <int EPI>
 static int32_t small_dispatch(const Ctx *ctx, const Problem *p, int n, int pdl, cudaStream_t st) {
     SmallArgs a{};
     a.n = n, a.pdl = pdl;
+    const int M = p[0].M, mt = M <= 16 ? 1 : (M <= 32 ? 2 : 4), bn = mt == 4 ? 64 : 32, max_split = mt == 4 ? 4 : kMaxSplit;
     int tiles = 0, K = 0;
     for (int i = 0; i < n; i++) {
         a.p[i] = p[i];
-        a.tiles[i] = (p[i].N + kBN - 1) / kBN;
+        a.tiles[i] = (p[i].N + bn - 1) / bn;
         tiles += a.tiles[i];
         K = std::max(K, p[i].K);
     }
-    const int M = p[0].M, mt = M <= 16 ? 1 : (M <= 32 ? 2 : 4);
     const int ctas = tiles * ((M + 16 * mt - 1) / (16 * mt)), nk = (K + kBK - 1) / kBK;
     // split k while the launch leaves SMs idle and every part keeps two tiles
     a.k_split = 1;
-    while (n == 1 && a.k_split < kMaxSplit && ctas * a.k_split * 2 <= 2 * ctx->sm_count && nk / (a.k_split * 2) >= 2) a.k_split *= 2;
+    while (n == 1 && a.k_split < max_split && ctas * a.k_split * 2 <= 2 * ctx->sm_count && nk / (a.k_split * 2) >= 2) a.k_split *= 2;
     switch (mt) {
-        case 1: return small_launch<1, 6, EPI>(a, tiles, M, st);
-        case 2: return small_launch<2, 5, EPI>(a, tiles, M, st);
-        default: return small_launch<4, 4, EPI>(a, tiles, M, st);
+        case 1: return small_launch<1, 1, 6, EPI>(a, tiles, M, st);
+        case 2: return small_launch<2, 1, 5, EPI>(a, tiles, M, st);
+        default: return small_launch<4, 2, 3, EPI>(a, tiles, M, st);
     }
 }
 

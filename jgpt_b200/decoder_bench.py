@@ -128,13 +128,13 @@ def _prefill(ctx, model, batch, seq_len, repeats):
     return float(np.median(best))
 
 
-def run_decoder(ctx, widths=(1024, 2048), batches=(1, 16, 64), prompts=((1, 2048), (8, 1024)), ctx_len=1024, steps=24, repeats=5, gpt=True):
+def run_decoder(ctx, widths=(1024, 2048), batches=(1, 16, 64), prompts=((1, 2048), (8, 1024)), ctx_len=1500, steps=24, repeats=5, models=("somopel", "gpt")):
     out = {"workload": f"{LAYERS} layers, vocabulary {VOCAB}, random weights; prefill = prompts of one call, decode at context {ctx_len}+",
            "timing": "prefill: CUDA events around the call; decode: host clock around a step that reads its ids back; medians", "sizes": []}
     for w in widths:
         row = {"width": w}
         for name, make in (("somopel", random_somopel), ("gpt", random_gpt)):
-            if name == "gpt" and not gpt:
+            if name not in models:
                 continue
             m = make(ctx, w, 8192)
             r = {}
