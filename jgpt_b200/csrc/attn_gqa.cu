@@ -326,10 +326,17 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
         __syncthreads();  // the copies below read what this CTA has just written
     }
     __nv_bfloat16 *mine = ring + (size_t)warp * ST * 32 * LD;
+    // physical blocks of this warp's next 32 pages, a page per lane: one trip to the table instead of one per page
+    int blocks = -1;
+    auto lookup = [&](int i) {
+        const int pg = pg0 + warp + 4 * (i + lane);
+        blocks = pg < pg1 ? page_of(a, sg.seq, pg * kBlockTokens) : -1;
+    };
     auto load = [&](int i) {  // the i-th page of this warp
         const int pg = pg0 + warp + 4 * i;
+        if ((i & 31) == 0) lookup(i);
+        const int phys = __shfl_sync(0xffffffffu, blocks, i & 31);
         if (pg < pg1) {
-            const int phys = page_of(a, sg.seq, pg * kBlockTokens);
             const __nv_bfloat16 *src = kv + ((size_t)(phys < 0 ? 0 : phys) * a.kv_heads + kvh) * (2 * kBlockTokens * D);
             __nv_bfloat16 *dst = mine + (size_t)(i % ST) * 32 * LD;
             for (int e = lane; e < 32 * CH; e += 32) {

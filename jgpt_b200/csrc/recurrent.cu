@@ -59,8 +59,11 @@ __device__ __forceinline__ float reduce8(const float (&lo)[4], const float (&hi)
     return (b2 ? s[1] : s[0]) + __shfl_xor_sync(0xffffffffu, b2 ? s[0] : s[1], 4);
 }
 
-template <class AT, int KIND, int DK>
-__global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const RecArgs a, const Seg *__restrict__ segs, const int *__restrict__ list,
+// SINGLE: every listed entry has one token (a decode step): no tile loop, no staging ahead, CTAs of at most 256 threads kept
+// small enough for several to share an SM, so that one's state is on its way while another computes.
+__host__ __device__ constexpr int rec_single_blocks(int DK) { return DK <= 64 ? 3 : (DK <= 128 ? 2 : 1); }
+template <class AT, int KIND, int DK, bool SINGLE>
+__global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_single_blocks(DK) : 1) recurrent_kernel(const RecArgs a, const Seg *__restrict__ segs, const int *__restrict__ list,
                                                                           int col_split, int tt,
                                                                           int pdl) {
     constexpr int NI = DK / 32;  // groups of four rows per lane
@@ -123,7 +126,7 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
     const int npairs = DK + DVc / 2;
     // raw rows of a tile into stage `buf`
     auto stage = [&](int buf, int t0) {
-        const int tn = min(tt, sgm.T - t0), per = RW / E;
+        const int tn = SINGLE ? 1 : min(tt, sgm.T - t0), per = RW / E;
         for (int e = tid; e < tn * per; e += nthreads) {
             const int t = e / per, c = (e % per) * E;
             const AT *row = proj + (size_t)(t0 + t) * a.ldp, *zr = z + (size_t)(t0 + t) * a.ldz, *src;
@@ -166,8 +169,8 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
         }
     };
     stage(0, 0);
-    for (int t0 = 0, buf = 0; t0 < sgm.T; t0 += tt, buf ^= 1) {
-        const int tn = min(tt, sgm.T - t0);
+    for (int t0 = 0, buf = 0; t0 < (SINGLE ? 1 : sgm.T); t0 += tt, buf ^= 1) {
+        const int tn = SINGLE ? 1 : min(tt, sgm.T - t0);
         const AT *raw = raw_s + (size_t)buf * tt * RW, *prev = raw_s + (size_t)(buf ^ 1) * tt * RW;
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
@@ -186,7 +189,7 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
                     y.x *= f, y.y *= f;
                     *reinterpret_cast<float2 *>(dst + t * ld) = y;
                 }
-                if (tn & 1) *reinterpret_cast<float2 *>(dst + tn * ld) = make_float2(0.f, 0.f);  // pads the last pair of tokens
+                if (!SINGLE && (tn & 1)) *reinterpret_cast<float2 *>(dst + tn * ld) = make_float2(0.f, 0.f);  // pads the last pair of tokens
             }
         }
         for (int idx = tid; idx < tn * (DK / 2); idx += nthreads) {
@@ -195,13 +198,13 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
             const float2 b = *reinterpret_cast<const float2 *>(a.decay_bias + h * DK + c);
             y.x += b.x, y.y += b.y;
             if (KIND == REC_GLA) y.x = -y.x, y.y = -y.y;  // sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau)
-            y.x = exp_f<AT>(-rate * softplus_f(y.x)), y.y = exp_f<AT>(-rate * softplus_f(y.y));
+            y.x = exp_f<AT>(-rate * softplus_f<AT>(y.x)), y.y = exp_f<AT>(-rate * softplus_f<AT>(y.y));
             *reinterpret_cast<float2 *>(sg + t * DK + c) = y;
         }
-        if (KIND == REC_GLA && (tn & 1))
+        if (!SINGLE && KIND == REC_GLA && (tn & 1))
             for (int c = tid; c < DK; c += nthreads) sg[tn * DK + c] = 1.f;
         __syncthreads();
-        if (t0 + tt < sgm.T) stage(buf ^ 1, t0 + tt);  // lands while this tile runs; the previous tile's rows are no longer needed
+        if (!SINGLE && t0 + tt < sgm.T) stage(buf ^ 1, t0 + tt);  // lands while this tile runs; the previous tile's rows are no longer needed
         if (KIND == REC_DELTA) {
             for (int t = warp; t < tn; t += nw) {
                 float qv[NI], kv[NI], qq = 0.f, kk = 0.f, qk = 0.f;
@@ -269,9 +272,9 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
             }
         } else {
             for (int t = 0; t < tn; t += 2) {
-                float of[2][4];
+                float of[2][4] = {};
 #pragma unroll
-                for (int e = 0; e < 2; e++) {
+                for (int e = 0; e < (SINGLE ? 1 : 2); e++) {
                     u64 qs[4] = {0, 0, 0, 0}, v2[4];
                     const float *qp = sq + (t + e) * DK + rl * 4, *kp = sk + (t + e) * DK + rl * 4, *gp = sg + (t + e) * DK + rl * 4;
                     const float4 v4 = *reinterpret_cast<const float4 *>(sv + (t + e) * DVc + vcol);
@@ -295,7 +298,7 @@ __global__ void __launch_bounds__(DK <= 128 ? 512 : 256) recurrent_kernel(const 
                     }
                 }
                 const float tot = reduce8(of[0], of[1], lane);
-                so[(t + (lane >> 4)) * DVc + vcol + (rl & 3)] = tot;  // row tn of an odd tile is a spare
+                if (!SINGLE || lane < 16) so[(t + (lane >> 4)) * DVc + vcol + (rl & 3)] = tot;  // row tn of an odd tile is a spare
             }
         }
         __syncthreads();
@@ -363,12 +366,11 @@ uint64_t rec_state_bytes(const RecArgs &a, int elem_bytes, uint64_t *conv_off) {
     return (s + conv + 255) / 256 * 256;
 }
 
-template <class AT, int KIND, int DK>
-static int32_t rec_launch(const StepDesc &d, const RecArgs &a, int pdl, int *split_out, cudaStream_t st) {
-    const bool single = d.n_tiles == 0;
-    if (d.n_short == 0) return JGPT_OK;
+template <class AT, int KIND, int DK, bool SINGLE>
+static int32_t rec_launch_form(const StepDesc &d, const RecArgs &a, int pdl, int *split_out, cudaStream_t st) {
+    const bool single = SINGLE;
     const int tt = single ? 2 : kTileTokens;
-    const int groups = a.DV / 16, max_groups = DK <= 128 ? 16 : 8;
+    const int groups = a.DV / 16, max_groups = DK <= 128 && !SINGLE ? 16 : 8;
     int split = 1;
     auto allowed = [&](int s) { return groups % s == 0; };
     while (split < groups && (!allowed(split) || groups / split > max_groups)) split++;
@@ -379,7 +381,7 @@ static int32_t rec_launch(const StepDesc &d, const RecArgs &a, int pdl, int *spl
         return sizeof(float) * ((size_t)tokens * row + 2 * tokens) + (size_t)stages * tokens * (row * sizeof(AT) + (KIND == REC_DELTA ? 16 : 0));
     };
     const size_t smem = smem_bytes(tt, DVc, single ? 1 : 2);
-    auto kern = recurrent_kernel<AT, KIND, DK>;
+    auto kern = recurrent_kernel<AT, KIND, DK, SINGLE>;
     static thread_local int set_for = -1;
     int dev = 0;
     JGPT_CUDA_TRY(cudaGetDevice(&dev));
@@ -395,6 +397,14 @@ static int32_t rec_launch(const StepDesc &d, const RecArgs &a, int pdl, int *spl
     cfg.dynamicSmemBytes = smem, cfg.stream = st, cfg.attrs = attr, cfg.numAttrs = (pdl & 1) ? 1 : 0;
     JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, kern, a, d.segs, d.short_segs, split, tt, pdl));
     return JGPT_OK;
+}
+
+template <class AT, int KIND, int DK>
+static int32_t rec_launch(const StepDesc &d, const RecArgs &a, int pdl, int *split_out, cudaStream_t st) {
+    if (d.n_short == 0) return JGPT_OK;
+    // heads wider than a single-token CTA's 128 columns keep the tile form, which normalises them without a second kernel
+    if (d.n_tiles == 0 && (a.DV <= 128 || DK > 128)) return rec_launch_form<AT, KIND, DK, true>(d, a, pdl, split_out, st);
+    return rec_launch_form<AT, KIND, DK, false>(d, a, pdl, split_out, st);
 }
 
 template <class AT, int KIND>

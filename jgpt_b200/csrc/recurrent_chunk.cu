@@ -172,7 +172,7 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
             const float2 b = *reinterpret_cast<const float2 *>(a.decay_bias + h * DK + c);
             y.x = zr[e].x + b.x, y.y = zr[e].y + b.y;
             if (KIND == REC_GLA) y.x = -y.x, y.y = -y.y;
-            y.x = exp_f<AT>(-rate * softplus_f(y.x)), y.y = exp_f<AT>(-rate * softplus_f(y.y));
+            y.x = exp_f<AT>(-rate * softplus_f<AT>(y.x)), y.y = exp_f<AT>(-rate * softplus_f<AT>(y.y));
         }
         *reinterpret_cast<float2 *>(sg + t * DK + c) = y;
     }

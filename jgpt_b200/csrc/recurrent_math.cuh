@@ -27,7 +27,12 @@ template <class AT>
 __device__ __forceinline__ float sigmoid_f(float x) {
     return sizeof(AT) == 4 ? 1.f / (1.f + expf(-x)) : __fdividef(1.f, 1.f + __expf(-x));
 }
-__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// log(1 + e^x).  bf16 mode: the fast logarithm; its absolute error (~1e-7, the rounding of a decay near 1) is what counts in
+// an exponent.
+template <class AT>
+__device__ __forceinline__ float softplus_f(float x) {
+    return fmaxf(x, 0.f) + (sizeof(AT) == 4 ? log1pf(expf(-fabsf(x))) : __logf(1.f + __expf(-fabsf(x))));
+}
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int off = 16; off >= 1; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
