@@ -9,8 +9,7 @@
 //     u_i + beta_i sum_{j<i} A_ij u_j = beta_i (v_i - (k_i b_i)^T S0)     i.e.  U = T V - (T K~) S0,  T = (I + diag(beta) A)^-1 diag(beta)
 //     o_i = (q_i b_i)^T S0 + sum_{j<=i} P_ij u_j
 //     S   = diag(b_16) S0 + sum_j (k_j b_16,j) u_j^T
-// the chunkwise form of linear attention and of the delta rule (WY representation) as published for gated linear attention
-// and gated delta networks, here with per-channel products kept in their safe form.
+// which follows from unrolling the rules over the chunk.
 //
 // Two kernels.  rec_prep_kernel, parallel over all chunks and heads: convolution, unit vectors, decays, and everything above
 // that does not involve S0, written as one record per (chunk, head).  rec_scan_kernel, serial over the chunks of a sequence
