@@ -335,14 +335,23 @@ JGPT_API int32_t jgpt_generate_greedy_rolling(jgpt_model model, jgpt_kvpool pool
  * scheduler and jgpt_model_destroy take it; entry points that need the fixed block return
  * JGPT_ERR_UNSUPPORTED.  The reference has one block design only (J/model/DecoderBlock.java).
  *
- * A layer is x += sum over its branches of out_scale * mixer(LN1(x)), then x += ff(LN2(x)) when ff > 0;
- * norms are layer norms with weight and bias, ff is W_down (gelu_tanh(W_gate h) * (W_up h)).
+ * A layer is x += m * ls1 * sum over its branches of out_scale * mixer(norm1(x)), then x += m * ls2 * ff(norm2(x)) when ff > 0;
+ * norms are layer norms with weight and bias or RMS norms with weight, m is residual_mult, the factors per column ls1, ls2 are
+ * there with layer_scale.  With depth_average what goes on from layer i is sum over j <= i + 1 of dwa_i[j] X_j, X_0 the
+ * embedding and X_(i+1) the result of layer i.
  * ------------------------------------------------------------------------------------------- */
 enum {
     JGPT_MIX_ATTENTION = 1, /* softmax attention over paged K/V, no rotation, positions of the query's chunk only */
     JGPT_MIX_GLA = 2,       /* gated linear attention: S <- diag(a) S + k v^T, a = sigmoid(W_a2 W_a1 h + bias)^(1/tau) */
-    JGPT_MIX_DELTA = 3      /* gated delta rule with a decay per key channel and short convolutions on q, k, v */
+    JGPT_MIX_DELTA = 3,     /* gated delta rule with a decay per key channel and short convolutions on q, k, v */
+    JGPT_MIX_HGRN2 = 4,     /* S <- diag(f) S + (1 - f) v^T, f = l + (1 - l) sigmoid(W_f h + bias); no output gate */
+    JGPT_MIX_WKV = 5,       /* o = (S + diag(u) k v^T)^T r, S <- diag(w) S + k v^T, w = exp(-exp(W_a2 tanh(W_a1 h_w) + bias)); r, k,
+                               v, g and w each read their own mix of h with the previous token's h; only layer norm kind RMS */
+    JGPT_MIX_LATENT = 6     /* softmax attention on a normed latent and one rotated key part shared by the heads, sliding window */
 };
+enum { JGPT_NORM_LAYER = 0, JGPT_NORM_RMS = 1 };
+enum { JGPT_FF_GATED_GELU = 0 /* W_down (gelu_tanh(W_gate h) * (W_up h)) */,
+       JGPT_FF_XIELU = 1 /* W_down xielu(W_up h), xielu(z) = a z^2 + z / 2 (z > 0), b (e^z - 1 - z) + z / 2, a = softplus(p), b = 1/2 + softplus(q) */ };
 enum { JGPT_DTYPE_BF16 = 0, /* bf16 products, activations and K/V; norms, scores, recurrences and the residual in fp32 */
        JGPT_DTYPE_F32 = 1 /* everything in fp32 (no reduced-precision matrix mode) */ };
 #define JGPT_MAX_BRANCHES 2
@@ -357,23 +366,43 @@ typedef struct {
     float score_scale;        /* attention */
     float tau;                /* gla */
     float out_scale;
+    int32_t window;           /* latent: position i sees j with 0 <= i - j < window; 0: every j <= i */
+    int32_t q_rank, kv_rank;  /* latent: sizes of the query and key latents (kv_rank up to 512) */
+    int32_t rot_dim;          /* latent: size of the rotated part of a query head and of the shared key part (up to 128) */
+    int32_t rot_dims;         /* of it the first rot_dims turn: dimension i with i + rot_dims / 2 */
+    int32_t kv_from;          /* latent: 0: a cache of its own; 1 + j: the cache of layer j */
+    double rot_base;          /* frequencies base^(-2 i / rot_dims) */
+    double rot_factor, rot_original, rot_fast, rot_slow; /* YaRN: slow dimensions divided by factor, cos and sin times 0.1 ln(factor) + 1;
+                                                            rot_factor 0: plain rotation */
 } jgpt_mixer_spec;
 typedef struct {
     int32_t n_branches;
     jgpt_mixer_spec branch[JGPT_MAX_BRANCHES];
-    int32_t ff; /* 0: no feed-forward part */
+    int32_t ff;      /* 0: no feed-forward part */
+    int32_t ff_kind; /* JGPT_FF_* */
 } jgpt_layer_spec;
 typedef struct {
     int32_t vocab, width, max_positions, n_layers;
     int32_t embed_norm; /* layer norm behind the embedding */
+    int32_t pos_table;     /* learned positions [max_positions, width] are added to the embedding */
+    int32_t norm;          /* JGPT_NORM_* (RMS: without pos_table and embed_norm) */
+    int32_t head;          /* logits from a matrix of their own (JGPT_W_HEAD) instead of the embedding */
+    int32_t layer_scale;   /* JGPT_W_LS1 / _LS2 (RMS only) */
+    int32_t depth_average; /* JGPT_W_DWA (RMS only) */
     float eps, embed_scale, logit_scale;
+    float residual_mult;
 } jgpt_decoder_spec;
 /* Tensors.  Of the model: layer = branch = -1; of a layer: branch = -1; of a mixer: layer and branch. */
 enum {
     JGPT_W_EMBED = 0, JGPT_W_POS, JGPT_W_EMBED_NORM, JGPT_W_EMBED_NORM_B, JGPT_W_FINAL_NORM, JGPT_W_FINAL_NORM_B,
+    JGPT_W_HEAD,
     JGPT_W_NORM1 = 10, JGPT_W_NORM1_B, JGPT_W_NORM2, JGPT_W_NORM2_B, JGPT_W_FF_GATE, JGPT_W_FF_UP, JGPT_W_FF_DOWN,
+    JGPT_W_LS1, JGPT_W_LS2, JGPT_W_DWA /* [layer + 2] */,
     JGPT_W_Q = 20, JGPT_W_K, JGPT_W_V, JGPT_W_O, JGPT_W_G /* output gate */, JGPT_W_B /* step size */, JGPT_W_A1, JGPT_W_A2,
-    JGPT_W_DECAY_BIAS, JGPT_W_A_LOG, JGPT_W_G1, JGPT_W_G2, JGPT_W_HEAD_NORM, JGPT_W_CONV_Q, JGPT_W_CONV_K, JGPT_W_CONV_V
+    JGPT_W_DECAY_BIAS, JGPT_W_A_LOG, JGPT_W_G1, JGPT_W_G2, JGPT_W_HEAD_NORM, JGPT_W_CONV_Q, JGPT_W_CONV_K, JGPT_W_CONV_V,
+    JGPT_W_MU_R, JGPT_W_MU_K, JGPT_W_MU_V, JGPT_W_MU_G, JGPT_W_MU_W, JGPT_W_BONUS /* u */, JGPT_W_LOWER /* l */, JGPT_W_F,
+    JGPT_W_DQ, JGPT_W_DQ_NORM, JGPT_W_UQ, JGPT_W_DKV, JGPT_W_DKV_NORM, JGPT_W_UK, JGPT_W_UV,
+    JGPT_W_FF_ACT /* of a layer: p, q */
 };
 
 /* max_rows bounds the rows (tokens) of one step. */

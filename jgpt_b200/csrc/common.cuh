@@ -66,9 +66,10 @@ struct SeqState {
 
 constexpr int kBlockTokens = 16;
 
-// Pages of one attention layer of a layered pool: [n_blocks][heads][K 16 x dim | V 16 x dim] elements at `offset` bytes.
+// Pages of one attention layer of a layered pool: [n_blocks][heads][K 16 x dim | V 16 x dim] elements at `offset` bytes, or
+// (parts == 1) one row of dim elements per token.
 struct KvLayerGeom {
-    int heads = 0, dim = 0;
+    int heads = 0, dim = 0, parts = 2;
     uint64_t offset = 0, block_bytes = 0;
 };
 

@@ -7,6 +7,10 @@
 //
 //   LN1 -> proj = h W_in^T -> [z = low-rank second factors] -> mixer kernels -> x += mixed W_out^T -> LN2 -> gelu pair -> x += act W_down^T
 //
+// With RMS norms the residual may be an average over the depth: every layer's result stays in a slot of its own, the norm in front of the
+// next layer forms the weighted sum on its way, and the product epilogues add (times the layer scale) to the slot.  A WKV layer's
+// norm writes five mixes with the previous token's row, which its input projections read as segments of one product.
+//
 // The residual x is fp32; rows entering a product are bf16 (or fp32 in the exact mode).  Head sizes are padded with zero
 // weights to what the kernels take, so every size of a configuration works; sums over a head use the true size.
 #include "decoder.cuh"
@@ -34,6 +38,16 @@ struct DBranch {
     void *w_a2 = nullptr, *w_g2 = nullptr;  // [heads * DK, ra], [heads * DV, rg]
     float *bias = nullptr, *a_log = nullptr, *norm = nullptr, *conv_q = nullptr, *conv_k = nullptr, *conv_v = nullptr;
     uint64_t have = 0;
+    float *bonus = nullptr, *lower = nullptr, *mu = nullptr;  // WKV [heads * DK], HGRN2 [heads * DK], WKV [5][width]
+    int f = -1;                                               // HGRN2: forget gate's columns in proj
+    // latent attention
+    int dq = -1, dkv = -1, dkr = -1;      // columns in proj: query latent, key latent, rotated key part
+    int DP = 0, DQ = 0, KR = 0, RR = 0, LDR = 0, qrp = 0;  // padded: head (unrotated), query head, latent, rotated part, page row, query latent
+    int rot = -1;                         // which rotation of the model
+    bool expand = false;                  // its head sizes have a written-out form
+    void *w_uq = nullptr, *w_absorb = nullptr, *w_ukv = nullptr;  // [heads * DQ, qrp], [heads * KR, DP], [heads * (DP + DV), KR]
+    float *dq_norm = nullptr, *dkv_norm = nullptr;
+    bool recurrent() const { return s.kind == JGPT_MIX_GLA || s.kind == JGPT_MIX_DELTA || s.kind == JGPT_MIX_HGRN2 || s.kind == JGPT_MIX_WKV; }
     int cols() const { return s.heads * (s.kind == JGPT_MIX_ATTENTION ? D : DV); }
 };
 
@@ -42,7 +56,11 @@ struct DLayer {
     int ff = 0, ffp = 0, n_in = 0, n_out = 0, n_z = 0;
     void *w_in = nullptr, *w_out = nullptr, *w_gu = nullptr, *w_down = nullptr;
     float *n1w = nullptr, *n1b = nullptr, *n2w = nullptr, *n2b = nullptr;
+    int ff_kind = 0;
+    float act_p0 = 0.f, act_p1 = 0.f;
+    float *ls1 = nullptr, *ls2 = nullptr, *dwa = nullptr;  // residual_mult x layer scale; depth average
     uint64_t have = 0;
+    const DBranch *shift() const { return br[0].s.kind == JGPT_MIX_WKV ? &br[0] : nullptr; }  // its input projections read mixes
 };
 
 struct Decoder {
@@ -51,7 +69,14 @@ struct Decoder {
     bool f32 = false;
     int eb = 2, R = 0, ldw = 0;  // element bytes, rows per step, padded width
     std::vector<DLayer> L;
-    void *embed = nullptr, *pos = nullptr;
+    void *embed = nullptr, *pos = nullptr, *head = nullptr;
+    bool rms = false;
+    std::vector<mix::Rotation> rots;
+    std::vector<jgpt_mixer_spec> rot_specs;
+    int max_window = 0;                // largest window of the latent layers (0: unbounded)
+    int lat_min = 0, kvx_rows = 0;     // entries of at least lat_min tokens run latent attention written out, in kvx_rows workspace rows
+    void *cq = nullptr, *q = nullptr, *qa = nullptr, *cx = nullptr, *kvx = nullptr;
+    float *slots = nullptr;            // [layers + 1][rows][width] with depth averages
     float *enw = nullptr, *enb = nullptr, *fnw = nullptr, *fnb = nullptr;
     uint64_t have = 0;
     std::vector<KvLayerGeom> kv;
@@ -120,13 +145,68 @@ int32_t decoder_destroy(Decoder *d) {
 
 static mix::RecArgs rec_args(const DBranch &b) {
     mix::RecArgs a{};
-    a.kind = b.s.kind == JGPT_MIX_DELTA ? mix::REC_DELTA : mix::REC_GLA;
+    a.kind = b.s.kind == JGPT_MIX_DELTA ? mix::REC_DELTA : b.s.kind == JGPT_MIX_HGRN2 ? mix::REC_HGRN2 : b.s.kind == JGPT_MIX_WKV ? mix::REC_WKV : mix::REC_GLA;
     a.q_off = b.q, a.k_off = b.k, a.v_off = b.v, a.b_off = b.b, a.g_off = b.g, a.z_off = b.za, a.zg_off = b.zg;
     a.heads = b.s.heads, a.kv_heads = b.s.kv_heads, a.DK = b.DK, a.DV = b.DV, a.dim = b.s.dim, a.vdim = b.s.vdim;
     a.tau = b.s.tau, a.out_scale = b.s.out_scale, a.taps = b.s.kind == JGPT_MIX_DELTA ? b.s.taps : 0;
     a.conv_q = b.conv_q, a.conv_k = b.conv_k, a.conv_v = b.conv_v, a.decay_bias = b.bias, a.a_log = b.a_log, a.norm_w = b.norm;
     a.conv_off = b.conv_off, a.out_off = b.out;
+    a.norm_stride = b.s.kind == JGPT_MIX_WKV ? b.DV : 0, a.bonus = b.bonus, a.lower = b.lower;
+    if (b.s.kind == JGPT_MIX_HGRN2) a.z_off = b.f;
     return a;
+}
+
+// Source row i lands in row (i / rgroup) * rpad + i % rgroup, columns likewise: padding per head.
+struct Grouping {
+    int group = 0, pad = 0;  // group == 0: no grouping
+    int at(int i) const { return group ? i / group * pad + i % group : i; }
+};
+
+static int32_t put_matrix(Decoder *d, void *dst, int ld, int row0, int col0, const float *src, int rows, int cols, Grouping rg, Grouping cg) {
+    const int last = rg.at(rows - 1) + 1;
+    const int width = cg.at(cols - 1) + 1;
+    std::vector<uint8_t> buf((size_t)last * width * d->eb, 0);
+    for (int r = 0; r < rows; r++)
+        for (int c = 0; c < cols; c++) {
+            const size_t o = (size_t)rg.at(r) * width + cg.at(c);
+            const float v = src[(size_t)r * cols + c];
+            if (d->f32) reinterpret_cast<float *>(buf.data())[o] = v;
+            else reinterpret_cast<__nv_bfloat16 *>(buf.data())[o] = __float2bfloat16(v);
+        }
+    JGPT_CUDA_TRY(cudaMemcpy2DAsync(reinterpret_cast<uint8_t *>(dst) + ((size_t)row0 * ld + col0) * d->eb, (size_t)ld * d->eb, buf.data(),
+                                    (size_t)width * d->eb, (size_t)width * d->eb, (size_t)last, cudaMemcpyHostToDevice, d->ctx->stream));
+    JGPT_CUDA_TRY(cudaStreamSynchronize(d->ctx->stream));
+    return JGPT_OK;
+}
+static int32_t put_floats(Decoder *d, float *dst, const float *src, int rows, int cols, Grouping rg) {
+    std::vector<float> buf((size_t)(rg.at(rows - 1) + 1) * cols, 0.f);
+    for (int r = 0; r < rows; r++) std::copy(src + (size_t)r * cols, src + (size_t)(r + 1) * cols, buf.begin() + (size_t)rg.at(r) * cols);
+    JGPT_CUDA_TRY(cudaMemcpyAsync(dst, buf.data(), sizeof(float) * buf.size(), cudaMemcpyHostToDevice, d->ctx->stream));
+    JGPT_CUDA_TRY(cudaStreamSynchronize(d->ctx->stream));
+    return JGPT_OK;
+}
+
+// Angles of a rotation: frequencies on the device, the magnitude of cos and sin.
+static int32_t add_rotation(Decoder *d, const jgpt_mixer_spec &s) {
+    const int half = s.rot_dims / 2;
+    std::vector<double> f((size_t)half);
+    auto dim_of = [&](double turns) { return s.rot_dims * std::log(s.rot_original / (2 * M_PI * turns)) / (2 * std::log(s.rot_base)); };
+    const bool yarn = s.rot_factor > 0;
+    const double lo = yarn ? std::max(std::floor(dim_of(s.rot_fast)), 0.0) : 0, hi = yarn ? std::min(std::ceil(dim_of(s.rot_slow)), s.rot_dims - 1.0) : 0;
+    for (int i = 0; i < half; i++) {
+        f[(size_t)i] = std::pow(s.rot_base, -2.0 * i / s.rot_dims);
+        if (!yarn) continue;
+        const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+        f[(size_t)i] = f[(size_t)i] / s.rot_factor * ramp + f[(size_t)i] * (1 - ramp);
+    }
+    mix::Rotation r{};
+    void *dev = nullptr;
+    TRY(dalloc(d, &dev, sizeof(double) * f.size()));
+    JGPT_CUDA_TRY(cudaMemcpyAsync(dev, f.data(), sizeof(double) * f.size(), cudaMemcpyHostToDevice, d->ctx->stream));
+    JGPT_CUDA_TRY(cudaStreamSynchronize(d->ctx->stream));
+    r.freq = (const double *)dev, r.half = half, r.mag = yarn ? (float)(0.1 * std::log(s.rot_factor) + 1.0) : 1.f;
+    d->rots.push_back(r), d->rot_specs.push_back(s);
+    return JGPT_OK;
 }
 
 // Sizes, column layouts and device memory of one layer.
@@ -184,19 +264,95 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
             }
             b.state_off = d->state_stride;
             d->state_stride += mix::rec_state_bytes(rec_args(b), eb, &b.conv_off);
+        } else if (s.kind == JGPT_MIX_HGRN2 || s.kind == JGPT_MIX_WKV) {
+            const bool wkv = s.kind == JGPT_MIX_WKV;
+            JGPT_REQUIRE(s.kv_heads == s.heads && (!wkv || (s.vdim == s.dim && s.rank_a > 0)), JGPT_ERR_INVALID_ARGUMENT,
+                         "layer %d: heads %d / %d, head sizes %d / %d, rank %d", index, s.heads, s.kv_heads, s.dim, s.vdim, s.rank_a);
+            JGPT_REQUIRE(!wkv || (ls.n_branches == 1 && d->rms), JGPT_ERR_UNSUPPORTED, "layer %d: WKV stands alone in its layer, behind an RMS norm", index);
+            b.DK = mix::rec_padded_key(s.dim), b.DV = wkv ? b.DK : mix::rec_padded_value(s.vdim);
+            JGPT_REQUIRE(b.DK > 0 && b.DV > 0, JGPT_ERR_UNSUPPORTED, "layer %d: head sizes %d / %d", index, s.dim, s.vdim);
+            const int hk = s.heads * b.DK;
+            b.q = seg(hk);
+            if (wkv) b.k = seg(hk);
+            b.v = seg(s.heads * b.DV);
+            TRY(dalloc(d, (void **)&b.bias, sizeof(float) * (uint64_t)hk));
+            TRY(dalloc(d, (void **)&b.norm, sizeof(float) * (uint64_t)b.DV * (wkv ? s.heads : 1)));
+            if (wkv) {
+                b.g = seg(hk);
+                b.ra = up(s.rank_a, 8), b.a1 = seg(s.rank_a);
+                b.za = zc, zc += hk;
+                TRY(dalloc(d, &b.w_a2, (uint64_t)hk * b.ra * eb));
+                TRY(dalloc(d, (void **)&b.bonus, sizeof(float) * (uint64_t)hk));
+                TRY(dalloc(d, (void **)&b.mu, sizeof(float) * 5 * (uint64_t)W));
+            } else {
+                b.f = seg(hk);
+                TRY(dalloc(d, (void **)&b.lower, sizeof(float) * (uint64_t)hk));
+            }
+            b.state_off = d->state_stride;
+            mix::RecArgs ra = rec_args(b);
+            ra.shift_width = wkv ? W : 0;
+            d->state_stride += mix::rec_state_bytes(ra, eb, &b.conv_off);
+        } else if (s.kind == JGPT_MIX_LATENT) {
+            JGPT_REQUIRE(s.q_rank > 0 && s.kv_rank > 0 && s.window >= 0 && s.rot_dims > 0 && s.rot_dims % 2 == 0 && s.rot_dims <= s.rot_dim && s.rot_base > 1.0,
+                         JGPT_ERR_INVALID_ARGUMENT, "layer %d: latents of %d / %d, window %d, rotation of %d / %d", index, s.q_rank, s.kv_rank, s.window,
+                         s.rot_dims, s.rot_dim);
+            b.KR = mix::latent_padded_rank(s.kv_rank), b.RR = mix::latent_padded_rot(s.rot_dim), b.LDR = b.KR + b.RR + 8;
+            JGPT_REQUIRE(b.KR > 0 && b.RR > 0, JGPT_ERR_UNSUPPORTED, "layer %d: latent of %d, rotated part of %d", index, s.kv_rank, s.rot_dim);
+            b.DP = up(s.dim, 8), b.DQ = b.DP + up(s.rot_dim, 8), b.DV = up(s.vdim, 8), b.qrp = up(s.q_rank, 8);
+            b.expand = !d->f32 && mix::latent_expandable(s.dim, s.rot_dim, s.vdim);
+            b.dq = seg(s.q_rank);
+            auto same_rotation = [&](const jgpt_mixer_spec &x) {
+                return x.rot_dims == s.rot_dims && x.rot_base == s.rot_base && x.rot_factor == s.rot_factor && x.rot_original == s.rot_original &&
+                       x.rot_fast == s.rot_fast && x.rot_slow == s.rot_slow;
+            };
+            if (s.kv_from == 0) {
+                b.dkv = seg(s.kv_rank), b.dkr = seg(s.rot_dim);
+                b.kv_layer = (int)d->kv.size();
+                KvLayerGeom geom;
+                geom.heads = 1, geom.dim = b.LDR, geom.parts = 1;
+                d->kv.push_back(geom);
+                TRY(dalloc(d, (void **)&b.dkv_norm, sizeof(float) * (uint64_t)s.kv_rank));
+            } else {
+                JGPT_REQUIRE(s.kv_from >= 1 && s.kv_from <= index, JGPT_ERR_INVALID_ARGUMENT, "layer %d reads the cache of layer %d", index, s.kv_from - 1);
+                const DBranch *from = nullptr;
+                for (const DBranch &x : d->L[(size_t)s.kv_from - 1].br)
+                    if (x.s.kind == JGPT_MIX_LATENT && x.s.kv_from == 0) from = &x;
+                JGPT_REQUIRE(from && from->s.kv_rank == s.kv_rank && from->s.rot_dim == s.rot_dim && same_rotation(from->s), JGPT_ERR_INVALID_ARGUMENT,
+                             "layer %d: layer %d has no cache of its sizes and rotation", index, s.kv_from - 1);
+                b.kv_layer = from->kv_layer;
+            }
+            for (size_t k = 0; k < d->rot_specs.size() && b.rot < 0; k++)
+                if (same_rotation(d->rot_specs[k])) b.rot = (int)k;
+            if (b.rot < 0) {
+                JGPT_REQUIRE(d->rots.size() < mix::kMaxRotations, JGPT_ERR_UNSUPPORTED, "more than %d different rotations", mix::kMaxRotations);
+                b.rot = (int)d->rots.size();
+                TRY(add_rotation(d, ls.branch[i]));
+            }
+            TRY(dalloc(d, &b.w_uq, (uint64_t)s.heads * b.DQ * b.qrp * eb));
+            TRY(dalloc(d, &b.w_absorb, (uint64_t)s.heads * b.KR * b.DP * eb));
+            TRY(dalloc(d, &b.w_ukv, (uint64_t)s.heads * (b.DP + b.DV) * b.KR * eb));
+            TRY(dalloc(d, (void **)&b.dq_norm, sizeof(float) * (uint64_t)s.q_rank));
         } else {
             return fail(JGPT_ERR_UNSUPPORTED, "layer %d: mixer kind %d", index, s.kind);
         }
         out += b.cols();
         y.br.push_back(b);
     }
-    y.n_in = in, y.n_out = up(out, 8), y.n_z = zc, y.ff = ls.ff, y.ffp = up(ls.ff, 16);
+    y.n_in = in, y.n_out = up(out, 8), y.n_z = zc, y.ff = ls.ff, y.ffp = up(ls.ff, 16), y.ff_kind = ls.ff_kind;
+    JGPT_REQUIRE(ls.ff_kind == JGPT_FF_GATED_GELU || ls.ff_kind == JGPT_FF_XIELU, JGPT_ERR_UNSUPPORTED, "layer %d: feed-forward kind %d", index, ls.ff_kind);
+    if (d->rms) {
+        TRY(dalloc(d, (void **)&y.ls1, sizeof(float) * (uint64_t)W));
+        TRY(dalloc(d, (void **)&y.ls2, sizeof(float) * (uint64_t)W));
+        const std::vector<float> mult((size_t)W, d->s.residual_mult);
+        for (float *p : {y.ls1, y.ls2}) TRY(put_floats(d, p, mult.data(), 1, W, Grouping()));
+    }
+    if (d->s.depth_average) TRY(dalloc(d, (void **)&y.dwa, sizeof(float) * (uint64_t)(index + 2)));
     TRY(dalloc(d, &y.w_in, (uint64_t)y.n_in * d->ldw * eb));
     TRY(dalloc(d, &y.w_out, (uint64_t)W * y.n_out * eb));
     TRY(dalloc(d, (void **)&y.n1w, sizeof(float) * (uint64_t)W));
     TRY(dalloc(d, (void **)&y.n1b, sizeof(float) * (uint64_t)W));
     if (y.ff) {
-        TRY(dalloc(d, &y.w_gu, 2ull * y.ffp * d->ldw * eb));
+        TRY(dalloc(d, &y.w_gu, (y.ff_kind == JGPT_FF_GATED_GELU ? 2ull : 1ull) * y.ffp * d->ldw * eb));
         TRY(dalloc(d, &y.w_down, (uint64_t)W * y.ffp * eb));
         TRY(dalloc(d, (void **)&y.n2w, sizeof(float) * (uint64_t)W));
         TRY(dalloc(d, (void **)&y.n2b, sizeof(float) * (uint64_t)W));
@@ -204,19 +360,28 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
     return JGPT_OK;
 }
 
-static size_t desc_ints(const Decoder *d) { return 18 * (size_t)d->R + 64; }
+static size_t desc_ints(const Decoder *d) { return 28 * (size_t)d->R + 128; }
 
 static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
     const uint64_t R = d->R, W = d->s.width, eb = d->eb;
     d->L.resize((size_t)d->s.n_layers);
     d->long_min = mix::rec_chunk_min_tokens(d->f32);
-    int n_in = 8, n_z = 8, n_out = 8, ffp = 16, raw = 0;
+    d->rms = d->s.norm == JGPT_NORM_RMS;
+    d->lat_min = env_int("JGPT_B200_LATENT_EXPAND_MIN", 64);
+    int n_in = 8, n_z = 8, n_out = 8, ffp = 16, raw = 0, mixes = 1, cq = 0, lq = 0, lqa = 0, cxw = 0, kvx = 0;
+    bool latent = false, unbounded = false, expand = true;
     for (int i = 0; i < d->s.n_layers; i++) {
         DLayer &y = d->L[(size_t)i];
         TRY(plan_layer(d, y, layers[i], i));
         n_in = std::max(n_in, y.n_in), n_z = std::max(n_z, y.n_z), n_out = std::max(n_out, y.n_out), ffp = std::max(ffp, y.ffp);
         for (const DBranch &b : y.br) {
-            if (b.s.kind == JGPT_MIX_ATTENTION) continue;
+            if (b.s.kind == JGPT_MIX_WKV) mixes = 5;
+            if (b.s.kind == JGPT_MIX_LATENT) {
+                latent = true, unbounded = unbounded || b.s.window == 0, d->max_window = std::max(d->max_window, b.s.window);
+                cq = std::max(cq, b.qrp), lq = std::max(lq, b.s.heads * b.DQ), lqa = std::max(lqa, b.s.heads * b.KR), cxw = std::max(cxw, b.KR + b.RR);
+                kvx = std::max(kvx, b.s.heads * (b.DP + b.DV)), expand = expand && b.expand;
+            }
+            if (!b.recurrent()) continue;
             raw = std::max(raw, b.s.heads * b.DV);
             if (const int t = d->long_min)
                 d->chunk_ws_floats = std::max(d->chunk_ws_floats, (uint64_t)(d->R / mix::kRecChunk + d->R / t + 1) * b.s.heads *
@@ -224,12 +389,27 @@ static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
         }
     }
     TRY(dalloc(d, &d->embed, (uint64_t)d->s.vocab * d->ldw * eb));
-    TRY(dalloc(d, &d->pos, (uint64_t)d->s.max_positions * d->ldw * eb));
+    if (d->s.pos_table) TRY(dalloc(d, &d->pos, (uint64_t)d->s.max_positions * d->ldw * eb));
+    if (d->s.head) TRY(dalloc(d, &d->head, (uint64_t)d->s.vocab * d->ldw * eb));
     for (float **p : {&d->enw, &d->enb, &d->fnw, &d->fnb}) TRY(dalloc(d, (void **)p, sizeof(float) * W));
     TRY(dalloc(d, (void **)&d->x, sizeof(float) * R * W));
+    if (d->s.depth_average) TRY(dalloc(d, (void **)&d->slots, sizeof(float) * (d->L.size() + 1) * R * W));
+    for (mix::Rotation &r : d->rots) TRY(dalloc(d, (void **)&r.out, sizeof(float2) * R * r.half));
+    if (unbounded) d->max_window = 0;
+    if (!latent || !expand) d->lat_min = 0;
+    if (latent) {
+        TRY(dalloc(d, &d->cq, R * cq * eb));
+        TRY(dalloc(d, &d->q, R * lq * eb));
+        TRY(dalloc(d, &d->qa, R * lqa * eb));
+        if (d->lat_min > 0) {
+            d->kvx_rows = 2 * d->R;
+            TRY(dalloc(d, &d->cx, (uint64_t)d->kvx_rows * cxw * eb));
+            TRY(dalloc(d, &d->kvx, (uint64_t)d->kvx_rows * kvx * eb));
+        }
+    }
     TRY(dalloc(d, (void **)&d->raw, sizeof(float) * R * raw));
     TRY(dalloc(d, (void **)&d->chunk_ws, sizeof(float) * d->chunk_ws_floats));
-    TRY(dalloc(d, &d->h, R * d->ldw * eb));
+    TRY(dalloc(d, &d->h, R * mixes * d->ldw * eb));
     TRY(dalloc(d, &d->proj, R * n_in * eb));
     TRY(dalloc(d, &d->z, R * n_z * eb));
     TRY(dalloc(d, &d->mixed, R * n_out * eb));
@@ -250,39 +430,17 @@ static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
 // ------------------------------------------------------------------------------------------------
 // Weights
 // ------------------------------------------------------------------------------------------------
-// Source row i lands in row (i / rgroup) * rpad + i % rgroup, columns likewise: padding per head.
-struct Grouping {
-    int group = 0, pad = 0;  // group == 0: no grouping
-    int at(int i) const { return group ? i / group * pad + i % group : i; }
-};
-
-static int32_t put_matrix(Decoder *d, void *dst, int ld, int row0, int col0, const float *src, int rows, int cols, Grouping rg, Grouping cg) {
-    const int last = rg.at(rows - 1) + 1;
-    const int width = cg.at(cols - 1) + 1;
-    std::vector<uint8_t> buf((size_t)last * width * d->eb, 0);
-    for (int r = 0; r < rows; r++)
-        for (int c = 0; c < cols; c++) {
-            const size_t o = (size_t)rg.at(r) * width + cg.at(c);
-            const float v = src[(size_t)r * cols + c];
-            if (d->f32) reinterpret_cast<float *>(buf.data())[o] = v;
-            else reinterpret_cast<__nv_bfloat16 *>(buf.data())[o] = __float2bfloat16(v);
-        }
-    JGPT_CUDA_TRY(cudaMemcpy2DAsync(reinterpret_cast<uint8_t *>(dst) + ((size_t)row0 * ld + col0) * d->eb, (size_t)ld * d->eb, buf.data(),
-                                    (size_t)width * d->eb, (size_t)width * d->eb, (size_t)last, cudaMemcpyHostToDevice, d->ctx->stream));
-    JGPT_CUDA_TRY(cudaStreamSynchronize(d->ctx->stream));
-    return JGPT_OK;
-}
-static int32_t put_floats(Decoder *d, float *dst, const float *src, int rows, int cols, Grouping rg) {
-    std::vector<float> buf((size_t)(rg.at(rows - 1) + 1) * cols, 0.f);
-    for (int r = 0; r < rows; r++) std::copy(src + (size_t)r * cols, src + (size_t)(r + 1) * cols, buf.begin() + (size_t)rg.at(r) * cols);
-    JGPT_CUDA_TRY(cudaMemcpyAsync(dst, buf.data(), sizeof(float) * buf.size(), cudaMemcpyHostToDevice, d->ctx->stream));
-    JGPT_CUDA_TRY(cudaStreamSynchronize(d->ctx->stream));
-    return JGPT_OK;
-}
-
 static uint64_t bit(int role) { return 1ull << role; }
 
 static uint64_t needed_roles(const jgpt_mixer_spec &s) {
+    if (s.kind == JGPT_MIX_LATENT)
+        return bit(JGPT_W_DQ) | bit(JGPT_W_DQ_NORM) | bit(JGPT_W_UQ) | bit(JGPT_W_UK) | bit(JGPT_W_UV) | bit(JGPT_W_O) |
+               (s.kv_from ? 0 : bit(JGPT_W_DKV) | bit(JGPT_W_DKV_NORM));
+    if (s.kind == JGPT_MIX_HGRN2)
+        return bit(JGPT_W_Q) | bit(JGPT_W_F) | bit(JGPT_W_V) | bit(JGPT_W_O) | bit(JGPT_W_DECAY_BIAS) | bit(JGPT_W_LOWER) | bit(JGPT_W_HEAD_NORM);
+    if (s.kind == JGPT_MIX_WKV)
+        return bit(JGPT_W_Q) | bit(JGPT_W_K) | bit(JGPT_W_V) | bit(JGPT_W_G) | bit(JGPT_W_O) | bit(JGPT_W_A1) | bit(JGPT_W_A2) | bit(JGPT_W_DECAY_BIAS) |
+               bit(JGPT_W_BONUS) | bit(JGPT_W_HEAD_NORM) | bit(JGPT_W_MU_R) | bit(JGPT_W_MU_K) | bit(JGPT_W_MU_V) | bit(JGPT_W_MU_G) | bit(JGPT_W_MU_W);
     uint64_t n = bit(JGPT_W_Q) | bit(JGPT_W_K) | bit(JGPT_W_V) | bit(JGPT_W_O);
     if (s.kind == JGPT_MIX_ATTENTION) return s.gate ? n | bit(JGPT_W_G) : n;
     n |= bit(JGPT_W_A1) | bit(JGPT_W_A2) | bit(JGPT_W_DECAY_BIAS) | bit(JGPT_W_HEAD_NORM);
@@ -291,13 +449,16 @@ static uint64_t needed_roles(const jgpt_mixer_spec &s) {
 }
 
 static int32_t missing_weights(const Decoder *d) {
-    const uint64_t top = bit(JGPT_W_EMBED) | bit(JGPT_W_POS) | bit(JGPT_W_FINAL_NORM) | bit(JGPT_W_FINAL_NORM_B) |
-                         (d->s.embed_norm ? bit(JGPT_W_EMBED_NORM) | bit(JGPT_W_EMBED_NORM_B) : 0);
+    const uint64_t beta = d->rms ? 0 : ~0ull;
+    const uint64_t top = bit(JGPT_W_EMBED) | (d->s.pos_table ? bit(JGPT_W_POS) : 0) | (d->s.head ? bit(JGPT_W_HEAD) : 0) | bit(JGPT_W_FINAL_NORM) |
+                         (beta & bit(JGPT_W_FINAL_NORM_B)) | (d->s.embed_norm ? bit(JGPT_W_EMBED_NORM) | bit(JGPT_W_EMBED_NORM_B) : 0);
     JGPT_REQUIRE((d->have & top) == top, JGPT_ERR_ILLEGAL_STATE, "embedding or final norm weights are not set");
     for (size_t i = 0; i < d->L.size(); i++) {
         const DLayer &y = d->L[i];
-        uint64_t n = bit(JGPT_W_NORM1) | bit(JGPT_W_NORM1_B);
-        if (y.ff) n |= bit(JGPT_W_NORM2) | bit(JGPT_W_NORM2_B) | bit(JGPT_W_FF_GATE) | bit(JGPT_W_FF_UP) | bit(JGPT_W_FF_DOWN);
+        uint64_t n = bit(JGPT_W_NORM1) | (beta & bit(JGPT_W_NORM1_B)) | (d->s.layer_scale ? bit(JGPT_W_LS1) : 0) | (d->s.depth_average ? bit(JGPT_W_DWA) : 0);
+        if (y.ff)
+            n |= bit(JGPT_W_NORM2) | (beta & bit(JGPT_W_NORM2_B)) | bit(JGPT_W_FF_UP) | bit(JGPT_W_FF_DOWN) | (d->s.layer_scale ? bit(JGPT_W_LS2) : 0) |
+                 (y.ff_kind == JGPT_FF_XIELU ? bit(JGPT_W_FF_ACT) : bit(JGPT_W_FF_GATE));
         JGPT_REQUIRE((y.have & n) == n, JGPT_ERR_ILLEGAL_STATE, "norm or feed-forward weights of layer %zu are not set", i);
         for (const DBranch &b : y.br)
             JGPT_REQUIRE((b.have & needed_roles(b.s)) == needed_roles(b.s), JGPT_ERR_ILLEGAL_STATE, "mixer weights of layer %zu are not set", i);
@@ -316,7 +477,12 @@ static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const flo
     if (layer < 0) {
         switch (role) {
             case JGPT_W_EMBED: TRY(shape(d->s.vocab, W)); TRY(put_matrix(d, d->embed, d->ldw, 0, 0, src, rows, cols, none, none)); break;
-            case JGPT_W_POS: TRY(shape(d->s.max_positions, W)); TRY(put_matrix(d, d->pos, d->ldw, 0, 0, src, rows, cols, none, none)); break;
+            case JGPT_W_HEAD:
+                JGPT_REQUIRE(d->head, JGPT_ERR_INVALID_ARGUMENT, "the logits come from the embedding");
+                TRY(shape(d->s.vocab, W));
+                TRY(put_matrix(d, d->head, d->ldw, 0, 0, src, rows, cols, none, none));
+                break;
+            case JGPT_W_POS: JGPT_REQUIRE(d->pos, JGPT_ERR_INVALID_ARGUMENT, "the model has no table of positions"); TRY(shape(d->s.max_positions, W)); TRY(put_matrix(d, d->pos, d->ldw, 0, 0, src, rows, cols, none, none)); break;
             case JGPT_W_EMBED_NORM: TRY(shape(1, W)); TRY(put_floats(d, d->enw, src, 1, W, none)); break;
             case JGPT_W_EMBED_NORM_B: TRY(shape(1, W)); TRY(put_floats(d, d->enb, src, 1, W, none)); break;
             case JGPT_W_FINAL_NORM: TRY(shape(1, W)); TRY(put_floats(d, d->fnw, src, 1, W, none)); break;
@@ -329,15 +495,42 @@ static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const flo
     DLayer &y = d->L[(size_t)layer];
     if (branch < 0) {
         const Grouping pair{16, 32};
-        const bool ff_role = role == JGPT_W_FF_GATE || role == JGPT_W_FF_UP || role == JGPT_W_FF_DOWN || role == JGPT_W_NORM2 || role == JGPT_W_NORM2_B;
+        const bool ff_role = role == JGPT_W_FF_ACT || role == JGPT_W_LS2 || role == JGPT_W_FF_GATE || role == JGPT_W_FF_UP || role == JGPT_W_FF_DOWN || role == JGPT_W_NORM2 || role == JGPT_W_NORM2_B;
         JGPT_REQUIRE(!ff_role || y.ff, JGPT_ERR_INVALID_ARGUMENT, "layer %d has no feed-forward part", layer);
         switch (role) {
             case JGPT_W_NORM1: TRY(shape(1, W)); TRY(put_floats(d, y.n1w, src, 1, W, none)); break;
             case JGPT_W_NORM1_B: TRY(shape(1, W)); TRY(put_floats(d, y.n1b, src, 1, W, none)); break;
             case JGPT_W_NORM2: TRY(shape(1, W)); TRY(put_floats(d, y.n2w, src, 1, W, none)); break;
             case JGPT_W_NORM2_B: TRY(shape(1, W)); TRY(put_floats(d, y.n2b, src, 1, W, none)); break;
+            case JGPT_W_LS1:
+            case JGPT_W_LS2: {
+                JGPT_REQUIRE(d->s.layer_scale, JGPT_ERR_INVALID_ARGUMENT, "the model has no layer scales");
+                TRY(shape(1, W));
+                std::vector<float> v(src, src + W);
+                for (float &x : v) x *= d->s.residual_mult;
+                TRY(put_floats(d, role == JGPT_W_LS1 ? y.ls1 : y.ls2, v.data(), 1, W, none));
+                break;
+            }
+            case JGPT_W_DWA:
+                JGPT_REQUIRE(y.dwa, JGPT_ERR_INVALID_ARGUMENT, "the model has no depth averages");
+                TRY(shape(1, layer + 2));
+                TRY(put_floats(d, y.dwa, src, 1, cols, none));
+                break;
+            case JGPT_W_FF_ACT: {
+                JGPT_REQUIRE(y.ff_kind == JGPT_FF_XIELU, JGPT_ERR_INVALID_ARGUMENT, "layer %d: the activation has no parameters", layer);
+                TRY(shape(1, 2));
+                auto softplus = [](double z) { return std::max(z, 0.0) + std::log1p(std::exp(-std::fabs(z))); };
+                y.act_p0 = (float)softplus(src[0]), y.act_p1 = (float)(0.5 + softplus(src[1]));
+                break;
+            }
             case JGPT_W_FF_GATE:
             case JGPT_W_FF_UP: {
+                if (y.ff_kind == JGPT_FF_XIELU) {
+                    JGPT_REQUIRE(role == JGPT_W_FF_UP, JGPT_ERR_INVALID_ARGUMENT, "layer %d: the feed-forward part has no gate", layer);
+                    TRY(shape(y.ff, W));
+                    TRY(put_matrix(d, y.w_gu, d->ldw, 0, 0, src, rows, cols, none, none));
+                    break;
+                }
                 // rows in groups of 16: gate, linear, gate, ... (two strided copies would overwrite each other's gaps)
                 TRY(shape(y.ff, W));
                 for (int r = 0; r < rows; r += 16)
@@ -378,7 +571,55 @@ static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const flo
         case JGPT_W_G2: TRY(shape(s.heads * s.vdim, s.rank_g)); TRY(put_matrix(d, b.w_g2, b.rg, 0, 0, src, rows, cols, vg, none)); break;
         case JGPT_W_DECAY_BIAS: TRY(shape(1, s.heads * s.dim)); TRY(put_floats(d, b.bias, src, cols, 1, kg)); break;
         case JGPT_W_A_LOG: TRY(shape(1, s.heads)); TRY(put_floats(d, b.a_log, src, 1, cols, none)); break;
-        case JGPT_W_HEAD_NORM: TRY(shape(1, s.vdim)); TRY(put_floats(d, b.norm, src, 1, cols, none)); break;
+        case JGPT_W_HEAD_NORM:
+            if (s.kind == JGPT_MIX_WKV) {
+                TRY(shape(1, s.heads * s.vdim));
+                TRY(put_floats(d, b.norm, src, cols, 1, vg));
+            } else {
+                TRY(shape(1, s.vdim));
+                TRY(put_floats(d, b.norm, src, 1, cols, none));
+            }
+            break;
+        case JGPT_W_BONUS: TRY(shape(s.heads, s.dim)); TRY(put_floats(d, b.bonus, src, rows * cols, 1, kg)); break;
+        case JGPT_W_LOWER: TRY(shape(1, s.heads * s.dim)); TRY(put_floats(d, b.lower, src, cols, 1, kg)); break;
+        case JGPT_W_F: TRY(into_proj(b.f, s.heads * s.dim, kg)); break;
+        case JGPT_W_MU_R:
+        case JGPT_W_MU_K:
+        case JGPT_W_MU_V:
+        case JGPT_W_MU_G:
+        case JGPT_W_MU_W: TRY(shape(1, W)); TRY(put_floats(d, b.mu + (size_t)(role - JGPT_W_MU_R) * W, src, 1, W, none)); break;
+        case JGPT_W_DQ: TRY(into_proj(b.dq, s.q_rank, none)); break;
+        case JGPT_W_DQ_NORM: TRY(shape(1, s.q_rank)); TRY(put_floats(d, b.dq_norm, src, 1, cols, none)); break;
+        case JGPT_W_DKV_NORM: TRY(shape(1, s.kv_rank)); TRY(put_floats(d, b.dkv_norm, src, 1, cols, none)); break;
+        case JGPT_W_DKV:
+            TRY(shape(s.kv_rank + s.rot_dim, W));
+            TRY(put_matrix(d, y.w_in, d->ldw, b.dkv, 0, src, s.kv_rank, W, none, none));
+            TRY(put_matrix(d, y.w_in, d->ldw, b.dkr, 0, src + (size_t)s.kv_rank * W, s.rot_dim, W, none, none));
+            break;
+        case JGPT_W_UQ:
+            TRY(shape(s.heads * (s.dim + s.rot_dim), s.q_rank));
+            for (int h = 0; h < s.heads; h++) {
+                const float *hs = src + (size_t)h * (s.dim + s.rot_dim) * s.q_rank;
+                TRY(put_matrix(d, b.w_uq, b.qrp, h * b.DQ, 0, hs, s.dim, s.q_rank, none, none));
+                TRY(put_matrix(d, b.w_uq, b.qrp, h * b.DQ + b.DP, 0, hs + (size_t)s.dim * s.q_rank, s.rot_dim, s.q_rank, none, none));
+            }
+            break;
+        case JGPT_W_UK: {
+            TRY(shape(s.heads * s.dim, s.kv_rank));
+            std::vector<float> t((size_t)s.kv_rank * s.dim);
+            for (int h = 0; h < s.heads; h++) {
+                for (int i = 0; i < s.dim; i++)
+                    for (int c = 0; c < s.kv_rank; c++) t[(size_t)c * s.dim + i] = src[((size_t)h * s.dim + i) * s.kv_rank + c];
+                TRY(put_matrix(d, b.w_absorb, b.DP, h * b.KR, 0, t.data(), s.kv_rank, s.dim, none, none));
+                TRY(put_matrix(d, b.w_ukv, b.KR, h * b.DP, 0, src + (size_t)h * s.dim * s.kv_rank, s.dim, s.kv_rank, none, none));
+            }
+            break;
+        }
+        case JGPT_W_UV:
+            TRY(shape(s.heads * s.vdim, s.kv_rank));
+            for (int h = 0; h < s.heads; h++)
+                TRY(put_matrix(d, b.w_ukv, b.KR, s.heads * b.DP + h * b.DV, 0, src + (size_t)h * s.vdim * s.kv_rank, s.vdim, s.kv_rank, none, none));
+            break;
         case JGPT_W_CONV_Q: TRY(shape(s.kv_heads * s.dim, s.taps)); TRY(put_floats(d, b.conv_q, src, rows, cols, kg)); break;
         case JGPT_W_CONV_K: TRY(shape(s.kv_heads * s.dim, s.taps)); TRY(put_floats(d, b.conv_k, src, rows, cols, kg)); break;
         case JGPT_W_CONV_V: TRY(shape(s.heads * s.vdim, s.taps)); TRY(put_floats(d, b.conv_v, src, rows, cols, vg)); break;
@@ -396,7 +637,8 @@ int32_t decoder_check_pool(const Decoder *d, const Pool *p) {
     JGPT_REQUIRE(p, JGPT_ERR_BAD_HANDLE, "bad kvpool handle");
     JGPT_REQUIRE(p->ctx == d->ctx, JGPT_ERR_INVALID_ARGUMENT, "model and KV pool live on different contexts");
     bool ok = p->layered && p->elem_bytes == d->eb && p->state_stride == d->state_stride && p->vlayers.size() == d->kv.size();
-    for (size_t i = 0; ok && i < d->kv.size(); i++) ok = p->vlayers[i].heads == d->kv[i].heads && p->vlayers[i].dim == d->kv[i].dim;
+    for (size_t i = 0; ok && i < d->kv.size(); i++)
+        ok = p->vlayers[i].heads == d->kv[i].heads && p->vlayers[i].dim == d->kv[i].dim && p->vlayers[i].parts == d->kv[i].parts;
     JGPT_REQUIRE(ok, JGPT_ERR_INVALID_ARGUMENT, "KV pool geometry does not match the model");
     return JGPT_OK;
 }
@@ -407,21 +649,100 @@ static int32_t product(Decoder *d, const nt::Problem *p, int n, nt::Epilogue epi
     return d->f32 ? nt::launch_f32(p, n, epi, d->ctx->stream) : nt::launch_bf16(d->ctx, p, n, epi, pdl, d->ctx->stream);
 }
 
-static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, uint64_t capture_rows) {
+// The residual in front of layer i (the number of layers: in front of the final norm).
+static mix::RowSource residual(const Decoder *d, size_t i) {
+    mix::RowSource r{};
+    if (i == 0) {
+        r.embed = d->embed, r.ld_embed = d->ldw, r.vocab = d->s.vocab, r.embed_scale = d->s.embed_scale;
+        for (const mix::Rotation &x : d->rots) r.rot[r.n_rot++] = x;
+    } else if (d->s.depth_average) {
+        r.slots = d->slots, r.slot_stride = (uint64_t)d->R * d->s.width, r.weights = d->L[i - 1].dwa, r.n_slots = (int)i + 1;
+    } else {
+        r.slots = d->x, r.n_slots = 1;
+    }
+    return r;
+}
+
+// Groups of long entries whose keys fit the workspace together.
+struct LatentBatch {
+    int first, n, rows, max_keys, tile0, n_tiles;
+};
+
+static int32_t enqueue_latent(Decoder *d, Pool *p, const mix::StepDesc &sd, const std::vector<LatentBatch> &batches, const DLayer &y, const DBranch &b, int pdl) {
+    const int R = sd.rows, eb = d->eb, H = b.s.heads;
+    cudaStream_t st = d->ctx->stream;
+    mix::LatentArgs a{};
+    a.proj = d->proj, a.ldp = y.n_in, a.dq_off = b.dq, a.c_off = b.dkv, a.r_off = b.dkr;
+    a.q_rank = b.s.q_rank, a.kv_rank = b.s.kv_rank, a.rot_dim = b.s.rot_dim, a.half = b.s.rot_dims / 2, a.eps = d->s.eps, a.scale = b.s.score_scale;
+    a.dq_norm = b.dq_norm, a.dkv_norm = b.dkv_norm, a.cq = d->cq, a.ldcq = b.qrp, a.own_cache = b.s.kv_from == 0;
+    a.KR = b.KR, a.RR = b.RR, a.LDR = b.LDR;
+    a.kv = p->vkv + p->vlayers[(size_t)b.kv_layer].offset, a.table = p->d_table, a.n_blocks = p->n_blocks, a.mbs = p->max_blocks_per_seq;
+    a.cs = d->rots[(size_t)b.rot].out, a.q = d->q, a.ldq = H * b.DQ, a.DQ = b.DQ, a.DP = b.DP, a.dim = b.s.dim, a.qa = d->qa;
+    a.heads = H, a.window = b.s.window, a.cx = d->cx, a.kvx = d->kvx, a.ldx = H * (b.DP + b.DV), a.DVm = b.DV, a.vdim = b.s.vdim;
+    a.out = d->mixed, a.ldo = y.n_out, a.out_off = b.out, a.sm_count = d->ctx->sm_count, a.status = d->ctx->d_status;
+    auto at = [&](void *base, size_t elements) { return reinterpret_cast<uint8_t *>(base) + elements * eb; };
+    TRY(mix::launch_latent_prep(d->f32, sd, a, pdl, st));
+    nt::Problem q{d->cq, b.w_uq, d->q, nullptr, R, a.ldq, b.qrp, b.qrp, b.qrp, a.ldq, 1.f};
+    TRY(product(d, &q, 1, nt::EPI_STORE, pdl));
+    if (const int n = sd.lat_hi - sd.lat_lo; n > 0) {
+        const size_t r0 = (size_t)sd.lat_lo;
+        nt::Problem in{at(d->q, r0 * a.ldq), b.w_absorb, at(d->qa, r0 * H * b.KR), nullptr, n, H * b.KR, b.DP, a.ldq, b.DP, H * b.KR, 1.f};
+        in.seg_n = b.KR, in.a_seg = b.DQ;
+        TRY(product(d, &in, 1, nt::EPI_STORE, pdl));
+        TRY(mix::launch_latent_attention(d->f32, sd, a, pdl, st));
+        nt::Problem out{at(d->qa, r0 * H * b.KR), at(b.w_ukv, (size_t)H * b.DP * b.KR), at(d->mixed, r0 * y.n_out + b.out), nullptr, n, H * b.DV, b.KR,
+                        H * b.KR, b.KR, y.n_out, 1.f};
+        out.seg_n = b.DV, out.a_seg = b.KR;
+        TRY(product(d, &out, 1, nt::EPI_STORE, pdl));
+    }
+    for (const LatentBatch &g : batches) {
+        TRY(mix::launch_latent_gather(sd, a, g.first, g.n, g.max_keys, pdl, st));
+        nt::Problem kv{d->cx, b.w_ukv, d->kvx, nullptr, g.rows, a.ldx, b.KR, b.KR + b.RR, b.KR, a.ldx, 1.f};
+        TRY(product(d, &kv, 1, nt::EPI_STORE, pdl));
+        TRY(mix::launch_latent_tiles(sd, a, g.tile0, g.n_tiles, pdl, st));
+    }
+    return JGPT_OK;
+}
+
+static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, const std::vector<LatentBatch> &batches, uint64_t capture_rows) {
     const int W = d->s.width, R = sd.rows, ldw = d->ldw, eb = d->eb;
     const float eps = d->s.eps;
     cudaStream_t st = d->ctx->stream;
     int *status = d->ctx->d_status;
     const int pdl = d->overlap && !d->f32 && !capture_rows ? 3 : 0;
+    const uint64_t slot = (uint64_t)d->R * W, mix_stride = (uint64_t)d->R * ldw;
+    const bool deep = d->s.depth_average;
     for (size_t i = 0; i < d->L.size(); i++) {
         DLayer &y = d->L[i];
-        if (i == 0)
+        float *from = d->x, *to = deep ? d->slots + (i + 1) * slot : d->x;  // residual in front of the layer, its result
+        if (d->rms) {
+            const DBranch *w = y.shift();
+            mix::ShiftArgs sh{};
+            if (w) {
+                for (int k = 0; k < 5; k++) sh.mu[k] = w->mu + (size_t)k * W;
+                sh.out_stride = mix_stride, sh.state = p->state + w->state_off + w->conv_off, sh.state_stride = p->state_stride, sh.max_seqs = p->max_seqs;
+            }
+            if (deep && i == 0) from = d->slots;
+            TRY(mix::launch_residual_norm(d->f32, sd, residual(d, i), nullptr, R, y.n1w, eps, i == 0 || deep ? from : nullptr, d->h, sh, W, ldw, status,
+                                          i == 0 ? pdl & 2 : pdl, st));
+        } else if (i == 0) {
             TRY(mix::launch_embed(d->f32, sd, d->embed, ldw, d->pos, ldw, d->s.embed_scale,
                                   d->s.embed_norm ? mix::NormW{d->enw, d->enb} : mix::NormW{nullptr, nullptr}, mix::NormW{y.n1w, y.n1b}, eps, d->x,
                                   d->h, W, ldw, d->s.vocab, d->s.max_positions, status, pdl & 2, st));
-        else TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n1w, y.n1b}, eps, d->h, R, W, ldw, pdl, st));
-        nt::Problem in{d->h, y.w_in, d->proj, nullptr, R, y.n_in, ldw, ldw, ldw, y.n_in, 1.f};
-        TRY(product(d, &in, 1, nt::EPI_STORE, pdl));
+        } else {
+            TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n1w, y.n1b}, eps, d->h, R, W, ldw, pdl, st));
+        }
+        if (const DBranch *w = y.shift()) {
+            uint8_t *h = reinterpret_cast<uint8_t *>(d->h), *win = reinterpret_cast<uint8_t *>(y.w_in), *proj = reinterpret_cast<uint8_t *>(d->proj);
+            const int hk = w->s.heads * w->DK;
+            nt::Problem in[2] = {{h, win, proj, nullptr, R, 4 * hk, ldw, ldw, ldw, y.n_in, 1.f},
+                                 {h + 4 * mix_stride * eb, win + (size_t)w->a1 * ldw * eb, proj + (size_t)w->a1 * eb, nullptr, R, w->ra, ldw, ldw, ldw, y.n_in, 1.f}};
+            in[0].seg_n = hk, in[0].a_seg = (long long)mix_stride, in[1].act = nt::ACT_TANH;
+            TRY(product(d, in, 2, nt::EPI_ACT, pdl));
+        } else {
+            nt::Problem in{d->h, y.w_in, d->proj, nullptr, R, y.n_in, ldw, ldw, ldw, y.n_in, 1.f};
+            TRY(product(d, &in, 1, nt::EPI_STORE, pdl));
+        }
         for (DBranch &b : y.br) {
             if (b.s.kind == JGPT_MIX_ATTENTION) {
                 mix::AttnArgs a{};
@@ -431,32 +752,48 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, uint
                 a.out = d->mixed, a.ldo = y.n_out, a.out_off = b.out;
                 a.sm_count = d->ctx->sm_count, a.status = status;
                 TRY(mix::launch_attention(d->f32, sd, a, pdl, st));
+            } else if (b.s.kind == JGPT_MIX_LATENT) {
+                TRY(enqueue_latent(d, p, sd, batches, y, b, pdl));
             } else {
                 uint8_t *proj = reinterpret_cast<uint8_t *>(d->proj), *z = reinterpret_cast<uint8_t *>(d->z);
                 nt::Problem zp[2];
                 int nz = 0;
-                zp[nz++] = nt::Problem{proj + (size_t)b.a1 * eb, b.w_a2, z + (size_t)b.za * eb, nullptr, R, b.s.heads * b.DK, b.ra, y.n_in, b.ra, y.n_z, 1.f};
+                if (b.a1 >= 0)
+                    zp[nz++] = nt::Problem{proj + (size_t)b.a1 * eb, b.w_a2, z + (size_t)b.za * eb, nullptr, R, b.s.heads * b.DK, b.ra, y.n_in, b.ra, y.n_z, 1.f};
                 if (b.g1 >= 0)
                     zp[nz++] = nt::Problem{proj + (size_t)b.g1 * eb, b.w_g2, z + (size_t)b.zg * eb, nullptr, R, b.s.heads * b.DV, b.rg, y.n_in, b.rg, y.n_z, 1.f};
-                TRY(product(d, zp, nz, nt::EPI_STORE, pdl));
+                if (nz) TRY(product(d, zp, nz, nt::EPI_STORE, pdl));
                 mix::RecArgs a = rec_args(b);
                 a.proj = d->proj, a.ldp = y.n_in, a.z = d->z, a.ldz = y.n_z, a.eps = eps;
+                if (b.s.kind == JGPT_MIX_HGRN2) a.z = d->proj, a.ldz = y.n_in;
                 a.state = p->state + b.state_off, a.state_stride = p->state_stride, a.max_seqs = p->max_seqs;
                 a.out = d->mixed, a.ldo = y.n_out, a.raw = d->raw, a.chunk_ws = d->chunk_ws, a.chunk_ws_floats = d->chunk_ws_floats, a.sm_count = d->ctx->sm_count, a.status = status;
                 TRY(mix::launch_recurrent(d->f32, sd, a, pdl, st));
             }
         }
-        nt::Problem out{d->mixed, y.w_out, d->x, nullptr, R, W, y.n_out, y.n_out, y.n_out, W, 1.f};
+        nt::Problem out{d->mixed, y.w_out, to, nullptr, R, W, y.n_out, y.n_out, y.n_out, W, 1.f};
+        out.res = from, out.colscale = y.ls1;
         TRY(product(d, &out, 1, nt::EPI_ADD_F32, pdl));
         if (y.ff) {
-            TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n2w, y.n2b}, eps, d->h, R, W, ldw, pdl, st));
-            nt::Problem gu{d->h, y.w_gu, d->act, nullptr, R, 2 * y.ffp, ldw, ldw, ldw, y.ffp, 1.f};
-            TRY(product(d, &gu, 1, nt::EPI_GATE_GELU, pdl));
-            nt::Problem down{d->act, y.w_down, d->x, nullptr, R, W, y.ffp, y.ffp, y.ffp, W, 1.f};
+            if (d->rms) {
+                mix::RowSource src{};
+                src.slots = to, src.n_slots = 1;
+                TRY(mix::launch_residual_norm(d->f32, sd, src, nullptr, R, y.n2w, eps, nullptr, d->h, mix::ShiftArgs{}, W, ldw, status, pdl, st));
+            } else {
+                TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n2w, y.n2b}, eps, d->h, R, W, ldw, pdl, st));
+            }
+            const bool gated = y.ff_kind == JGPT_FF_GATED_GELU;
+            nt::Problem gu{d->h, y.w_gu, d->act, nullptr, R, gated ? 2 * y.ffp : y.ffp, ldw, ldw, ldw, y.ffp, 1.f};
+            if (!gated) gu.act = nt::ACT_XIELU, gu.p0 = y.act_p0, gu.p1 = y.act_p1;
+            TRY(product(d, &gu, 1, gated ? nt::EPI_GATE_GELU : nt::EPI_ACT, pdl));
+            nt::Problem down{d->act, y.w_down, to, nullptr, R, W, y.ffp, y.ffp, y.ffp, W, 1.f};
+            down.colscale = y.ls2;
             TRY(product(d, &down, 1, nt::EPI_ADD_F32, pdl));
         }
-        if (capture_rows)
+        if (capture_rows) {
+            if (deep) TRY(mix::launch_residual_norm(d->f32, sd, residual(d, i + 1), nullptr, R, d->fnw, eps, d->x, nullptr, mix::ShiftArgs{}, W, ldw, status, 0, st));
             JGPT_CUDA_TRY(cudaMemcpyAsync(d->capture + (uint64_t)i * capture_rows * W, d->x, sizeof(float) * capture_rows * W, cudaMemcpyDeviceToHost, st));
+        }
     }
     return JGPT_OK;
 }
@@ -465,8 +802,11 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, uint
 static int32_t enqueue_head(Decoder *d, const mix::StepDesc &sd, int w0, int n, bool pick, const SampleSpec &spec) {
     cudaStream_t st = d->ctx->stream;
     const int pdl = d->overlap && !d->f32 && w0 == 0 ? 3 : 0;
-    TRY(mix::launch_layer_norm(d->f32, d->x, sd.want + w0, mix::NormW{d->fnw, d->fnb}, d->s.eps, d->h, n, d->s.width, d->ldw, pdl, st));
-    nt::Problem p{d->h, d->embed, d->logits, nullptr, n, d->s.vocab, d->ldw, d->ldw, d->ldw, d->s.vocab, d->s.logit_scale};
+    if (d->rms)
+        TRY(mix::launch_residual_norm(d->f32, sd, residual(d, d->L.size()), sd.want + w0, n, d->fnw, d->s.eps, nullptr, d->h, mix::ShiftArgs{}, d->s.width,
+                                      d->ldw, d->ctx->d_status, pdl, st));
+    else TRY(mix::launch_layer_norm(d->f32, d->x, sd.want + w0, mix::NormW{d->fnw, d->fnb}, d->s.eps, d->h, n, d->s.width, d->ldw, pdl, st));
+    nt::Problem p{d->h, d->head ? d->head : d->embed, d->logits, nullptr, n, d->s.vocab, d->ldw, d->ldw, d->ldw, d->s.vocab, d->s.logit_scale};
     TRY(product(d, &p, 1, nt::EPI_SCALE_F32, pdl & 1));
     if (!pick) return JGPT_OK;
     if (spec.temperature > 0.f) return launch_sample(d->logits, d->samp, n, d->s.vocab, spec, d->d_u + w0, d->d_next + w0, st);
@@ -552,6 +892,7 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
         return o;
     };
     const size_t o_tok = take((size_t)rows), o_pos = take((size_t)rows), o_seq = take((size_t)rows), o_seg = take(6 * (size_t)c.n);
+    const size_t o_ent = take((size_t)rows), o_lat_short = take((size_t)c.n), o_lat_long = take(4 * (size_t)c.n);
     const size_t o_single = take((size_t)c.n), o_short = take((size_t)c.n), o_want = take((size_t)c.n_want), o_long = take(2 * (size_t)c.n);
     int max_len = 0, n_short = 0, n_long = 0, n_chunks = 0;
     const int long_min = d->long_min;
@@ -561,7 +902,7 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
         const SeqState &ss = p->seqs[(size_t)s];
         segs[i] = mix::Seg{s, r0, T, ss.len, ss.conv_set, 0};
         max_len = std::max(max_len, ss.len + T);
-        for (int t = 0; t < T; t++) hd[o_tok + r0 + t] = c.ids[r0 + t], hd[o_pos + r0 + t] = ss.len + t, hd[o_seq + r0 + t] = s;
+        for (int t = 0; t < T; t++) hd[o_tok + r0 + t] = c.ids[r0 + t], hd[o_pos + r0 + t] = ss.len + t, hd[o_seq + r0 + t] = s, hd[o_ent + r0 + t] = i;
         if (T == 1) hd[o_single + n_single++] = i;
         if (long_min == 0 || T < long_min) hd[o_short + n_short++] = i;
         else {
@@ -585,13 +926,38 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
         if (T > 1)
             for (int t = 0; t < T; t += qt) hd[o_tile + 2 * n_tiles] = i, hd[o_tile + 2 * n_tiles + 1] = t, n_tiles++;
     }
-    at = o_tile + 2 * (size_t)n_tiles;
+    at = o_tile;
+    take(2 * (size_t)n_tiles);
+    // latent attention: long entries in batches that fit the workspace, with tiles of query tokens of their own; the others'
+    // rows as one range (running tokens and short portions lie together in what the scheduler sends)
+    mix::StepDesc sd{};
+    std::vector<LatentBatch> batches;
+    const size_t o_lat_tile = at;
+    int n_lat_long = 0, n_lat_tiles = 0;
+    sd.lat_lo = rows;
+    mix::LatentEntry *lat_long = reinterpret_cast<mix::LatentEntry *>(hd + o_lat_long);
+    for (int i = 0; d->cq && i < c.n; i++) {
+        const int T = segs[i].T, pos0 = segs[i].pos0, back = d->max_window > 0 ? std::min(pos0, d->max_window - 1) : pos0;
+        if (d->lat_min == 0 || T < std::max(d->lat_min, 2) || (long long)back + T > d->kvx_rows) {
+            sd.lat_lo = std::min(sd.lat_lo, segs[i].row0), sd.lat_hi = segs[i].row0 + T;
+            if (T > 1) hd[o_lat_short + sd.n_lat_short++] = i, sd.lat_short_max = std::max(sd.lat_short_max, T);
+            continue;
+        }
+        if (batches.empty() || batches.back().rows + back + T > d->kvx_rows) batches.push_back(LatentBatch{n_lat_long, 0, 0, 0, n_lat_tiles, 0});
+        LatentBatch &g = batches.back();
+        lat_long[n_lat_long] = mix::LatentEntry{i, pos0 - back, back + T, g.rows};
+        for (int t = 0; t < T; t += mix::kLatentTile, g.n_tiles++)
+            hd[o_lat_tile + 2 * n_lat_tiles] = n_lat_long, hd[o_lat_tile + 2 * n_lat_tiles + 1] = t, n_lat_tiles++;
+        g.n++, g.rows += back + T, g.max_keys = std::max(g.max_keys, back + T), n_lat_long++;
+    }
+    at = o_lat_tile + 2 * (size_t)n_lat_tiles;
     JGPT_REQUIRE(at <= desc_ints(d), JGPT_ERR_INVALID_ARGUMENT, "step descriptors need %zu words, there are %zu", at, desc_ints(d));
     cudaStream_t st = d->ctx->stream;
-    mix::StepDesc sd{};
     const int *dd = d->d_desc;
     sd.tok = dd + o_tok, sd.pos = dd + o_pos, sd.seq = dd + o_seq, sd.segs = reinterpret_cast<const mix::Seg *>(dd + o_seg);
     sd.tiles = reinterpret_cast<const int2 *>(dd + o_tile), sd.singles = dd + o_single, sd.want = dd + o_want;
+    sd.ent = dd + o_ent, sd.lat_short = dd + o_lat_short, sd.lat_long = reinterpret_cast<const mix::LatentEntry *>(dd + o_lat_long);
+    sd.lat_tiles = reinterpret_cast<const int2 *>(dd + o_lat_tile);
     sd.rows = rows, sd.n_segs = c.n, sd.n_tiles = n_tiles, sd.n_singles = n_single, sd.n_want = c.n_want, sd.max_len = max_len;
     sd.qt = qt;
     sd.short_segs = dd + o_short, sd.long_segs = reinterpret_cast<const int2 *>(dd + o_long), sd.chunks = reinterpret_cast<const int2 *>(dd + o_chunk);
@@ -612,7 +978,7 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
     }
     auto enqueue = [&]() -> int32_t {
         JGPT_CUDA_TRY(cudaMemcpyAsync(d->d_desc, hd, sizeof(int) * at, cudaMemcpyHostToDevice, st));
-        TRY(enqueue_layers(d, p, sd, cap_rows));
+        TRY(enqueue_layers(d, p, sd, batches, cap_rows));
         for (int w0 = 0; w0 < c.n_want; w0 += d->logit_rows) {
             const int n = std::min(d->logit_rows, c.n_want - w0);
             TRY(enqueue_head(d, sd, w0, n, pick, c.spec));
@@ -753,6 +1119,10 @@ int32_t jgpt_decoder_create(jgpt_ctx ctxh, const jgpt_decoder_spec *spec, const 
     JGPT_REQUIRE(spec && layers && out, JGPT_ERR_INVALID_ARGUMENT, "null pointer");
     JGPT_REQUIRE(spec->vocab > 0 && spec->width > 0 && spec->max_positions > 0 && spec->n_layers > 0 && max_rows > 0, JGPT_ERR_INVALID_ARGUMENT,
                  "model dimensions must be positive");
+    const bool rms = spec->norm == JGPT_NORM_RMS;
+    JGPT_REQUIRE(rms || spec->norm == JGPT_NORM_LAYER, JGPT_ERR_UNSUPPORTED, "norm %d", spec->norm);
+    JGPT_REQUIRE(rms ? !spec->pos_table && !spec->embed_norm : !spec->layer_scale && !spec->depth_average && spec->residual_mult == 1.f, JGPT_ERR_UNSUPPORTED,
+                 "layer norms go with embedding norms and learned positions, RMS norms with residual factors and depth averages");
     JGPT_REQUIRE(dtype == JGPT_DTYPE_BF16 || dtype == JGPT_DTYPE_F32, JGPT_ERR_INVALID_ARGUMENT, "dtype %d", dtype);
     JGPT_CUDA_TRY(make_current(c));
     Decoder *d = new Decoder();

@@ -25,7 +25,7 @@ constexpr int kBK = 128, kMaxSplit = 8;
 
 struct SmallArgs {
     Problem p[2];
-    int tiles[2];   // column tiles of each product
+    int tiles[2], per_seg[2];   // column tiles of each product, of each of its segments
     int n, k_split, pdl;
 };
 
@@ -56,8 +56,9 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
     if (second) tile -= args.tiles[0];
     const Problem &P = second ? args.p[1] : args.p[0];
     const int M = P.M, N = P.N, K = P.K, lda = P.lda, ldw = P.ldw;
-    const int m0 = blockIdx.y * BM, n0 = tile * kBN;
-    const __nv_bfloat16 *__restrict__ A = reinterpret_cast<const __nv_bfloat16 *>(P.A);
+    const int per_seg = args.per_seg[second], seg = tile / per_seg, seg_n = P.seg_n;
+    const int m0 = blockIdx.y * BM, n0 = seg * seg_n + tile % per_seg * kBN, n_end = min(N, (seg + 1) * seg_n), cn = seg * P.c_seg;
+    const __nv_bfloat16 *__restrict__ A = reinterpret_cast<const __nv_bfloat16 *>(P.A) + seg * P.a_seg;
     const __nv_bfloat16 *__restrict__ W = reinterpret_cast<const __nv_bfloat16 *>(P.W);
     const int nk_all = (K + kBK - 1) / kBK;
     const int kt0 = k_part * nk_all / args.k_split, nk = (k_part + 1) * nk_all / args.k_split - kt0;
@@ -67,7 +68,7 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
 #pragma unroll
         for (int i = 0; i < 2 * NH; i++) {
             const int r = r16 + 16 * i, k = k0 + c16 * 8;
-            const bool ok = n0 + r < N && k < K;
+            const bool ok = n0 + r < n_end && k < K;
             cp_async16(Ws + ((size_t)buf * kBN + r) * kBK + ((c16 ^ (r & 7)) * 8), ok ? W + (size_t)(n0 + r) * ldw + k : W, ok);
         }
     };
@@ -179,10 +180,12 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
             const float up = __shfl_down_sync(0xffffffffu, sum[i], 16);
             if ((c & 31) < 16 && m < M && n + 16 < N)
                 reinterpret_cast<__nv_bfloat16 *>(P.C)[(size_t)m * P.ldc + n / 32 * 16 + (c & 15)] = __float2bfloat16(gelu_tanh(sum[i]) * up);
-        } else if (m < M && n < N) {
-            if (EPI == EPI_STORE) reinterpret_cast<__nv_bfloat16 *>(P.C)[(size_t)m * P.ldc + n] = __float2bfloat16(sum[i]);
-            if (EPI == EPI_ADD_F32) reinterpret_cast<float *>(P.C)[(size_t)m * P.ldc + n] += sum[i];
-            if (EPI == EPI_SCALE_F32) reinterpret_cast<float *>(P.C)[(size_t)m * P.ldc + n] = sum[i] * P.scale;
+        } else if (m < M && n < n_end) {
+            const size_t at = (size_t)m * P.ldc + n + cn;
+            if (EPI == EPI_STORE) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(sum[i]);
+            if (EPI == EPI_ACT) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(activate(P.act, P.p0, P.p1, sum[i]));
+            if (EPI == EPI_ADD_F32) reinterpret_cast<float *>(P.C)[at] = P.res[at] + (P.colscale ? P.colscale[n] * sum[i] : sum[i]);
+            if (EPI == EPI_SCALE_F32) reinterpret_cast<float *>(P.C)[at] = sum[i] * P.scale;
         }
     }
 }
@@ -225,7 +228,7 @@ static int32_t small_dispatch(const Ctx *ctx, const Problem *p, int n, int pdl, 
     int tiles = 0, K = 0;
     for (int i = 0; i < n; i++) {
         a.p[i] = p[i];
-        a.tiles[i] = (p[i].N + bn - 1) / bn;
+        a.per_seg[i] = (p[i].seg_n + bn - 1) / bn, a.tiles[i] = p[i].segments() * a.per_seg[i];
         tiles += a.tiles[i];
         K = std::max(K, p[i].K);
     }
@@ -245,8 +248,20 @@ int umma_min_rows() {
     return v;
 }
 
-int32_t launch_bf16(const Ctx *ctx, const Problem *p, int n, Epilogue epi, int pdl, cudaStream_t st) {
+// Defaults spelled out: one segment, the residual in C itself.
+static int32_t complete(const Problem *p, int n, Problem (&q)[2]) {
     JGPT_REQUIRE(n >= 1 && n <= 2 && p[0].M > 0, JGPT_ERR_INVALID_ARGUMENT, "1 or 2 products per launch");
+    for (int i = 0; i < n; i++) {
+        q[i] = p[i];
+        if (q[i].seg_n <= 0) q[i].seg_n = q[i].N;
+        if (!q[i].res) q[i].res = reinterpret_cast<const float *>(q[i].C);
+    }
+    return JGPT_OK;
+}
+
+int32_t launch_bf16(const Ctx *ctx, const Problem *problems, int n, Epilogue epi, int pdl, cudaStream_t st) {
+    Problem p[2];
+    if (int32_t rc = complete(problems, n, p)) return rc;
     bool big = p[0].M >= umma_min_rows() && umma_min_rows() > 0;
     for (int i = 0; i < n; i++) big = big && !p[i].rowsel;
     if (big) {
@@ -259,6 +274,7 @@ int32_t launch_bf16(const Ctx *ctx, const Problem *p, int n, Epilogue epi, int p
         case EPI_ADD_F32: return small_dispatch<EPI_ADD_F32>(ctx, p, n, pdl, st);
         case EPI_SCALE_F32: return small_dispatch<EPI_SCALE_F32>(ctx, p, n, pdl, st);
         case EPI_GATE_GELU: return small_dispatch<EPI_GATE_GELU>(ctx, p, n, pdl, st);
+        case EPI_ACT: return small_dispatch<EPI_ACT>(ctx, p, n, pdl, st);
     }
     return fail(JGPT_ERR_INVALID_ARGUMENT, "unknown epilogue");
 }
@@ -272,16 +288,17 @@ __global__ void __launch_bounds__(256) gemm_nt_f32_kernel(const Problem P0, cons
     __shared__ float As[BK][BT + 1], Ws[BK][BT + 1];
     const Problem &P = blockIdx.z == 0 ? P0 : P1;
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-    const int m0 = blockIdx.y * BT, n0 = blockIdx.x * BT;
+    const int per_seg = (P.seg_n + BT - 1) / BT, seg = blockIdx.x / per_seg, cn = seg * P.c_seg;
+    const int m0 = blockIdx.y * BT, n0 = seg * P.seg_n + blockIdx.x % per_seg * BT, n_end = min(P.N, (seg + 1) * P.seg_n);
     if (n0 >= P.N) return;
-    const float *__restrict__ A = reinterpret_cast<const float *>(P.A);
+    const float *__restrict__ A = reinterpret_cast<const float *>(P.A) + seg * P.a_seg;
     const float *__restrict__ W = reinterpret_cast<const float *>(P.W);
     float acc[4][4] = {};
     for (int k0 = 0; k0 < P.K; k0 += BK) {
         for (int e = tid; e < BT * BK; e += 256) {
             const int r = e / BK, k = k0 + e % BK, m = m0 + r, n = n0 + r;
             As[e % BK][r] = (m < P.M && k < P.K) ? A[(size_t)(P.rowsel ? P.rowsel[m] : m) * P.lda + k] : 0.f;
-            Ws[e % BK][r] = (n < P.N && k < P.K) ? W[(size_t)n * P.ldw + k] : 0.f;
+            Ws[e % BK][r] = (n < n_end && k < P.K) ? W[(size_t)n * P.ldw + k] : 0.f;
         }
         __syncthreads();
 #pragma unroll
@@ -311,25 +328,29 @@ __global__ void __launch_bounds__(256) gemm_nt_f32_kernel(const Problem P0, cons
 #pragma unroll
             for (int j = 0; j < 4; j++) {
                 const int n = n0 + tx + 16 * j;
-                if (n >= P.N) continue;
-                float *c = C + (size_t)m * P.ldc + n;
-                if (EPI == EPI_STORE) *c = acc[i][j];
-                if (EPI == EPI_ADD_F32) *c += acc[i][j];
-                if (EPI == EPI_SCALE_F32) *c = acc[i][j] * P.scale;
+                if (n >= n_end) continue;
+                const size_t at = (size_t)m * P.ldc + n + cn;
+                if (EPI == EPI_STORE) C[at] = acc[i][j];
+                if (EPI == EPI_ACT) C[at] = activate(P.act, P.p0, P.p1, acc[i][j]);
+                if (EPI == EPI_ADD_F32) C[at] = P.res[at] + (P.colscale ? P.colscale[n] * acc[i][j] : acc[i][j]);
+                if (EPI == EPI_SCALE_F32) C[at] = acc[i][j] * P.scale;
             }
         }
     }
 }
 
-int32_t launch_f32(const Problem *p, int n, Epilogue epi, cudaStream_t st) {
-    JGPT_REQUIRE(n >= 1 && n <= 2 && p[0].M > 0, JGPT_ERR_INVALID_ARGUMENT, "1 or 2 products per launch");
+int32_t launch_f32(const Problem *problems, int n, Epilogue epi, cudaStream_t st) {
+    Problem p[2];
+    if (int32_t rc = complete(problems, n, p)) return rc;
     const Problem &q = p[n - 1];
-    const dim3 grid((unsigned)((std::max(p[0].N, q.N) + 63) / 64), (unsigned)((p[0].M + 63) / 64), (unsigned)n);
+    auto tiles = [](const Problem &x) { return x.segments() * ((x.seg_n + 63) / 64); };
+    const dim3 grid((unsigned)std::max(tiles(p[0]), tiles(q)), (unsigned)((p[0].M + 63) / 64), (unsigned)n);
     switch (epi) {
         case EPI_STORE: gemm_nt_f32_kernel<EPI_STORE><<<grid, 256, 0, st>>>(p[0], q); break;
         case EPI_ADD_F32: gemm_nt_f32_kernel<EPI_ADD_F32><<<grid, 256, 0, st>>>(p[0], q); break;
         case EPI_SCALE_F32: gemm_nt_f32_kernel<EPI_SCALE_F32><<<grid, 256, 0, st>>>(p[0], q); break;
         case EPI_GATE_GELU: gemm_nt_f32_kernel<EPI_GATE_GELU><<<grid, 256, 0, st>>>(p[0], q); break;
+        case EPI_ACT: gemm_nt_f32_kernel<EPI_ACT><<<grid, 256, 0, st>>>(p[0], q); break;
     }
     JGPT_CUDA_TRY(cudaGetLastError());
     return JGPT_OK;

@@ -52,6 +52,10 @@ struct UmmaArgs {
     int M, N, K, ldc, mt, nt, pdl;
     float scale;
     int *status;
+    int per_seg, seg_n, c_seg, a_x, a_y;  // column tiles and columns of a segment; its shift in C; its operand's shift (columns, rows)
+    const float *res, *colscale;
+    int act;
+    float p0, p1;
 };
 
 __device__ __forceinline__ void tile_of(const UmmaArgs &a, int t, int &m, int &n) {
@@ -99,13 +103,14 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
             for (int t = blockIdx.x; t < total && !*s_abort; t += gridDim.x) {
                 int m, n;
                 tile_of(a, t, m, n);
+                const int seg = n / a.per_seg, ax = seg * a.a_x, ay = seg * a.a_y + m * UM, wy = seg * a.seg_n + n % a.per_seg * BN;
                 for (int kt = 0; kt < nk; kt++, it++) {
                     const uint32_t s = it % ST, use = it / ST;
                     if (use > 0 && !mbar_wait_bounded(&empty_bar[s], (use - 1) & 1u, a.status, s_abort)) break;
                     uint8_t *dst = tiles + (size_t)s * SB;
                     mbar_expect_tx(&full_bar[s], SB);
-                    tma_2d(dst, &amap, kt * UK, m * UM, &full_bar[s]);
-                    tma_2d(dst + A_BYTES, &wmap, kt * UK, n * BN, &full_bar[s]);
+                    tma_2d(dst, &amap, ax + kt * UK, ay, &full_bar[s]);
+                    tma_2d(dst + A_BYTES, &wmap, kt * UK, wy, &full_bar[s]);
                 }
             }
             if (*s_abort) {  // copies already issued still target this CTA's shared memory: give each a bounded chance to land
@@ -140,13 +145,14 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
         }
     } else {
         const int quarter = warp & 3, half = (warp - 2) >> 2;
-        const bool vec4 = (a.ldc & 3) == 0;
+        const bool vec4 = (a.ldc & 3) == 0 && (a.c_seg & 3) == 0;
         uint32_t j = 0;
         for (int t = blockIdx.x; t < total; t += gridDim.x, j++) {
             const uint32_t buf = j & 1u, round = j >> 1, acc = tmem + buf * BN;
             int mi, ni;
             tile_of(a, t, mi, ni);
-            const int m = mi * UM + quarter * 32 + lane, n0 = ni * BN;
+            const int seg = ni / a.per_seg, m = mi * UM + quarter * 32 + lane, n0 = seg * a.seg_n + ni % a.per_seg * BN;
+            const int n_end = min(a.N, (seg + 1) * a.seg_n), cn = seg * a.c_seg;
             int ok = 0;
             if (lane == 0) ok = mbar_wait_bounded(&acc_full[buf], round & 1u, a.status, s_abort) ? 1 : 0;
             ok = __shfl_sync(0xffffffffu, ok, 0);
@@ -154,15 +160,19 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
             tc_fence_after();
 #pragma unroll 1
             for (int c0 = half * (BN / 2); c0 < (half + 1) * (BN / 2); c0 += 32) {
-                if (n0 + c0 >= a.N) break;  // uniform across the warp
+                if (n0 + c0 >= n_end) break;  // uniform across the warp
                 float v[32];
                 load_acc32(acc, quarter, c0, v);
                 if (m >= a.M) continue;
-                if (EPI == EPI_STORE) {
-                    __nv_bfloat16 *c = reinterpret_cast<__nv_bfloat16 *>(a.C) + (size_t)m * a.ldc + n0 + c0;
+                if (EPI == EPI_STORE || EPI == EPI_ACT) {
+                    __nv_bfloat16 *c = reinterpret_cast<__nv_bfloat16 *>(a.C) + (size_t)m * a.ldc + n0 + c0 + cn;
+                    if (EPI == EPI_ACT) {
+#pragma unroll
+                        for (int q = 0; q < 32; q++) v[q] = activate(a.act, a.p0, a.p1, v[q]);
+                    }
 #pragma unroll
                     for (int q = 0; q < 4; q++)
-                        if (n0 + c0 + 8 * q < a.N)  // N is a multiple of 8 here
+                        if (n0 + c0 + 8 * q < n_end)  // N and seg_n are multiples of 8 here
                             *reinterpret_cast<uint4 *>(c + 8 * q) = make_uint4(pack_bf16(v[8 * q], v[8 * q + 1]), pack_bf16(v[8 * q + 2], v[8 * q + 3]),
                                                                                pack_bf16(v[8 * q + 4], v[8 * q + 5]), pack_bf16(v[8 * q + 6], v[8 * q + 7]));
                 } else if (EPI == EPI_GATE_GELU) {
@@ -174,15 +184,22 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
                         *reinterpret_cast<uint4 *>(c + 8 * q) = make_uint4(pack_bf16(v[8 * q], v[8 * q + 1]), pack_bf16(v[8 * q + 2], v[8 * q + 3]),
                                                                            pack_bf16(v[8 * q + 4], v[8 * q + 5]), pack_bf16(v[8 * q + 6], v[8 * q + 7]));
                 } else {
-                    float *c = reinterpret_cast<float *>(a.C) + (size_t)m * a.ldc + n0 + c0;
+                    const size_t at = (size_t)m * a.ldc + n0 + c0 + cn;
+                    float *c = reinterpret_cast<float *>(a.C) + at;
+                    const float *res = a.res + at;
+                    if (EPI == EPI_ADD_F32 && a.colscale) {
+#pragma unroll
+                        for (int q = 0; q < 32; q++)
+                            if (n0 + c0 + q < n_end) v[q] *= __ldg(a.colscale + n0 + c0 + q);
+                    }
 #pragma unroll
                     for (int q = 0; q < 8; q++) {
                         const int n = n0 + c0 + 4 * q;
                         float4 o = make_float4(v[4 * q], v[4 * q + 1], v[4 * q + 2], v[4 * q + 3]);
                         if (EPI == EPI_SCALE_F32) o.x *= a.scale, o.y *= a.scale, o.z *= a.scale, o.w *= a.scale;
-                        if (vec4 && n + 3 < a.N) {
+                        if (vec4 && n + 3 < n_end) {
                             if (EPI == EPI_ADD_F32) {
-                                const float4 r = *reinterpret_cast<const float4 *>(c + 4 * q);
+                                const float4 r = *reinterpret_cast<const float4 *>(res + 4 * q);
                                 o.x += r.x, o.y += r.y, o.z += r.z, o.w += r.w;
                             }
                             *reinterpret_cast<float4 *>(c + 4 * q) = o;
@@ -190,7 +207,7 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
                             const float e[4] = {o.x, o.y, o.z, o.w};
 #pragma unroll
                             for (int i = 0; i < 4; i++)
-                                if (n + i < a.N) c[4 * q + i] = EPI == EPI_ADD_F32 ? c[4 * q + i] + e[i] : e[i];
+                                if (n + i < n_end) c[4 * q + i] = EPI == EPI_ADD_F32 ? res[4 * q + i] + e[i] : e[i];
                         }
                     }
                 }
@@ -235,10 +252,12 @@ static int32_t make_map(CUtensorMap *map, const void *base, int rows, int K, int
 template <int BN, int EPI>
 static int32_t umma_launch(const Ctx *ctx, const Problem &p, int pdl, cudaStream_t st) {
     CUtensorMap am, wm;
-    int32_t rc = make_map(&am, p.A, p.M, p.K, p.lda, UM);
+    const int segs = p.segments(), ay = (int)(p.a_seg / p.lda), ax = (int)(p.a_seg % p.lda), per_seg = (p.segment_cols() + BN - 1) / BN;
+    int32_t rc = make_map(&am, p.A, p.M + (segs - 1) * ay, p.K + (segs - 1) * ax, p.lda, UM);
     if (!rc) rc = make_map(&wm, p.W, p.N, p.K, p.ldw, BN);
     if (rc) return rc;
-    UmmaArgs a{p.C, p.M, p.N, p.K, p.ldc, (p.M + UM - 1) / UM, (p.N + BN - 1) / BN, pdl, p.scale, ctx->d_status};
+    UmmaArgs a{p.C, p.M, p.N, p.K, p.ldc, (p.M + UM - 1) / UM, segs * per_seg, pdl, p.scale, ctx->d_status,
+               per_seg, p.segment_cols(), p.c_seg, ax, ay, p.res, p.colscale, p.act, p.p0, p.p1};
     auto kern = gemm_nt_umma_kernel<BN, EPI>;
     static thread_local int set_for = -1;
     if (set_for != ctx->device) {
@@ -258,7 +277,7 @@ static int32_t umma_launch(const Ctx *ctx, const Problem &p, int pdl, cudaStream
 template <int EPI>
 static int32_t umma_pick(const Ctx *ctx, const Problem &p, int pdl, cudaStream_t st) {
     const int mt = (p.M + UM - 1) / UM;
-    auto tiles = [&](int bn) { return mt * ((p.N + bn - 1) / bn); };
+    auto tiles = [&](int bn) { return mt * p.segments() * ((p.segment_cols() + bn - 1) / bn); };
     if (tiles(256) >= ctx->sm_count) return umma_launch<256, EPI>(ctx, p, pdl, st);
     if (tiles(128) >= ctx->sm_count * 2 / 3) return umma_launch<128, EPI>(ctx, p, pdl, st);
     return umma_launch<64, EPI>(ctx, p, pdl, st);
@@ -269,7 +288,11 @@ int32_t launch_bf16_umma(const Ctx *ctx, const Problem &p, Epilogue epi, int pdl
                  JGPT_ERR_INVALID_ARGUMENT, "operand rows must start on 16-byte boundaries");
     JGPT_REQUIRE((epi != EPI_STORE || (p.N % 8 == 0 && p.ldc % 8 == 0)) && (epi != EPI_GATE_GELU || (p.N % 32 == 0 && p.ldc % 8 == 0)),
                  JGPT_ERR_INVALID_ARGUMENT, "output columns %d, stride %d", p.N, p.ldc);
+    JGPT_REQUIRE((epi != EPI_ACT || (p.N % 8 == 0 && p.ldc % 8 == 0)) &&
+                     (p.segments() == 1 || (p.seg_n % 8 == 0 && p.c_seg % 8 == 0 && p.a_seg % 8 == 0 && epi != EPI_GATE_GELU)),
+                 JGPT_ERR_INVALID_ARGUMENT, "segments of %d columns, shifts %lld / %d", p.seg_n, p.a_seg, p.c_seg);
     switch (epi) {
+        case EPI_ACT: return umma_pick<EPI_ACT>(ctx, p, pdl, st);
         case EPI_STORE: return umma_pick<EPI_STORE>(ctx, p, pdl, st);
         case EPI_ADD_F32: return umma_pick<EPI_ADD_F32>(ctx, p, pdl, st);
         case EPI_SCALE_F32: return umma_pick<EPI_SCALE_F32>(ctx, p, pdl, st);

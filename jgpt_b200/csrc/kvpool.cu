@@ -344,7 +344,7 @@ int32_t pool_create_layered(Ctx *c, const std::vector<KvLayerGeom> &layers, int 
     p->ctx = c, p->layered = true, p->elem_bytes = elem_bytes, p->n_blocks = n_blocks, p->max_seqs = max_seqs;
     p->max_blocks_per_seq = max_blocks_per_seq, p->max_positions = max_blocks_per_seq * kBlockTokens, p->state_stride = state_stride;
     for (KvLayerGeom g : layers) {
-        g.offset = p->kv_bytes, g.block_bytes = 2ull * kBlockTokens * g.heads * g.dim * elem_bytes;
+        g.offset = p->kv_bytes, g.block_bytes = (uint64_t)g.parts * kBlockTokens * g.heads * g.dim * elem_bytes;
         p->kv_bytes += g.block_bytes * (uint64_t)n_blocks;
         p->vlayers.push_back(g);
     }

@@ -17,7 +17,7 @@ struct Seg {
 
 // What a step brings, on the device.
 struct StepDesc {
-    const int *tok, *pos, *seq;  // per row
+    const int *tok, *pos, *seq, *ent;  // per row: token, position, sequence, entry
     const Seg *segs;
     const int2 *tiles;           // (entry, first token) of every query tile of the entries with more than one token
     const int *singles;          // entries with one token
@@ -25,7 +25,12 @@ struct StepDesc {
     const int2 *long_segs;       // the others: (entry, index of its first chunk)
     const int2 *chunks;          // (entry, first token) of the long entries' chunks of kRecChunk tokens
     const int *want;             // rows whose logits are wanted
-    int rows, n_segs, n_tiles, n_singles, n_short, n_long, n_chunks, n_want;
+    const struct LatentEntry *lat_long;  // entries whose latent attention runs on written-out keys and values
+    const int2 *lat_tiles;       // (index in lat_long, first token) of their query tiles
+    const int *lat_short;        // entries with more than one token whose latent attention stays on the latents
+    int rows, n_segs, n_tiles, n_singles, n_short, n_long, n_chunks, n_want, n_lat_short;
+    int lat_short_max;           // tokens of the longest of the latter
+    int lat_lo, lat_hi;          // rows from the first to the last of the entries that stay on the latents
     int qt;                      // tokens per query tile
     int max_len;                 // upper bound of pos0 + T (sizes the split of single-token attention)
 };
@@ -41,6 +46,38 @@ int32_t launch_embed(bool f32, const StepDesc &d, const void *embed, int ld_embe
                      cudaStream_t st);
 int32_t launch_layer_norm(bool f32, const float *x, const int *rowsel, NormW w, float eps, void *h, int rows, int W, int ldh, int pdl,
                           cudaStream_t st);
+
+// A row of the residual stream: the embedding of the row's token, or the weighted sum of the earlier layers' results
+// (a plain residual is the sum over one slot without weights).
+constexpr int kMaxRotations = 4;
+struct Rotation {        // cos and sin of every row's angles, [rows][half] pairs, times mag
+    const double *freq;
+    float2 *out;
+    int half;
+    float mag;
+};
+struct RowSource {
+    const void *embed;   // null: slots
+    int ld_embed, vocab;
+    float embed_scale;
+    const float *slots, *weights;
+    uint64_t slot_stride;
+    int n_slots;
+    Rotation rot[kMaxRotations];  // written beside the embedding
+    int n_rot;
+};
+// Five mixes of a row with the one before it, h + (h' - h) mu_s; h' of an entry's first row comes from the sequence's state
+// [2][W] (the copy conv_set names), its last row goes into the other copy.
+struct ShiftArgs {
+    const float *mu[5];  // null mu[0]: no mixes
+    uint64_t out_stride; // elements between the mixes of h
+    uint8_t *state;      // of slot 0, at the history
+    uint64_t state_stride;
+    int max_seqs;
+};
+// x[r] = source (when x is set), h[r] = x[r] / rms * gamma, as mixes when sh has them; rowsel picks rows (null: all).
+int32_t launch_residual_norm(bool f32, const StepDesc &d, const RowSource &src, const int *rowsel, int rows, const float *gamma, float eps, float *x,
+                             void *h, const ShiftArgs &sh, int W, int ldh, int *status, int pdl, cudaStream_t st);
 
 // ---- attn_gqa.cu -----------------------------------------------------------------------------------
 struct AttnArgs {
@@ -62,12 +99,12 @@ int attn_padded_head(int dim, int vdim);          // 0: not supported
 int attn_query_tile(int heads, int kv_heads);     // tokens per query tile of the multi-token kernel
 
 // ---- recurrent.cu ----------------------------------------------------------------------------------
-enum RecKind : int { REC_GLA = 0, REC_DELTA = 1 };
+enum RecKind : int { REC_GLA = 0, REC_DELTA = 1, REC_HGRN2 = 2, REC_WKV = 3 };
 struct RecArgs {
     int kind;
     const void *proj;   // [rows, ldp]
     int ldp, q_off, k_off, v_off, b_off, g_off;  // b: step-size column (delta); g: output gate inside proj (GLA)
-    const void *z;      // [rows, ldz]: decay logits at z_off, output gate at zg_off (delta)
+    const void *z;      // [rows, ldz]: decay logits at z_off, output gate at zg_off (delta); HGRN2: proj itself
     int ldz, z_off, zg_off;
     int heads, kv_heads, DK, DV;  // padded head sizes
     int dim, vdim;      // true head sizes
@@ -76,7 +113,11 @@ struct RecArgs {
     int taps;
     const float *decay_bias;  // [heads * DK]
     const float *a_log;       // [heads] (delta)
-    const float *norm_w;      // [DV]
+    const float *norm_w;      // [DV], or [heads * DV]: norm_stride is DV then
+    int norm_stride;
+    const float *bonus;       // [heads * DK] weight of the current token (WKV)
+    const float *lower;       // [heads * DK] lower bound of the forget gate (HGRN2)
+    int shift_width;          // width of the previous token's input kept in the state (WKV)
     uint8_t *state;     // of sequence slot 0, this layer's part
     uint64_t state_stride;    // bytes between sequence slots
     uint64_t conv_off;  // byte offset of the convolution history [2][taps - 1][channels] inside the part
@@ -97,6 +138,48 @@ int32_t launch_recurrent(bool f32, const StepDesc &d, const RecArgs &a, int pdl,
 int rec_padded_key(int dim);    // 0: not supported
 int rec_padded_value(int vdim);
 uint64_t rec_state_bytes(const RecArgs &a, int elem_bytes, uint64_t *conv_off);
+
+// ---- attn_latent.cu ----------------------------------------------------------------------------------
+// Latent attention.  A page row is [latent c, padded to KR | rotated key part, padded to RR | 8 unused], LDR elements.
+// On the latents ("absorbed"): scores q~ . c + q_rot . k_rot with q~ = W_uk^T q per head, the output a weighted sum of c.
+// Written out: keys [W_uk c | k_rot] and values W_uv c per head in a workspace, for entries with many query rows.
+struct LatentEntry {
+    int entry, key0, n_keys, row0;  // the keys of positions [key0, key0 + n_keys) in workspace rows [row0, ..)
+};
+struct LatentArgs {
+    const void *proj;   // [rows, ldp]: query latent at dq_off, key latent at c_off, rotated part behind it at r_off
+    int ldp, dq_off, c_off, r_off;
+    int q_rank, kv_rank, rot_dim, half;
+    float eps, scale;
+    const float *dq_norm, *dkv_norm;
+    void *cq;           // [rows, ldcq]
+    int ldcq, own_cache;
+    int KR, RR, LDR;
+    void *kv;           // pages [block][16][LDR]
+    const int *table;
+    int n_blocks, mbs;
+    const float2 *cs;   // [rows][half]
+    const void *q;      // [rows, ldq], head h at h * DQ: [dim, padded to DP | rot_dim ...]
+    int ldq, DQ, DP, dim;
+    void *qa;           // [rows, heads * KR]: q~, replaced by the weighted sums
+    int heads, window;
+    // written-out form
+    void *cx;           // [workspace rows][KR + RR]
+    const void *kvx;    // [workspace rows][ldx]: keys at h * DP, values at heads * DP + h * DVm
+    int ldx, DVm, vdim;
+    void *out;          // [rows, ldo], head h at out_off + h * DVm
+    int ldo, out_off;
+    int sm_count;
+    int *status;
+};
+int latent_padded_rank(int kv_rank);   // KR; 0: not supported by the tensor-core kernel
+int latent_padded_rot(int rot_dim);
+bool latent_expandable(int dim, int rot_dim, int vdim);
+int32_t launch_latent_prep(bool f32, const StepDesc &d, const LatentArgs &a, int pdl, cudaStream_t st);
+int32_t launch_latent_attention(bool f32, const StepDesc &d, const LatentArgs &a, int pdl, cudaStream_t st);
+int32_t launch_latent_gather(const StepDesc &d, const LatentArgs &a, int first, int n, int max_keys, int pdl, cudaStream_t st);
+int32_t launch_latent_tiles(const StepDesc &d, const LatentArgs &a, int first_tile, int n_tiles, int pdl, cudaStream_t st);
+constexpr int kLatentTile = 64;  // query tokens per tile of the written-out form
 
 }  // namespace mix
 }  // namespace jgpt

@@ -1,4 +1,6 @@
-// Embedding and layer norm of the layered decoder.  The residual stream and the norms are fp32.
+// Embedding and norms of the layered decoder: layer norm over a plain residual, RMS norm over a residual that may be the
+// embedding, a weighted sum of the earlier layers' results, and mixed with the previous token's row.  The residual stream and
+// the norms are fp32.
 #include "mixers.cuh"
 #include "ptx.cuh"
 
@@ -124,6 +126,116 @@ int32_t launch_layer_norm(bool f32, const float *x, const int *rowsel, NormW w, 
     JGPT_REQUIRE(smem <= 48 * 1024 - 256, JGPT_ERR_UNSUPPORTED, "width %d", W);
     if (f32) return launch(layer_norm_kernel<float>, rows, smem, pdl, st, x, rowsel, (const NormW)w, eps, (float *)h, W, ldh, pdl);
     return launch(layer_norm_kernel<__nv_bfloat16>, rows, smem, pdl, st, x, rowsel, (const NormW)w, eps, (__nv_bfloat16 *)h, W, ldh, pdl);
+}
+
+// ------------------------------------------------------------------------------------------------
+// RMS norm
+// ------------------------------------------------------------------------------------------------
+// Row `src` of the residual into shared memory (and to x), its 1 / rms returned.
+template <class AT, bool EMBED>
+__device__ __forceinline__ float residual_row(const RowSource &s, const int *__restrict__ tok, int src, float eps, float *row, float *x, int W, float *red, int *status) {
+    float q = 0.f;
+    if (EMBED) {
+        int t = tok[src];
+        if (t < 0 || t >= s.vocab) {
+            if (threadIdx.x == 0) atomicOr(status, DEV_STATUS_BAD_POSITION);
+            t = 0;
+        }
+        const AT *e = reinterpret_cast<const AT *>(s.embed) + (size_t)t * s.ld_embed;
+        for (int j = threadIdx.x; j < W; j += kNormThreads) {
+            const float v = load_act(e + j) * s.embed_scale;
+            row[j] = v, q += v * v;
+            if (x) x[(size_t)src * W + j] = v;
+        }
+    } else if ((W & 3) == 0) {
+        const float *base = s.slots + (size_t)src * W;
+        for (int j = threadIdx.x * 4; j < W; j += kNormThreads * 4) {
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (!s.weights) v = *reinterpret_cast<const float4 *>(base + j);
+            else {
+#pragma unroll 8
+                for (int i = 0; i < s.n_slots; i++) {
+                    const float4 y = *reinterpret_cast<const float4 *>(base + i * s.slot_stride + j);
+                    const float w = __ldg(s.weights + i);
+                    v.x = fmaf(w, y.x, v.x), v.y = fmaf(w, y.y, v.y), v.z = fmaf(w, y.z, v.z), v.w = fmaf(w, y.w, v.w);
+                }
+            }
+            *reinterpret_cast<float4 *>(row + j) = v;
+            if (x) *reinterpret_cast<float4 *>(x + (size_t)src * W + j) = v;
+            q += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+    } else {
+        const float *base = s.slots + (size_t)src * W;
+        for (int j = threadIdx.x; j < W; j += kNormThreads) {
+            float v = s.weights ? 0.f : base[j];
+            if (s.weights)
+                for (int i = 0; i < s.n_slots; i++) v = fmaf(__ldg(s.weights + i), base[i * s.slot_stride + j], v);
+            row[j] = v, q += v * v;
+            if (x) x[(size_t)src * W + j] = v;
+        }
+    }
+    return 1.f / sqrtf(block_sum(q, red) / (float)W + eps);
+}
+
+template <class AT, bool EMBED>
+__global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const StepDesc d, const RowSource s, const int *__restrict__ rowsel,
+                                                                     const float *__restrict__ gamma, float eps, float *x, AT *__restrict__ h,
+                                                                     const ShiftArgs sh, int W, int ldh, int *status, int pdl) {
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[kNormThreads / 32];
+    const int r = blockIdx.x;
+    if (pdl & 2) griddep_launch_dependents();
+    if (pdl & 1) griddep_wait();
+    const int src = rowsel ? rowsel[r] : r;
+    const float inv = residual_row<AT, EMBED>(s, d.tok, src, eps, row, x, W, red, status);
+    if (EMBED) {
+        for (int k = 0; k < s.n_rot; k++)
+            for (int i = threadIdx.x; i < s.rot[k].half; i += kNormThreads) {
+                double sn, cs;
+                sincos((double)d.pos[src] * s.rot[k].freq[i], &sn, &cs);
+                s.rot[k].out[(size_t)src * s.rot[k].half + i] = make_float2((float)cs * s.rot[k].mag, (float)sn * s.rot[k].mag);
+            }
+    }
+    if (!h) return;
+    if (!sh.mu[0]) {
+        for (int j = threadIdx.x; j < ldh; j += kNormThreads) store_act(h + (size_t)r * ldh + j, j < W ? row[j] * inv * gamma[j] : 0.f);
+        return;
+    }
+    // the row before: recomputed the same way inside an entry, read from the state in front of it
+    float *before = row + (W + 3) / 4 * 4;
+    const Seg sg = d.segs[d.ent[src]];
+    if (sg.seq < 0 || sg.seq >= sh.max_seqs) {
+        if (threadIdx.x == 0) atomicOr(status, DEV_STATUS_BAD_SEQ);
+        return;
+    }
+    float *hist = reinterpret_cast<float *>(sh.state + (uint64_t)sg.seq * sh.state_stride);
+    const bool first = src == sg.row0, last = src == sg.row0 + sg.T - 1;
+    float binv = 0.f;
+    if (!first) binv = residual_row<AT, EMBED>(s, d.tok, src - 1, eps, before, nullptr, W, red, status);
+    for (int j = threadIdx.x; j < ldh; j += kNormThreads) {
+        float v = 0.f, dv = 0.f;
+        if (j < W) {
+            v = row[j] * inv * gamma[j];
+            const float p = first ? (sg.pos0 > 0 ? hist[(size_t)sg.conv_set * W + j] : 0.f) : before[j] * binv * gamma[j];
+            dv = p - v;
+            if (last) hist[(size_t)(1 - sg.conv_set) * W + j] = v;
+        }
+#pragma unroll
+        for (int m = 0; m < 5; m++) store_act(h + m * sh.out_stride + (size_t)r * ldh + j, j < W ? fmaf(dv, sh.mu[m][j], v) : 0.f);
+    }
+}
+
+int32_t launch_residual_norm(bool f32, const StepDesc &d, const RowSource &s, const int *rowsel, int rows, const float *gamma, float eps, float *x,
+                             void *h, const ShiftArgs &sh, int W, int ldh, int *status, int pdl, cudaStream_t st) {
+    const size_t smem = sizeof(float) * (size_t)((W + 3) / 4 * 4) * (sh.mu[0] ? 2 : 1);
+    JGPT_REQUIRE(smem <= 48 * 1024 - 256, JGPT_ERR_UNSUPPORTED, "width %d", W);
+    auto run = [&](auto kern, auto *act) {
+        return launch(kern, rows, smem, pdl, st, (const StepDesc)d, (const RowSource)s, rowsel, gamma, eps, x, (decltype(act))h, (const ShiftArgs)sh, W, ldh,
+                      status, pdl);
+    };
+    if (f32) return s.embed ? run(residual_norm_kernel<float, true>, (float *)nullptr) : run(residual_norm_kernel<float, false>, (float *)nullptr);
+    return s.embed ? run(residual_norm_kernel<__nv_bfloat16, true>, (__nv_bfloat16 *)nullptr)
+                   : run(residual_norm_kernel<__nv_bfloat16, false>, (__nv_bfloat16 *)nullptr);
 }
 
 }  // namespace mix

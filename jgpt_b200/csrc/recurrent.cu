@@ -1,9 +1,11 @@
-// Recurrent mixers of the layered decoder, token by token: gated linear attention and the gated delta rule, both with a
-// decay per key channel (long entries of a bf16 step take the chunked form, recurrent_chunk.cu), as ONE kernel from the layer's projections to the gated, normalised head outputs - for prompts, portions of
+// Recurrent mixers of the layered decoder, token by token: gated linear attention, the gated delta rule, HGRN2 and WKV, all with
+// a decay per key channel (long entries of a bf16 step take the chunked form, recurrent_chunk.cu), as ONE kernel from the layer's projections to the gated, normalised head outputs - for prompts, portions of
 // prompts and single tokens alike, so a token's arithmetic does not depend on how its sequence was cut.
 //
 //   GLA    S <- diag(a) S + k v^T;                       o = S^T q
 //   DELTA  S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q   (o read off as S_decayed^T q + (q.k) u)
+//   HGRN2  S <- diag(f) S + (1 - f) v^T;                 o = S^T q
+//   WKV    o = (S + diag(u) k v^T)^T r, read off as S^T r + (r.(u k)) v;  S <- diag(w) S + k v^T
 //
 // A CTA owns one (sequence, head); a warp owns 16 value columns with every key row of the state in registers: lane =
 // (row lane 0..7, column lane 0..3), DK / 8 rows x 4 columns, rows in pairs for the packed fp32 instructions
@@ -73,7 +75,8 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
     const int h = blockIdx.x % a.heads, split = blockIdx.x / a.heads, col0 = split * DVc;
     constexpr int E = 16 / sizeof(AT);  // elements of a 16-byte chunk
     // a token's raw row: q, k, v, decay logits, output gate, then (delta) the chunk that holds its step size
-    const int RW = 3 * DK + 2 * DVc + (KIND == REC_DELTA ? E : 0), RK = DK, RV = 2 * DK, RZ = RV + DVc, RG = RZ + DK, RB = RG + DVc;
+    const int RK = DK, RV = rec_has_key(KIND) ? 2 * DK : DK, RZ = RV + DVc, RG = RZ + DK, RB = rec_has_gate(KIND) ? RG + DVc : RG,
+              RW = RB + (KIND == REC_DELTA ? E : 0);
     float *sq = rec_smem, *sk = sq + tt * DK, *sg = sk + tt * DK, *sv = sg + tt * DK, *so = sv + tt * DVc, *sbeta = so + tt * DVc,
           *sqk = sbeta + tt;
     AT *raw_s = reinterpret_cast<AT *>(sqk + tt);  // [2][tt][RW]; one stage is enough for a single token
@@ -182,11 +185,17 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
                 if (a.taps <= 4) convolve(std::integral_constant<int, 4>(), idx, raw, prev, t0, tn, dst, ld);
                 else convolve(std::integral_constant<int, kMaxTaps>(), idx, raw, prev, t0, tn, dst, ld);
             } else {
-                const float f = idx < DK / 2 ? qscale : 1.f;
+                if (!rec_has_key(KIND) && idx >= DK / 2 && idx < DK) {  // its key comes with the forget gate
+                    if (!SINGLE && (tn & 1)) *reinterpret_cast<float2 *>(dst + tn * ld) = make_float2(0.f, 0.f);
+                    continue;
+                }
+                const float f = KIND == REC_GLA && idx < DK / 2 ? qscale : 1.f;
+                const int from = idx < DK ? 2 * idx : RV + 2 * (idx - DK);
 #pragma unroll 4
                 for (int t = 0; t < tn; t++) {
-                    float2 y = load2(raw + (size_t)t * RW + 2 * idx);
-                    y.x *= f, y.y *= f;
+                    float2 y = load2(raw + (size_t)t * RW + from);
+                    if (KIND == REC_HGRN2 && idx < DK / 2) y.x *= sigmoid_f<AT>(y.x), y.y *= sigmoid_f<AT>(y.y);
+                    else y.x *= f, y.y *= f;
                     *reinterpret_cast<float2 *>(dst + t * ld) = y;
                 }
                 if (!SINGLE && (tn & 1)) *reinterpret_cast<float2 *>(dst + tn * ld) = make_float2(0.f, 0.f);  // pads the last pair of tokens
@@ -198,10 +207,19 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
             const float2 b = *reinterpret_cast<const float2 *>(a.decay_bias + h * DK + c);
             y.x += b.x, y.y += b.y;
             if (KIND == REC_GLA) y.x = -y.x, y.y = -y.y;  // sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau)
-            y.x = exp_f<AT>(-rate * softplus_f<AT>(y.x)), y.y = exp_f<AT>(-rate * softplus_f<AT>(y.y));
+            if (KIND == REC_HGRN2) {
+                const float2 low = *reinterpret_cast<const float2 *>(a.lower + h * DK + c);
+                const float2 f0 = forget_write<AT>(y.x, low.x), f1 = forget_write<AT>(y.y, low.y);
+                y = make_float2(f0.x, f1.x);
+                *reinterpret_cast<float2 *>(sk + t * DK + c) = make_float2(f0.y, f1.y);
+            } else if (KIND == REC_WKV) {
+                y.x = exp_neg_exp<AT>(y.x), y.y = exp_neg_exp<AT>(y.y);
+            } else {
+                y.x = exp_f<AT>(-rate * softplus_f<AT>(y.x)), y.y = exp_f<AT>(-rate * softplus_f<AT>(y.y));
+            }
             *reinterpret_cast<float2 *>(sg + t * DK + c) = y;
         }
-        if (!SINGLE && KIND == REC_GLA && (tn & 1))
+        if (!SINGLE && KIND != REC_DELTA && (tn & 1))
             for (int c = tid; c < DK; c += nthreads) sg[tn * DK + c] = 1.f;
         __syncthreads();
         if (!SINGLE && t0 + tt < sgm.T) stage(buf ^ 1, t0 + tt);  // lands while this tile runs; the previous tile's rows are no longer needed
@@ -218,6 +236,16 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
 #pragma unroll
                 for (int i = 0; i < NI; i++) sq[t * DK + lane + 32 * i] = qv[i] * fq, sk[t * DK + lane + 32 * i] = kv[i] * fk;
                 if (lane == 0) sqk[t] = qk * fq * fk, sbeta[t] = sigmoid_f<AT>(load1(raw + (size_t)t * RW + RB + h % E));
+            }
+            __syncthreads();
+        }
+        if (KIND == REC_WKV) {  // what the current token adds to its own output: (r . (u k)) v
+            for (int t = warp; t < tn; t += nw) {
+                float rk = 0.f;
+#pragma unroll
+                for (int i = 0; i < NI; i++) rk += sq[t * DK + lane + 32 * i] * sk[t * DK + lane + 32 * i] * a.bonus[h * DK + lane + 32 * i];
+                rk = warp_sum(rk);
+                if (lane == 0) sqk[t] = rk;
             }
             __syncthreads();
         }
@@ -286,9 +314,10 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
                         const ulonglong2 g2 = *reinterpret_cast<const ulonglong2 *>(gp + 32 * i);
 #pragma unroll
                         for (int c = 0; c < 4; c++) {
+                            if (KIND == REC_WKV) qs[c] = fma2(q2.x, st[2 * i][c], qs[c]), qs[c] = fma2(q2.y, st[2 * i + 1][c], qs[c]);
                             st[2 * i][c] = fma2(k2.x, v2[c], mul2(g2.x, st[2 * i][c]));
                             st[2 * i + 1][c] = fma2(k2.y, v2[c], mul2(g2.y, st[2 * i + 1][c]));
-                            qs[c] = fma2(q2.x, st[2 * i][c], qs[c]), qs[c] = fma2(q2.y, st[2 * i + 1][c], qs[c]);
+                            if (KIND != REC_WKV) qs[c] = fma2(q2.x, st[2 * i][c], qs[c]), qs[c] = fma2(q2.y, st[2 * i + 1][c], qs[c]);
                         }
                     }
 #pragma unroll
@@ -297,7 +326,8 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
                         of[e][c] = y.x + y.y;
                     }
                 }
-                const float tot = reduce8(of[0], of[1], lane);
+                float tot = reduce8(of[0], of[1], lane);
+                if (KIND == REC_WKV && t + (lane >> 4) < tn) tot = fmaf(sqk[t + (lane >> 4)], sv[(t + (lane >> 4)) * DVc + vcol + (rl & 3)], tot);
                 if (!SINGLE || lane < 16) so[(t + (lane >> 4)) * DVc + vcol + (rl & 3)] = tot;  // row tn of an odd tile is a spare
             }
         }
@@ -316,10 +346,9 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
                 const float inv = a.out_scale / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
                 AT *o = reinterpret_cast<AT *>(a.out) + (size_t)(sgm.row0 + t0 + t) * a.ldo + a.out_off + h * DVc;
                 const AT *gp = raw + (size_t)t * RW + RG;
-                for (int c = lane; c < DVc; c += 32) {
-                    const float gt = load1(gp + c), sgt = sigmoid_f<AT>(gt);
-                    store1(o + c, so[t * DVc + c] * inv * a.norm_w[c] * (KIND == REC_DELTA ? sgt : gt * sgt));
-                }
+                const float *nm = a.norm_w + h * a.norm_stride;
+                for (int c = lane; c < DVc; c += 32)
+                    store1(o + c, so[t * DVc + c] * inv * nm[c] * (rec_has_gate(KIND) ? out_gate<AT, KIND>(load1(gp + c)) : 1.f));
             }
         }
     }
@@ -360,10 +389,10 @@ int rec_padded_value(int vdim) { return vdim > 0 && vdim <= 256 ? (vdim + 15) / 
 
 uint64_t rec_state_bytes(const RecArgs &a, int elem_bytes, uint64_t *conv_off) {
     const uint64_t s = (uint64_t)a.heads * a.DK * a.DV * sizeof(float);
-    *conv_off = s;
+    *conv_off = s;  // the convolution's history, or WKV's previous rows
     const uint64_t channels = 2ull * a.kv_heads * a.DK + (uint64_t)a.heads * a.DV;
     const uint64_t conv = a.taps > 1 ? 2ull * (uint64_t)(a.taps - 1) * channels * (uint64_t)elem_bytes : 0;
-    return (s + conv + 255) / 256 * 256;
+    return (s + conv + 2 * sizeof(float) * (uint64_t)a.shift_width + 255) / 256 * 256;
 }
 
 template <class AT, int KIND, int DK, bool SINGLE>
@@ -431,8 +460,13 @@ static int32_t rec_run(const StepDesc &d, const RecArgs &a, int pdl, cudaStream_
 
 int32_t launch_recurrent(bool f32, const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st) {
     JGPT_REQUIRE(a.taps <= kMaxTaps, JGPT_ERR_UNSUPPORTED, "convolutions of up to %d taps", kMaxTaps);
-    if (f32) return a.kind == REC_DELTA ? rec_run<float, REC_DELTA>(d, a, pdl, st) : rec_run<float, REC_GLA>(d, a, pdl, st);
-    return a.kind == REC_DELTA ? rec_run<__nv_bfloat16, REC_DELTA>(d, a, pdl, st) : rec_run<__nv_bfloat16, REC_GLA>(d, a, pdl, st);
+    switch (a.kind) {
+        case REC_GLA: return f32 ? rec_run<float, REC_GLA>(d, a, pdl, st) : rec_run<__nv_bfloat16, REC_GLA>(d, a, pdl, st);
+        case REC_DELTA: return f32 ? rec_run<float, REC_DELTA>(d, a, pdl, st) : rec_run<__nv_bfloat16, REC_DELTA>(d, a, pdl, st);
+        case REC_HGRN2: return f32 ? rec_run<float, REC_HGRN2>(d, a, pdl, st) : rec_run<__nv_bfloat16, REC_HGRN2>(d, a, pdl, st);
+        case REC_WKV: return f32 ? rec_run<float, REC_WKV>(d, a, pdl, st) : rec_run<__nv_bfloat16, REC_WKV>(d, a, pdl, st);
+    }
+    return fail(JGPT_ERR_INVALID_ARGUMENT, "recurrence %d", a.kind);
 }
 
 }  // namespace mix

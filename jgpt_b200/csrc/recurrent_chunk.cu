@@ -9,7 +9,8 @@
 //     u_i + beta_i sum_{j<i} A_ij u_j = beta_i (v_i - (k_i b_i)^T S0)     i.e.  U = T V - (T K~) S0,  T = (I + diag(beta) A)^-1 diag(beta)
 //     o_i = (q_i b_i)^T S0 + sum_{j<=i} P_ij u_j
 //     S   = diag(b_16) S0 + sum_j (k_j b_16,j) u_j^T
-// which follows from unrolling the rules over the chunk.
+// which follows from unrolling the rules over the chunk.  HGRN2 is GLA with k = 1 - g.  WKV reads before it writes:
+//     P_ij = sum_d r_i k_j b_i-1,j  (j < i),  P_ii = sum_d r_i u k_i,  and r_i b_i-1 in place of q_i b_i.
 //
 // Two kernels.  rec_prep_kernel, parallel over all chunks and heads: convolution, unit vectors, decays, and everything above
 // that does not involve S0, written as one record per (chunk, head).  rec_scan_kernel, serial over the chunks of a sequence
@@ -153,12 +154,17 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
             if (a.taps <= 4) convolve(std::integral_constant<int, 4>(), pc, ch, dst, ld);
             else convolve(std::integral_constant<int, kMaxTaps>(), pc, ch, dst, ld);
         } else {
+            if (!rec_has_key(KIND) && idx >= DK / 2 && idx < DK) continue;  // its key comes with the forget gate
             float2 x[kC];
-            const float f = idx < DK / 2 ? qscale : 1.f;
+            const float f = KIND == REC_GLA && idx < DK / 2 ? qscale : 1.f;
 #pragma unroll
             for (int t = 0; t < kC; t++) x[t] = t < tn ? load2(proj + (size_t)(t0 + t) * a.ldp + pc) : make_float2(0.f, 0.f);
 #pragma unroll
-            for (int t = 0; t < kC; t++) *reinterpret_cast<float2 *>(dst + t * ld) = make_float2(x[t].x * f, x[t].y * f);
+            for (int t = 0; t < kC; t++) {
+                if (KIND == REC_HGRN2 && idx < DK / 2) x[t].x *= sigmoid_f<AT>(x[t].x), x[t].y *= sigmoid_f<AT>(x[t].y);
+                else x[t].x *= f, x[t].y *= f;
+                *reinterpret_cast<float2 *>(dst + t * ld) = x[t];
+            }
         }
     }
     // ---- decays (1 past the end: the state stays) and step sizes ----
@@ -166,13 +172,22 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
     for (int e = 0; e < ZN; e++) {
         const int idx = e * 256 + tid, t = idx / (DK / 2), c = 2 * (idx % (DK / 2));
         if (t >= kC) break;
-        float2 y = make_float2(1.f, 1.f);
+        float2 y = make_float2(1.f, 1.f), w = make_float2(0.f, 0.f);
         if (t < tn) {
             const float2 b = *reinterpret_cast<const float2 *>(a.decay_bias + h * DK + c);
             y.x = zr[e].x + b.x, y.y = zr[e].y + b.y;
             if (KIND == REC_GLA) y.x = -y.x, y.y = -y.y;
-            y.x = exp_f<AT>(-rate * softplus_f<AT>(y.x)), y.y = exp_f<AT>(-rate * softplus_f<AT>(y.y));
+            if (KIND == REC_HGRN2) {
+                const float2 low = *reinterpret_cast<const float2 *>(a.lower + h * DK + c);
+                const float2 f0 = forget_write<AT>(y.x, low.x), f1 = forget_write<AT>(y.y, low.y);
+                y = make_float2(f0.x, f1.x), w = make_float2(f0.y, f1.y);
+            } else if (KIND == REC_WKV) {
+                y.x = exp_neg_exp<AT>(y.x), y.y = exp_neg_exp<AT>(y.y);
+            } else {
+                y.x = exp_f<AT>(-rate * softplus_f<AT>(y.x)), y.y = exp_f<AT>(-rate * softplus_f<AT>(y.y));
+            }
         }
+        if (KIND == REC_HGRN2) *reinterpret_cast<float2 *>(sk + t * DK + c) = w;
         *reinterpret_cast<float2 *>(sg + t * DK + c) = y;
     }
     if (KIND == REC_DELTA && tid < kC) sbeta[tid] = tid < tn ? sigmoid_f<AT>(bl) : 0.f;
@@ -194,7 +209,11 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
     // ---- A and P: warp w takes keys j = w and 15 - w; the key decays step by step on its way to later tokens ----
     {
         const int js[2] = {warp, 15 - warp};
-        float v[2][32];
+        float v[2][32], bonus[NI];
+        if (KIND == REC_WKV) {
+#pragma unroll
+            for (int c = 0; c < NI; c++) bonus[c] = a.bonus[h * DK + lane + 32 * c];
+        }
 #pragma unroll
         for (int s = 0; s < 2; s++) {
             const int j = js[s];
@@ -207,6 +226,11 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
                 if (i >= j) {
 #pragma unroll
                     for (int c = 0; c < NI; c++) {
+                        if (KIND == REC_WKV) {  // the bonus for itself, undecayed for the next token
+                            p = fmaf(sq[i * DK + lane + 32 * c], i == j ? kk[c] * bonus[c] : kk[c], p);
+                            if (i > j) kk[c] *= sg[i * DK + lane + 32 * c];
+                            continue;
+                        }
                         if (i > j) kk[c] *= sg[i * DK + lane + 32 * c];
                         p = fmaf(sq[i * DK + lane + 32 * c], kk[c], p);
                         if (KIND == REC_DELTA) w = fmaf(sk[i * DK + lane + 32 * c], kk[c], w);
@@ -221,7 +245,7 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
                 else sA[(lane - 16) * kC + j] = tot;
             }
         }
-        if (KIND == REC_GLA) {
+        if (KIND != REC_DELTA) {
             const float tot = reduce32(v[0], lane);
             sP[(lane & 15) * kC + js[lane >> 4]] = tot;
         }
@@ -249,8 +273,9 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
             float kt[kC], b = 1.f;
 #pragma unroll
             for (int t = 0; t < kC; t++) {
+                if (KIND == REC_WKV) rq[at_tok(t, d, DK)] = sq[t * DK + d] * b;
                 b *= sg[t * DK + d];
-                rq[at_tok(t, d, DK)] = sq[t * DK + d] * b;
+                if (KIND != REC_WKV) rq[at_tok(t, d, DK)] = sq[t * DK + d] * b;
                 kt[t] = sk[t * DK + d] * b;
             }
             rb[d] = b;
@@ -484,7 +509,7 @@ static int32_t chunk_launch(const StepDesc &d, const RecArgs &a, int pdl, cudaSt
     int nw = std::min(groups, max_warps);
     while (nw > 1 && (groups % nw != 0 || (long long)a.heads * d.n_long * (groups / nw) < a.sm_count)) nw--;
     const size_t smem = sizeof(float) * kScanStages * scan_stage_floats(KIND, DK, 16 * nw);
-    rc = launch_early(rec_scan_kernel<KIND, DK>, dim3((unsigned)(a.heads * (groups / nw)), (unsigned)d.n_long), 32 * nw, smem, set2,
+    rc = launch_early(rec_scan_kernel<KIND == REC_DELTA ? REC_DELTA : REC_GLA, DK>, dim3((unsigned)(a.heads * (groups / nw)), (unsigned)d.n_long), 32 * nw, smem, set2,
                       sizeof(float) * kScanStages * scan_stage_floats(KIND, DK, 16 * max_warps), pdl, st, a, d.segs, d.long_segs, pdl);
     if (rc) return rc;
     return launch_early(rec_chunk_norm_kernel<AT, KIND>, dim3((unsigned)d.n_chunks, (unsigned)((kC * a.heads + 63) / 64)), 256, 0, set3, 0, pdl, st, a, d.segs,
@@ -506,8 +531,13 @@ static int32_t chunk_dispatch(const StepDesc &d, const RecArgs &a, int pdl, cuda
 
 int32_t launch_recurrent_chunks(bool f32, const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st) {
     if (d.n_chunks == 0) return JGPT_OK;
-    if (f32) return a.kind == REC_DELTA ? chunk_dispatch<float, REC_DELTA>(d, a, pdl, st) : chunk_dispatch<float, REC_GLA>(d, a, pdl, st);
-    return a.kind == REC_DELTA ? chunk_dispatch<__nv_bfloat16, REC_DELTA>(d, a, pdl, st) : chunk_dispatch<__nv_bfloat16, REC_GLA>(d, a, pdl, st);
+    switch (a.kind) {
+        case REC_GLA: return f32 ? chunk_dispatch<float, REC_GLA>(d, a, pdl, st) : chunk_dispatch<__nv_bfloat16, REC_GLA>(d, a, pdl, st);
+        case REC_DELTA: return f32 ? chunk_dispatch<float, REC_DELTA>(d, a, pdl, st) : chunk_dispatch<__nv_bfloat16, REC_DELTA>(d, a, pdl, st);
+        case REC_HGRN2: return f32 ? chunk_dispatch<float, REC_HGRN2>(d, a, pdl, st) : chunk_dispatch<__nv_bfloat16, REC_HGRN2>(d, a, pdl, st);
+        case REC_WKV: return f32 ? chunk_dispatch<float, REC_WKV>(d, a, pdl, st) : chunk_dispatch<__nv_bfloat16, REC_WKV>(d, a, pdl, st);
+    }
+    return fail(JGPT_ERR_INVALID_ARGUMENT, "recurrence %d", a.kind);
 }
 
 }  // namespace mix

@@ -39,6 +39,24 @@ __device__ __forceinline__ float warp_sum(float v) {
     return v;
 }
 
+// exp(-exp(y)): the decay of WKV.
+template <class AT>
+__device__ __forceinline__ float exp_neg_exp(float y) {
+    return exp_f<AT>(-exp_f<AT>(y));
+}
+// Forget gate f = l + (1 - l) sigmoid(z) of HGRN2 and 1 - f = (1 - l) sigmoid(-z), which a difference would round away.
+template <class AT>
+__device__ __forceinline__ float2 forget_write(float z, float low) {
+    return make_float2(low + (1.f - low) * sigmoid_f<AT>(z), (1.f - low) * sigmoid_f<AT>(-z));
+}
+__host__ __device__ constexpr bool rec_has_key(int kind) { return kind != REC_HGRN2; }   // a projection of its own for k
+__host__ __device__ constexpr bool rec_has_gate(int kind) { return kind != REC_HGRN2; }  // an output gate
+// Gate factor of a head's output from the gate projection.
+template <class AT, int KIND>
+__device__ __forceinline__ float out_gate(float g) {
+    return KIND == REC_DELTA ? sigmoid_f<AT>(g) : g * sigmoid_f<AT>(g);
+}
+
 // RMS norm over a head's value columns and its output gate, by one warp: raw fp32 values -> activations.
 template <class AT, int KIND>
 __device__ __forceinline__ void norm_gate_head(const RecArgs &a, int r, int h, int lane) {
@@ -49,10 +67,8 @@ __device__ __forceinline__ void norm_gate_head(const RecArgs &a, int r, int h, i
     AT *o = reinterpret_cast<AT *>(a.out) + (size_t)r * a.ldo + a.out_off + h * a.DV;
     const AT *gp = KIND == REC_DELTA ? reinterpret_cast<const AT *>(a.z) + (size_t)r * a.ldz + a.zg_off + h * a.DV
                                      : reinterpret_cast<const AT *>(a.proj) + (size_t)r * a.ldp + a.g_off + h * a.DV;
-    for (int c = lane; c < a.DV; c += 32) {
-        const float gt = load1(gp + c), sgt = sigmoid_f<AT>(gt);
-        store1(o + c, raw[c] * inv * a.norm_w[c] * (KIND == REC_DELTA ? sgt : gt * sgt));
-    }
+    const float *nw = a.norm_w + h * a.norm_stride;
+    for (int c = lane; c < a.DV; c += 32) store1(o + c, raw[c] * inv * nw[c] * (rec_has_gate(KIND) ? out_gate<AT, KIND>(load1(gp + c)) : 1.f));
 }
 
 }  // namespace mix

@@ -15,30 +15,37 @@ from . import binding as B
 from .kv_cache import KvPool
 from .runtime import Context
 
-MIX_ATTENTION, MIX_GLA, MIX_DELTA = 1, 2, 3
+MIX_ATTENTION, MIX_GLA, MIX_DELTA, MIX_HGRN2, MIX_WKV, MIX_LATENT = range(1, 7)
+NORM_LAYER, NORM_RMS = 0, 1
+FF_GATED_GELU, FF_XIELU = 0, 1
+NO_LIMIT = 1 << 30  # positions of a model without a table of them
 DTYPES = {"bfloat16": 0, "float32": 1}
 BLOCK_TOKENS = 16
 
 
 class _MixerSpec(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("kind", "heads", "kv_heads", "dim", "vdim", "chunk", "gate", "taps", "rank_a", "rank_g")] + \
-               [(n, C.c_float) for n in ("score_scale", "tau", "out_scale")]
+               [(n, C.c_float) for n in ("score_scale", "tau", "out_scale")] + \
+               [(n, C.c_int32) for n in ("window", "q_rank", "kv_rank", "rot_dim", "rot_dims", "kv_from")] + \
+               [(n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")]
 
 
 class _LayerSpec(C.Structure):
-    _fields_ = [("n_branches", C.c_int32), ("branch", _MixerSpec * 2), ("ff", C.c_int32)]
+    _fields_ = [("n_branches", C.c_int32), ("branch", _MixerSpec * 2), ("ff", C.c_int32), ("ff_kind", C.c_int32)]
 
 
 class _DecoderSpec(C.Structure):
-    _fields_ = [(n, C.c_int32) for n in ("vocab", "width", "max_positions", "n_layers", "embed_norm")] + \
-               [(n, C.c_float) for n in ("eps", "embed_scale", "logit_scale")]
+    _fields_ = [(n, C.c_int32) for n in ("vocab", "width", "max_positions", "n_layers", "embed_norm", "pos_table", "norm", "head", "layer_scale",
+                                           "depth_average")] + \
+               [(n, C.c_float) for n in ("eps", "embed_scale", "logit_scale", "residual_mult")]
 
 
 # tensor roles (JGPT_W_* of the header)
-W_EMBED, W_POS, W_EMBED_NORM, W_EMBED_NORM_B, W_FINAL_NORM, W_FINAL_NORM_B = range(6)
-W_NORM1, W_NORM1_B, W_NORM2, W_NORM2_B, W_FF_GATE, W_FF_UP, W_FF_DOWN = range(10, 17)
+W_EMBED, W_POS, W_EMBED_NORM, W_EMBED_NORM_B, W_FINAL_NORM, W_FINAL_NORM_B, W_HEAD = range(7)
+W_NORM1, W_NORM1_B, W_NORM2, W_NORM2_B, W_FF_GATE, W_FF_UP, W_FF_DOWN, W_LS1, W_LS2, W_DWA = range(10, 20)
 (W_Q, W_K, W_V, W_O, W_G, W_B, W_A1, W_A2, W_DECAY_BIAS, W_A_LOG, W_G1, W_G2, W_HEAD_NORM, W_CONV_Q, W_CONV_K,
- W_CONV_V) = range(20, 36)
+ W_CONV_V, W_MU_R, W_MU_K, W_MU_V, W_MU_G, W_MU_W, W_BONUS, W_LOWER, W_F, W_DQ, W_DQ_NORM, W_UQ, W_DKV, W_DKV_NORM, W_UK, W_UV,
+ W_FF_ACT) = range(20, 52)
 
 
 @dataclass
@@ -56,6 +63,17 @@ class Mixer:
     score_scale: float = 1.0
     tau: float = 1.0
     out_scale: float = 1.0
+    window: int = 0
+    q_rank: int = 0
+    kv_rank: int = 0
+    rot_dim: int = 0
+    rot_dims: int = 0
+    kv_from: int = 0  # 1 + the layer whose latent cache is read, 0: its own
+    rot_base: float = 0.0
+    rot_factor: float = 0.0
+    rot_original: float = 0.0
+    rot_fast: float = 0.0
+    rot_slow: float = 0.0
     tensors: dict = field(default_factory=dict)  # role -> tensor name
 
 
@@ -64,6 +82,7 @@ class Layer:
     branches: list
     ff: int = 0
     tensors: dict = field(default_factory=dict)
+    ff_kind: int = FF_GATED_GELU
 
 
 @dataclass
@@ -76,6 +95,12 @@ class DecoderConfig:
     embed_norm: bool = False
     embed_scale: float = 1.0
     logit_scale: float = 1.0
+    pos_table: bool = True
+    norm: int = NORM_LAYER
+    head: bool = False
+    layer_scale: bool = False
+    depth_average: bool = False
+    residual_mult: float = 1.0
     tensors: dict = field(default_factory=dict)
 
     def all_tensors(self):
@@ -101,12 +126,14 @@ class DecoderModel:
         for spec, layer in zip(layers, config.layers):
             if not 1 <= len(layer.branches) <= 2:
                 raise ValueError(f"a layer has one or two mixer branches, not {len(layer.branches)}")
-            spec.n_branches, spec.ff = len(layer.branches), layer.ff
+            spec.n_branches, spec.ff, spec.ff_kind = len(layer.branches), layer.ff, layer.ff_kind
             for b, m in zip(spec.branch, layer.branches):
                 for n, _ in _MixerSpec._fields_:
                     setattr(b, n, int(m.gate) if n == "gate" else getattr(m, n))
-        top = _DecoderSpec(config.vocab, config.width, config.max_positions, len(config.layers), int(config.embed_norm),
-                           config.eps, config.embed_scale, config.logit_scale)
+        top = _DecoderSpec(n_layers=len(config.layers))
+        for n, t in _DecoderSpec._fields_:
+            if n != "n_layers":
+                setattr(top, n, int(getattr(config, n)) if t is C.c_int32 else getattr(config, n))
         h = C.c_uint64()
         B.check(self._lib.jgpt_decoder_create(ctx.handle, C.byref(top), layers, DTYPES[dtype], maxRows, C.byref(h)))
         self.handle = h.value
@@ -126,7 +153,7 @@ class DecoderModel:
                 raise ValueError(f"{name}: {e}") from None
 
     def newPool(self, n_blocks, max_seqs, max_blocks_per_seq=None) -> "DecoderPool":
-        return DecoderPool(self, n_blocks, max_seqs, max_blocks_per_seq or -(-self.maxSeqLen // BLOCK_TOKENS))
+        return DecoderPool(self, n_blocks, max_seqs, max_blocks_per_seq or min(n_blocks, -(-self.maxSeqLen // BLOCK_TOKENS)))
 
     # ---- forward step --------------------------------------------------------------------------
     def step(self, pool: KvPool, seqs, tokens, want=(), want_logits=True, want_next=False):

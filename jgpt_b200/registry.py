@@ -96,3 +96,55 @@ def somopel(c, shape_of) -> D.DecoderConfig:
     _norm(names, D.W_FINAL_NORM, "final.norm")
     return D.DecoderConfig(c["vocab"], c["width"], c["max_positions"], c["norm"]["eps"], layers, embed_norm=True,
                            embed_scale=c["embedding"]["scale"], logit_scale=c["logit_scale"], tensors=names)
+
+
+# ---- Zusepel -------------------------------------------------------------------------------------------
+def _hgrn2(m, p):
+    return D.Mixer(D.MIX_HGRN2, m["heads"], m["heads"], m["dim"], m["vdim"],
+                   tensors={D.W_Q: p + "q", D.W_F: p + "f", D.W_DECAY_BIAS: p + "f.b", D.W_LOWER: p + "lower", D.W_V: p + "v", D.W_HEAD_NORM: p + "norm",
+                            D.W_O: p + "o"})
+
+
+def _wkv(m, p, shape_of):
+    return D.Mixer(D.MIX_WKV, m["heads"], m["heads"], m["dim"], m["dim"], rank_a=shape_of(p + "w1")[0],
+                   tensors={D.W_MU_R: p + "mu.r", D.W_MU_K: p + "mu.k", D.W_MU_V: p + "mu.v", D.W_MU_G: p + "mu.g", D.W_MU_W: p + "mu.w", D.W_Q: p + "r",
+                            D.W_K: p + "k", D.W_V: p + "v", D.W_G: p + "g", D.W_A1: p + "w1", D.W_A2: p + "w2", D.W_DECAY_BIAS: p + "w0",
+                            D.W_BONUS: p + "u", D.W_HEAD_NORM: p + "norm", D.W_O: p + "o"})
+
+
+def _latent(m, p):
+    rot, names = m["rot"], {D.W_DQ: p + "dq", D.W_DQ_NORM: p + "dq.norm", D.W_UQ: p + "uq", D.W_UK: p + "uk", D.W_UV: p + "uv", D.W_O: p + "o"}
+    shared = m.get("kv_from")
+    if shared is None:
+        names.update({D.W_DKV: p + "dkv", D.W_DKV_NORM: p + "dkv.norm"})
+    yarn = rot.get("scaling")
+    return D.Mixer(D.MIX_LATENT, m["heads"], m["heads"], m["dim"], m["vdim"], window=(m.get("mask") or {}).get("size", 0), q_rank=m["q_rank"],
+                   kv_rank=m["kv_rank"], rot_dim=m["rot_dim"], rot_dims=rot["dims"], kv_from=0 if shared is None else 1 + shared, score_scale=m["scale"],
+                   rot_base=rot["base"], **({"rot_" + k: yarn[k] for k in ("factor", "original", "fast", "slow")} if yarn else {}), tensors=names)
+
+
+@register("Zusepel")
+def zusepel(c, shape_of) -> D.DecoderConfig:
+    """Layers of three kinds in any order: 'latent_attention' (sliding window, YaRN rotation, a layer may read an earlier
+    layer's cache), 'wkv' and 'hgrn2' (recurrences); RMS norms, layer scales, averages over the depth, an xIELU feed-forward
+    part, no table of positions."""
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        p, m, mlp = f"l{i}.", e["mixer"], e["mlp"]
+        names = {D.W_NORM1: p + "norm1", D.W_LS1: p + "ls1", D.W_DWA: p + "dwa"}
+        if e["type"] == "latent_attention":
+            mixer = _latent(m, p + "mix.")
+        elif e["type"] == "wkv":
+            mixer = _wkv(m, p + "mix.", shape_of)
+        elif e["type"] == "hgrn2":
+            mixer = _hgrn2(m, p + "mix.")
+        else:
+            raise ValueError(f"layer {i}: mixer type {e['type']!r}")
+        if mlp is not None:
+            if mlp["kind"] != "dense":
+                raise ValueError(f"layer {i}: feed-forward kind {mlp['kind']!r}")
+            names.update({D.W_NORM2: p + "norm2", D.W_LS2: p + "ls2", D.W_FF_UP: p + "mlp.up", D.W_FF_DOWN: p + "mlp.down", D.W_FF_ACT: p + "mlp.act"})
+        layers.append(D.Layer([mixer], mlp["ff"] if mlp else 0, names, D.FF_XIELU))
+    names = {D.W_EMBED: "embed", D.W_FINAL_NORM: "final.norm", D.W_HEAD: "head"}
+    return D.DecoderConfig(c["vocab"], c["width"], D.NO_LIMIT, c["norm"]["eps"], layers, pos_table=False, norm=D.NORM_RMS, head=True, layer_scale=True,
+                           depth_average=True, residual_mult=c["residual_mult"], tensors=names)
