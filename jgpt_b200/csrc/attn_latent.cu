@@ -14,6 +14,7 @@
 #include "attn_mma.cuh"
 
 #include <algorithm>
+#include <type_traits>
 
 namespace jgpt {
 namespace mix {
@@ -30,35 +31,44 @@ __device__ __forceinline__ float rotated(const AT *x, const float2 *cs, int half
     return j < half ? u * t.x - v * t.y : v * t.x + u * t.y;
 }
 
-// One warp per (row, part): part 0 the query latent, part 1 the key latent and the rotated part.
+// A block per row, 128 threads per part: part 0 the query latent, part 1 the key latent and the rotated part.
 template <class AT>
-__global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs a, const int *__restrict__ seq, const int *__restrict__ pos, int rows, int pdl) {
-    const int item = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, parts = a.own_cache ? 2 : 1;
+__global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs a, const int *__restrict__ seq, const int *__restrict__ pos, int pdl) {
+    constexpr int NT = 128;
+    __shared__ float red[8];
+    const int r = blockIdx.x, part = threadIdx.x / NT, t = threadIdx.x % NT;
     if (pdl & 2) griddep_launch_dependents();
     if (pdl & 1) griddep_wait();
-    if (item >= rows * parts) return;
-    const int r = item / parts, part = item % parts;
     const AT *proj = reinterpret_cast<const AT *>(a.proj) + (size_t)r * a.ldp;
     const AT *src = proj + (part ? a.c_off : a.dq_off);
     const float *gamma = part ? a.dkv_norm : a.dq_norm;
     const int n = part ? a.kv_rank : a.q_rank, padded = part ? a.KR : a.ldcq;
-    float ss = 0.f;
-    for (int j = lane; j < n; j += 32) {
-        const float v = act_load(src + j);
-        ss += v * v;
+    float ss = 0.f, v[8];  // the first 1024 elements stay in registers
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+        v[i] = t + NT * i < n ? act_load(src + t + NT * i) : 0.f;
+        ss += v[i] * v[i];
     }
+    for (int j = t + NT * 8; j < n; j += NT) ss += act_load(src + j) * act_load(src + j);
 #pragma unroll
     for (int off = 16; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
-    const float inv = 1.f / sqrtf(ss / (float)n + a.eps);
+    if ((t & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    const float inv = 1.f / sqrtf((red[4 * part] + red[4 * part + 1] + red[4 * part + 2] + red[4 * part + 3]) / (float)n + a.eps);
     AT *dst = reinterpret_cast<AT *>(a.cq) + (size_t)r * a.ldcq;
     if (part) {
         const int phys = page_of(a, seq[r], pos[r]);
         if (phys < 0) return;
         dst = reinterpret_cast<AT *>(a.kv) + ((size_t)phys * kBlockTokens + pos[r] % kBlockTokens) * a.LDR;
     }
-    for (int j = lane; j < padded; j += 32) act_store(dst + j, j < n ? act_load(src + j) * inv * gamma[j] : 0.f);
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+        const int j = t + NT * i;
+        if (j < padded) act_store(dst + j, j < n ? v[i] * inv * gamma[j] : 0.f);
+    }
+    for (int j = t + NT * 8; j < padded; j += NT) act_store(dst + j, j < n ? act_load(src + j) * inv * gamma[j] : 0.f);
     if (part)
-        for (int j = lane; j < a.RR; j += 32)
+        for (int j = t; j < a.RR; j += NT)
             act_store(dst + a.KR + j, j < a.rot_dim ? rotated(proj + a.r_off, a.cs + (size_t)r * a.half, a.half, j) : 0.f);
 }
 
@@ -110,279 +120,295 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentArgs a, co
 // ------------------------------------------------------------------------------------------------
 // On the latents, bf16
 // ------------------------------------------------------------------------------------------------
-// CTA = 16 MT (token, head) rows of an entry, eight warps, tiles of 64 keys = four pages brought in by bulk copies (a page is
-// contiguous, its row stride an odd number of 16-byte units, so ldmatrix is free of bank conflicts).  A warp scores eight keys
-// of a tile for all rows; the row maxima and the weights (bf16 high and low parts) meet in shared memory; then a warp adds up
-// its eighth of the latent's columns.  A cluster splits the keys; partial sums meet through cluster shared memory.
-constexpr int kLatKeys = 64, kLatPages = kLatKeys / kBlockTokens, kLatLP = kLatKeys + 8;
-constexpr size_t kMaxSmem = 232448;
+// CTA = 16 MT (token, head) rows of an entry, eight warps and a ninth that brings in tiles of 32 keys = two pages by bulk copies (a
+// page is contiguous, its row stride an odd number of 16-byte units, so ldmatrix is free of bank conflicts).  A warp scores eight
+// keys over half of the row's elements; the halves meet in shared memory, where every warp turns an eighth of the rows into
+// weights (bf16 high and low parts) and then adds up its eighth of the latent's columns.  A cluster splits the keys; partial sums
+// meet through cluster shared memory.
+constexpr int kLatKeys = 32, kLatPages = kLatKeys / kBlockTokens, kLatLS = kLatKeys + 8, kLatThreads = 288;
+constexpr size_t kMaxSmem = 232448 - 4096;  // dynamic; the rest is for static shared memory
 
 template <int MT>
 __host__ __device__ constexpr size_t latent_fixed_smem(int LDR) {
-    return (size_t)16 * MT * LDR * 2 + 2 * (size_t)16 * MT * kLatLP * 2 + sizeof(float) * 8 * 16 * MT;
+    return (size_t)16 * MT * LDR * 2 + sizeof(float) * 2 * 16 * MT * kLatLS + 2 * (size_t)16 * MT * kLatLS * 2;
 }
 
 template <int NTW, int MT>
-__global__ void __launch_bounds__(256, 1) latent_attn_kernel(const LatentArgs a, const Seg *__restrict__ segs, const int *__restrict__ list, int stages, int pdl) {
-    constexpr int KR = NTW * 64, ROWS = 16 * MT, MAXST = 8;
+__global__ void __launch_bounds__(kLatThreads, MT == 1 ? 2 : 1) latent_attn_kernel(const LatentArgs a, const Seg *__restrict__ segs, int stages, int pdl) {
+    constexpr int KR = NTW * 64, ROWS = 16 * MT, MAXST = 8, TPR = 256 / ROWS;
     extern __shared__ __align__(128) uint8_t lat_smem[];
-    __shared__ __align__(8) uint64_t full[MAXST];
+    __shared__ __align__(8) uint64_t full[MAXST], empty[MAXST];
     __shared__ int s_abort_mem;
+    __shared__ float s_ml[8][ROWS][2];           // row maxima and sums of every CTA of the cluster
+    __shared__ float s_m[ROWS], s_l[ROWS], s_f[ROWS];  // this CTA's running maxima, sums, the last tile's factors
     volatile int *s_abort = &s_abort_mem;
     const int LDR = a.LDR, RR = a.RR, H = a.heads;
     const uint32_t page_bytes = (uint32_t)(kBlockTokens * LDR * 2);
-    __nv_bfloat16 *ring = reinterpret_cast<__nv_bfloat16 *>(lat_smem);  // [stages][64][LDR]
-    __nv_bfloat16 *qs = ring + (size_t)stages * kLatKeys * LDR;         // [ROWS][LDR]
-    __nv_bfloat16 *ph = qs + (size_t)ROWS * LDR, *pl = ph + ROWS * kLatLP;
-    float *red = reinterpret_cast<float *>(pl + ROWS * kLatLP);         // [8][ROWS]
+    __nv_bfloat16 *ring = reinterpret_cast<__nv_bfloat16 *>(lat_smem);     // [stages][32][LDR]
+    __nv_bfloat16 *qs = ring + (size_t)stages * kLatKeys * LDR;            // [ROWS][LDR]
+    float *sp = reinterpret_cast<float *>(qs + (size_t)ROWS * LDR);        // [2][ROWS][kLatLS] half scores
+    __nv_bfloat16 *ph = reinterpret_cast<__nv_bfloat16 *>(sp + 2 * ROWS * kLatLS), *pl = ph + ROWS * kLatLS;  // [ROWS][kLatLS] weights
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t2 = 2 * (lane & 3);
     const int nsplit = gridDim.x, split = blockIdx.x, r0 = blockIdx.y * ROWS;
     if (pdl & 2) griddep_launch_dependents();
-    const Seg sg = segs[list[blockIdx.z]];
+    const Seg sg = segs[blockIdx.z];
     const int rows = sg.T * H;
-    if (r0 >= rows) return;
+    if (r0 >= rows) return;  // the whole cluster
+    if (nsplit > 1) cluster_arrive();
     const int first = window_first(sg.pos0 + r0 / H, a.window), last = sg.pos0 + min(rows - 1, r0 + ROWS - 1) / H;
     const int lo_page = first / kBlockTokens, n_pages = last / kBlockTokens - lo_page + 1;
     const int pg0 = lo_page + split * n_pages / nsplit, pg1 = lo_page + (split + 1) * n_pages / nsplit;
     const int n_tiles = (pg1 - pg0 + kLatPages - 1) / kLatPages;
     if (tid == 0) {
-        for (int s = 0; s < stages; s++) mbar_init(&full[s], 1);
+        for (int s = 0; s < stages; s++) mbar_init(&full[s], 1), mbar_init(&empty[s], 8);
         *s_abort = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
+    if (tid < ROWS) s_m[tid] = -INFINITY, s_l[tid] = 0.f;
+    // blocks of 32 pages, a page per lane (tables do not change inside a step)
+    int blocks = 0;
+    auto lookup = [&](int i) {
+        const int pg = pg0 + i * kLatPages + lane;
+        blocks = pg < pg1 ? max(page_of(a, sg.seq, pg * kBlockTokens), 0) : 0;
+    };
+    if (warp == 8) lookup(0);
     __syncthreads();
     if (pdl & 1) griddep_wait();
 
-    // warp 0 brings tiles in: lanes 0-3 a page each, its block looked up a tile ahead
-    int phys = 0;
-    auto lookup = [&](int i) {
-        const int pg = pg0 + i * kLatPages + lane;
-        phys = lane < kLatPages && pg < pg1 ? max(page_of(a, sg.seq, pg * kBlockTokens), 0) : 0;
-    };
-    auto fetch = [&](int i) {
-        const int s = i % stages, pg = pg0 + i * kLatPages, n = min(kLatPages, pg1 - pg);
-        if (lane == 0) mbar_expect_tx(&full[s], (uint32_t)n * page_bytes);
-        __syncwarp();
-        if (lane < n)
-            bulk_g2s(ring + ((size_t)s * kLatKeys + lane * kBlockTokens) * LDR, reinterpret_cast<const uint8_t *>(a.kv) + (size_t)phys * page_bytes, page_bytes,
-                     &full[s]);
-        lookup(i + 1);
-    };
-    int issued = 0;
-    if (warp == 0) {
-        lookup(0);
-        for (; issued < stages && issued < n_tiles; issued++) fetch(issued);
-    }
-    {  // query rows: q~, then the rotated part
-        const __nv_bfloat16 *qa = reinterpret_cast<const __nv_bfloat16 *>(a.qa) + (size_t)sg.row0 * H * KR;
-        for (int e = tid; e < ROWS * (KR / 8); e += 256) {
-            const int r = e / (KR / 8), c = e % (KR / 8) * 8;
-            const bool ok = r0 + r < rows;
-            cp_async16(qs + (size_t)r * LDR + c, qa + (size_t)(ok ? r0 + r : 0) * KR + c, ok);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-        for (int e = tid; e < ROWS * RR; e += 256) {
-            const int r = e / RR, j = e % RR, t = (r0 + r) / H, h = (r0 + r) % H;
-            float v = 0.f;
-            if (r0 + r < rows && j < a.rot_dim)
-                v = rotated(reinterpret_cast<const __nv_bfloat16 *>(a.q) + (size_t)(sg.row0 + t) * a.ldq + (size_t)h * a.DQ + a.DP,
-                            a.cs + (size_t)(sg.row0 + t) * a.half, a.half, j);
-            qs[(size_t)r * LDR + KR + j] = __float2bfloat16(v);
-        }
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
-    __syncthreads();
-
-    int lo[MT][2], hi[MT][2];
-    float m[MT][2], l[MT][2], o[MT][NTW][4];
-#pragma unroll
-    for (int i = 0; i < MT; i++)
-#pragma unroll
-        for (int e = 0; e < 2; e++) {
-            const int r = r0 + i * 16 + g + 8 * e;
-            hi[i][e] = r < rows ? sg.pos0 + r / H : -1;
-            lo[i][e] = r < rows ? window_first(hi[i][e], a.window) : 0;
-            m[i][e] = -INFINITY, l[i][e] = 0.f;
-        }
+    float o[MT][NTW][4];
 #pragma unroll
     for (int i = 0; i < MT; i++)
 #pragma unroll
         for (int n = 0; n < NTW; n++)
 #pragma unroll
             for (int e = 0; e < 4; e++) o[i][n][e] = 0.f;
-    const float sl = a.scale * 1.4426950408889634f;
-    const int ksteps = (KR + RR) / 16, end_key = min(last, pg1 * kBlockTokens - 1);
-    bool failed = false;
-    for (int it = 0; it < n_tiles; it++) {
-        const int s = it % stages, kb = (pg0 + it * kLatPages) * kBlockTokens;
-        __nv_bfloat16 *ks = ring + (size_t)s * kLatKeys * LDR;
-        const bool ok = mbar_wait_bounded(&full[s], (uint32_t)(it / stages) & 1u, a.status, s_abort);
-        if (kb + kLatKeys - 1 > end_key) {  // nothing is known about what lies behind the last key: its weight is zero, its values must be too
-            const int v0 = end_key - kb + 1, per = LDR / 8;
-            for (int e = tid; e < (kLatKeys - v0) * per; e += 256) *reinterpret_cast<uint4 *>(ks + (size_t)(v0 + e / per) * LDR + e % per * 8) = make_uint4(0, 0, 0, 0);
+    if (warp == 8) {
+        for (int i = 0; i < n_tiles; i++) {
+            const int s = i % stages, pg = pg0 + i * kLatPages, n = min(kLatPages, pg1 - pg), at = i % (32 / kLatPages) * kLatPages;
+            if (i > 0 && at == 0) lookup(i);
+            const int phys = __shfl_sync(0xffffffffu, blocks, at + lane % kLatPages);
+            if (i >= stages && !mbar_wait_bounded(&empty[s], (uint32_t)(i / stages - 1) & 1u, a.status, s_abort)) break;
+            if (lane == 0) mbar_expect_tx(&full[s], (uint32_t)n * page_bytes);
+            __syncwarp();
+            if (lane < n)
+                bulk_g2s(ring + ((size_t)s * kLatKeys + lane * kBlockTokens) * LDR, reinterpret_cast<const uint8_t *>(a.kv) + (size_t)phys * page_bytes,
+                         page_bytes, &full[s]);
         }
-        float sc[MT][4];
+        __syncwarp();
+        if (*s_abort)  // a wait ran out: give copies in flight a bounded chance to land before the memory goes
+            for (int s = 0; s < stages; s++)
+                for (uint32_t k = 0; k < (1u << 12) && !mbar_try_wait(&full[s], 0); k++) {
+                }
+    } else {
+        {  // query rows: q~, then the rotated part, TPR threads per row
+            const int r = tid / TPR, j0 = tid % TPR, t = (r0 + r) / H, h = (r0 + r) % H;
+            const bool ok = r0 + r < rows;
+            const __nv_bfloat16 *qa = reinterpret_cast<const __nv_bfloat16 *>(a.qa) + ((size_t)sg.row0 * H + (ok ? r0 + r : 0)) * KR;
+            for (int c = j0 * 8; c < KR; c += TPR * 8) cp_async16(qs + (size_t)r * LDR + c, qa + c, ok);
+            asm volatile("cp.async.commit_group;" ::: "memory");
+            const __nv_bfloat16 *qr = reinterpret_cast<const __nv_bfloat16 *>(a.q) + (size_t)(sg.row0 + (ok ? t : 0)) * a.ldq + (size_t)h * a.DQ + a.DP;
+            const float2 *cs = a.cs + (size_t)(sg.row0 + (ok ? t : 0)) * a.half;
+#pragma unroll 4
+            for (int j = j0; j < RR; j += TPR) qs[(size_t)r * LDR + KR + j] = __float2bfloat16(ok && j < a.rot_dim ? rotated(qr, cs, a.half, j) : 0.f);
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        named_bar_sync(1, 256);
+        // this lane's row and pair of keys when scores become weights: 16 lanes per row, two rows of a warp at a time
+        int lo[MT], hi[MT];
 #pragma unroll
-        for (int i = 0; i < MT; i++)
+        for (int i = 0; i < MT; i++) {
+            const int r = r0 + warp * 2 * MT + 2 * i + (lane >> 4);
+            hi[i] = r < rows ? sg.pos0 + r / H : -1;
+            lo[i] = r < rows ? window_first(hi[i], a.window) : 0;
+        }
+        const float sl = a.scale * 1.4426950408889634f;
+        const int ksteps = (KR + RR) / 16, khalf = (ksteps / 2 + 1) / 2 * 2, k_from = warp < 4 ? 0 : khalf, k_to = warp < 4 ? khalf : ksteps;
+        const int end_key = min(last, pg1 * kBlockTokens - 1);
+        for (int it = 0; it < n_tiles; it++) {
+            const int s = it % stages, kb = (pg0 + it * kLatPages) * kBlockTokens;
+            __nv_bfloat16 *ks = ring + (size_t)s * kLatKeys * LDR;
+            // when the wait runs out the status word is set: what follows works on whatever is there, and nobody looks at it
+            mbar_wait_bounded(&full[s], (uint32_t)(it / stages) & 1u, a.status, s_abort);
+            if (kb + kLatKeys - 1 > end_key) {  // nothing is known about what lies behind the last key: its weight is zero, its values must be too
+                const int v0 = end_key - kb + 1, per = LDR / 8;
+                for (int e = tid; e < (kLatKeys - v0) * per; e += 256) *reinterpret_cast<uint4 *>(ks + (size_t)(v0 + e / per) * LDR + e % per * 8) = make_uint4(0, 0, 0, 0);
+            }
+            {  // eight keys, half of the elements; even and odd steps are two chains of products, operands of six steps in flight
+                float sc[MT][4], sc2[MT][4];
 #pragma unroll
-            for (int e = 0; e < 4; e++) sc[i][e] = 0.f;
-        const __nv_bfloat16 *kw = ks + (size_t)(warp * 8 + (lane & 7)) * LDR + (lane >> 3) * 8, *qw = qs + (size_t)(lane & 15) * LDR + (lane >> 4) * 8;
-        auto score = [&](int kk, uint32_t b0, uint32_t b1) {
+                for (int i = 0; i < MT; i++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) sc[i][e] = sc2[i][e] = 0.f;
+                const __nv_bfloat16 *kw = ks + (size_t)((warp & 3) * 8 + (lane & 7)) * LDR + (lane >> 3) * 8, *qw = qs + (size_t)(lane & 15) * LDR + (lane >> 4) * 8;
+                auto steps = [&](auto count, int kk) {
+                    constexpr int P = decltype(count)::value;  // pairs of steps
+                    uint32_t b[P][4], q[2 * P][MT][4];
+#pragma unroll
+                    for (int p = 0; p < P; p++) {
+                        ldmatrix_x4(b[p], kw + (kk + 2 * p) * 16);
+#pragma unroll
+                        for (int i = 0; i < MT; i++) {
+                            ldmatrix_x4(q[2 * p][i], qw + (size_t)i * 16 * LDR + (kk + 2 * p) * 16);
+                            ldmatrix_x4(q[2 * p + 1][i], qw + (size_t)i * 16 * LDR + (kk + 2 * p + 1) * 16);
+                        }
+                    }
+#pragma unroll
+                    for (int p = 0; p < P; p++)
+#pragma unroll
+                        for (int i = 0; i < MT; i++) {
+                            mma_bf16(sc[i], q[2 * p][i], b[p][0], b[p][1]);
+                            mma_bf16(sc2[i], q[2 * p + 1][i], b[p][2], b[p][3]);
+                        }
+                };
+                int kk = k_from;
+                for (; kk + 6 <= k_to; kk += 6) steps(std::integral_constant<int, 3>(), kk);
+                for (; kk + 2 <= k_to; kk += 2) steps(std::integral_constant<int, 1>(), kk);
+                if (kk < k_to) {  // the upper two matrices would lie past the row: their lanes read the lower ones again
+                    uint32_t b[4], q[4];
+                    ldmatrix_x4(b, kw + kk * 16 - (lane >= 16 ? 16 : 0));
+#pragma unroll
+                    for (int i = 0; i < MT; i++) {
+                        ldmatrix_x4(q, qw + (size_t)i * 16 * LDR + kk * 16);
+                        mma_bf16(sc[i], q, b[0], b[1]);
+                    }
+                }
+                float *w = sp + (size_t)(warp >> 2) * ROWS * kLatLS + (warp & 3) * 8 + t2;
+#pragma unroll
+                for (int i = 0; i < MT; i++)
+#pragma unroll
+                    for (int e = 0; e < 2; e++)
+                        *reinterpret_cast<float2 *>(w + (i * 16 + g + 8 * e) * kLatLS) = make_float2(sc[i][2 * e] + sc2[i][2 * e], sc[i][2 * e + 1] + sc2[i][2 * e + 1]);
+            }
+            named_bar_sync(1, 256);
 #pragma unroll
             for (int i = 0; i < MT; i++) {
-                uint32_t q[4];
-                ldmatrix_x4(q, qw + (size_t)i * 16 * LDR + kk * 16);
-                mma_bf16(sc[i], q, b0, b1);
-            }
-        };
-        int kk = 0;
-#pragma unroll 4
-        for (; kk + 1 < ksteps; kk += 2) {
-            uint32_t b[4];
-            ldmatrix_x4(b, kw + kk * 16);
-            score(kk, b[0], b[1]);
-            score(kk + 1, b[2], b[3]);
-        }
-        if (kk < ksteps) {  // the upper two matrices would lie past the row: their lanes read the lower ones again
-            uint32_t b[4];
-            ldmatrix_x4(b, kw + kk * 16 - (lane >= 16 ? 16 : 0));
-            score(kk, b[0], b[1]);
-        }
-        const int key = kb + warp * 8 + t2;
+                const int r = warp * 2 * MT + 2 * i + (lane >> 4), c = 2 * (lane & 15), key = kb + c, top = min(hi[i], end_key);
+                const float2 u = *reinterpret_cast<const float2 *>(sp + r * kLatLS + c), w = *reinterpret_cast<const float2 *>(sp + (ROWS + r) * kLatLS + c);
+                const float m0 = s_m[r];
+                const float x0 = key >= lo[i] && key <= top ? (u.x + w.x) * sl : -INFINITY, x1 = key + 1 >= lo[i] && key + 1 <= top ? (u.y + w.y) * sl : -INFINITY;
+                float mx = fmaxf(x0, x1);
 #pragma unroll
-        for (int i = 0; i < MT; i++)
-#pragma unroll
-            for (int e = 0; e < 2; e++) {
-                float mx = -INFINITY;
-#pragma unroll
-                for (int c = 0; c < 2; c++) {
-                    float &x = sc[i][2 * e + c];
-                    x = key + c >= lo[i][e] && key + c <= min(hi[i][e], end_key) ? x * sl : -INFINITY;
-                    mx = fmaxf(mx, x);
-                }
-                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-                if ((lane & 3) == 0) red[warp * ROWS + i * 16 + g + 8 * e] = mx;
-            }
-        if (__syncthreads_or(!ok)) {
-            failed = true;
-            break;
-        }
-        float f[MT][2];
-        bool moved = false;
-#pragma unroll
-        for (int i = 0; i < MT; i++)
-#pragma unroll
-            for (int e = 0; e < 2; e++) {
-                float mn = m[i][e];
-#pragma unroll
-                for (int w = 0; w < 8; w++) mn = fmaxf(mn, red[w * ROWS + i * 16 + g + 8 * e]);
-                f[i][e] = mn == -INFINITY ? 1.f : fast_exp2(m[i][e] - mn);
-                m[i][e] = mn;
-                const float ref = mn == -INFINITY ? 0.f : mn;
-                const float p0 = fast_exp2(sc[i][2 * e] - ref), p1 = fast_exp2(sc[i][2 * e + 1] - ref);
-                l[i][e] = l[i][e] * f[i][e] + p0 + p1;
-                moved = moved || f[i][e] != 1.f;
+                for (int off = 8; off >= 1; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+                mx = fmaxf(mx, m0);
+                const float ref = mx == -INFINITY ? 0.f : mx, p0 = fast_exp2(x0 - ref), p1 = fast_exp2(x1 - ref);
                 uint32_t h2, l2;
                 split_pair(p0, p1, h2, l2);
-                const int at = (i * 16 + g + 8 * e) * kLatLP + warp * 8 + t2;
-                *reinterpret_cast<uint32_t *>(ph + at) = h2, *reinterpret_cast<uint32_t *>(pl + at) = l2;
+                *reinterpret_cast<uint32_t *>(ph + r * kLatLS + c) = h2, *reinterpret_cast<uint32_t *>(pl + r * kLatLS + c) = l2;
+                float sum = p0 + p1;
+#pragma unroll
+                for (int off = 8; off >= 1; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+                if ((lane & 15) == 0) {
+                    const float f = mx == -INFINITY ? 1.f : fast_exp2(m0 - mx);
+                    s_m[r] = mx, s_f[r] = f, s_l[r] = s_l[r] * f + sum;
+                }
             }
-        __syncthreads();
-        if (__any_sync(0xffffffffu, moved)) {
+            named_bar_sync(1, 256);
+            const __nv_bfloat16 *vw = ks + (size_t)(((lane >> 3) & 1) * 8 + (lane & 7)) * LDR + warp * NTW * 8 + (lane >> 4) * 8;
+            const int pw = (lane & 15) * kLatLS + (lane >> 4) * 8;
+            bool moved = false;
+            float f[MT][2];
 #pragma unroll
             for (int i = 0; i < MT; i++)
 #pragma unroll
-                for (int n = 0; n < NTW; n++) o[i][n][0] *= f[i][0], o[i][n][1] *= f[i][0], o[i][n][2] *= f[i][1], o[i][n][3] *= f[i][1];
-        }
-        const __nv_bfloat16 *vw = ks + (size_t)(((lane >> 3) & 1) * 8 + (lane & 7)) * LDR + warp * NTW * 8 + (lane >> 4) * 8;
-        const int pw = (lane & 15) * kLatLP + (lane >> 4) * 8;
+                for (int e = 0; e < 2; e++) {
+                    f[i][e] = s_f[i * 16 + g + 8 * e];
+                    moved = moved || f[i][e] != 1.f;
+                }
+            if (__any_sync(0xffffffffu, moved)) {
 #pragma unroll
-        for (int k16 = 0; k16 < kLatKeys / 16; k16++) {
-            uint32_t wh[MT][4], wl[MT][4];
+                for (int i = 0; i < MT; i++)
 #pragma unroll
-            for (int i = 0; i < MT; i++) {
-                ldmatrix_x4(wh[i], ph + i * 16 * kLatLP + pw + k16 * 16);
-                ldmatrix_x4(wl[i], pl + i * 16 * kLatLP + pw + k16 * 16);
+                    for (int n = 0; n < NTW; n++) o[i][n][0] *= f[i][0], o[i][n][1] *= f[i][0], o[i][n][2] *= f[i][1], o[i][n][3] *= f[i][1];
             }
 #pragma unroll
-            for (int n = 0; n < NTW; n += 2) {
-                uint32_t b[4];
-                ldmatrix_x4_trans(b, vw + (size_t)k16 * 16 * LDR + n * 8);
+            for (int k16 = 0; k16 < kLatKeys / 16; k16++) {
+                uint32_t wh[MT][4], wl[MT][4], b[NTW / 2][4];
+#pragma unroll
+                for (int n = 0; n < NTW / 2; n++) ldmatrix_x4_trans(b[n], vw + (size_t)k16 * 16 * LDR + n * 16);
 #pragma unroll
                 for (int i = 0; i < MT; i++) {
-                    mma_bf16(o[i][n], wh[i], b[0], b[1]);
-                    mma_bf16(o[i][n], wl[i], b[0], b[1]);
-                    mma_bf16(o[i][n + 1], wh[i], b[2], b[3]);
-                    mma_bf16(o[i][n + 1], wl[i], b[2], b[3]);
+                    ldmatrix_x4(wh[i], ph + i * 16 * kLatLS + pw + k16 * 16);
+                    ldmatrix_x4(wl[i], pl + i * 16 * kLatLS + pw + k16 * 16);
                 }
+#pragma unroll
+                for (int n = 0; n < NTW / 2; n++)
+#pragma unroll
+                    for (int i = 0; i < MT; i++) {
+                        mma_bf16(o[i][2 * n], wh[i], b[n][0], b[n][1]);
+                        mma_bf16(o[i][2 * n + 1], wh[i], b[n][2], b[n][3]);
+                        mma_bf16(o[i][2 * n], wl[i], b[n][0], b[n][1]);
+                        mma_bf16(o[i][2 * n + 1], wl[i], b[n][2], b[n][3]);
+                    }
             }
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&empty[s]);  // this warp is done with the stage
         }
-        __syncthreads();  // the stage, the maxima and the weights are free
-        if (warp == 0 && issued < n_tiles) fetch(issued++);
     }
-    if (failed) {  // give copies in flight a bounded chance to land, then leave together
-        if (tid == 0)
-            for (int i = 0; i < stages; i++)
-                for (uint32_t k = 0; k < (1u << 16) && !mbar_try_wait(&full[i], (uint32_t)((n_tiles - 1 - i) / stages) & 1u); k++) {
-                }
-        __syncthreads();
-        return;
-    }
-#pragma unroll
-    for (int i = 0; i < MT; i++)
-#pragma unroll
-        for (int e = 0; e < 2; e++) {
-            l[i][e] += __shfl_xor_sync(0xffffffffu, l[i][e], 1);
-            l[i][e] += __shfl_xor_sync(0xffffffffu, l[i][e], 2);
-            if ((lane & 3) == 0) red[warp * ROWS + i * 16 + g + 8 * e] = l[i][e];
-        }
     __syncthreads();
-#pragma unroll
-    for (int i = 0; i < MT; i++)
-#pragma unroll
-        for (int e = 0; e < 2; e++) {
-            l[i][e] = 0.f;
-#pragma unroll
-            for (int w = 0; w < 8; w++) l[i][e] += red[w * ROWS + i * 16 + g + 8 * e];
-        }
     __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(a.qa) + ((size_t)sg.row0 * H + r0) * KR;
     if (nsplit == 1) {
+        if (warp == 8) return;
 #pragma unroll
         for (int i = 0; i < MT; i++)
 #pragma unroll
             for (int e = 0; e < 2; e++) {
                 const int r = i * 16 + g + 8 * e;
                 if (r0 + r >= rows) continue;
-                const float f = l[i][e] > 0.f ? 1.f / l[i][e] : 0.f;
+                const float l = s_l[r], f = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll
                 for (int n = 0; n < NTW; n++)
                     *reinterpret_cast<uint32_t *>(out + (size_t)r * KR + (warp * NTW + n) * 8 + t2) = bf16_pair(o[i][n][2 * e] * f, o[i][n][2 * e + 1] * f);
             }
         return;
     }
-    float *mo = reinterpret_cast<float *>(lat_smem), *ml = mo + (size_t)ROWS * KR;  // [ROWS][KR], [ROWS][m, l], in place of the ring
+    float *mo = reinterpret_cast<float *>(lat_smem);  // [ROWS][KR], in place of the ring
+    cluster_wait();                                   // every CTA of the cluster has started: its shared memory may be written
+    for (int e = tid; e < ROWS * nsplit; e += kLatThreads) {
+        st_cluster_f32(&s_ml[split][e % ROWS][0], (uint32_t)(e / ROWS), s_m[e % ROWS]);
+        st_cluster_f32(&s_ml[split][e % ROWS][1], (uint32_t)(e / ROWS), s_l[e % ROWS]);
+    }
+    if (warp < 8) {
 #pragma unroll
-    for (int i = 0; i < MT; i++)
+        for (int i = 0; i < MT; i++)
 #pragma unroll
-        for (int e = 0; e < 2; e++) {
-            const int r = i * 16 + g + 8 * e;
-            if (warp == 0 && (lane & 3) == 0) ml[2 * r] = m[i][e], ml[2 * r + 1] = l[i][e];
+            for (int e = 0; e < 2; e++)
 #pragma unroll
-            for (int n = 0; n < NTW; n++)
-                *reinterpret_cast<float2 *>(mo + (size_t)r * KR + (warp * NTW + n) * 8 + t2) = make_float2(o[i][n][2 * e], o[i][n][2 * e + 1]);
-        }
+                for (int n = 0; n < NTW; n++)
+                    *reinterpret_cast<float2 *>(mo + (size_t)(i * 16 + g + 8 * e) * KR + (warp * NTW + n) * 8 + t2) = make_float2(o[i][n][2 * e], o[i][n][2 * e + 1]);
+    }
     cluster_sync();
-    const int valid = min(ROWS, rows - r0), c0 = split * KR / nsplit, cn = (split + 1) * KR / nsplit - c0;
-    for (int e = tid; e < valid * cn; e += 256) {
-        const int r = e / cn, c = c0 + e % cn;
-        float mx = -INFINITY, sum = 0.f, acc = 0.f;
-        for (int s = 0; s < nsplit; s++) mx = fmaxf(mx, ld_cluster_f32(ml + 2 * r, (uint32_t)s));
-        for (int s = 0; s < nsplit; s++) {
-            const float ms = ld_cluster_f32(ml + 2 * r, (uint32_t)s), f = ms == -INFINITY ? 0.f : fast_exp2(ms - mx);
-            sum += f * ld_cluster_f32(ml + 2 * r + 1, (uint32_t)s), acc += f * ld_cluster_f32(mo + (size_t)r * KR + c, (uint32_t)s);
+    // every part's weight per row, then this CTA's share of the columns (the split is 2, 4 or 8)
+    const int valid = min(ROWS, rows - r0), cn = KR / nsplit, c0 = split * cn;
+    if (tid < ROWS) {
+        float ms[8], mx = -INFINITY, sum = 0.f;
+#pragma unroll
+        for (int s = 0; s < 8; s++) {
+            ms[s] = s < nsplit ? s_ml[s][tid][0] : -INFINITY;
+            mx = fmaxf(mx, ms[s]);
         }
-        out[(size_t)r * KR + c] = __float2bfloat16(sum > 0.f ? acc / sum : 0.f);
+#pragma unroll
+        for (int s = 0; s < 8; s++) {
+            ms[s] = ms[s] == -INFINITY ? 0.f : fast_exp2(ms[s] - mx);
+            if (s < nsplit) sum += ms[s] * s_ml[s][tid][1];
+        }
+#pragma unroll
+        for (int s = 0; s < 8; s++) sp[s * ROWS + tid] = sum > 0.f ? ms[s] / sum : 0.f;
+    }
+    __syncthreads();
+    for (int e = tid; e < valid * (cn / 4); e += kLatThreads) {
+        const int r = e / (cn / 4), c = c0 + e % (cn / 4) * 4;
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int s0 = 0; s0 < nsplit; s0 += 4) {
+            float4 x[4];
+#pragma unroll
+            for (int s = 0; s < 4; s++) x[s] = s0 + s < nsplit ? ld_cluster_f32x4(mo + (size_t)r * KR + c, (uint32_t)(s0 + s)) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int s = 0; s < 4; s++) {
+                const float w = sp[(s0 + s) * ROWS + r];
+                acc.x = fmaf(w, x[s].x, acc.x), acc.y = fmaf(w, x[s].y, acc.y), acc.z = fmaf(w, x[s].z, acc.z), acc.w = fmaf(w, x[s].w, acc.w);
+            }
+        }
+        *reinterpret_cast<uint2 *>(out + (size_t)r * KR + c) = make_uint2(bf16_pair(acc.x, acc.y), bf16_pair(acc.z, acc.w));
     }
     cluster_sync();  // nobody leaves while its shared memory is being read
 }
@@ -404,14 +430,15 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const LatentArgs a, 
     for (int j = lane; j < n; j += 32) dst[j] = src[j];
 }
 
-// CTA = 64 query tokens of one head: 4 warps x 16 rows; tiles of 64 keys through two stages.
+// CTA = 64 query tokens of one head: 4 warps x 16 rows; tiles of 32 keys through two stages (small, for three CTAs on an SM).
+constexpr int kTileKeys = 32;
 template <int DK, int DV>
-__host__ __device__ constexpr size_t latent_tile_smem() { return (size_t)64 * (DK + 8) * 2 + 2 * (size_t)kLatKeys * (DK + DV + 16) * 2; }
+__host__ __device__ constexpr size_t latent_tile_smem() { return (size_t)64 * (DK + 8) * 2 + 2 * (size_t)kTileKeys * (DK + DV + 16) * 2; }
 
 template <int DK, int DV>
-__global__ void __launch_bounds__(128) latent_tile_kernel(const LatentArgs a, const Seg *__restrict__ segs, const LatentEntry *__restrict__ entries,
+__global__ void __launch_bounds__(128, DK <= 192 ? 3 : 1) latent_tile_kernel(const LatentArgs a, const Seg *__restrict__ segs, const LatentEntry *__restrict__ entries,
                                                           const int2 *__restrict__ tiles, int pdl) {
-    constexpr int LK = DK + 8, LV = DV + 8, CK = DK / 8, CV = DV / 8;
+    constexpr int LK = DK + 8, LV = DV + 8, CK = DK / 8;
     extern __shared__ __align__(128) uint8_t lat_smem[];
     __nv_bfloat16 *qs = reinterpret_cast<__nv_bfloat16 *>(lat_smem), *kv_s = qs + 64 * LK;  // stages: [K 64 x LK | V 64 x LV]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, h = blockIdx.y;
@@ -437,21 +464,23 @@ __global__ void __launch_bounds__(128) latent_tile_kernel(const LatentArgs a, co
     const __nv_bfloat16 *vx = reinterpret_cast<const __nv_bfloat16 *>(a.kvx) + (size_t)en.row0 * a.ldx + (size_t)a.heads * a.DP + (size_t)h * a.DVm;
     const int n_keys = p1 - en.key0 + 1;
     auto load = [&](int stage, int kb) {
-        __nv_bfloat16 *dk = kv_s + (size_t)stage * kLatKeys * (LK + LV), *dv = dk + kLatKeys * LK;
-        for (int e = tid; e < kLatKeys * (CK + CV); e += 128) {
-            const int j = e / (CK + CV), x = e % (CK + CV), key = kb + j;
-            const bool in = key < n_keys;
-            const size_t row = in ? key : 0;
-            if (x < CK) {
-                const int c = x * 8;
-                const bool rot = c >= a.DP;
-                const bool ok = in && c < a.DP + a.RR;
-                cp_async16(dk + j * LK + c, rot ? cx + row * (a.KR + a.RR) + (ok ? c - a.DP : 0) : kx + row * a.ldx + c, ok);
-            } else {
-                const int c = (x - CK) * 8;
-                const bool ok = in && c < a.DVm;
-                cp_async16(dv + j * LV + c, vx + row * a.ldx + (ok ? c : 0), ok);
-            }
+        // four threads per key, chunks 4 i + (tid & 3)
+        const int j = tid >> 2, key = kb + j;
+        const bool in = key < n_keys;
+        const size_t row = in ? key : 0;
+        __nv_bfloat16 *dk = kv_s + (size_t)stage * kTileKeys * (LK + LV) + j * LK, *dv = kv_s + (size_t)stage * kTileKeys * (LK + LV) + kTileKeys * LK + j * LV;
+        const __nv_bfloat16 *kr = kx + row * a.ldx, *rr = cx + row * (a.KR + a.RR), *vr = vx + row * a.ldx;
+#pragma unroll
+        for (int i = 0; i < DK / 32; i++) {
+            const int c = (4 * i + (tid & 3)) * 8;
+            const bool ok = in && c < a.DP + a.RR;
+            cp_async16(dk + c, c < a.DP ? kr + c : rr + (ok ? c - a.DP : 0), ok);
+        }
+#pragma unroll
+        for (int i = 0; i < DV / 32; i++) {
+            const int c = (4 * i + (tid & 3)) * 8;
+            const bool ok = in && c < a.DVm;
+            cp_async16(dv + c, vr + (ok ? c : 0), ok);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -472,17 +501,17 @@ __global__ void __launch_bounds__(128) latent_tile_kernel(const LatentArgs a, co
     const float sl = a.scale * 1.4426950408889634f;
     const int vis_lo = window_first(p1, a.window) - en.key0;
     int it = 0;
-    for (int kb = start; kb < n_keys; kb += kLatKeys, it++) {
-        if (kb + kLatKeys < n_keys) {
-            load((it + 1) & 1, kb + kLatKeys);
+    for (int kb = start; kb < n_keys; kb += kTileKeys, it++) {
+        if (kb + kTileKeys < n_keys) {
+            load((it + 1) & 1, kb + kTileKeys);
             asm volatile("cp.async.wait_group 1;" ::: "memory");
         } else {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-        const __nv_bfloat16 *ks = kv_s + (size_t)(it & 1) * kLatKeys * (LK + LV);
-        const bool masked = kb + kLatKeys - 1 > p0 - en.key0 || kb < vis_lo;
-        attend_tile<DK, DV, kLatKeys>(qfrag, ks, ks + kLatKeys * LK, kb, masked, lo, hi, sl, m, l, o, lane);
+        const __nv_bfloat16 *ks = kv_s + (size_t)(it & 1) * kTileKeys * (LK + LV);
+        const bool masked = kb + kTileKeys - 1 > p0 - en.key0 || kb < vis_lo;
+        attend_tile<DK, DV, kTileKeys>(qfrag, ks, ks + kTileKeys * LK, kb, masked, lo, hi, sl, m, l, o, lane);
         __syncthreads();
     }
 #pragma unroll
@@ -544,30 +573,32 @@ static int32_t opt_in(K kern, size_t smem, int &set_for) {
 }
 
 int32_t launch_latent_prep(bool f32, const StepDesc &d, const LatentArgs &a, int pdl, cudaStream_t st) {
-    const dim3 grid((unsigned)((d.rows * (a.own_cache ? 2 : 1) + 7) / 8));
-    if (f32) return launch(latent_prep_kernel<float>, grid, 256, 0, 1, pdl, st, a, d.seq, d.pos, d.rows, pdl);
-    return launch(latent_prep_kernel<__nv_bfloat16>, grid, 256, 0, 1, pdl, st, a, d.seq, d.pos, d.rows, pdl);
+    const dim3 grid((unsigned)d.rows);
+    const int threads = a.own_cache ? 256 : 128;
+    if (f32) return launch(latent_prep_kernel<float>, grid, threads, 0, 1, pdl, st, a, d.seq, d.pos, pdl);
+    return launch(latent_prep_kernel<__nv_bfloat16>, grid, threads, 0, 1, pdl, st, a, d.seq, d.pos, pdl);
 }
 
 template <int NTW, int MT>
-static int32_t attn_run(const StepDesc &d, const LatentArgs &a, const int *list, int n, int max_rows, bool single, int pdl, cudaStream_t st) {
+static int32_t attn_run(const StepDesc &d, const LatentArgs &a, const Seg *list, int n, int max_rows, bool single, int pdl, cudaStream_t st) {
     auto kern = latent_attn_kernel<NTW, MT>;
     static thread_local int set_for = -1;
-    if (int32_t rc = opt_in(kern, kMaxSmem - 1024, set_for)) return rc;
+    if (int32_t rc = opt_in(kern, kMaxSmem, set_for)) return rc;
     const size_t fixed = latent_fixed_smem<MT>(a.LDR), stage = (size_t)kLatKeys * a.LDR * 2;
-    const int stages = (int)std::min<size_t>(4, (kMaxSmem - 1024 - fixed) / stage), blocks = (max_rows + 16 * MT - 1) / (16 * MT);
-    JGPT_REQUIRE(stages >= 2, JGPT_ERR_UNSUPPORTED, "latent of %d, rotated part of %d", a.KR, a.RR);
+    const size_t room = MT == 1 ? kMaxSmem / 2 : kMaxSmem;  // two CTAs of 16 rows share an SM
+    const int stages = (int)std::min<size_t>(6, (std::max(room, fixed + 2 * stage) - fixed) / stage), blocks = (max_rows + 16 * MT - 1) / (16 * MT);
+    JGPT_REQUIRE(stages >= 2 && fixed + stages * stage <= kMaxSmem, JGPT_ERR_UNSUPPORTED, "latent of %d, rotated part of %d", a.KR, a.RR);
     int split = 1;
-    if (single) {  // the grid stays within one CTA per SM, every CTA keeps two tiles
+    if (single) {  // the grid stays within what the SMs hold, every CTA keeps two tiles
         const int keys = a.window > 0 ? std::min(a.window, d.max_len) : d.max_len, tiles = keys / kLatKeys + 1;
-        while (split < 8 && n * blocks * split * 2 <= a.sm_count && tiles >= split * 2 * 2) split *= 2;
+        while (split < 8 && n * blocks * split * 2 <= (MT == 1 ? 2 : 1) * a.sm_count && tiles >= split * 2 * 2) split *= 2;
     }
     const dim3 grid((unsigned)split, (unsigned)blocks, (unsigned)n);
-    return launch(kern, grid, 256, fixed + stages * stage, split, pdl, st, a, d.segs, list, stages, pdl);
+    return launch(kern, grid, kLatThreads, fixed + stages * stage, split, pdl, st, a, list, stages, pdl);
 }
 
 template <int NTW>
-static int32_t attn_rows(const StepDesc &d, const LatentArgs &a, const int *list, int n, int max_rows, bool single, int pdl, cudaStream_t st) {
+static int32_t attn_rows(const StepDesc &d, const LatentArgs &a, const Seg *list, int n, int max_rows, bool single, int pdl, cudaStream_t st) {
     return max_rows <= 16 ? attn_run<NTW, 1>(d, a, list, n, max_rows, single, pdl, st) : attn_run<NTW, 2>(d, a, list, n, max_rows, single, pdl, st);
 }
 
@@ -577,7 +608,7 @@ int32_t launch_latent_attention(bool f32, const StepDesc &d, const LatentArgs &a
         JGPT_CUDA_TRY(cudaGetLastError());
         return JGPT_OK;
     }
-    auto run = [&](const int *list, int n, int max_rows, bool single) -> int32_t {
+    auto run = [&](const Seg *list, int n, int max_rows, bool single) -> int32_t {
         switch (a.KR) {
             case 128: return attn_rows<2>(d, a, list, n, max_rows, single, pdl, st);
             case 256: return attn_rows<4>(d, a, list, n, max_rows, single, pdl, st);
@@ -587,7 +618,7 @@ int32_t launch_latent_attention(bool f32, const StepDesc &d, const LatentArgs &a
         return fail(JGPT_ERR_UNSUPPORTED, "latent of %d", a.KR);
     };
     if (d.n_singles)
-        if (int32_t rc = run(d.singles, d.n_singles, a.heads, true)) return rc;
+        if (int32_t rc = run(d.lat_singles, d.n_singles, a.heads, true)) return rc;
     return d.n_lat_short ? run(d.lat_short, d.n_lat_short, d.lat_short_max * a.heads, false) : JGPT_OK;
 }
 

@@ -360,7 +360,7 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
     return JGPT_OK;
 }
 
-static size_t desc_ints(const Decoder *d) { return 28 * (size_t)d->R + 128; }
+static size_t desc_ints(const Decoder *d) { return 40 * (size_t)d->R + 128; }
 
 static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
     const uint64_t R = d->R, W = d->s.width, eb = d->eb;
@@ -892,7 +892,7 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
         return o;
     };
     const size_t o_tok = take((size_t)rows), o_pos = take((size_t)rows), o_seq = take((size_t)rows), o_seg = take(6 * (size_t)c.n);
-    const size_t o_ent = take((size_t)rows), o_lat_short = take((size_t)c.n), o_lat_long = take(4 * (size_t)c.n);
+    const size_t o_ent = take((size_t)rows), o_lat_single = take(6 * (size_t)c.n), o_lat_short = take(6 * (size_t)c.n), o_lat_long = take(4 * (size_t)c.n);
     const size_t o_single = take((size_t)c.n), o_short = take((size_t)c.n), o_want = take((size_t)c.n_want), o_long = take(2 * (size_t)c.n);
     int max_len = 0, n_short = 0, n_long = 0, n_chunks = 0;
     const int long_min = d->long_min;
@@ -936,11 +936,14 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
     int n_lat_long = 0, n_lat_tiles = 0;
     sd.lat_lo = rows;
     mix::LatentEntry *lat_long = reinterpret_cast<mix::LatentEntry *>(hd + o_lat_long);
+    mix::Seg *lat_single = reinterpret_cast<mix::Seg *>(hd + o_lat_single), *lat_short = reinterpret_cast<mix::Seg *>(hd + o_lat_short);
+    int n_lat_single = 0;
     for (int i = 0; d->cq && i < c.n; i++) {
         const int T = segs[i].T, pos0 = segs[i].pos0, back = d->max_window > 0 ? std::min(pos0, d->max_window - 1) : pos0;
         if (d->lat_min == 0 || T < std::max(d->lat_min, 2) || (long long)back + T > d->kvx_rows) {
             sd.lat_lo = std::min(sd.lat_lo, segs[i].row0), sd.lat_hi = segs[i].row0 + T;
-            if (T > 1) hd[o_lat_short + sd.n_lat_short++] = i, sd.lat_short_max = std::max(sd.lat_short_max, T);
+            if (T > 1) lat_short[sd.n_lat_short++] = segs[i], sd.lat_short_max = std::max(sd.lat_short_max, T);
+            else lat_single[n_lat_single++] = segs[i];
             continue;
         }
         if (batches.empty() || batches.back().rows + back + T > d->kvx_rows) batches.push_back(LatentBatch{n_lat_long, 0, 0, 0, n_lat_tiles, 0});
@@ -956,7 +959,7 @@ int32_t decoder_step(Decoder *d, Pool *p, jgpt_kvpool poolh, const StepCall &c) 
     const int *dd = d->d_desc;
     sd.tok = dd + o_tok, sd.pos = dd + o_pos, sd.seq = dd + o_seq, sd.segs = reinterpret_cast<const mix::Seg *>(dd + o_seg);
     sd.tiles = reinterpret_cast<const int2 *>(dd + o_tile), sd.singles = dd + o_single, sd.want = dd + o_want;
-    sd.ent = dd + o_ent, sd.lat_short = dd + o_lat_short, sd.lat_long = reinterpret_cast<const mix::LatentEntry *>(dd + o_lat_long);
+    sd.ent = dd + o_ent, sd.lat_singles = reinterpret_cast<const mix::Seg *>(dd + o_lat_single), sd.lat_short = reinterpret_cast<const mix::Seg *>(dd + o_lat_short), sd.lat_long = reinterpret_cast<const mix::LatentEntry *>(dd + o_lat_long);
     sd.lat_tiles = reinterpret_cast<const int2 *>(dd + o_lat_tile);
     sd.rows = rows, sd.n_segs = c.n, sd.n_tiles = n_tiles, sd.n_singles = n_single, sd.n_want = c.n_want, sd.max_len = max_len;
     sd.qt = qt;

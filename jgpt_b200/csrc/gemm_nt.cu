@@ -183,7 +183,7 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
         } else if (m < M && n < n_end) {
             const size_t at = (size_t)m * P.ldc + n + cn;
             if (EPI == EPI_STORE) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(sum[i]);
-            if (EPI == EPI_ACT) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(activate(P.act, P.p0, P.p1, sum[i]));
+            if (EPI == EPI_ACT) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(activate_fast(P.act, P.p0, P.p1, sum[i]));
             if (EPI == EPI_ADD_F32) reinterpret_cast<float *>(P.C)[at] = P.res[at] + (P.colscale ? P.colscale[n] * sum[i] : sum[i]);
             if (EPI == EPI_SCALE_F32) reinterpret_cast<float *>(P.C)[at] = sum[i] * P.scale;
         }

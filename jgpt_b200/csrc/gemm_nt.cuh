@@ -45,8 +45,16 @@ __device__ __forceinline__ float gelu_tanh(float z) {
 
 // xIELU: a z^2 + z / 2 for positive z, b (e^z - 1 - z) + z / 2 otherwise.
 __device__ __forceinline__ float xielu(float z, float a, float b) { return 0.5f * z + (z > 0.f ? a * z * z : b * (expm1f(z) - z)); }
+// The same with the fast exponential, for results that are rounded to bf16: e^z - 1 - z from its series near 0.
+__device__ __forceinline__ float xielu_fast(float z, float a, float b) {
+    const float e = z > -0.03125f ? z * z * fmaf(z, fmaf(z, 1.f / 24.f, 1.f / 6.f), 0.5f) : __expf(z) - 1.f - z;
+    return fmaf(0.5f, z, z > 0.f ? a * z * z : b * e);
+}
 __device__ __forceinline__ float activate(int act, float p0, float p1, float z) {
     return act == ACT_XIELU ? xielu(z, p0, p1) : (act == ACT_TANH ? tanhf(z) : z);
+}
+__device__ __forceinline__ float activate_fast(int act, float p0, float p1, float z) {
+    return act == ACT_XIELU ? xielu_fast(z, p0, p1) : (act == ACT_TANH ? tanhf(z) : z);
 }
 
 // Runs 1 or 2 independent products (same M) in one launch.  K, lda, ldw and (bf16) the operand addresses must allow

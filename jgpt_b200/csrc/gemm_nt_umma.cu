@@ -166,9 +166,12 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
                 if (m >= a.M) continue;
                 if (EPI == EPI_STORE || EPI == EPI_ACT) {
                     __nv_bfloat16 *c = reinterpret_cast<__nv_bfloat16 *>(a.C) + (size_t)m * a.ldc + n0 + c0 + cn;
-                    if (EPI == EPI_ACT) {
+                    if (EPI == EPI_ACT && a.act == ACT_XIELU) {
 #pragma unroll
-                        for (int q = 0; q < 32; q++) v[q] = activate(a.act, a.p0, a.p1, v[q]);
+                        for (int q = 0; q < 32; q++) v[q] = xielu_fast(v[q], a.p0, a.p1);
+                    } else if (EPI == EPI_ACT && a.act == ACT_TANH) {
+#pragma unroll
+                        for (int q = 0; q < 32; q++) v[q] = tanhf(v[q]);
                     }
 #pragma unroll
                     for (int q = 0; q < 4; q++)

@@ -27,7 +27,7 @@ struct StepDesc {
     const int *want;             // rows whose logits are wanted
     const struct LatentEntry *lat_long;  // entries whose latent attention runs on written-out keys and values
     const int2 *lat_tiles;       // (index in lat_long, first token) of their query tiles
-    const int *lat_short;        // entries with more than one token whose latent attention stays on the latents
+    const Seg *lat_singles, *lat_short;  // entries with one token; with more whose latent attention stays on the latents
     int rows, n_segs, n_tiles, n_singles, n_short, n_long, n_chunks, n_want, n_lat_short;
     int lat_short_max;           // tokens of the longest of the latter
     int lat_lo, lat_hi;          // rows from the first to the last of the entries that stay on the latents

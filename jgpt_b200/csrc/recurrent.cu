@@ -372,12 +372,13 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
     }
 }
 
-// RMS norm and gate of heads whose columns were cut over several CTAs.  One warp per (row, head).
+// RMS norm and gate of heads whose columns were cut over several CTAs.
 template <class AT, int KIND>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const RecArgs a, int rows) {
     const int item = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (item >= rows * a.heads) return;
-    norm_gate_head<AT, KIND>(a, item / a.heads, item % a.heads, lane);
+    const int per = norm_heads_per_warp(a.DV), groups = (a.heads + per - 1) / per;
+    if (item >= rows * groups) return;
+    norm_gate_group<AT, KIND>(a, item / groups, item % groups * per, lane);
 }
 
 int rec_padded_key(int dim) {

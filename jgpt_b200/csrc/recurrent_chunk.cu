@@ -465,7 +465,7 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecArgs a, const Se
         for (int e = 0; e < 4; e++) S[(size_t)(8 * n + 2 * t + (e & 1)) * 16 + g + 8 * (e >> 1)] = st[n][e];
 }
 
-// RMS norm and gate of the chunked rows, one warp per (row, head).
+// RMS norm and gate of the chunked rows.
 template <class AT, int KIND>
 __global__ void __launch_bounds__(256) rec_chunk_norm_kernel(const RecArgs a, const Seg *__restrict__ segs, const int2 *__restrict__ chunks, int pdl) {
     if (pdl & 2) griddep_launch_dependents();
@@ -473,8 +473,9 @@ __global__ void __launch_bounds__(256) rec_chunk_norm_kernel(const RecArgs a, co
     const Seg sgm = segs[ck.x];
     const int tn = min(kC, sgm.T - ck.y), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (pdl & 1) griddep_wait();
-    for (int i = blockIdx.y * 8 + warp; i < tn * a.heads; i += 8 * gridDim.y)
-        norm_gate_head<AT, KIND>(a, sgm.row0 + ck.y + i / a.heads, i % a.heads, lane);
+    const int per = norm_heads_per_warp(a.DV), groups = (a.heads + per - 1) / per;
+    for (int i = blockIdx.y * 8 + warp; i < tn * groups; i += 8 * gridDim.y)
+        norm_gate_group<AT, KIND>(a, sgm.row0 + ck.y + i / groups, i % groups * per, lane);
 }
 
 template <class K, class... Args>
@@ -512,7 +513,7 @@ static int32_t chunk_launch(const StepDesc &d, const RecArgs &a, int pdl, cudaSt
     rc = launch_early(rec_scan_kernel<KIND == REC_DELTA ? REC_DELTA : REC_GLA, DK>, dim3((unsigned)(a.heads * (groups / nw)), (unsigned)d.n_long), 32 * nw, smem, set2,
                       sizeof(float) * kScanStages * scan_stage_floats(KIND, DK, 16 * max_warps), pdl, st, a, d.segs, d.long_segs, pdl);
     if (rc) return rc;
-    return launch_early(rec_chunk_norm_kernel<AT, KIND>, dim3((unsigned)d.n_chunks, (unsigned)((kC * a.heads + 63) / 64)), 256, 0, set3, 0, pdl, st, a, d.segs,
+    return launch_early(rec_chunk_norm_kernel<AT, KIND>, dim3((unsigned)d.n_chunks, (unsigned)((kC * (a.heads / norm_heads_per_warp(a.DV) + 1) + 31) / 32)), 256, 0, set3, 0, pdl, st, a, d.segs,
                         d.chunks, pdl);
 }
 

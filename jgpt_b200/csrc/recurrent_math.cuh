@@ -57,18 +57,51 @@ __device__ __forceinline__ float out_gate(float g) {
     return KIND == REC_DELTA ? sigmoid_f<AT>(g) : g * sigmoid_f<AT>(g);
 }
 
-// RMS norm over a head's value columns and its output gate, by one warp: raw fp32 values -> activations.
-template <class AT, int KIND>
-__device__ __forceinline__ void norm_gate_head(const RecArgs &a, int r, int h, int lane) {
+// RMS norm over a head's value columns and its output gate: raw fp32 values -> activations.  A warp takes heads h0, h0 + 1, ... of a
+// row, LANES lanes each with four columns at a time.
+template <class AT, int KIND, int LANES>
+__device__ __forceinline__ void norm_gate_heads(const RecArgs &a, int r, int h0, int lane) {
+    constexpr int NV = LANES == 32 ? 2 : 1;  // up to 256 columns
+    const int h = h0 + lane / LANES, c0 = lane % LANES * 4;
+    const bool on = h < a.heads;
     const float *raw = a.raw + (size_t)r * a.heads * a.DV + h * a.DV;
+    float4 x[NV];
     float ss = 0.f;
-    for (int c = lane; c < a.DV; c += 32) ss += raw[c] * raw[c];
-    const float inv = a.out_scale / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const int c = c0 + 128 * i;
+        x[i] = on && c < a.DV ? *reinterpret_cast<const float4 *>(raw + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+    }
     AT *o = reinterpret_cast<AT *>(a.out) + (size_t)r * a.ldo + a.out_off + h * a.DV;
     const AT *gp = KIND == REC_DELTA ? reinterpret_cast<const AT *>(a.z) + (size_t)r * a.ldz + a.zg_off + h * a.DV
                                      : reinterpret_cast<const AT *>(a.proj) + (size_t)r * a.ldp + a.g_off + h * a.DV;
     const float *nw = a.norm_w + h * a.norm_stride;
-    for (int c = lane; c < a.DV; c += 32) store1(o + c, raw[c] * inv * nw[c] * (rec_has_gate(KIND) ? out_gate<AT, KIND>(load1(gp + c)) : 1.f));
+#pragma unroll
+    for (int off = LANES / 2; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+    const float inv = a.out_scale / sqrtf(ss / (float)a.vdim + a.eps);
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const int c = c0 + 128 * i;
+        if (!on || c >= a.DV) continue;
+        const float4 w = *reinterpret_cast<const float4 *>(nw + c);
+        float2 lo = make_float2(x[i].x * inv * w.x, x[i].y * inv * w.y), hi = make_float2(x[i].z * inv * w.z, x[i].w * inv * w.w);
+        if (rec_has_gate(KIND)) {
+            const float2 g0 = load2(gp + c), g1 = load2(gp + c + 2);
+            lo.x *= out_gate<AT, KIND>(g0.x), lo.y *= out_gate<AT, KIND>(g0.y), hi.x *= out_gate<AT, KIND>(g1.x), hi.y *= out_gate<AT, KIND>(g1.y);
+        }
+        store2(o + c, lo), store2(o + c + 2, hi);
+    }
+}
+// Heads a warp takes at once: eight lanes cover 32 columns.
+__host__ __device__ inline int norm_heads_per_warp(int DV) { return DV <= 32 ? 4 : (DV <= 64 ? 2 : 1); }
+template <class AT, int KIND>
+__device__ __forceinline__ void norm_gate_group(const RecArgs &a, int r, int h0, int lane) {
+    switch (norm_heads_per_warp(a.DV)) {
+        case 4: return norm_gate_heads<AT, KIND, 8>(a, r, h0, lane);
+        case 2: return norm_gate_heads<AT, KIND, 16>(a, r, h0, lane);
+        default: return norm_gate_heads<AT, KIND, 32>(a, r, h0, lane);
+    }
 }
 
 }  // namespace mix

@@ -1,5 +1,5 @@
-"""Prefill and decode throughput of a layered decoder (the Somopel design with random weights) beside the fixed-block GPT
-model at equal width, depth, feed-forward size and vocabulary: ``bench.py --workload decoder``."""
+"""Prefill and decode throughput of the layered designs (Zusepel, Somopel; random weights) beside the fixed-block GPT model at
+equal width, depth, feed-forward parameters and vocabulary: ``bench.py --workload decoder``."""
 from __future__ import annotations
 
 import time
@@ -58,16 +58,63 @@ def random_somopel(ctx, width, max_rows, rank=64):
                 lin(q + n, k, width), lin(q + n + ".conv", k, t)
             lin(q + "b", H, width), vec(q + "A_log", H), vec(q + "dt_bias", H * dk), lin(q + "o", width, H * dv)
             lin(q + "a1", rank, width), lin(q + "a2", H * dk, rank), lin(q + "g1", rank, width), lin(q + "g2", H * dv, rank), vec(q + "norm", dv)
+    return _random_model(ctx, cfg, shapes, max_rows)
+
+
+def _random_model(ctx, cfg, shapes, max_rows, seed=0):
+    rng = np.random.default_rng(seed)
     noise = rng.standard_normal(1 << 22, dtype=np.float32)
 
     def get(n):  # slices of one noise block: making fresh numbers for every weight takes longer than the benchmark
         s = shapes[n]
         k = int(np.prod(s))
         x = np.resize(noise[int(rng.integers(0, 1 << 20)):], k).reshape(s)
+        if n.endswith(".lower"):
+            return 0.5 + 0.1 * np.tanh(x)
+        if n.endswith(".w0"):
+            return x - 4
         return x / np.sqrt(s[1]) if len(s) == 2 else 1 + 0.1 * x
     model = D.DecoderModel(ctx, registry.describe(cfg, shapes.__getitem__), "bfloat16", max_rows)
     model.loadTensors(get)
     return model
+
+
+def zusepel_config(width):
+    """Latent attention with 128 + 64 / 128 heads on a latent of 512 (window 512), WKV heads of 64, HGRN2 heads of 128."""
+    h, mlp = width // 128, {"kind": "dense", "ff": width * 33 // 8}  # as many parameters as a gated part of 11 / 4
+    rot = {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+    latent = {"heads": h, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": width * 3 // 8, "kv_rank": 512, "mask": {"size": 512}, "rot": rot,
+              "scale": 192 ** -0.5}
+    block = [("latent_attention", latent), ("wkv", {"heads": 2 * h, "dim": 64}), ("hgrn2", {"heads": h, "dim": 128, "vdim": 128})]
+    layers = [{"type": t, "mixer": m, "mlp": mlp} for t, m in block * (LAYERS // 3)]
+    layers[3] = {**layers[3], "mixer": {**latent, "kv_from": 0}}
+    return {"architecture": "Zusepel", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6}, "residual_mult": 0.7, "layers": layers}
+
+
+def random_zusepel(ctx, width, max_rows, rank=64):
+    cfg = zusepel_config(width)
+    shapes = {"embed": (VOCAB, width), "head": (VOCAB, width), "final.norm": (width,)}
+    for i, e in enumerate(cfg["layers"]):
+        p, m, ff = f"l{i}.", e["mixer"], e["mlp"]["ff"]
+        new = {n: (width,) for n in ("norm1", "norm2", "ls1", "ls2")}
+        new.update({"dwa": (i + 2,), "mlp.up": (ff, width), "mlp.down": (width, ff), "mlp.act": (2,)})
+        H, d = m["heads"], m["dim"]
+        if e["type"] == "latent_attention":
+            r, v = m["rot_dim"], m["vdim"]
+            new.update({"mix.dq": (m["q_rank"], width), "mix.dq.norm": (m["q_rank"],), "mix.uq": (H * (d + r), m["q_rank"]), "mix.uk": (H * d, m["kv_rank"]),
+                        "mix.uv": (H * v, m["kv_rank"]), "mix.o": (width, H * v)})
+            if "kv_from" not in m:
+                new.update({"mix.dkv": (m["kv_rank"] + r, width), "mix.dkv.norm": (m["kv_rank"],)})
+        elif e["type"] == "wkv":
+            new.update({f"mix.mu.{s}": (width,) for s in "rkvgw"})
+            new.update({f"mix.{s}": (H * d, width) for s in "rkvg"})
+            new.update({"mix.w1": (rank, width), "mix.w2": (H * d, rank), "mix.w0": (H * d,), "mix.u": (H, d), "mix.norm": (H * d,), "mix.o": (width, H * d)})
+        else:
+            v = m["vdim"]
+            new.update({"mix.q": (H * d, width), "mix.f": (H * d, width), "mix.f.b": (H * d,), "mix.lower": (H * d,), "mix.v": (H * v, width), "mix.norm": (v,),
+                        "mix.o": (width, H * v)})
+        shapes.update({p + n: s for n, s in new.items()})
+    return _random_model(ctx, cfg, shapes, max_rows)
 
 
 def random_gpt(ctx, width, max_rows):
@@ -128,12 +175,12 @@ def _prefill(ctx, model, batch, seq_len, repeats):
     return float(np.median(best))
 
 
-def run_decoder(ctx, widths=(1024, 2048), batches=(1, 16, 64), prompts=((1, 2048), (8, 1024)), ctx_len=1500, steps=24, repeats=5, models=("somopel", "gpt")):
+def run_decoder(ctx, widths=(1024, 2048), batches=(1, 16, 64), prompts=((1, 2048), (8, 1024)), ctx_len=1500, steps=24, repeats=5, models=("zusepel", "somopel", "gpt")):
     out = {"workload": f"{LAYERS} layers, vocabulary {VOCAB}, random weights; prefill = prompts of one call, decode at context {ctx_len}+",
            "timing": "prefill: CUDA events around the call; decode: host clock around a step that reads its ids back; medians", "sizes": []}
     for w in widths:
         row = {"width": w}
-        for name, make in (("somopel", random_somopel), ("gpt", random_gpt)):
+        for name, make in (("zusepel", random_zusepel), ("somopel", random_somopel), ("gpt", random_gpt)):
             if name not in models:
                 continue
             m = make(ctx, w, 8192)

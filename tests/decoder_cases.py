@@ -90,8 +90,10 @@ def tokens(cfg, n, seed=0):
 class Case:
     """A configuration with its weights, and the oracle's logits of token lists (computed once each)."""
 
+    make_weights, forward = staticmethod(weights), staticmethod(R.forward)
+
     def __init__(self, cfg, seed=0, edit=None, **kw):
-        self.cfg, self.W = cfg, weights(cfg, seed, **kw)
+        self.cfg, self.W = cfg, self.make_weights(cfg, seed, **kw)
         if edit:
             edit(self.W)
             self.W = {k: bf16(v) for k, v in self.W.items()}
@@ -105,7 +107,7 @@ class Case:
     def ref(self, toks, cfg=None):
         key = (tuple(int(t) for t in toks), id(cfg))
         if key not in self._ref:
-            self._ref[key] = R.forward(cfg or self.cfg, self.W, np.asarray(toks))
+            self._ref[key] = self.forward(cfg or self.cfg, self.W, np.asarray(toks))
         return self._ref[key]
 
 
@@ -149,3 +151,38 @@ def cut(toks, sizes):
         out.append(toks[at:at + n])
         at, i = at + n, i + 1
     return out
+
+
+def mixed_plan(toks, seed, live=3):
+    """Requests that start, pause, go on in portions or single tokens, and end: at most `live` at a time."""
+    rng = np.random.default_rng(seed)
+    at, active, todo, plan = {n: 0 for n in toks}, [], list(toks), []
+    while todo or active:
+        while todo and len(active) < live:
+            active.append(todo.pop(0))
+        step = []
+        for n in list(active):
+            if rng.random() < 0.2:
+                continue  # left out of this step
+            k = int(rng.choice([1, 1, 1, 2, 3, 16, 29, 64, 90]))
+            step.append((n, toks[n][at[n]:at[n] + k]))
+            at[n] += k
+        for n in list(active):
+            if at[n] >= len(toks[n]):
+                active.remove(n)
+                step.append((n, None))
+        plan.append(step)
+    return plan
+
+
+def greedy(case, prompt, n):
+    """The oracle's greedy continuation and the smallest margin between its best two logits."""
+    out, margin = list(prompt), np.inf
+    for _ in range(n):
+        lg = case.forward(case.cfg, case.W, np.array(out))[-1]
+        top = np.sort(lg)[-2:]
+        margin = min(margin, top[1] - top[0])
+        out.append(int(lg.argmax()))
+        if out[-1] == 0:
+            break
+    return out[len(prompt):], margin

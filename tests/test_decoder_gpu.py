@@ -160,7 +160,7 @@ def test_chunked_recurrences_at_full_precision(ctx, cases, name, monkeypatch):
         t = dc.tokens(c.cfg, 320, 17)
         _close(dc.run_steps(m, pool, [[("a", p)] for p in dc.cut(t, sizes)])["a"], c.ref(t), "float32")
     toks = {f"r{i}": dc.tokens(c.cfg, L, 50 + i) for i, L in enumerate([1, 150, 33, 64, 17, 2])}
-    got = dc.run_steps(m, pool, _mixed_plan(toks, 3))
+    got = dc.run_steps(m, pool, dc.mixed_plan(toks, 3))
     for r, t in toks.items():
         _close(got[r], c.ref(t), "float32")
     pool.close(), m.close()
@@ -195,28 +195,6 @@ def test_long_decoding(ctx, cases, dtype):
     pool.close(), m.close()
 
 
-def _mixed_plan(toks, seed, live=3):
-    """Requests that start, pause, go on in portions or single tokens, and end: at most `live` at a time."""
-    rng = np.random.default_rng(seed)
-    at, active, todo, plan = {n: 0 for n in toks}, [], list(toks), []
-    while todo or active:
-        while todo and len(active) < live:
-            active.append(todo.pop(0))
-        step = []
-        for n in list(active):
-            if rng.random() < 0.2:
-                continue  # left out of this step
-            k = int(rng.choice([1, 1, 1, 2, 3, 16, 29, 64]))
-            step.append((n, toks[n][at[n]:at[n] + k]))
-            at[n] += k
-        for n in list(active):
-            if at[n] >= len(toks[n]):
-                active.remove(n)
-                step.append((n, None))
-        plan.append(step)
-    return plan
-
-
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("name", ["order", "ragged_sizes", "wide_groups"])
 def test_mixed_batches_with_blocks_and_slots_used_again(ctx, cases, name, dtype):
@@ -229,7 +207,7 @@ def test_mixed_batches_with_blocks_and_slots_used_again(ctx, cases, name, dtype)
     from jgpt_b200 import binding as B
     B.check(m._lib.jgpt_dev_memset(ctx.handle, p, 0xFF, n))
     toks = {f"r{i}": dc.tokens(c.cfg, L, 50 + i) for i, L in enumerate([1, 150, 33, 200, 64, 17, 2, 180, 90])}
-    got = dc.run_steps(m, pool, _mixed_plan(toks, 7))
+    got = dc.run_steps(m, pool, dc.mixed_plan(toks, 7))
     for r, t in toks.items():
         _close(got[r], c.ref(t), dtype)
     assert pool.free_blocks() == 40
@@ -307,24 +285,12 @@ def test_first_tokens_and_convolution_history(ctx):
 
 
 # ---- scheduler, generation, sampling -------------------------------------------------------------------------
-def _oracle_greedy(c, prompt, n):
-    out, margin = list(prompt), np.inf
-    for _ in range(n):
-        lg = R.forward(c.cfg, c.W, np.array(out))[-1]
-        top = np.sort(lg)[-2:]
-        margin = min(margin, top[1] - top[0])
-        out.append(int(lg.argmax()))
-        if out[-1] == 0:
-            break
-    return out[len(prompt):], margin
-
-
 def test_greedy_generation_equals_the_oracle(ctx, cases):
     c = cases["ragged_sizes"]
     m = c.model(ctx, "float32", max_rows=16)
     for i, L in enumerate([1, 5, 40]):  # the longest prompt goes in as portions
         prompt = dc.tokens(c.cfg, L, 200 + i)
-        want, margin = _oracle_greedy(c, prompt, 12)
+        want, margin = dc.greedy(c, prompt, 12)
         assert margin > 1e-4
         got = m.generateGpuKv(prompt, 12)
         assert got[L:L + len(want)].tolist() == want and (got[L + len(want):] == 0).all()
@@ -346,7 +312,7 @@ def test_continuous_batching(ctx, cases, dtype):
         got, state, _ = batch.result(r)
         assert state == 2
         if dtype == "float32":
-            want, margin = _oracle_greedy(c, p, 10)
+            want, margin = dc.greedy(c, p, 10)
             assert margin < 1e-4 or got.tolist() == want
         else:
             lg = R.forward(c.cfg, c.W, np.concatenate([p, got]))  # every pick is near the oracle's best
@@ -431,4 +397,4 @@ def test_trace_run_and_generate_command_lines(ctx, cases, tmp_path):
     assert r.returncode == 0, r.stderr
     lines = [json.loads(x) for x in r.stdout.splitlines() if x.startswith("{")]
     for line, p in zip(lines, (t[:5], t[5:8])):
-        assert line["tokens"] == _oracle_greedy(c, p, 6)[0]
+        assert line["tokens"] == dc.greedy(c, p, 6)[0]
