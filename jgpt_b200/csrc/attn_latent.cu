@@ -14,7 +14,6 @@
 #include "attn_mma.cuh"
 
 #include <algorithm>
-#include <type_traits>
 
 namespace jgpt {
 namespace mix {
@@ -31,44 +30,85 @@ __device__ __forceinline__ float rotated(const AT *x, const float2 *cs, int half
     return j < half ? u * t.x - v * t.y : v * t.x + u * t.y;
 }
 
-// A block per row, 128 threads per part: part 0 the query latent, part 1 the key latent and the rotated part.
+__device__ __forceinline__ void load8(const __nv_bfloat16 *p, float (&v)[8]) {
+    const uint4 u = *reinterpret_cast<const uint4 *>(p);
+    const __nv_bfloat162 *h = reinterpret_cast<const __nv_bfloat162 *>(&u);
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const float2 f = __bfloat1622float2(h[i]);
+        v[2 * i] = f.x, v[2 * i + 1] = f.y;
+    }
+}
+__device__ __forceinline__ void load8(const float *p, float (&v)[8]) {
+#pragma unroll
+    for (int i = 0; i < 8; i += 4) {
+        const float4 f = *reinterpret_cast<const float4 *>(p + i);
+        v[i] = f.x, v[i + 1] = f.y, v[i + 2] = f.z, v[i + 3] = f.w;
+    }
+}
+__device__ __forceinline__ void store8(__nv_bfloat16 *p, const float (&v)[8]) {
+    *reinterpret_cast<uint4 *>(p) = make_uint4(bf16_pair(v[0], v[1]), bf16_pair(v[2], v[3]), bf16_pair(v[4], v[5]), bf16_pair(v[6], v[7]));
+}
+__device__ __forceinline__ void store8(float *p, const float (&v)[8]) {
+    *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]), *reinterpret_cast<float4 *>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+
+// A warp per (row, part): part 0 the query latent, part 1 the key latent and the rotated part.  Latents start at multiples of
+// eight columns and are followed by zeros up to the next one.
 template <class AT>
-__global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs a, const int *__restrict__ seq, const int *__restrict__ pos, int pdl) {
-    constexpr int NT = 128;
-    __shared__ float red[8];
-    const int r = blockIdx.x, part = threadIdx.x / NT, t = threadIdx.x % NT;
+__global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs a, const int *__restrict__ seq, const int *__restrict__ pos, int rows, int pdl) {
+    constexpr int NV = 4;  // the first 1024 elements stay in registers
+    const int item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31, parts = a.own_cache ? 2 : 1;
     if (pdl & 2) griddep_launch_dependents();
     if (pdl & 1) griddep_wait();
+    if (item >= rows * parts) return;
+    const int r = item / parts, part = item % parts;
     const AT *proj = reinterpret_cast<const AT *>(a.proj) + (size_t)r * a.ldp;
     const AT *src = proj + (part ? a.c_off : a.dq_off);
     const float *gamma = part ? a.dkv_norm : a.dq_norm;
     const int n = part ? a.kv_rank : a.q_rank, padded = part ? a.KR : a.ldcq;
-    float ss = 0.f, v[8];  // the first 1024 elements stay in registers
-#pragma unroll
-    for (int i = 0; i < 8; i++) {
-        v[i] = t + NT * i < n ? act_load(src + t + NT * i) : 0.f;
-        ss += v[i] * v[i];
-    }
-    for (int j = t + NT * 8; j < n; j += NT) ss += act_load(src + j) * act_load(src + j);
-#pragma unroll
-    for (int off = 16; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
-    if ((t & 31) == 0) red[threadIdx.x >> 5] = ss;
-    __syncthreads();
-    const float inv = 1.f / sqrtf((red[4 * part] + red[4 * part + 1] + red[4 * part + 2] + red[4 * part + 3]) / (float)n + a.eps);
     AT *dst = reinterpret_cast<AT *>(a.cq) + (size_t)r * a.ldcq;
     if (part) {
         const int phys = page_of(a, seq[r], pos[r]);
         if (phys < 0) return;
         dst = reinterpret_cast<AT *>(a.kv) + ((size_t)phys * kBlockTokens + pos[r] % kBlockTokens) * a.LDR;
     }
+    float v[NV][8], ss = 0.f;
+    auto squares = [&](const float (&x)[8]) {
 #pragma unroll
-    for (int i = 0; i < 8; i++) {
-        const int j = t + NT * i;
-        if (j < padded) act_store(dst + j, j < n ? v[i] * inv * gamma[j] : 0.f);
+        for (int e = 0; e < 8; e++) ss += x[e] * x[e];
+    };
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const int j = (lane + 32 * i) * 8;
+        if (j < n) load8(src + j, v[i]);
+        else {
+#pragma unroll
+            for (int e = 0; e < 8; e++) v[i][e] = 0.f;
+        }
+        squares(v[i]);
     }
-    for (int j = t + NT * 8; j < padded; j += NT) act_store(dst + j, j < n ? act_load(src + j) * inv * gamma[j] : 0.f);
+    for (int j = (lane + 32 * NV) * 8; j < n; j += 256) {
+        float x[8];
+        load8(src + j, x), squares(x);
+    }
+#pragma unroll
+    for (int off = 16; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+    const float inv = 1.f / sqrtf(ss / (float)n + a.eps);
+    auto put = [&](int j, float (&x)[8]) {
+#pragma unroll
+        for (int e = 0; e < 8; e++) x[e] = j + e < n ? x[e] * inv * __ldg(gamma + j + e) : 0.f;
+        store8(dst + j, x);
+    };
+#pragma unroll
+    for (int i = 0; i < NV; i++)
+        if ((lane + 32 * i) * 8 < padded) put((lane + 32 * i) * 8, v[i]);
+    for (int j = (lane + 32 * NV) * 8; j < padded; j += 256) {
+        float x[8];
+        load8(src + min(j, (n - 1) / 8 * 8), x), put(j, x);
+    }
     if (part)
-        for (int j = t; j < a.RR; j += NT)
+        for (int j = lane; j < a.RR; j += 32)
             act_store(dst + a.KR + j, j < a.rot_dim ? rotated(proj + a.r_off, a.cs + (size_t)r * a.half, a.half, j) : 0.f);
 }
 
@@ -121,16 +161,18 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentArgs a, co
 // On the latents, bf16
 // ------------------------------------------------------------------------------------------------
 // CTA = 16 MT (token, head) rows of an entry, eight warps and a ninth that brings in tiles of 32 keys = two pages by bulk copies (a
-// page is contiguous, its row stride an odd number of 16-byte units, so ldmatrix is free of bank conflicts).  A warp scores eight
-// keys over half of the row's elements; the halves meet in shared memory, where every warp turns an eighth of the rows into
-// weights (bf16 high and low parts) and then adds up its eighth of the latent's columns.  A cluster splits the keys; partial sums
+// page is contiguous, its row stride an odd number of 16-byte units, so ldmatrix is free of bank conflicts).  A warp scores the
+// tile's keys over an eighth of the row's elements (its part of the query rows stays in registers: shared memory bandwidth is what
+// a tile costs); the parts meet in shared memory, where every warp turns an eighth of the rows into weights (bf16 high and low
+// parts) and then adds up its eighth of the latent's columns.  A cluster splits the keys; partial sums
 // meet through cluster shared memory.
 constexpr int kLatKeys = 32, kLatPages = kLatKeys / kBlockTokens, kLatLS = kLatKeys + 8, kLatThreads = 288;
 constexpr size_t kMaxSmem = 232448 - 4096;  // dynamic; the rest is for static shared memory
 
 template <int MT>
 __host__ __device__ constexpr size_t latent_fixed_smem(int LDR) {
-    return (size_t)16 * MT * LDR * 2 + sizeof(float) * 2 * 16 * MT * kLatLS + 2 * (size_t)16 * MT * kLatLS * 2;
+    const size_t query = (size_t)16 * MT * LDR * 2, scores = sizeof(float) * 8 * 16 * MT * kLatLS;  // one after the other in the same place
+    return (query > scores ? query : scores) + 2 * (size_t)16 * MT * kLatLS * 2;
 }
 
 template <int NTW, int MT>
@@ -145,9 +187,9 @@ __global__ void __launch_bounds__(kLatThreads, MT == 1 ? 2 : 1) latent_attn_kern
     const int LDR = a.LDR, RR = a.RR, H = a.heads;
     const uint32_t page_bytes = (uint32_t)(kBlockTokens * LDR * 2);
     __nv_bfloat16 *ring = reinterpret_cast<__nv_bfloat16 *>(lat_smem);     // [stages][32][LDR]
-    __nv_bfloat16 *qs = ring + (size_t)stages * kLatKeys * LDR;            // [ROWS][LDR]
-    float *sp = reinterpret_cast<float *>(qs + (size_t)ROWS * LDR);        // [2][ROWS][kLatLS] half scores
-    __nv_bfloat16 *ph = reinterpret_cast<__nv_bfloat16 *>(sp + 2 * ROWS * kLatLS), *pl = ph + ROWS * kLatLS;  // [ROWS][kLatLS] weights
+    __nv_bfloat16 *ph = ring + (size_t)stages * kLatKeys * LDR, *pl = ph + ROWS * kLatLS;  // [ROWS][kLatLS] weights
+    __nv_bfloat16 *qs = pl + ROWS * kLatLS;                                // [ROWS][LDR], until the operands are in registers
+    float *sp = reinterpret_cast<float *>(qs);                             // [8][ROWS][kLatLS] parts of the scores
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t2 = 2 * (lane & 3);
     const int nsplit = gridDim.x, split = blockIdx.x, r0 = blockIdx.y * ROWS;
     if (pdl & 2) griddep_launch_dependents();
@@ -222,7 +264,16 @@ __global__ void __launch_bounds__(kLatThreads, MT == 1 ? 2 : 1) latent_attn_kern
             lo[i] = r < rows ? window_first(hi[i], a.window) : 0;
         }
         const float sl = a.scale * 1.4426950408889634f;
-        const int ksteps = (KR + RR) / 16, khalf = (ksteps / 2 + 1) / 2 * 2, k_from = warp < 4 ? 0 : khalf, k_to = warp < 4 ? khalf : ksteps;
+        // this warp's k steps, and the query rows' operands for them
+        constexpr int NQ = (KR / 16 + kMaxRot / 16 + 7) / 8;
+        const int ksteps = (KR + RR) / 16, k_from = warp * ksteps / 8, k_n = (warp + 1) * ksteps / 8 - k_from;
+        uint32_t q[NQ][MT][4];
+#pragma unroll
+        for (int k = 0; k < NQ; k++)
+#pragma unroll
+            for (int i = 0; i < MT; i++)
+                if (k < k_n) ldmatrix_x4(q[k][i], qs + (size_t)(i * 16 + (lane & 15)) * LDR + (lane >> 4) * 8 + (k_from + k) * 16);
+        named_bar_sync(1, 256);  // the scores take the query rows' place
         const int end_key = min(last, pg1 * kBlockTokens - 1);
         for (int it = 0; it < n_tiles; it++) {
             const int s = it % stages, kb = (pg0 + it * kLatPages) * kBlockTokens;
@@ -233,59 +284,50 @@ __global__ void __launch_bounds__(kLatThreads, MT == 1 ? 2 : 1) latent_attn_kern
                 const int v0 = end_key - kb + 1, per = LDR / 8;
                 for (int e = tid; e < (kLatKeys - v0) * per; e += 256) *reinterpret_cast<uint4 *>(ks + (size_t)(v0 + e / per) * LDR + e % per * 8) = make_uint4(0, 0, 0, 0);
             }
-            {  // eight keys, half of the elements; even and odd steps are two chains of products, operands of six steps in flight
-                float sc[MT][4], sc2[MT][4];
+            {  // all keys, an eighth of the elements
+                float sc[MT][4][4];
 #pragma unroll
                 for (int i = 0; i < MT; i++)
 #pragma unroll
-                    for (int e = 0; e < 4; e++) sc[i][e] = sc2[i][e] = 0.f;
-                const __nv_bfloat16 *kw = ks + (size_t)((warp & 3) * 8 + (lane & 7)) * LDR + (lane >> 3) * 8, *qw = qs + (size_t)(lane & 15) * LDR + (lane >> 4) * 8;
-                auto steps = [&](auto count, int kk) {
-                    constexpr int P = decltype(count)::value;  // pairs of steps
-                    uint32_t b[P][4], q[2 * P][MT][4];
+                    for (int e = 0; e < 16; e++) sc[i][e >> 2][e & 3] = 0.f;
+                const __nv_bfloat16 *kw = ks + (size_t)(((lane >> 4) << 3) + (lane & 7)) * LDR + ((lane >> 3) & 1) * 8 + k_from * 16;
 #pragma unroll
-                    for (int p = 0; p < P; p++) {
-                        ldmatrix_x4(b[p], kw + (kk + 2 * p) * 16);
-#pragma unroll
-                        for (int i = 0; i < MT; i++) {
-                            ldmatrix_x4(q[2 * p][i], qw + (size_t)i * 16 * LDR + (kk + 2 * p) * 16);
-                            ldmatrix_x4(q[2 * p + 1][i], qw + (size_t)i * 16 * LDR + (kk + 2 * p + 1) * 16);
-                        }
-                    }
-#pragma unroll
-                    for (int p = 0; p < P; p++)
-#pragma unroll
-                        for (int i = 0; i < MT; i++) {
-                            mma_bf16(sc[i], q[2 * p][i], b[p][0], b[p][1]);
-                            mma_bf16(sc2[i], q[2 * p + 1][i], b[p][2], b[p][3]);
-                        }
-                };
-                int kk = k_from;
-                for (; kk + 6 <= k_to; kk += 6) steps(std::integral_constant<int, 3>(), kk);
-                for (; kk + 2 <= k_to; kk += 2) steps(std::integral_constant<int, 1>(), kk);
-                if (kk < k_to) {  // the upper two matrices would lie past the row: their lanes read the lower ones again
-                    uint32_t b[4], q[4];
-                    ldmatrix_x4(b, kw + kk * 16 - (lane >= 16 ? 16 : 0));
+                for (int k = 0; k < NQ; k++) {
+                    if (k >= k_n) break;
+                    uint32_t b0[4], b1[4];
+                    ldmatrix_x4(b0, kw + k * 16);
+                    ldmatrix_x4(b1, kw + (size_t)16 * LDR + k * 16);
 #pragma unroll
                     for (int i = 0; i < MT; i++) {
-                        ldmatrix_x4(q, qw + (size_t)i * 16 * LDR + kk * 16);
-                        mma_bf16(sc[i], q, b[0], b[1]);
+                        mma_bf16(sc[i][0], q[k][i], b0[0], b0[1]);
+                        mma_bf16(sc[i][1], q[k][i], b0[2], b0[3]);
+                        mma_bf16(sc[i][2], q[k][i], b1[0], b1[1]);
+                        mma_bf16(sc[i][3], q[k][i], b1[2], b1[3]);
                     }
                 }
-                float *w = sp + (size_t)(warp >> 2) * ROWS * kLatLS + (warp & 3) * 8 + t2;
+                float *w = sp + (size_t)warp * ROWS * kLatLS + t2;
 #pragma unroll
                 for (int i = 0; i < MT; i++)
 #pragma unroll
                     for (int e = 0; e < 2; e++)
-                        *reinterpret_cast<float2 *>(w + (i * 16 + g + 8 * e) * kLatLS) = make_float2(sc[i][2 * e] + sc2[i][2 * e], sc[i][2 * e + 1] + sc2[i][2 * e + 1]);
+#pragma unroll
+                        for (int c = 0; c < 4; c++)
+                            *reinterpret_cast<float2 *>(w + (i * 16 + g + 8 * e) * kLatLS + c * 8) = make_float2(sc[i][c][2 * e], sc[i][c][2 * e + 1]);
             }
             named_bar_sync(1, 256);
 #pragma unroll
             for (int i = 0; i < MT; i++) {
                 const int r = warp * 2 * MT + 2 * i + (lane >> 4), c = 2 * (lane & 15), key = kb + c, top = min(hi[i], end_key);
-                const float2 u = *reinterpret_cast<const float2 *>(sp + r * kLatLS + c), w = *reinterpret_cast<const float2 *>(sp + (ROWS + r) * kLatLS + c);
+                float2 u[8];
+#pragma unroll
+                for (int k = 0; k < 8; k++) u[k] = *reinterpret_cast<const float2 *>(sp + (k * ROWS + r) * kLatLS + c);
                 const float m0 = s_m[r];
-                const float x0 = key >= lo[i] && key <= top ? (u.x + w.x) * sl : -INFINITY, x1 = key + 1 >= lo[i] && key + 1 <= top ? (u.y + w.y) * sl : -INFINITY;
+#pragma unroll
+                for (int k = 4; k >= 1; k >>= 1)
+#pragma unroll
+                    for (int j = 0; j < 4; j++)
+                        if (j < k) u[j].x += u[j + k].x, u[j].y += u[j + k].y;
+                const float x0 = key >= lo[i] && key <= top ? u[0].x * sl : -INFINITY, x1 = key + 1 >= lo[i] && key + 1 <= top ? u[0].y * sl : -INFINITY;
                 float mx = fmaxf(x0, x1);
 #pragma unroll
                 for (int off = 8; off >= 1; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
@@ -573,10 +615,10 @@ static int32_t opt_in(K kern, size_t smem, int &set_for) {
 }
 
 int32_t launch_latent_prep(bool f32, const StepDesc &d, const LatentArgs &a, int pdl, cudaStream_t st) {
-    const dim3 grid((unsigned)d.rows);
-    const int threads = a.own_cache ? 256 : 128;
-    if (f32) return launch(latent_prep_kernel<float>, grid, threads, 0, 1, pdl, st, a, d.seq, d.pos, pdl);
-    return launch(latent_prep_kernel<__nv_bfloat16>, grid, threads, 0, 1, pdl, st, a, d.seq, d.pos, pdl);
+    const int items = d.rows * (a.own_cache ? 2 : 1), warps = items <= 4 * a.sm_count ? 2 : 8;
+    const dim3 grid((unsigned)((items + warps - 1) / warps));
+    if (f32) return launch(latent_prep_kernel<float>, grid, 32 * warps, 0, 1, pdl, st, a, d.seq, d.pos, d.rows, pdl);
+    return launch(latent_prep_kernel<__nv_bfloat16>, grid, 32 * warps, 0, 1, pdl, st, a, d.seq, d.pos, d.rows, pdl);
 }
 
 template <int NTW, int MT>
