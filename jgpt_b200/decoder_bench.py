@@ -82,13 +82,13 @@ def _random_model(ctx, cfg, shapes, max_rows, seed=0):
 def zusepel_config(width):
     """Latent attention with 128 + 64 / 128 heads on a latent of 512 (window 512), WKV heads of 64, HGRN2 heads of 128."""
     h, mlp = width // 128, {"kind": "dense", "ff": width * 33 // 8}  # as many parameters as a gated part of 11 / 4
-    rot = {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+    rot = {"base": 10000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
     latent = {"heads": h, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": width * 3 // 8, "kv_rank": 512, "mask": {"size": 512}, "rot": rot,
               "scale": 192 ** -0.5}
     block = [("latent_attention", latent), ("wkv", {"heads": 2 * h, "dim": 64}), ("hgrn2", {"heads": h, "dim": 128, "vdim": 128})]
     layers = [{"type": t, "mixer": m, "mlp": mlp} for t, m in block * (LAYERS // 3)]
     layers[3] = {**layers[3], "mixer": {**latent, "kv_from": 0}}
-    return {"architecture": "Zusepel", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6}, "residual_mult": 0.7, "layers": layers}
+    return {"architecture": "Zusepel", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6}, "residual_mult": 0.9, "layers": layers}
 
 
 def random_zusepel(ctx, width, max_rows, rank=64):
