@@ -338,10 +338,12 @@ JGPT_API int32_t jgpt_generate_greedy_rolling(jgpt_model model, jgpt_kvpool pool
  * A layer is x += m * ls1 * sum over its branches of out_scale * mixer(norm1(x)), then x += m * ls2 * ff(norm2(x)) when ff > 0;
  * norms are layer norms with weight and bias or RMS norms with weight, m is residual_mult, the factors per column ls1, ls2 are
  * there with layer_scale.  With depth_average what goes on from layer i is sum over j <= i + 1 of dwa_i[j] X_j, X_0 the
- * embedding and X_(i+1) the result of layer i.
+ * embedding and X_(i+1) the result of layer i.  With norm_after the parts read x itself and the norms come behind the sums:
+ * x <- norm1(residual_scale * x + sum of mixers(x)), then x <- norm2(residual_scale * x + ff(x)); RMS norms.
  * ------------------------------------------------------------------------------------------- */
 enum {
-    JGPT_MIX_ATTENTION = 1, /* softmax attention over paged K/V, no rotation, positions of the query's chunk only */
+    JGPT_MIX_ATTENTION = 1, /* softmax attention over paged K/V (all positions before the query or those of its chunk); biases, norms
+                               and rotation of query and key heads, two maps per head and output gates as the fields below say */
     JGPT_MIX_GLA = 2,       /* gated linear attention: S <- diag(a) S + k v^T, a = sigmoid(W_a2 W_a1 h + bias)^(1/tau) */
     JGPT_MIX_DELTA = 3,     /* gated delta rule with a decay per key channel and short convolutions on q, k, v */
     JGPT_MIX_HGRN2 = 4,     /* S <- diag(f) S + (1 - f) v^T, f = l + (1 - l) sigmoid(W_f h + bias); no output gate */
@@ -351,7 +353,10 @@ enum {
 };
 enum { JGPT_NORM_LAYER = 0, JGPT_NORM_RMS = 1 };
 enum { JGPT_FF_GATED_GELU = 0 /* W_down (gelu_tanh(W_gate h) * (W_up h)) */,
+       JGPT_FF_GATED_RELU = 2 /* W_down (relu(W_gate h) * (W_up h)) */,
+       JGPT_FF_MOE = 3 /* a mixture of experts W_down act(W_up h), see jgpt_moe_spec */,
        JGPT_FF_XIELU = 1 /* W_down xielu(W_up h), xielu(z) = a z^2 + z / 2 (z > 0), b (e^z - 1 - z) + z / 2, a = softplus(p), b = 1/2 + softplus(q) */ };
+enum { JGPT_ACT_RELU = 0, JGPT_ACT_RELU2 = 1 /* relu(z)^2 */, JGPT_ACT_GELU_TANH = 2 };
 enum { JGPT_DTYPE_BF16 = 0, /* bf16 products, activations and K/V; norms, scores, recurrences and the residual in fp32 */
        JGPT_DTYPE_F32 = 1 /* everything in fp32 (no reduced-precision matrix mode) */ };
 #define JGPT_MAX_BRANCHES 2
@@ -360,7 +365,7 @@ typedef struct {
     int32_t heads, kv_heads;  /* attention: query / key heads; delta: value heads / query-key heads */
     int32_t dim, vdim;        /* query-key and value head size, up to 256 each */
     int32_t chunk;            /* attention: position i sees j <= i with i / chunk == j / chunk; 0: every j <= i */
-    int32_t gate;             /* attention: output of head h times sigmoid(W_g h)_h */
+    int32_t gate;             /* attention: 1: output of head h times sigmoid(W_g h)_h; 2: element by element, W_g [heads * vdim, width] */
     int32_t taps;             /* delta: columns of the causal convolutions, 1..8 */
     int32_t rank_a, rank_g;   /* inner sizes of the two-factor decay and output-gate projections */
     float score_scale;        /* attention */
@@ -374,12 +379,28 @@ typedef struct {
     double rot_base;          /* frequencies base^(-2 i / rot_dims) */
     double rot_factor, rot_original, rot_fast, rot_slow; /* YaRN: slow dimensions divided by factor, cos and sin times 0.1 ln(factor) + 1;
                                                             rot_factor 0: plain rotation */
+    /* attention only; with rot_dims > 0 the first rot_dims dimensions of every query and key head (map) turn */
+    int32_t rot_interleaved;  /* pairs (2 i, 2 i + 1) instead of (i, i + rot_dims / 2) */
+    int32_t qkv_bias;         /* JGPT_W_Q_BIAS, _K_BIAS, _V_BIAS are added in the projections */
+    int32_t qk_norm;          /* RMS norm of every query and key head (map) with JGPT_W_Q_NORM / _K_NORM [dim], before the rotation */
+    int32_t maps;             /* 0, 1: one; 2: differential, q and k hold [map 1 | map 2] per head: o = a1 - lambda a2 with lambda =
+                                 exp(lq1 . lk1) - exp(lq2 . lk2) + diff, then o / rms(o) * (1 - diff); dim up to 128 then */
+    float diff;
 } jgpt_mixer_spec;
+/* Mixture of experts.  Scores are the softmax of W_router h over experts + identity outputs; the top largest scores + correction
+ * are chosen among the `keep` of `groups` equal groups of neighbours with the largest such score; weights are the chosen scores
+ * over their sum.  The last `identity` outputs stand for h itself.  A shared expert of size shared_ff (0: none) runs for every
+ * token, times sigmoid(W_sg h). */
+typedef struct {
+    int32_t experts, identity, top, groups, keep, ff, shared_ff;
+    int32_t act, shared_act;  /* JGPT_ACT_* of the experts W_down act(W_up h) */
+} jgpt_moe_spec;
 typedef struct {
     int32_t n_branches;
     jgpt_mixer_spec branch[JGPT_MAX_BRANCHES];
-    int32_t ff;      /* 0: no feed-forward part */
+    int32_t ff;      /* 0: no feed-forward part (mixtures: moe.ff once more) */
     int32_t ff_kind; /* JGPT_FF_* */
+    jgpt_moe_spec moe;
 } jgpt_layer_spec;
 typedef struct {
     int32_t vocab, width, max_positions, n_layers;
@@ -391,8 +412,12 @@ typedef struct {
     int32_t depth_average; /* JGPT_W_DWA (RMS only) */
     float eps, embed_scale, logit_scale;
     float residual_mult;
+    int32_t norm_after;    /* norms behind the sums instead of in front of the parts (RMS only, without layer_scale and depth_average) */
+    float residual_scale;  /* with norm_after */
 } jgpt_decoder_spec;
-/* Tensors.  Of the model: layer = branch = -1; of a layer: branch = -1; of a mixer: layer and branch. */
+/* Tensors.  Of the model: layer = branch = -1; of a layer: branch = -1; of a mixer: layer and branch; of an expert: layer and
+ * branch = JGPT_EXPERT(e). */
+#define JGPT_EXPERT(e) (JGPT_MAX_BRANCHES + (e))
 enum {
     JGPT_W_EMBED = 0, JGPT_W_POS, JGPT_W_EMBED_NORM, JGPT_W_EMBED_NORM_B, JGPT_W_FINAL_NORM, JGPT_W_FINAL_NORM_B,
     JGPT_W_HEAD,
@@ -402,7 +427,10 @@ enum {
     JGPT_W_DECAY_BIAS, JGPT_W_A_LOG, JGPT_W_G1, JGPT_W_G2, JGPT_W_HEAD_NORM, JGPT_W_CONV_Q, JGPT_W_CONV_K, JGPT_W_CONV_V,
     JGPT_W_MU_R, JGPT_W_MU_K, JGPT_W_MU_V, JGPT_W_MU_G, JGPT_W_MU_W, JGPT_W_BONUS /* u */, JGPT_W_LOWER /* l */, JGPT_W_F,
     JGPT_W_DQ, JGPT_W_DQ_NORM, JGPT_W_UQ, JGPT_W_DKV, JGPT_W_DKV_NORM, JGPT_W_UK, JGPT_W_UV,
-    JGPT_W_FF_ACT /* of a layer: p, q */
+    JGPT_W_FF_ACT /* of a layer: p, q */,
+    JGPT_W_Q_BIAS, JGPT_W_K_BIAS, JGPT_W_V_BIAS, JGPT_W_Q_NORM, JGPT_W_K_NORM, JGPT_W_LQ1, JGPT_W_LK1, JGPT_W_LQ2, JGPT_W_LK2,
+    JGPT_W_ROUTER = 64 /* of a layer, as the next four: [experts + identity, width] */, JGPT_W_CORRECTION, JGPT_W_SHARED_GATE /* [1, width] */,
+    JGPT_W_SHARED_UP, JGPT_W_SHARED_DOWN, JGPT_W_EXPERT_UP /* of an expert, as the next */, JGPT_W_EXPERT_DOWN
 };
 
 /* max_rows bounds the rows (tokens) of one step. */

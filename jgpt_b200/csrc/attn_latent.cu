@@ -30,29 +30,6 @@ __device__ __forceinline__ float rotated(const AT *x, const float2 *cs, int half
     return j < half ? u * t.x - v * t.y : v * t.x + u * t.y;
 }
 
-__device__ __forceinline__ void load8(const __nv_bfloat16 *p, float (&v)[8]) {
-    const uint4 u = *reinterpret_cast<const uint4 *>(p);
-    const __nv_bfloat162 *h = reinterpret_cast<const __nv_bfloat162 *>(&u);
-#pragma unroll
-    for (int i = 0; i < 4; i++) {
-        const float2 f = __bfloat1622float2(h[i]);
-        v[2 * i] = f.x, v[2 * i + 1] = f.y;
-    }
-}
-__device__ __forceinline__ void load8(const float *p, float (&v)[8]) {
-#pragma unroll
-    for (int i = 0; i < 8; i += 4) {
-        const float4 f = *reinterpret_cast<const float4 *>(p + i);
-        v[i] = f.x, v[i + 1] = f.y, v[i + 2] = f.z, v[i + 3] = f.w;
-    }
-}
-__device__ __forceinline__ void store8(__nv_bfloat16 *p, const float (&v)[8]) {
-    *reinterpret_cast<uint4 *>(p) = make_uint4(bf16_pair(v[0], v[1]), bf16_pair(v[2], v[3]), bf16_pair(v[4], v[5]), bf16_pair(v[6], v[7]));
-}
-__device__ __forceinline__ void store8(float *p, const float (&v)[8]) {
-    *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]), *reinterpret_cast<float4 *>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
-}
-
 // A warp per (row, part): part 0 the query latent, part 1 the key latent and the rotated part.  Latents start at multiples of
 // eight columns and are followed by zeros up to the next one.
 template <class AT>

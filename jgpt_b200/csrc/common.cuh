@@ -67,7 +67,7 @@ struct SeqState {
 constexpr int kBlockTokens = 16;
 
 // Pages of one attention layer of a layered pool: [n_blocks][heads][K 16 x dim | V 16 x dim] elements at `offset` bytes, or
-// (parts == 1) one row of dim elements per token.
+// (parts == 1) dim elements per token and head, laid out as the layer's kernels like.
 struct KvLayerGeom {
     int heads = 0, dim = 0, parts = 2;
     uint64_t offset = 0, block_bytes = 0;

@@ -1,6 +1,7 @@
 // Layered decoder: configuration, weights, step function.
 //
-// A layer is  x <- x + sum of its mixer branches(LN1(x)),  then  x <- x + ff(LN2(x))  when it has a feed-forward part.
+// A layer is  x <- x + sum of its mixer branches(LN1(x)),  then  x <- x + ff(LN2(x))  when it has a feed-forward part (norms may
+// come behind the sums instead, see below).
 // All branches of a layer read the same normalised rows, so their input projections are ONE product over concatenated
 // weights, and their output projections are ONE product over concatenated (gated, scaled) head outputs that adds to the
 // residual in its epilogue:
@@ -10,6 +11,10 @@
 // With RMS norms the residual may be an average over the depth: every layer's result stays in a slot of its own, the norm in front of the
 // next layer forms the weighted sum on its way, and the product epilogues add (times the layer scale) to the slot.  A WKV layer's
 // norm writes five mixes with the previous token's row, which its input projections read as segments of one product.
+//
+// With norms behind the sums the parts read x itself: the product epilogues form residual factor x x + part, the norm kernel
+// behind them writes x and its rounding for the next product.  A mixture of experts is router -> route (choice, lists, tiles) ->
+// up products of all experts and the shared one -> down products -> the norm kernel adds a token's weighted rows on its way.
 //
 // The residual x is fp32; rows entering a product are bf16 (or fp32 in the exact mode).  Head sizes are padded with zero
 // weights to what the kernels take, so every size of a configuration works; sums over a head use the true size.
@@ -28,7 +33,11 @@ static int up(int n, int m) { return (n + m - 1) / m * m; }
 
 struct DBranch {
     jgpt_mixer_spec s{};
-    int D = 0, DK = 0, DV = 0;          // padded head sizes (attention: D; recurrent: DK, DV)
+    int DK = 0, DV = 0;                 // padded head sizes (of one map)
+    int maps = 1;
+    float lambda = 0.f;                 // differential attention: from the four vectors below
+    std::vector<float> lambda_part[4];
+    float *q_norm = nullptr, *k_norm = nullptr;
     int q = -1, k = -1, v = -1, g = -1, a1 = -1, b = -1, g1 = -1;  // column offsets inside proj
     int za = -1, zg = -1;               // column offsets inside z
     int ra = 0, rg = 0;                 // padded ranks
@@ -48,7 +57,7 @@ struct DBranch {
     void *w_uq = nullptr, *w_absorb = nullptr, *w_ukv = nullptr;  // [heads * DQ, qrp], [heads * KR, DP], [heads * (DP + DV), KR]
     float *dq_norm = nullptr, *dkv_norm = nullptr;
     bool recurrent() const { return s.kind == JGPT_MIX_GLA || s.kind == JGPT_MIX_DELTA || s.kind == JGPT_MIX_HGRN2 || s.kind == JGPT_MIX_WKV; }
-    int cols() const { return s.heads * (s.kind == JGPT_MIX_ATTENTION ? D : DV); }
+    int cols() const { return s.heads * DV; }
 };
 
 struct DLayer {
@@ -60,6 +69,14 @@ struct DLayer {
     float act_p0 = 0.f, act_p1 = 0.f;
     float *ls1 = nullptr, *ls2 = nullptr, *dwa = nullptr;  // residual_mult x layer scale; depth average
     uint64_t have = 0;
+    float *bias_in = nullptr;  // of the input projections
+    // mixture of experts: [experts + identity (+ 1: the shared expert's gate), ldw], then all experts' up [effp, ldw] and down [ldw, effp]
+    jgpt_moe_spec moe{};
+    int effp = 0, sffp = 0, n_router = 0;
+    void *w_router = nullptr, *w_eup = nullptr, *w_edown = nullptr, *w_sup = nullptr, *w_sdown = nullptr;
+    float *correction = nullptr;
+    uint64_t have_moe = 0;
+    std::vector<uint8_t> have_expert;
     const DBranch *shift() const { return br[0].s.kind == JGPT_MIX_WKV ? &br[0] : nullptr; }  // its input projections read mixes
 };
 
@@ -85,6 +102,10 @@ struct Decoder {
     // workspace
     float *x = nullptr, *raw = nullptr, *chunk_ws = nullptr, *logits = nullptr;
     void *h = nullptr, *proj = nullptr, *z = nullptr, *mixed = nullptr, *act = nullptr;
+    // mixtures: activations of the experts' rows, their results, the same of the shared expert; routing
+    void *e_act = nullptr, *e_out = nullptr, *s_act = nullptr, *s_out = nullptr;
+    float *r_logits = nullptr;
+    mix::RouteArgs route{};
     int *d_desc = nullptr, *h_desc = nullptr;
     int *d_next = nullptr, *h_next = nullptr;
     float *d_u = nullptr, *h_u = nullptr, *samp = nullptr;
@@ -209,6 +230,45 @@ static int32_t add_rotation(Decoder *d, const jgpt_mixer_spec &s) {
     return JGPT_OK;
 }
 
+static bool same_rotation(const jgpt_mixer_spec &x, const jgpt_mixer_spec &s) {
+    return x.rot_dims == s.rot_dims && x.rot_base == s.rot_base && x.rot_factor == s.rot_factor && x.rot_original == s.rot_original &&
+           x.rot_fast == s.rot_fast && x.rot_slow == s.rot_slow;
+}
+static int32_t find_rotation(Decoder *d, const jgpt_mixer_spec &s, int *rot) {
+    for (size_t k = 0; k < d->rot_specs.size(); k++)
+        if (same_rotation(d->rot_specs[k], s)) {
+            *rot = (int)k;
+            return JGPT_OK;
+        }
+    JGPT_REQUIRE(d->rots.size() < mix::kMaxRotations, JGPT_ERR_UNSUPPORTED, "more than %d different rotations", mix::kMaxRotations);
+    *rot = (int)d->rots.size();
+    return add_rotation(d, s);
+}
+
+// Sizes, weights and choice of a mixture.
+static int32_t plan_moe(Decoder *d, DLayer &y, const jgpt_moe_spec &m, int index) {
+    const int out = m.experts + m.identity;
+    JGPT_REQUIRE(m.experts > 0 && m.identity >= 0 && m.ff > 0 && m.shared_ff >= 0 && m.groups > 0 && out % m.groups == 0 && m.keep > 0 && m.keep <= m.groups &&
+                     m.top > 0 && m.top <= out / m.groups * m.keep,
+                 JGPT_ERR_INVALID_ARGUMENT, "layer %d: %d + %d experts of %d in %d groups, %d of %d kept, shared part of %d", index, m.experts, m.identity, m.ff,
+                 m.groups, m.top, m.keep, m.shared_ff);
+    auto known = [](int act) { return act == JGPT_ACT_RELU || act == JGPT_ACT_RELU2 || act == JGPT_ACT_GELU_TANH; };
+    JGPT_REQUIRE(known(m.act) && known(m.shared_act), JGPT_ERR_UNSUPPORTED, "layer %d: activations %d / %d", index, m.act, m.shared_act);
+    JGPT_REQUIRE(d->s.norm_after, JGPT_ERR_UNSUPPORTED, "layer %d: mixtures of experts go with norms behind the sums", index);
+    const uint64_t eb = d->eb, ldw = d->ldw;
+    y.moe = m, y.effp = up(m.ff, 16), y.sffp = up(m.shared_ff, 16), y.n_router = out + (m.shared_ff ? 1 : 0);
+    y.have_expert.assign((size_t)m.experts, 0);
+    TRY(dalloc(d, &y.w_router, y.n_router * ldw * eb));
+    TRY(dalloc(d, (void **)&y.correction, sizeof(float) * (uint64_t)out));
+    TRY(dalloc(d, &y.w_eup, (uint64_t)m.experts * y.effp * ldw * eb));
+    TRY(dalloc(d, &y.w_edown, (uint64_t)m.experts * y.effp * ldw * eb));
+    if (m.shared_ff) {
+        TRY(dalloc(d, &y.w_sup, y.sffp * ldw * eb));
+        TRY(dalloc(d, &y.w_sdown, y.sffp * ldw * eb));
+    }
+    return JGPT_OK;
+}
+
 // Sizes, column layouts and device memory of one layer.
 static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int index) {
     JGPT_REQUIRE(ls.n_branches >= 1 && ls.n_branches <= JGPT_MAX_BRANCHES, JGPT_ERR_INVALID_ARGUMENT, "layer %d: %d mixer branches", index,
@@ -229,13 +289,21 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
                      "layer %d: heads %d / %d, head sizes %d / %d", index, s.heads, s.kv_heads, s.dim, s.vdim);
         b.out = out;
         if (s.kind == JGPT_MIX_ATTENTION) {
-            b.D = mix::attn_padded_head(s.dim, s.vdim);
-            JGPT_REQUIRE(b.D > 0, JGPT_ERR_UNSUPPORTED, "layer %d: head sizes %d / %d", index, s.dim, s.vdim);
-            b.q = seg(s.heads * b.D), b.k = seg(s.kv_heads * b.D), b.v = seg(s.kv_heads * b.D);
-            if (s.gate) b.g = seg(s.heads);
+            b.maps = std::max(s.maps, 1);
+            JGPT_REQUIRE(b.maps <= 2 && s.gate >= 0 && s.gate <= 2, JGPT_ERR_UNSUPPORTED, "layer %d: %d attention maps, gate %d", index, b.maps, s.gate);
+            JGPT_REQUIRE(mix::attn_padded_head(s.dim, s.vdim, b.maps, &b.DK, &b.DV), JGPT_ERR_UNSUPPORTED, "layer %d: head sizes %d / %d", index, s.dim, s.vdim);
+            JGPT_REQUIRE(s.rot_dims >= 0 && s.rot_dims % 2 == 0 && s.rot_dims <= s.dim && (s.rot_dims == 0 || (s.rot_base > 1.0 && d->rms)), JGPT_ERR_INVALID_ARGUMENT,
+                         "layer %d: rotation of %d of %d", index, s.rot_dims, s.dim);
+            b.q = seg(s.heads * b.maps * b.DK), b.k = seg(s.kv_heads * b.maps * b.DK), b.v = seg(s.kv_heads * b.DV);
+            if (s.gate) b.g = seg(s.gate == mix::GATE_HEAD ? s.heads : s.heads * b.DV);
+            if (s.rot_dims) TRY(find_rotation(d, s, &b.rot));
+            if (s.qk_norm) {
+                TRY(dalloc(d, (void **)&b.q_norm, sizeof(float) * (uint64_t)s.dim));
+                TRY(dalloc(d, (void **)&b.k_norm, sizeof(float) * (uint64_t)s.dim));
+            }
             b.kv_layer = (int)d->kv.size();
             KvLayerGeom geom;
-            geom.heads = s.kv_heads, geom.dim = b.D;
+            geom.heads = s.kv_heads, geom.dim = b.maps * b.DK + b.DV, geom.parts = 1;
             d->kv.push_back(geom);
         } else if (s.kind == JGPT_MIX_GLA || s.kind == JGPT_MIX_DELTA) {
             const bool delta = s.kind == JGPT_MIX_DELTA;
@@ -301,10 +369,6 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
             b.DP = up(s.dim, 8), b.DQ = b.DP + up(s.rot_dim, 8), b.DV = up(s.vdim, 8), b.qrp = up(s.q_rank, 8);
             b.expand = !d->f32 && mix::latent_expandable(s.dim, s.rot_dim, s.vdim);
             b.dq = seg(s.q_rank);
-            auto same_rotation = [&](const jgpt_mixer_spec &x) {
-                return x.rot_dims == s.rot_dims && x.rot_base == s.rot_base && x.rot_factor == s.rot_factor && x.rot_original == s.rot_original &&
-                       x.rot_fast == s.rot_fast && x.rot_slow == s.rot_slow;
-            };
             if (s.kv_from == 0) {
                 b.dkv = seg(s.kv_rank), b.dkr = seg(s.rot_dim);
                 b.kv_layer = (int)d->kv.size();
@@ -317,17 +381,11 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
                 const DBranch *from = nullptr;
                 for (const DBranch &x : d->L[(size_t)s.kv_from - 1].br)
                     if (x.s.kind == JGPT_MIX_LATENT && x.s.kv_from == 0) from = &x;
-                JGPT_REQUIRE(from && from->s.kv_rank == s.kv_rank && from->s.rot_dim == s.rot_dim && same_rotation(from->s), JGPT_ERR_INVALID_ARGUMENT,
+                JGPT_REQUIRE(from && from->s.kv_rank == s.kv_rank && from->s.rot_dim == s.rot_dim && same_rotation(from->s, s), JGPT_ERR_INVALID_ARGUMENT,
                              "layer %d: layer %d has no cache of its sizes and rotation", index, s.kv_from - 1);
                 b.kv_layer = from->kv_layer;
             }
-            for (size_t k = 0; k < d->rot_specs.size() && b.rot < 0; k++)
-                if (same_rotation(d->rot_specs[k])) b.rot = (int)k;
-            if (b.rot < 0) {
-                JGPT_REQUIRE(d->rots.size() < mix::kMaxRotations, JGPT_ERR_UNSUPPORTED, "more than %d different rotations", mix::kMaxRotations);
-                b.rot = (int)d->rots.size();
-                TRY(add_rotation(d, ls.branch[i]));
-            }
+            TRY(find_rotation(d, s, &b.rot));
             TRY(dalloc(d, &b.w_uq, (uint64_t)s.heads * b.DQ * b.qrp * eb));
             TRY(dalloc(d, &b.w_absorb, (uint64_t)s.heads * b.KR * b.DP * eb));
             TRY(dalloc(d, &b.w_ukv, (uint64_t)s.heads * (b.DP + b.DV) * b.KR * eb));
@@ -339,8 +397,12 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
         y.br.push_back(b);
     }
     y.n_in = in, y.n_out = up(out, 8), y.n_z = zc, y.ff = ls.ff, y.ffp = up(ls.ff, 16), y.ff_kind = ls.ff_kind;
-    JGPT_REQUIRE(ls.ff_kind == JGPT_FF_GATED_GELU || ls.ff_kind == JGPT_FF_XIELU, JGPT_ERR_UNSUPPORTED, "layer %d: feed-forward kind %d", index, ls.ff_kind);
-    if (d->rms) {
+    JGPT_REQUIRE(ls.ff_kind >= JGPT_FF_GATED_GELU && ls.ff_kind <= JGPT_FF_MOE, JGPT_ERR_UNSUPPORTED, "layer %d: feed-forward kind %d", index, ls.ff_kind);
+    JGPT_REQUIRE(!d->s.norm_after || !y.shift(), JGPT_ERR_UNSUPPORTED, "layer %d: WKV mixes normed inputs", index);
+    for (const DBranch &b : y.br)
+        if (b.s.kind == JGPT_MIX_ATTENTION && b.s.qkv_bias && !y.bias_in) TRY(dalloc(d, (void **)&y.bias_in, sizeof(float) * (uint64_t)y.n_in));
+    if (y.ff && y.ff_kind == JGPT_FF_MOE) TRY(plan_moe(d, y, ls.moe, index));
+    if (d->rms && !d->s.norm_after) {
         TRY(dalloc(d, (void **)&y.ls1, sizeof(float) * (uint64_t)W));
         TRY(dalloc(d, (void **)&y.ls2, sizeof(float) * (uint64_t)W));
         const std::vector<float> mult((size_t)W, d->s.residual_mult);
@@ -352,8 +414,10 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
     TRY(dalloc(d, (void **)&y.n1w, sizeof(float) * (uint64_t)W));
     TRY(dalloc(d, (void **)&y.n1b, sizeof(float) * (uint64_t)W));
     if (y.ff) {
-        TRY(dalloc(d, &y.w_gu, (y.ff_kind == JGPT_FF_GATED_GELU ? 2ull : 1ull) * y.ffp * d->ldw * eb));
-        TRY(dalloc(d, &y.w_down, (uint64_t)W * y.ffp * eb));
+        if (y.ff_kind != JGPT_FF_MOE) {
+            TRY(dalloc(d, &y.w_gu, (y.ff_kind == JGPT_FF_XIELU ? 1ull : 2ull) * y.ffp * d->ldw * eb));
+            TRY(dalloc(d, &y.w_down, (uint64_t)W * y.ffp * eb));
+        }
         TRY(dalloc(d, (void **)&y.n2w, sizeof(float) * (uint64_t)W));
         TRY(dalloc(d, (void **)&y.n2b, sizeof(float) * (uint64_t)W));
     }
@@ -369,11 +433,15 @@ static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
     d->rms = d->s.norm == JGPT_NORM_RMS;
     d->lat_min = env_int("JGPT_B200_LATENT_EXPAND_MIN", 64);
     int n_in = 8, n_z = 8, n_out = 8, ffp = 16, raw = 0, mixes = 1, cq = 0, lq = 0, lqa = 0, cxw = 0, kvx = 0;
+    int top = 0, experts = 0, outputs = 0, effp = 0, sffp = 0, tiles = 0;
     bool latent = false, unbounded = false, expand = true;
     for (int i = 0; i < d->s.n_layers; i++) {
         DLayer &y = d->L[(size_t)i];
         TRY(plan_layer(d, y, layers[i], i));
         n_in = std::max(n_in, y.n_in), n_z = std::max(n_z, y.n_z), n_out = std::max(n_out, y.n_out), ffp = std::max(ffp, y.ffp);
+        top = std::max(top, y.moe.top), experts = std::max(experts, y.moe.experts), outputs = std::max(outputs, y.n_router);
+        effp = std::max(effp, y.effp), sffp = std::max(sffp, y.sffp);
+        if (y.effp) tiles = std::max(tiles, std::min(y.moe.experts, d->R * y.moe.top) + d->R * y.moe.top / 16);
         for (const DBranch &b : y.br) {
             if (b.s.kind == JGPT_MIX_WKV) mixes = 5;
             if (b.s.kind == JGPT_MIX_LATENT) {
@@ -395,6 +463,25 @@ static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
     TRY(dalloc(d, (void **)&d->x, sizeof(float) * R * W));
     if (d->s.depth_average) TRY(dalloc(d, (void **)&d->slots, sizeof(float) * (d->L.size() + 1) * R * W));
     for (mix::Rotation &r : d->rots) TRY(dalloc(d, (void **)&r.out, sizeof(float2) * R * r.half));
+    if (top) {
+        const uint64_t copies = R * (uint64_t)top;
+        mix::RouteArgs &r = d->route;
+        TRY(dalloc(d, &d->e_act, copies * effp * eb));
+        TRY(dalloc(d, &d->e_out, copies * d->ldw * eb));
+        TRY(dalloc(d, &d->s_act, R * sffp * eb));
+        TRY(dalloc(d, &d->s_out, R * (sffp ? d->ldw : 0) * eb));
+        r.ld = up(outputs, 4), r.cap = d->R;
+        TRY(dalloc(d, (void **)&d->r_logits, sizeof(float) * R * r.ld));
+        TRY(dalloc(d, (void **)&r.slots, sizeof(mix::RouteSlot) * copies));
+        TRY(dalloc(d, (void **)&r.row_weights, sizeof(float2) * R));
+        TRY(dalloc(d, (void **)&r.list, sizeof(int) * R * experts));
+        TRY(dalloc(d, (void **)&r.counts, sizeof(int) * (uint64_t)experts));
+        TRY(dalloc(d, (void **)&r.offsets, sizeof(int) * (uint64_t)experts));
+        TRY(dalloc(d, (void **)&r.ticket, sizeof(int)));
+        TRY(dalloc(d, (void **)&r.tiles, sizeof(nt::RowTile) * (uint64_t)tiles));
+        TRY(dalloc(d, (void **)&r.n_tiles, sizeof(int)));
+        r.logits = d->r_logits;
+    }
     if (unbounded) d->max_window = 0;
     if (!latent || !expand) d->lat_min = 0;
     if (latent) {
@@ -442,7 +529,10 @@ static uint64_t needed_roles(const jgpt_mixer_spec &s) {
         return bit(JGPT_W_Q) | bit(JGPT_W_K) | bit(JGPT_W_V) | bit(JGPT_W_G) | bit(JGPT_W_O) | bit(JGPT_W_A1) | bit(JGPT_W_A2) | bit(JGPT_W_DECAY_BIAS) |
                bit(JGPT_W_BONUS) | bit(JGPT_W_HEAD_NORM) | bit(JGPT_W_MU_R) | bit(JGPT_W_MU_K) | bit(JGPT_W_MU_V) | bit(JGPT_W_MU_G) | bit(JGPT_W_MU_W);
     uint64_t n = bit(JGPT_W_Q) | bit(JGPT_W_K) | bit(JGPT_W_V) | bit(JGPT_W_O);
-    if (s.kind == JGPT_MIX_ATTENTION) return s.gate ? n | bit(JGPT_W_G) : n;
+    if (s.kind == JGPT_MIX_ATTENTION)
+        return n | (s.gate ? bit(JGPT_W_G) : 0) | (s.qkv_bias ? bit(JGPT_W_Q_BIAS) | bit(JGPT_W_K_BIAS) | bit(JGPT_W_V_BIAS) : 0) |
+               (s.qk_norm ? bit(JGPT_W_Q_NORM) | bit(JGPT_W_K_NORM) : 0) |
+               (s.maps > 1 ? bit(JGPT_W_LQ1) | bit(JGPT_W_LK1) | bit(JGPT_W_LQ2) | bit(JGPT_W_LK2) : 0);
     n |= bit(JGPT_W_A1) | bit(JGPT_W_A2) | bit(JGPT_W_DECAY_BIAS) | bit(JGPT_W_HEAD_NORM);
     if (s.kind == JGPT_MIX_GLA) return n | bit(JGPT_W_G);
     return n | bit(JGPT_W_B) | bit(JGPT_W_A_LOG) | bit(JGPT_W_G1) | bit(JGPT_W_G2) | bit(JGPT_W_CONV_Q) | bit(JGPT_W_CONV_K) | bit(JGPT_W_CONV_V);
@@ -456,7 +546,15 @@ static int32_t missing_weights(const Decoder *d) {
     for (size_t i = 0; i < d->L.size(); i++) {
         const DLayer &y = d->L[i];
         uint64_t n = bit(JGPT_W_NORM1) | (beta & bit(JGPT_W_NORM1_B)) | (d->s.layer_scale ? bit(JGPT_W_LS1) : 0) | (d->s.depth_average ? bit(JGPT_W_DWA) : 0);
-        if (y.ff)
+        if (y.effp) {
+            n |= bit(JGPT_W_NORM2);
+            const uint64_t e = bit(JGPT_W_EXPERT_UP - 64) | bit(JGPT_W_EXPERT_DOWN - 64);
+            const uint64_t m = bit(JGPT_W_ROUTER - 64) | bit(JGPT_W_CORRECTION - 64) |
+                               (y.sffp ? bit(JGPT_W_SHARED_GATE - 64) | bit(JGPT_W_SHARED_UP - 64) | bit(JGPT_W_SHARED_DOWN - 64) : 0);
+            JGPT_REQUIRE((y.have_moe & m) == m, JGPT_ERR_ILLEGAL_STATE, "router or shared expert of layer %zu are not set", i);
+            for (size_t k = 0; k < y.have_expert.size(); k++)
+                JGPT_REQUIRE((y.have_expert[k] & e) == e, JGPT_ERR_ILLEGAL_STATE, "expert %zu of layer %zu is not set", k, i);
+        } else if (y.ff)
             n |= bit(JGPT_W_NORM2) | (beta & bit(JGPT_W_NORM2_B)) | bit(JGPT_W_FF_UP) | bit(JGPT_W_FF_DOWN) | (d->s.layer_scale ? bit(JGPT_W_LS2) : 0) |
                  (y.ff_kind == JGPT_FF_XIELU ? bit(JGPT_W_FF_ACT) : bit(JGPT_W_FF_GATE));
         JGPT_REQUIRE((y.have & n) == n, JGPT_ERR_ILLEGAL_STATE, "norm or feed-forward weights of layer %zu are not set", i);
@@ -493,10 +591,42 @@ static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const flo
         return JGPT_OK;
     }
     DLayer &y = d->L[(size_t)layer];
+    if (branch >= JGPT_MAX_BRANCHES) {
+        const int e = branch - JGPT_MAX_BRANCHES, ldw = d->ldw;
+        JGPT_REQUIRE(e < (int)y.have_expert.size(), JGPT_ERR_OUT_OF_RANGE, "layer %d has %zu experts", layer, y.have_expert.size());
+        auto expert = [&](void *base) { return reinterpret_cast<uint8_t *>(base) + (size_t)e * y.effp * ldw * d->eb; };
+        if (role == JGPT_W_EXPERT_UP) {
+            TRY(shape(y.moe.ff, W));
+            TRY(put_matrix(d, expert(y.w_eup), ldw, 0, 0, src, rows, cols, none, none));
+        } else if (role == JGPT_W_EXPERT_DOWN) {
+            TRY(shape(W, y.moe.ff));
+            TRY(put_matrix(d, expert(y.w_edown), y.effp, 0, 0, src, rows, cols, none, none));
+        } else {
+            return fail(JGPT_ERR_INVALID_ARGUMENT, "tensor %d does not belong to an expert", role);
+        }
+        y.have_expert[(size_t)e] |= (uint8_t)bit(role - 64);
+        return JGPT_OK;
+    }
+    if (branch < 0 && role >= 64) {
+        const int out = y.moe.experts + y.moe.identity;
+        const bool shared = role == JGPT_W_SHARED_GATE || role == JGPT_W_SHARED_UP || role == JGPT_W_SHARED_DOWN;
+        JGPT_REQUIRE(y.effp && role < 128 && (!shared || y.sffp), JGPT_ERR_INVALID_ARGUMENT, "layer %d has no %s", layer, shared ? "shared expert" : "mixture of experts");
+        switch (role) {
+            case JGPT_W_ROUTER: TRY(shape(out, W)); TRY(put_matrix(d, y.w_router, d->ldw, 0, 0, src, rows, cols, none, none)); break;
+            case JGPT_W_SHARED_GATE: TRY(shape(1, W)); TRY(put_matrix(d, y.w_router, d->ldw, out, 0, src, rows, cols, none, none)); break;
+            case JGPT_W_CORRECTION: TRY(shape(1, out)); TRY(put_floats(d, y.correction, src, 1, out, none)); break;
+            case JGPT_W_SHARED_UP: TRY(shape(y.moe.shared_ff, W)); TRY(put_matrix(d, y.w_sup, d->ldw, 0, 0, src, rows, cols, none, none)); break;
+            case JGPT_W_SHARED_DOWN: TRY(shape(W, y.moe.shared_ff)); TRY(put_matrix(d, y.w_sdown, y.sffp, 0, 0, src, rows, cols, none, none)); break;
+            default: return fail(JGPT_ERR_INVALID_ARGUMENT, "tensor %d does not belong to a layer", role);
+        }
+        y.have_moe |= bit(role - 64);
+        return JGPT_OK;
+    }
     if (branch < 0) {
         const Grouping pair{16, 32};
         const bool ff_role = role == JGPT_W_FF_ACT || role == JGPT_W_LS2 || role == JGPT_W_FF_GATE || role == JGPT_W_FF_UP || role == JGPT_W_FF_DOWN || role == JGPT_W_NORM2 || role == JGPT_W_NORM2_B;
-        JGPT_REQUIRE(!ff_role || y.ff, JGPT_ERR_INVALID_ARGUMENT, "layer %d has no feed-forward part", layer);
+        const bool ff_norm = role == JGPT_W_NORM2 || role == JGPT_W_NORM2_B;
+        JGPT_REQUIRE(!ff_role || (y.ff && (ff_norm || !y.effp)), JGPT_ERR_INVALID_ARGUMENT, "layer %d has no such feed-forward part", layer);
         switch (role) {
             case JGPT_W_NORM1: TRY(shape(1, W)); TRY(put_floats(d, y.n1w, src, 1, W, none)); break;
             case JGPT_W_NORM1_B: TRY(shape(1, W)); TRY(put_floats(d, y.n1b, src, 1, W, none)); break;
@@ -550,20 +680,38 @@ static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const flo
     JGPT_REQUIRE(role >= 0 && role < 63 && (needed_roles(s) & bit(role)), JGPT_ERR_INVALID_ARGUMENT, "tensor %d does not belong to mixer kind %d", role,
                  s.kind);
     const bool att = s.kind == JGPT_MIX_ATTENTION;
-    const Grouping kg{s.dim, att ? b.D : b.DK}, vg{s.vdim, att ? b.D : b.DV};
-    const int vheads = att ? s.kv_heads : s.heads, qheads = att ? s.heads : s.kv_heads;
+    const Grouping kg{s.dim, b.DK}, vg{s.vdim, b.DV};
+    const int vheads = att ? s.kv_heads : s.heads, qheads = att ? s.heads * b.maps : s.kv_heads, kheads = s.kv_heads * (att ? b.maps : 1);
     auto into_proj = [&](int off, int n, Grouping g) -> int32_t {
         TRY(shape(n, W));
         return put_matrix(d, y.w_in, d->ldw, off, 0, src, rows, cols, g, none);
     };
     switch (role) {
         case JGPT_W_Q: TRY(into_proj(b.q, qheads * s.dim, kg)); break;
-        case JGPT_W_K: TRY(into_proj(b.k, s.kv_heads * s.dim, kg)); break;
+        case JGPT_W_K: TRY(into_proj(b.k, kheads * s.dim, kg)); break;
         case JGPT_W_V: TRY(into_proj(b.v, vheads * s.vdim, vg)); break;
         case JGPT_W_G:
-            if (att) TRY(into_proj(b.g, s.heads, none));
+            if (att && s.gate == mix::GATE_HEAD) TRY(into_proj(b.g, s.heads, none));
             else TRY(into_proj(b.g, s.heads * s.vdim, vg));
             break;
+        case JGPT_W_Q_BIAS: TRY(shape(1, qheads * s.dim)); TRY(put_floats(d, y.bias_in + b.q, src, cols, 1, kg)); break;
+        case JGPT_W_K_BIAS: TRY(shape(1, kheads * s.dim)); TRY(put_floats(d, y.bias_in + b.k, src, cols, 1, kg)); break;
+        case JGPT_W_V_BIAS: TRY(shape(1, vheads * s.vdim)); TRY(put_floats(d, y.bias_in + b.v, src, cols, 1, vg)); break;
+        case JGPT_W_Q_NORM: TRY(shape(1, s.dim)); TRY(put_floats(d, b.q_norm, src, 1, cols, none)); break;
+        case JGPT_W_K_NORM: TRY(shape(1, s.dim)); TRY(put_floats(d, b.k_norm, src, 1, cols, none)); break;
+        case JGPT_W_LQ1:
+        case JGPT_W_LK1:
+        case JGPT_W_LQ2:
+        case JGPT_W_LK2: {
+            TRY(shape(1, s.dim));
+            b.lambda_part[role - JGPT_W_LQ1].assign(src, src + s.dim);
+            double dot[2] = {0, 0};
+            for (int k = 0; k < 2; k++)
+                if (const std::vector<float> &u = b.lambda_part[2 * k], &v = b.lambda_part[2 * k + 1]; u.size() == v.size())
+                    for (size_t j = 0; j < u.size(); j++) dot[k] += (double)u[j] * v[j];
+            b.lambda = (float)(std::exp(dot[0]) - std::exp(dot[1]) + (double)s.diff);
+            break;
+        }
         case JGPT_W_B: TRY(into_proj(b.b, s.heads, none)); break;
         case JGPT_W_A1: TRY(into_proj(b.a1, s.rank_a, none)); break;
         case JGPT_W_G1: TRY(into_proj(b.g1, s.rank_g, none)); break;
@@ -704,6 +852,31 @@ static int32_t enqueue_latent(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
     return JGPT_OK;
 }
 
+// Router, choice, products of the experts; the norm kernel adds what m says.
+static int32_t enqueue_moe(Decoder *d, const DLayer &y, int R, int pdl, mix::MoeSum &m) {
+    const int ldw = d->ldw, T = nt::group_tile_rows(d->f32, R, y.moe.top, y.moe.experts);
+    auto act = [](int a) { return a == JGPT_ACT_RELU2 ? nt::ACT_RELU2 : (a == JGPT_ACT_RELU ? nt::ACT_RELU : nt::ACT_GELU); };
+    mix::RouteArgs r = d->route;
+    nt::Problem logits{d->h, y.w_router, d->r_logits, nullptr, R, y.n_router, ldw, ldw, ldw, r.ld, 1.f};
+    TRY(product(d, &logits, 1, nt::EPI_SCALE_F32, pdl));
+    r.experts = y.moe.experts, r.identity = y.moe.identity, r.top = y.moe.top, r.groups = y.moe.groups, r.keep = y.moe.keep, r.shared = y.sffp ? 1 : 0;
+    r.correction = y.correction, r.tile_rows = T, r.max_tiles = std::min(y.moe.experts, R * y.moe.top) + R * y.moe.top / T;
+    TRY(mix::launch_route(r, R, pdl, d->ctx->stream));
+    nt::RowGroups g;
+    g.tiles = r.tiles, g.n_tiles = r.n_tiles, g.max_tiles = r.max_tiles, g.rows = T, g.n_groups = y.moe.experts, g.a_rows = R, g.w_group = (long long)y.effp * ldw;
+    nt::Problem in[2] = {{d->h, y.w_eup, d->e_act, r.list, R, y.effp, ldw, ldw, ldw, y.effp, 1.f}, {d->h, y.w_sup, d->s_act, nullptr, R, y.sffp, ldw, ldw, ldw, y.sffp, 1.f}};
+    in[0].grp = g, in[0].act = act(y.moe.act), in[1].act = act(y.moe.shared_act);
+    TRY(product(d, in, y.sffp ? 2 : 1, nt::EPI_ACT, pdl));
+    g.a_rows = R * y.moe.top, g.early = true;
+    nt::Problem out[2] = {{d->e_act, y.w_edown, d->e_out, nullptr, R, ldw, y.effp, y.effp, y.effp, ldw, 1.f},
+                          {d->s_act, y.w_sdown, d->s_out, nullptr, R, ldw, y.sffp, y.sffp, y.sffp, ldw, 1.f}};
+    out[0].grp = g;
+    TRY(product(d, out, y.sffp ? 2 : 1, nt::EPI_STORE, pdl));
+    m.out = d->e_out, m.shared = y.sffp ? d->s_out : nullptr, m.ld = ldw, m.top = y.moe.top, m.cap = r.cap, m.slots = r.slots, m.row_weights = r.row_weights;
+    m.offsets = r.offsets, m.alpha = d->s.residual_scale;
+    return JGPT_OK;
+}
+
 static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, const std::vector<LatentBatch> &batches, uint64_t capture_rows) {
     const int W = d->s.width, R = sd.rows, ldw = d->ldw, eb = d->eb;
     const float eps = d->s.eps;
@@ -711,11 +884,15 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
     int *status = d->ctx->d_status;
     const int pdl = d->overlap && !d->f32 && !capture_rows ? 3 : 0;
     const uint64_t slot = (uint64_t)d->R * W, mix_stride = (uint64_t)d->R * ldw;
-    const bool deep = d->s.depth_average;
+    const bool deep = d->s.depth_average, after = d->s.norm_after;
+    const float res_scale = after ? d->s.residual_scale : 1.f;
     for (size_t i = 0; i < d->L.size(); i++) {
         DLayer &y = d->L[i];
         float *from = d->x, *to = deep ? d->slots + (i + 1) * slot : d->x;  // residual in front of the layer, its result
-        if (d->rms) {
+        if (after) {  // the norms behind the sums leave h
+            if (i == 0)
+                TRY(mix::launch_residual_norm(d->f32, sd, residual(d, 0), nullptr, R, nullptr, eps, d->x, d->h, mix::ShiftArgs{}, W, ldw, status, pdl & 2, st));
+        } else if (d->rms) {
             const DBranch *w = y.shift();
             mix::ShiftArgs sh{};
             if (w) {
@@ -741,13 +918,18 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
             TRY(product(d, in, 2, nt::EPI_ACT, pdl));
         } else {
             nt::Problem in{d->h, y.w_in, d->proj, nullptr, R, y.n_in, ldw, ldw, ldw, y.n_in, 1.f};
+            in.bias = y.bias_in;
             TRY(product(d, &in, 1, nt::EPI_STORE, pdl));
         }
         for (DBranch &b : y.br) {
             if (b.s.kind == JGPT_MIX_ATTENTION) {
                 mix::AttnArgs a{};
                 a.proj = d->proj, a.ldp = y.n_in, a.q_off = b.q, a.k_off = b.k, a.v_off = b.v, a.g_off = b.g;
-                a.heads = b.s.heads, a.kv_heads = b.s.kv_heads, a.D = b.D, a.chunk = b.s.chunk, a.scale = b.s.score_scale, a.out_scale = b.s.out_scale;
+                a.heads = b.s.heads, a.kv_heads = b.s.kv_heads, a.maps = b.maps, a.DK = b.DK, a.DV = b.DV, a.dim = b.s.dim, a.vdim = b.s.vdim;
+                a.gate = b.s.gate, a.chunk = b.s.chunk, a.scale = b.s.score_scale, a.out_scale = b.s.out_scale;
+                a.q_norm = b.q_norm, a.k_norm = b.k_norm, a.eps = eps, a.interleaved = b.s.rot_interleaved;
+                if (b.rot >= 0) a.cs = d->rots[(size_t)b.rot].out, a.half = b.s.rot_dims / 2;
+                a.lambda = b.lambda, a.diff_scale = 1.f - b.s.diff;
                 a.kv = p->vkv + p->vlayers[(size_t)b.kv_layer].offset, a.table = p->d_table, a.n_blocks = p->n_blocks, a.mbs = p->max_blocks_per_seq;
                 a.out = d->mixed, a.ldo = y.n_out, a.out_off = b.out;
                 a.sm_count = d->ctx->sm_count, a.status = status;
@@ -772,24 +954,30 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
             }
         }
         nt::Problem out{d->mixed, y.w_out, to, nullptr, R, W, y.n_out, y.n_out, y.n_out, W, 1.f};
-        out.res = from, out.colscale = y.ls1;
+        out.res = from, out.colscale = y.ls1, out.res_scale = res_scale;
         TRY(product(d, &out, 1, nt::EPI_ADD_F32, pdl));
-        if (y.ff) {
-            if (d->rms) {
+        if (after) TRY(mix::launch_post_norm(d->f32, d->x, R, y.n1w, eps, d->h, mix::MoeSum{}, W, ldw, pdl, st));
+        mix::MoeSum moe{};
+        if (y.effp) {
+            TRY(enqueue_moe(d, y, R, pdl, moe));
+        } else if (y.ff) {
+            if (d->rms && !after) {
                 mix::RowSource src{};
                 src.slots = to, src.n_slots = 1;
                 TRY(mix::launch_residual_norm(d->f32, sd, src, nullptr, R, y.n2w, eps, nullptr, d->h, mix::ShiftArgs{}, W, ldw, status, pdl, st));
-            } else {
+            } else if (!after) {
                 TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n2w, y.n2b}, eps, d->h, R, W, ldw, pdl, st));
             }
-            const bool gated = y.ff_kind == JGPT_FF_GATED_GELU;
+            const bool gated = y.ff_kind != JGPT_FF_XIELU;
             nt::Problem gu{d->h, y.w_gu, d->act, nullptr, R, gated ? 2 * y.ffp : y.ffp, ldw, ldw, ldw, y.ffp, 1.f};
+            gu.act = y.ff_kind == JGPT_FF_GATED_RELU ? nt::ACT_RELU : nt::ACT_GELU;
             if (!gated) gu.act = nt::ACT_XIELU, gu.p0 = y.act_p0, gu.p1 = y.act_p1;
-            TRY(product(d, &gu, 1, gated ? nt::EPI_GATE_GELU : nt::EPI_ACT, pdl));
+            TRY(product(d, &gu, 1, gated ? nt::EPI_GATE : nt::EPI_ACT, pdl));
             nt::Problem down{d->act, y.w_down, to, nullptr, R, W, y.ffp, y.ffp, y.ffp, W, 1.f};
-            down.colscale = y.ls2;
+            down.colscale = y.ls2, down.res_scale = res_scale;
             TRY(product(d, &down, 1, nt::EPI_ADD_F32, pdl));
         }
+        if (after && y.ff) TRY(mix::launch_post_norm(d->f32, d->x, R, y.n2w, eps, d->h, moe, W, ldw, pdl, st));
         if (capture_rows) {
             if (deep) TRY(mix::launch_residual_norm(d->f32, sd, residual(d, i + 1), nullptr, R, d->fnw, eps, d->x, nullptr, mix::ShiftArgs{}, W, ldw, status, 0, st));
             JGPT_CUDA_TRY(cudaMemcpyAsync(d->capture + (uint64_t)i * capture_rows * W, d->x, sizeof(float) * capture_rows * W, cudaMemcpyDeviceToHost, st));
@@ -1126,6 +1314,8 @@ int32_t jgpt_decoder_create(jgpt_ctx ctxh, const jgpt_decoder_spec *spec, const 
     JGPT_REQUIRE(rms || spec->norm == JGPT_NORM_LAYER, JGPT_ERR_UNSUPPORTED, "norm %d", spec->norm);
     JGPT_REQUIRE(rms ? !spec->pos_table && !spec->embed_norm : !spec->layer_scale && !spec->depth_average && spec->residual_mult == 1.f, JGPT_ERR_UNSUPPORTED,
                  "layer norms go with embedding norms and learned positions, RMS norms with residual factors and depth averages");
+    JGPT_REQUIRE(!spec->norm_after || (rms && !spec->layer_scale && !spec->depth_average && spec->residual_mult == 1.f), JGPT_ERR_UNSUPPORTED,
+                 "norms behind the sums are RMS norms over a plain residual");
     JGPT_REQUIRE(dtype == JGPT_DTYPE_BF16 || dtype == JGPT_DTYPE_F32, JGPT_ERR_INVALID_ARGUMENT, "dtype %d", dtype);
     JGPT_CUDA_TRY(make_current(c));
     Decoder *d = new Decoder();

@@ -40,7 +40,7 @@ constexpr size_t small_smem(int k_split) {
     return std::max(std::max(small_ring_bytes<MT, NH, STAGES>(), small_red_bytes<MT, NH>()), sizeof(float) * (size_t)(k_split - 1) * 16 * MT * 32 * NH);
 }
 
-template <int MT, int NH, int STAGES, int EPI>
+template <int MT, int NH, int STAGES, int EPI, bool GROUPED>
 __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args) {
     constexpr int BM = 16 * MT, kBN = 32 * NH, KS = 8 / NH;
     extern __shared__ __align__(128) uint8_t nt_smem[];
@@ -55,11 +55,28 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
     const bool second = args.n > 1 && tile >= args.tiles[0];
     if (second) tile -= args.tiles[0];
     const Problem &P = second ? args.p[1] : args.p[0];
-    const int M = P.M, N = P.N, K = P.K, lda = P.lda, ldw = P.ldw;
-    const int per_seg = args.per_seg[second], seg = tile / per_seg, seg_n = P.seg_n;
-    const int m0 = blockIdx.y * BM, n0 = seg * seg_n + tile % per_seg * kBN, n_end = min(N, (seg + 1) * seg_n), cn = seg * P.c_seg;
-    const __nv_bfloat16 *__restrict__ A = reinterpret_cast<const __nv_bfloat16 *>(P.A) + seg * P.a_seg;
+    const int N = P.N, K = P.K, lda = P.lda, ldw = P.ldw, per_seg = args.per_seg[second];
+    int M = P.M, m0 = blockIdx.y * BM, seg = tile / per_seg, src0 = 0;
+    bool wait = args.pdl & 1;
     const __nv_bfloat16 *__restrict__ W = reinterpret_cast<const __nv_bfloat16 *>(P.W);
+    if (GROUPED) {  // a grid of one dimension: the groups' row tiles, then those of the product beside them
+        if (!second) {
+            if (wait && !P.grp.early) griddep_wait(), wait = false;
+            if (args.pdl & 2) griddep_launch_dependents();
+            if (seg >= *P.grp.n_tiles) {
+                if (wait) griddep_wait();  // whoever comes next counts on this launch having waited
+                return;
+            }
+            const RowTile t = P.grp.tiles[seg];
+            m0 = t.row0, M = t.row_end, src0 = t.src0 - t.row0, W += t.group * P.grp.w_group;
+        } else {
+            if (args.pdl & 2) griddep_launch_dependents();
+            m0 = seg * BM;
+        }
+        seg = 0;
+    }
+    const int seg_n = P.seg_n, n0 = seg * seg_n + tile % per_seg * kBN, n_end = min(N, (seg + 1) * seg_n), cn = seg * P.c_seg;
+    const __nv_bfloat16 *__restrict__ A = reinterpret_cast<const __nv_bfloat16 *>(P.A) + seg * P.a_seg;
     const int nk_all = (K + kBK - 1) / kBK;
     const int kt0 = k_part * nk_all / args.k_split, nk = (k_part + 1) * nk_all / args.k_split - kt0;
 
@@ -72,19 +89,19 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
             cp_async16(Ws + ((size_t)buf * kBN + r) * kBK + ((c16 ^ (r & 7)) * 8), ok ? W + (size_t)(n0 + r) * ldw + k : W, ok);
         }
     };
-    if (args.pdl & 2) griddep_launch_dependents();
+    if (!GROUPED && (args.pdl & 2)) griddep_launch_dependents();
     // weights do not depend on the previous kernel: the first tiles are requested before the wait
 #pragma unroll
     for (int s = 0; s < STAGES - 1; s++)
         if (s < nk) load_w(s, (kt0 + s) * kBK);
-    if (args.pdl & 1) griddep_wait();
+    if (wait) griddep_wait();
     const __nv_bfloat16 *a_src[MT];
     bool a_ok[MT];
 #pragma unroll
     for (int i = 0; i < MT; i++) {
         const int m = m0 + r16 + 16 * i;
         a_ok[i] = m < M;
-        a_src[i] = A + (size_t)(a_ok[i] ? (P.rowsel ? P.rowsel[m] : m) : 0) * lda;
+        a_src[i] = A + (size_t)(a_ok[i] ? (P.rowsel ? P.rowsel[m + src0] : m) : 0) * lda;
     }
     auto load_a = [&](int buf, int k0) {
 #pragma unroll
@@ -175,24 +192,24 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
 #pragma unroll
     for (int i = 0; i < PER; i++) {
         const int e = tid + 256 * i, m = m0 + e / kBN, c = e % kBN, n = n0 + c;
-        if (EPI == EPI_GATE_GELU) {
+        if (EPI == EPI_GATE) {
             // lanes 0-15 of a warp hold the gate of a row's 16 outputs, lanes 16-31 the linear part
             const float up = __shfl_down_sync(0xffffffffu, sum[i], 16);
             if ((c & 31) < 16 && m < M && n + 16 < N)
-                reinterpret_cast<__nv_bfloat16 *>(P.C)[(size_t)m * P.ldc + n / 32 * 16 + (c & 15)] = __float2bfloat16(gelu_tanh(sum[i]) * up);
+                reinterpret_cast<__nv_bfloat16 *>(P.C)[(size_t)m * P.ldc + n / 32 * 16 + (c & 15)] = __float2bfloat16(activate<true>(P.act, 0.f, 0.f, sum[i]) * up);
         } else if (m < M && n < n_end) {
             const size_t at = (size_t)m * P.ldc + n + cn;
-            if (EPI == EPI_STORE) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(sum[i]);
-            if (EPI == EPI_ACT) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(activate_fast(P.act, P.p0, P.p1, sum[i]));
-            if (EPI == EPI_ADD_F32) reinterpret_cast<float *>(P.C)[at] = P.res[at] + (P.colscale ? P.colscale[n] * sum[i] : sum[i]);
+            if (EPI == EPI_STORE) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(P.bias ? sum[i] + P.bias[n] : sum[i]);
+            if (EPI == EPI_ACT) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(activate<true>(P.act, P.p0, P.p1, sum[i]));
+            if (EPI == EPI_ADD_F32) reinterpret_cast<float *>(P.C)[at] = P.res_scale * P.res[at] + (P.colscale ? P.colscale[n] * sum[i] : sum[i]);
             if (EPI == EPI_SCALE_F32) reinterpret_cast<float *>(P.C)[at] = sum[i] * P.scale;
         }
     }
 }
 
-template <int MT, int NH, int STAGES, int EPI>
+template <int MT, int NH, int STAGES, int EPI, bool GROUPED>
 static int32_t small_launch(const SmallArgs &args, int total_tiles, int M, cudaStream_t st) {
-    auto kern = gemm_nt_small_kernel<MT, NH, STAGES, EPI>;
+    auto kern = gemm_nt_small_kernel<MT, NH, STAGES, EPI, GROUPED>;
     const size_t smem = small_smem<MT, NH, STAGES>(args.k_split);
     static thread_local int set_for = -1;  // the opt-in to more than 48 KiB, once per device
     int dev = 0;
@@ -214,32 +231,34 @@ static int32_t small_launch(const SmallArgs &args, int total_tiles, int M, cudaS
         attr[na].val.programmaticStreamSerializationAllowed = 1;
         na++;
     }
-    cfg.gridDim = dim3((unsigned)(total_tiles * args.k_split), (unsigned)((M + 16 * MT - 1) / (16 * MT)));
+    cfg.gridDim = dim3((unsigned)(total_tiles * args.k_split), GROUPED ? 1u : (unsigned)((M + 16 * MT - 1) / (16 * MT)));
     cfg.blockDim = dim3(256), cfg.dynamicSmemBytes = smem, cfg.stream = st, cfg.attrs = attr, cfg.numAttrs = (unsigned)na;
     JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, kern, args));
     return JGPT_OK;
 }
 
-template <int EPI>
+template <int EPI, bool GROUPED = false>
 static int32_t small_dispatch(const Ctx *ctx, const Problem *p, int n, int pdl, cudaStream_t st) {
     SmallArgs a{};
     a.n = n, a.pdl = pdl;
-    const int M = p[0].M, mt = M <= 16 ? 1 : (M <= 32 ? 2 : 4), bn = mt == 4 ? 64 : 32, max_split = mt == 4 ? 4 : kMaxSplit;
+    const int M = p[0].M, tall = GROUPED ? p[0].grp.rows : M;
+    const int mt = tall <= 16 ? 1 : (tall <= 32 ? 2 : 4), bn = mt == 4 ? 64 : 32, max_split = mt == 4 ? 4 : kMaxSplit;
     int tiles = 0, K = 0;
     for (int i = 0; i < n; i++) {
         a.p[i] = p[i];
         a.per_seg[i] = (p[i].seg_n + bn - 1) / bn, a.tiles[i] = p[i].segments() * a.per_seg[i];
+        if (GROUPED) a.tiles[i] *= i == 0 ? p[0].grp.max_tiles : (M + 16 * mt - 1) / (16 * mt);
         tiles += a.tiles[i];
         K = std::max(K, p[i].K);
     }
     const int ctas = tiles * ((M + 16 * mt - 1) / (16 * mt)), nk = (K + kBK - 1) / kBK;
     // split k while the launch leaves SMs idle and every part keeps two tiles
     a.k_split = 1;
-    while (n == 1 && a.k_split < max_split && ctas * a.k_split * 2 <= 2 * ctx->sm_count && nk / (a.k_split * 2) >= 2) a.k_split *= 2;
+    while (n == 1 && !GROUPED && a.k_split < max_split && ctas * a.k_split * 2 <= 2 * ctx->sm_count && nk / (a.k_split * 2) >= 2) a.k_split *= 2;
     switch (mt) {
-        case 1: return small_launch<1, 1, 6, EPI>(a, tiles, M, st);
-        case 2: return small_launch<2, 1, 5, EPI>(a, tiles, M, st);
-        default: return small_launch<4, 2, 3, EPI>(a, tiles, M, st);
+        case 1: return small_launch<1, 1, 6, EPI, GROUPED>(a, tiles, M, st);
+        case 2: return small_launch<2, 1, 5, EPI, GROUPED>(a, tiles, M, st);
+        default: return small_launch<4, 2, 3, EPI, GROUPED>(a, tiles, M, st);
     }
 }
 
@@ -248,32 +267,46 @@ int umma_min_rows() {
     return v;
 }
 
+int group_tile_rows(bool f32, int rows, int copies, int groups) {
+    if (f32) return 64;
+    if (umma_min_rows() > 0 && rows >= umma_min_rows()) return 128;
+    const int mean = (rows * copies + groups - 1) / groups;
+    return mean <= 8 ? 16 : (mean <= 16 ? 32 : 64);
+}
+
 // Defaults spelled out: one segment, the residual in C itself.
-static int32_t complete(const Problem *p, int n, Problem (&q)[2]) {
+static int32_t complete(const Problem *p, int n, Epilogue epi, Problem (&q)[2]) {
     JGPT_REQUIRE(n >= 1 && n <= 2 && p[0].M > 0, JGPT_ERR_INVALID_ARGUMENT, "1 or 2 products per launch");
     for (int i = 0; i < n; i++) {
         q[i] = p[i];
         if (q[i].seg_n <= 0) q[i].seg_n = q[i].N;
         if (!q[i].res) q[i].res = reinterpret_cast<const float *>(q[i].C);
+        JGPT_REQUIRE(!q[i].grp.tiles || (i == 0 && (epi == EPI_STORE || epi == EPI_ACT) && q[i].segments() == 1 && q[i].grp.max_tiles > 0),
+                     JGPT_ERR_INVALID_ARGUMENT, "rows in groups: the first product of a launch, one segment, stored or activated");
     }
     return JGPT_OK;
 }
 
 int32_t launch_bf16(const Ctx *ctx, const Problem *problems, int n, Epilogue epi, int pdl, cudaStream_t st) {
     Problem p[2];
-    if (int32_t rc = complete(problems, n, p)) return rc;
+    if (int32_t rc = complete(problems, n, epi, p)) return rc;
     bool big = p[0].M >= umma_min_rows() && umma_min_rows() > 0;
-    for (int i = 0; i < n; i++) big = big && !p[i].rowsel;
+    for (int i = 0; i < n; i++) big = big && (!p[i].rowsel || p[i].grp.tiles);
+    if (p[0].grp.tiles) {
+        const int rows = p[0].grp.rows;
+        JGPT_REQUIRE(big ? rows == 128 : (rows == 16 || rows == 32 || rows == 64), JGPT_ERR_INVALID_ARGUMENT, "row tiles of %d", rows);
+        if (!big) return epi == EPI_ACT ? small_dispatch<EPI_ACT, true>(ctx, p, n, pdl, st) : small_dispatch<EPI_STORE, true>(ctx, p, n, pdl, st);
+    }
     if (big) {
         for (int i = 0; i < n; i++)
-            if (int32_t rc = launch_bf16_umma(ctx, p[i], epi, i == 0 ? pdl : 0, st)) return rc;
+            if (int32_t rc = launch_bf16_umma(ctx, p[i], epi, pdl, st)) return rc;
         return JGPT_OK;
     }
     switch (epi) {
         case EPI_STORE: return small_dispatch<EPI_STORE>(ctx, p, n, pdl, st);
         case EPI_ADD_F32: return small_dispatch<EPI_ADD_F32>(ctx, p, n, pdl, st);
         case EPI_SCALE_F32: return small_dispatch<EPI_SCALE_F32>(ctx, p, n, pdl, st);
-        case EPI_GATE_GELU: return small_dispatch<EPI_GATE_GELU>(ctx, p, n, pdl, st);
+        case EPI_GATE: return small_dispatch<EPI_GATE>(ctx, p, n, pdl, st);
         case EPI_ACT: return small_dispatch<EPI_ACT>(ctx, p, n, pdl, st);
     }
     return fail(JGPT_ERR_INVALID_ARGUMENT, "unknown epilogue");
@@ -289,15 +322,21 @@ __global__ void __launch_bounds__(256) gemm_nt_f32_kernel(const Problem P0, cons
     const Problem &P = blockIdx.z == 0 ? P0 : P1;
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
     const int per_seg = (P.seg_n + BT - 1) / BT, seg = blockIdx.x / per_seg, cn = seg * P.c_seg;
-    const int m0 = blockIdx.y * BT, n0 = seg * P.seg_n + blockIdx.x % per_seg * BT, n_end = min(P.N, (seg + 1) * P.seg_n);
+    const int n0 = seg * P.seg_n + blockIdx.x % per_seg * BT, n_end = min(P.N, (seg + 1) * P.seg_n);
     if (n0 >= P.N) return;
     const float *__restrict__ A = reinterpret_cast<const float *>(P.A) + seg * P.a_seg;
     const float *__restrict__ W = reinterpret_cast<const float *>(P.W);
+    int m0 = blockIdx.y * BT, m_end = P.M, src0 = 0;
+    if (P.grp.tiles) {
+        if ((int)blockIdx.y >= *P.grp.n_tiles) return;
+        const RowTile t = P.grp.tiles[blockIdx.y];
+        m0 = t.row0, m_end = t.row_end, src0 = t.src0 - t.row0, W += t.group * P.grp.w_group;
+    }
     float acc[4][4] = {};
     for (int k0 = 0; k0 < P.K; k0 += BK) {
         for (int e = tid; e < BT * BK; e += 256) {
             const int r = e / BK, k = k0 + e % BK, m = m0 + r, n = n0 + r;
-            As[e % BK][r] = (m < P.M && k < P.K) ? A[(size_t)(P.rowsel ? P.rowsel[m] : m) * P.lda + k] : 0.f;
+            As[e % BK][r] = (m < m_end && k < P.K) ? A[(size_t)(P.rowsel ? P.rowsel[m + src0] : m) * P.lda + k] : 0.f;
             Ws[e % BK][r] = (n < n_end && k < P.K) ? W[(size_t)n * P.ldw + k] : 0.f;
         }
         __syncthreads();
@@ -317,12 +356,12 @@ __global__ void __launch_bounds__(256) gemm_nt_f32_kernel(const Problem P0, cons
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         const int m = m0 + ty * 4 + i;
-        if (m >= P.M) continue;
-        if (EPI == EPI_GATE_GELU) {  // columns tx (+ 32) of a group of 32 are the gate, tx + 16 the linear part
+        if (m >= m_end) continue;
+        if (EPI == EPI_GATE) {  // columns tx (+ 32) of a group of 32 are the gate, tx + 16 the linear part
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
                 const int n = n0 + tx + 16 * j;
-                if (n + 16 < P.N) C[(size_t)m * P.ldc + n / 32 * 16 + tx] = gelu_tanh(acc[i][j]) * acc[i][j + 1];
+                if (n + 16 < P.N) C[(size_t)m * P.ldc + n / 32 * 16 + tx] = activate<false>(P.act, 0.f, 0.f, acc[i][j]) * acc[i][j + 1];
             }
         } else {
 #pragma unroll
@@ -330,9 +369,9 @@ __global__ void __launch_bounds__(256) gemm_nt_f32_kernel(const Problem P0, cons
                 const int n = n0 + tx + 16 * j;
                 if (n >= n_end) continue;
                 const size_t at = (size_t)m * P.ldc + n + cn;
-                if (EPI == EPI_STORE) C[at] = acc[i][j];
-                if (EPI == EPI_ACT) C[at] = activate(P.act, P.p0, P.p1, acc[i][j]);
-                if (EPI == EPI_ADD_F32) C[at] = P.res[at] + (P.colscale ? P.colscale[n] * acc[i][j] : acc[i][j]);
+                if (EPI == EPI_STORE) C[at] = P.bias ? acc[i][j] + P.bias[n] : acc[i][j];
+                if (EPI == EPI_ACT) C[at] = activate<false>(P.act, P.p0, P.p1, acc[i][j]);
+                if (EPI == EPI_ADD_F32) C[at] = P.res_scale * P.res[at] + (P.colscale ? P.colscale[n] * acc[i][j] : acc[i][j]);
                 if (EPI == EPI_SCALE_F32) C[at] = acc[i][j] * P.scale;
             }
         }
@@ -341,15 +380,20 @@ __global__ void __launch_bounds__(256) gemm_nt_f32_kernel(const Problem P0, cons
 
 int32_t launch_f32(const Problem *problems, int n, Epilogue epi, cudaStream_t st) {
     Problem p[2];
-    if (int32_t rc = complete(problems, n, p)) return rc;
+    if (int32_t rc = complete(problems, n, epi, p)) return rc;
     const Problem &q = p[n - 1];
+    if (p[0].grp.tiles && n == 2) {
+        if (int32_t rc = launch_f32(p, 1, epi, st)) return rc;
+        return launch_f32(p + 1, 1, epi, st);
+    }
+    JGPT_REQUIRE(!p[0].grp.tiles || p[0].grp.rows <= 64, JGPT_ERR_INVALID_ARGUMENT, "row tiles of %d", p[0].grp.rows);
     auto tiles = [](const Problem &x) { return x.segments() * ((x.seg_n + 63) / 64); };
-    const dim3 grid((unsigned)std::max(tiles(p[0]), tiles(q)), (unsigned)((p[0].M + 63) / 64), (unsigned)n);
+    const dim3 grid((unsigned)std::max(tiles(p[0]), tiles(q)), (unsigned)(p[0].grp.tiles ? p[0].grp.max_tiles : (p[0].M + 63) / 64), (unsigned)n);
     switch (epi) {
         case EPI_STORE: gemm_nt_f32_kernel<EPI_STORE><<<grid, 256, 0, st>>>(p[0], q); break;
         case EPI_ADD_F32: gemm_nt_f32_kernel<EPI_ADD_F32><<<grid, 256, 0, st>>>(p[0], q); break;
         case EPI_SCALE_F32: gemm_nt_f32_kernel<EPI_SCALE_F32><<<grid, 256, 0, st>>>(p[0], q); break;
-        case EPI_GATE_GELU: gemm_nt_f32_kernel<EPI_GATE_GELU><<<grid, 256, 0, st>>>(p[0], q); break;
+        case EPI_GATE: gemm_nt_f32_kernel<EPI_GATE><<<grid, 256, 0, st>>>(p[0], q); break;
         case EPI_ACT: gemm_nt_f32_kernel<EPI_ACT><<<grid, 256, 0, st>>>(p[0], q); break;
     }
     JGPT_CUDA_TRY(cudaGetLastError());

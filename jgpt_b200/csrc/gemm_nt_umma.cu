@@ -8,6 +8,8 @@
 //
 // Persistent CTAs of 320 threads: warp 0 issues the copies, warp 1 owns the tensor memory and issues the MMAs, warps 2-9
 // drain the accumulator (TMEM lane quarter = warp % 4, half the tile's columns each) while the next tile is multiplied.
+// Rows in groups (experts): the device's list of row tiles takes the place of the row grid, the weight tile's rows shift by group,
+// and an operand with a row list comes in through gather copies, four rows each, one per lane of the copying warp.
 // Output tiles are walked in groups of eight row tiles, rows fastest, so CTAs side by side share weight tiles in L2.
 // Every wait is bounded; on expiry the status word gets DEV_STATUS_WAIT_TIMEOUT and the CTA winds down.
 #include <cuda.h>
@@ -47,19 +49,32 @@ __device__ __forceinline__ void tma_2d(void *smem_dst, const CUtensorMap *map, i
                  : "memory");
 }
 
+// Four rows of 64 elements; the map's box is one row.
+__device__ __forceinline__ void tma_gather4(void *smem_dst, const CUtensorMap *map, int x, const int (&y)[4], uint64_t *bar) {
+    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile::gather4.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4, %5, %6}], [%7];" ::"r"(
+                     smem_u32(smem_dst)),
+                 "l"(map), "r"(x), "r"(y[0]), "r"(y[1]), "r"(y[2]), "r"(y[3]), "r"(smem_u32(bar))
+                 : "memory");
+}
+
+enum RowMode : int { ROWS_ALL = 0, ROWS_GROUPS = 1, ROWS_GATHERED = 2 };
+
 struct UmmaArgs {
     void *C;
     int M, N, K, ldc, mt, nt, pdl;
     float scale;
     int *status;
     int per_seg, seg_n, c_seg, a_x, a_y;  // column tiles and columns of a segment; its shift in C; its operand's shift (columns, rows)
-    const float *res, *colscale;
+    const float *res, *colscale, *bias;
     int act;
-    float p0, p1;
+    float p0, p1, res_scale;
+    const RowTile *tiles;  // groups: the row tiles, how many, each group's rows of W, the operand's row list
+    const int *n_tiles, *rowsel;
+    int w_rows;
 };
 
-__device__ __forceinline__ void tile_of(const UmmaArgs &a, int t, int &m, int &n) {
-    const int per = kGroupM * a.nt, g = t / per, r = t % per, gm = min(kGroupM, a.mt - g * kGroupM);
+__device__ __forceinline__ void tile_of(const UmmaArgs &a, int mt, int t, int &m, int &n) {
+    const int per = kGroupM * a.nt, g = t / per, r = t % per, gm = min(kGroupM, mt - g * kGroupM);
     m = g * kGroupM + r % gm, n = r / gm;
 }
 
@@ -68,7 +83,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<const uint32_t *>(&v);
 }
 
-template <int BN, int EPI>
+template <int BN, int EPI, int ROWS>
 __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __grid_constant__ CUtensorMap amap, const __grid_constant__ CUtensorMap wmap,
                                                                        const UmmaArgs a) {
     constexpr int ST = stages<BN>();
@@ -80,7 +95,7 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
     __shared__ int s_abort_mem;
     volatile int *s_abort = &s_abort_mem;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int nk = (a.K + UK - 1) / UK, total = a.mt * a.nt;
+    const int nk = (a.K + UK - 1) / UK;
     uint8_t *tiles = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(umma_raw) + 1023) & ~(uintptr_t)1023);
 
     if (tid == 0) {
@@ -96,14 +111,50 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
     const uint32_t tmem = s_tmem;
     if (a.pdl & 2) griddep_launch_dependents();
     if (a.pdl & 1) griddep_wait();
+    const int mt = ROWS == ROWS_ALL ? a.mt : min(*a.n_tiles, a.mt), total = mt * a.nt;
 
     if (warp == 0) {
-        if (lane == 0) {
+        if (ROWS == ROWS_GATHERED) {
+            uint32_t it = 0;
+            for (int t = blockIdx.x; t < total; t += gridDim.x) {
+                int m, n, rows[4];
+                tile_of(a, mt, t, m, n);
+                const RowTile rt = a.tiles[m];
+#pragma unroll
+                for (int i = 0; i < 4; i++) rows[i] = a.rowsel[rt.src0 + (rt.row0 + 4 * lane + i < rt.row_end ? 4 * lane + i : 0)];
+                bool ok = true;
+                for (int kt = 0; kt < nk; kt++, it++) {
+                    const uint32_t s = it % ST, use = it / ST;
+                    int free = 1;
+                    uint8_t *dst = tiles + (size_t)s * SB;
+                    if (lane == 0) {
+                        if (use > 0) free = mbar_wait_bounded(&empty_bar[s], (use - 1) & 1u, a.status, s_abort);
+                        if (free) {
+                            mbar_expect_tx(&full_bar[s], SB);
+                            tma_2d(dst + A_BYTES, &wmap, kt * UK, rt.group * a.w_rows + n * BN, &full_bar[s]);
+                        }
+                    }
+                    if (!__shfl_sync(0xffffffffu, free, 0)) {
+                        ok = false;
+                        break;
+                    }
+                    tma_gather4(dst + lane * 4 * UK * 2, &amap, kt * UK, rows, &full_bar[s]);
+                }
+                if (!ok) break;
+            }
+            if (*s_abort && lane == 0) {
+                for (uint32_t k = it > (uint32_t)ST ? it - ST : 0; k < it; k++)
+                    for (uint32_t i = 0; i < (1u << 16) && !mbar_try_wait(&full_bar[k % ST], (k / ST) & 1u); i++) {
+                    }
+            }
+        } else if (lane == 0) {
             uint32_t it = 0;
             for (int t = blockIdx.x; t < total && !*s_abort; t += gridDim.x) {
                 int m, n;
-                tile_of(a, t, m, n);
-                const int seg = n / a.per_seg, ax = seg * a.a_x, ay = seg * a.a_y + m * UM, wy = seg * a.seg_n + n % a.per_seg * BN;
+                tile_of(a, mt, t, m, n);
+                const int seg = n / a.per_seg, ax = seg * a.a_x;
+                int ay = seg * a.a_y + m * UM, wy = seg * a.seg_n + n % a.per_seg * BN;
+                if (ROWS != ROWS_ALL) ay = a.tiles[m].row0, wy += a.tiles[m].group * a.w_rows;
                 for (int kt = 0; kt < nk; kt++, it++) {
                     const uint32_t s = it % ST, use = it / ST;
                     if (use > 0 && !mbar_wait_bounded(&empty_bar[s], (use - 1) & 1u, a.status, s_abort)) break;
@@ -150,8 +201,9 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
         for (int t = blockIdx.x; t < total; t += gridDim.x, j++) {
             const uint32_t buf = j & 1u, round = j >> 1, acc = tmem + buf * BN;
             int mi, ni;
-            tile_of(a, t, mi, ni);
-            const int seg = ni / a.per_seg, m = mi * UM + quarter * 32 + lane, n0 = seg * a.seg_n + ni % a.per_seg * BN;
+            tile_of(a, mt, t, mi, ni);
+            const int row0 = ROWS == ROWS_ALL ? mi * UM : a.tiles[mi].row0, m_end = ROWS == ROWS_ALL ? a.M : a.tiles[mi].row_end;
+            const int seg = ni / a.per_seg, m = row0 + quarter * 32 + lane, n0 = seg * a.seg_n + ni % a.per_seg * BN;
             const int n_end = min(a.N, (seg + 1) * a.seg_n), cn = seg * a.c_seg;
             int ok = 0;
             if (lane == 0) ok = mbar_wait_bounded(&acc_full[buf], round & 1u, a.status, s_abort) ? 1 : 0;
@@ -163,7 +215,7 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
                 if (n0 + c0 >= n_end) break;  // uniform across the warp
                 float v[32];
                 load_acc32(acc, quarter, c0, v);
-                if (m >= a.M) continue;
+                if (m >= m_end) continue;
                 if (EPI == EPI_STORE || EPI == EPI_ACT) {
                     __nv_bfloat16 *c = reinterpret_cast<__nv_bfloat16 *>(a.C) + (size_t)m * a.ldc + n0 + c0 + cn;
                     if (EPI == EPI_ACT && a.act == ACT_XIELU) {
@@ -172,16 +224,32 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
                     } else if (EPI == EPI_ACT && a.act == ACT_TANH) {
 #pragma unroll
                         for (int q = 0; q < 32; q++) v[q] = tanhf(v[q]);
+                    } else if (EPI == EPI_ACT && a.act == ACT_RELU2) {
+#pragma unroll
+                        for (int q = 0; q < 32; q++) v[q] = fmaxf(v[q], 0.f), v[q] *= v[q];
+                    } else if (EPI == EPI_ACT) {
+#pragma unroll
+                        for (int q = 0; q < 32; q++) v[q] = activate<true>(a.act, a.p0, a.p1, v[q]);
+                    }
+                    if (EPI == EPI_STORE && a.bias) {
+#pragma unroll
+                        for (int q = 0; q < 32; q++)
+                            if (n0 + c0 + q < n_end) v[q] += __ldg(a.bias + n0 + c0 + q);
                     }
 #pragma unroll
                     for (int q = 0; q < 4; q++)
                         if (n0 + c0 + 8 * q < n_end)  // N and seg_n are multiples of 8 here
                             *reinterpret_cast<uint4 *>(c + 8 * q) = make_uint4(pack_bf16(v[8 * q], v[8 * q + 1]), pack_bf16(v[8 * q + 2], v[8 * q + 3]),
                                                                                pack_bf16(v[8 * q + 4], v[8 * q + 5]), pack_bf16(v[8 * q + 6], v[8 * q + 7]));
-                } else if (EPI == EPI_GATE_GELU) {
+                } else if (EPI == EPI_GATE) {
                     __nv_bfloat16 *c = reinterpret_cast<__nv_bfloat16 *>(a.C) + (size_t)m * a.ldc + (n0 + c0) / 2;
+                    if (a.act == ACT_RELU) {
 #pragma unroll
-                    for (int q = 0; q < 16; q++) v[q] = gelu_tanh(v[q]) * v[16 + q];
+                        for (int q = 0; q < 16; q++) v[q] = fmaxf(v[q], 0.f) * v[16 + q];
+                    } else {
+#pragma unroll
+                        for (int q = 0; q < 16; q++) v[q] = gelu_tanh(v[q]) * v[16 + q];
+                    }
 #pragma unroll
                     for (int q = 0; q < 2; q++)
                         *reinterpret_cast<uint4 *>(c + 8 * q) = make_uint4(pack_bf16(v[8 * q], v[8 * q + 1]), pack_bf16(v[8 * q + 2], v[8 * q + 3]),
@@ -203,14 +271,14 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
                         if (vec4 && n + 3 < n_end) {
                             if (EPI == EPI_ADD_F32) {
                                 const float4 r = *reinterpret_cast<const float4 *>(res + 4 * q);
-                                o.x += r.x, o.y += r.y, o.z += r.z, o.w += r.w;
+                                o.x = fmaf(a.res_scale, r.x, o.x), o.y = fmaf(a.res_scale, r.y, o.y), o.z = fmaf(a.res_scale, r.z, o.z), o.w = fmaf(a.res_scale, r.w, o.w);
                             }
                             *reinterpret_cast<float4 *>(c + 4 * q) = o;
                         } else {
                             const float e[4] = {o.x, o.y, o.z, o.w};
 #pragma unroll
                             for (int i = 0; i < 4; i++)
-                                if (n + i < n_end) c[4 * q + i] = EPI == EPI_ADD_F32 ? res[4 * q + i] + e[i] : e[i];
+                                if (n + i < n_end) c[4 * q + i] = EPI == EPI_ADD_F32 ? fmaf(a.res_scale, res[4 * q + i], e[i]) : e[i];
                         }
                     }
                 }
@@ -252,16 +320,18 @@ static int32_t make_map(CUtensorMap *map, const void *base, int rows, int K, int
     return JGPT_OK;
 }
 
-template <int BN, int EPI>
+template <int BN, int EPI, int ROWS>
 static int32_t umma_launch(const Ctx *ctx, const Problem &p, int pdl, cudaStream_t st) {
     CUtensorMap am, wm;
     const int segs = p.segments(), ay = (int)(p.a_seg / p.lda), ax = (int)(p.a_seg % p.lda), per_seg = (p.segment_cols() + BN - 1) / BN;
-    int32_t rc = make_map(&am, p.A, p.M + (segs - 1) * ay, p.K + (segs - 1) * ax, p.lda, UM);
-    if (!rc) rc = make_map(&wm, p.W, p.N, p.K, p.ldw, BN);
+    const int w_rows = ROWS == ROWS_ALL ? 0 : (int)(p.grp.w_group / p.ldw), mt = ROWS == ROWS_ALL ? (p.M + UM - 1) / UM : p.grp.max_tiles;
+    int32_t rc = make_map(&am, p.A, ROWS == ROWS_ALL ? p.M + (segs - 1) * ay : p.grp.a_rows, p.K + (segs - 1) * ax, p.lda, ROWS == ROWS_GATHERED ? 1 : UM);
+    if (!rc) rc = make_map(&wm, p.W, ROWS == ROWS_ALL ? p.N : (p.grp.n_groups - 1) * w_rows + p.N, p.K, p.ldw, BN);
     if (rc) return rc;
-    UmmaArgs a{p.C, p.M, p.N, p.K, p.ldc, (p.M + UM - 1) / UM, segs * per_seg, pdl, p.scale, ctx->d_status,
-               per_seg, p.segment_cols(), p.c_seg, ax, ay, p.res, p.colscale, p.act, p.p0, p.p1};
-    auto kern = gemm_nt_umma_kernel<BN, EPI>;
+    UmmaArgs a{p.C, p.M, p.N, p.K, p.ldc, mt, segs * per_seg, pdl, p.scale, ctx->d_status,
+               per_seg, p.segment_cols(), p.c_seg, ax, ay, p.res, p.colscale, p.bias, p.act, p.p0, p.p1, p.res_scale,
+               p.grp.tiles, p.grp.n_tiles, p.rowsel, w_rows};
+    auto kern = gemm_nt_umma_kernel<BN, EPI, ROWS>;
     static thread_local int set_for = -1;
     if (set_for != ctx->device) {
         JGPT_CUDA_TRY(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)umma_smem<BN>()));
@@ -277,29 +347,34 @@ static int32_t umma_launch(const Ctx *ctx, const Problem &p, int pdl, cudaStream
     return JGPT_OK;
 }
 
-template <int EPI>
+template <int EPI, int ROWS = ROWS_ALL>
 static int32_t umma_pick(const Ctx *ctx, const Problem &p, int pdl, cudaStream_t st) {
-    const int mt = (p.M + UM - 1) / UM;
+    const int mt = ROWS == ROWS_ALL ? (p.M + UM - 1) / UM : p.grp.max_tiles;
     auto tiles = [&](int bn) { return mt * p.segments() * ((p.segment_cols() + bn - 1) / bn); };
-    if (tiles(256) >= ctx->sm_count) return umma_launch<256, EPI>(ctx, p, pdl, st);
-    if (tiles(128) >= ctx->sm_count * 2 / 3) return umma_launch<128, EPI>(ctx, p, pdl, st);
-    return umma_launch<64, EPI>(ctx, p, pdl, st);
+    if (tiles(256) >= ctx->sm_count) return umma_launch<256, EPI, ROWS>(ctx, p, pdl, st);
+    if (tiles(128) >= ctx->sm_count * 2 / 3) return umma_launch<128, EPI, ROWS>(ctx, p, pdl, st);
+    return umma_launch<64, EPI, ROWS>(ctx, p, pdl, st);
 }
 
 int32_t launch_bf16_umma(const Ctx *ctx, const Problem &p, Epilogue epi, int pdl, cudaStream_t st) {
     JGPT_REQUIRE(p.lda % 8 == 0 && p.ldw % 8 == 0 && (reinterpret_cast<uintptr_t>(p.A) & 15) == 0 && (reinterpret_cast<uintptr_t>(p.W) & 15) == 0,
                  JGPT_ERR_INVALID_ARGUMENT, "operand rows must start on 16-byte boundaries");
-    JGPT_REQUIRE((epi != EPI_STORE || (p.N % 8 == 0 && p.ldc % 8 == 0)) && (epi != EPI_GATE_GELU || (p.N % 32 == 0 && p.ldc % 8 == 0)),
+    JGPT_REQUIRE((epi != EPI_STORE || (p.N % 8 == 0 && p.ldc % 8 == 0)) && (epi != EPI_GATE || ((p.act == ACT_GELU || p.act == ACT_RELU) && p.N % 32 == 0 && p.ldc % 8 == 0)),
                  JGPT_ERR_INVALID_ARGUMENT, "output columns %d, stride %d", p.N, p.ldc);
     JGPT_REQUIRE((epi != EPI_ACT || (p.N % 8 == 0 && p.ldc % 8 == 0)) &&
-                     (p.segments() == 1 || (p.seg_n % 8 == 0 && p.c_seg % 8 == 0 && p.a_seg % 8 == 0 && epi != EPI_GATE_GELU)),
+                     (p.segments() == 1 || (p.seg_n % 8 == 0 && p.c_seg % 8 == 0 && p.a_seg % 8 == 0 && epi != EPI_GATE)),
                  JGPT_ERR_INVALID_ARGUMENT, "segments of %d columns, shifts %lld / %d", p.seg_n, p.a_seg, p.c_seg);
+    if (p.grp.tiles) {
+        JGPT_REQUIRE(p.grp.n_groups > 0 && p.grp.a_rows > 0 && p.grp.w_group % p.ldw == 0, JGPT_ERR_INVALID_ARGUMENT, "groups of rows");
+        if (epi == EPI_ACT) return p.rowsel ? umma_pick<EPI_ACT, ROWS_GATHERED>(ctx, p, pdl, st) : umma_pick<EPI_ACT, ROWS_GROUPS>(ctx, p, pdl, st);
+        return p.rowsel ? umma_pick<EPI_STORE, ROWS_GATHERED>(ctx, p, pdl, st) : umma_pick<EPI_STORE, ROWS_GROUPS>(ctx, p, pdl, st);
+    }
     switch (epi) {
         case EPI_ACT: return umma_pick<EPI_ACT>(ctx, p, pdl, st);
         case EPI_STORE: return umma_pick<EPI_STORE>(ctx, p, pdl, st);
         case EPI_ADD_F32: return umma_pick<EPI_ADD_F32>(ctx, p, pdl, st);
         case EPI_SCALE_F32: return umma_pick<EPI_SCALE_F32>(ctx, p, pdl, st);
-        case EPI_GATE_GELU: return umma_pick<EPI_GATE_GELU>(ctx, p, pdl, st);
+        case EPI_GATE: return umma_pick<EPI_GATE>(ctx, p, pdl, st);
     }
     return fail(JGPT_ERR_INVALID_ARGUMENT, "unknown epilogue");
 }

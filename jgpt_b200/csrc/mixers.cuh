@@ -5,6 +5,7 @@
 #include <cuda_bf16.h>
 
 #include "common.cuh"
+#include "gemm_nt.cuh"
 
 namespace jgpt {
 namespace mix {
@@ -49,7 +50,7 @@ int32_t launch_layer_norm(bool f32, const float *x, const int *rowsel, NormW w, 
 
 // A row of the residual stream: the embedding of the row's token, or the weighted sum of the earlier layers' results
 // (a plain residual is the sum over one slot without weights).
-constexpr int kMaxRotations = 4;
+constexpr int kMaxRotations = 16;
 struct Rotation {        // cos and sin of every row's angles, [rows][half] pairs, times mag
     const double *freq;
     float2 *out;
@@ -75,27 +76,71 @@ struct ShiftArgs {
     uint64_t state_stride;
     int max_seqs;
 };
-// x[r] = source (when x is set), h[r] = x[r] / rms * gamma, as mixes when sh has them; rowsel picks rows (null: all).
+// x[r] = source (when x is set), h[r] = x[r] / rms * gamma (x[r] itself without gamma), as mixes when sh has them; rowsel picks
+// rows (null: all).
 int32_t launch_residual_norm(bool f32, const StepDesc &d, const RowSource &src, const int *rowsel, int rows, const float *gamma, float eps, float *x,
                              void *h, const ShiftArgs &sh, int W, int ldh, int *status, int pdl, cudaStream_t st);
 
+// The norm behind a sum: x[r] = S[r] / rms * gamma and h[r] = x[r], S = x itself, or with a mixture of experts
+// S[r] = (alpha + weight of the identity experts) x[r] + sum of weight_s out[row of slot s] + shared gate * shared[r].
+struct RouteSlot {
+    int expert, rank;  // expert < 0: none; its row of the experts' products is offsets[expert] + rank
+    float weight;
+};
+struct MoeSum {
+    const void *out, *shared;  // [.., ld] activations; out null: no mixture; shared null: no shared expert
+    int ld, top, cap;
+    const RouteSlot *slots;    // [rows][top]
+    const float2 *row_weights; // [rows]: identity experts, shared gate
+    const int *offsets;
+    float alpha;
+};
+int32_t launch_post_norm(bool f32, float *x, int rows, const float *gamma, float eps, void *h, const MoeSum &m, int W, int ldh, int pdl, cudaStream_t st);
+
+// ---- moe.cu ------------------------------------------------------------------------------------------
+struct RouteArgs {
+    const float *logits;       // [rows, ld]: experts, identity experts, the shared expert's gate (when shared is set)
+    int ld, experts, identity, top, groups, keep, shared;
+    const float *correction;   // [experts + identity]
+    RouteSlot *slots;
+    float2 *row_weights;
+    int *list, *counts, *offsets, *ticket;  // rows of every expert [experts][cap]; counts and ticket are zero between launches
+    int cap;
+    nt::RowTile *tiles;
+    int *n_tiles;
+    int max_tiles, tile_rows;
+};
+int32_t launch_route(const RouteArgs &a, int rows, int pdl, cudaStream_t st);
+
 // ---- attn_gqa.cu -----------------------------------------------------------------------------------
+// Query heads in groups that share a key head.  Differential attention has two maps: a head's query and key are [map 1 | map 2],
+// each map is an attention of its own over the same values, the second one's result times lambda is taken off the first one's
+// and the difference brought to unit root mean square.  Padded sizes: DK per map, DV.
+enum HeadGate : int { GATE_NONE = 0, GATE_HEAD = 1, GATE_ELEMENT = 2 };
 struct AttnArgs {
-    const void *proj;   // [rows, ldp] projections of the layer
-    int ldp, q_off, k_off, v_off, g_off;  // column offsets; g_off < 0: no output gate
-    int heads, kv_heads, D;  // query heads, key heads, padded head size (q, k and v alike)
+    void *proj;         // [rows, ldp] projections of the layer
+    int ldp, q_off, k_off, v_off, g_off;  // column offsets
+    int heads, kv_heads, maps, DK, DV, dim, vdim;
+    int gate;           // HeadGate: sigmoid of one column per head, or of a column per element of the output
     int chunk;          // a query sees the keys of its own chunk of this many positions (0: all earlier positions)
     float scale, out_scale;
-    void *kv;           // this layer's pages: [block][kv head][K 16 x D | V 16 x D]
+    const float *q_norm, *k_norm;  // weights of the RMS norm of every query and key head (map); null: none
+    float eps;
+    const float2 *cs;   // [rows][half] cos and sin; the first 2 half elements of every head (map) turn; null: no rotation
+    int half, interleaved;         // pairs (2 i, 2 i + 1), or (i, i + half)
+    float lambda, diff_scale;
+    void *kv;           // this layer's pages: [block][kv head][K 16 x (maps DK) | V 16 x DV]
     const int *table;
     int n_blocks, mbs;
-    void *out;          // [rows, ldo], head h at out_off + h * D
+    void *out;          // [rows, ldo], head h at out_off + h * DV
     int ldo, out_off;
     int sm_count;
     int *status;
+    __host__ __device__ bool prepared() const { return q_norm || cs; }  // heads are normed or rotated on their way
+    __host__ __device__ int page_head() const { return kBlockTokens * (maps * DK + DV); }
 };
 int32_t launch_attention(bool f32, const StepDesc &d, const AttnArgs &a, int pdl, cudaStream_t st);
-int attn_padded_head(int dim, int vdim);          // 0: not supported
+bool attn_padded_head(int dim, int vdim, int maps, int *DK, int *DV);  // false: not supported
 int attn_query_tile(int heads, int kv_heads);     // tokens per query tile of the multi-token kernel
 
 // ---- recurrent.cu ----------------------------------------------------------------------------------

@@ -198,7 +198,7 @@ __global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const StepD
     }
     if (!h) return;
     if (!sh.mu[0]) {
-        for (int j = threadIdx.x; j < ldh; j += kNormThreads) store_act(h + (size_t)r * ldh + j, j < W ? row[j] * inv * gamma[j] : 0.f);
+        for (int j = threadIdx.x; j < ldh; j += kNormThreads) store_act(h + (size_t)r * ldh + j, j < W ? (gamma ? row[j] * inv * gamma[j] : row[j]) : 0.f);
         return;
     }
     // the row before: recomputed the same way inside an entry, read from the state in front of it
@@ -236,6 +236,99 @@ int32_t launch_residual_norm(bool f32, const StepDesc &d, const RowSource &s, co
     if (f32) return s.embed ? run(residual_norm_kernel<float, true>, (float *)nullptr) : run(residual_norm_kernel<float, false>, (float *)nullptr);
     return s.embed ? run(residual_norm_kernel<__nv_bfloat16, true>, (__nv_bfloat16 *)nullptr)
                    : run(residual_norm_kernel<__nv_bfloat16, false>, (__nv_bfloat16 *)nullptr);
+}
+
+// ------------------------------------------------------------------------------------------------
+// RMS norm behind a sum
+// ------------------------------------------------------------------------------------------------
+__device__ __forceinline__ float4 load4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16 *p) {
+    const uint2 u = *reinterpret_cast<const uint2 *>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16 *p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+}
+__device__ __forceinline__ void add_scaled(float4 &s, float w, const float4 &v) {
+    s.x = fmaf(w, v.x, s.x), s.y = fmaf(w, v.y, s.y), s.z = fmaf(w, v.z, s.z), s.w = fmaf(w, v.w, s.w);
+}
+
+constexpr int kMaxTop = 32;
+
+template <class AT, bool MOE>
+__global__ void __launch_bounds__(kNormThreads) post_norm_kernel(float *__restrict__ x, const float *__restrict__ gamma, float eps, AT *__restrict__ h, const MoeSum m,
+                                                                 int W, int ldh, int pdl) {
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[kNormThreads / 32], weight[kMaxTop];
+    __shared__ long long from[kMaxTop];
+    const int r = blockIdx.x, tid = threadIdx.x;
+    if (pdl & 2) griddep_launch_dependents();
+    if (pdl & 1) griddep_wait();
+    float *xr = x + (size_t)r * W;
+    const AT *out = reinterpret_cast<const AT *>(m.out), *shared = reinterpret_cast<const AT *>(m.shared) + (size_t)r * m.ld;
+    float keep = 1.f, gate = 0.f;
+    if (MOE) {
+        if (tid < m.top) {
+            const RouteSlot s = m.slots[(size_t)r * m.top + tid];
+            const bool ok = s.expert >= 0 && s.rank >= 0 && s.rank < m.cap;
+            weight[tid] = ok ? s.weight : 0.f, from[tid] = ok ? (long long)(m.offsets[s.expert] + s.rank) * m.ld : -1;
+        }
+        const float2 w = m.row_weights[r];
+        keep = m.alpha + w.x, gate = w.y;
+        __syncthreads();
+    }
+    float q = 0.f;
+    if ((W & 3) == 0) {
+        for (int j = tid * 4; j < W; j += kNormThreads * 4) {
+            float4 v = load4(xr + j);
+            if (MOE) {
+                v.x *= keep, v.y *= keep, v.z *= keep, v.w *= keep;
+#pragma unroll 8
+                for (int s = 0; s < m.top; s++)
+                    if (from[s] >= 0) add_scaled(v, weight[s], load4(out + from[s] + j));
+                if (m.shared) add_scaled(v, gate, load4(shared + j));
+            }
+            store4(row + j, v);
+            q += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+    } else {
+        for (int j = tid; j < W; j += kNormThreads) {
+            float v = xr[j];
+            if (MOE) {
+                v *= keep;
+                for (int s = 0; s < m.top; s++)
+                    if (from[s] >= 0) v = fmaf(weight[s], load_act(out + from[s] + j), v);
+                if (m.shared) v = fmaf(gate, load_act(shared + j), v);
+            }
+            row[j] = v, q += v * v;
+        }
+    }
+    const float inv = 1.f / sqrtf(block_sum(q, red) / (float)W + eps);
+    AT *hr = h + (size_t)r * ldh;
+    if ((W & 3) == 0) {
+        for (int j = tid * 4; j < W; j += kNormThreads * 4) {
+            const float4 v = load4(row + j), g = load4(gamma + j), y = make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w);
+            store4(xr + j, y), store4(hr + j, y);
+        }
+        for (int j = W + tid; j < ldh; j += kNormThreads) store_act(hr + j, 0.f);
+        return;
+    }
+    for (int j = tid; j < ldh; j += kNormThreads) {
+        const float y = j < W ? row[j] * inv * gamma[j] : 0.f;
+        if (j < W) xr[j] = y;
+        store_act(hr + j, y);
+    }
+}
+
+int32_t launch_post_norm(bool f32, float *x, int rows, const float *gamma, float eps, void *h, const MoeSum &m, int W, int ldh, int pdl, cudaStream_t st) {
+    const size_t smem = sizeof(float) * (size_t)((W + 3) / 4 * 4);
+    JGPT_REQUIRE(smem <= 47 * 1024 && m.top <= kMaxTop, JGPT_ERR_UNSUPPORTED, "width %d, %d experts per token", W, m.top);
+    auto run = [&](auto kern, auto *act) { return launch(kern, rows, smem, pdl, st, x, gamma, eps, (decltype(act))h, (const MoeSum)m, W, ldh, pdl); };
+    if (f32) return m.out ? run(post_norm_kernel<float, true>, (float *)nullptr) : run(post_norm_kernel<float, false>, (float *)nullptr);
+    return m.out ? run(post_norm_kernel<__nv_bfloat16, true>, (__nv_bfloat16 *)nullptr) : run(post_norm_kernel<__nv_bfloat16, false>, (__nv_bfloat16 *)nullptr);
 }
 
 }  // namespace mix

@@ -17,7 +17,9 @@ from .runtime import Context
 
 MIX_ATTENTION, MIX_GLA, MIX_DELTA, MIX_HGRN2, MIX_WKV, MIX_LATENT = range(1, 7)
 NORM_LAYER, NORM_RMS = 0, 1
-FF_GATED_GELU, FF_XIELU = 0, 1
+FF_GATED_GELU, FF_XIELU, FF_GATED_RELU, FF_MOE = range(4)
+ACT_RELU, ACT_RELU2, ACT_GELU_TANH = range(3)
+GATE_NONE, GATE_HEAD, GATE_ELEMENT = range(3)
 NO_LIMIT = 1 << 30  # positions of a model without a table of them
 DTYPES = {"bfloat16": 0, "float32": 1}
 BLOCK_TOKENS = 16
@@ -27,17 +29,23 @@ class _MixerSpec(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("kind", "heads", "kv_heads", "dim", "vdim", "chunk", "gate", "taps", "rank_a", "rank_g")] + \
                [(n, C.c_float) for n in ("score_scale", "tau", "out_scale")] + \
                [(n, C.c_int32) for n in ("window", "q_rank", "kv_rank", "rot_dim", "rot_dims", "kv_from")] + \
-               [(n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")]
+               [(n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")] + \
+               [(n, C.c_int32) for n in ("rot_interleaved", "qkv_bias", "qk_norm", "maps")] + [("diff", C.c_float)]
+
+
+class _MoeSpec(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("experts", "identity", "top", "groups", "keep", "ff", "shared_ff", "act", "shared_act")]
 
 
 class _LayerSpec(C.Structure):
-    _fields_ = [("n_branches", C.c_int32), ("branch", _MixerSpec * 2), ("ff", C.c_int32), ("ff_kind", C.c_int32)]
+    _fields_ = [("n_branches", C.c_int32), ("branch", _MixerSpec * 2), ("ff", C.c_int32), ("ff_kind", C.c_int32), ("moe", _MoeSpec)]
 
 
 class _DecoderSpec(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("vocab", "width", "max_positions", "n_layers", "embed_norm", "pos_table", "norm", "head", "layer_scale",
                                            "depth_average")] + \
-               [(n, C.c_float) for n in ("eps", "embed_scale", "logit_scale", "residual_mult")]
+               [(n, C.c_float) for n in ("eps", "embed_scale", "logit_scale", "residual_mult")] + \
+               [("norm_after", C.c_int32), ("residual_scale", C.c_float)]
 
 
 # tensor roles (JGPT_W_* of the header)
@@ -45,7 +53,9 @@ W_EMBED, W_POS, W_EMBED_NORM, W_EMBED_NORM_B, W_FINAL_NORM, W_FINAL_NORM_B, W_HE
 W_NORM1, W_NORM1_B, W_NORM2, W_NORM2_B, W_FF_GATE, W_FF_UP, W_FF_DOWN, W_LS1, W_LS2, W_DWA = range(10, 20)
 (W_Q, W_K, W_V, W_O, W_G, W_B, W_A1, W_A2, W_DECAY_BIAS, W_A_LOG, W_G1, W_G2, W_HEAD_NORM, W_CONV_Q, W_CONV_K,
  W_CONV_V, W_MU_R, W_MU_K, W_MU_V, W_MU_G, W_MU_W, W_BONUS, W_LOWER, W_F, W_DQ, W_DQ_NORM, W_UQ, W_DKV, W_DKV_NORM, W_UK, W_UV,
- W_FF_ACT) = range(20, 52)
+ W_FF_ACT, W_Q_BIAS, W_K_BIAS, W_V_BIAS, W_Q_NORM, W_K_NORM, W_LQ1, W_LK1, W_LQ2, W_LK2) = range(20, 61)
+W_ROUTER, W_CORRECTION, W_SHARED_GATE, W_SHARED_UP, W_SHARED_DOWN, W_EXPERT_UP, W_EXPERT_DOWN = range(64, 71)
+MAX_BRANCHES = 2
 
 
 @dataclass
@@ -56,7 +66,7 @@ class Mixer:
     dim: int
     vdim: int
     chunk: int = 0
-    gate: bool = False
+    gate: int = GATE_NONE
     taps: int = 0
     rank_a: int = 0
     rank_g: int = 0
@@ -74,7 +84,27 @@ class Mixer:
     rot_original: float = 0.0
     rot_fast: float = 0.0
     rot_slow: float = 0.0
+    rot_interleaved: bool = False
+    qkv_bias: bool = False
+    qk_norm: bool = False
+    maps: int = 1  # 2: differential, the second map's output times lambda is taken off the first one's
+    diff: float = 0.0
     tensors: dict = field(default_factory=dict)  # role -> tensor name
+
+
+@dataclass
+class Moe:
+    """Experts W_down act(W_up h): the last ``identity`` router outputs hand h on, a shared expert runs for every token."""
+    experts: int
+    top: int
+    ff: int
+    identity: int = 0
+    groups: int = 1
+    keep: int = 1
+    shared_ff: int = 0
+    act: int = ACT_RELU2
+    shared_act: int = ACT_RELU2
+    tensors: list = field(default_factory=list)  # per expert: role -> tensor name
 
 
 @dataclass
@@ -83,6 +113,7 @@ class Layer:
     ff: int = 0
     tensors: dict = field(default_factory=dict)
     ff_kind: int = FF_GATED_GELU
+    moe: Moe | None = None
 
 
 @dataclass
@@ -101,6 +132,8 @@ class DecoderConfig:
     layer_scale: bool = False
     depth_average: bool = False
     residual_mult: float = 1.0
+    norm_after: bool = False
+    residual_scale: float = 1.0
     tensors: dict = field(default_factory=dict)
 
     def all_tensors(self):
@@ -113,6 +146,9 @@ class DecoderConfig:
             for j, m in enumerate(layer.branches):
                 for role, name in m.tensors.items():
                     yield i, j, role, name
+            for e, names in enumerate(layer.moe.tensors if layer.moe else ()):
+                for role, name in names.items():
+                    yield i, MAX_BRANCHES + e, role, name
 
 
 class DecoderModel:
@@ -128,8 +164,11 @@ class DecoderModel:
                 raise ValueError(f"a layer has one or two mixer branches, not {len(layer.branches)}")
             spec.n_branches, spec.ff, spec.ff_kind = len(layer.branches), layer.ff, layer.ff_kind
             for b, m in zip(spec.branch, layer.branches):
-                for n, _ in _MixerSpec._fields_:
-                    setattr(b, n, int(m.gate) if n == "gate" else getattr(m, n))
+                for n, t in _MixerSpec._fields_:
+                    setattr(b, n, int(getattr(m, n)) if t is C.c_int32 else getattr(m, n))
+            if layer.moe:
+                for n, _ in _MoeSpec._fields_:
+                    setattr(spec.moe, n, getattr(layer.moe, n))
         top = _DecoderSpec(n_layers=len(config.layers))
         for n, t in _DecoderSpec._fields_:
             if n != "n_layers":

@@ -45,13 +45,19 @@ def load_model(ctx, folder, dtype="bfloat16", max_rows=2048) -> D.DecoderModel:
         w.close()
 
 
+def _rotation(rot):
+    yarn = rot.get("scaling")
+    return {"rot_dims": rot["dims"], "rot_base": rot["base"],
+            **({"rot_" + k: yarn[k] for k in ("factor", "original", "fast", "slow")} if yarn else {})}
+
+
 # ---- Somopel -------------------------------------------------------------------------------------------
 def _norm(names, role, name):
     names[role], names[role + 1] = name, name + ".b"
 
 
 def _attention(m, p, shape_of, out_scale):
-    return D.Mixer(D.MIX_ATTENTION, m["heads"], m["kv_heads"], m["dim"], m["vdim"], chunk=m["mask"]["size"], gate=True,
+    return D.Mixer(D.MIX_ATTENTION, m["heads"], m["kv_heads"], m["dim"], m["vdim"], chunk=m["mask"]["size"], gate=D.GATE_HEAD,
                    score_scale=m["scale"], out_scale=out_scale,
                    tensors={D.W_Q: p + "q", D.W_K: p + "k", D.W_V: p + "v", D.W_G: p + "g", D.W_O: p + "o"})
 
@@ -113,14 +119,13 @@ def _wkv(m, p, shape_of):
 
 
 def _latent(m, p):
-    rot, names = m["rot"], {D.W_DQ: p + "dq", D.W_DQ_NORM: p + "dq.norm", D.W_UQ: p + "uq", D.W_UK: p + "uk", D.W_UV: p + "uv", D.W_O: p + "o"}
+    names = {D.W_DQ: p + "dq", D.W_DQ_NORM: p + "dq.norm", D.W_UQ: p + "uq", D.W_UK: p + "uk", D.W_UV: p + "uv", D.W_O: p + "o"}
     shared = m.get("kv_from")
     if shared is None:
         names.update({D.W_DKV: p + "dkv", D.W_DKV_NORM: p + "dkv.norm"})
-    yarn = rot.get("scaling")
     return D.Mixer(D.MIX_LATENT, m["heads"], m["heads"], m["dim"], m["vdim"], window=(m.get("mask") or {}).get("size", 0), q_rank=m["q_rank"],
-                   kv_rank=m["kv_rank"], rot_dim=m["rot_dim"], rot_dims=rot["dims"], kv_from=0 if shared is None else 1 + shared, score_scale=m["scale"],
-                   rot_base=rot["base"], **({"rot_" + k: yarn[k] for k in ("factor", "original", "fast", "slow")} if yarn else {}), tensors=names)
+                   kv_rank=m["kv_rank"], rot_dim=m["rot_dim"], kv_from=0 if shared is None else 1 + shared, score_scale=m["scale"],
+                   **_rotation(m["rot"]), tensors=names)
 
 
 @register("Zusepel")
@@ -148,3 +153,58 @@ def zusepel(c, shape_of) -> D.DecoderConfig:
     names = {D.W_EMBED: "embed", D.W_FINAL_NORM: "final.norm", D.W_HEAD: "head"}
     return D.DecoderConfig(c["vocab"], c["width"], D.NO_LIMIT, c["norm"]["eps"], layers, pos_table=False, norm=D.NORM_RMS, head=True, layer_scale=True,
                            depth_average=True, residual_mult=c["residual_mult"], tensors=names)
+
+
+# ---- Nefipel -------------------------------------------------------------------------------------------
+def _gated_heads(m, p):
+    return D.Mixer(D.MIX_ATTENTION, m["heads"], m["kv_heads"], m["dim"], m["vdim"], gate=D.GATE_ELEMENT, score_scale=m["scale"], qkv_bias=True,
+                   qk_norm=True, **_rotation(m["rot"]),
+                   tensors={D.W_Q: p + "q", D.W_K: p + "k", D.W_V: p + "v", D.W_Q_BIAS: p + "q.b", D.W_K_BIAS: p + "k.b", D.W_V_BIAS: p + "v.b",
+                            D.W_Q_NORM: p + "q.norm", D.W_K_NORM: p + "k.norm", D.W_G: p + "g", D.W_O: p + "o"})
+
+
+def _differential(m, p):
+    return D.Mixer(D.MIX_ATTENTION, m["heads"], m["kv_heads"], m["dim"], m["vdim"], score_scale=m["scale"], qk_norm=True, rot_interleaved=True,
+                   maps=2, diff=m["diff"], **_rotation(m["rot"]),
+                   tensors={D.W_Q: p + "q", D.W_K: p + "k", D.W_V: p + "v", D.W_Q_NORM: p + "q.norm", D.W_K_NORM: p + "k.norm", D.W_LQ1: p + "lq1",
+                            D.W_LK1: p + "lk1", D.W_LQ2: p + "lq2", D.W_LK2: p + "lk2", D.W_O: p + "o"})
+
+
+def _mixture(mlp, p, names):
+    r, shared, groups = mlp["router"], mlp.get("shared"), mlp["router"].get("groups") or {}
+    names.update({D.W_ROUTER: p + "router", D.W_CORRECTION: p + "correction"})
+    if shared:
+        names.update({D.W_SHARED_GATE: p + "shared.sg", D.W_SHARED_UP: p + "shared.up", D.W_SHARED_DOWN: p + "shared.down"})
+    return D.Moe(r["experts"], r["top"], mlp["expert"]["ff"], identity=r.get("identity", 0), groups=groups.get("count", 1), keep=groups.get("keep", 1),
+                 shared_ff=shared["ff"] if shared else 0,
+                 tensors=[{D.W_EXPERT_UP: f"{p}e{e}.up", D.W_EXPERT_DOWN: f"{p}e{e}.down"} for e in range(r["experts"])])
+
+
+@register("Nefipel")
+def nefipel(c, shape_of) -> D.DecoderConfig:
+    """Layers of two kinds in any order: 'attention' (normed, rotated heads with biases, a gate per element of the output) and
+    'attention_2' (two maps per head, the second taken off the first); norms behind the sums; dense gated-relu parts and
+    mixtures of experts with identity experts and a gated shared expert; tied logits."""
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        p, m, mlp = f"l{i}.", e["mixer"], e["mlp"]
+        names, ff, kind, moe = {D.W_NORM1: p + "norm1"}, 0, D.FF_GATED_RELU, None
+        if e["type"] == "attention":
+            mixer = _gated_heads(m, p + "mix.")
+        elif e["type"] == "attention_2":
+            mixer = _differential(m, p + "mix.")
+        else:
+            raise ValueError(f"layer {i}: mixer type {e['type']!r}")
+        if mlp is not None:
+            names[D.W_NORM2] = p + "norm2"
+            if mlp["kind"] == "dense":
+                ff = mlp["ff"]
+                names.update({D.W_FF_GATE: p + "mlp.gate", D.W_FF_UP: p + "mlp.up", D.W_FF_DOWN: p + "mlp.down"})
+            elif mlp["kind"] == "moe":
+                kind, ff, moe = D.FF_MOE, mlp["expert"]["ff"], _mixture(mlp, p + "mlp.", names)
+            else:
+                raise ValueError(f"layer {i}: feed-forward kind {mlp['kind']!r}")
+        layers.append(D.Layer([mixer], ff, names, kind, moe))
+    return D.DecoderConfig(c["vocab"], c["width"], D.NO_LIMIT, c["norm"]["eps"], layers, pos_table=False, norm=D.NORM_RMS,
+                           embed_scale=c["embedding"]["scale"], norm_after=True, residual_scale=c["postln_alpha"],
+                           tensors={D.W_EMBED: "embed", D.W_FINAL_NORM: "final.norm"})
