@@ -1,4 +1,4 @@
-"""Prefill and decode throughput of the layered designs (Zusepel, Somopel; random weights) beside the fixed-block GPT model at
+"""Prefill and decode throughput of the layered designs (Nefipel, Zusepel, Somopel; random weights) beside the fixed-block GPT model at
 equal width, depth, feed-forward parameters and vocabulary: ``bench.py --workload decoder``."""
 from __future__ import annotations
 
@@ -73,6 +73,10 @@ def _random_model(ctx, cfg, shapes, max_rows, seed=0):
             return 0.5 + 0.1 * np.tanh(x)
         if n.endswith(".w0"):
             return x - 4
+        if n.endswith(".correction"):
+            return 0.005 * x
+        if n.endswith((".q.b", ".k.b", ".v.b", ".lq1", ".lk1", ".lq2", ".lk2")):
+            return 0.1 * x
         return x / np.sqrt(s[1]) if len(s) == 2 else 1 + 0.1 * x
     model = D.DecoderModel(ctx, registry.describe(cfg, shapes.__getitem__), "bfloat16", max_rows)
     model.loadTensors(get)
@@ -113,6 +117,44 @@ def random_zusepel(ctx, width, max_rows, rank=64):
             v = m["vdim"]
             new.update({"mix.q": (H * d, width), "mix.f": (H * d, width), "mix.f.b": (H * d,), "mix.lower": (H * d,), "mix.v": (H * v, width), "mix.norm": (v,),
                         "mix.o": (width, H * v)})
+        shapes.update({p + n: s for n, s in new.items()})
+    return _random_model(ctx, cfg, shapes, max_rows)
+
+
+def nefipel_config(width):
+    """Heads of 128 in groups of four, then two maps of 64 over values of 128; dense gated parts in every other layer, else 60
+    experts and 4 identity experts, 8 of them a token, and a shared one: as many multiplications a token as a dense part has."""
+    h = width // 128
+    att = {"heads": h, "kv_heads": max(h // 4, 1), "dim": 128, "vdim": 128, "rot": {"base": 10000.0, "dims": 64}, "scale": 128 ** -0.5}
+    yarn = {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    diff = {"heads": h, "kv_heads": max(h // 4, 1), "dim": 64, "vdim": 128, "rot": {"base": 10000.0, "dims": 64, "scaling": yarn}, "scale": 0.125, "diff": 0.5}
+    moe = {"kind": "moe", "expert": {"ff": width * 3 // 8}, "shared": {"ff": width * 9 // 8},
+           "router": {"experts": 60, "identity": 4, "top": 8, "groups": {"count": 8, "keep": 4}}}
+    block = [{"type": "attention", "mixer": att, "mlp": {"kind": "dense", "ff": width * 11 // 4}}, {"type": "attention_2", "mixer": diff, "mlp": moe}]
+    return {"architecture": "Nefipel", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6}, "postln_alpha": 2.5, "embedding": {"scale": 16.0},
+            "layers": block * (LAYERS // 2)}
+
+
+def random_nefipel(ctx, width, max_rows):
+    cfg = nefipel_config(width)
+    shapes = {"embed": (VOCAB, width), "final.norm": (width,)}
+    for i, e in enumerate(cfg["layers"]):
+        p, m, mlp = f"l{i}.", e["mixer"], e["mlp"]
+        H, G, d, v, maps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], 2 if e["type"] == "attention_2" else 1
+        new = {"norm1": (width,), "norm2": (width,), "mix.q": (H * maps * d, width), "mix.k": (G * maps * d, width), "mix.v": (G * v, width),
+               "mix.o": (width, H * v), "mix.q.norm": (d,), "mix.k.norm": (d,)}
+        if maps == 1:
+            new.update({"mix.q.b": (H * d,), "mix.k.b": (G * d,), "mix.v.b": (G * v,), "mix.g": (H * v, width)})
+        else:
+            new.update({"mix." + n: (d,) for n in ("lq1", "lk1", "lq2", "lk2")})
+        if mlp["kind"] == "dense":
+            new.update({"mlp.gate": (mlp["ff"], width), "mlp.up": (mlp["ff"], width), "mlp.down": (width, mlp["ff"])})
+        else:
+            n, f, s = mlp["router"]["experts"], mlp["expert"]["ff"], mlp["shared"]["ff"]
+            new.update({"mlp.router": (n + mlp["router"]["identity"], width), "mlp.correction": (n + mlp["router"]["identity"],), "mlp.shared.sg": (1, width),
+                        "mlp.shared.up": (s, width), "mlp.shared.down": (width, s)})
+            for k in range(n):
+                new.update({f"mlp.e{k}.up": (f, width), f"mlp.e{k}.down": (width, f)})
         shapes.update({p + n: s for n, s in new.items()})
     return _random_model(ctx, cfg, shapes, max_rows)
 
@@ -175,12 +217,12 @@ def _prefill(ctx, model, batch, seq_len, repeats):
     return float(np.median(best))
 
 
-def run_decoder(ctx, widths=(1024, 2048), batches=(1, 16, 64), prompts=((1, 2048), (8, 1024)), ctx_len=1500, steps=24, repeats=5, models=("zusepel", "somopel", "gpt")):
+def run_decoder(ctx, widths=(1024, 2048), batches=(1, 16, 64), prompts=((1, 2048), (8, 1024)), ctx_len=1500, steps=24, repeats=5, models=("nefipel", "zusepel", "somopel", "gpt")):
     out = {"workload": f"{LAYERS} layers, vocabulary {VOCAB}, random weights; prefill = prompts of one call, decode at context {ctx_len}+",
            "timing": "prefill: CUDA events around the call; decode: host clock around a step that reads its ids back; medians", "sizes": []}
     for w in widths:
         row = {"width": w}
-        for name, make in (("zusepel", random_zusepel), ("somopel", random_somopel), ("gpt", random_gpt)):
+        for name, make in (("nefipel", random_nefipel), ("zusepel", random_zusepel), ("somopel", random_somopel), ("gpt", random_gpt)):
             if name not in models:
                 continue
             m = make(ctx, w, 8192)

@@ -98,17 +98,32 @@ def expert(h, up, down):
     return linear(relu(linear(h, up)) ** 2, down)
 
 
+def open_groups(choice, r):
+    """Which outputs may be chosen: those of the groups whose best choice score is among the largest."""
+    g = r.get("groups") or {"count": 1, "keep": 1}
+    size = choice.size // g["count"]
+    best = np.argsort(-choice.reshape(g["count"], size).max(1), kind="stable")[:g["keep"]]
+    return np.isin(np.arange(choice.size) // size, best)
+
+
 def route(z, correction, r):
     """One token: router logits -> [(expert, weight)]; the correction takes part in the choice only."""
     s = np.exp(z - z.max())
     s = s / s.sum()
-    choice, n = s + correction, z.size
-    g = r.get("groups") or {"count": 1, "keep": 1}
-    size = n // g["count"]
-    best = np.argsort(-choice.reshape(g["count"], size).max(1), kind="stable")[:g["keep"]]
-    open_ = np.isin(np.arange(n) // size, best)
-    chosen = np.argsort(-np.where(open_, choice, -np.inf), kind="stable")[:r["top"]]
+    choice = s + correction
+    chosen = np.argsort(-np.where(open_groups(choice, r), choice, -np.inf), kind="stable")[:r["top"]]
     return [(int(e), s[e] / (s[chosen].sum() + 1e-20)) for e in chosen]
+
+
+def route_margin(z, correction, r):
+    """How far one choice score is from changing what is chosen."""
+    s = np.exp(z - z.max())
+    choice = s / s.sum() + correction
+    ok, g = open_groups(choice, r), r.get("groups") or {"count": 1, "keep": 1}
+    inside, best = -np.sort(-choice[ok]), -np.sort(-choice.reshape(g["count"], -1).max(1))
+    gaps = [inside[r["top"] - 1] - inside[r["top"]]] if inside.size > r["top"] else []
+    gaps += [best[g["keep"] - 1] - best[g["keep"]]] if g["keep"] < g["count"] else []
+    return min(gaps, default=np.inf)
 
 
 def mixture(h, W, mlp):
