@@ -2,10 +2,11 @@
 // the kernels are built for), all earlier positions or those of the query's chunk, optional norms and rotation of the heads,
 // one or two maps per head (mixers.cuh), an optional output gate per head or per element.
 //
-//   attn_prep_kernel     query heads normed and rotated in place, keys likewise and values into the pages
+//   attn_prep_kernel     keys (normed and rotated) and values into the pages; in the exact mode query heads in place
 //   attn_rows_kernel     one warp per (row, head), fp32: the exact mode
-//   attn_tile_kernel     portions of prompts, bf16 tensor cores
-//   attn_single_kernel   single tokens, bf16 tensor cores over a split sequence, with the preparation of its own heads
+//   attn_tile_kernel     portions of prompts, bf16 tensor cores; prepares its query heads
+//   attn_single_kernel   single tokens, bf16 tensor cores over a split sequence; prepares its query heads, and its key unless
+//                        attn_prep_kernel has done so
 #include "mixers.cuh"
 
 #include <algorithm>
@@ -19,82 +20,97 @@ __host__ __device__ __forceinline__ int first_visible(int pos, int chunk) { retu
 
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 
-// A head (map) of a row in the 8-element pieces of `lanes` neighbouring lanes (a power of two; every lane of the warp takes
-// part): norm over its dim elements, rotation.  buf: 8 floats per lane of the group.
-__device__ __forceinline__ void prepare_head(float (&x)[8], int piece, int lanes, int dim, const float *w, float eps, const float2 *cs, int half,
-                                             int interleaved, float *buf) {
+// What happens to a query or key head (map) behind its projection: norm, rotation.
+struct HeadPrep {
+    const float *w;  // null: no norm
+    const float2 *cs;
+    int dim, half, interleaved;
+    float eps;
+};
+__device__ __forceinline__ HeadPrep head_prep(const AttnArgs &a, bool key, int row) {
+    return HeadPrep{key ? a.k_norm : a.q_norm, a.cs + (size_t)row * a.half, a.dim, a.half, a.interleaved, a.eps};
+}
+// The head lies in 8-element pieces in `lanes` neighbouring lanes (a power of two; every lane of the warp takes part); src: its
+// start in memory.
+template <class AT>
+__device__ __forceinline__ void prepare_head(float (&x)[8], const AT *src, int piece, int lanes, const HeadPrep &h) {
     const int j0 = piece * 8;
-    if (w) {
+    float inv = 1.f;
+    if (h.w) {
         float ss = 0.f;
 #pragma unroll
         for (int e = 0; e < 8; e++) ss += x[e] * x[e];
         for (int off = lanes >> 1; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
-        const float inv = 1.f / sqrtf(ss / (float)dim + eps);
+        inv = 1.f / sqrtf(ss / (float)h.dim + h.eps);
 #pragma unroll
-        for (int e = 0; e < 8; e++) x[e] = j0 + e < dim ? x[e] * inv * __ldg(w + j0 + e) : 0.f;
+        for (int e = 0; e < 8; e++) x[e] = j0 + e < h.dim ? x[e] * inv * __ldg(h.w + j0 + e) : 0.f;
     }
-    if (!half) return;
-    if (interleaved) {
+    if (!h.half) return;
+    if (h.interleaved) {
 #pragma unroll
         for (int e = 0; e < 8; e += 2)
-            if (j0 + e < 2 * half) {
-                const float2 t = __ldg(cs + ((j0 + e) >> 1));
+            if (j0 + e < 2 * h.half) {
+                const float2 t = __ldg(h.cs + ((j0 + e) >> 1));
                 const float u = x[e], v = x[e + 1];
                 x[e] = u * t.x - v * t.y, x[e + 1] = v * t.x + u * t.y;
             }
-        return;
-    }
+    } else if ((h.half & 7) == 0) {  // the other element of a pair is in the same place of another lane
+        const int hp = h.half >> 3, lane = threadIdx.x & 31;
+        const bool first = piece < hp, turns = piece < 2 * hp;
+        const int other = turns ? (first ? lane + hp : lane - hp) : lane;
 #pragma unroll
-    for (int e = 0; e < 8; e++) buf[j0 + e] = x[e];
-    __syncwarp();
+        for (int e = 0; e < 8; e++) {
+            const float y = __shfl_sync(0xffffffffu, x[e], other);
+            if (!turns) continue;
+            const float2 t = __ldg(h.cs + (first ? j0 + e : j0 + e - h.half));
+            x[e] = first ? x[e] * t.x - y * t.y : x[e] * t.x + y * t.y;
+        }
+    } else {
 #pragma unroll
-    for (int e = 0; e < 8; e++) {
-        const int j = j0 + e;
-        if (j >= 2 * half) continue;
-        const float2 t = __ldg(cs + (j < half ? j : j - half));
-        x[e] = j < half ? x[e] * t.x - buf[j + half] * t.y : x[e] * t.x + buf[j - half] * t.y;
+        for (int e = 0; e < 8; e++) {
+            const int j = j0 + e, p = j < h.half ? j + h.half : j - h.half;
+            if (j >= 2 * h.half) continue;
+            const float2 t = __ldg(h.cs + (j < h.half ? j : p));
+            const float y = act_load(src + p) * inv * (h.w ? __ldg(h.w + p) : 1.f);
+            x[e] = j < h.half ? x[e] * t.x - y * t.y : x[e] * t.x + y * t.y;
+        }
+        __syncwarp();  // whoever writes the head back does so after this
     }
-    __syncwarp();
 }
-__host__ __device__ __forceinline__ int head_lanes(int DK) { return DK <= 32 ? 4 : (DK <= 64 ? 8 : (DK <= 128 ? 16 : 32)); }
+__host__ __device__ constexpr int head_lanes(int DK) { return DK <= 32 ? 4 : (DK <= 64 ? 8 : (DK <= 128 ? 16 : 32)); }
 
-// Vectors of a row: its query maps (when they are prepared), key maps, values; a vector per head_lanes(DK) lanes.
+// A block (or several, in y) per row: its query maps (with `queries`, in place), key maps and values (into the page), a vector per
+// head_lanes(DK) lanes.
 template <class AT>
-__global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a, const int *__restrict__ seq, const int *__restrict__ pos, int rows, int pdl) {
-    __shared__ float bufs[256 * 8];
+__global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a, const int *__restrict__ seq, const int *__restrict__ pos, int queries, int pdl) {
     if (pdl & 2) griddep_launch_dependents();
-    const int lanes = head_lanes(a.DK), nq = a.prepared() ? a.heads * a.maps : 0, nk = a.kv_heads * a.maps, nv = nq + nk + a.kv_heads;
-    const long long item = ((long long)blockIdx.x * 256 + threadIdx.x) / lanes;
-    const bool ok = item < (long long)rows * nv;
-    const int r = ok ? (int)(item / nv) : 0, i = ok ? (int)(item % nv) : 0, piece = threadIdx.x & (lanes - 1);
+    const int lanes = head_lanes(a.DK), nq = queries ? a.heads * a.maps : 0, nk = a.kv_heads * a.maps, nv = nq + nk + a.kv_heads;
+    const int r = blockIdx.x, i = (blockIdx.y * blockDim.x + threadIdx.x) / lanes, piece = threadIdx.x & (lanes - 1);
+    const int p = pos[r], row = p % kBlockTokens, phys = page_of(a, seq[r], p), kw = a.maps * a.DK;
     if (pdl & 1) griddep_wait();
     AT *proj = reinterpret_cast<AT *>(a.proj) + (size_t)r * a.ldp;
-    const int p = pos[r];
-    AT *page = nullptr;
-    if (i >= nq) {
-        const int phys = page_of(a, seq[r], p), g = i < nq + nk ? (i - nq) / a.maps : i - nq - nk;
-        if (phys >= 0) page = reinterpret_cast<AT *>(a.kv) + ((size_t)phys * a.kv_heads + g) * a.page_head();
+    const bool query = i < nq, value = i >= nq + nk && i < nv, key = i >= nq && i < nq + nk;
+    const int g = key ? (i - nq) / a.maps : (value ? i - nq - nk : 0);
+    AT *page = reinterpret_cast<AT *>(a.kv) + ((size_t)max(phys, 0) * a.kv_heads + g) * a.page_head();
+    if (value && phys >= 0) {
+        AT *dst = page + kBlockTokens * page_row(kw) + row * page_row(a.DV);
+        for (int c = piece; c < a.DV / 8; c += lanes) {
+            float x[8];
+            load8(proj + a.v_off + g * a.DV + c * 8, x), store8(dst + page_chunk(a.DV, row, c) * 8, x);
+        }
     }
-    const bool value = i >= nq + nk, mine = ok && (i < nq || page);
-    if (value && mine) {
-        const AT *src = proj + a.v_off + (i - nq - nk) * a.DV;
-        AT *dst = page + kBlockTokens * a.maps * a.DK + (size_t)(p % kBlockTokens) * a.DV;
-        constexpr int E = 16 / sizeof(AT);
-        for (int c = piece * E; c < a.DV; c += lanes * E) *reinterpret_cast<uint4 *>(dst + c) = *reinterpret_cast<const uint4 *>(src + c);
-    }
+    const AT *src = proj + (query ? a.q_off + i * a.DK : a.k_off + (key ? i - nq : 0) * a.DK);
     float x[8];
-    AT *src = proj + (i < nq ? a.q_off + i * a.DK : a.k_off + (i - nq) * a.DK) + piece * 8;
-    const bool load = mine && !value && piece * 8 < a.DK;
-    if (load) load8(src, x);
+    const bool load = (query || key) && piece * 8 < a.DK;
+    if (load) load8(src + piece * 8, x);
     else {
 #pragma unroll
         for (int e = 0; e < 8; e++) x[e] = 0.f;
     }
-    if (a.prepared())
-        prepare_head(x, piece, lanes, a.dim, i < nq ? a.q_norm : a.k_norm, a.eps, a.cs + (size_t)r * a.half, a.half, a.interleaved, bufs + (threadIdx.x - piece) * 8);
+    if (a.prepared()) prepare_head(x, src, piece, lanes, head_prep(a, !query, r));
     if (!load) return;
-    if (i < nq) store8(src, x);
-    else store8(page + (size_t)(p % kBlockTokens) * a.maps * a.DK + (i - nq) % a.maps * a.DK + piece * 8, x);
+    if (query) store8(proj + a.q_off + i * a.DK + piece * 8, x);
+    else if (phys >= 0) store8(page + row * page_row(kw) + page_chunk(kw, row, (i - nq) % a.maps * (a.DK / 8) + piece) * 8, x);
 }
 
 // One warp per (row, query head): lane l holds elements l, l + 32, ... of q and of the output.
@@ -115,20 +131,21 @@ __global__ void __launch_bounds__(256) attn_rows_kernel(const AttnArgs a, const 
         for (int j = first_visible(p, a.chunk); j <= p; j++) {
             const int phys = page_of(a, s, j);
             if (phys < 0) break;
-            const AT *k = reinterpret_cast<const AT *>(a.kv) + ((size_t)phys * a.kv_heads + g) * a.page_head();
-            const AT *v = k + kBlockTokens * kw + (size_t)(j % kBlockTokens) * a.DV + lane;
-            k += (size_t)(j % kBlockTokens) * kw + map * a.DK + lane;
+            const int row = j % kBlockTokens;
+            const AT *k = reinterpret_cast<const AT *>(a.kv) + ((size_t)phys * a.kv_heads + g) * a.page_head() + row * page_row(kw);
+            const AT *v = k + kBlockTokens * page_row(kw) + row * (page_row(a.DV) - page_row(kw));
+            auto at = [&](int D, int e) { return page_chunk(D, row, e >> 3) * 8 + (e & 7); };
             float d = 0.f;
 #pragma unroll
             for (int e = 0; e < MAXE; e++)
-                if (e < nk) d = fmaf(q[e], act_load(k + 32 * e), d);
+                if (e < nk) d = fmaf(q[e], act_load(k + at(kw, map * a.DK + lane + 32 * e)), d);
 #pragma unroll
             for (int off = 16; off >= 1; off >>= 1) d += __shfl_xor_sync(0xffffffffu, d, off);
             const float mn = fmaxf(m, d), fo = expf(m - mn), w = expf(d - mn);
             m = mn, l = l * fo + w;
 #pragma unroll
             for (int e = 0; e < MAXE; e++)
-                if (e < nv) o[e] = fmaf(w, act_load(v + 32 * e), o[e] * fo);
+                if (e < nv) o[e] = fmaf(w, act_load(v + at(a.DV, lane + 32 * e)), o[e] * fo);
         }
         f = l > 0.f ? 1.f / l : 0.f;
     }
@@ -163,53 +180,121 @@ __device__ __forceinline__ const __nv_bfloat16 *gate_at(const AttnArgs &a, int r
     return reinterpret_cast<const __nv_bfloat16 *>(a.proj) + (size_t)row * a.ldp + a.g_off + h * a.DV + c;
 }
 
-// Entries with several tokens (queries are prepared, K / V in the pages).  CTA = 64 rows of one key head: 4 warps x 16 rows for
-// each map; tiles of 64 keys through two stages.  The second map's warps hand their rows over in shared memory.
-constexpr int kTileKeys = 64;
+// Pages of a key head: 16 rows of K (all maps), 16 of V.
+template <int KW, int DV>
+struct Page {
+    static constexpr int LK = page_row(KW), LV = page_row(DV), ELEMS = 16 * (LK + LV);
+    static constexpr uint32_t BYTES = ELEMS * 2;
+    template <class T>
+    __device__ static T *k(T *page, int row, int chunk) { return page + row * LK + page_chunk(KW, row, chunk) * 8; }
+    template <class T>
+    __device__ static T *v(T *page, int row, int chunk) { return page + 16 * LK + row * LV + page_chunk(DV, row, chunk) * 8; }
+    // values of rows that nobody has written: a weight of zero does not hide what is not a number
+    __device__ static void clear_values(__nv_bfloat16 *page, int from, int lane) {
+        for (int e = from * (LV / 8) + lane; e < 16 * (LV / 8); e += 32) reinterpret_cast<uint4 *>(page + 16 * LK)[e] = make_uint4(0, 0, 0, 0);
+    }
+};
+
+// Entries with several tokens (K / V are in the pages).  CTA = 64 rows of one key head (32 with two maps): four warps of 16 rows of
+// one map, prepared on their way in; a fifth warp brings in tiles of KT keys, a bulk copy per page.  The second map's warps hand
+// their rows over in shared memory.
 template <int DK, int DV, int MAPS>
-__host__ __device__ constexpr size_t tile_smem() { return (size_t)2 * (MAPS * 64 * (DK + 8) + 2 * kTileKeys * (MAPS * (DK + 8) + DV + 8)); }
+struct Tile {
+    using P = Page<MAPS * DK, DV>;
+    static constexpr int KT = 64, ST = 2, PAGES = KT / 16, LQ = DK + 8, ROWS = 64 / MAPS, BLOCKS = DV <= 128 ? 2 : 1;
+    static constexpr size_t stage_elems = (size_t)PAGES * P::ELEMS, ring = ST * stage_elems * 2, hand = MAPS == 2 ? (size_t)ROWS * (DV + 8) * 4 : 0;
+    static constexpr size_t smem = (ring > hand ? ring : hand) + (size_t)64 * LQ * 2;
+};
 
 template <int DK, int DV, int MAPS>
-__global__ void __launch_bounds__(128 * MAPS) attn_tile_kernel(const AttnArgs a, const Seg *__restrict__ segs, const int2 *__restrict__ tiles, int qt, int pdl) {
-    constexpr int LK = DK + 8, LV = DV + 8, CK = DK / 8, CV = DV / 8, NT = 128 * MAPS, STAGE = kTileKeys * (MAPS * LK + LV), KW = MAPS * DK;
-    extern __shared__ __align__(16) uint8_t attn_smem[];
-    __nv_bfloat16 *qs = reinterpret_cast<__nv_bfloat16 *>(attn_smem), *kv_s = qs + MAPS * 64 * LK;  // stages: [K 64 x LK] per map, [V 64 x LV]
-    const int tid = threadIdx.x, lane = tid & 31, g = lane >> 2, map = tid / 128, warp = (tid % 128) >> 5;
-    const int grp = a.heads / a.kv_heads, kvh = blockIdx.y, r0 = blockIdx.z * 64;
+__global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_kernel(const AttnArgs a, const Seg *__restrict__ segs, const int2 *__restrict__ tiles, int qt, int pdl) {
+    using T = Tile<DK, DV, MAPS>;
+    using P = typename T::P;
+    constexpr int LQ = T::LQ, KT = T::KT, ST = T::ST, PAGES = T::PAGES, NC = 128, LV = DV + 8, ROWS = T::ROWS;
+    extern __shared__ __align__(128) uint8_t attn_smem[];
+    __nv_bfloat16 *ring = reinterpret_cast<__nv_bfloat16 *>(attn_smem);  // stages of PAGES pages
+    __nv_bfloat16 *qs = reinterpret_cast<__nv_bfloat16 *>(attn_smem + T::smem) - 64 * LQ;
+    __shared__ __align__(8) uint64_t full[ST], empty[ST];
+    __shared__ int s_abort_mem;
+    volatile int *s_abort = &s_abort_mem;
+    const int tid = threadIdx.x, lane = tid & 31, g = lane >> 2, wid = tid >> 5, map = wid / (ROWS / 16), warp = wid % (ROWS / 16);
+    const int grp = a.heads / a.kv_heads, kvh = blockIdx.y, r0 = blockIdx.z * ROWS;
     if (pdl & 2) griddep_launch_dependents();
     const int2 tile = tiles[gridDim.x - 1 - blockIdx.x];  // the last tiles of a prompt see most keys
     const Seg sg = segs[tile.x];
     const int nt = min(qt, sg.T - tile.y), rows = nt * grp, row_base = sg.row0 + tile.y;
     if (r0 >= rows) return;
-    const int p0 = sg.pos0 + tile.y, p1 = sg.pos0 + tile.y + (min(rows, r0 + 64) - 1) / grp;
-    const __nv_bfloat16 *proj = reinterpret_cast<const __nv_bfloat16 *>(a.proj);
-    const __nv_bfloat16 *kv = reinterpret_cast<const __nv_bfloat16 *>(a.kv);
-    if (pdl & 1) griddep_wait();
-    for (int e = tid; e < MAPS * 64 * CK; e += NT) {
-        const int m = e / (64 * CK), r = r0 + e / CK % 64, c = e % CK;
-        const bool ok = r < rows;
-        const int t = ok ? r / grp : 0, h = kvh * grp + (ok ? r % grp : 0);
-        cp_async16(qs + (e / CK) * LK + c * 8, proj + (size_t)(row_base + t) * a.ldp + a.q_off + (h * MAPS + m) * DK + c * 8, ok);
+    const int p0 = sg.pos0 + tile.y, b0 = p0 + r0 / grp, p1 = p0 + (min(rows, r0 + ROWS) - 1) / grp;  // positions: of the tile, of the block's rows
+    const int first = first_visible(b0, a.chunk) / kBlockTokens * kBlockTokens, n_tiles = (p1 - first) / KT + 1;
+    if (tid == 0) {
+        for (int s = 0; s < ST; s++) mbar_init(&full[s], 1), mbar_init(&empty[s], NC / 32);
+        *s_abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
-    const int first = first_visible(p0 + r0 / grp, a.chunk) / kBlockTokens * kBlockTokens;
-    auto load = [&](int stage, int kb) {
-        __nv_bfloat16 *dst = kv_s + (size_t)stage * STAGE;
-        for (int e = tid; e < kTileKeys * (MAPS * CK + CV); e += NT) {
-            const int j = e / (MAPS * CK + CV), c = e % (MAPS * CK + CV), key = kb + j, m = c / CK;
-            const int phys = key <= p1 ? page_of(a, sg.seq, key) : -1;
-            const __nv_bfloat16 *src = kv + ((size_t)(phys < 0 ? 0 : phys) * a.kv_heads + kvh) * (kBlockTokens * (KW + DV));
-            if (MAPS * CK > c) cp_async16(dst + (m * kTileKeys + j) * LK + c % CK * 8, src + (key % kBlockTokens) * KW + c * 8, phys >= 0);
-            else cp_async16(dst + MAPS * kTileKeys * LK + j * LV + (c - MAPS * CK) * 8, src + kBlockTokens * KW + (key % kBlockTokens) * DV + (c - MAPS * CK) * 8, phys >= 0);
+    __syncthreads();
+    if (pdl & 1) griddep_wait();
+    if (tid >= NC) {
+        const __nv_bfloat16 *kv = reinterpret_cast<const __nv_bfloat16 *>(a.kv) + (size_t)kvh * P::ELEMS;
+        auto lookup = [&](int it) {
+            const int key = first + it * KT + lane * 16;
+            return lane < PAGES && it < n_tiles && key <= p1 ? page_of(a, sg.seq, key) : -1;
+        };
+        int phys = lookup(0), it = 0;
+        for (; it < n_tiles; it++) {
+            const int next = lookup(it + 1), s = it % ST;
+            int ok = 1;
+            const uint32_t pages = __popc(__ballot_sync(0xffffffffu, phys >= 0));
+            if (lane == 0) {
+                if (it >= ST) ok = mbar_wait_bounded(&empty[s], (it / ST - 1) & 1, a.status, s_abort);
+                if (ok) mbar_expect_tx(&full[s], pages * P::BYTES);
+            }
+            if (!__shfl_sync(0xffffffffu, ok, 0)) break;
+            if (phys >= 0) bulk_g2s(ring + s * T::stage_elems + lane * P::ELEMS, kv + (size_t)phys * a.kv_heads * P::ELEMS, P::BYTES, &full[s]);
+            phys = next;
         }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    load(0, first);
+        if (*s_abort && lane == 0)  // copies in flight still target this CTA's shared memory: a bounded chance to land
+            for (int k = max(it - ST, 0); k < it; k++)
+                for (uint32_t i = 0; i < (1u << 16) && !mbar_try_wait(&full[k % ST], (k / ST) & 1u); i++) {
+                }
+        return;
+    }
+    {
+        constexpr int LANES = head_lanes(DK), PER = NC / LANES, N = 64 / PER;  // vectors at a time, rounds
+        const __nv_bfloat16 *proj = reinterpret_cast<const __nv_bfloat16 *>(a.proj);
+        const int piece = tid & (LANES - 1);
+        auto source = [&](int v, int &row) {  // vector v = row of the block, map
+            const int r = r0 + v / MAPS, t = r / grp, h = kvh * grp + r % grp;
+            row = row_base + t;
+            return r < rows ? proj + (size_t)row * a.ldp + a.q_off + (h * MAPS + v % MAPS) * DK : nullptr;
+        };
+        uint4 raw[N];
+#pragma unroll
+        for (int n = 0; n < N; n++) {
+            int row;
+            const __nv_bfloat16 *src = source(n * PER + tid / LANES, row);
+            raw[n] = src && piece * 8 < DK ? *reinterpret_cast<const uint4 *>(src + piece * 8) : make_uint4(0, 0, 0, 0);
+        }
+#pragma unroll
+        for (int n = 0; n < N; n++) {
+            const int v = n * PER + tid / LANES;
+            if (a.prepared()) {
+                int row;
+                const __nv_bfloat16 *src = source(v, row);
+                float x[8];
+                load8(reinterpret_cast<const __nv_bfloat16 *>(&raw[n]), x);
+                prepare_head(x, src ? src : proj, piece, LANES, head_prep(a, false, src ? row : row_base));
+                store8(reinterpret_cast<__nv_bfloat16 *>(&raw[n]), x);
+            }
+            if (piece * 8 < DK) *reinterpret_cast<uint4 *>(qs + (v % MAPS * ROWS + v / MAPS) * LQ + piece * 8) = raw[n];
+        }
+        named_bar_sync(1, NC);
+    }
     int lo[2], hi[2], rt[2];
 #pragma unroll
     for (int e = 0; e < 2; e++) {
         const int r = r0 + warp * 16 + g + 8 * e;
         rt[e] = r < rows ? r : -1;
-        hi[e] = p0 + (r < rows ? r / grp : r0 / grp);
+        hi[e] = p0 + (r < rows ? r : r0) / grp;
         lo[e] = first_visible(hi[e], a.chunk);
     }
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[DV / 8][4];
@@ -218,23 +303,25 @@ __global__ void __launch_bounds__(128 * MAPS) attn_tile_kernel(const AttnArgs a,
 #pragma unroll
         for (int e = 0; e < 4; e++) o[n][e] = 0.f;
     auto qfrag = [&](int kk, uint32_t (&f)[4]) {
-        ldmatrix_x4(f, qs + (size_t)(map * 64 + warp * 16 + (lane & 15)) * LK + kk * 16 + (lane >> 4) * 8);
+        ldmatrix_x4(f, qs + (size_t)(map * ROWS + warp * 16 + (lane & 15)) * LQ + kk * 16 + (lane >> 4) * 8);
     };
     const float sl = a.scale * 1.4426950408889634f;
     const int vis_lo = first_visible(p1, a.chunk);
-    int it = 0;
-    for (int kb = first; kb <= p1; kb += kTileKeys, it++) {
-        if (kb + kTileKeys <= p1) {
-            load((it + 1) & 1, kb + kTileKeys);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
+    for (int it = 0; it < n_tiles; it++) {
+        const int s = it % ST, kb = first + it * KT;
+        if (!__all_sync(0xffffffffu, mbar_wait_bounded(&full[s], (it / ST) & 1, a.status, s_abort))) break;
+        __nv_bfloat16 *stage = ring + s * T::stage_elems;
+        if (kb + KT > p1 + 1) {  // every warp clears what it is going to read
+#pragma unroll
+            for (int i = 0; i < PAGES; i++)
+                if (kb + 16 * i + 15 > p1) P::clear_values(stage + i * P::ELEMS, max(p1 + 1 - kb - 16 * i, 0), lane);
+            __syncwarp();
         }
-        __syncthreads();
-        const __nv_bfloat16 *ks = kv_s + (size_t)(it & 1) * STAGE;
-        const bool masked = kb + kTileKeys - 1 > p0 + r0 / grp || kb < vis_lo;
-        attend_tile<DK, DV, kTileKeys>(qfrag, ks + map * kTileKeys * LK, ks + MAPS * kTileKeys * LK, kb, masked, lo, hi, sl, m, l, o, lane);
-        __syncthreads();
+        auto kat = [&](int r, int c) { return P::k(stage + (r >> 4) * P::ELEMS, r & 15, map * (DK / 8) + c); };
+        auto vat = [&](int r, int c) { return P::v(stage + (r >> 4) * P::ELEMS, r & 15, c); };
+        attend_tile<DK, DV, KT>(qfrag, kat, vat, kb, kb + KT - 1 > b0 || kb < vis_lo, lo, hi, sl, m, l, o, lane);
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&empty[s]);
     }
     float f[2];
 #pragma unroll
@@ -244,7 +331,8 @@ __global__ void __launch_bounds__(128 * MAPS) attn_tile_kernel(const AttnArgs a,
         f[e] = l[e] > 0.f ? 1.f / l[e] : 0.f;
     }
     if (MAPS == 2) {
-        float *other = reinterpret_cast<float *>(kv_s);  // [64][DV + 8]
+        float *other = reinterpret_cast<float *>(ring);  // [ROWS][DV + 8]
+        named_bar_sync(1, NC);  // every warp is done with the stages
         const int t2 = 2 * (lane & 3);
         if (map == 1) {
 #pragma unroll
@@ -253,7 +341,7 @@ __global__ void __launch_bounds__(128 * MAPS) attn_tile_kernel(const AttnArgs a,
                 for (int n = 0; n < DV / 8; n++)
                     *reinterpret_cast<float2 *>(other + (warp * 16 + g + 8 * e) * LV + n * 8 + t2) = make_float2(o[n][2 * e] * f[e], o[n][2 * e + 1] * f[e]);
         }
-        __syncthreads();
+        named_bar_sync(1, NC);
         if (map == 1) return;
 #pragma unroll
         for (int e = 0; e < 2; e++) {
@@ -290,96 +378,113 @@ __global__ void __launch_bounds__(128 * MAPS) attn_tile_kernel(const AttnArgs a,
 }
 
 // Entries with one token: a cluster of CTAs per (entry, key head) cuts the visible pages between them, a warp takes every
-// fourth page of its CTA through its own copy ring (no block barrier in the loop), and the partial softmax states meet through
-// cluster shared memory.  The query rows are the heads of the group times the maps: with two maps a row is zero outside its own
-// map's half of the key, so one product scores both.  With one map CTA r of the cluster finishes its share of the head's columns,
-// with two a warp somewhere in the cluster finishes a head.  With FUSED the kernel prepares its heads itself, and the CTA that
-// owns the last page writes the token's K and V into it first.
+// fourth page of its CTA through its own ring of bulk copies (no block barrier in the loop), and the partial softmax states meet
+// through cluster shared memory.  The query rows are the heads of the group times the maps: with two maps a row is zero outside its
+// own map's half of the key, so one product scores both.  With one map CTA r of the cluster finishes its share of the head's
+// columns, with two a warp somewhere in the cluster finishes a head.  With FUSED the token's own K and V are not in the pages yet:
+// the CTA that owns the last page prepares and writes them, and patches its copy of the page; earlier pages are requested before
+// the wait for the launch in front.
 template <int DK, int DV>
-__host__ __device__ constexpr int single_stages() { return DK + DV <= 256 ? 3 : 2; }
-template <int DK, int DV>
-__host__ __device__ constexpr size_t single_ring() {
-    const size_t ring = (size_t)4 * single_stages<DK, DV>() * 16 * (DK + DV + 16) * 2, part = sizeof(float) * 4 * 16 * (DV + 4);
-    return ring > part ? ring : part;  // the warps' partial states take the ring's place
-}
-template <int DK, int DV>
-__host__ __device__ constexpr size_t single_smem() {
-    return single_ring<DK, DV>() + sizeof(float) * 16 * (DV + 4) + (size_t)16 * (DK + 8) * 2;  // the CTA's merged state and the query rows are their own
-}
+struct Single {
+    using P = Page<DK, DV>;
+    static constexpr int ST = 4 * 6 * P::BYTES <= 104 * 1024 ? 6 : (4 * 4 * P::BYTES <= 104 * 1024 ? 4 : (4 * 3 * P::BYTES <= 104 * 1024 ? 3 : 2));
+    static constexpr int PW = DV + 4, LQ = DK + 8;
+    static constexpr size_t ring_bytes = 4 * ST * (size_t)P::BYTES, part_bytes = sizeof(float) * 4 * 16 * PW, front = ring_bytes > part_bytes ? ring_bytes : part_bytes;
+    static constexpr size_t merged_bytes = sizeof(float) * 16 * PW, query_bytes = (size_t)2 * (16 * LQ + DK + DV);
+    static constexpr size_t smem = front + (merged_bytes > query_bytes ? merged_bytes : query_bytes);
+};
 
 template <int DK, int DV>  // DK: of all maps together
 __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, const Seg *__restrict__ segs, const int *__restrict__ singles, int row_blocks,
                                                           int fused, int pdl) {
-    constexpr int LK = DK + 8, LV = DV + 8, CK = DK / 8, CV = DV / 8, ST = single_stages<DK, DV>(), PW = DV + 4, PAGE = 16 * (LK + LV);
-    extern __shared__ __align__(16) uint8_t attn_smem[];
-    __nv_bfloat16 *ring = reinterpret_cast<__nv_bfloat16 *>(attn_smem);                      // [4 warps][ST][K 16 x LK | V 16 x LV]
-    float *part = reinterpret_cast<float *>(attn_smem);                                      // [4 warps][16][m, l, -, -, o[DV]], after the loop
-    float *merged = reinterpret_cast<float *>(attn_smem + single_ring<DK, DV>());            // [16][m, l, -, -, o[DV]] of this CTA
-    __nv_bfloat16 *qs = reinterpret_cast<__nv_bfloat16 *>(merged + 16 * PW);                 // [16][LK]
-    __shared__ float bufs[128 * 8];
+    using S = Single<DK, DV>;
+    using P = typename S::P;
+    constexpr int LQ = S::LQ, ST = S::ST, PW = S::PW, CV = DV / 8;
+    extern __shared__ __align__(128) uint8_t attn_smem[];
+    __nv_bfloat16 *ring = reinterpret_cast<__nv_bfloat16 *>(attn_smem);        // [4 warps][ST] pages
+    float *part = reinterpret_cast<float *>(attn_smem);                        // [4 warps][16][m, l, -, -, o[DV]], after the loop
+    float *merged = reinterpret_cast<float *>(attn_smem + S::front);           // [16][m, l, -, -, o[DV]] of this CTA, after the loop
+    __nv_bfloat16 *qs = reinterpret_cast<__nv_bfloat16 *>(attn_smem + S::front), *own = qs + 16 * LQ;  // query rows [16][LQ]; the token's [K | V]
+    __shared__ __align__(8) uint64_t full[4][ST];
+    __shared__ int s_abort_mem;
+    volatile int *s_abort = &s_abort_mem;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t2 = 2 * (lane & 3);
     const int nsplit = gridDim.x, split = blockIdx.x, maps = a.maps, hpb = 16 / maps, dk = DK / maps;
     const int rb = blockIdx.y % row_blocks, kvh = blockIdx.y / row_blocks, grp = a.heads / a.kv_heads, h0 = kvh * grp + rb * hpb, nh = min(hpb, grp - rb * hpb);
     if (pdl & 2) griddep_launch_dependents();
     const Seg sg = segs[singles[blockIdx.z]];
     const int p = sg.pos0, row = sg.row0, first = first_visible(p, a.chunk), lo_page = first / kBlockTokens, n_pages = p / kBlockTokens - lo_page + 1;
-    const int pg0 = lo_page + split * n_pages / nsplit, pg1 = lo_page + (split + 1) * n_pages / nsplit;
-    const __nv_bfloat16 *proj = reinterpret_cast<const __nv_bfloat16 *>(a.proj) + (size_t)row * a.ldp;
-    __nv_bfloat16 *kv = reinterpret_cast<__nv_bfloat16 *>(a.kv);
-    for (int e = tid; e < 16 * LK / 8; e += 128) reinterpret_cast<uint4 *>(qs)[e] = make_uint4(0, 0, 0, 0);
-    if (pdl & 1) griddep_wait();
+    const int pg0 = lo_page + split * n_pages / nsplit, pg1 = lo_page + (split + 1) * n_pages / nsplit, last = p / kBlockTokens;
+    __nv_bfloat16 *kv = reinterpret_cast<__nv_bfloat16 *>(a.kv) + (size_t)kvh * P::ELEMS;
+    if (lane == 0) {
+        for (int s = 0; s < ST; s++) mbar_init(&full[warp][s], 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (tid == 0) *s_abort = 0;
+    for (int e = tid; e < 16 * LQ / 8; e += 128) reinterpret_cast<uint4 *>(qs)[e] = make_uint4(0, 0, 0, 0);
     __syncthreads();
+    __nv_bfloat16 *mine = ring + (size_t)warp * ST * P::ELEMS;
+    // physical blocks of this warp's next 32 pages, a page per lane: one trip to the table instead of one per page
+    int blocks = -1;
+    auto load = [&](int i) {  // the i-th page of this warp
+        const int pg = pg0 + warp + 4 * i;
+        if ((i & 31) == 0) {
+            const int at = pg + 4 * lane;
+            blocks = at < pg1 ? page_of(a, sg.seq, at * kBlockTokens) : -1;
+        }
+        const int phys = __shfl_sync(0xffffffffu, blocks, i & 31);
+        if (pg < pg1 && lane == 0) {
+            mbar_expect_tx(&full[warp][i % ST], phys >= 0 ? P::BYTES : 0);
+            if (phys >= 0) bulk_g2s(mine + (size_t)(i % ST) * P::ELEMS, kv + (size_t)phys * a.kv_heads * P::ELEMS, P::BYTES, &full[warp][i % ST]);
+        }
+    };
+    const bool append = fused && split == nsplit - 1;
+    if (fused) {
+#pragma unroll
+        for (int i = 0; i < ST; i++) load(i);
+    }
+    if (pdl & 1) griddep_wait();
+    if (!fused) {
+#pragma unroll
+        for (int i = 0; i < ST; i++) load(i);
+    }
+    const __nv_bfloat16 *proj = reinterpret_cast<const __nv_bfloat16 *>(a.proj) + (size_t)row * a.ldp;
     {
         // heads of the group, then (with the last page) the key's maps
         const int lanes = head_lanes(dk), piece = tid & (lanes - 1), slots = 128 / lanes, nq = nh * maps;
-        const bool append = fused && split == nsplit - 1;
-        const int phys = append ? page_of(a, sg.seq, p) : -1, total = nq + (phys >= 0 ? maps : 0);
-        __nv_bfloat16 *page = kv + ((size_t)(phys < 0 ? 0 : phys) * a.kv_heads + kvh) * (16 * (DK + DV));
+        const int phys = append ? page_of(a, sg.seq, p) : -1, total = nq + (append ? maps : 0), r = p % kBlockTokens;
+        __nv_bfloat16 *page = kv + (size_t)max(phys, 0) * a.kv_heads * P::ELEMS;
         for (int v0 = 0; v0 < total; v0 += slots) {
             const int v = v0 + tid / lanes;
             const bool load = v < total && piece * 8 < dk, key = v >= nq;
+            const __nv_bfloat16 *src = proj + (key ? a.k_off + (kvh * maps + min(v - nq, maps - 1)) * dk : a.q_off + (h0 * maps + v) * dk);
             float x[8];
-            if (load) load8(proj + (key ? a.k_off + (kvh * maps + v - nq) * dk : a.q_off + (h0 * maps + v) * dk) + piece * 8, x);
+            if (load) load8(src + piece * 8, x);
             else {
 #pragma unroll
                 for (int e = 0; e < 8; e++) x[e] = 0.f;
             }
-            if (fused && a.prepared())
-                prepare_head(x, piece, lanes, a.dim, key ? a.k_norm : a.q_norm, a.eps, a.cs + (size_t)row * a.half, a.half, a.interleaved, bufs + (tid - piece) * 8);
+            if (a.prepared()) prepare_head(x, src, piece, lanes, head_prep(a, key, row));
             if (!load) continue;
-            if (key) store8(page + (size_t)(p % kBlockTokens) * DK + (v - nq) * dk + piece * 8, x);
-            else store8(qs + ((v % maps) * hpb + v / maps) * LK + (v % maps) * dk + piece * 8, x);
+            if (key) {
+                const int c = (v - nq) * (dk / 8) + piece;
+                store8(own + c * 8, x);
+                if (phys >= 0) store8(P::k(page, r, c), x);
+            } else {
+                store8(qs + ((v % maps) * hpb + v / maps) * LQ + (v % maps) * dk + piece * 8, x);
+            }
         }
-        if (phys >= 0)
-            for (int c = tid; c < CV; c += 128)
-                *reinterpret_cast<uint4 *>(page + 16 * DK + (size_t)(p % kBlockTokens) * DV + c * 8) = *reinterpret_cast<const uint4 *>(proj + a.v_off + kvh * DV + c * 8);
-        __syncthreads();  // the copies below read what this CTA has just written
+        if (append)
+            for (int c = tid; c < CV; c += 128) {
+                const uint4 x = *reinterpret_cast<const uint4 *>(proj + a.v_off + kvh * DV + c * 8);
+                *reinterpret_cast<uint4 *>(own + DK + c * 8) = x;
+                if (phys >= 0) *reinterpret_cast<uint4 *>(P::v(page, r, c)) = x;
+            }
+        __syncthreads();
     }
-    __nv_bfloat16 *mine = ring + (size_t)warp * ST * PAGE;
-    // physical blocks of this warp's next 32 pages, a page per lane: one trip to the table instead of one per page
-    int blocks = -1;
-    auto lookup = [&](int i) {
-        const int pg = pg0 + warp + 4 * (i + lane);
-        blocks = pg < pg1 ? page_of(a, sg.seq, pg * kBlockTokens) : -1;
-    };
-    auto load = [&](int i) {  // the i-th page of this warp
-        const int pg = pg0 + warp + 4 * i;
-        if ((i & 31) == 0) lookup(i);
-        const int phys = __shfl_sync(0xffffffffu, blocks, i & 31);
-        if (pg < pg1) {
-            const __nv_bfloat16 *src = kv + ((size_t)(phys < 0 ? 0 : phys) * a.kv_heads + kvh) * (16 * (DK + DV));
-            __nv_bfloat16 *dst = mine + (size_t)(i % ST) * PAGE;
-            const int live = phys < 0 ? 0 : p + 1 - pg * kBlockTokens;  // rows of the page that hold tokens
-            for (int e = lane; e < 16 * CK; e += 32) cp_async16(dst + e / CK * LK + e % CK * 8, src + e * 8, e / CK < live);
-            for (int e = lane; e < 16 * CV; e += 32) cp_async16(dst + 16 * LK + e / CV * LV + e % CV * 8, src + 16 * DK + e * 8, e / CV < live);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-#pragma unroll
-    for (int i = 0; i < ST - 1; i++) load(i);
     uint32_t q[DK / 16][4];
 #pragma unroll
-    for (int kk = 0; kk < DK / 16; kk++) ldmatrix_x4(q[kk], qs + (size_t)(lane & 15) * LK + kk * 16 + (lane >> 4) * 8);
+    for (int kk = 0; kk < DK / 16; kk++) ldmatrix_x4(q[kk], qs + (size_t)(lane & 15) * LQ + kk * 16 + (lane >> 4) * 8);
     auto qfrag = [&](int kk, uint32_t (&f)[4]) { f[0] = q[kk][0], f[1] = q[kk][1], f[2] = q[kk][2], f[3] = q[kk][3]; };
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[DV / 8][4];
 #pragma unroll
@@ -389,15 +494,29 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
     const int lo[2] = {first, first}, hi[2] = {p, p};
     const float sl = a.scale * 1.4426950408889634f;
     for (int i = 0; pg0 + warp + 4 * i < pg1; i++) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(ST - 2) : "memory");
+        const int pg = pg0 + warp + 4 * i, kb = pg * kBlockTokens;
+        if (!__all_sync(0xffffffffu, mbar_wait_bounded(&full[warp][i % ST], (i / ST) & 1, a.status, s_abort))) break;
+        __nv_bfloat16 *page = mine + (size_t)(i % ST) * P::ELEMS;
+        if (pg == last) {
+            const int r = p % kBlockTokens;
+            P::clear_values(page, r + (fused ? 0 : 1), lane);
+            __syncwarp();
+            if (fused) {
+                for (int c = lane; c < DK / 8; c += 32) *reinterpret_cast<uint4 *>(P::k(page, r, c)) = *reinterpret_cast<const uint4 *>(own + c * 8);
+                for (int c = lane; c < CV; c += 32) *reinterpret_cast<uint4 *>(P::v(page, r, c)) = *reinterpret_cast<const uint4 *>(own + DK + c * 8);
+                __syncwarp();
+            }
+        }
+        auto kat = [&](int r, int c) { return P::k(page, r, c); };
+        auto vat = [&](int r, int c) { return P::v(page, r, c); };
+        attend_tile<DK, DV, 16>(qfrag, kat, vat, kb, kb < first || kb + 15 > p, lo, hi, sl, m, l, o, lane);
         __syncwarp();
-        const __nv_bfloat16 *ks = mine + (size_t)(i % ST) * PAGE;
-        const int kb = (pg0 + warp + 4 * i) * kBlockTokens;
-        attend_tile<DK, DV, 16>(qfrag, ks, ks + 16 * LK, kb, kb < first || kb + 15 > p, lo, hi, sl, m, l, o, lane);
-        __syncwarp();
-        load(i + ST - 1);
+        load(i + ST);
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    if (*s_abort && lane == 0)  // copies in flight still target this CTA's shared memory: a bounded chance to land
+        for (int i = 0; pg0 + warp + 4 * i < pg1; i++)
+            for (uint32_t k = 0; k < (1u << 14) && !mbar_try_wait(&full[warp][i % ST], (i / ST) & 1u); k++) {
+            }
     __syncthreads();  // every warp is done with its ring
 #pragma unroll
     for (int e = 0; e < 2; e++) {
@@ -508,14 +627,17 @@ bool attn_padded_head(int dim, int vdim, int maps, int *DK, int *DV) {
 }
 int attn_query_tile(int heads, int kv_heads) { return std::max(1, 64 / (heads / kv_heads)); }
 
-static long long prep_blocks(const AttnArgs &a, int rows) {
-    const long long vectors = (long long)rows * ((a.prepared() ? a.heads * a.maps : 0) + a.kv_heads * (a.maps + 1));
-    return (vectors * head_lanes(a.DK) + 255) / 256;
+// Threads of a row's preparation: one block, or several of 256.
+static void prep_shape(const AttnArgs &a, bool queries, int rows, dim3 *grid, dim3 *block) {
+    const int threads = ((queries ? a.heads * a.maps : 0) + a.kv_heads * (a.maps + 1)) * head_lanes(a.DK);
+    *block = dim3((unsigned)std::min(256, (threads + 31) / 32 * 32)), *grid = dim3((unsigned)rows, (threads + block->x - 1) / block->x);
 }
 
 template <class AT>
 static int32_t rows_attention(const StepDesc &d, const AttnArgs &a, cudaStream_t st) {
-    attn_prep_kernel<AT><<<(unsigned)prep_blocks(a, d.rows), 256, 0, st>>>(a, d.seq, d.pos, d.rows, 0);
+    dim3 grid, block;
+    prep_shape(a, a.prepared(), d.rows, &grid, &block);
+    attn_prep_kernel<AT><<<grid, block, 0, st>>>(a, d.seq, d.pos, a.prepared(), 0);
     attn_rows_kernel<AT><<<(unsigned)((d.rows * (long long)a.heads + 7) / 8), 256, 0, st>>>(a, d.seq, d.pos, d.rows);
     JGPT_CUDA_TRY(cudaGetLastError());
     return JGPT_OK;
@@ -546,17 +668,19 @@ static int32_t tensor_attention(const StepDesc &d, const AttnArgs &a, int pdl, c
         return n + 1;
     };
     if (d.n_tiles) {
-        cfg.gridDim = dim3((unsigned)prep_blocks(a, d.rows)), cfg.blockDim = dim3(256), cfg.dynamicSmemBytes = 0, cfg.numAttrs = (unsigned)early(0);
-        JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, attn_prep_kernel<__nv_bfloat16>, a, d.seq, d.pos, d.rows, pdl));
+        using T = Tile<DK, DV, MAPS>;
+        prep_shape(a, false, d.rows, &cfg.gridDim, &cfg.blockDim);
+        cfg.dynamicSmemBytes = 0, cfg.numAttrs = (unsigned)early(0);
+        JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, attn_prep_kernel<__nv_bfloat16>, a, d.seq, d.pos, 0, pdl));
         static thread_local int set_for = -1;
-        if (int32_t rc = opt_in(attn_tile_kernel<DK, DV, MAPS>, tile_smem<DK, DV, MAPS>(), set_for)) return rc;
-        cfg.gridDim = dim3((unsigned)d.n_tiles, (unsigned)a.kv_heads, (unsigned)((d.qt * grp + 63) / 64)), cfg.blockDim = dim3(128 * MAPS);
-        cfg.dynamicSmemBytes = tile_smem<DK, DV, MAPS>(), cfg.numAttrs = (unsigned)early(0);
+        if (int32_t rc = opt_in(attn_tile_kernel<DK, DV, MAPS>, T::smem, set_for)) return rc;
+        cfg.gridDim = dim3((unsigned)d.n_tiles, (unsigned)a.kv_heads, (unsigned)((d.qt * grp + T::ROWS - 1) / T::ROWS)), cfg.blockDim = dim3(160);
+        cfg.dynamicSmemBytes = T::smem, cfg.numAttrs = (unsigned)early(0);
         JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, attn_tile_kernel<DK, DV, MAPS>, a, d.segs, d.tiles, d.qt, pdl));
     }
     if (d.n_singles) {
         static thread_local int set_for = -1;
-        if (int32_t rc = opt_in(attn_single_kernel<KW, DV>, single_smem<KW, DV>(), set_for)) return rc;
+        if (int32_t rc = opt_in(attn_single_kernel<KW, DV>, (Single<KW, DV>::smem), set_for)) return rc;
         const int row_blocks = (grp * MAPS + 15) / 16, ctas = d.n_singles * a.kv_heads * row_blocks;
         const int keys = a.chunk > 0 ? std::min(a.chunk, d.max_len) : d.max_len, pages = keys / kBlockTokens + 1;
         int split = 1;  // every warp keeps two pages, the grid stays around two CTAs per SM
@@ -568,7 +692,7 @@ static int32_t tensor_attention(const StepDesc &d, const AttnArgs &a, int pdl, c
             na++;
         }
         cfg.gridDim = dim3((unsigned)split, (unsigned)(a.kv_heads * row_blocks), (unsigned)d.n_singles), cfg.blockDim = dim3(128);
-        cfg.dynamicSmemBytes = single_smem<KW, DV>(), cfg.numAttrs = (unsigned)na;
+        cfg.dynamicSmemBytes = (Single<KW, DV>::smem), cfg.numAttrs = (unsigned)na;
         JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, attn_single_kernel<KW, DV>, a, d.segs, d.singles, row_blocks, d.n_tiles ? 0 : 1, pdl));
     }
     return JGPT_OK;

@@ -530,7 +530,9 @@ __global__ void __launch_bounds__(128, DK <= 192 ? 3 : 1) latent_tile_kernel(con
         __syncthreads();
         const __nv_bfloat16 *ks = kv_s + (size_t)(it & 1) * kTileKeys * (LK + LV);
         const bool masked = kb + kTileKeys - 1 > p0 - en.key0 || kb < vis_lo;
-        attend_tile<DK, DV, kTileKeys>(qfrag, ks, ks + kTileKeys * LK, kb, masked, lo, hi, sl, m, l, o, lane);
+        auto kat = [&](int r, int c) { return ks + r * LK + c * 8; };
+        auto vat = [&](int r, int c) { return ks + kTileKeys * LK + r * LV + c * 8; };
+        attend_tile<DK, DV, kTileKeys>(qfrag, kat, vat, kb, masked, lo, hi, sl, m, l, o, lane);
         __syncthreads();
     }
 #pragma unroll

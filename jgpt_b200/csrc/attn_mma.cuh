@@ -69,13 +69,12 @@ __device__ __forceinline__ void store8(float *p, const float (&v)[8]) {
     *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]), *reinterpret_cast<float4 *>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
 }
 
-// 16 rows x KT keys of one warp against staged K rows (stride DK + 8) and V rows (stride DV + 8): scores, online softmax, P.V.
-// lo / hi: visible key range of this thread's rows g and g + 8 (inclusive); kb: first key of the tile.
-template <int DK, int DV, int KT, class QFrag>
-__device__ __forceinline__ void attend_tile(const QFrag &qfrag, const __nv_bfloat16 *ks, const __nv_bfloat16 *vs, int kb, bool masked,
-                                            const int (&lo)[2], const int (&hi)[2], float scale_log2, float (&m)[2], float (&l)[2],
-                                            float (&o)[DV / 8][4], int lane) {
-    constexpr int LK = DK + 8, LV = DV + 8, NT = KT / 8;
+// 16 rows x KT keys of one warp against staged K and V rows: scores, online softmax, P.V.  kat / vat (row, chunk): address of the
+// chunk-th 8 elements of a row.  lo / hi: visible key range of this thread's rows g and g + 8 (inclusive); kb: first key of the tile.
+template <int DK, int DV, int KT, class QFrag, class KAt, class VAt>
+__device__ __forceinline__ void attend_tile(const QFrag &qfrag, const KAt &kat, const VAt &vat, int kb, bool masked, const int (&lo)[2],
+                                            const int (&hi)[2], float scale_log2, float (&m)[2], float (&l)[2], float (&o)[DV / 8][4], int lane) {
+    constexpr int NT = KT / 8;
     float s[NT][4];
 #pragma unroll
     for (int j = 0; j < NT; j++)
@@ -88,7 +87,7 @@ __device__ __forceinline__ void attend_tile(const QFrag &qfrag, const __nv_bfloa
 #pragma unroll
         for (int j = 0; j < NT; j += 2) {
             uint32_t b[4];
-            ldmatrix_x4(b, ks + (size_t)(j * 8 + ((lane >> 4) << 3) + (lane & 7)) * LK + kk * 16 + ((lane >> 3) & 1) * 8);
+            ldmatrix_x4(b, kat(j * 8 + ((lane >> 4) << 3) + (lane & 7), kk * 2 + ((lane >> 3) & 1)));
             mma_bf16(s[j], a, b[0], b[1]);
             mma_bf16(s[j + 1], a, b[2], b[3]);
         }
@@ -135,7 +134,7 @@ __device__ __forceinline__ void attend_tile(const QFrag &qfrag, const __nv_bfloa
 #pragma unroll
         for (int n = 0; n < DV / 8; n += 2) {
             uint32_t b[4];
-            ldmatrix_x4_trans(b, vs + (size_t)(kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * LV + n * 8 + (lane >> 4) * 8);
+            ldmatrix_x4_trans(b, vat(kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), n + (lane >> 4)));
             mma_bf16(o[n], ph, b[0], b[1]);
             mma_bf16(o[n], pl, b[0], b[1]);
             mma_bf16(o[n + 1], ph, b[2], b[3]);

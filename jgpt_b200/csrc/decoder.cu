@@ -303,7 +303,7 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
             }
             b.kv_layer = (int)d->kv.size();
             KvLayerGeom geom;
-            geom.heads = s.kv_heads, geom.dim = b.maps * b.DK + b.DV, geom.parts = 1;
+            geom.heads = s.kv_heads, geom.dim = mix::page_row(b.maps * b.DK) + mix::page_row(b.DV), geom.parts = 1;
             d->kv.push_back(geom);
         } else if (s.kind == JGPT_MIX_GLA || s.kind == JGPT_MIX_DELTA) {
             const bool delta = s.kind == JGPT_MIX_DELTA;
@@ -864,7 +864,10 @@ static int32_t enqueue_moe(Decoder *d, const DLayer &y, int R, int pdl, mix::Moe
     TRY(mix::launch_route(r, R, pdl, d->ctx->stream));
     nt::RowGroups g;
     g.tiles = r.tiles, g.n_tiles = r.n_tiles, g.max_tiles = r.max_tiles, g.rows = T, g.n_groups = y.moe.experts, g.a_rows = R, g.w_group = (long long)y.effp * ldw;
+    const bool copied = T == nt::kLargeTile;  // the tcgen05 product reads its rows group by group, from the place of the results to come
+    if (copied) TRY(mix::launch_moe_gather(r, d->h, d->e_out, ldw, pdl, d->ctx->stream));
     nt::Problem in[2] = {{d->h, y.w_eup, d->e_act, r.list, R, y.effp, ldw, ldw, ldw, y.effp, 1.f}, {d->h, y.w_sup, d->s_act, nullptr, R, y.sffp, ldw, ldw, ldw, y.sffp, 1.f}};
+    if (copied) in[0].A = d->e_out, in[0].rowsel = nullptr, g.a_rows = R * y.moe.top;
     in[0].grp = g, in[0].act = act(y.moe.act), in[1].act = act(y.moe.shared_act);
     TRY(product(d, in, y.sffp ? 2 : 1, nt::EPI_ACT, pdl));
     g.a_rows = R * y.moe.top, g.early = true;

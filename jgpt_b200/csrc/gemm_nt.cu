@@ -269,9 +269,9 @@ int umma_min_rows() {
 
 int group_tile_rows(bool f32, int rows, int copies, int groups) {
     if (f32) return 64;
-    if (umma_min_rows() > 0 && rows >= umma_min_rows()) return 128;
+    if (umma_min_rows() > 0 && rows >= umma_min_rows()) return kLargeTile;
     const int mean = (rows * copies + groups - 1) / groups;
-    return mean <= 8 ? 16 : (mean <= 16 ? 32 : 64);
+    return mean <= 10 ? 16 : (mean <= 22 ? 32 : 64);
 }
 
 // Defaults spelled out: one segment, the residual in C itself.
@@ -291,10 +291,10 @@ int32_t launch_bf16(const Ctx *ctx, const Problem *problems, int n, Epilogue epi
     Problem p[2];
     if (int32_t rc = complete(problems, n, epi, p)) return rc;
     bool big = p[0].M >= umma_min_rows() && umma_min_rows() > 0;
-    for (int i = 0; i < n; i++) big = big && (!p[i].rowsel || p[i].grp.tiles);
+    for (int i = 0; i < n; i++) big = big && !p[i].rowsel;
     if (p[0].grp.tiles) {
         const int rows = p[0].grp.rows;
-        JGPT_REQUIRE(big ? rows == 128 : (rows == 16 || rows == 32 || rows == 64), JGPT_ERR_INVALID_ARGUMENT, "row tiles of %d", rows);
+        JGPT_REQUIRE(big ? rows == kLargeTile : (rows == 16 || rows == 32 || rows == 64), JGPT_ERR_INVALID_ARGUMENT, "row tiles of %d", rows);
         if (!big) return epi == EPI_ACT ? small_dispatch<EPI_ACT, true>(ctx, p, n, pdl, st) : small_dispatch<EPI_STORE, true>(ctx, p, n, pdl, st);
     }
     if (big) {

@@ -38,7 +38,7 @@ struct Problem {
     const void *A;     // [M, lda]
     const void *W;     // [N, ldw]
     void *C;           // [M, ldc]
-    const int *rowsel; // optional: row m of A is rowsel[m] (the large-M kernel takes it with rows in groups only)
+    const int *rowsel; // optional: row m of A is rowsel[m] (not for the large-M kernel)
     int M, N, K, lda, ldw, ldc;
     float scale = 1.f;
     // Segments: columns [s seg_n, (s + 1) seg_n) read the operand at A + s a_seg (elements) and land at column n + s c_seg of C.
@@ -90,7 +90,9 @@ int32_t launch_f32(const Problem *p, int n, Epilogue epi, cudaStream_t st);
 
 // From this many rows on launch_bf16 takes the tcgen05 kernel.
 int umma_min_rows();
-// Rows of a tile (RowGroups::rows) for products of `rows` rows, each of which is in `copies` of the groups.
+// Rows of a tile (RowGroups::rows) for products of `rows` rows, each of which is in `copies` of the groups; kLargeTile: the large-M
+// kernel, whose operand holds the rows group by group.
+constexpr int kLargeTile = 128;
 int group_tile_rows(bool f32, int rows, int copies, int groups);
 int32_t launch_bf16_umma(const Ctx *ctx, const Problem &p, Epilogue epi, int pdl, cudaStream_t st);
 

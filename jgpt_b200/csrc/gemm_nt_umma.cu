@@ -8,8 +8,8 @@
 //
 // Persistent CTAs of 320 threads: warp 0 issues the copies, warp 1 owns the tensor memory and issues the MMAs, warps 2-9
 // drain the accumulator (TMEM lane quarter = warp % 4, half the tile's columns each) while the next tile is multiplied.
-// Rows in groups (experts): the device's list of row tiles takes the place of the row grid, the weight tile's rows shift by group,
-// and an operand with a row list comes in through gather copies, four rows each, one per lane of the copying warp.
+// Rows in groups (experts): the device's list of row tiles takes the place of the row grid and the weight tile's rows
+// shift by group.
 // Output tiles are walked in groups of eight row tiles, rows fastest, so CTAs side by side share weight tiles in L2.
 // Every wait is bounded; on expiry the status word gets DEV_STATUS_WAIT_TIMEOUT and the CTA winds down.
 #include <cuda.h>
@@ -49,15 +49,7 @@ __device__ __forceinline__ void tma_2d(void *smem_dst, const CUtensorMap *map, i
                  : "memory");
 }
 
-// Four rows of 64 elements; the map's box is one row.
-__device__ __forceinline__ void tma_gather4(void *smem_dst, const CUtensorMap *map, int x, const int (&y)[4], uint64_t *bar) {
-    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile::gather4.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4, %5, %6}], [%7];" ::"r"(
-                     smem_u32(smem_dst)),
-                 "l"(map), "r"(x), "r"(y[0]), "r"(y[1]), "r"(y[2]), "r"(y[3]), "r"(smem_u32(bar))
-                 : "memory");
-}
-
-enum RowMode : int { ROWS_ALL = 0, ROWS_GROUPS = 1, ROWS_GATHERED = 2 };
+enum RowMode : int { ROWS_ALL = 0, ROWS_GROUPS = 1 };
 
 struct UmmaArgs {
     void *C;
@@ -68,8 +60,8 @@ struct UmmaArgs {
     const float *res, *colscale, *bias;
     int act;
     float p0, p1, res_scale;
-    const RowTile *tiles;  // groups: the row tiles, how many, each group's rows of W, the operand's row list
-    const int *n_tiles, *rowsel;
+    const RowTile *tiles;  // groups: the row tiles, how many, each group's rows of W
+    const int *n_tiles;
     int w_rows;
 };
 
@@ -114,40 +106,7 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
     const int mt = ROWS == ROWS_ALL ? a.mt : min(*a.n_tiles, a.mt), total = mt * a.nt;
 
     if (warp == 0) {
-        if (ROWS == ROWS_GATHERED) {
-            uint32_t it = 0;
-            for (int t = blockIdx.x; t < total; t += gridDim.x) {
-                int m, n, rows[4];
-                tile_of(a, mt, t, m, n);
-                const RowTile rt = a.tiles[m];
-#pragma unroll
-                for (int i = 0; i < 4; i++) rows[i] = a.rowsel[rt.src0 + (rt.row0 + 4 * lane + i < rt.row_end ? 4 * lane + i : 0)];
-                bool ok = true;
-                for (int kt = 0; kt < nk; kt++, it++) {
-                    const uint32_t s = it % ST, use = it / ST;
-                    int free = 1;
-                    uint8_t *dst = tiles + (size_t)s * SB;
-                    if (lane == 0) {
-                        if (use > 0) free = mbar_wait_bounded(&empty_bar[s], (use - 1) & 1u, a.status, s_abort);
-                        if (free) {
-                            mbar_expect_tx(&full_bar[s], SB);
-                            tma_2d(dst + A_BYTES, &wmap, kt * UK, rt.group * a.w_rows + n * BN, &full_bar[s]);
-                        }
-                    }
-                    if (!__shfl_sync(0xffffffffu, free, 0)) {
-                        ok = false;
-                        break;
-                    }
-                    tma_gather4(dst + lane * 4 * UK * 2, &amap, kt * UK, rows, &full_bar[s]);
-                }
-                if (!ok) break;
-            }
-            if (*s_abort && lane == 0) {
-                for (uint32_t k = it > (uint32_t)ST ? it - ST : 0; k < it; k++)
-                    for (uint32_t i = 0; i < (1u << 16) && !mbar_try_wait(&full_bar[k % ST], (k / ST) & 1u); i++) {
-                    }
-            }
-        } else if (lane == 0) {
+        if (lane == 0) {
             uint32_t it = 0;
             for (int t = blockIdx.x; t < total && !*s_abort; t += gridDim.x) {
                 int m, n;
@@ -325,12 +284,12 @@ static int32_t umma_launch(const Ctx *ctx, const Problem &p, int pdl, cudaStream
     CUtensorMap am, wm;
     const int segs = p.segments(), ay = (int)(p.a_seg / p.lda), ax = (int)(p.a_seg % p.lda), per_seg = (p.segment_cols() + BN - 1) / BN;
     const int w_rows = ROWS == ROWS_ALL ? 0 : (int)(p.grp.w_group / p.ldw), mt = ROWS == ROWS_ALL ? (p.M + UM - 1) / UM : p.grp.max_tiles;
-    int32_t rc = make_map(&am, p.A, ROWS == ROWS_ALL ? p.M + (segs - 1) * ay : p.grp.a_rows, p.K + (segs - 1) * ax, p.lda, ROWS == ROWS_GATHERED ? 1 : UM);
+    int32_t rc = make_map(&am, p.A, ROWS == ROWS_ALL ? p.M + (segs - 1) * ay : p.grp.a_rows, p.K + (segs - 1) * ax, p.lda, UM);
     if (!rc) rc = make_map(&wm, p.W, ROWS == ROWS_ALL ? p.N : (p.grp.n_groups - 1) * w_rows + p.N, p.K, p.ldw, BN);
     if (rc) return rc;
     UmmaArgs a{p.C, p.M, p.N, p.K, p.ldc, mt, segs * per_seg, pdl, p.scale, ctx->d_status,
                per_seg, p.segment_cols(), p.c_seg, ax, ay, p.res, p.colscale, p.bias, p.act, p.p0, p.p1, p.res_scale,
-               p.grp.tiles, p.grp.n_tiles, p.rowsel, w_rows};
+               p.grp.tiles, p.grp.n_tiles, w_rows};
     auto kern = gemm_nt_umma_kernel<BN, EPI, ROWS>;
     static thread_local int set_for = -1;
     if (set_for != ctx->device) {
@@ -366,8 +325,7 @@ int32_t launch_bf16_umma(const Ctx *ctx, const Problem &p, Epilogue epi, int pdl
                  JGPT_ERR_INVALID_ARGUMENT, "segments of %d columns, shifts %lld / %d", p.seg_n, p.a_seg, p.c_seg);
     if (p.grp.tiles) {
         JGPT_REQUIRE(p.grp.n_groups > 0 && p.grp.a_rows > 0 && p.grp.w_group % p.ldw == 0, JGPT_ERR_INVALID_ARGUMENT, "groups of rows");
-        if (epi == EPI_ACT) return p.rowsel ? umma_pick<EPI_ACT, ROWS_GATHERED>(ctx, p, pdl, st) : umma_pick<EPI_ACT, ROWS_GROUPS>(ctx, p, pdl, st);
-        return p.rowsel ? umma_pick<EPI_STORE, ROWS_GATHERED>(ctx, p, pdl, st) : umma_pick<EPI_STORE, ROWS_GROUPS>(ctx, p, pdl, st);
+        return epi == EPI_ACT ? umma_pick<EPI_ACT, ROWS_GROUPS>(ctx, p, pdl, st) : umma_pick<EPI_STORE, ROWS_GROUPS>(ctx, p, pdl, st);
     }
     switch (epi) {
         case EPI_ACT: return umma_pick<EPI_ACT>(ctx, p, pdl, st);

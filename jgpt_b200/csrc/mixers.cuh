@@ -111,11 +111,17 @@ struct RouteArgs {
     int max_tiles, tile_rows;
 };
 int32_t launch_route(const RouteArgs &a, int rows, int pdl, cudaStream_t st);
+// out[row of a tile] = the row of h that the tile's list names, ld bf16 elements each.
+int32_t launch_moe_gather(const RouteArgs &a, const void *h, void *out, int ld, int pdl, cudaStream_t st);
 
 // ---- attn_gqa.cu -----------------------------------------------------------------------------------
 // Query heads in groups that share a key head.  Differential attention has two maps: a head's query and key are [map 1 | map 2],
 // each map is an attention of its own over the same values, the second one's result times lambda is taken off the first one's
 // and the difference brought to unit root mean square.  Padded sizes: DK per map, DV.
+// Rows of a page are stored the way shared memory wants them: 16-byte pieces permuted by the row, or a row of an odd number of
+// pieces, so that a page comes in as one bulk copy and eight rows are read without bank conflicts.
+__host__ __device__ constexpr int page_row(int D) { return D % 64 == 0 ? D : D + 8; }
+__host__ __device__ constexpr int page_chunk(int D, int row, int chunk) { return D % 64 == 0 ? chunk ^ (row & 7) : chunk; }
 enum HeadGate : int { GATE_NONE = 0, GATE_HEAD = 1, GATE_ELEMENT = 2 };
 struct AttnArgs {
     void *proj;         // [rows, ldp] projections of the layer
@@ -129,7 +135,7 @@ struct AttnArgs {
     const float2 *cs;   // [rows][half] cos and sin; the first 2 half elements of every head (map) turn; null: no rotation
     int half, interleaved;         // pairs (2 i, 2 i + 1), or (i, i + half)
     float lambda, diff_scale;
-    void *kv;           // this layer's pages: [block][kv head][K 16 x (maps DK) | V 16 x DV]
+    void *kv;           // this layer's pages: [block][kv head][K 16 x page_row(maps DK) | V 16 x page_row(DV)]
     const int *table;
     int n_blocks, mbs;
     void *out;          // [rows, ldo], head h at out_off + h * DV
@@ -137,7 +143,7 @@ struct AttnArgs {
     int sm_count;
     int *status;
     __host__ __device__ bool prepared() const { return q_norm || cs; }  // heads are normed or rotated on their way
-    __host__ __device__ int page_head() const { return kBlockTokens * (maps * DK + DV); }
+    __host__ __device__ int page_head() const { return kBlockTokens * (page_row(maps * DK) + page_row(DV)); }
 };
 int32_t launch_attention(bool f32, const StepDesc &d, const AttnArgs &a, int pdl, cudaStream_t st);
 bool attn_padded_head(int dim, int vdim, int maps, int *DK, int *DV);  // false: not supported

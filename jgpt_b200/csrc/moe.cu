@@ -1,94 +1,102 @@
 // Routing of the mixture of experts: a token's experts and their weights from its router logits, the rows of every expert, and the
 // row tiles of the experts' products.
 //
-// One launch: a warp per token picks its experts and takes a place in each one's list (lists have room for every row, since a token
-// picks an expert once); the block that finishes last turns the counts into offsets and tiles and leaves the counters at zero.
-// Places depend on the order of arrival, results do not: every row of a product stands alone.
+// One launch: a warp per token picks its experts, a block counts its tokens' picks and takes places in the experts' lists (lists
+// have room for every row, since a token picks an expert once); the block that finishes last turns the counts into offsets and
+// tiles and leaves the counters at zero.  Decode-sized steps are one block and need no counters.  Places depend on the order of
+// arrival, results do not: every row of a product stands alone.
+#include <algorithm>
+
 #include "mixers.cuh"
 #include "ptx.cuh"
 
 namespace jgpt {
 namespace mix {
 
-constexpr int kRouteWarps = 4;
+constexpr unsigned kAll = 0xffffffffu;
 
-// The largest value of the warp's v and its index, the lowest one among equals.
-__device__ __forceinline__ void warp_best(float &v, int &i) {
-#pragma unroll
-    for (int off = 16; off >= 1; off >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, v, off);
-        const int oi = __shfl_xor_sync(0xffffffffu, i, off);
-        if (ov > v || (ov == v && oi < i)) v = ov, i = oi;
-    }
-}
 __device__ __forceinline__ int warp_scan(int v) {  // inclusive
     const int lane = threadIdx.x & 31;
 #pragma unroll
     for (int off = 1; off < 32; off <<= 1) {
-        const int o = __shfl_up_sync(0xffffffffu, v, off);
+        const int o = __shfl_up_sync(kAll, v, off);
         if (lane >= off) v += o;
     }
     return v;
 }
+// Orders like the float, never 0: 0 stands for out of the question.
+__device__ __forceinline__ uint32_t order_key(float v) {
+    const uint32_t u = __float_as_uint(v);
+    return u & 0x80000000u ? max(~u, 1u) : u | 0x80000000u;
+}
 
-// Experts of one token by one warp: lane s gets the s-th choice and its weight.  score, choice: E values of shared memory each.
-__device__ __forceinline__ void choose_experts(const RouteArgs &a, const float *logits, float *score, float *choice, float *group, int &expert, float &weight) {
+// Lane l's entries are l, l + 32, ...: the best of all n keys, the lowest index among equals (n: none left).
+struct Best {
+    uint32_t key = 0;
+    int at = 0;
+    __device__ void scan(const uint32_t *keys, int n) {
+        key = 0, at = n;
+        for (int e = threadIdx.x & 31; e < n; e += 32)
+            if (keys[e] > key) key = keys[e], at = e;
+    }
+    __device__ int of_warp(int n) const {
+        const uint32_t top = __reduce_max_sync(kAll, key);
+        return top ? (int)__reduce_min_sync(kAll, key == top ? (unsigned)at : (unsigned)n) : n;
+    }
+};
+
+// Experts of one token by one warp: lane s gets the s-th choice (-1: none) and its weight.  score, choice: E words of shared memory
+// each, group: a word per group.
+__device__ __forceinline__ void choose_experts(const RouteArgs &a, const float *logits, float *score, uint32_t *choice, uint32_t *group, int &expert, float &weight) {
     const int lane = threadIdx.x & 31, E = a.experts + a.identity, size = E / a.groups;
     float mx = -INFINITY, sum = 0.f;
     for (int e = lane; e < E; e += 32) score[e] = logits[e], mx = fmaxf(mx, score[e]);
 #pragma unroll
-    for (int off = 16; off >= 1; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+    for (int off = 16; off >= 1; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(kAll, mx, off));
     for (int e = lane; e < E; e += 32) score[e] = expf(score[e] - mx), sum += score[e];
 #pragma unroll
-    for (int off = 16; off >= 1; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
-    for (int e = lane; e < E; e += 32) score[e] /= sum, choice[e] = score[e] + a.correction[e];
-    __syncwarp();
+    for (int off = 16; off >= 1; off >>= 1) sum += __shfl_xor_sync(kAll, sum, off);
+    for (int e = lane; e < E; e += 32) score[e] /= sum, choice[e] = order_key(score[e] + a.correction[e]);
+    Best best;
     if (a.keep < a.groups) {
+        __syncwarp();
         for (int g = lane; g < a.groups; g += 32) {
-            float best = -INFINITY;
-            for (int e = g * size; e < (g + 1) * size; e++) best = fmaxf(best, choice[e]);
-            group[g] = best;
+            uint32_t k = 0;
+            for (int e = g * size; e < (g + 1) * size; e++) k = max(k, choice[e]);
+            group[g] = k;
         }
-        __syncwarp();
         for (int k = 0; k < a.keep; k++) {
-            float v = -INFINITY;
-            int at = a.groups;
-            for (int g = lane; g < a.groups; g += 32)
-                if (group[g] > v) v = group[g], at = g;
-            warp_best(v, at);
-            if (lane == 0 && at < a.groups) group[at] = __int_as_float(0x7fc00000);  // NaN: taken, and no larger than anything
-            __syncwarp();
+            best.scan(group, a.groups);
+            const int at = best.of_warp(a.groups);
+            if (at < a.groups && (at & 31) == lane) group[at] = 0;
         }
-        for (int e = lane; e < E; e += 32)
-            if (!isnan(group[e / size])) choice[e] = -INFINITY;
         __syncwarp();
+        for (int e = lane; e < E; e += 32)
+            if (group[e / size]) choice[e] = 0;  // a group that was not taken
     }
     expert = -1, weight = 0.f;
     float total = 0.f;
+    best.scan(choice, E);
     for (int s = 0; s < a.top; s++) {
-        float v = -INFINITY;
-        int at = E;
-        for (int e = lane; e < E; e += 32)
-            if (choice[e] > v) v = choice[e], at = e;
-        warp_best(v, at);
-        if (at >= E) break;  // nothing comparable left
-        const float w = score[at];
+        const int at = best.of_warp(E);
+        if (at >= E) break;
+        const float w = __shfl_sync(kAll, best.at == at ? score[at] : 0.f, at & 31);
         total += w;
         if (lane == s) expert = at, weight = w;
-        if (lane == 0) choice[at] = -INFINITY;
-        __syncwarp();
+        if ((at & 31) == lane) choice[at] = 0, best.scan(choice, E);
     }
     weight /= total + 1e-20f;
+    __syncwarp();  // the words are free for the next token
 }
 
-// Offsets and tiles from the counts, by one block; the counters go back to zero.
-__device__ __forceinline__ void plan_tiles(const RouteArgs &a) {
+// Offsets and tiles from the experts' counts, by one warp.
+template <class Count>
+__device__ __forceinline__ void plan_tiles(const RouteArgs &a, const Count &count) {
     const int lane = threadIdx.x & 31;
-    if (threadIdx.x >= 32) return;
     int rows = 0, tiles = 0;
     for (int e0 = 0; e0 < a.experts; e0 += 32) {
         const int e = e0 + lane;
-        const int n = e < a.experts ? min(atomicExch(a.counts + e, 0), a.cap) : 0, nt = (n + a.tile_rows - 1) / a.tile_rows;
+        const int n = e < a.experts ? min(count(e), a.cap) : 0, nt = (n + a.tile_rows - 1) / a.tile_rows;
         const int rs = warp_scan(n), ts = warp_scan(nt), row0 = rows + rs - n, t0 = tiles + ts - nt;
         if (e < a.experts) {
             a.offsets[e] = row0;
@@ -96,56 +104,105 @@ __device__ __forceinline__ void plan_tiles(const RouteArgs &a) {
                 if (t0 + t < a.max_tiles)
                     a.tiles[t0 + t] = nt::RowTile{e, row0 + t * a.tile_rows, min(row0 + n, row0 + (t + 1) * a.tile_rows), e * a.cap + t * a.tile_rows};
         }
-        rows += __shfl_sync(0xffffffffu, rs, 31), tiles += __shfl_sync(0xffffffffu, ts, 31);
+        rows += __shfl_sync(kAll, rs, 31), tiles += __shfl_sync(kAll, ts, 31);
     }
     if (lane == 0) *a.n_tiles = min(tiles, a.max_tiles);
 }
 
-__global__ void __launch_bounds__(32 * kRouteWarps) route_kernel(const RouteArgs a, int rows, int pdl) {
-    extern __shared__ float route_smem[];
+__host__ __device__ __forceinline__ int route_words(const RouteArgs &a) { return 2 * (a.experts + a.identity) + a.groups; }  // of a warp
+
+__global__ void __launch_bounds__(1024) route_kernel(const RouteArgs a, int rows, int per_block, int pdl) {
+    extern __shared__ uint32_t route_smem[];
     __shared__ int last;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, E = a.experts + a.identity, r = blockIdx.x * kRouteWarps + warp;
-    float *score = route_smem + warp * (2 * E + a.groups), *choice = score + E, *group = choice + E;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5, E = a.experts + a.identity;
+    const int r0 = blockIdx.x * per_block, n = min(per_block, rows - r0);
+    float *score = reinterpret_cast<float *>(route_smem + warp * route_words(a));
+    uint32_t *choice = reinterpret_cast<uint32_t *>(score) + E, *group = choice + E;
+    int *counts = reinterpret_cast<int *>(route_smem) + warps * route_words(a), *base = counts + a.experts;
+    RouteSlot *slots = reinterpret_cast<RouteSlot *>(base + a.experts);
     if (pdl & 2) griddep_launch_dependents();
+    for (int e = tid; e < a.experts; e += blockDim.x) counts[e] = 0;
     if (pdl & 1) griddep_wait();
-    if (r < rows) {
+    __syncthreads();
+    for (int t = warp; t < n; t += warps) {
+        const float *logits = a.logits + (size_t)(r0 + t) * a.ld;
         int expert;
         float weight;
-        const float *logits = a.logits + (size_t)r * a.ld;
         choose_experts(a, logits, score, choice, group, expert, weight);
-        const bool real = lane < a.top && expert >= 0 && expert < a.experts;
-        int rank = -1;
-        if (real) {
-            rank = atomicAdd(a.counts + expert, 1);
-            if (rank < a.cap) a.list[(size_t)expert * a.cap + rank] = r;
-        }
-        float id = lane < a.top && expert >= a.experts ? weight : 0.f;
+        const bool real = expert >= 0 && expert < a.experts;
+        if (lane < a.top) slots[t * a.top + lane] = RouteSlot{real ? expert : -1, real ? atomicAdd(counts + expert, 1) : -1, real ? weight : 0.f};
+        float id = expert >= a.experts ? weight : 0.f;
 #pragma unroll
-        for (int off = 16; off >= 1; off >>= 1) id += __shfl_xor_sync(0xffffffffu, id, off);
-        if (lane < a.top) a.slots[(size_t)r * a.top + lane] = RouteSlot{real ? expert : -1, rank, real ? weight : 0.f};
-        if (lane == 0) a.row_weights[r] = make_float2(id, a.shared ? 1.f / (1.f + expf(-logits[E])) : 0.f);
+        for (int off = 16; off >= 1; off >>= 1) id += __shfl_xor_sync(kAll, id, off);
+        if (lane == 0) a.row_weights[r0 + t] = make_float2(id, a.shared ? 1.f / (1.f + expf(-logits[E])) : 0.f);
     }
-    __threadfence();
     __syncthreads();
-    if (threadIdx.x == 0) last = atomicAdd(a.ticket, 1) == (int)gridDim.x - 1;
+    const bool alone = gridDim.x == 1;
+    for (int e = tid; e < a.experts; e += blockDim.x) base[e] = alone || counts[e] == 0 ? 0 : atomicAdd(a.counts + e, counts[e]);
     __syncthreads();
-    if (!last) return;
+    for (int i = tid; i < n * a.top; i += blockDim.x) {
+        RouteSlot s = slots[i];
+        if (s.expert >= 0) {
+            s.rank += base[s.expert];
+            if (s.rank < a.cap) a.list[(size_t)s.expert * a.cap + s.rank] = r0 + i / a.top;
+        }
+        a.slots[(size_t)r0 * a.top + i] = s;
+    }
+    if (alone) {
+        if (warp == 0) plan_tiles(a, [&](int e) { return counts[e]; });
+        return;
+    }
+    if (tid == 0) __threadfence(), last = atomicAdd(a.ticket, 1) == (int)gridDim.x - 1;
+    __syncthreads();
+    if (!last || warp != 0) return;
     __threadfence();
-    if (threadIdx.x == 0) *a.ticket = 0;
-    plan_tiles(a);
+    if (lane == 0) *a.ticket = 0;
+    plan_tiles(a, [&](int e) { return atomicExch(a.counts + e, 0); });
 }
 
-int32_t launch_route(const RouteArgs &a, int rows, int pdl, cudaStream_t st) {
-    const size_t smem = sizeof(float) * kRouteWarps * (size_t)(2 * (a.experts + a.identity) + a.groups);
-    JGPT_REQUIRE(smem <= 47 * 1024 && a.top <= 32, JGPT_ERR_UNSUPPORTED, "%d router outputs, %d chosen", a.experts + a.identity, a.top);
+// A block per 16 rows of a tile.  (Nothing here is __restrict__: reads of what counts as constant may move up past the wait.)
+__global__ void __launch_bounds__(256) moe_gather_kernel(const RouteArgs a, const uint4 *h, uint4 *out, int chunks, int pdl) {
+    if (pdl & 2) griddep_launch_dependents();
+    if (pdl & 1) griddep_wait();
+    if ((int)blockIdx.x >= *a.n_tiles) return;
+    const nt::RowTile t = a.tiles[blockIdx.x];
+    const int row0 = t.row0 + blockIdx.y * 16, n = min(16, t.row_end - row0), *from = a.list + t.src0 + blockIdx.y * 16;
+    for (int i0 = threadIdx.x; i0 < n * chunks; i0 += 8 * 256) {
+        uint4 x[8];
+#pragma unroll
+        for (int k = 0; k < 8; k++)
+            if (const int i = i0 + 256 * k; i < n * chunks) x[k] = h[(size_t)from[i / chunks] * chunks + i % chunks];
+#pragma unroll
+        for (int k = 0; k < 8; k++)
+            if (const int i = i0 + 256 * k; i < n * chunks) out[(size_t)row0 * chunks + i] = x[k];
+    }
+}
+
+template <class... Args>
+static int32_t launch(void (*kern)(Args...), dim3 grid, int threads, size_t smem, int pdl, cudaStream_t st, Args... args) {
     cudaLaunchConfig_t cfg = {};
     cudaLaunchAttribute attr[1];
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
     attr[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.gridDim = dim3((unsigned)((rows + kRouteWarps - 1) / kRouteWarps)), cfg.blockDim = dim3(32 * kRouteWarps), cfg.dynamicSmemBytes = smem, cfg.stream = st;
+    cfg.gridDim = grid, cfg.blockDim = dim3((unsigned)threads), cfg.dynamicSmemBytes = smem, cfg.stream = st;
     cfg.attrs = attr, cfg.numAttrs = (pdl & 1) ? 1 : 0;
-    JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, route_kernel, a, rows, pdl));
+    JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, kern, args...));
     return JGPT_OK;
+}
+
+int32_t launch_route(const RouteArgs &a, int rows, int pdl, cudaStream_t st) {
+    const bool alone = rows <= 128 && sizeof(RouteSlot) * (size_t)rows * a.top <= 24 * 1024;
+    const int per_block = alone ? rows : 32;
+    auto smem = [&](int warps) { return 4 * ((size_t)warps * route_words(a) + 2 * (size_t)a.experts) + sizeof(RouteSlot) * (size_t)per_block * a.top; };
+    int warps = std::min(alone ? 32 : 16, per_block);
+    while (warps > 1 && smem(warps) > 47 * 1024) warps /= 2;
+    JGPT_REQUIRE(smem(warps) <= 47 * 1024 && a.top <= 32, JGPT_ERR_UNSUPPORTED, "%d router outputs, %d chosen", a.experts + a.identity, a.top);
+    return launch(route_kernel, dim3((unsigned)((rows + per_block - 1) / per_block)), 32 * warps, smem(warps), pdl, st, a, rows, per_block, pdl);
+}
+
+int32_t launch_moe_gather(const RouteArgs &a, const void *h, void *out, int ld, int pdl, cudaStream_t st) {
+    return launch(moe_gather_kernel, dim3((unsigned)a.max_tiles, (unsigned)((a.tile_rows + 15) / 16)), 256, 0, pdl, st, a,
+                  reinterpret_cast<const uint4 *>(h), reinterpret_cast<uint4 *>(out), ld / 8, pdl);
 }
 
 }  // namespace mix

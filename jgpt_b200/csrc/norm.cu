@@ -75,7 +75,7 @@ __global__ void __launch_bounds__(kNormThreads) embed_norm_kernel(const int *__r
 }
 
 template <class AT>
-__global__ void __launch_bounds__(kNormThreads) layer_norm_kernel(const float *__restrict__ x, const int *__restrict__ rowsel, const NormW w,
+__global__ void __launch_bounds__(kNormThreads) layer_norm_kernel(const float *x, const int *__restrict__ rowsel, const NormW w,
                                                                   float eps, AT *__restrict__ h, int W, int ldh, int pdl) {
     extern __shared__ float row[];
     __shared__ float red[kNormThreads / 32];
@@ -259,7 +259,7 @@ __device__ __forceinline__ void add_scaled(float4 &s, float w, const float4 &v) 
 constexpr int kMaxTop = 32;
 
 template <class AT, bool MOE>
-__global__ void __launch_bounds__(kNormThreads) post_norm_kernel(float *__restrict__ x, const float *__restrict__ gamma, float eps, AT *__restrict__ h, const MoeSum m,
+__global__ void __launch_bounds__(kNormThreads) post_norm_kernel(float *x, const float *__restrict__ gamma, float eps, AT *__restrict__ h, const MoeSum m,
                                                                  int W, int ldh, int pdl) {
     extern __shared__ __align__(16) float row[];
     __shared__ float red[kNormThreads / 32], weight[kMaxTop];
