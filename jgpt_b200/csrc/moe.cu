@@ -3,10 +3,8 @@
 //
 // One launch: a warp per token picks its experts, a block counts its tokens' picks and takes places in the experts' lists (lists
 // have room for every row, since a token picks an expert once); the block that finishes last turns the counts into offsets and
-// tiles and leaves the counters at zero.  Decode-sized steps are one block and need no counters.  Places depend on the order of
+// tiles and leaves the counters at zero.  Places depend on the order of
 // arrival, results do not: every row of a product stands alone.
-#include <algorithm>
-
 #include "mixers.cuh"
 #include "ptx.cuh"
 
@@ -14,6 +12,7 @@ namespace jgpt {
 namespace mix {
 
 constexpr unsigned kAll = 0xffffffffu;
+constexpr int kRouteWarps = 8;
 
 __device__ __forceinline__ int warp_scan(int v) {  // inclusive
     const int lane = threadIdx.x & 31;
@@ -30,63 +29,72 @@ __device__ __forceinline__ uint32_t order_key(float v) {
     return u & 0x80000000u ? max(~u, 1u) : u | 0x80000000u;
 }
 
-// Lane l's entries are l, l + 32, ...: the best of all n keys, the lowest index among equals (n: none left).
-struct Best {
-    uint32_t key = 0;
-    int at = 0;
-    __device__ void scan(const uint32_t *keys, int n) {
-        key = 0, at = n;
-        for (int e = threadIdx.x & 31; e < n; e += 32)
-            if (keys[e] > key) key = keys[e], at = e;
-    }
-    __device__ int of_warp(int n) const {
-        const uint32_t top = __reduce_max_sync(kAll, key);
-        return top ? (int)__reduce_min_sync(kAll, key == top ? (unsigned)at : (unsigned)n) : n;
-    }
-};
+// The warp's best key and its index, the lowest one among equals; -1: no key but zeros.
+__device__ __forceinline__ int best_of_warp(uint32_t key, int at) {
+    const uint32_t top = __reduce_max_sync(kAll, key);
+    return top ? (int)__reduce_min_sync(kAll, key == top ? (unsigned)at : kAll) : -1;
+}
 
-// Experts of one token by one warp: lane s gets the s-th choice (-1: none) and its weight.  score, choice: E words of shared memory
-// each, group: a word per group.
-__device__ __forceinline__ void choose_experts(const RouteArgs &a, const float *logits, float *score, uint32_t *choice, uint32_t *group, int &expert, float &weight) {
+// Experts of one token by one warp, which holds outputs lane + 32 i: lane s gets the s-th choice (-1: none) and its weight.
+// group: a word of shared memory per group.
+template <int NPL>
+__device__ __forceinline__ void choose_experts(const RouteArgs &a, const float *logits, uint32_t *group, int &expert, float &weight) {
     const int lane = threadIdx.x & 31, E = a.experts + a.identity, size = E / a.groups;
-    float mx = -INFINITY, sum = 0.f;
-    for (int e = lane; e < E; e += 32) score[e] = logits[e], mx = fmaxf(mx, score[e]);
+    float score[NPL], mx = -INFINITY, sum = 0.f;
+    uint32_t key[NPL];
+#pragma unroll
+    for (int i = 0; i < NPL; i++) score[i] = lane + 32 * i < E ? logits[lane + 32 * i] : -INFINITY, mx = fmaxf(mx, score[i]);
 #pragma unroll
     for (int off = 16; off >= 1; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(kAll, mx, off));
-    for (int e = lane; e < E; e += 32) score[e] = expf(score[e] - mx), sum += score[e];
+#pragma unroll
+    for (int i = 0; i < NPL; i++) score[i] = expf(score[i] - mx), sum += score[i];
 #pragma unroll
     for (int off = 16; off >= 1; off >>= 1) sum += __shfl_xor_sync(kAll, sum, off);
-    for (int e = lane; e < E; e += 32) score[e] /= sum, choice[e] = order_key(score[e] + a.correction[e]);
-    Best best;
+    const float inv = 1.f / sum;
+#pragma unroll
+    for (int i = 0; i < NPL; i++) score[i] *= inv, key[i] = lane + 32 * i < E ? order_key(score[i] + __ldg(a.correction + lane + 32 * i)) : 0;
     if (a.keep < a.groups) {
+        for (int g = lane; g < a.groups; g += 32) group[g] = 0;
         __syncwarp();
-        for (int g = lane; g < a.groups; g += 32) {
-            uint32_t k = 0;
-            for (int e = g * size; e < (g + 1) * size; e++) k = max(k, choice[e]);
-            group[g] = k;
+        int mine[NPL];
+#pragma unroll
+        for (int i = 0; i < NPL; i++) {
+            mine[i] = lane + 32 * i < E ? (lane + 32 * i) / size : 0;
+            if (key[i]) atomicMax(group + mine[i], key[i]);
         }
+        __syncwarp();
         for (int k = 0; k < a.keep; k++) {
-            best.scan(group, a.groups);
-            const int at = best.of_warp(a.groups);
-            if (at < a.groups && (at & 31) == lane) group[at] = 0;
+            uint32_t top = 0;
+            int at = 0;
+            for (int g = lane; g < a.groups; g += 32)
+                if (group[g] > top) top = group[g], at = g;
+            const int taken = best_of_warp(top, at);
+            if (taken >= 0 && (taken & 31) == lane) group[taken] = 0;
         }
         __syncwarp();
-        for (int e = lane; e < E; e += 32)
-            if (group[e / size]) choice[e] = 0;  // a group that was not taken
+#pragma unroll
+        for (int i = 0; i < NPL; i++)
+            if (group[mine[i]]) key[i] = 0;  // a group that was not taken
+        __syncwarp();                        // the words are free for the next token
     }
     expert = -1, weight = 0.f;
     float total = 0.f;
-    best.scan(choice, E);
     for (int s = 0; s < a.top; s++) {
-        const int at = best.of_warp(E);
-        if (at >= E) break;
-        const float w = __shfl_sync(kAll, best.at == at ? score[at] : 0.f, at & 31);
-        total += w;
-        if (lane == s) expert = at, weight = w;
-        if ((at & 31) == lane) choice[at] = 0, best.scan(choice, E);
+        uint32_t top = 0;
+        int at = 0;
+        float w = 0.f;
+#pragma unroll
+        for (int i = 0; i < NPL; i++)
+            if (key[i] > top) top = key[i], at = lane + 32 * i, w = score[i];
+        const int taken = best_of_warp(top, at);
+        if (taken < 0) break;
+        w = __shfl_sync(kAll, w, taken & 31), total += w;
+        if (lane == s) expert = taken, weight = w;
+#pragma unroll
+        for (int i = 0; i < NPL; i++)
+            if (lane + 32 * i == taken) key[i] = 0;
     }
     weight /= total + 1e-20f;
-    __syncwarp();  // the words are free for the next token
 }
 
 // Offsets and tiles from the experts' counts, by one warp.
@@ -109,26 +117,24 @@ __device__ __forceinline__ void plan_tiles(const RouteArgs &a, const Count &coun
     if (lane == 0) *a.n_tiles = min(tiles, a.max_tiles);
 }
 
-__host__ __device__ __forceinline__ int route_words(const RouteArgs &a) { return 2 * (a.experts + a.identity) + a.groups; }  // of a warp
-
-__global__ void __launch_bounds__(1024) route_kernel(const RouteArgs a, int rows, int per_block, int pdl) {
+template <int NPL>
+__global__ void __launch_bounds__(32 * kRouteWarps) route_kernel(const RouteArgs a, int rows, int per_block, int pdl) {
     extern __shared__ uint32_t route_smem[];
     __shared__ int last;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5, E = a.experts + a.identity;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, E = a.experts + a.identity;
     const int r0 = blockIdx.x * per_block, n = min(per_block, rows - r0);
-    float *score = reinterpret_cast<float *>(route_smem + warp * route_words(a));
-    uint32_t *choice = reinterpret_cast<uint32_t *>(score) + E, *group = choice + E;
-    int *counts = reinterpret_cast<int *>(route_smem) + warps * route_words(a), *base = counts + a.experts;
+    uint32_t *group = route_smem + warp * a.groups;
+    int *counts = reinterpret_cast<int *>(route_smem) + kRouteWarps * a.groups, *base = counts + a.experts;
     RouteSlot *slots = reinterpret_cast<RouteSlot *>(base + a.experts);
     if (pdl & 2) griddep_launch_dependents();
     for (int e = tid; e < a.experts; e += blockDim.x) counts[e] = 0;
     if (pdl & 1) griddep_wait();
     __syncthreads();
-    for (int t = warp; t < n; t += warps) {
+    for (int t = warp; t < n; t += kRouteWarps) {
         const float *logits = a.logits + (size_t)(r0 + t) * a.ld;
         int expert;
         float weight;
-        choose_experts(a, logits, score, choice, group, expert, weight);
+        choose_experts<NPL>(a, logits, group, expert, weight);
         const bool real = expert >= 0 && expert < a.experts;
         if (lane < a.top) slots[t * a.top + lane] = RouteSlot{real ? expert : -1, real ? atomicAdd(counts + expert, 1) : -1, real ? weight : 0.f};
         float id = expert >= a.experts ? weight : 0.f;
@@ -191,13 +197,15 @@ static int32_t launch(void (*kern)(Args...), dim3 grid, int threads, size_t smem
 }
 
 int32_t launch_route(const RouteArgs &a, int rows, int pdl, cudaStream_t st) {
-    const bool alone = rows <= 128 && sizeof(RouteSlot) * (size_t)rows * a.top <= 24 * 1024;
-    const int per_block = alone ? rows : 32;
-    auto smem = [&](int warps) { return 4 * ((size_t)warps * route_words(a) + 2 * (size_t)a.experts) + sizeof(RouteSlot) * (size_t)per_block * a.top; };
-    int warps = std::min(alone ? 32 : 16, per_block);
-    while (warps > 1 && smem(warps) > 47 * 1024) warps /= 2;
-    JGPT_REQUIRE(smem(warps) <= 47 * 1024 && a.top <= 32, JGPT_ERR_UNSUPPORTED, "%d router outputs, %d chosen", a.experts + a.identity, a.top);
-    return launch(route_kernel, dim3((unsigned)((rows + per_block - 1) / per_block)), 32 * warps, smem(warps), pdl, st, a, rows, per_block, pdl);
+    // few tokens: one per warp, and one block for as many as it has warps; many: four per warp
+    const int per_block = rows <= 512 ? kRouteWarps : 4 * kRouteWarps, E = a.experts + a.identity;
+    const size_t smem = 4 * ((size_t)kRouteWarps * a.groups + 2 * (size_t)a.experts) + sizeof(RouteSlot) * (size_t)per_block * a.top;
+    JGPT_REQUIRE(smem <= 47 * 1024 && a.top <= 32 && E <= 1024, JGPT_ERR_UNSUPPORTED, "%d router outputs, %d chosen", E, a.top);
+    auto run = [&](auto kern) { return launch(kern, dim3((unsigned)((rows + per_block - 1) / per_block)), 32 * kRouteWarps, smem, pdl, st, a, rows, per_block, pdl); };
+    if (E <= 32) return run(route_kernel<1>);
+    if (E <= 64) return run(route_kernel<2>);
+    if (E <= 128) return run(route_kernel<4>);
+    return E <= 256 ? run(route_kernel<8>) : run(route_kernel<32>);
 }
 
 int32_t launch_moe_gather(const RouteArgs &a, const void *h, void *out, int ld, int pdl, cudaStream_t st) {

@@ -131,7 +131,7 @@ def nefipel_config(width):
     moe = {"kind": "moe", "expert": {"ff": width * 3 // 8}, "shared": {"ff": width * 9 // 8},
            "router": {"experts": 60, "identity": 4, "top": 8, "groups": {"count": 8, "keep": 4}}}
     block = [{"type": "attention", "mixer": att, "mlp": {"kind": "dense", "ff": width * 11 // 4}}, {"type": "attention_2", "mixer": diff, "mlp": moe}]
-    return {"architecture": "Nefipel", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6}, "postln_alpha": 2.5, "embedding": {"scale": 16.0},
+    return {"architecture": "Nefipel", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6}, "postln_alpha": 2.5, "embedding": {"scale": 8.0},
             "layers": block * (LAYERS // 2)}
 
 

@@ -107,7 +107,7 @@ def _alone(ctx, layer, dtype, sizes=(200, 1, 2, 40, 7, 50), width=64, edit=None,
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("kw", [dict(), dict(heads=1, kv_heads=1, dim=8, vdim=8, rot_dims=2), dict(heads=33, kv_heads=1, dim=16, vdim=24),
-                                dict(dim=128, vdim=128, rot_dims=128), dict(dim=90, vdim=33, rot_dims=50), dict(dim=64, vdim=32, rot_dims=32),
+                                dict(dim=128, vdim=128, rot_dims=128), dict(dim=90, vdim=33, rot_dims=50), dict(dim=60, vdim=30, rot_dims=28),
                                 dict(heads=2, dim=130, vdim=190, rot_dims=20), dict(dim=31, vdim=60, rot_dims=6)])
 def test_gated_attention_alone(ctx, kw, dtype):
     _alone(ctx, nc.att(mlp=None, **kw), dtype)
@@ -115,7 +115,7 @@ def test_gated_attention_alone(ctx, kw, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("kw", [dict(), dict(heads=1, kv_heads=1, dim=6, vdim=16), dict(heads=18, kv_heads=1, dim=16, vdim=32), dict(dim=64, vdim=128, yarn=None),
-                                dict(dim=48, vdim=96, rot_dims=48), dict(heads=9, kv_heads=3, dim=128, vdim=256), dict(dim=90, vdim=180, rot_dims=10),
+                                dict(dim=44, vdim=90, rot_dims=44), dict(heads=9, kv_heads=3, dim=128, vdim=256), dict(dim=90, vdim=180, rot_dims=10),
                                 dict(dim=128, vdim=100, rot_dims=62), dict(dim=24, vdim=50, at=0.9)])
 def test_differential_attention_alone(ctx, kw, dtype):
     _alone(ctx, nc.diff(mlp=None, **kw), dtype)
