@@ -23,6 +23,7 @@ GATE_NONE, GATE_HEAD, GATE_ELEMENT = range(3)
 NO_LIMIT = 1 << 30  # positions of a model without a table of them
 DTYPES = {"bfloat16": 0, "float32": 1}
 BLOCK_TOKENS = 16
+MAX_BRANCHES = 2
 
 
 class _MixerSpec(C.Structure):
@@ -38,7 +39,7 @@ class _MoeSpec(C.Structure):
 
 
 class _LayerSpec(C.Structure):
-    _fields_ = [("n_branches", C.c_int32), ("branch", _MixerSpec * 2), ("ff", C.c_int32), ("ff_kind", C.c_int32), ("moe", _MoeSpec)]
+    _fields_ = [("n_branches", C.c_int32), ("branch", _MixerSpec * MAX_BRANCHES), ("ff", C.c_int32), ("ff_kind", C.c_int32), ("moe", _MoeSpec)]
 
 
 class _DecoderSpec(C.Structure):
@@ -55,7 +56,6 @@ W_NORM1, W_NORM1_B, W_NORM2, W_NORM2_B, W_FF_GATE, W_FF_UP, W_FF_DOWN, W_LS1, W_
  W_CONV_V, W_MU_R, W_MU_K, W_MU_V, W_MU_G, W_MU_W, W_BONUS, W_LOWER, W_F, W_DQ, W_DQ_NORM, W_UQ, W_DKV, W_DKV_NORM, W_UK, W_UV,
  W_FF_ACT, W_Q_BIAS, W_K_BIAS, W_V_BIAS, W_Q_NORM, W_K_NORM, W_LQ1, W_LK1, W_LQ2, W_LK2) = range(20, 61)
 W_ROUTER, W_CORRECTION, W_SHARED_GATE, W_SHARED_UP, W_SHARED_DOWN, W_EXPERT_UP, W_EXPERT_DOWN = range(64, 71)
-MAX_BRANCHES = 2
 
 
 @dataclass

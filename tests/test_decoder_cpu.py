@@ -80,13 +80,13 @@ def test_abi_structures_match_the_header():
     def fields(name):
         body = re.search(r"typedef struct \{([^{}]*)\} %s;" % name, src).group(1)
         out = []
-        for t, names in re.findall(r"(int32_t|float|double|jgpt_mixer_spec)\s+([^;]+);", body):
+        for t, names in re.findall(r"(int32_t|float|double|jgpt_\w+_spec)\s+([^;]+);", body):
             out += [(n.strip().split("[")[0], t) for n in names.split(",")]
         return out
 
-    ct = {C.c_int32: "int32_t", C.c_float: "float", C.c_double: "double"}
-    for name, cls in (("jgpt_mixer_spec", D._MixerSpec), ("jgpt_layer_spec", D._LayerSpec), ("jgpt_decoder_spec", D._DecoderSpec)):
-        assert fields(name) == [(n, ct.get(t, "jgpt_mixer_spec")) for n, t in cls._fields_], name
+    ct = {C.c_int32: "int32_t", C.c_float: "float", C.c_double: "double", D._MixerSpec * D.MAX_BRANCHES: "jgpt_mixer_spec", D._MoeSpec: "jgpt_moe_spec"}
+    for name, cls in (("jgpt_mixer_spec", D._MixerSpec), ("jgpt_moe_spec", D._MoeSpec), ("jgpt_layer_spec", D._LayerSpec), ("jgpt_decoder_spec", D._DecoderSpec)):
+        assert fields(name) == [(n, ct[t]) for n, t in cls._fields_], name
     roles = re.search(r"JGPT_W_EMBED = 0.*?\};", src, re.S).group(0)
     at, value = -1, {}
     for n, v in re.findall(r"(JGPT_W_\w+)(?:\s*=\s*(\d+))?", roles):
