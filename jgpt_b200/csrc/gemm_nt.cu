@@ -241,7 +241,9 @@ template <int EPI, bool GROUPED = false>
 static int32_t small_dispatch(const Ctx *ctx, const Problem *p, int n, int pdl, cudaStream_t st) {
     SmallArgs a{};
     a.n = n, a.pdl = pdl;
-    const int M = p[0].M, tall = GROUPED ? p[0].grp.rows : M;
+    const int M = p[0].M;
+    // few columns (a router's): lower tiles, so that the launch has more CTAs
+    const int tall = GROUPED ? p[0].grp.rows : (n == 1 && p[0].N <= 256 ? std::min(M, 32) : M);
     const int mt = tall <= 16 ? 1 : (tall <= 32 ? 2 : 4), bn = mt == 4 ? 64 : 32, max_split = mt == 4 ? 4 : kMaxSplit;
     int tiles = 0, K = 0;
     for (int i = 0; i < n; i++) {
