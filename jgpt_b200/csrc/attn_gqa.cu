@@ -50,7 +50,7 @@ __device__ __forceinline__ void prepare_head(float (&x)[8], const AT *src, int p
 #pragma unroll
         for (int e = 0; e < 8; e += 2)
             if (j0 + e < 2 * h.half) {
-                const float2 t = __ldg(h.cs + ((j0 + e) >> 1));
+                const float2 t = h.cs[((j0 + e) >> 1)];
                 const float u = x[e], v = x[e + 1];
                 x[e] = u * t.x - v * t.y, x[e + 1] = v * t.x + u * t.y;
             }
@@ -62,7 +62,7 @@ __device__ __forceinline__ void prepare_head(float (&x)[8], const AT *src, int p
         for (int e = 0; e < 8; e++) {
             const float y = __shfl_sync(0xffffffffu, x[e], other);
             if (!turns) continue;
-            const float2 t = __ldg(h.cs + (first ? j0 + e : j0 + e - h.half));
+            const float2 t = h.cs[(first ? j0 + e : j0 + e - h.half)];
             x[e] = first ? x[e] * t.x - y * t.y : x[e] * t.x + y * t.y;
         }
     } else {
@@ -70,7 +70,7 @@ __device__ __forceinline__ void prepare_head(float (&x)[8], const AT *src, int p
         for (int e = 0; e < 8; e++) {
             const int j = j0 + e, p = j < h.half ? j + h.half : j - h.half;
             if (j >= 2 * h.half) continue;
-            const float2 t = __ldg(h.cs + (j < h.half ? j : p));
+            const float2 t = h.cs[(j < h.half ? j : p)];
             const float y = act_load(src + p) * inv * (h.w ? __ldg(h.w + p) : 1.f);
             x[e] = j < h.half ? x[e] * t.x - y * t.y : x[e] * t.x + y * t.y;
         }
