@@ -339,7 +339,10 @@ JGPT_API int32_t jgpt_generate_greedy_rolling(jgpt_model model, jgpt_kvpool pool
  * norms are layer norms with weight and bias or RMS norms with weight, m is residual_mult, the factors per column ls1, ls2 are
  * there with layer_scale.  With depth_average what goes on from layer i is sum over j <= i + 1 of dwa_i[j] X_j, X_0 the
  * embedding and X_(i+1) the result of layer i.  With norm_after the parts read x itself and the norms come behind the sums:
- * x <- norm1(residual_scale * x + sum of mixers(x)), then x <- norm2(residual_scale * x + ff(x)); RMS norms.
+ * x <- norm1(residual_scale * x + sum of mixers(x)), then x <- norm2(residual_scale * x + ff(x)); RMS norms.  With norm_both there
+ * are norms on either side: x += m * post1(g1 * sum of mixers(h)), h = norm1(x), then x += m * post2(g2 * ff(h)), h = norm2(x); with
+ * residual_gate g = sigmoid(W_rg h + b) element by element (else 1); with token_shift the mixers read h + (h' - h) * shift, h'
+ * being the h of the token before (zeros for the first).
  * ------------------------------------------------------------------------------------------- */
 enum {
     JGPT_MIX_ATTENTION = 1, /* softmax attention over paged K/V (all positions before the query or those of its chunk); biases, norms
@@ -349,11 +352,19 @@ enum {
     JGPT_MIX_HGRN2 = 4,     /* S <- diag(f) S + (1 - f) v^T, f = l + (1 - l) sigmoid(W_f h + bias); no output gate */
     JGPT_MIX_WKV = 5,       /* o = (S + diag(u) k v^T)^T r, S <- diag(w) S + k v^T, w = exp(-exp(W_a2 tanh(W_a1 h_w) + bias)); r, k,
                                v, g and w each read their own mix of h with the previous token's h; only layer norm kind RMS */
-    JGPT_MIX_LATENT = 6     /* softmax attention on a normed latent and one rotated key part shared by the heads, sliding window */
+    JGPT_MIX_LATENT = 6,    /* softmax attention on a normed latent and one rotated key part shared by the heads, sliding window */
+    JGPT_MIX_GENERAL_DELTA = 7 /* S <- diag(w) S - (a u) (u^T S) + k v^T with the old S on the right and u = k / |k|, o = S^T r;
+                               w = exp(-rate sigmoid(W_a2 tanh(W_a1 h) + bias)), a = sigmoid(W_b h + bias) per key channel */
 };
+/* Norm of the query and key rows of attention: none; of every head (map) with JGPT_W_Q_NORM / _K_NORM [dim]; of all heads' rows
+ * at once with weights of that size; of every head without weights. */
+enum { JGPT_QK_NORM_NONE = 0, JGPT_QK_NORM_HEAD = 1, JGPT_QK_NORM_ALL = 2, JGPT_QK_NORM_UNIT = 3 };
+/* A score that takes part in the sum under the softmax weights and has no value: none; JGPT_W_SINK [heads]; 0. */
+enum { JGPT_SINK_NONE = 0, JGPT_SINK_LEARNED = 1, JGPT_SINK_ZERO = 2 };
 enum { JGPT_NORM_LAYER = 0, JGPT_NORM_RMS = 1 };
 enum { JGPT_FF_GATED_GELU = 0 /* W_down (gelu_tanh(W_gate h) * (W_up h)) */,
        JGPT_FF_GATED_RELU = 2 /* W_down (relu(W_gate h) * (W_up h)) */,
+       JGPT_FF_RELU2 = 4 /* W_down relu(W_up h)^2 */,
        JGPT_FF_MOE = 3 /* a mixture of experts W_down act(W_up h), see jgpt_moe_spec */,
        JGPT_FF_XIELU = 1 /* W_down xielu(W_up h), xielu(z) = a z^2 + z / 2 (z > 0), b (e^z - 1 - z) + z / 2, a = softplus(p), b = 1/2 + softplus(q) */ };
 enum { JGPT_ACT_RELU = 0, JGPT_ACT_RELU2 = 1 /* relu(z)^2 */, JGPT_ACT_GELU_TANH = 2 };
@@ -371,7 +382,7 @@ typedef struct {
     float score_scale;        /* attention */
     float tau;                /* gla */
     float out_scale;
-    int32_t window;           /* latent: position i sees j with 0 <= i - j < window; 0: every j <= i */
+    int32_t window;           /* attention, latent: position i sees j with 0 <= i - j < window; 0: every j <= i */
     int32_t q_rank, kv_rank;  /* latent: sizes of the query and key latents (kv_rank up to 512) */
     int32_t rot_dim;          /* latent: size of the rotated part of a query head and of the shared key part (up to 128) */
     int32_t rot_dims;         /* of it the first rot_dims turn: dimension i with i + rot_dims / 2 */
@@ -382,10 +393,14 @@ typedef struct {
     /* attention only; with rot_dims > 0 the first rot_dims dimensions of every query and key head (map) turn */
     int32_t rot_interleaved;  /* pairs (2 i, 2 i + 1) instead of (i, i + rot_dims / 2) */
     int32_t qkv_bias;         /* JGPT_W_Q_BIAS, _K_BIAS, _V_BIAS are added in the projections */
-    int32_t qk_norm;          /* RMS norm of every query and key head (map) with JGPT_W_Q_NORM / _K_NORM [dim], before the rotation */
+    int32_t qk_norm;          /* JGPT_QK_NORM_*: RMS norm of queries and keys in front of the rotation */
     int32_t maps;             /* 0, 1: one; 2: differential, q and k hold [map 1 | map 2] per head: o = a1 - lambda a2 with lambda =
                                  exp(lq1 . lk1) - exp(lq2 . lk2) + diff, then o / rms(o) * (1 - diff); dim up to 128 then */
     float diff;
+    int32_t keep;             /* with window: every position also sees the first `keep` */
+    int32_t sink;             /* JGPT_SINK_* */
+    int32_t v_mix;            /* values become (1 - l) v + l v_first, l = JGPT_W_VMIX, v_first those of the first such layer (which has no l) */
+    float decay_rate;         /* general delta */
 } jgpt_mixer_spec;
 /* Mixture of experts.  Scores are the softmax of W_router h over experts + identity outputs; the top largest scores + correction
  * are chosen among the `keep` of `groups` equal groups of neighbours with the largest such score; weights are the chosen scores
@@ -414,6 +429,9 @@ typedef struct {
     float residual_mult;
     int32_t norm_after;    /* norms behind the sums instead of in front of the parts (RMS only, without layer_scale and depth_average) */
     float residual_scale;  /* with norm_after */
+    int32_t norm_both;     /* norms in front of and behind the parts (RMS only); the next two go with it */
+    int32_t token_shift;   /* JGPT_W_SHIFT */
+    int32_t residual_gate; /* JGPT_W_RG1, _RG1_B, _RG2, _RG2_B */
 } jgpt_decoder_spec;
 /* Tensors.  Of the model: layer = branch = -1; of a layer: branch = -1; of a mixer: layer and branch; of an expert: layer and
  * branch = JGPT_EXPERT(e). */
@@ -429,8 +447,10 @@ enum {
     JGPT_W_DQ, JGPT_W_DQ_NORM, JGPT_W_UQ, JGPT_W_DKV, JGPT_W_DKV_NORM, JGPT_W_UK, JGPT_W_UV,
     JGPT_W_FF_ACT /* of a layer: p, q */,
     JGPT_W_Q_BIAS, JGPT_W_K_BIAS, JGPT_W_V_BIAS, JGPT_W_Q_NORM, JGPT_W_K_NORM, JGPT_W_LQ1, JGPT_W_LK1, JGPT_W_LQ2, JGPT_W_LK2,
+    JGPT_W_SINK, JGPT_W_VMIX /* [1] */, JGPT_W_B_BIAS,
     JGPT_W_ROUTER = 64 /* of a layer, as the next four: [experts + identity, width] */, JGPT_W_CORRECTION, JGPT_W_SHARED_GATE /* [1, width] */,
-    JGPT_W_SHARED_UP, JGPT_W_SHARED_DOWN, JGPT_W_EXPERT_UP /* of an expert, as the next */, JGPT_W_EXPERT_DOWN
+    JGPT_W_SHARED_UP, JGPT_W_SHARED_DOWN, JGPT_W_EXPERT_UP /* of an expert, as the next */, JGPT_W_EXPERT_DOWN,
+    JGPT_W_POST1 = 80 /* of a layer, as the others: norms behind the parts */, JGPT_W_POST2, JGPT_W_SHIFT, JGPT_W_RG1, JGPT_W_RG1_B, JGPT_W_RG2, JGPT_W_RG2_B
 };
 
 /* max_rows bounds the rows (tokens) of one step. */

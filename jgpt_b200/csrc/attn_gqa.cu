@@ -1,6 +1,7 @@
 // Paged attention of the layered decoder: query heads in groups that share a key head, head sizes up to 256 (padded to what
-// the kernels are built for), all earlier positions or those of the query's chunk, optional norms and rotation of the heads,
-// one or two maps per head (mixers.cuh), an optional output gate per head or per element.
+// the kernels are built for), all earlier positions, those of the query's chunk, or a window and the first tokens, optional norms
+// and rotation of the heads, sinks, values mixed with another layer's, one or two maps per head (mixers.cuh), an optional output
+// gate per head or per element.
 //
 //   attn_prep_kernel     keys (normed and rotated) and values into the pages; in the exact mode query heads in place
 //   attn_rows_kernel     one warp per (row, head), fp32: the exact mode
@@ -16,34 +17,47 @@
 namespace jgpt {
 namespace mix {
 
-__host__ __device__ __forceinline__ int first_visible(int pos, int chunk) { return chunk > 0 ? pos / chunk * chunk : 0; }
+// First key of the chunk or window of a position; with a window the keys before a.keep are seen as well.
+__host__ __device__ __forceinline__ int first_visible(int pos, const AttnArgs &a) {
+    if (a.window > 0) return pos >= a.window ? pos - a.window + 1 : 0;
+    return a.chunk > 0 ? pos / a.chunk * a.chunk : 0;
+}
+// Keys in front of the window that are visited on their own: none, or [0, keep) when the window's first page lies behind them.
+__device__ __forceinline__ int kept_apart(int first_page_key, const AttnArgs &a) { return a.keep > 0 && first_page_key >= a.keep ? a.keep : 0; }
 
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 
 // What happens to a query or key head (map) behind its projection: norm, rotation.
 struct HeadPrep {
-    const float *w;  // null: no norm
+    const float *w;  // weights of the norm, null: 1
     const float2 *cs;
-    int dim, half, interleaved;
-    float eps;
+    int dim, half, interleaved, norm;
+    float eps, inv;  // inv: of the whole row
 };
-__device__ __forceinline__ HeadPrep head_prep(const AttnArgs &a, bool key, int row) {
-    return HeadPrep{key ? a.k_norm : a.q_norm, a.cs + (size_t)row * a.half, a.dim, a.half, a.interleaved, a.eps};
+// head: which of the row's (its weights, when the whole row has some); inv: 1 / root mean square of the row, when that is what the norm takes
+__device__ __forceinline__ HeadPrep head_prep(const AttnArgs &a, bool key, int row, int head, float inv) {
+    const float *w = key ? a.k_norm : a.q_norm;
+    return HeadPrep{w + (a.qk_norm == QK_NORM_ALL ? head * a.DK : 0), a.cs + (size_t)row * a.half, a.dim, a.half, a.interleaved, a.qk_norm, a.eps, inv};
 }
+__device__ __forceinline__ float head_weight(const HeadPrep &h, int j) { return h.norm == QK_NORM_UNIT ? 1.f : __ldg(h.w + j); }
 // The head lies in 8-element pieces in `lanes` neighbouring lanes (a power of two; every lane of the warp takes part); src: its
 // start in memory.
 template <class AT>
 __device__ __forceinline__ void prepare_head(float (&x)[8], const AT *src, int piece, int lanes, const HeadPrep &h) {
     const int j0 = piece * 8;
     float inv = 1.f;
-    if (h.w) {
+    if (h.norm == QK_NORM_ALL) {
+        inv = h.inv;
+#pragma unroll
+        for (int e = 0; e < 8; e++) x[e] = j0 + e < h.dim ? x[e] * inv * __ldg(h.w + j0 + e) : 0.f;
+    } else if (h.norm) {
         float ss = 0.f;
 #pragma unroll
         for (int e = 0; e < 8; e++) ss += x[e] * x[e];
         for (int off = lanes >> 1; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
         inv = 1.f / sqrtf(ss / (float)h.dim + h.eps);
 #pragma unroll
-        for (int e = 0; e < 8; e++) x[e] = j0 + e < h.dim ? x[e] * inv * __ldg(h.w + j0 + e) : 0.f;
+        for (int e = 0; e < 8; e++) x[e] = j0 + e < h.dim ? x[e] * inv * head_weight(h, j0 + e) : 0.f;
     }
     if (!h.half) return;
     if (h.interleaved) {
@@ -71,7 +85,7 @@ __device__ __forceinline__ void prepare_head(float (&x)[8], const AT *src, int p
             const int j = j0 + e, p = j < h.half ? j + h.half : j - h.half;
             if (j >= 2 * h.half) continue;
             const float2 t = h.cs[(j < h.half ? j : p)];
-            const float y = act_load(src + p) * inv * (h.w ? __ldg(h.w + p) : 1.f);
+            const float y = act_load(src + p) * inv * (h.norm ? head_weight(h, p) : 1.f);
             x[e] = j < h.half ? x[e] * t.x - y * t.y : x[e] * t.x + y * t.y;
         }
         __syncwarp();  // whoever writes the head back does so after this
@@ -79,38 +93,88 @@ __device__ __forceinline__ void prepare_head(float (&x)[8], const AT *src, int p
 }
 __host__ __device__ constexpr int head_lanes(int DK) { return DK <= 32 ? 4 : (DK <= 64 ? 8 : (DK <= 128 ? 16 : 32)); }
 
+// 1 / root mean square of n heads of a row (padding is zero), by all threads of the block.
+template <class AT>
+__device__ __forceinline__ float row_rms(const AT *src, int n, const AttnArgs &a, float *red) {
+    float ss = 0.f;
+    for (int c = threadIdx.x * 8; c < n * a.DK; c += blockDim.x * 8) {
+        float x[8];
+        load8(src + c, x);
+#pragma unroll
+        for (int e = 0; e < 8; e++) ss += x[e] * x[e];
+    }
+#pragma unroll
+    for (int off = 16; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+    __syncthreads();  // the previous use of red is over
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+    for (int w = 0; w < (int)blockDim.x / 32; w++) ss += red[w];
+    return 1.f / sqrtf(ss / (float)(n * a.dim) + a.eps);
+}
+
+// Eight values of a key head from column c on, mixed with another layer's (whose heads may be cut differently).
+template <class AT>
+__device__ __forceinline__ void load_values(const AttnArgs &a, int row, int g, int c, float (&x)[8]) {
+    load8(reinterpret_cast<const AT *>(a.proj) + (size_t)row * a.ldp + a.v_off + g * a.DV + c, x);
+    if (!a.v_first) return;
+    const AT *first = reinterpret_cast<const AT *>(a.v_first) + (size_t)row * a.ld_first;
+    float y[8];
+    if (a.vdim_first == a.vdim && c + 8 <= a.DV_first) {
+        load8(first + g * a.DV_first + c, y);
+    } else {
+#pragma unroll
+        for (int e = 0; e < 8; e++) {
+            const int i = g * a.vdim + c + e;
+            y[e] = c + e < a.vdim ? act_load(first + i / a.vdim_first * a.DV_first + i % a.vdim_first) : 0.f;
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < 8; e++) x[e] = fmaf(a.v_share, y[e], (1.f - a.v_share) * x[e]);
+}
+
 // A block (or several, in y) per row: its query maps (with `queries`, in place), key maps and values (into the page), a vector per
 // head_lanes(DK) lanes.
 template <class AT>
 __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a, const int *__restrict__ seq, const int *__restrict__ pos, int queries, int pdl) {
     if (pdl & 2) griddep_launch_dependents();
+    __shared__ float red[8];
     const int lanes = head_lanes(a.DK), nq = queries ? a.heads * a.maps : 0, nk = a.kv_heads * a.maps, nv = nq + nk + a.kv_heads;
-    const int r = blockIdx.x, i = (blockIdx.y * blockDim.x + threadIdx.x) / lanes, piece = threadIdx.x & (lanes - 1);
+    const int r = blockIdx.x, piece = threadIdx.x & (lanes - 1), per = blockDim.x / lanes;
     const int p = pos[r], row = p % kBlockTokens, phys = page_of(a, seq[r], p), kw = a.maps * a.DK;
     if (pdl & 1) griddep_wait();
     AT *proj = reinterpret_cast<AT *>(a.proj) + (size_t)r * a.ldp;
-    const bool query = i < nq, value = i >= nq + nk && i < nv, key = i >= nq && i < nq + nk;
-    const int g = key ? (i - nq) / a.maps : (value ? i - nq - nk : 0);
-    AT *page = reinterpret_cast<AT *>(a.kv) + ((size_t)max(phys, 0) * a.kv_heads + g) * a.page_head();
-    if (value && phys >= 0) {
-        AT *dst = page + kBlockTokens * page_row(kw) + row * page_row(a.DV);
-        for (int c = piece; c < a.DV / 8; c += lanes) {
-            float x[8];
-            load8(proj + a.v_off + g * a.DV + c * 8, x), store8(dst + page_chunk(a.DV, row, c) * 8, x);
+    float2 inv = make_float2(1.f, 1.f);
+    if (a.qk_norm == QK_NORM_ALL) {  // one block has the row then
+        inv.x = row_rms(proj + a.q_off, a.heads, a, red), inv.y = row_rms(proj + a.k_off, a.kv_heads, a, red);
+        if (threadIdx.x == 0) a.row_inv[r] = inv;
+    }
+    for (int i0 = blockIdx.y * per; i0 < nv; i0 += gridDim.y * per) {
+        const int i = i0 + threadIdx.x / lanes;
+        const bool query = i < nq, value = i >= nq + nk && i < nv, key = i >= nq && i < nq + nk;
+        const int g = key ? (i - nq) / a.maps : (value ? i - nq - nk : 0);
+        AT *page = reinterpret_cast<AT *>(a.kv) + ((size_t)max(phys, 0) * a.kv_heads + g) * a.page_head();
+        if (value && phys >= 0) {
+            AT *dst = page + kBlockTokens * page_row(kw) + row * page_row(a.DV);
+            for (int c = piece; c < a.DV / 8; c += lanes) {
+                float x[8];
+                load_values<AT>(a, r, g, c * 8, x), store8(dst + page_chunk(a.DV, row, c) * 8, x);
+            }
         }
-    }
-    const AT *src = proj + (query ? a.q_off + i * a.DK : a.k_off + (key ? i - nq : 0) * a.DK);
-    float x[8];
-    const bool load = (query || key) && piece * 8 < a.DK;
-    if (load) load8(src + piece * 8, x);
-    else {
+        const int head = query ? i : (key ? i - nq : 0);
+        const AT *src = proj + (query ? a.q_off : a.k_off) + head * a.DK;
+        float x[8];
+        const bool load = (query || key) && piece * 8 < a.DK;
+        if (load) load8(src + piece * 8, x);
+        else {
 #pragma unroll
-        for (int e = 0; e < 8; e++) x[e] = 0.f;
+            for (int e = 0; e < 8; e++) x[e] = 0.f;
+        }
+        if (a.prepared()) prepare_head(x, src, piece, lanes, head_prep(a, !query, r, head, query ? inv.x : inv.y));
+        if (!load) continue;
+        if (query) store8(proj + a.q_off + i * a.DK + piece * 8, x);
+        else if (phys >= 0) store8(page + row * page_row(kw) + page_chunk(kw, row, (i - nq) % a.maps * (a.DK / 8) + piece) * 8, x);
     }
-    if (a.prepared()) prepare_head(x, src, piece, lanes, head_prep(a, !query, r));
-    if (!load) return;
-    if (query) store8(proj + a.q_off + i * a.DK + piece * 8, x);
-    else if (phys >= 0) store8(page + row * page_row(kw) + page_chunk(kw, row, (i - nq) % a.maps * (a.DK / 8) + piece) * 8, x);
 }
 
 // One warp per (row, query head): lane l holds elements l, l + 32, ... of q and of the output.
@@ -128,7 +192,9 @@ __global__ void __launch_bounds__(256) attn_rows_kernel(const AttnArgs a, const 
 #pragma unroll
         for (int e = 0; e < MAXE; e++)
             q[e] = e < nk ? act_load(proj + a.q_off + (h * a.maps + map) * a.DK + lane + 32 * e) * a.scale : 0.f, first[e] = map ? o[e] * f : 0.f, o[e] = 0.f;
-        for (int j = first_visible(p, a.chunk); j <= p; j++) {
+        const int seen = first_visible(p, a);
+        for (int j = min(a.keep, seen) > 0 ? 0 : seen; j <= p; j++) {
+            if (j == min(a.keep, seen)) j = seen;
             const int phys = page_of(a, s, j);
             if (phys < 0) break;
             const int row = j % kBlockTokens;
@@ -146,6 +212,12 @@ __global__ void __launch_bounds__(256) attn_rows_kernel(const AttnArgs a, const 
 #pragma unroll
             for (int e = 0; e < MAXE; e++)
                 if (e < nv) o[e] = fmaf(w, act_load(v + at(a.DV, lane + 32 * e)), o[e] * fo);
+        }
+        if (a.sink) {
+            const float mn = fmaxf(m, a.sink[h]), fo = expf(m - mn);
+            l = l * fo + expf(a.sink[h] - mn);
+#pragma unroll
+            for (int e = 0; e < MAXE; e++) o[e] *= fo;
         }
         f = l > 0.f ? 1.f / l : 0.f;
     }
@@ -225,7 +297,10 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
     const int nt = min(qt, sg.T - tile.y), rows = nt * grp, row_base = sg.row0 + tile.y;
     if (r0 >= rows) return;
     const int p0 = sg.pos0 + tile.y, b0 = p0 + r0 / grp, p1 = p0 + (min(rows, r0 + ROWS) - 1) / grp;  // positions: of the tile, of the block's rows
-    const int first = first_visible(b0, a.chunk) / kBlockTokens * kBlockTokens, n_tiles = (p1 - first) / KT + 1;
+    // keys in tiles: the kept ones when they lie apart, then those from the first one that the block's first row sees
+    const int win = first_visible(b0, a) / kBlockTokens * kBlockTokens, kept = kept_apart(win, a), first = a.keep && !kept ? 0 : win;
+    const int n_kept = (kept + KT - 1) / KT, n_tiles = n_kept + (p1 - first) / KT + 1;
+    auto tile_key = [&](int it) { return it < n_kept ? it * KT : first + (it - n_kept) * KT; };
     if (tid == 0) {
         for (int s = 0; s < ST; s++) mbar_init(&full[s], 1), mbar_init(&empty[s], NC / 32);
         *s_abort = 0;
@@ -236,7 +311,7 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
     if (tid >= NC) {
         const __nv_bfloat16 *kv = reinterpret_cast<const __nv_bfloat16 *>(a.kv) + (size_t)kvh * P::ELEMS;
         auto lookup = [&](int it) {
-            const int key = first + it * KT + lane * 16;
+            const int key = tile_key(it) + lane * 16;
             return lane < PAGES && it < n_tiles && key <= p1 ? page_of(a, sg.seq, key) : -1;
         };
         int phys = lookup(0), it = 0;
@@ -262,27 +337,28 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
         constexpr int LANES = head_lanes(DK), PER = NC / LANES, N = 64 / PER;  // vectors at a time, rounds
         const __nv_bfloat16 *proj = reinterpret_cast<const __nv_bfloat16 *>(a.proj);
         const int piece = tid & (LANES - 1);
-        auto source = [&](int v, int &row) {  // vector v = row of the block, map
-            const int r = r0 + v / MAPS, t = r / grp, h = kvh * grp + r % grp;
-            row = row_base + t;
+        auto source = [&](int v, int &row, int &h) {  // vector v = row of the block, map
+            const int r = r0 + v / MAPS, t = r / grp;
+            h = kvh * grp + r % grp, row = row_base + t;
             return r < rows ? proj + (size_t)row * a.ldp + a.q_off + (h * MAPS + v % MAPS) * DK : nullptr;
         };
         uint4 raw[N];
 #pragma unroll
         for (int n = 0; n < N; n++) {
-            int row;
-            const __nv_bfloat16 *src = source(n * PER + tid / LANES, row);
+            int row, h;
+            const __nv_bfloat16 *src = source(n * PER + tid / LANES, row, h);
             raw[n] = src && piece * 8 < DK ? *reinterpret_cast<const uint4 *>(src + piece * 8) : make_uint4(0, 0, 0, 0);
         }
 #pragma unroll
         for (int n = 0; n < N; n++) {
             const int v = n * PER + tid / LANES;
             if (a.prepared()) {
-                int row;
-                const __nv_bfloat16 *src = source(v, row);
+                int row, h;
+                const __nv_bfloat16 *src = source(v, row, h);
+                if (!src) row = row_base, h = kvh * grp;
                 float x[8];
                 load8(reinterpret_cast<const __nv_bfloat16 *>(&raw[n]), x);
-                prepare_head(x, src ? src : proj, piece, LANES, head_prep(a, false, src ? row : row_base));
+                prepare_head(x, src ? src : proj, piece, LANES, head_prep(a, false, row, h, a.qk_norm == QK_NORM_ALL ? a.row_inv[row].x : 1.f));
                 store8(reinterpret_cast<__nv_bfloat16 *>(&raw[n]), x);
             }
             if (piece * 8 < DK) *reinterpret_cast<uint4 *>(qs + (v % MAPS * ROWS + v / MAPS) * LQ + piece * 8) = raw[n];
@@ -295,7 +371,7 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
         const int r = r0 + warp * 16 + g + 8 * e;
         rt[e] = r < rows ? r : -1;
         hi[e] = p0 + (r < rows ? r : r0) / grp;
-        lo[e] = first_visible(hi[e], a.chunk);
+        lo[e] = first_visible(hi[e], a);
     }
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[DV / 8][4];
 #pragma unroll
@@ -306,9 +382,10 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
         ldmatrix_x4(f, qs + (size_t)(map * ROWS + warp * 16 + (lane & 15)) * LQ + kk * 16 + (lane >> 4) * 8);
     };
     const float sl = a.scale * 1.4426950408889634f;
-    const int vis_lo = first_visible(p1, a.chunk);
+    const int vis_lo = first_visible(p1, a);
     for (int it = 0; it < n_tiles; it++) {
-        const int s = it % ST, kb = first + it * KT;
+        const int s = it % ST, kb = tile_key(it);
+        const bool apart = it < n_kept;
         if (!__all_sync(0xffffffffu, mbar_wait_bounded(&full[s], (it / ST) & 1, a.status, s_abort))) break;
         __nv_bfloat16 *stage = ring + s * T::stage_elems;
         if (kb + KT > p1 + 1) {  // every warp clears what it is going to read
@@ -319,7 +396,12 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
         }
         auto kat = [&](int r, int c) { return P::k(stage + (r >> 4) * P::ELEMS, r & 15, map * (DK / 8) + c); };
         auto vat = [&](int r, int c) { return P::v(stage + (r >> 4) * P::ELEMS, r & 15, c); };
-        attend_tile<DK, DV, KT>(qfrag, kat, vat, kb, kb + KT - 1 > b0 || kb < vis_lo, lo, hi, sl, m, l, o, lane);
+        if (apart) {
+            const int all[2] = {0, 0}, top[2] = {kept - 1, kept - 1};
+            attend_tile<DK, DV, KT>(qfrag, kat, vat, kb, kb + KT > kept, all, top, 0, sl, m, l, o, lane);
+        } else {
+            attend_tile<DK, DV, KT>(qfrag, kat, vat, kb, kb + KT - 1 > b0 || kb < vis_lo, lo, hi, a.keep, sl, m, l, o, lane);
+        }
         __syncwarp();
         if (lane == 0) mbar_arrive(&empty[s]);
     }
@@ -329,6 +411,10 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
         l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
         l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
         f[e] = l[e] > 0.f ? 1.f / l[e] : 0.f;
+        if (MAPS == 1 && a.sink && rt[e] >= 0) {  // its share: relative to the larger of the two scores
+            const float sk = a.sink[kvh * grp + rt[e] % grp] * 1.4426950408889634f, mn = fmaxf(m[e], sk), w = fast_exp2(m[e] - mn);
+            f[e] = w / (l[e] * w + fast_exp2(sk - mn));
+        }
     }
     if (MAPS == 2) {
         float *other = reinterpret_cast<float *>(ring);  // [ROWS][DV + 8]
@@ -406,6 +492,7 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
     float *merged = reinterpret_cast<float *>(attn_smem + S::front);           // [16][m, l, -, -, o[DV]] of this CTA, after the loop
     __nv_bfloat16 *qs = reinterpret_cast<__nv_bfloat16 *>(attn_smem + S::front), *own = qs + 16 * LQ;  // query rows [16][LQ]; the token's [K | V]
     __shared__ __align__(8) uint64_t full[4][ST];
+    __shared__ float red[4];
     __shared__ int s_abort_mem;
     volatile int *s_abort = &s_abort_mem;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t2 = 2 * (lane & 3);
@@ -413,8 +500,11 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
     const int rb = blockIdx.y % row_blocks, kvh = blockIdx.y / row_blocks, grp = a.heads / a.kv_heads, h0 = kvh * grp + rb * hpb, nh = min(hpb, grp - rb * hpb);
     if (pdl & 2) griddep_launch_dependents();
     const Seg sg = segs[singles[blockIdx.z]];
-    const int p = sg.pos0, row = sg.row0, first = first_visible(p, a.chunk), lo_page = first / kBlockTokens, n_pages = p / kBlockTokens - lo_page + 1;
-    const int pg0 = lo_page + split * n_pages / nsplit, pg1 = lo_page + (split + 1) * n_pages / nsplit, last = p / kBlockTokens;
+    // pages in order: the kept ones when they lie apart, then those from the first one seen; this CTA has [pg0, pg1) of them
+    const int p = sg.pos0, row = sg.row0, first = first_visible(p, a), win_page = first / kBlockTokens, kept = kept_apart(win_page * kBlockTokens, a);
+    const int lo_page = a.keep && !kept ? 0 : win_page, n_kept = (kept + kBlockTokens - 1) / kBlockTokens, last = p / kBlockTokens, n_pages = n_kept + last - lo_page + 1;
+    const int pg0 = split * n_pages / nsplit, pg1 = (split + 1) * n_pages / nsplit;
+    auto page_at = [&](int i) { return i < n_kept ? i : i - n_kept + lo_page; };
     __nv_bfloat16 *kv = reinterpret_cast<__nv_bfloat16 *>(a.kv) + (size_t)kvh * P::ELEMS;
     if (lane == 0) {
         for (int s = 0; s < ST; s++) mbar_init(&full[warp][s], 1);
@@ -430,7 +520,7 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
         const int pg = pg0 + warp + 4 * i;
         if ((i & 31) == 0) {
             const int at = pg + 4 * lane;
-            blocks = at < pg1 ? page_of(a, sg.seq, at * kBlockTokens) : -1;
+            blocks = at < pg1 ? page_of(a, sg.seq, page_at(at) * kBlockTokens) : -1;
         }
         const int phys = __shfl_sync(0xffffffffu, blocks, i & 31);
         if (pg < pg1 && lane == 0) {
@@ -450,6 +540,15 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
     }
     const __nv_bfloat16 *proj = reinterpret_cast<const __nv_bfloat16 *>(a.proj) + (size_t)row * a.ldp;
     {
+        float2 inv = make_float2(1.f, 1.f);
+        if (a.qk_norm == QK_NORM_ALL) {
+            if (fused) {
+                inv.x = row_rms(proj + a.q_off, a.heads, a, red);
+                if (append) inv.y = row_rms(proj + a.k_off, a.kv_heads, a, red);
+            } else {
+                inv = a.row_inv[row];
+            }
+        }
         // heads of the group, then (with the last page) the key's maps
         const int lanes = head_lanes(dk), piece = tid & (lanes - 1), slots = 128 / lanes, nq = nh * maps;
         const int phys = append ? page_of(a, sg.seq, p) : -1, total = nq + (append ? maps : 0), r = p % kBlockTokens;
@@ -464,7 +563,7 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
 #pragma unroll
                 for (int e = 0; e < 8; e++) x[e] = 0.f;
             }
-            if (a.prepared()) prepare_head(x, src, piece, lanes, head_prep(a, key, row));
+            if (a.prepared()) prepare_head(x, src, piece, lanes, head_prep(a, key, row, key ? kvh : min(h0 + v, a.heads - 1), key ? inv.y : inv.x));
             if (!load) continue;
             if (key) {
                 const int c = (v - nq) * (dk / 8) + piece;
@@ -476,9 +575,10 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
         }
         if (append)
             for (int c = tid; c < CV; c += 128) {
-                const uint4 x = *reinterpret_cast<const uint4 *>(proj + a.v_off + kvh * DV + c * 8);
-                *reinterpret_cast<uint4 *>(own + DK + c * 8) = x;
-                if (phys >= 0) *reinterpret_cast<uint4 *>(P::v(page, r, c)) = x;
+                float x[8];
+                load_values<__nv_bfloat16>(a, row, kvh, c * 8, x);
+                store8(own + DK + c * 8, x);
+                if (phys >= 0) store8(P::v(page, r, c), x);
             }
         __syncthreads();
     }
@@ -491,10 +591,11 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
     for (int n = 0; n < DV / 8; n++)
 #pragma unroll
         for (int e = 0; e < 4; e++) o[n][e] = 0.f;
-    const int lo[2] = {first, first}, hi[2] = {p, p};
+    const int lo[2] = {first, first}, hi[2] = {p, p}, kept_lo[2] = {0, 0}, kept_hi[2] = {kept - 1, kept - 1};
     const float sl = a.scale * 1.4426950408889634f;
     for (int i = 0; pg0 + warp + 4 * i < pg1; i++) {
-        const int pg = pg0 + warp + 4 * i, kb = pg * kBlockTokens;
+        const bool apart = pg0 + warp + 4 * i < n_kept;
+        const int pg = page_at(pg0 + warp + 4 * i), kb = pg * kBlockTokens;
         if (!__all_sync(0xffffffffu, mbar_wait_bounded(&full[warp][i % ST], (i / ST) & 1, a.status, s_abort))) break;
         __nv_bfloat16 *page = mine + (size_t)(i % ST) * P::ELEMS;
         if (pg == last) {
@@ -509,7 +610,8 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
         }
         auto kat = [&](int r, int c) { return P::k(page, r, c); };
         auto vat = [&](int r, int c) { return P::v(page, r, c); };
-        attend_tile<DK, DV, 16>(qfrag, kat, vat, kb, kb < first || kb + 15 > p, lo, hi, sl, m, l, o, lane);
+        if (apart) attend_tile<DK, DV, 16>(qfrag, kat, vat, kb, kb + 16 > kept, kept_lo, kept_hi, 0, sl, m, l, o, lane);
+        else attend_tile<DK, DV, 16>(qfrag, kat, vat, kb, kb < first || kb + 15 > p, lo, hi, a.keep, sl, m, l, o, lane);
         __syncwarp();
         load(i + ST);
     }
@@ -550,9 +652,13 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
         const int c0 = split * DV / nsplit, cn = (split + 1) * DV / nsplit - c0;
         for (int e = tid; e < nh * cn; e += 128) {
             const int r = e / cn, c = c0 + e % cn;
-            float mx = -INFINITY, sum = 0.f, acc = 0.f;
+            const float sk = a.sink ? a.sink[h0 + r] * 1.4426950408889634f : -INFINITY;
+            float mx = sk, sum = 0.f, acc = 0.f;
             if (nsplit == 1) {
-                sum = merged[r * PW + 1], acc = merged[r * PW + 4 + c];
+                const float ms = merged[r * PW];
+                mx = fmaxf(mx, ms);
+                const float f = a.sink && ms != -INFINITY ? fast_exp2(ms - mx) : 1.f;
+                sum = f * merged[r * PW + 1], acc = f * merged[r * PW + 4 + c];
             } else {
                 for (int s = 0; s < nsplit; s++) mx = fmaxf(mx, ld_cluster_f32(merged + r * PW, (uint32_t)s));
                 for (int s = 0; s < nsplit; s++) {
@@ -560,6 +666,7 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
                     sum += f * ld_cluster_f32(merged + r * PW + 1, (uint32_t)s), acc += f * ld_cluster_f32(merged + r * PW + 4 + c, (uint32_t)s);
                 }
             }
+            if (a.sink) sum += fast_exp2(sk - mx);
             float v = acc * (sum > 0.f ? 1.f / sum : 0.f) * row_factor(a, row, h0 + r);
             if (a.gate == GATE_ELEMENT) v *= sigmoid(act_load(gate_at(a, row, h0 + r, c)));
             out[(size_t)r * DV + c] = __float2bfloat16(v);
@@ -616,7 +723,7 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
 struct HeadSizes {
     int maps, DK, DV;
 };
-constexpr HeadSizes kHeadSizes[] = {{1, 32, 32},  {1, 64, 32},  {1, 64, 64},  {1, 96, 96},  {1, 128, 64}, {1, 128, 128}, {1, 192, 192}, {1, 256, 256},
+constexpr HeadSizes kHeadSizes[] = {{1, 32, 32},  {1, 64, 32},  {1, 64, 64},  {1, 96, 64},  {1, 96, 96},  {1, 128, 64}, {1, 128, 128}, {1, 192, 192}, {1, 256, 256},
                                     {2, 32, 32},  {2, 32, 64},  {2, 64, 64},  {2, 64, 96},  {2, 64, 128}, {2, 96, 192},  {2, 128, 128}, {2, 128, 256}};
 
 bool attn_padded_head(int dim, int vdim, int maps, int *DK, int *DV) {
@@ -630,7 +737,7 @@ int attn_query_tile(int heads, int kv_heads) { return std::max(1, 64 / (heads / 
 // Threads of a row's preparation: one block, or several of 256.
 static void prep_shape(const AttnArgs &a, bool queries, int rows, dim3 *grid, dim3 *block) {
     const int threads = ((queries ? a.heads * a.maps : 0) + a.kv_heads * (a.maps + 1)) * head_lanes(a.DK);
-    *block = dim3((unsigned)std::min(256, (threads + 31) / 32 * 32)), *grid = dim3((unsigned)rows, (threads + block->x - 1) / block->x);
+    *block = dim3((unsigned)std::min(256, (threads + 31) / 32 * 32)), *grid = dim3((unsigned)rows, a.qk_norm == QK_NORM_ALL ? 1u : (threads + block->x - 1) / block->x);
 }
 
 template <class AT>
@@ -682,7 +789,7 @@ static int32_t tensor_attention(const StepDesc &d, const AttnArgs &a, int pdl, c
         static thread_local int set_for = -1;
         if (int32_t rc = opt_in(attn_single_kernel<KW, DV>, (Single<KW, DV>::smem), set_for)) return rc;
         const int row_blocks = (grp * MAPS + 15) / 16, ctas = d.n_singles * a.kv_heads * row_blocks;
-        const int keys = a.chunk > 0 ? std::min(a.chunk, d.max_len) : d.max_len, pages = keys / kBlockTokens + 1;
+        const int range = a.window > 0 ? a.window + a.keep : a.chunk, keys = range > 0 ? std::min(range, d.max_len) : d.max_len, pages = keys / kBlockTokens + 1;
         int split = 1;  // every warp keeps two pages, the grid stays around two CTAs per SM
         while (split < 8 && ctas * split * 2 <= 2 * a.sm_count && pages >= split * 2 * 8) split *= 2;
         int na = early(0);

@@ -16,6 +16,10 @@
 // behind them writes x and its rounding for the next product.  A mixture of experts is router -> route (choice, lists, tiles) ->
 // up products of all experts and the shared one -> down products -> the norm kernel adds a token's weighted rows on its way.
 //
+// With norms on both sides of the parts the norm kernel between two parts does everything but products: it gates and norms the part's
+// result, adds it to x (two arrays in turn), norms x for the next part and mixes in the row before.  The gate's projection rides
+// with the next part's first product: a second segment of it reads the rows as they were before the shift.
+//
 // The residual x is fp32; rows entering a product are bf16 (or fp32 in the exact mode).  Head sizes are padded with zero
 // weights to what the kernels take, so every size of a configuration works; sums over a head use the true size.
 #include "decoder.cuh"
@@ -35,6 +39,8 @@ struct DBranch {
     jgpt_mixer_spec s{};
     int DK = 0, DV = 0;                 // padded head sizes (of one map)
     int maps = 1;
+    const DBranch *v_first = nullptr;   // values are mixed with this branch's
+    float v_share = 0.f, *sink = nullptr;
     float lambda = 0.f;                 // differential attention: from the four vectors below
     std::vector<float> lambda_part[4];
     float *q_norm = nullptr, *k_norm = nullptr;
@@ -56,13 +62,19 @@ struct DBranch {
     bool expand = false;                  // its head sizes have a written-out form
     void *w_uq = nullptr, *w_absorb = nullptr, *w_ukv = nullptr;  // [heads * DQ, qrp], [heads * KR, DP], [heads * (DP + DV), KR]
     float *dq_norm = nullptr, *dkv_norm = nullptr;
-    bool recurrent() const { return s.kind == JGPT_MIX_GLA || s.kind == JGPT_MIX_DELTA || s.kind == JGPT_MIX_HGRN2 || s.kind == JGPT_MIX_WKV; }
+    float *removal_bias = nullptr;        // general delta [heads * DK]
+    bool recurrent() const { return s.kind == JGPT_MIX_GLA || s.kind == JGPT_MIX_DELTA || s.kind == JGPT_MIX_HGRN2 || s.kind == JGPT_MIX_WKV || s.kind == JGPT_MIX_GENERAL_DELTA; }
     int cols() const { return s.heads * DV; }
 };
 
 struct DLayer {
     std::vector<DBranch> br;
     int ff = 0, ffp = 0, n_in = 0, n_out = 0, n_z = 0;
+    int n_mix = 0, n_up = 0;                 // columns of the mixers in proj, of the first feed-forward product; gates lie behind
+    int tanh_from = 0, tanh_to = 0;          // columns of proj with an activation
+    float *post1 = nullptr, *post2 = nullptr, *share = nullptr, *bias_up = nullptr;
+    uint64_t shift_off = 0, have_both = 0;
+    bool v_source = false;                   // its projections stay for the layers that mix in its values
     void *w_in = nullptr, *w_out = nullptr, *w_gu = nullptr, *w_down = nullptr;
     float *n1w = nullptr, *n1b = nullptr, *n2w = nullptr, *n2b = nullptr;
     int ff_kind = 0;
@@ -88,6 +100,8 @@ struct Decoder {
     std::vector<DLayer> L;
     void *embed = nullptr, *pos = nullptr, *head = nullptr;
     bool rms = false;
+    const DBranch *v_first = nullptr;
+    int v_first_ld = 0;
     std::vector<mix::Rotation> rots;
     std::vector<jgpt_mixer_spec> rot_specs;
     int max_window = 0;                // largest window of the latent layers (0: unbounded)
@@ -100,12 +114,14 @@ struct Decoder {
     uint64_t state_stride = 0;
     std::vector<void *> allocs;
     // workspace
-    float *x = nullptr, *raw = nullptr, *chunk_ws = nullptr, *logits = nullptr;
-    void *h = nullptr, *proj = nullptr, *z = nullptr, *mixed = nullptr, *act = nullptr;
+    float *x = nullptr, *x_next = nullptr, *raw = nullptr, *chunk_ws = nullptr, *logits = nullptr;
+    void *h = nullptr, *proj = nullptr, *proj_first = nullptr, *y = nullptr, *z = nullptr, *mixed = nullptr, *act = nullptr;
     // mixtures: activations of the experts' rows, their results, the same of the shared expert; routing
     void *e_act = nullptr, *e_out = nullptr, *s_act = nullptr, *s_out = nullptr;
     float *r_logits = nullptr;
     mix::RouteArgs route{};
+    mix::PartNorm open{};              // what the layers left for the final norm
+    float2 *row_inv = nullptr;         // 1 / root mean square of a row's queries and keys
     int *d_desc = nullptr, *h_desc = nullptr;
     int *d_next = nullptr, *h_next = nullptr;
     float *d_u = nullptr, *h_u = nullptr, *samp = nullptr;
@@ -166,13 +182,14 @@ int32_t decoder_destroy(Decoder *d) {
 
 static mix::RecArgs rec_args(const DBranch &b) {
     mix::RecArgs a{};
-    a.kind = b.s.kind == JGPT_MIX_DELTA ? mix::REC_DELTA : b.s.kind == JGPT_MIX_HGRN2 ? mix::REC_HGRN2 : b.s.kind == JGPT_MIX_WKV ? mix::REC_WKV : mix::REC_GLA;
+    a.kind = b.s.kind == JGPT_MIX_DELTA ? mix::REC_DELTA : b.s.kind == JGPT_MIX_HGRN2 ? mix::REC_HGRN2 : b.s.kind == JGPT_MIX_WKV ? mix::REC_WKV
+             : b.s.kind == JGPT_MIX_GENERAL_DELTA ? mix::REC_GENERAL : mix::REC_GLA;
     a.q_off = b.q, a.k_off = b.k, a.v_off = b.v, a.b_off = b.b, a.g_off = b.g, a.z_off = b.za, a.zg_off = b.zg;
     a.heads = b.s.heads, a.kv_heads = b.s.kv_heads, a.DK = b.DK, a.DV = b.DV, a.dim = b.s.dim, a.vdim = b.s.vdim;
     a.tau = b.s.tau, a.out_scale = b.s.out_scale, a.taps = b.s.kind == JGPT_MIX_DELTA ? b.s.taps : 0;
     a.conv_q = b.conv_q, a.conv_k = b.conv_k, a.conv_v = b.conv_v, a.decay_bias = b.bias, a.a_log = b.a_log, a.norm_w = b.norm;
     a.conv_off = b.conv_off, a.out_off = b.out;
-    a.norm_stride = b.s.kind == JGPT_MIX_WKV ? b.DV : 0, a.bonus = b.bonus, a.lower = b.lower;
+    a.norm_stride = b.s.kind == JGPT_MIX_WKV || b.s.kind == JGPT_MIX_GENERAL_DELTA ? b.DV : 0, a.removal_bias = b.removal_bias, a.rate = b.s.decay_rate, a.bonus = b.bonus, a.lower = b.lower;
     if (b.s.kind == JGPT_MIX_HGRN2) a.z_off = b.f;
     return a;
 }
@@ -297,9 +314,26 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
             b.q = seg(s.heads * b.maps * b.DK), b.k = seg(s.kv_heads * b.maps * b.DK), b.v = seg(s.kv_heads * b.DV);
             if (s.gate) b.g = seg(s.gate == mix::GATE_HEAD ? s.heads : s.heads * b.DV);
             if (s.rot_dims) TRY(find_rotation(d, s, &b.rot));
-            if (s.qk_norm) {
-                TRY(dalloc(d, (void **)&b.q_norm, sizeof(float) * (uint64_t)s.dim));
-                TRY(dalloc(d, (void **)&b.k_norm, sizeof(float) * (uint64_t)s.dim));
+            JGPT_REQUIRE(s.qk_norm >= 0 && s.qk_norm <= JGPT_QK_NORM_UNIT && (s.qk_norm != JGPT_QK_NORM_ALL || b.maps == 1), JGPT_ERR_UNSUPPORTED,
+                         "layer %d: norm %d of queries and keys, %d maps", index, s.qk_norm, b.maps);
+            JGPT_REQUIRE(s.window >= 0 && s.keep >= 0 && !(s.window && s.chunk) && (s.window || !s.keep) && s.sink >= 0 && s.sink <= JGPT_SINK_ZERO &&
+                             (!s.sink || b.maps == 1),
+                         JGPT_ERR_INVALID_ARGUMENT, "layer %d: window %d with %d kept, chunk %d, sink %d, %d maps", index, s.window, s.keep, s.chunk, s.sink, b.maps);
+            if (s.qk_norm == JGPT_QK_NORM_HEAD || s.qk_norm == JGPT_QK_NORM_ALL) {
+                const bool all = s.qk_norm == JGPT_QK_NORM_ALL;
+                TRY(dalloc(d, (void **)&b.q_norm, sizeof(float) * (uint64_t)(all ? s.heads * b.DK : s.dim)));
+                TRY(dalloc(d, (void **)&b.k_norm, sizeof(float) * (uint64_t)(all ? s.kv_heads * b.DK : s.dim)));
+            }
+            if (s.sink) TRY(dalloc(d, (void **)&b.sink, sizeof(float) * (uint64_t)s.heads));  // zeros
+            if (s.v_mix) {
+                JGPT_REQUIRE(ls.n_branches == 1, JGPT_ERR_UNSUPPORTED, "layer %d: mixed values stand alone in their layer", index);
+                if (d->v_first) {
+                    JGPT_REQUIRE(d->v_first->s.kv_heads * d->v_first->s.vdim == s.kv_heads * s.vdim, JGPT_ERR_INVALID_ARGUMENT,
+                                 "layer %d: values of %d x %d are mixed with %d x %d", index, s.kv_heads, s.vdim, d->v_first->s.kv_heads, d->v_first->s.vdim);
+                    b.v_first = d->v_first;
+                } else {
+                    y.v_source = true;
+                }
             }
             b.kv_layer = (int)d->kv.size();
             KvLayerGeom geom;
@@ -360,6 +394,21 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
             mix::RecArgs ra = rec_args(b);
             ra.shift_width = wkv ? W : 0;
             d->state_stride += mix::rec_state_bytes(ra, eb, &b.conv_off);
+        } else if (s.kind == JGPT_MIX_GENERAL_DELTA) {
+            JGPT_REQUIRE(s.kv_heads == s.heads && s.rank_a > 0 && s.decay_rate > 0.f && d->rms && ls.n_branches == 1, JGPT_ERR_INVALID_ARGUMENT,
+                         "layer %d: heads %d / %d, rank %d, decay rate %g, %d branches", index, s.heads, s.kv_heads, s.rank_a, (double)s.decay_rate, ls.n_branches);
+            b.DK = mix::rec_padded_key(s.dim), b.DV = mix::rec_padded_value(s.vdim);
+            JGPT_REQUIRE(b.DK > 0 && b.DV > 0, JGPT_ERR_UNSUPPORTED, "layer %d: head sizes %d / %d", index, s.dim, s.vdim);
+            const int hk = s.heads * b.DK, hv = s.heads * b.DV;
+            b.q = seg(hk), b.k = seg(hk), b.v = seg(hv), b.g = seg(hv), b.b = seg(hk);
+            b.ra = up(s.rank_a, 8), b.a1 = seg(s.rank_a), y.tanh_from = b.a1, y.tanh_to = b.a1 + b.ra;
+            b.za = zc, zc += hk;
+            TRY(dalloc(d, &b.w_a2, (uint64_t)hk * b.ra * eb));
+            TRY(dalloc(d, (void **)&b.bias, sizeof(float) * (uint64_t)hk));
+            TRY(dalloc(d, (void **)&b.removal_bias, sizeof(float) * (uint64_t)hk));
+            TRY(dalloc(d, (void **)&b.norm, sizeof(float) * (uint64_t)hv));
+            b.state_off = d->state_stride;
+            d->state_stride += mix::rec_state_bytes(rec_args(b), eb, &b.conv_off);
         } else if (s.kind == JGPT_MIX_LATENT) {
             JGPT_REQUIRE(s.q_rank > 0 && s.kv_rank > 0 && s.window >= 0 && s.rot_dims > 0 && s.rot_dims % 2 == 0 && s.rot_dims <= s.rot_dim && s.rot_base > 1.0,
                          JGPT_ERR_INVALID_ARGUMENT, "layer %d: latents of %d / %d, window %d, rotation of %d / %d", index, s.q_rank, s.kv_rank, s.window,
@@ -396,13 +445,26 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
         out += b.cols();
         y.br.push_back(b);
     }
+    const bool gated = d->s.residual_gate;
+    y.n_mix = in;
+    if (gated) in += d->ldw;
     y.n_in = in, y.n_out = up(out, 8), y.n_z = zc, y.ff = ls.ff, y.ffp = up(ls.ff, 16), y.ff_kind = ls.ff_kind;
-    JGPT_REQUIRE(ls.ff_kind >= JGPT_FF_GATED_GELU && ls.ff_kind <= JGPT_FF_MOE, JGPT_ERR_UNSUPPORTED, "layer %d: feed-forward kind %d", index, ls.ff_kind);
-    JGPT_REQUIRE(!d->s.norm_after || !y.shift(), JGPT_ERR_UNSUPPORTED, "layer %d: WKV mixes normed inputs", index);
-    for (const DBranch &b : y.br)
-        if (b.s.kind == JGPT_MIX_ATTENTION && b.s.qkv_bias && !y.bias_in) TRY(dalloc(d, (void **)&y.bias_in, sizeof(float) * (uint64_t)y.n_in));
+    JGPT_REQUIRE(ls.ff_kind >= JGPT_FF_GATED_GELU && ls.ff_kind <= JGPT_FF_RELU2, JGPT_ERR_UNSUPPORTED, "layer %d: feed-forward kind %d", index, ls.ff_kind);
+    JGPT_REQUIRE((!d->s.norm_after && !d->s.norm_both) || !y.shift(), JGPT_ERR_UNSUPPORTED, "layer %d: WKV mixes inputs normed in front of it alone", index);
+    const bool one_up = y.ff_kind == JGPT_FF_XIELU || y.ff_kind == JGPT_FF_RELU2;
+    JGPT_REQUIRE(!gated || !y.ff || one_up, JGPT_ERR_UNSUPPORTED, "layer %d: a gated result of feed-forward kind %d", index, y.ff_kind);
+    y.n_up = y.ffp + (gated ? d->ldw : 0);
+    bool biased = gated;
+    for (const DBranch &b : y.br) biased = biased || (b.s.kind == JGPT_MIX_ATTENTION && b.s.qkv_bias);
+    if (biased) TRY(dalloc(d, (void **)&y.bias_in, sizeof(float) * (uint64_t)y.n_in));
     if (y.ff && y.ff_kind == JGPT_FF_MOE) TRY(plan_moe(d, y, ls.moe, index));
-    if (d->rms && !d->s.norm_after) {
+    if (d->s.norm_both) {
+        for (float **p : {&y.post1, &y.post2, &y.share}) TRY(dalloc(d, (void **)p, sizeof(float) * (uint64_t)d->ldw));
+        if (gated && y.ff) TRY(dalloc(d, (void **)&y.bias_up, sizeof(float) * (uint64_t)y.n_up));
+        y.shift_off = d->state_stride;
+        if (d->s.token_shift) d->state_stride += up((int)(2 * sizeof(float)) * d->ldw, 256);
+    }
+    if (d->rms && !d->s.norm_after && !d->s.norm_both) {
         TRY(dalloc(d, (void **)&y.ls1, sizeof(float) * (uint64_t)W));
         TRY(dalloc(d, (void **)&y.ls2, sizeof(float) * (uint64_t)W));
         const std::vector<float> mult((size_t)W, d->s.residual_mult);
@@ -410,15 +472,15 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
     }
     if (d->s.depth_average) TRY(dalloc(d, (void **)&y.dwa, sizeof(float) * (uint64_t)(index + 2)));
     TRY(dalloc(d, &y.w_in, (uint64_t)y.n_in * d->ldw * eb));
-    TRY(dalloc(d, &y.w_out, (uint64_t)W * y.n_out * eb));
-    TRY(dalloc(d, (void **)&y.n1w, sizeof(float) * (uint64_t)W));
+    TRY(dalloc(d, &y.w_out, (uint64_t)d->ldw * y.n_out * eb));
+    TRY(dalloc(d, (void **)&y.n1w, sizeof(float) * (uint64_t)d->ldw));
     TRY(dalloc(d, (void **)&y.n1b, sizeof(float) * (uint64_t)W));
     if (y.ff) {
         if (y.ff_kind != JGPT_FF_MOE) {
-            TRY(dalloc(d, &y.w_gu, (y.ff_kind == JGPT_FF_XIELU ? 1ull : 2ull) * y.ffp * d->ldw * eb));
-            TRY(dalloc(d, &y.w_down, (uint64_t)W * y.ffp * eb));
+            TRY(dalloc(d, &y.w_gu, (uint64_t)(one_up ? y.n_up : 2 * y.ffp) * d->ldw * eb));
+            TRY(dalloc(d, &y.w_down, (uint64_t)d->ldw * y.ffp * eb));
         }
-        TRY(dalloc(d, (void **)&y.n2w, sizeof(float) * (uint64_t)W));
+        TRY(dalloc(d, (void **)&y.n2w, sizeof(float) * (uint64_t)d->ldw));
         TRY(dalloc(d, (void **)&y.n2b, sizeof(float) * (uint64_t)W));
     }
     return JGPT_OK;
@@ -432,13 +494,17 @@ static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
     d->long_min = mix::rec_chunk_min_tokens(d->f32);
     d->rms = d->s.norm == JGPT_NORM_RMS;
     d->lat_min = env_int("JGPT_B200_LATENT_EXPAND_MIN", 64);
-    int n_in = 8, n_z = 8, n_out = 8, ffp = 16, raw = 0, mixes = 1, cq = 0, lq = 0, lqa = 0, cxw = 0, kvx = 0;
+    int n_in = 8, n_z = 8, n_out = 8, ffp = 16, raw = 0, mixes = d->s.norm_both ? 2 : 1, cq = 0, lq = 0, lqa = 0, cxw = 0, kvx = 0;
     int top = 0, experts = 0, outputs = 0, effp = 0, sffp = 0, tiles = 0;
     bool latent = false, unbounded = false, expand = true;
     for (int i = 0; i < d->s.n_layers; i++) {
         DLayer &y = d->L[(size_t)i];
         TRY(plan_layer(d, y, layers[i], i));
-        n_in = std::max(n_in, y.n_in), n_z = std::max(n_z, y.n_z), n_out = std::max(n_out, y.n_out), ffp = std::max(ffp, y.ffp);
+        n_in = std::max(n_in, y.n_in), n_z = std::max(n_z, y.n_z), n_out = std::max(n_out, y.n_out), ffp = std::max(ffp, y.n_up);
+        if (y.v_source) {
+            d->v_first = &y.br[0], d->v_first_ld = y.n_in;
+            TRY(dalloc(d, &d->proj_first, R * y.n_in * eb));
+        }
         top = std::max(top, y.moe.top), experts = std::max(experts, y.moe.experts), outputs = std::max(outputs, y.n_router);
         effp = std::max(effp, y.effp), sffp = std::max(sffp, y.sffp);
         if (y.effp) tiles = std::max(tiles, std::min(y.moe.experts, d->R * y.moe.top) + d->R * y.moe.top / 16);
@@ -459,8 +525,12 @@ static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
     TRY(dalloc(d, &d->embed, (uint64_t)d->s.vocab * d->ldw * eb));
     if (d->s.pos_table) TRY(dalloc(d, &d->pos, (uint64_t)d->s.max_positions * d->ldw * eb));
     if (d->s.head) TRY(dalloc(d, &d->head, (uint64_t)d->s.vocab * d->ldw * eb));
-    for (float **p : {&d->enw, &d->enb, &d->fnw, &d->fnb}) TRY(dalloc(d, (void **)p, sizeof(float) * W));
-    TRY(dalloc(d, (void **)&d->x, sizeof(float) * R * W));
+    for (float **p : {&d->enw, &d->enb, &d->fnw, &d->fnb}) TRY(dalloc(d, (void **)p, sizeof(float) * d->ldw));
+    TRY(dalloc(d, (void **)&d->x, sizeof(float) * R * d->ldw));
+    if (d->s.norm_both) {
+        TRY(dalloc(d, (void **)&d->x_next, sizeof(float) * R * d->ldw));
+        TRY(dalloc(d, &d->y, R * d->ldw * eb));
+    }
     if (d->s.depth_average) TRY(dalloc(d, (void **)&d->slots, sizeof(float) * (d->L.size() + 1) * R * W));
     for (mix::Rotation &r : d->rots) TRY(dalloc(d, (void **)&r.out, sizeof(float2) * R * r.half));
     if (top) {
@@ -494,6 +564,7 @@ static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
             TRY(dalloc(d, &d->kvx, (uint64_t)d->kvx_rows * kvx * eb));
         }
     }
+    TRY(dalloc(d, (void **)&d->row_inv, sizeof(float2) * R));
     TRY(dalloc(d, (void **)&d->raw, sizeof(float) * R * raw));
     TRY(dalloc(d, (void **)&d->chunk_ws, sizeof(float) * d->chunk_ws_floats));
     TRY(dalloc(d, &d->h, R * mixes * d->ldw * eb));
@@ -519,7 +590,11 @@ static int32_t build(Decoder *d, const jgpt_layer_spec *layers) {
 // ------------------------------------------------------------------------------------------------
 static uint64_t bit(int role) { return 1ull << role; }
 
-static uint64_t needed_roles(const jgpt_mixer_spec &s) {
+static uint64_t needed_roles(const DBranch &b) {
+    const jgpt_mixer_spec &s = b.s;
+    if (s.kind == JGPT_MIX_GENERAL_DELTA)
+        return bit(JGPT_W_Q) | bit(JGPT_W_K) | bit(JGPT_W_V) | bit(JGPT_W_G) | bit(JGPT_W_O) | bit(JGPT_W_A1) | bit(JGPT_W_A2) | bit(JGPT_W_DECAY_BIAS) |
+               bit(JGPT_W_B) | bit(JGPT_W_B_BIAS) | bit(JGPT_W_HEAD_NORM);
     if (s.kind == JGPT_MIX_LATENT)
         return bit(JGPT_W_DQ) | bit(JGPT_W_DQ_NORM) | bit(JGPT_W_UQ) | bit(JGPT_W_UK) | bit(JGPT_W_UV) | bit(JGPT_W_O) |
                (s.kv_from ? 0 : bit(JGPT_W_DKV) | bit(JGPT_W_DKV_NORM));
@@ -531,7 +606,8 @@ static uint64_t needed_roles(const jgpt_mixer_spec &s) {
     uint64_t n = bit(JGPT_W_Q) | bit(JGPT_W_K) | bit(JGPT_W_V) | bit(JGPT_W_O);
     if (s.kind == JGPT_MIX_ATTENTION)
         return n | (s.gate ? bit(JGPT_W_G) : 0) | (s.qkv_bias ? bit(JGPT_W_Q_BIAS) | bit(JGPT_W_K_BIAS) | bit(JGPT_W_V_BIAS) : 0) |
-               (s.qk_norm ? bit(JGPT_W_Q_NORM) | bit(JGPT_W_K_NORM) : 0) |
+               (b.q_norm ? bit(JGPT_W_Q_NORM) | bit(JGPT_W_K_NORM) : 0) | (s.sink == JGPT_SINK_LEARNED ? bit(JGPT_W_SINK) : 0) |
+               (b.v_first ? bit(JGPT_W_VMIX) : 0) |
                (s.maps > 1 ? bit(JGPT_W_LQ1) | bit(JGPT_W_LK1) | bit(JGPT_W_LQ2) | bit(JGPT_W_LK2) : 0);
     n |= bit(JGPT_W_A1) | bit(JGPT_W_A2) | bit(JGPT_W_DECAY_BIAS) | bit(JGPT_W_HEAD_NORM);
     if (s.kind == JGPT_MIX_GLA) return n | bit(JGPT_W_G);
@@ -556,10 +632,16 @@ static int32_t missing_weights(const Decoder *d) {
                 JGPT_REQUIRE((y.have_expert[k] & e) == e, JGPT_ERR_ILLEGAL_STATE, "expert %zu of layer %zu is not set", k, i);
         } else if (y.ff)
             n |= bit(JGPT_W_NORM2) | (beta & bit(JGPT_W_NORM2_B)) | bit(JGPT_W_FF_UP) | bit(JGPT_W_FF_DOWN) | (d->s.layer_scale ? bit(JGPT_W_LS2) : 0) |
-                 (y.ff_kind == JGPT_FF_XIELU ? bit(JGPT_W_FF_ACT) : bit(JGPT_W_FF_GATE));
+                 (y.ff_kind == JGPT_FF_XIELU ? bit(JGPT_W_FF_ACT) : y.ff_kind == JGPT_FF_RELU2 ? 0 : bit(JGPT_W_FF_GATE));
         JGPT_REQUIRE((y.have & n) == n, JGPT_ERR_ILLEGAL_STATE, "norm or feed-forward weights of layer %zu are not set", i);
+        if (d->s.norm_both) {
+            auto at = [](int role) { return bit(role - JGPT_W_POST1); };
+            const uint64_t m = at(JGPT_W_POST1) | (d->s.token_shift ? at(JGPT_W_SHIFT) : 0) | (d->s.residual_gate ? at(JGPT_W_RG1) | at(JGPT_W_RG1_B) : 0) |
+                               (y.ff ? at(JGPT_W_POST2) | (d->s.residual_gate ? at(JGPT_W_RG2) | at(JGPT_W_RG2_B) : 0) : 0);
+            JGPT_REQUIRE((y.have_both & m) == m, JGPT_ERR_ILLEGAL_STATE, "norms behind the parts, shift or gates of layer %zu are not set", i);
+        }
         for (const DBranch &b : y.br)
-            JGPT_REQUIRE((b.have & needed_roles(b.s)) == needed_roles(b.s), JGPT_ERR_ILLEGAL_STATE, "mixer weights of layer %zu are not set", i);
+            JGPT_REQUIRE((b.have & needed_roles(b)) == needed_roles(b), JGPT_ERR_ILLEGAL_STATE, "mixer weights of layer %zu are not set", i);
     }
     return JGPT_OK;
 }
@@ -605,6 +687,22 @@ static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const flo
             return fail(JGPT_ERR_INVALID_ARGUMENT, "tensor %d does not belong to an expert", role);
         }
         y.have_expert[(size_t)e] |= (uint8_t)bit(role - 64);
+        return JGPT_OK;
+    }
+    if (branch < 0 && role >= JGPT_W_POST1) {
+        const bool ff_role = role == JGPT_W_POST2 || role == JGPT_W_RG2 || role == JGPT_W_RG2_B, gate = role >= JGPT_W_RG1;
+        JGPT_REQUIRE(d->s.norm_both && role <= JGPT_W_RG2_B && (!ff_role || y.ff) && (!gate || d->s.residual_gate) && (role != JGPT_W_SHIFT || d->s.token_shift),
+                     JGPT_ERR_INVALID_ARGUMENT, "tensor %d does not belong to layer %d", role, layer);
+        switch (role) {
+            case JGPT_W_POST1: TRY(shape(1, W)); TRY(put_floats(d, y.post1, src, 1, W, none)); break;
+            case JGPT_W_POST2: TRY(shape(1, W)); TRY(put_floats(d, y.post2, src, 1, W, none)); break;
+            case JGPT_W_SHIFT: TRY(shape(1, W)); TRY(put_floats(d, y.share, src, 1, W, none)); break;
+            case JGPT_W_RG1: TRY(shape(W, W)); TRY(put_matrix(d, y.w_in, d->ldw, y.n_mix, 0, src, W, W, none, none)); break;
+            case JGPT_W_RG1_B: TRY(shape(1, W)); TRY(put_floats(d, y.bias_in + y.n_mix, src, 1, W, none)); break;
+            case JGPT_W_RG2: TRY(shape(W, W)); TRY(put_matrix(d, y.w_gu, d->ldw, y.ffp, 0, src, W, W, none, none)); break;
+            case JGPT_W_RG2_B: TRY(shape(1, W)); TRY(put_floats(d, y.bias_up + y.ffp, src, 1, W, none)); break;
+        }
+        y.have_both |= bit(role - JGPT_W_POST1);
         return JGPT_OK;
     }
     if (branch < 0 && role >= 64) {
@@ -655,7 +753,7 @@ static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const flo
             }
             case JGPT_W_FF_GATE:
             case JGPT_W_FF_UP: {
-                if (y.ff_kind == JGPT_FF_XIELU) {
+                if (y.ff_kind == JGPT_FF_XIELU || y.ff_kind == JGPT_FF_RELU2) {
                     JGPT_REQUIRE(role == JGPT_W_FF_UP, JGPT_ERR_INVALID_ARGUMENT, "layer %d: the feed-forward part has no gate", layer);
                     TRY(shape(y.ff, W));
                     TRY(put_matrix(d, y.w_gu, d->ldw, 0, 0, src, rows, cols, none, none));
@@ -677,7 +775,7 @@ static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const flo
     JGPT_REQUIRE(branch < (int)y.br.size(), JGPT_ERR_OUT_OF_RANGE, "layer %d has %zu mixer branches", layer, y.br.size());
     DBranch &b = y.br[(size_t)branch];
     const jgpt_mixer_spec &s = b.s;
-    JGPT_REQUIRE(role >= 0 && role < 63 && (needed_roles(s) & bit(role)), JGPT_ERR_INVALID_ARGUMENT, "tensor %d does not belong to mixer kind %d", role,
+    JGPT_REQUIRE(role >= 0 && role < 64 && (needed_roles(b) & bit(role)), JGPT_ERR_INVALID_ARGUMENT, "tensor %d does not belong to mixer kind %d", role,
                  s.kind);
     const bool att = s.kind == JGPT_MIX_ATTENTION;
     const Grouping kg{s.dim, b.DK}, vg{s.vdim, b.DV};
@@ -697,8 +795,17 @@ static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const flo
         case JGPT_W_Q_BIAS: TRY(shape(1, qheads * s.dim)); TRY(put_floats(d, y.bias_in + b.q, src, cols, 1, kg)); break;
         case JGPT_W_K_BIAS: TRY(shape(1, kheads * s.dim)); TRY(put_floats(d, y.bias_in + b.k, src, cols, 1, kg)); break;
         case JGPT_W_V_BIAS: TRY(shape(1, vheads * s.vdim)); TRY(put_floats(d, y.bias_in + b.v, src, cols, 1, vg)); break;
-        case JGPT_W_Q_NORM: TRY(shape(1, s.dim)); TRY(put_floats(d, b.q_norm, src, 1, cols, none)); break;
-        case JGPT_W_K_NORM: TRY(shape(1, s.dim)); TRY(put_floats(d, b.k_norm, src, 1, cols, none)); break;
+        case JGPT_W_Q_NORM:
+        case JGPT_W_K_NORM: {
+            float *dst = role == JGPT_W_Q_NORM ? b.q_norm : b.k_norm;
+            const bool all = s.qk_norm == JGPT_QK_NORM_ALL;
+            TRY(shape(1, all ? (role == JGPT_W_Q_NORM ? s.heads : s.kv_heads) * s.dim : s.dim));
+            TRY(all ? put_floats(d, dst, src, cols, 1, kg) : put_floats(d, dst, src, 1, cols, none));
+            break;
+        }
+        case JGPT_W_SINK: TRY(shape(1, s.heads)); TRY(put_floats(d, b.sink, src, 1, cols, none)); break;
+        case JGPT_W_VMIX: TRY(shape(1, 1)); b.v_share = src[0]; break;
+        case JGPT_W_B_BIAS: TRY(shape(1, s.heads * s.dim)); TRY(put_floats(d, b.removal_bias, src, cols, 1, kg)); break;
         case JGPT_W_LQ1:
         case JGPT_W_LK1:
         case JGPT_W_LQ2:
@@ -712,7 +819,10 @@ static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const flo
             b.lambda = (float)(std::exp(dot[0]) - std::exp(dot[1]) + (double)s.diff);
             break;
         }
-        case JGPT_W_B: TRY(into_proj(b.b, s.heads, none)); break;
+        case JGPT_W_B:
+            if (s.kind == JGPT_MIX_GENERAL_DELTA) TRY(into_proj(b.b, s.heads * s.dim, kg));
+            else TRY(into_proj(b.b, s.heads, none));
+            break;
         case JGPT_W_A1: TRY(into_proj(b.a1, s.rank_a, none)); break;
         case JGPT_W_G1: TRY(into_proj(b.g1, s.rank_g, none)); break;
         case JGPT_W_A2: TRY(shape(s.heads * s.dim, s.rank_a)); TRY(put_matrix(d, b.w_a2, b.ra, 0, 0, src, rows, cols, kg, none)); break;
@@ -720,7 +830,7 @@ static int32_t set_tensor(Decoder *d, int layer, int branch, int role, const flo
         case JGPT_W_DECAY_BIAS: TRY(shape(1, s.heads * s.dim)); TRY(put_floats(d, b.bias, src, cols, 1, kg)); break;
         case JGPT_W_A_LOG: TRY(shape(1, s.heads)); TRY(put_floats(d, b.a_log, src, 1, cols, none)); break;
         case JGPT_W_HEAD_NORM:
-            if (s.kind == JGPT_MIX_WKV) {
+            if (s.kind == JGPT_MIX_WKV || s.kind == JGPT_MIX_GENERAL_DELTA) {
                 TRY(shape(1, s.heads * s.vdim));
                 TRY(put_floats(d, b.norm, src, cols, 1, vg));
             } else {
@@ -880,6 +990,33 @@ static int32_t enqueue_moe(Decoder *d, const DLayer &y, int R, int pdl, mix::Moe
     return JGPT_OK;
 }
 
+static void set_activation(const DLayer &y, nt::Problem &p) {
+    switch (y.ff_kind) {
+        case JGPT_FF_XIELU: p.act = nt::ACT_XIELU, p.p0 = y.act_p0, p.p1 = y.act_p1; break;
+        case JGPT_FF_RELU2: p.act = nt::ACT_RELU2; break;
+        case JGPT_FF_GATED_RELU: p.act = nt::ACT_RELU; break;
+        default: p.act = nt::ACT_GELU;
+    }
+}
+
+// Norms on both sides: the state of the residual stream between two launches, x and the part whose result it still lacks.
+static mix::PartNorm open_norm(const Decoder *d) {
+    mix::PartNorm n{};
+    n.mult = d->s.residual_mult;
+    return n;
+}
+// Adds what is open, norms the sum for the next part; afterwards nothing is open.
+template <class Fn>
+static int32_t close_norm(Decoder *d, const mix::StepDesc &sd, mix::PartNorm &open, const float *pre, void *h, int pdl, Fn &&more) {
+    mix::PartNorm n = open;
+    n.x_out = n.x == d->x ? d->x_next : d->x, n.pre = pre, n.h = h;
+    more(n);
+    TRY(mix::launch_part_norm(d->f32, sd, residual(d, 0), n, nullptr, sd.rows, d->s.eps, d->s.width, d->ldw, d->ctx->sm_count, d->ctx->d_status,
+                              n.x ? pdl : pdl & 2, d->ctx->stream));
+    open = open_norm(d), open.x = n.x_out;
+    return JGPT_OK;
+}
+
 static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, const std::vector<LatentBatch> &batches, uint64_t capture_rows) {
     const int W = d->s.width, R = sd.rows, ldw = d->ldw, eb = d->eb;
     const float eps = d->s.eps;
@@ -887,12 +1024,20 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
     int *status = d->ctx->d_status;
     const int pdl = d->overlap && !d->f32 && !capture_rows ? 3 : 0;
     const uint64_t slot = (uint64_t)d->R * W, mix_stride = (uint64_t)d->R * ldw;
-    const bool deep = d->s.depth_average, after = d->s.norm_after;
+    const bool deep = d->s.depth_average, after = d->s.norm_after, both = d->s.norm_both, gated_result = d->s.residual_gate;
+    mix::PartNorm next = d->open = open_norm(d);
     const float res_scale = after ? d->s.residual_scale : 1.f;
     for (size_t i = 0; i < d->L.size(); i++) {
         DLayer &y = d->L[i];
         float *from = d->x, *to = deep ? d->slots + (i + 1) * slot : d->x;  // residual in front of the layer, its result
-        if (after) {  // the norms behind the sums leave h
+        uint8_t *rows_shifted = reinterpret_cast<uint8_t *>(d->h), *rows_plain = d->s.token_shift ? rows_shifted + mix_stride * eb : rows_shifted;
+        void *layer_proj = y.v_source ? d->proj_first : d->proj;
+        if (both) {
+            TRY(close_norm(d, sd, next, y.n1w, rows_plain, pdl, [&](mix::PartNorm &n) {
+                if (!d->s.token_shift) return;
+                n.shifted = rows_shifted, n.share = y.share, n.state = p->state + y.shift_off, n.state_stride = p->state_stride, n.max_seqs = p->max_seqs;
+            }));
+        } else if (after) {  // the norms behind the sums leave h
             if (i == 0)
                 TRY(mix::launch_residual_norm(d->f32, sd, residual(d, 0), nullptr, R, nullptr, eps, d->x, d->h, mix::ShiftArgs{}, W, ldw, status, pdl & 2, st));
         } else if (d->rms) {
@@ -920,18 +1065,24 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
             in[0].seg_n = hk, in[0].a_seg = (long long)mix_stride, in[1].act = nt::ACT_TANH;
             TRY(product(d, in, 2, nt::EPI_ACT, pdl));
         } else {
-            nt::Problem in{d->h, y.w_in, d->proj, nullptr, R, y.n_in, ldw, ldw, ldw, y.n_in, 1.f};
+            nt::Problem in{d->h, y.w_in, layer_proj, nullptr, R, y.n_in, ldw, ldw, ldw, y.n_in, 1.f};
             in.bias = y.bias_in;
-            TRY(product(d, &in, 1, nt::EPI_STORE, pdl));
+            if (gated_result && d->s.token_shift) in.seg_n = y.n_mix, in.a_seg = (long long)mix_stride, in.a_cap = 1;
+            if (y.tanh_to) in.act = nt::ACT_TANH, in.act_from = y.tanh_from, in.act_to = y.tanh_to;
+            TRY(product(d, &in, 1, y.tanh_to ? nt::EPI_ACT : nt::EPI_STORE, pdl));
         }
         for (DBranch &b : y.br) {
             if (b.s.kind == JGPT_MIX_ATTENTION) {
                 mix::AttnArgs a{};
-                a.proj = d->proj, a.ldp = y.n_in, a.q_off = b.q, a.k_off = b.k, a.v_off = b.v, a.g_off = b.g;
+                a.proj = layer_proj, a.ldp = y.n_in, a.q_off = b.q, a.k_off = b.k, a.v_off = b.v, a.g_off = b.g;
                 a.heads = b.s.heads, a.kv_heads = b.s.kv_heads, a.maps = b.maps, a.DK = b.DK, a.DV = b.DV, a.dim = b.s.dim, a.vdim = b.s.vdim;
                 a.gate = b.s.gate, a.chunk = b.s.chunk, a.scale = b.s.score_scale, a.out_scale = b.s.out_scale;
                 a.q_norm = b.q_norm, a.k_norm = b.k_norm, a.eps = eps, a.interleaved = b.s.rot_interleaved;
                 if (b.rot >= 0) a.cs = d->rots[(size_t)b.rot].out, a.half = b.s.rot_dims / 2;
+                a.qk_norm = b.s.qk_norm, a.row_inv = d->row_inv, a.window = b.s.window, a.keep = b.s.keep, a.sink = b.sink;
+                if (const DBranch *f = b.v_first)
+                    a.v_first = reinterpret_cast<uint8_t *>(d->proj_first) + (size_t)f->v * eb, a.ld_first = d->v_first_ld, a.vdim_first = f->s.vdim, a.DV_first = f->DV,
+                    a.v_share = b.v_share;
                 a.lambda = b.lambda, a.diff_scale = 1.f - b.s.diff;
                 a.kv = p->vkv + p->vlayers[(size_t)b.kv_layer].offset, a.table = p->d_table, a.n_blocks = p->n_blocks, a.mbs = p->max_blocks_per_seq;
                 a.out = d->mixed, a.ldo = y.n_out, a.out_off = b.out;
@@ -956,6 +1107,34 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
                 TRY(mix::launch_recurrent(d->f32, sd, a, pdl, st));
             }
         }
+        if (both) {
+            nt::Problem out{d->mixed, y.w_out, d->y, nullptr, R, ldw, y.n_out, y.n_out, y.n_out, ldw, 1.f};
+            TRY(product(d, &out, 1, nt::EPI_STORE, pdl));
+            next.y = d->y, next.post = y.post1;
+            if (gated_result) next.gate = reinterpret_cast<uint8_t *>(layer_proj) + (size_t)y.n_mix * eb, next.ldg = y.n_in;
+            if (y.ff) {
+                TRY(close_norm(d, sd, next, y.n2w, d->h, pdl, [](mix::PartNorm &) {}));
+                const bool one = y.ff_kind == JGPT_FF_XIELU || y.ff_kind == JGPT_FF_RELU2;
+                const int n_act = one ? y.n_up : y.ffp;
+                nt::Problem in{d->h, y.w_gu, d->act, nullptr, R, one ? y.n_up : 2 * y.ffp, ldw, ldw, ldw, n_act, 1.f};
+                set_activation(y, in);
+                in.act_to = one ? y.ffp : in.act_to, in.bias = y.bias_up;
+                TRY(product(d, &in, 1, one ? nt::EPI_ACT : nt::EPI_GATE, pdl));
+                nt::Problem down{d->act, y.w_down, d->y, nullptr, R, ldw, y.ffp, n_act, y.ffp, ldw, 1.f};
+                TRY(product(d, &down, 1, nt::EPI_STORE, pdl));
+                next.y = d->y, next.post = y.post2;
+                if (gated_result) next.gate = reinterpret_cast<uint8_t *>(d->act) + (size_t)y.ffp * eb, next.ldg = n_act;
+            }
+            d->open = next;
+            if (capture_rows) {  // the sum as it will be formed in front of the next part
+                mix::PartNorm n = next;
+                n.x_out = next.x == d->x ? d->x_next : d->x;
+                TRY(mix::launch_part_norm(d->f32, sd, residual(d, 0), n, nullptr, R, eps, W, ldw, d->ctx->sm_count, status, 0, st));
+                JGPT_CUDA_TRY(cudaMemcpy2DAsync(d->capture + (uint64_t)i * capture_rows * W, sizeof(float) * W, n.x_out, sizeof(float) * ldw, sizeof(float) * W, capture_rows,
+                                                cudaMemcpyDeviceToHost, st));
+            }
+            continue;
+        }
         nt::Problem out{d->mixed, y.w_out, to, nullptr, R, W, y.n_out, y.n_out, y.n_out, W, 1.f};
         out.res = from, out.colscale = y.ls1, out.res_scale = res_scale;
         TRY(product(d, &out, 1, nt::EPI_ADD_F32, pdl));
@@ -971,10 +1150,9 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
             } else if (!after) {
                 TRY(mix::launch_layer_norm(d->f32, d->x, nullptr, mix::NormW{y.n2w, y.n2b}, eps, d->h, R, W, ldw, pdl, st));
             }
-            const bool gated = y.ff_kind != JGPT_FF_XIELU;
+            const bool gated = y.ff_kind != JGPT_FF_XIELU && y.ff_kind != JGPT_FF_RELU2;
             nt::Problem gu{d->h, y.w_gu, d->act, nullptr, R, gated ? 2 * y.ffp : y.ffp, ldw, ldw, ldw, y.ffp, 1.f};
-            gu.act = y.ff_kind == JGPT_FF_GATED_RELU ? nt::ACT_RELU : nt::ACT_GELU;
-            if (!gated) gu.act = nt::ACT_XIELU, gu.p0 = y.act_p0, gu.p1 = y.act_p1;
+            set_activation(y, gu);
             TRY(product(d, &gu, 1, gated ? nt::EPI_GATE : nt::EPI_ACT, pdl));
             nt::Problem down{d->act, y.w_down, to, nullptr, R, W, y.ffp, y.ffp, y.ffp, W, 1.f};
             down.colscale = y.ls2, down.res_scale = res_scale;
@@ -993,7 +1171,11 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
 static int32_t enqueue_head(Decoder *d, const mix::StepDesc &sd, int w0, int n, bool pick, const SampleSpec &spec) {
     cudaStream_t st = d->ctx->stream;
     const int pdl = d->overlap && !d->f32 && w0 == 0 ? 3 : 0;
-    if (d->rms)
+    if (d->s.norm_both) {
+        mix::PartNorm last = d->open;
+        last.pre = d->fnw, last.h = d->h;
+        TRY(mix::launch_part_norm(d->f32, sd, residual(d, 0), last, sd.want + w0, n, d->s.eps, d->s.width, d->ldw, d->ctx->sm_count, d->ctx->d_status, pdl, st));
+    } else if (d->rms)
         TRY(mix::launch_residual_norm(d->f32, sd, residual(d, d->L.size()), sd.want + w0, n, d->fnw, d->s.eps, nullptr, d->h, mix::ShiftArgs{}, d->s.width,
                                       d->ldw, d->ctx->d_status, pdl, st));
     else TRY(mix::launch_layer_norm(d->f32, d->x, sd.want + w0, mix::NormW{d->fnw, d->fnb}, d->s.eps, d->h, n, d->s.width, d->ldw, pdl, st));
@@ -1319,6 +1501,9 @@ int32_t jgpt_decoder_create(jgpt_ctx ctxh, const jgpt_decoder_spec *spec, const 
                  "layer norms go with embedding norms and learned positions, RMS norms with residual factors and depth averages");
     JGPT_REQUIRE(!spec->norm_after || (rms && !spec->layer_scale && !spec->depth_average && spec->residual_mult == 1.f), JGPT_ERR_UNSUPPORTED,
                  "norms behind the sums are RMS norms over a plain residual");
+    JGPT_REQUIRE(!spec->norm_both || (rms && !spec->norm_after && !spec->layer_scale && !spec->depth_average), JGPT_ERR_UNSUPPORTED,
+                 "norms on both sides are RMS norms without layer scales and depth averages");
+    JGPT_REQUIRE(spec->norm_both || (!spec->token_shift && !spec->residual_gate), JGPT_ERR_UNSUPPORTED, "token shifts and gated results go with norms on both sides");
     JGPT_REQUIRE(dtype == JGPT_DTYPE_BF16 || dtype == JGPT_DTYPE_F32, JGPT_ERR_INVALID_ARGUMENT, "dtype %d", dtype);
     JGPT_CUDA_TRY(make_current(c));
     Decoder *d = new Decoder();

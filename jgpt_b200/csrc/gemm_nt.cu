@@ -76,7 +76,7 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
         seg = 0;
     }
     const int seg_n = P.seg_n, n0 = seg * seg_n + tile % per_seg * kBN, n_end = min(N, (seg + 1) * seg_n), cn = seg * P.c_seg;
-    const __nv_bfloat16 *__restrict__ A = reinterpret_cast<const __nv_bfloat16 *>(P.A) + seg * P.a_seg;
+    const __nv_bfloat16 *__restrict__ A = reinterpret_cast<const __nv_bfloat16 *>(P.A) + min(seg, P.a_cap) * P.a_seg;
     const int nk_all = (K + kBK - 1) / kBK;
     const int kt0 = k_part * nk_all / args.k_split, nk = (k_part + 1) * nk_all / args.k_split - kt0;
 
@@ -200,7 +200,10 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
         } else if (m < M && n < n_end) {
             const size_t at = (size_t)m * P.ldc + n + cn;
             if (EPI == EPI_STORE) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(P.bias ? sum[i] + P.bias[n] : sum[i]);
-            if (EPI == EPI_ACT) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(activate<true>(P.act, P.p0, P.p1, sum[i]));
+            if (EPI == EPI_ACT) {
+                const float v = P.bias ? sum[i] + P.bias[n] : sum[i];
+                reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(n >= P.act_from && n < P.act_to ? activate<true>(P.act, P.p0, P.p1, v) : v);
+            }
             if (EPI == EPI_ADD_F32) reinterpret_cast<float *>(P.C)[at] = P.res_scale * P.res[at] + (P.colscale ? P.colscale[n] * sum[i] : sum[i]);
             if (EPI == EPI_SCALE_F32) reinterpret_cast<float *>(P.C)[at] = sum[i] * P.scale;
         }
@@ -248,7 +251,7 @@ static int32_t small_dispatch(const Ctx *ctx, const Problem *p, int n, int pdl, 
     int tiles = 0, K = 0;
     for (int i = 0; i < n; i++) {
         a.p[i] = p[i];
-        a.per_seg[i] = (p[i].seg_n + bn - 1) / bn, a.tiles[i] = p[i].segments() * a.per_seg[i];
+        a.per_seg[i] = (p[i].seg_n + bn - 1) / bn, a.tiles[i] = p[i].column_tiles(bn);
         if (GROUPED) a.tiles[i] *= i == 0 ? p[0].grp.max_tiles : (M + 16 * mt - 1) / (16 * mt);
         tiles += a.tiles[i];
         K = std::max(K, p[i].K);
@@ -326,7 +329,7 @@ __global__ void __launch_bounds__(256) gemm_nt_f32_kernel(const Problem P0, cons
     const int per_seg = (P.seg_n + BT - 1) / BT, seg = blockIdx.x / per_seg, cn = seg * P.c_seg;
     const int n0 = seg * P.seg_n + blockIdx.x % per_seg * BT, n_end = min(P.N, (seg + 1) * P.seg_n);
     if (n0 >= P.N) return;
-    const float *__restrict__ A = reinterpret_cast<const float *>(P.A) + seg * P.a_seg;
+    const float *__restrict__ A = reinterpret_cast<const float *>(P.A) + min(seg, P.a_cap) * P.a_seg;
     const float *__restrict__ W = reinterpret_cast<const float *>(P.W);
     int m0 = blockIdx.y * BT, m_end = P.M, src0 = 0;
     if (P.grp.tiles) {
@@ -372,7 +375,10 @@ __global__ void __launch_bounds__(256) gemm_nt_f32_kernel(const Problem P0, cons
                 if (n >= n_end) continue;
                 const size_t at = (size_t)m * P.ldc + n + cn;
                 if (EPI == EPI_STORE) C[at] = P.bias ? acc[i][j] + P.bias[n] : acc[i][j];
-                if (EPI == EPI_ACT) C[at] = activate<false>(P.act, P.p0, P.p1, acc[i][j]);
+                if (EPI == EPI_ACT) {
+                    const float v = P.bias ? acc[i][j] + P.bias[n] : acc[i][j];
+                    C[at] = n >= P.act_from && n < P.act_to ? activate<false>(P.act, P.p0, P.p1, v) : v;
+                }
                 if (EPI == EPI_ADD_F32) C[at] = P.res_scale * P.res[at] + (P.colscale ? P.colscale[n] * acc[i][j] : acc[i][j]);
                 if (EPI == EPI_SCALE_F32) C[at] = acc[i][j] * P.scale;
             }
@@ -389,7 +395,7 @@ int32_t launch_f32(const Problem *problems, int n, Epilogue epi, cudaStream_t st
         return launch_f32(p + 1, 1, epi, st);
     }
     JGPT_REQUIRE(!p[0].grp.tiles || p[0].grp.rows <= 64, JGPT_ERR_INVALID_ARGUMENT, "row tiles of %d", p[0].grp.rows);
-    auto tiles = [](const Problem &x) { return x.segments() * ((x.seg_n + 63) / 64); };
+    auto tiles = [](const Problem &x) { return x.column_tiles(64); };
     const dim3 grid((unsigned)std::max(tiles(p[0]), tiles(q)), (unsigned)(p[0].grp.tiles ? p[0].grp.max_tiles : (p[0].M + 63) / 64), (unsigned)n);
     switch (epi) {
         case EPI_STORE: gemm_nt_f32_kernel<EPI_STORE><<<grid, 256, 0, st>>>(p[0], q); break;

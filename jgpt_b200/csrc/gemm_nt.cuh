@@ -15,7 +15,7 @@ enum Epilogue : int {
     EPI_ADD_F32 = 1,   // C (fp32) = residual factor * residual + column factor * sum; every element is read and written by one thread
     EPI_SCALE_F32 = 2, // C (fp32) = sum * scale
     EPI_GATE = 3,      // W rows alternate in groups of 16: 16 of the gate, 16 of the linear part; C [M, N / 2] = act(gate) * linear
-    EPI_ACT = 4,       // C (activation type) = act(sum), the function picked per product
+    EPI_ACT = 4,       // C (activation type) = act(sum + bias), the function picked per product, for all columns or a range of them
 };
 enum Activation : int { ACT_NONE = 0, ACT_TANH = 1, ACT_XIELU = 2, ACT_GELU = 3, ACT_RELU = 4, ACT_RELU2 = 5 };
 
@@ -43,16 +43,22 @@ struct Problem {
     float scale = 1.f;
     // Segments: columns [s seg_n, (s + 1) seg_n) read the operand at A + s a_seg (elements) and land at column n + s c_seg of C.
     // a_seg is a multiple of lda (other rows) or less than lda (other columns of the same rows).  0: one segment.
-    int seg_n = 0, c_seg = 0;
+    // From segment a_cap on the operand stays where it is.
+    int seg_n = 0, c_seg = 0, a_cap = 1 << 30;
     long long a_seg = 0;
     const float *res = nullptr, *colscale = nullptr;  // EPI_ADD_F32: residual [M, ldc] (null: C itself), factor per column (null: 1)
     int act = ACT_NONE;                               // EPI_ACT
     float p0 = 0.f, p1 = 0.f;                         // its parameters
-    const float *bias = nullptr;                      // EPI_STORE: per column
+    int act_from = 0, act_to = 1 << 30;               // its columns; the others get the bias alone
+    const float *bias = nullptr;                      // EPI_STORE, EPI_ACT: per column
     float res_scale = 1.f;                            // EPI_ADD_F32
     RowGroups grp;                                    // tiles set: rows in groups (EPI_STORE, EPI_ACT; one segment)
     int segments() const { return seg_n > 0 ? (N + seg_n - 1) / seg_n : 1; }
     int segment_cols() const { return seg_n > 0 ? seg_n : N; }
+    int column_tiles(int bn) const {  // the last segment may be shorter
+        const int s = segments(), c = segment_cols();
+        return (s - 1) * ((c + bn - 1) / bn) + (N - (s - 1) * c + bn - 1) / bn;
+    }
 };
 
 // gelu(z) in its tanh form, 0.5 z (1 + tanh(u)) = z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3).

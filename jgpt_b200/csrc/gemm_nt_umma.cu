@@ -56,9 +56,9 @@ struct UmmaArgs {
     int M, N, K, ldc, mt, nt, pdl;
     float scale;
     int *status;
-    int per_seg, seg_n, c_seg, a_x, a_y;  // column tiles and columns of a segment; its shift in C; its operand's shift (columns, rows)
+    int per_seg, seg_n, c_seg, a_x, a_y, a_cap;  // column tiles and columns of a segment; its shift in C; its operand's shift (columns, rows), up to a_cap times
     const float *res, *colscale, *bias;
-    int act;
+    int act, act_from, act_to;
     float p0, p1, res_scale;
     const RowTile *tiles;  // groups: the row tiles, how many, each group's rows of W
     const int *n_tiles;
@@ -111,8 +111,8 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
             for (int t = blockIdx.x; t < total && !*s_abort; t += gridDim.x) {
                 int m, n;
                 tile_of(a, mt, t, m, n);
-                const int seg = n / a.per_seg, ax = seg * a.a_x;
-                int ay = seg * a.a_y + m * UM, wy = seg * a.seg_n + n % a.per_seg * BN;
+                const int seg = n / a.per_seg, shift = min(seg, a.a_cap), ax = shift * a.a_x;
+                int ay = shift * a.a_y + m * UM, wy = seg * a.seg_n + n % a.per_seg * BN;
                 if (ROWS != ROWS_ALL) ay = a.tiles[m].row0, wy += a.tiles[m].group * a.w_rows;
                 for (int kt = 0; kt < nk; kt++, it++) {
                     const uint32_t s = it % ST, use = it / ST;
@@ -177,7 +177,19 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
                 if (m >= m_end) continue;
                 if (EPI == EPI_STORE || EPI == EPI_ACT) {
                     __nv_bfloat16 *c = reinterpret_cast<__nv_bfloat16 *>(a.C) + (size_t)m * a.ldc + n0 + c0 + cn;
-                    if (EPI == EPI_ACT && a.act == ACT_XIELU) {
+                    const int n1 = n0 + c0;
+                    if (a.bias) {
+#pragma unroll
+                        for (int q = 0; q < 32; q++)
+                            if (n1 + q < n_end) v[q] += __ldg(a.bias + n1 + q);
+                    }
+                    if (EPI == EPI_ACT && (n1 < a.act_from || n1 + 32 > a.act_to)) {
+                        if (n1 + 32 > a.act_from && n1 < a.act_to) {
+#pragma unroll
+                            for (int q = 0; q < 32; q++)
+                                if (n1 + q >= a.act_from && n1 + q < a.act_to) v[q] = activate<true>(a.act, a.p0, a.p1, v[q]);
+                        }
+                    } else if (EPI == EPI_ACT && a.act == ACT_XIELU) {
 #pragma unroll
                         for (int q = 0; q < 32; q++) v[q] = xielu_fast(v[q], a.p0, a.p1);
                     } else if (EPI == EPI_ACT && a.act == ACT_TANH) {
@@ -189,11 +201,6 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
                     } else if (EPI == EPI_ACT) {
 #pragma unroll
                         for (int q = 0; q < 32; q++) v[q] = activate<true>(a.act, a.p0, a.p1, v[q]);
-                    }
-                    if (EPI == EPI_STORE && a.bias) {
-#pragma unroll
-                        for (int q = 0; q < 32; q++)
-                            if (n0 + c0 + q < n_end) v[q] += __ldg(a.bias + n0 + c0 + q);
                     }
 #pragma unroll
                     for (int q = 0; q < 4; q++)
@@ -282,13 +289,13 @@ static int32_t make_map(CUtensorMap *map, const void *base, int rows, int K, int
 template <int BN, int EPI, int ROWS>
 static int32_t umma_launch(const Ctx *ctx, const Problem &p, int pdl, cudaStream_t st) {
     CUtensorMap am, wm;
-    const int segs = p.segments(), ay = (int)(p.a_seg / p.lda), ax = (int)(p.a_seg % p.lda), per_seg = (p.segment_cols() + BN - 1) / BN;
+    const int segs = p.segments(), shifts = std::min(segs - 1, p.a_cap), ay = (int)(p.a_seg / p.lda), ax = (int)(p.a_seg % p.lda), per_seg = (p.segment_cols() + BN - 1) / BN;
     const int w_rows = ROWS == ROWS_ALL ? 0 : (int)(p.grp.w_group / p.ldw), mt = ROWS == ROWS_ALL ? (p.M + UM - 1) / UM : p.grp.max_tiles;
-    int32_t rc = make_map(&am, p.A, ROWS == ROWS_ALL ? p.M + (segs - 1) * ay : p.grp.a_rows, p.K + (segs - 1) * ax, p.lda, UM);
+    int32_t rc = make_map(&am, p.A, ROWS == ROWS_ALL ? p.M + shifts * ay : p.grp.a_rows, p.K + shifts * ax, p.lda, UM);
     if (!rc) rc = make_map(&wm, p.W, ROWS == ROWS_ALL ? p.N : (p.grp.n_groups - 1) * w_rows + p.N, p.K, p.ldw, BN);
     if (rc) return rc;
-    UmmaArgs a{p.C, p.M, p.N, p.K, p.ldc, mt, segs * per_seg, pdl, p.scale, ctx->d_status,
-               per_seg, p.segment_cols(), p.c_seg, ax, ay, p.res, p.colscale, p.bias, p.act, p.p0, p.p1, p.res_scale,
+    UmmaArgs a{p.C, p.M, p.N, p.K, p.ldc, mt, p.column_tiles(BN), pdl, p.scale, ctx->d_status,
+               per_seg, p.segment_cols(), p.c_seg, ax, ay, p.a_cap, p.res, p.colscale, p.bias, p.act, p.act_from, p.act_to, p.p0, p.p1, p.res_scale,
                p.grp.tiles, p.grp.n_tiles, w_rows};
     auto kern = gemm_nt_umma_kernel<BN, EPI, ROWS>;
     static thread_local int set_for = -1;
@@ -309,7 +316,7 @@ static int32_t umma_launch(const Ctx *ctx, const Problem &p, int pdl, cudaStream
 template <int EPI, int ROWS = ROWS_ALL>
 static int32_t umma_pick(const Ctx *ctx, const Problem &p, int pdl, cudaStream_t st) {
     const int mt = ROWS == ROWS_ALL ? (p.M + UM - 1) / UM : p.grp.max_tiles;
-    auto tiles = [&](int bn) { return mt * p.segments() * ((p.segment_cols() + bn - 1) / bn); };
+    auto tiles = [&](int bn) { return mt * p.column_tiles(bn); };
     if (tiles(256) >= ctx->sm_count) return umma_launch<256, EPI, ROWS>(ctx, p, pdl, st);
     if (tiles(128) >= ctx->sm_count * 2 / 3) return umma_launch<128, EPI, ROWS>(ctx, p, pdl, st);
     return umma_launch<64, EPI, ROWS>(ctx, p, pdl, st);

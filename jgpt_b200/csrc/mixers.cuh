@@ -97,6 +97,26 @@ struct MoeSum {
 };
 int32_t launch_post_norm(bool f32, float *x, int rows, const float *gamma, float eps, void *h, const MoeSum &m, int W, int ldh, int pdl, cudaStream_t st);
 
+// Between two parts with norms on either side: x[r] = source + mult * rms_norm(y[r] * sigmoid(gate[r])) * post, h[r] = rms_norm(x[r]) * pre,
+// shifted[r] = h + (h' - h) share with h' as for ShiftArgs.  x, h, y and shifted have rows of ldw elements, zeros past W; weights likewise.
+struct PartNorm {
+    const float *x;            // residual so far; null: the embedding
+    const void *y, *gate;      // y null: nothing is added; gate null: 1
+    int ldg;
+    const float *post;
+    float mult;
+    float *x_out;              // null: not stored
+    const float *pre;
+    void *h;                   // null: the residual only
+    void *shifted;             // null: no token shift
+    const float *share;
+    uint8_t *state;            // of slot 0, at the row kept, [2][ldw]
+    uint64_t state_stride;
+    int max_seqs;
+};
+int32_t launch_part_norm(bool f32, const StepDesc &d, const RowSource &embed, const PartNorm &p, const int *rowsel, int rows, float eps, int W, int ldw,
+                         int sm_count, int *status, int pdl, cudaStream_t st);
+
 // ---- moe.cu ------------------------------------------------------------------------------------------
 struct RouteArgs {
     const float *logits;       // [rows, ld]: experts, identity experts, the shared expert's gate (when shared is set)
@@ -122,16 +142,24 @@ int32_t launch_moe_gather(const RouteArgs &a, const void *h, void *out, int ld, 
 // pieces, so that a page comes in as one bulk copy and eight rows are read without bank conflicts.
 __host__ __device__ constexpr int page_row(int D) { return D % 64 == 0 ? D : D + 8; }
 __host__ __device__ constexpr int page_chunk(int D, int row, int chunk) { return D % 64 == 0 ? chunk ^ (row & 7) : chunk; }
+enum QkNorm : int { QK_NORM_NONE = 0, QK_NORM_HEAD = 1, QK_NORM_ALL = 2, QK_NORM_UNIT = 3 };  // per head with weights; over the whole row; per head without
 enum HeadGate : int { GATE_NONE = 0, GATE_HEAD = 1, GATE_ELEMENT = 2 };
 struct AttnArgs {
     void *proj;         // [rows, ldp] projections of the layer
     int ldp, q_off, k_off, v_off, g_off;  // column offsets
     int heads, kv_heads, maps, DK, DV, dim, vdim;
     int gate;           // HeadGate: sigmoid of one column per head, or of a column per element of the output
+    int window, keep;   // a query sees the last `window` positions and the first `keep` (window 0: as chunk says)
     int chunk;          // a query sees the keys of its own chunk of this many positions (0: all earlier positions)
     float scale, out_scale;
-    const float *q_norm, *k_norm;  // weights of the RMS norm of every query and key head (map); null: none
+    int qk_norm;        // QkNorm
+    const float *q_norm, *k_norm;  // its weights: [dim], or padded [heads * DK] for whole rows
+    float2 *row_inv;    // [rows] 1 / root mean square of the query and key rows, written in steps with prompts
     float eps;
+    const float *sink;  // [heads] score without a value; null: none
+    const void *v_first;  // values become (1 - share) v + share v_first; null: no mixing
+    int ld_first, vdim_first, DV_first;
+    float v_share;
     const float2 *cs;   // [rows][half] cos and sin; the first 2 half elements of every head (map) turn; null: no rotation
     int half, interleaved;         // pairs (2 i, 2 i + 1), or (i, i + half)
     float lambda, diff_scale;
@@ -142,7 +170,7 @@ struct AttnArgs {
     int ldo, out_off;
     int sm_count;
     int *status;
-    __host__ __device__ bool prepared() const { return q_norm || cs; }  // heads are normed or rotated on their way
+    __host__ __device__ bool prepared() const { return qk_norm || cs; }  // heads are normed or rotated on their way
     __host__ __device__ int page_head() const { return kBlockTokens * (page_row(maps * DK) + page_row(DV)); }
 };
 int32_t launch_attention(bool f32, const StepDesc &d, const AttnArgs &a, int pdl, cudaStream_t st);
@@ -150,11 +178,11 @@ bool attn_padded_head(int dim, int vdim, int maps, int *DK, int *DV);  // false:
 int attn_query_tile(int heads, int kv_heads);     // tokens per query tile of the multi-token kernel
 
 // ---- recurrent.cu ----------------------------------------------------------------------------------
-enum RecKind : int { REC_GLA = 0, REC_DELTA = 1, REC_HGRN2 = 2, REC_WKV = 3 };
+enum RecKind : int { REC_GLA = 0, REC_DELTA = 1, REC_HGRN2 = 2, REC_WKV = 3, REC_GENERAL = 4 };
 struct RecArgs {
     int kind;
     const void *proj;   // [rows, ldp]
-    int ldp, q_off, k_off, v_off, b_off, g_off;  // b: step-size column (delta); g: output gate inside proj (GLA)
+    int ldp, q_off, k_off, v_off, b_off, g_off;  // b: step-size column (delta), removal rates (general); g: output gate inside proj (all but delta)
     const void *z;      // [rows, ldz]: decay logits at z_off, output gate at zg_off (delta); HGRN2: proj itself
     int ldz, z_off, zg_off;
     int heads, kv_heads, DK, DV;  // padded head sizes
@@ -166,6 +194,8 @@ struct RecArgs {
     const float *a_log;       // [heads] (delta)
     const float *norm_w;      // [DV], or [heads * DV]: norm_stride is DV then
     int norm_stride;
+    const float *removal_bias;  // [heads * DK], and the rate of the decay (general)
+    float rate;
     const float *bonus;       // [heads * DK] weight of the current token (WKV)
     const float *lower;       // [heads * DK] lower bound of the forget gate (HGRN2)
     int shift_width;          // width of the previous token's input kept in the state (WKV)

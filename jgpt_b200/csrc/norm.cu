@@ -1,6 +1,9 @@
 // Embedding and norms of the layered decoder: layer norm over a plain residual, RMS norm over a residual that may be the
 // embedding, a weighted sum of the earlier layers' results, and mixed with the previous token's row.  The residual stream and
 // the norms are fp32.
+#include <algorithm>
+#include <type_traits>
+
 #include "mixers.cuh"
 #include "ptx.cuh"
 
@@ -329,6 +332,150 @@ int32_t launch_post_norm(bool f32, float *x, int rows, const float *gamma, float
     auto run = [&](auto kern, auto *act) { return launch(kern, rows, smem, pdl, st, x, gamma, eps, (decltype(act))h, (const MoeSum)m, W, ldh, pdl); };
     if (f32) return m.out ? run(post_norm_kernel<float, true>, (float *)nullptr) : run(post_norm_kernel<float, false>, (float *)nullptr);
     return m.out ? run(post_norm_kernel<__nv_bfloat16, true>, (__nv_bfloat16 *)nullptr) : run(post_norm_kernel<__nv_bfloat16, false>, (__nv_bfloat16 *)nullptr);
+}
+
+// ------------------------------------------------------------------------------------------------
+// RMS norms on both sides of a part
+// ------------------------------------------------------------------------------------------------
+__device__ __forceinline__ float dot4(const float4 &v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+template <class AT>
+__device__ __forceinline__ float sigmoid_act(float z) {
+    return sizeof(AT) == 4 ? 1.f / (1.f + expf(-z)) : __fdividef(1.f, 1.f + __expf(-z));
+}
+
+// A block takes `per` rows one after the other, 4 NV columns per thread in registers: the row in front of each is at hand for the
+// token shift.  Only the row in front of the block's first one is computed twice, so x is read and written in different arrays.
+template <class AT, bool EMBED, int NV>
+__global__ void __launch_bounds__(kNormThreads) part_norm_kernel(const StepDesc d, const RowSource s, const PartNorm a, const int *rowsel, int rows, int per,
+                                                                 float eps, int W, int ldw, int *status, int pdl) {
+    __shared__ float red[kNormThreads / 32];
+    const int tid = threadIdx.x, r0 = blockIdx.x * per, r1 = min(rows, r0 + per);
+    if (pdl & 2) griddep_launch_dependents();
+    int first = r0;
+    if (a.shifted && r0 > d.segs[d.ent[r0]].row0) first = r0 - 1;
+    if (pdl & 1) griddep_wait();
+    float4 before[NV];
+    for (int r = first; r < r1; r++) {
+        const int src = rowsel ? rowsel[r] : r;
+        const bool own = r >= r0;
+        float4 x[NV];
+        if (EMBED) {
+            int t = d.tok[src];
+            if (t < 0 || t >= s.vocab) {
+                if (tid == 0) atomicOr(status, DEV_STATUS_BAD_POSITION);
+                t = 0;
+            }
+            const AT *e = reinterpret_cast<const AT *>(s.embed) + (size_t)t * s.ld_embed;
+#pragma unroll
+            for (int i = 0; i < NV; i++) {
+                const int j = (tid + i * kNormThreads) * 4;
+                x[i] = j < ldw ? load4(e + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+                x[i].x *= s.embed_scale, x[i].y *= s.embed_scale, x[i].z *= s.embed_scale, x[i].w *= s.embed_scale;
+            }
+            if (own)
+                for (int k = 0; k < s.n_rot; k++)
+                    for (int i = tid; i < s.rot[k].half; i += kNormThreads) {
+                        double sn, cs;
+                        sincos((double)d.pos[src] * s.rot[k].freq[i], &sn, &cs);
+                        s.rot[k].out[(size_t)src * s.rot[k].half + i] = make_float2((float)cs * s.rot[k].mag, (float)sn * s.rot[k].mag);
+                    }
+        } else {
+            const float *xr = a.x + (size_t)src * ldw;
+#pragma unroll
+            for (int i = 0; i < NV; i++) {
+                const int j = (tid + i * kNormThreads) * 4;
+                x[i] = j < ldw ? load4(xr + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+        }
+        if (a.y) {
+            const AT *yr = reinterpret_cast<const AT *>(a.y) + (size_t)src * ldw, *gr = reinterpret_cast<const AT *>(a.gate) + (size_t)src * a.ldg;
+            float4 y[NV];
+            float q = 0.f;
+#pragma unroll
+            for (int i = 0; i < NV; i++) {
+                const int j = (tid + i * kNormThreads) * 4;
+                y[i] = j < ldw ? load4(yr + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+                if (a.gate && j < ldw) {
+                    const float4 g = load4(gr + j);
+                    y[i].x *= sigmoid_act<AT>(g.x), y[i].y *= sigmoid_act<AT>(g.y), y[i].z *= sigmoid_act<AT>(g.z), y[i].w *= sigmoid_act<AT>(g.w);
+                }
+                q += dot4(y[i]);
+            }
+            const float f = a.mult / sqrtf(block_sum(q, red) / (float)W + eps);
+#pragma unroll
+            for (int i = 0; i < NV; i++) {
+                const int j = (tid + i * kNormThreads) * 4;
+                if (j >= ldw) continue;
+                const float4 w = load4(a.post + j);
+                x[i].x = fmaf(f * y[i].x, w.x, x[i].x), x[i].y = fmaf(f * y[i].y, w.y, x[i].y);
+                x[i].z = fmaf(f * y[i].z, w.z, x[i].z), x[i].w = fmaf(f * y[i].w, w.w, x[i].w);
+            }
+        }
+        if (own && a.x_out) {
+#pragma unroll
+            for (int i = 0; i < NV; i++) {
+                const int j = (tid + i * kNormThreads) * 4;
+                if (j < ldw) store4(a.x_out + (size_t)src * ldw + j, x[i]);
+            }
+        }
+        if (!a.h) continue;
+        float q = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; i++) q += dot4(x[i]);
+        const float f = 1.f / sqrtf(block_sum(q, red) / (float)W + eps);
+#pragma unroll
+        for (int i = 0; i < NV; i++) {
+            const int j = (tid + i * kNormThreads) * 4;
+            if (j >= ldw) continue;
+            const float4 w = load4(a.pre + j);
+            x[i].x *= f * w.x, x[i].y *= f * w.y, x[i].z *= f * w.z, x[i].w *= f * w.w;
+            if (own) store4(reinterpret_cast<AT *>(a.h) + (size_t)r * ldw + j, x[i]);
+        }
+        if (!a.shifted) continue;
+        if (own) {
+            const Seg sg = d.segs[d.ent[r]];
+            const bool ok = sg.seq >= 0 && sg.seq < a.max_seqs;
+            if (!ok && tid == 0) atomicOr(status, DEV_STATUS_BAD_SEQ);
+            float *hist = reinterpret_cast<float *>(a.state + (uint64_t)(ok ? sg.seq : 0) * a.state_stride);
+            const bool front = r == sg.row0, last = r == sg.row0 + sg.T - 1;
+#pragma unroll
+            for (int i = 0; i < NV; i++) {
+                const int j = (tid + i * kNormThreads) * 4;
+                if (j >= ldw) continue;
+                float4 b = before[i];
+                if (front) b = ok && sg.pos0 > 0 ? load4(hist + (size_t)sg.conv_set * ldw + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+                if (last && ok) store4(hist + (size_t)(1 - sg.conv_set) * ldw + j, x[i]);
+                const float4 m = load4(a.share + j);
+                b.x = fmaf(b.x - x[i].x, m.x, x[i].x), b.y = fmaf(b.y - x[i].y, m.y, x[i].y);
+                b.z = fmaf(b.z - x[i].z, m.z, x[i].z), b.w = fmaf(b.w - x[i].w, m.w, x[i].w);
+                store4(reinterpret_cast<AT *>(a.shifted) + (size_t)r * ldw + j, b);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < NV; i++) before[i] = x[i];
+    }
+}
+
+int32_t launch_part_norm(bool f32, const StepDesc &d, const RowSource &embed, const PartNorm &p, const int *rowsel, int rows, float eps, int W, int ldw,
+                         int sm_count, int *status, int pdl, cudaStream_t st) {
+    const int per = std::max(1, std::min(8, rows / (8 * sm_count)));
+    const int nv = (ldw + 4 * kNormThreads - 1) / (4 * kNormThreads);
+    JGPT_REQUIRE(nv <= 16, JGPT_ERR_UNSUPPORTED, "width %d", W);
+    JGPT_REQUIRE(!p.shifted || !rowsel, JGPT_ERR_INVALID_ARGUMENT, "the token shift takes all rows");
+    auto run = [&](auto kern) {
+        return launch(kern, (rows + per - 1) / per, 0, pdl, st, (const StepDesc)d, (const RowSource)embed, (const PartNorm)p, rowsel, rows, per, eps, W, ldw, status, pdl);
+    };
+    auto pick = [&](auto act, auto from_embed) {
+        typedef decltype(act) AT;
+        constexpr bool E = decltype(from_embed)::value;
+        return nv <= 1   ? run(part_norm_kernel<AT, E, 1>)
+               : nv <= 2 ? run(part_norm_kernel<AT, E, 2>)
+               : nv <= 4 ? run(part_norm_kernel<AT, E, 4>)
+               : nv <= 8 ? run(part_norm_kernel<AT, E, 8>)
+                         : run(part_norm_kernel<AT, E, 16>);
+    };
+    if (f32) return p.x ? pick(0.f, std::false_type()) : pick(0.f, std::true_type());
+    return p.x ? pick(__nv_bfloat16(), std::false_type()) : pick(__nv_bfloat16(), std::true_type());
 }
 
 }  // namespace mix

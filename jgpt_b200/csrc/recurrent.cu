@@ -1,9 +1,11 @@
-// Recurrent mixers of the layered decoder, token by token: gated linear attention, the gated delta rule, HGRN2 and WKV, all with
+// Recurrent mixers of the layered decoder, token by token: gated linear attention, the gated delta rule, the generalised delta rule, HGRN2 and WKV, all with
 // a decay per key channel (long entries of a bf16 step take the chunked form, recurrent_chunk.cu), as ONE kernel from the layer's projections to the gated, normalised head outputs - for prompts, portions of
 // prompts and single tokens alike, so a token's arithmetic does not depend on how its sequence was cut.
 //
 //   GLA    S <- diag(a) S + k v^T;                       o = S^T q
 //   DELTA  S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q   (o read off as S_decayed^T q + (q.k) u)
+//   GENERAL S <- diag(w) S - (a u) (u^T S) + k v^T with the old S on the right, u = k / n, n = |k|;  o = S^T q.  With s = S^T u:
+//          S <- diag(w) S + u (n v)^T - (a u) s^T,  o read off as S^T (w q) - (q.(a u)) s + (q.u) n v
 //   HGRN2  S <- diag(f) S + (1 - f) v^T;                 o = S^T q
 //   WKV    o = (S + diag(u) k v^T)^T r, read off as S^T r + (r.(u k)) v;  S <- diag(w) S + k v^T
 //
@@ -25,7 +27,8 @@
 namespace jgpt {
 namespace mix {
 
-constexpr int kTileTokens = 16;
+// Tokens of a tile; fewer where two stages of raw rows would not fit.
+__host__ __device__ constexpr int rec_tile_tokens(int kind, int DK, size_t elem) { return kind == REC_GENERAL && DK * elem > 192 * 4 ? 8 : 16; }
 
 typedef unsigned long long u64;
 __device__ __forceinline__ u64 pack2(float lo, float hi) {
@@ -76,10 +79,10 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
     constexpr int E = 16 / sizeof(AT);  // elements of a 16-byte chunk
     // a token's raw row: q, k, v, decay logits, output gate, then (delta) the chunk that holds its step size
     const int RK = DK, RV = rec_has_key(KIND) ? 2 * DK : DK, RZ = RV + DVc, RG = RZ + DK, RB = rec_has_gate(KIND) ? RG + DVc : RG,
-              RW = RB + (KIND == REC_DELTA ? E : 0);
-    float *sq = rec_smem, *sk = sq + tt * DK, *sg = sk + tt * DK, *sv = sg + tt * DK, *so = sv + tt * DVc, *sbeta = so + tt * DVc,
-          *sqk = sbeta + tt;
-    AT *raw_s = reinterpret_cast<AT *>(sqk + tt);  // [2][tt][RW]; one stage is enough for a single token
+              RW = RB + (KIND == REC_DELTA ? E : KIND == REC_GENERAL ? DK : 0);  // general: the removal rates' projection
+    float *sq = rec_smem, *sk = sq + tt * DK, *sg = sk + tt * DK, *sa = sg + (rec_key_vectors(KIND) - 3) * tt * DK, *sv = sa + tt * DK, *so = sv + tt * DVc,
+          *sbeta = so + tt * DVc, *sqk = sbeta + tt, *sqa = sqk + tt;
+    AT *raw_s = reinterpret_cast<AT *>(sqk + (KIND == REC_GENERAL ? 3 : 1) * tt);  // [2][tt][RW]; one stage is enough for a single token
 
     if (pdl & 2) griddep_launch_dependents();
     const Seg sgm = segs[list[blockIdx.y]];
@@ -138,7 +141,7 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
             else if (c < RZ) src = row + a.v_off + h * a.DV + col0 + c - RV;
             else if (c < RG) src = zr + a.z_off + h * DK + c - RZ;
             else if (c < RB) src = (KIND == REC_DELTA ? zr + a.zg_off : row + a.g_off) + h * a.DV + col0 + c - RG;
-            else src = row + a.b_off + h / E * E;
+            else src = KIND == REC_GENERAL ? row + a.b_off + h * DK + c - RB : row + a.b_off + h / E * E;
             cp_async16(raw_s + ((size_t)buf * tt + t) * RW + c, src, true);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -214,12 +217,18 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
                 *reinterpret_cast<float2 *>(sk + t * DK + c) = make_float2(f0.y, f1.y);
             } else if (KIND == REC_WKV) {
                 y.x = exp_neg_exp<AT>(y.x), y.y = exp_neg_exp<AT>(y.y);
+            } else if (KIND == REC_GENERAL) {
+                y.x = exp_f<AT>(-a.rate * sigmoid_f<AT>(y.x)), y.y = exp_f<AT>(-a.rate * sigmoid_f<AT>(y.y));
+                float2 m = load2(raw + (size_t)t * RW + RB + c);
+                const float2 mb = *reinterpret_cast<const float2 *>(a.removal_bias + h * DK + c);
+                m.x = sigmoid_f<AT>(m.x + mb.x), m.y = sigmoid_f<AT>(m.y + mb.y);
+                *reinterpret_cast<float2 *>(sa + t * DK + c) = m;
             } else {
                 y.x = exp_f<AT>(-rate * softplus_f<AT>(y.x)), y.y = exp_f<AT>(-rate * softplus_f<AT>(y.y));
             }
             *reinterpret_cast<float2 *>(sg + t * DK + c) = y;
         }
-        if (!SINGLE && KIND != REC_DELTA && (tn & 1))
+        if (!SINGLE && KIND != REC_DELTA && KIND != REC_GENERAL && (tn & 1))
             for (int c = tid; c < DK; c += nthreads) sg[tn * DK + c] = 1.f;
         __syncthreads();
         if (!SINGLE && t0 + tt < sgm.T) stage(buf ^ 1, t0 + tt);  // lands while this tile runs; the previous tile's rows are no longer needed
@@ -239,6 +248,24 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
             }
             __syncthreads();
         }
+        if (KIND == REC_GENERAL) {
+            for (int t = warp; t < tn; t += nw) {
+                float kv[NI], kk = 0.f, qu = 0.f, qa = 0.f;
+#pragma unroll
+                for (int i = 0; i < NI; i++) kv[i] = sk[t * DK + lane + 32 * i], kk += kv[i] * kv[i];
+                const float n = sqrtf(warp_sum(kk) + 1e-6f), f = 1.f / n;
+#pragma unroll
+                for (int i = 0; i < NI; i++) {
+                    const int at = t * DK + lane + 32 * i;
+                    const float u = kv[i] * f, au = sa[at] * u, q = sq[at];
+                    qu += q * u, qa += q * au;
+                    sk[at] = u, sa[at] = au, sq[at] = q * sg[at];
+                }
+                qu = warp_sum(qu), qa = warp_sum(qa);
+                if (lane == 0) sbeta[t] = n, sqk[t] = qu, sqa[t] = qa;
+            }
+            __syncthreads();
+        }
         if (KIND == REC_WKV) {  // what the current token adds to its own output: (r . (u k)) v
             for (int t = warp; t < tn; t += nw) {
                 float rk = 0.f;
@@ -251,7 +278,54 @@ __global__ void __launch_bounds__(SINGLE || DK > 128 ? 256 : 512, SINGLE ? rec_s
         }
         // ---- the recurrence: every warp on its own columns ----
         const int vcol = warp * 16 + cl * 4;
-        if (KIND == REC_DELTA) {
+        if (KIND == REC_GENERAL) {
+            for (int t = 0; t < tn; t++) {
+                u64 ks[4] = {0, 0, 0, 0}, qs[4] = {0, 0, 0, 0};
+                const float *qp = sq + t * DK + rl * 4, *kp = sk + t * DK + rl * 4, *gp = sg + t * DK + rl * 4, *ap = sa + t * DK + rl * 4;
+#pragma unroll
+                for (int i = 0; i < NI; i++) {
+                    const ulonglong2 q2 = *reinterpret_cast<const ulonglong2 *>(qp + 32 * i), k2 = *reinterpret_cast<const ulonglong2 *>(kp + 32 * i);
+#pragma unroll
+                    for (int c = 0; c < 4; c++) {
+                        ks[c] = fma2(k2.x, st[2 * i][c], ks[c]), ks[c] = fma2(k2.y, st[2 * i + 1][c], ks[c]);
+                        qs[c] = fma2(q2.x, st[2 * i][c], qs[c]), qs[c] = fma2(q2.y, st[2 * i + 1][c], qs[c]);
+                    }
+                }
+                float kf[4], qf[4];
+#pragma unroll
+                for (int c = 0; c < 4; c++) {
+                    const float2 x = unpack2(ks[c]), y = unpack2(qs[c]);
+                    kf[c] = x.x + x.y, qf[c] = y.x + y.y;
+                }
+                const float tot = reduce8(kf, qf, lane);
+                const float4 v4 = *reinterpret_cast<const float4 *>(sv + t * DVc + vcol);
+                const float n = sbeta[t];
+                float nv[4], s[4];
+#pragma unroll
+                for (int c = 0; c < 4; c++) {
+                    s[c] = __shfl_sync(0xffffffffu, tot, ((c & 2) << 2) | ((c & 1) << 2) | cl);
+                    nv[c] = n * (c == 0 ? v4.x : c == 1 ? v4.y : c == 2 ? v4.z : v4.w);
+                }
+                if (lane & 16) {
+                    const int c = rl & 3;
+                    const float sc = c == 0 ? s[0] : c == 1 ? s[1] : c == 2 ? s[2] : s[3], nc = c == 0 ? nv[0] : c == 1 ? nv[1] : c == 2 ? nv[2] : nv[3];
+                    so[t * DVc + vcol + c] = fmaf(sqk[t], nc, fmaf(-sqa[t], sc, tot));
+                }
+                u64 n2[4], s2[4];
+#pragma unroll
+                for (int c = 0; c < 4; c++) n2[c] = pack2(nv[c], nv[c]), s2[c] = pack2(-s[c], -s[c]);
+#pragma unroll
+                for (int i = 0; i < NI; i++) {
+                    const ulonglong2 k2 = *reinterpret_cast<const ulonglong2 *>(kp + 32 * i), g2 = *reinterpret_cast<const ulonglong2 *>(gp + 32 * i),
+                                     a2 = *reinterpret_cast<const ulonglong2 *>(ap + 32 * i);
+#pragma unroll
+                    for (int c = 0; c < 4; c++) {
+                        st[2 * i][c] = fma2(a2.x, s2[c], fma2(k2.x, n2[c], mul2(g2.x, st[2 * i][c])));
+                        st[2 * i + 1][c] = fma2(a2.y, s2[c], fma2(k2.y, n2[c], mul2(g2.y, st[2 * i + 1][c])));
+                    }
+                }
+            }
+        } else if (KIND == REC_DELTA) {
             for (int t = 0; t < tn; t++) {
                 u64 ks[4] = {0, 0, 0, 0}, qs[4] = {0, 0, 0, 0};
                 const float *qp = sq + t * DK + rl * 4, *kp = sk + t * DK + rl * 4, *gp = sg + t * DK + rl * 4;
@@ -399,7 +473,8 @@ uint64_t rec_state_bytes(const RecArgs &a, int elem_bytes, uint64_t *conv_off) {
 template <class AT, int KIND, int DK, bool SINGLE>
 static int32_t rec_launch_form(const StepDesc &d, const RecArgs &a, int pdl, int *split_out, cudaStream_t st) {
     const bool single = SINGLE;
-    const int tt = single ? 2 : kTileTokens;
+    constexpr int tile_tokens = rec_tile_tokens(KIND, DK, sizeof(AT));
+    const int tt = single ? 2 : tile_tokens;
     const int groups = a.DV / 16, max_groups = DK <= 128 && !SINGLE ? 16 : 8;
     int split = 1;
     auto allowed = [&](int s) { return groups % s == 0; };
@@ -407,8 +482,8 @@ static int32_t rec_launch_form(const StepDesc &d, const RecArgs &a, int pdl, int
     *split_out = split;
     const int nw = groups / split, DVc = nw * 16;
     auto smem_bytes = [](int tokens, int cols, int stages) {
-        const size_t row = 3 * DK + 2 * (size_t)cols;
-        return sizeof(float) * ((size_t)tokens * row + 2 * tokens) + (size_t)stages * tokens * (row * sizeof(AT) + (KIND == REC_DELTA ? 16 : 0));
+        const size_t row = rec_key_vectors(KIND) * DK + 2 * (size_t)cols;
+        return sizeof(float) * ((size_t)tokens * row + (KIND == REC_GENERAL ? 4 : 2) * tokens) + (size_t)stages * tokens * (row * sizeof(AT) + (KIND == REC_DELTA ? 16 : 0));
     };
     const size_t smem = smem_bytes(tt, DVc, single ? 1 : 2);
     auto kern = recurrent_kernel<AT, KIND, DK, SINGLE>;
@@ -416,7 +491,7 @@ static int32_t rec_launch_form(const StepDesc &d, const RecArgs &a, int pdl, int
     int dev = 0;
     JGPT_CUDA_TRY(cudaGetDevice(&dev));
     if (set_for != dev) {
-        JGPT_CUDA_TRY(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_bytes(kTileTokens, 16 * max_groups, 2)));
+        JGPT_CUDA_TRY(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_bytes(tile_tokens, 16 * max_groups, 2)));
         set_for = dev;
     }
     cudaLaunchConfig_t cfg = {};
@@ -466,6 +541,7 @@ int32_t launch_recurrent(bool f32, const StepDesc &d, const RecArgs &a, int pdl,
         case REC_DELTA: return f32 ? rec_run<float, REC_DELTA>(d, a, pdl, st) : rec_run<__nv_bfloat16, REC_DELTA>(d, a, pdl, st);
         case REC_HGRN2: return f32 ? rec_run<float, REC_HGRN2>(d, a, pdl, st) : rec_run<__nv_bfloat16, REC_HGRN2>(d, a, pdl, st);
         case REC_WKV: return f32 ? rec_run<float, REC_WKV>(d, a, pdl, st) : rec_run<__nv_bfloat16, REC_WKV>(d, a, pdl, st);
+        case REC_GENERAL: return f32 ? rec_run<float, REC_GENERAL>(d, a, pdl, st) : rec_run<__nv_bfloat16, REC_GENERAL>(d, a, pdl, st);
     }
     return fail(JGPT_ERR_INVALID_ARGUMENT, "recurrence %d", a.kind);
 }

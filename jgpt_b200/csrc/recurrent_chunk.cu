@@ -11,6 +11,10 @@
 //     S   = diag(b_16) S0 + sum_j (k_j b_16,j) u_j^T
 // which follows from unrolling the rules over the chunk.  HGRN2 is GLA with k = 1 - g.  WKV reads before it writes:
 //     P_ij = sum_d r_i k_j b_i-1,j  (j < i),  P_ii = sum_d r_i u k_i,  and r_i b_i-1 in place of q_i b_i.
+// The generalised delta rule S <- diag(w) S - (a u) (u^T S) + k v^T, with s_i = S_(i-1)^T u_i, is
+//     s_i = (u_i b_i-1)^T S0 + sum_{j<i} C_ij v_j - sum_{j<i} A_ij s_j,   A_ij = sum_d u_i (a u)_j b_i-1,j,  C_ij = sum_d u_i k_j b_i-1,j
+// so with T = (I + A)^-1 the rows U = -s are  U = -(T U~) S0 - T C V:  the form above with (a u)_j in place of k_j, and the terms
+// sum_j (k_j b_16,j) v_j^T of the state and sum_{j<=i} R_ij v_j of the output (R_ij = sum_d q_i k_j b_ij) beside it.
 //
 // Two kernels.  rec_prep_kernel, parallel over all chunks and heads: convolution, unit vectors, decays, and everything above
 // that does not involve S0, written as one record per (chunk, head).  rec_scan_kernel, serial over the chunks of a sequence
@@ -31,10 +35,13 @@ static_assert(kC == 16, "the layouts below are for 16 tokens");
 
 // Record of one (chunk, head), floats:
 //   [DELTA: -W [16 tok][DK]] [Q~ [16 tok][DK]] [K^ [DK][16 tok]] [b_16 [DK]] [P [16 i][16 j]] [U0 [DV][16 tok]]
+// GENERAL: -W, Q~, K^ with (a u), K^ with k, b_16, P with (a u), R, then for every 16 value columns U0 [16][16 tok] and V [16][16 tok].
 // 8-float groups inside a row are permuted so that the fragment loads are free of bank conflicts.
-__host__ __device__ constexpr int rec_mats(int kind) { return kind == REC_DELTA ? 3 : 2; }
+__host__ __device__ constexpr int rec_mats(int kind) { return kind == REC_GENERAL ? 4 : kind == REC_DELTA ? 3 : 2; }
+__host__ __device__ constexpr int rec_updates(int kind) { return kind == REC_GENERAL ? 2 : 1; }  // outer products per token
+__host__ __device__ constexpr bool rec_has_w(int kind) { return kind == REC_DELTA || kind == REC_GENERAL; }
 __host__ __device__ constexpr uint64_t record_floats(int kind, int DK, int DV) {
-    return (uint64_t)rec_mats(kind) * kC * DK + DK + kC * kC + (uint64_t)kC * DV;
+    return (uint64_t)rec_mats(kind) * kC * DK + DK + (uint64_t)rec_updates(kind) * (kC * kC + kC * (uint64_t)DV);
 }
 uint64_t rec_chunk_record_floats(int kind, int DK, int DV) { return record_floats(kind, DK, DV); }
 int rec_chunk_min_tokens(bool f32) {
@@ -84,6 +91,7 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, DV = a.DV;
     float *sq = prep_smem, *sk = sq + kC * DK, *sg = sk + kC * DK, *sv = sg + kC * DK;  // [16][DK], [16][DV]
     float *sA = sv + kC * DV, *sP = sA + kC * kC, *sT = sP + kC * kC, *sbeta = sT + kC * kC;
+    float *sR = sbeta + kC, *sC = sR + kC * kC, *sa = sC + kC * kC;  // general
     if (pdl & 2) griddep_launch_dependents();
     const int2 ck = chunks[blockIdx.x];
     const Seg sgm = segs[ck.x];
@@ -120,6 +128,15 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
     for (int e = 0; e < ZN; e++) {
         const int idx = e * 256 + tid, t = idx / (DK / 2), c = 2 * (idx % (DK / 2));
         zr[e] = t < tn ? load2(z + (size_t)(t0 + t) * a.ldz + a.z_off + h * DK + c) : make_float2(0.f, 0.f);
+        if (KIND == REC_GENERAL && t < kC) {
+            float2 m = make_float2(0.f, 0.f);
+            if (t < tn) {
+                const float2 mb = *reinterpret_cast<const float2 *>(a.removal_bias + h * DK + c);
+                m = load2(proj + (size_t)(t0 + t) * a.ldp + a.b_off + h * DK + c);
+                m.x = sigmoid_f<AT>(m.x + mb.x), m.y = sigmoid_f<AT>(m.y + mb.y);
+            }
+            *reinterpret_cast<float2 *>(sa + t * DK + c) = m;
+        }
     }
     float bl = 0.f;
     if (KIND == REC_DELTA && tid < tn) bl = load1(proj + (size_t)(t0 + tid) * a.ldp + a.b_off + h);
@@ -183,6 +200,8 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
                 y = make_float2(f0.x, f1.x), w = make_float2(f0.y, f1.y);
             } else if (KIND == REC_WKV) {
                 y.x = exp_neg_exp<AT>(y.x), y.y = exp_neg_exp<AT>(y.y);
+            } else if (KIND == REC_GENERAL) {
+                y.x = exp_f<AT>(-a.rate * sigmoid_f<AT>(y.x)), y.y = exp_f<AT>(-a.rate * sigmoid_f<AT>(y.y));
             } else {
                 y.x = exp_f<AT>(-rate * softplus_f<AT>(y.x)), y.y = exp_f<AT>(-rate * softplus_f<AT>(y.y));
             }
@@ -206,6 +225,18 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
         }
         __syncthreads();
     }
+    if (KIND == REC_GENERAL) {  // |k| beside the unit key, which the removal rates are multiplied with
+        for (int t = warp; t < kC; t += 8) {
+            float kv[NI], kk = 0.f;
+#pragma unroll
+            for (int i = 0; i < NI; i++) kv[i] = sk[t * DK + lane + 32 * i], kk += kv[i] * kv[i];
+            const float n = sqrtf(warp_sum(kk) + 1e-6f), f = 1.f / n;
+#pragma unroll
+            for (int i = 0; i < NI; i++) sk[t * DK + lane + 32 * i] = kv[i] * f, sa[t * DK + lane + 32 * i] *= kv[i] * f;
+            if (lane == 0) sbeta[t] = n;
+        }
+        __syncthreads();
+    }
     // ---- A and P: warp w takes keys j = w and 15 - w; the key decays step by step on its way to later tokens ----
     {
         const int js[2] = {warp, 15 - warp};
@@ -214,8 +245,38 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
 #pragma unroll
             for (int c = 0; c < NI; c++) bonus[c] = a.bonus[h * DK + lane + 32 * c];
         }
+        if (KIND == REC_GENERAL) {
+#pragma unroll 1
+            for (int s = 0; s < 2; s++) {
+                const int j = js[s];
+                const float n = sbeta[j];
+                float kd[NI], ad[NI], w[2][32];  // unit key and removal row on their way; rows P, A and R, C
 #pragma unroll
-        for (int s = 0; s < 2; s++) {
+                for (int c = 0; c < NI; c++) kd[c] = sk[j * DK + lane + 32 * c], ad[c] = sa[j * DK + lane + 32 * c];
+#pragma unroll
+                for (int i = 0; i < kC; i++) {
+                    float p = 0.f, x = 0.f, y = 0.f, z = 0.f;
+                    if (i >= j) {
+#pragma unroll
+                        for (int c = 0; c < NI; c++) {
+                            if (i > j) {
+                                const float u = sk[i * DK + lane + 32 * c], g = sg[i * DK + lane + 32 * c];
+                                x = fmaf(u, ad[c], x), z = fmaf(u, kd[c], z);
+                                ad[c] *= g, kd[c] *= g;
+                            }
+                            const float q = sq[i * DK + lane + 32 * c];
+                            p = fmaf(q, ad[c], p), y = fmaf(q, kd[c], y);
+                        }
+                    }
+                    w[0][i] = p, w[0][16 + i] = x, w[1][i] = y, w[1][16 + i] = z;
+                }
+                const float t0 = reduce32(w[0], lane), t1 = n * reduce32(w[1], lane);
+                if (lane < 16) sP[lane * kC + j] = t0, sR[lane * kC + j] = t1;
+                else sA[(lane - 16) * kC + j] = t0, sC[(lane - 16) * kC + j] = t1;
+            }
+        }
+#pragma unroll
+        for (int s = 0; s < (KIND == REC_GENERAL ? 0 : 2); s++) {
             const int j = js[s];
             float kk[NI];
 #pragma unroll
@@ -245,13 +306,13 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
                 else sA[(lane - 16) * kC + j] = tot;
             }
         }
-        if (KIND != REC_DELTA) {
+        if (KIND != REC_DELTA && KIND != REC_GENERAL) {
             const float tot = reduce32(v[0], lane);
             sP[(lane & 15) * kC + js[lane >> 4]] = tot;
         }
     }
     __syncthreads();
-    if (KIND == REC_DELTA && tid < kC) {  // column tid of T by forward substitution
+    if (rec_has_w(KIND) && tid < kC) {  // column tid of T by forward substitution
         float t[kC];
 #pragma unroll
         for (int i = 0; i < kC; i++) {
@@ -259,14 +320,15 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
 #pragma unroll
             for (int j = 0; j < kC; j++)
                 if (j < i) s = fmaf(-sA[i * kC + j], t[j], s);
-            t[i] = sbeta[i] * s;
+            t[i] = KIND == REC_DELTA ? sbeta[i] * s : s;
             sT[i * kC + tid] = t[i];
         }
     }
-    if (KIND == REC_DELTA) __syncthreads();
+    if (rec_has_w(KIND)) __syncthreads();
     // ---- the record ----
     float *rec = a.chunk_ws + ((size_t)blockIdx.x * a.heads + h) * record_floats(KIND, DK, DV);
-    float *rw = rec, *rq = rec + (KIND == REC_DELTA ? kC * DK : 0), *rk = rq + kC * DK, *rb = rk + kC * DK, *rp = rb + DK, *ru = rp + kC * kC;
+    float *rw = rec, *rq = rec + (rec_has_w(KIND) ? kC * DK : 0), *rk = rq + kC * DK, *rb = rk + rec_updates(KIND) * kC * DK, *rp = rb + DK,
+          *ru = rp + rec_updates(KIND) * kC * kC;
     for (int idx = tid; idx < DK + DV; idx += 256) {
         if (idx < DK) {
             const int d = idx;
@@ -274,12 +336,13 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
 #pragma unroll
             for (int t = 0; t < kC; t++) {
                 if (KIND == REC_WKV) rq[at_tok(t, d, DK)] = sq[t * DK + d] * b;
+                if (KIND == REC_GENERAL) kt[t] = sk[t * DK + d] * b;
                 b *= sg[t * DK + d];
                 if (KIND != REC_WKV) rq[at_tok(t, d, DK)] = sq[t * DK + d] * b;
-                kt[t] = sk[t * DK + d] * b;
+                if (KIND != REC_GENERAL) kt[t] = sk[t * DK + d] * b;
             }
             rb[d] = b;
-            if (KIND == REC_DELTA) {
+            if (rec_has_w(KIND)) {
 #pragma unroll
                 for (int i = 0; i < kC; i++) {
                     rw[at_tok(i, d, DK)] = -lower_dot(sT, i, kt);
@@ -288,10 +351,19 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
             b = 1.f;
 #pragma unroll
             for (int t = kC - 1; t >= 0; t--) {
-                kt[t] = sk[t * DK + d] * b;
+                kt[t] = (KIND == REC_GENERAL ? sa : sk)[t * DK + d] * b;
                 b *= sg[t * DK + d];
             }
             store_row16(rk, d, kt);
+            if (KIND == REC_GENERAL) {
+                b = 1.f;
+#pragma unroll
+                for (int t = kC - 1; t >= 0; t--) {
+                    kt[t] = sbeta[t] * sk[t * DK + d] * b;
+                    b *= sg[t * DK + d];
+                }
+                store_row16(rk + kC * DK, d, kt);
+            }
         } else {
             const int c = idx - DK;
             float vv[kC];
@@ -303,10 +375,23 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecArgs a, const Se
                     vv[i] = lower_dot(sT, i, vv);
                 }
             }
+            if (KIND == REC_GENERAL) {  // V, then -T C V; C is strictly lower triangular
+                float *cols = ru + c / 16 * (2 * 16 * kC);
+                store_row16(cols + 16 * kC, c % 16, vv);
+#pragma unroll
+                for (int i = kC - 1; i >= 0; i--) vv[i] = lower_dot(sC, i, vv);
+#pragma unroll
+                for (int i = kC - 1; i >= 0; i--) vv[i] = -lower_dot(sT, i, vv);
+                store_row16(cols, c % 16, vv);
+                continue;
+            }
             store_row16(ru, c, vv);
         }
     }
-    for (int e = tid; e < kC * kC; e += 256) rp[at_16(e / kC, e % kC)] = e / kC >= e % kC ? sP[e] : 0.f;
+    for (int e = tid; e < kC * kC; e += 256) {
+        rp[at_16(e / kC, e % kC)] = e / kC >= e % kC ? sP[e] : 0.f;
+        if (KIND == REC_GENERAL) rp[kC * kC + at_16(e / kC, e % kC)] = e / kC >= e % kC ? sR[e] : 0.f;
+    }
     // ---- convolution history for the next step, by the entry's last chunk ----
     if (KIND == REC_DELTA && a.taps > 1 && t0 + kC >= sgm.T) {
         AT *next = reinterpret_cast<AT *>(part + a.conv_off) + (size_t)(1 - sgm.conv_set) * (a.taps - 1) * channels;
@@ -343,20 +428,22 @@ __device__ __forceinline__ void mma3(float (&acc)[4], float (&cor)[4], const Spl
     mma_tf32(cor, x.hi, y.lo[0], y.lo[1]);
 }
 
-constexpr int kScanStages = 3;
+// Two stages where three do not fit beside one another.
+__host__ __device__ constexpr int scan_stages(int kind, int DK) { return kind == REC_GENERAL && DK > 192 ? 2 : 3; }
 __host__ __device__ constexpr size_t scan_stage_floats(int kind, int DK, int cols) { return (size_t)record_floats(kind, DK, cols); }
 
 template <int KIND, int DK>
 __global__ void __launch_bounds__(256) rec_scan_kernel(const RecArgs a, const Seg *__restrict__ segs, const int2 *__restrict__ longs, int pdl) {
     constexpr int NT = DK / 8;
-    constexpr uint32_t COMMON = (uint32_t)(rec_mats(KIND) * kC * DK + DK + kC * kC);
+    constexpr int UPD = rec_updates(KIND), kScanStages = scan_stages(KIND, DK);
+    constexpr uint32_t COMMON = (uint32_t)(rec_mats(KIND) * kC * DK + DK + UPD * kC * kC);
     extern __shared__ __align__(16) float scan_smem[];
     __shared__ __align__(8) uint64_t full[kScanStages];
     __shared__ int s_abort_mem;
     volatile int *s_abort = &s_abort_mem;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int cols = blockDim.x / 2, h = blockIdx.x % a.heads, col0 = blockIdx.x / a.heads * cols;  // value columns of this CTA
-    const uint32_t STAGE = COMMON + (uint32_t)kC * cols;
+    const uint32_t STAGE = COMMON + (uint32_t)(UPD * kC) * cols;
     if (pdl & 2) griddep_launch_dependents();
     const int2 ls = longs[blockIdx.y];
     const Seg sgm = segs[ls.x];
@@ -387,7 +474,7 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecArgs a, const Se
         float *dst = scan_smem + (size_t)s * STAGE;
         mbar_expect_tx(&full[s], STAGE * 4);
         bulk_g2s(dst, rec, COMMON * 4, &full[s]);
-        bulk_g2s(dst + COMMON, rec + COMMON + (size_t)kC * col0, (uint32_t)(kC * cols * 4), &full[s]);
+        bulk_g2s(dst + COMMON, rec + COMMON + (size_t)(UPD * kC) * col0, (uint32_t)(UPD * kC * cols * 4), &full[s]);
     };
     int issued = 0;
     if (tid == 0)
@@ -404,8 +491,8 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecArgs a, const Se
             return;
         }
         const float *m = scan_smem + (size_t)s * STAGE;
-        const float *mw = m, *mq = m + (KIND == REC_DELTA ? kC * DK : 0), *mk = mq + kC * DK, *mb = mk + kC * DK, *mp = mb + DK,
-                    *mu = m + COMMON + (size_t)warp * 16 * kC;
+        const float *mw = m, *mq = m + (rec_has_w(KIND) ? kC * DK : 0), *mk = mq + kC * DK, *mb = mk + UPD * kC * DK, *mp = mb + DK,
+                    *mu = m + COMMON + (size_t)warp * 16 * UPD * kC;
         // U0 and O, tokens 8 n + 2 t (+ 1) of columns g, g + 8
         float u[2][4], uc[2][4], o[2][4], oc[2][4];
 #pragma unroll
@@ -421,21 +508,33 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecArgs a, const Se
 #pragma unroll
             for (int n = 0; n < 2; n++) {
                 const int at = at_tok(8 * n + g, 8 * k + 2 * t, DK);
-                if (KIND == REC_DELTA) mma3(u[n], uc[n], sa, SplitB(*reinterpret_cast<const float2 *>(mw + at)));
+                if (rec_has_w(KIND)) mma3(u[n], uc[n], sa, SplitB(*reinterpret_cast<const float2 *>(mw + at)));
                 mma3(o[n], oc[n], sa, SplitB(*reinterpret_cast<const float2 *>(mq + at)));
             }
         }
-        if (KIND == REC_DELTA) {
+        if (rec_has_w(KIND)) {
 #pragma unroll
             for (int n = 0; n < 2; n++)
 #pragma unroll
                 for (int e = 0; e < 4; e++) u[n][e] += uc[n][e];
         }
         const SplitA ua[2] = {SplitA(u[0]), SplitA(u[1])};
+        if (KIND == REC_GENERAL) {  // V takes the place of U0 for the second set of products
+#pragma unroll
+            for (int n = 0; n < 2; n++) {
+                const float *mv = mu + 16 * kC;
+                const float2 x = *reinterpret_cast<const float2 *>(mv + at_16(g, 8 * n + 2 * t)), y = *reinterpret_cast<const float2 *>(mv + at_16(g + 8, 8 * n + 2 * t));
+                u[n][0] = x.x, u[n][1] = x.y, u[n][2] = y.x, u[n][3] = y.y;
+            }
+        }
+        const SplitA va[2] = {SplitA(u[0]), SplitA(u[1])};
 #pragma unroll
         for (int k = 0; k < 2; k++)
 #pragma unroll
-            for (int n = 0; n < 2; n++) mma3(o[n], oc[n], ua[k], SplitB(*reinterpret_cast<const float2 *>(mp + at_16(8 * n + g, 8 * k + 2 * t))));
+            for (int n = 0; n < 2; n++) {
+                mma3(o[n], oc[n], ua[k], SplitB(*reinterpret_cast<const float2 *>(mp + at_16(8 * n + g, 8 * k + 2 * t))));
+                if (KIND == REC_GENERAL) mma3(o[n], oc[n], va[k], SplitB(*reinterpret_cast<const float2 *>(mp + kC * kC + at_16(8 * n + g, 8 * k + 2 * t))));
+            }
         // the state moves on
 #pragma unroll
         for (int n = 0; n < NT; n++) {
@@ -443,7 +542,10 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecArgs a, const Se
             float cor[4] = {0.f, 0.f, 0.f, 0.f};
             st[n][0] *= b.x, st[n][1] *= b.y, st[n][2] *= b.x, st[n][3] *= b.y;
 #pragma unroll
-            for (int k = 0; k < 2; k++) mma3(st[n], cor, ua[k], SplitB(*reinterpret_cast<const float2 *>(mk + at_16(8 * n + g, 8 * k + 2 * t))));
+            for (int k = 0; k < 2; k++) {
+                mma3(st[n], cor, ua[k], SplitB(*reinterpret_cast<const float2 *>(mk + at_16(8 * n + g, 8 * k + 2 * t))));
+                if (KIND == REC_GENERAL) mma3(st[n], cor, va[k], SplitB(*reinterpret_cast<const float2 *>(mk + kC * DK + at_16(8 * n + g, 8 * k + 2 * t))));
+            }
 #pragma unroll
             for (int e = 0; e < 4; e++) st[n][e] += cor[e];
         }
@@ -500,7 +602,7 @@ template <class AT, int KIND, int DK>
 static int32_t chunk_launch(const StepDesc &d, const RecArgs &a, int pdl, cudaStream_t st) {
     JGPT_REQUIRE((uint64_t)d.n_chunks * a.heads * record_floats(KIND, DK, a.DV) <= a.chunk_ws_floats, JGPT_ERR_INVALID_ARGUMENT,
                  "%d chunks exceed the workspace", d.n_chunks);
-    auto prep_smem = [](int DV) { return sizeof(float) * ((size_t)kC * (3 * DK + DV) + 3 * kC * kC + kC); };
+    auto prep_smem = [](int DV) { return sizeof(float) * ((size_t)kC * (rec_key_vectors(KIND) * DK + DV) + (KIND == REC_GENERAL ? 5 : 3) * kC * kC + kC); };
     static thread_local int set1 = -1, set2 = -1, set3 = -1;
     int32_t rc = launch_early(rec_prep_kernel<AT, KIND, DK>, dim3((unsigned)d.n_chunks, (unsigned)a.heads), 256, prep_smem(a.DV), set1, prep_smem(256), pdl,
                               st, a, d.segs, d.chunks, pdl);
@@ -509,9 +611,10 @@ static int32_t chunk_launch(const StepDesc &d, const RecArgs &a, int pdl, cudaSt
     const int groups = a.DV / 16, max_warps = DK <= 128 ? 8 : 4;
     int nw = std::min(groups, max_warps);
     while (nw > 1 && (groups % nw != 0 || (long long)a.heads * d.n_long * (groups / nw) < a.sm_count)) nw--;
-    const size_t smem = sizeof(float) * kScanStages * scan_stage_floats(KIND, DK, 16 * nw);
-    rc = launch_early(rec_scan_kernel<KIND == REC_DELTA ? REC_DELTA : REC_GLA, DK>, dim3((unsigned)(a.heads * (groups / nw)), (unsigned)d.n_long), 32 * nw, smem, set2,
-                      sizeof(float) * kScanStages * scan_stage_floats(KIND, DK, 16 * max_warps), pdl, st, a, d.segs, d.long_segs, pdl);
+    constexpr int form = rec_has_w(KIND) ? KIND : REC_GLA, stages = scan_stages(form, DK);
+    const size_t smem = sizeof(float) * stages * scan_stage_floats(KIND, DK, 16 * nw);
+    rc = launch_early(rec_scan_kernel<form, DK>, dim3((unsigned)(a.heads * (groups / nw)), (unsigned)d.n_long), 32 * nw, smem, set2,
+                      sizeof(float) * stages * scan_stage_floats(KIND, DK, 16 * max_warps), pdl, st, a, d.segs, d.long_segs, pdl);
     if (rc) return rc;
     return launch_early(rec_chunk_norm_kernel<AT, KIND>, dim3((unsigned)d.n_chunks, (unsigned)((kC * (a.heads / norm_heads_per_warp(a.DV) + 1) + 31) / 32)), 256, 0, set3, 0, pdl, st, a, d.segs,
                         d.chunks, pdl);
@@ -537,6 +640,7 @@ int32_t launch_recurrent_chunks(bool f32, const StepDesc &d, const RecArgs &a, i
         case REC_DELTA: return f32 ? chunk_dispatch<float, REC_DELTA>(d, a, pdl, st) : chunk_dispatch<__nv_bfloat16, REC_DELTA>(d, a, pdl, st);
         case REC_HGRN2: return f32 ? chunk_dispatch<float, REC_HGRN2>(d, a, pdl, st) : chunk_dispatch<__nv_bfloat16, REC_HGRN2>(d, a, pdl, st);
         case REC_WKV: return f32 ? chunk_dispatch<float, REC_WKV>(d, a, pdl, st) : chunk_dispatch<__nv_bfloat16, REC_WKV>(d, a, pdl, st);
+        case REC_GENERAL: return f32 ? chunk_dispatch<float, REC_GENERAL>(d, a, pdl, st) : chunk_dispatch<__nv_bfloat16, REC_GENERAL>(d, a, pdl, st);
     }
     return fail(JGPT_ERR_INVALID_ARGUMENT, "recurrence %d", a.kind);
 }

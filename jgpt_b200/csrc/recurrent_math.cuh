@@ -49,12 +49,13 @@ template <class AT>
 __device__ __forceinline__ float2 forget_write(float z, float low) {
     return make_float2(low + (1.f - low) * sigmoid_f<AT>(z), (1.f - low) * sigmoid_f<AT>(-z));
 }
+__host__ __device__ constexpr int rec_key_vectors(int kind) { return kind == REC_GENERAL ? 4 : 3; }  // vectors of key channels per token: q, k, decays, removal
 __host__ __device__ constexpr bool rec_has_key(int kind) { return kind != REC_HGRN2; }   // a projection of its own for k
 __host__ __device__ constexpr bool rec_has_gate(int kind) { return kind != REC_HGRN2; }  // an output gate
 // Gate factor of a head's output from the gate projection.
 template <class AT, int KIND>
 __device__ __forceinline__ float out_gate(float g) {
-    return KIND == REC_DELTA ? sigmoid_f<AT>(g) : g * sigmoid_f<AT>(g);
+    return KIND == REC_DELTA || KIND == REC_GENERAL ? sigmoid_f<AT>(g) : g * sigmoid_f<AT>(g);
 }
 
 // RMS norm over a head's value columns and its output gate: raw fp32 values -> activations.  A warp takes heads h0, h0 + 1, ... of a

@@ -15,11 +15,13 @@ from . import binding as B
 from .kv_cache import KvPool
 from .runtime import Context
 
-MIX_ATTENTION, MIX_GLA, MIX_DELTA, MIX_HGRN2, MIX_WKV, MIX_LATENT = range(1, 7)
+MIX_ATTENTION, MIX_GLA, MIX_DELTA, MIX_HGRN2, MIX_WKV, MIX_LATENT, MIX_GENERAL_DELTA = range(1, 8)
 NORM_LAYER, NORM_RMS = 0, 1
-FF_GATED_GELU, FF_XIELU, FF_GATED_RELU, FF_MOE = range(4)
+FF_GATED_GELU, FF_XIELU, FF_GATED_RELU, FF_MOE, FF_RELU2 = range(5)
 ACT_RELU, ACT_RELU2, ACT_GELU_TANH = range(3)
 GATE_NONE, GATE_HEAD, GATE_ELEMENT = range(3)
+QK_NORM_NONE, QK_NORM_HEAD, QK_NORM_ALL, QK_NORM_UNIT = range(4)
+SINK_NONE, SINK_LEARNED, SINK_ZERO = range(3)
 NO_LIMIT = 1 << 30  # positions of a model without a table of them
 DTYPES = {"bfloat16": 0, "float32": 1}
 BLOCK_TOKENS = 16
@@ -31,7 +33,8 @@ class _MixerSpec(C.Structure):
                [(n, C.c_float) for n in ("score_scale", "tau", "out_scale")] + \
                [(n, C.c_int32) for n in ("window", "q_rank", "kv_rank", "rot_dim", "rot_dims", "kv_from")] + \
                [(n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")] + \
-               [(n, C.c_int32) for n in ("rot_interleaved", "qkv_bias", "qk_norm", "maps")] + [("diff", C.c_float)]
+               [(n, C.c_int32) for n in ("rot_interleaved", "qkv_bias", "qk_norm", "maps")] + [("diff", C.c_float)] + \
+               [(n, C.c_int32) for n in ("keep", "sink", "v_mix")] + [("decay_rate", C.c_float)]
 
 
 class _MoeSpec(C.Structure):
@@ -46,7 +49,7 @@ class _DecoderSpec(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("vocab", "width", "max_positions", "n_layers", "embed_norm", "pos_table", "norm", "head", "layer_scale",
                                            "depth_average")] + \
                [(n, C.c_float) for n in ("eps", "embed_scale", "logit_scale", "residual_mult")] + \
-               [("norm_after", C.c_int32), ("residual_scale", C.c_float)]
+               [("norm_after", C.c_int32), ("residual_scale", C.c_float)] + [(n, C.c_int32) for n in ("norm_both", "token_shift", "residual_gate")]
 
 
 # tensor roles (JGPT_W_* of the header)
@@ -54,8 +57,10 @@ W_EMBED, W_POS, W_EMBED_NORM, W_EMBED_NORM_B, W_FINAL_NORM, W_FINAL_NORM_B, W_HE
 W_NORM1, W_NORM1_B, W_NORM2, W_NORM2_B, W_FF_GATE, W_FF_UP, W_FF_DOWN, W_LS1, W_LS2, W_DWA = range(10, 20)
 (W_Q, W_K, W_V, W_O, W_G, W_B, W_A1, W_A2, W_DECAY_BIAS, W_A_LOG, W_G1, W_G2, W_HEAD_NORM, W_CONV_Q, W_CONV_K,
  W_CONV_V, W_MU_R, W_MU_K, W_MU_V, W_MU_G, W_MU_W, W_BONUS, W_LOWER, W_F, W_DQ, W_DQ_NORM, W_UQ, W_DKV, W_DKV_NORM, W_UK, W_UV,
- W_FF_ACT, W_Q_BIAS, W_K_BIAS, W_V_BIAS, W_Q_NORM, W_K_NORM, W_LQ1, W_LK1, W_LQ2, W_LK2) = range(20, 61)
+ W_FF_ACT, W_Q_BIAS, W_K_BIAS, W_V_BIAS, W_Q_NORM, W_K_NORM, W_LQ1, W_LK1, W_LQ2, W_LK2, W_SINK,
+ W_VMIX, W_B_BIAS) = range(20, 64)
 W_ROUTER, W_CORRECTION, W_SHARED_GATE, W_SHARED_UP, W_SHARED_DOWN, W_EXPERT_UP, W_EXPERT_DOWN = range(64, 71)
+W_POST1, W_POST2, W_SHIFT, W_RG1, W_RG1_B, W_RG2, W_RG2_B = range(80, 87)
 
 
 @dataclass
@@ -86,9 +91,13 @@ class Mixer:
     rot_slow: float = 0.0
     rot_interleaved: bool = False
     qkv_bias: bool = False
-    qk_norm: bool = False
+    qk_norm: int = QK_NORM_NONE
     maps: int = 1  # 2: differential, the second map's output times lambda is taken off the first one's
     diff: float = 0.0
+    keep: int = 0
+    sink: int = SINK_NONE
+    v_mix: bool = False
+    decay_rate: float = 1.0
     tensors: dict = field(default_factory=dict)  # role -> tensor name
 
 
@@ -134,6 +143,9 @@ class DecoderConfig:
     residual_mult: float = 1.0
     norm_after: bool = False
     residual_scale: float = 1.0
+    norm_both: bool = False
+    token_shift: bool = False
+    residual_gate: bool = False
     tensors: dict = field(default_factory=dict)
 
     def all_tensors(self):

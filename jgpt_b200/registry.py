@@ -6,6 +6,7 @@ weight file for sizes that only the tensors hold.
 from __future__ import annotations
 
 import json
+import math
 import os
 
 from . import decoder as D
@@ -158,13 +159,13 @@ def zusepel(c, shape_of) -> D.DecoderConfig:
 # ---- Nefipel -------------------------------------------------------------------------------------------
 def _gated_heads(m, p):
     return D.Mixer(D.MIX_ATTENTION, m["heads"], m["kv_heads"], m["dim"], m["vdim"], gate=D.GATE_ELEMENT, score_scale=m["scale"], qkv_bias=True,
-                   qk_norm=True, **_rotation(m["rot"]),
+                   qk_norm=D.QK_NORM_HEAD, **_rotation(m["rot"]),
                    tensors={D.W_Q: p + "q", D.W_K: p + "k", D.W_V: p + "v", D.W_Q_BIAS: p + "q.b", D.W_K_BIAS: p + "k.b", D.W_V_BIAS: p + "v.b",
                             D.W_Q_NORM: p + "q.norm", D.W_K_NORM: p + "k.norm", D.W_G: p + "g", D.W_O: p + "o"})
 
 
 def _differential(m, p):
-    return D.Mixer(D.MIX_ATTENTION, m["heads"], m["kv_heads"], m["dim"], m["vdim"], score_scale=m["scale"], qk_norm=True, rot_interleaved=True,
+    return D.Mixer(D.MIX_ATTENTION, m["heads"], m["kv_heads"], m["dim"], m["vdim"], score_scale=m["scale"], qk_norm=D.QK_NORM_HEAD, rot_interleaved=True,
                    maps=2, diff=m["diff"], **_rotation(m["rot"]),
                    tensors={D.W_Q: p + "q", D.W_K: p + "k", D.W_V: p + "v", D.W_Q_NORM: p + "q.norm", D.W_K_NORM: p + "k.norm", D.W_LQ1: p + "lq1",
                             D.W_LK1: p + "lk1", D.W_LQ2: p + "lq2", D.W_LK2: p + "lk2", D.W_O: p + "o"})
@@ -208,3 +209,58 @@ def nefipel(c, shape_of) -> D.DecoderConfig:
     return D.DecoderConfig(c["vocab"], c["width"], D.NO_LIMIT, c["norm"]["eps"], layers, pos_table=False, norm=D.NORM_RMS,
                            embed_scale=c["embedding"]["scale"], norm_after=True, residual_scale=c["postln_alpha"],
                            tensors={D.W_EMBED: "embed", D.W_FINAL_NORM: "final.norm"})
+
+
+# ---- Lipelix -------------------------------------------------------------------------------------------
+def _mixed_values(m, p, first):
+    """The first layer that mixes its values is the one they come from: it has no share of its own."""
+    if not m.get("v_mix"):
+        return False, {}
+    return True, {} if first else {D.W_VMIX: p + "vmix"}
+
+
+def _normed_rows(m, p, v_mix, names):
+    return D.Mixer(D.MIX_ATTENTION, m["heads"], m["kv_heads"], m["dim"], m["vdim"], score_scale=m["scale"], qk_norm=D.QK_NORM_ALL, sink=D.SINK_LEARNED,
+                   v_mix=v_mix, **_rotation(m["rot"]),
+                   tensors={D.W_Q: p + "q", D.W_K: p + "k", D.W_V: p + "v", D.W_Q_NORM: p + "q.norm", D.W_K_NORM: p + "k.norm", D.W_SINK: p + "sink",
+                            D.W_O: p + "o", **names})
+
+
+def _windowed(m, p, v_mix, names):
+    return D.Mixer(D.MIX_ATTENTION, m["heads"], m["kv_heads"], m["dim"], m["vdim"], score_scale=m["scale"], qk_norm=D.QK_NORM_UNIT, sink=D.SINK_ZERO,
+                   window=m["mask"]["size"], keep=m["mask"].get("keep_first", 0), v_mix=v_mix, **_rotation(m["rot"]),
+                   tensors={D.W_Q: p + "q", D.W_K: p + "k", D.W_V: p + "v", D.W_O: p + "o", **names})
+
+
+def _general_delta(m, p, shape_of):
+    return D.Mixer(D.MIX_GENERAL_DELTA, m["heads"], m["heads"], m["dim"], m["dim"], rank_a=shape_of(p + "w1")[0], decay_rate=math.exp(-0.5),
+                   tensors={D.W_Q: p + "r", D.W_K: p + "k", D.W_V: p + "v", D.W_G: p + "g", D.W_B: p + "a", D.W_B_BIAS: p + "a.b", D.W_A1: p + "w1",
+                            D.W_A2: p + "w2", D.W_DECAY_BIAS: p + "w0", D.W_HEAD_NORM: p + "norm", D.W_O: p + "o"})
+
+
+@register("Lipelix")
+def lipelix(c, shape_of) -> D.DecoderConfig:
+    """Layers of three kinds in any order: 'attention' (queries and keys normed as whole rows, all earlier positions, a learned
+    sink), 'attention_2' (a sliding window with kept first tokens, unit heads, a sink of score 0) and 'general_delta' (recurrence);
+    norms on both sides of every part, gated results, a token shift, values mixed with the first layer's."""
+    layers, source = [], None
+    for i, e in enumerate(c["layers"]):
+        p, m, mlp = f"l{i}.", e["mixer"], e["mlp"]
+        names = {D.W_NORM1: p + "norm1", D.W_POST1: p + "norm1b", D.W_SHIFT: p + "shift", D.W_RG1: p + "rg1", D.W_RG1_B: p + "rg1.b"}
+        if e["type"] in ("attention", "attention_2"):
+            v_mix, extra = _mixed_values(m, p + "mix.", source is None)
+            source = i if source is None and v_mix else source
+            mixer = (_normed_rows if e["type"] == "attention" else _windowed)(m, p + "mix.", v_mix, extra)
+        elif e["type"] == "general_delta":
+            mixer = _general_delta(m, p + "mix.", shape_of)
+        else:
+            raise ValueError(f"layer {i}: mixer type {e['type']!r}")
+        if mlp is not None:
+            if mlp["kind"] != "dense":
+                raise ValueError(f"layer {i}: feed-forward kind {mlp['kind']!r}")
+            names.update({D.W_NORM2: p + "norm2", D.W_POST2: p + "norm2b", D.W_RG2: p + "rg2", D.W_RG2_B: p + "rg2.b", D.W_FF_UP: p + "mlp.up",
+                          D.W_FF_DOWN: p + "mlp.down"})
+        layers.append(D.Layer([mixer], mlp["ff"] if mlp else 0, names, D.FF_RELU2))
+    return D.DecoderConfig(c["vocab"], c["width"], D.NO_LIMIT, c["norm"]["eps"], layers, pos_table=False, norm=D.NORM_RMS, head=True,
+                           embed_scale=c["embedding"]["scale"], residual_mult=c["residual_mult"], norm_both=True, token_shift=True, residual_gate=True,
+                           tensors={D.W_EMBED: "embed", D.W_FINAL_NORM: "final.norm", D.W_HEAD: "head"})
