@@ -642,7 +642,7 @@ def main():
     ap.add_argument("--launch-overlap", type=int, default=2, help="with --quick --per-layer: 0 ordinary launches, 1 / 2 overlapped")
     ap.add_argument("--batch", type=int, default=64, help="sequences per step for --workload decodestep")
     ap.add_argument("--decoder-widths", default="1024,2048", help="model widths for --workload decoder")
-    ap.add_argument("--decoder-model", default="nefipel", choices=["nefipel", "zusepel", "somopel", "gpt"], help="--workload decoder --quick: the model to run")
+    ap.add_argument("--decoder-model", default="lipelix", choices=["lipelix", "nefipel", "zusepel", "somopel", "gpt"], help="--workload decoder --quick: the model to run")
     ap.add_argument("--decoder-part", default="all", choices=["all", "prefill", "decode"], help="--workload decoder: what to run")
     ap.add_argument("--gather-depth", type=int, default=4, help="continuous batching: steps a rank may run ahead of the token-id gather")
     ap.add_argument("--workload", default="microbench", choices=["microbench", "decode35m", "decodestep", "prefill", "contbatch", "longctx", "kvstore", "phases", "fusedphases", "steptimeline", "decoder"],

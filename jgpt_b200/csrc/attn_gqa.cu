@@ -93,24 +93,26 @@ __device__ __forceinline__ void prepare_head(float (&x)[8], const AT *src, int p
 }
 __host__ __device__ constexpr int head_lanes(int DK) { return DK <= 32 ? 4 : (DK <= 64 ? 8 : (DK <= 128 ? 16 : 32)); }
 
-// 1 / root mean square of n heads of a row (padding is zero), by all threads of the block.
+// 1 / root mean square of all query heads and of all key heads of a row (padding is zero), by all threads of the block.
 template <class AT>
-__device__ __forceinline__ float row_rms(const AT *src, int n, const AttnArgs &a, float *red) {
-    float ss = 0.f;
-    for (int c = threadIdx.x * 8; c < n * a.DK; c += blockDim.x * 8) {
-        float x[8];
-        load8(src + c, x);
+__device__ __forceinline__ float2 row_rms(const AT *proj, const AttnArgs &a, float2 *red) {
+    float2 ss = make_float2(0.f, 0.f);
+    const int nq = a.heads * a.DK, n = nq + a.kv_heads * a.DK;
+    for (int c = threadIdx.x * 8; c < n; c += blockDim.x * 8) {
+        float x[8], s = 0.f;
+        load8(proj + (c < nq ? a.q_off + c : a.k_off + c - nq), x);
 #pragma unroll
-        for (int e = 0; e < 8; e++) ss += x[e] * x[e];
+        for (int e = 0; e < 8; e++) s += x[e] * x[e];
+        if (c < nq) ss.x += s;
+        else ss.y += s;
     }
 #pragma unroll
-    for (int off = 16; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
-    __syncthreads();  // the previous use of red is over
+    for (int off = 16; off >= 1; off >>= 1) ss.x += __shfl_xor_sync(0xffffffffu, ss.x, off), ss.y += __shfl_xor_sync(0xffffffffu, ss.y, off);
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
     __syncthreads();
-    ss = 0.f;
-    for (int w = 0; w < (int)blockDim.x / 32; w++) ss += red[w];
-    return 1.f / sqrtf(ss / (float)(n * a.dim) + a.eps);
+    ss = make_float2(0.f, 0.f);
+    for (int w = 0; w < (int)blockDim.x / 32; w++) ss.x += red[w].x, ss.y += red[w].y;
+    return make_float2(1.f / sqrtf(ss.x / (float)(a.heads * a.dim) + a.eps), 1.f / sqrtf(ss.y / (float)(a.kv_heads * a.dim) + a.eps));
 }
 
 // Eight values of a key head from column c on, mixed with another layer's (whose heads may be cut differently).
@@ -119,36 +121,42 @@ __device__ __forceinline__ void load_values(const AttnArgs &a, int row, int g, i
     load8(reinterpret_cast<const AT *>(a.proj) + (size_t)row * a.ldp + a.v_off + g * a.DV + c, x);
     if (!a.v_first) return;
     const AT *first = reinterpret_cast<const AT *>(a.v_first) + (size_t)row * a.ld_first;
-    float y[8];
+    const float keep = 1.f - a.v_share;
     if (a.vdim_first == a.vdim && c + 8 <= a.DV_first) {
+        float y[8];
         load8(first + g * a.DV_first + c, y);
-    } else {
 #pragma unroll
-        for (int e = 0; e < 8; e++) {
-            const int i = g * a.vdim + c + e;
-            y[e] = c + e < a.vdim ? act_load(first + i / a.vdim_first * a.DV_first + i % a.vdim_first) : 0.f;
-        }
+        for (int e = 0; e < 8; e++) x[e] = fmaf(a.v_share, y[e], keep * x[e]);
+        return;
+    }
+    AT mixed[8];
+    const AT *own = reinterpret_cast<const AT *>(a.proj) + (size_t)row * a.ldp + a.v_off + g * a.DV + c;
+#pragma unroll 1
+    for (int e = 0; e < 8; e++) {
+        const int i = g * a.vdim + c + e;
+        act_store(mixed + e, c + e < a.vdim ? fmaf(a.v_share, act_load(first + i / a.vdim_first * a.DV_first + i % a.vdim_first), keep * act_load(own + e)) : 0.f);
     }
 #pragma unroll
-    for (int e = 0; e < 8; e++) x[e] = fmaf(a.v_share, y[e], (1.f - a.v_share) * x[e]);
+    for (int e = 0; e < 8; e++) x[e] = act_load(mixed + e);
 }
 
 // A block (or several, in y) per row: its query maps (with `queries`, in place), key maps and values (into the page), a vector per
-// head_lanes(DK) lanes.
-template <class AT>
+// head_lanes(DK) lanes.  WIDE: norms over the whole row, by the one block that has it, and mixed values.
+template <class AT, bool WIDE>
 __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a, const int *__restrict__ seq, const int *__restrict__ pos, int queries, int pdl) {
+    __shared__ float2 red[8];
     if (pdl & 2) griddep_launch_dependents();
-    __shared__ float red[8];
     const int lanes = head_lanes(a.DK), nq = queries ? a.heads * a.maps : 0, nk = a.kv_heads * a.maps, nv = nq + nk + a.kv_heads;
     const int r = blockIdx.x, piece = threadIdx.x & (lanes - 1), per = blockDim.x / lanes;
     const int p = pos[r], row = p % kBlockTokens, phys = page_of(a, seq[r], p), kw = a.maps * a.DK;
     if (pdl & 1) griddep_wait();
     AT *proj = reinterpret_cast<AT *>(a.proj) + (size_t)r * a.ldp;
     float2 inv = make_float2(1.f, 1.f);
-    if (a.qk_norm == QK_NORM_ALL) {  // one block has the row then
-        inv.x = row_rms(proj + a.q_off, a.heads, a, red), inv.y = row_rms(proj + a.k_off, a.kv_heads, a, red);
+    if (WIDE && a.qk_norm == QK_NORM_ALL) {
+        inv = row_rms(proj, a, red);
         if (threadIdx.x == 0) a.row_inv[r] = inv;
     }
+#pragma unroll 1
     for (int i0 = blockIdx.y * per; i0 < nv; i0 += gridDim.y * per) {
         const int i = i0 + threadIdx.x / lanes;
         const bool query = i < nq, value = i >= nq + nk && i < nv, key = i >= nq && i < nq + nk;
@@ -156,9 +164,12 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a, const 
         AT *page = reinterpret_cast<AT *>(a.kv) + ((size_t)max(phys, 0) * a.kv_heads + g) * a.page_head();
         if (value && phys >= 0) {
             AT *dst = page + kBlockTokens * page_row(kw) + row * page_row(a.DV);
+#pragma unroll 1
             for (int c = piece; c < a.DV / 8; c += lanes) {
                 float x[8];
-                load_values<AT>(a, r, g, c * 8, x), store8(dst + page_chunk(a.DV, row, c) * 8, x);
+                if (WIDE) load_values<AT>(a, r, g, c * 8, x);
+                else load8(proj + a.v_off + g * a.DV + c * 8, x);
+                store8(dst + page_chunk(a.DV, row, c) * 8, x);
             }
         }
         const int head = query ? i : (key ? i - nq : 0);
@@ -171,9 +182,9 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a, const 
             for (int e = 0; e < 8; e++) x[e] = 0.f;
         }
         if (a.prepared()) prepare_head(x, src, piece, lanes, head_prep(a, !query, r, head, query ? inv.x : inv.y));
-        if (!load) continue;
-        if (query) store8(proj + a.q_off + i * a.DK + piece * 8, x);
-        else if (phys >= 0) store8(page + row * page_row(kw) + page_chunk(kw, row, (i - nq) % a.maps * (a.DK / 8) + piece) * 8, x);
+        if (load && query) store8(proj + a.q_off + i * a.DK + piece * 8, x);
+        else if (load && phys >= 0) store8(page + row * page_row(kw) + page_chunk(kw, row, (i - nq) % a.maps * (a.DK / 8) + piece) * 8, x);
+        if (!WIDE) break;
     }
 }
 
@@ -278,7 +289,8 @@ struct Tile {
     static constexpr size_t smem = (ring > hand ? ring : hand) + (size_t)64 * LQ * 2;
 };
 
-template <int DK, int DV, int MAPS>
+// WINDOW: a window with kept tokens.
+template <int DK, int DV, int MAPS, bool WINDOW>
 __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_kernel(const AttnArgs a, const Seg *__restrict__ segs, const int2 *__restrict__ tiles, int qt, int pdl) {
     using T = Tile<DK, DV, MAPS>;
     using P = typename T::P;
@@ -298,7 +310,7 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
     if (r0 >= rows) return;
     const int p0 = sg.pos0 + tile.y, b0 = p0 + r0 / grp, p1 = p0 + (min(rows, r0 + ROWS) - 1) / grp;  // positions: of the tile, of the block's rows
     // keys in tiles: the kept ones when they lie apart, then those from the first one that the block's first row sees
-    const int win = first_visible(b0, a) / kBlockTokens * kBlockTokens, kept = kept_apart(win, a), first = a.keep && !kept ? 0 : win;
+    const int win = first_visible(b0, a) / kBlockTokens * kBlockTokens, kept = WINDOW ? kept_apart(win, a) : 0, first = WINDOW && a.keep && !kept ? 0 : win;
     const int n_kept = (kept + KT - 1) / KT, n_tiles = n_kept + (p1 - first) / KT + 1;
     auto tile_key = [&](int it) { return it < n_kept ? it * KT : first + (it - n_kept) * KT; };
     if (tid == 0) {
@@ -385,7 +397,7 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
     const int vis_lo = first_visible(p1, a);
     for (int it = 0; it < n_tiles; it++) {
         const int s = it % ST, kb = tile_key(it);
-        const bool apart = it < n_kept;
+        const bool apart = WINDOW && it < n_kept;
         if (!__all_sync(0xffffffffu, mbar_wait_bounded(&full[s], (it / ST) & 1, a.status, s_abort))) break;
         __nv_bfloat16 *stage = ring + s * T::stage_elems;
         if (kb + KT > p1 + 1) {  // every warp clears what it is going to read
@@ -396,11 +408,11 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
         }
         auto kat = [&](int r, int c) { return P::k(stage + (r >> 4) * P::ELEMS, r & 15, map * (DK / 8) + c); };
         auto vat = [&](int r, int c) { return P::v(stage + (r >> 4) * P::ELEMS, r & 15, c); };
-        if (apart) {
-            const int all[2] = {0, 0}, top[2] = {kept - 1, kept - 1};
-            attend_tile<DK, DV, KT>(qfrag, kat, vat, kb, kb + KT > kept, all, top, 0, sl, m, l, o, lane);
+        if (WINDOW) {
+            const int from[2] = {apart ? 0 : lo[0], apart ? 0 : lo[1]}, to[2] = {apart ? kept - 1 : hi[0], apart ? kept - 1 : hi[1]};
+            attend_tile<DK, DV, KT, true>(qfrag, kat, vat, kb, apart || kb + KT - 1 > b0 || kb < vis_lo, from, to, a.keep, sl, m, l, o, lane);
         } else {
-            attend_tile<DK, DV, KT>(qfrag, kat, vat, kb, kb + KT - 1 > b0 || kb < vis_lo, lo, hi, a.keep, sl, m, l, o, lane);
+            attend_tile<DK, DV, KT, false>(qfrag, kat, vat, kb, kb + KT - 1 > b0 || kb < vis_lo, lo, hi, 0, sl, m, l, o, lane);
         }
         __syncwarp();
         if (lane == 0) mbar_arrive(&empty[s]);
@@ -492,7 +504,7 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
     float *merged = reinterpret_cast<float *>(attn_smem + S::front);           // [16][m, l, -, -, o[DV]] of this CTA, after the loop
     __nv_bfloat16 *qs = reinterpret_cast<__nv_bfloat16 *>(attn_smem + S::front), *own = qs + 16 * LQ;  // query rows [16][LQ]; the token's [K | V]
     __shared__ __align__(8) uint64_t full[4][ST];
-    __shared__ float red[4];
+    __shared__ float2 red[4];
     __shared__ int s_abort_mem;
     volatile int *s_abort = &s_abort_mem;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t2 = 2 * (lane & 3);
@@ -543,8 +555,7 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
         float2 inv = make_float2(1.f, 1.f);
         if (a.qk_norm == QK_NORM_ALL) {
             if (fused) {
-                inv.x = row_rms(proj + a.q_off, a.heads, a, red);
-                if (append) inv.y = row_rms(proj + a.k_off, a.kv_heads, a, red);
+                inv = row_rms(proj, a, red);
             } else {
                 inv = a.row_inv[row];
             }
@@ -591,7 +602,6 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
     for (int n = 0; n < DV / 8; n++)
 #pragma unroll
         for (int e = 0; e < 4; e++) o[n][e] = 0.f;
-    const int lo[2] = {first, first}, hi[2] = {p, p}, kept_lo[2] = {0, 0}, kept_hi[2] = {kept - 1, kept - 1};
     const float sl = a.scale * 1.4426950408889634f;
     for (int i = 0; pg0 + warp + 4 * i < pg1; i++) {
         const bool apart = pg0 + warp + 4 * i < n_kept;
@@ -610,8 +620,8 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
         }
         auto kat = [&](int r, int c) { return P::k(page, r, c); };
         auto vat = [&](int r, int c) { return P::v(page, r, c); };
-        if (apart) attend_tile<DK, DV, 16>(qfrag, kat, vat, kb, kb + 16 > kept, kept_lo, kept_hi, 0, sl, m, l, o, lane);
-        else attend_tile<DK, DV, 16>(qfrag, kat, vat, kb, kb < first || kb + 15 > p, lo, hi, a.keep, sl, m, l, o, lane);
+        const int from = apart ? 0 : first, to = apart ? kept - 1 : p, lo[2] = {from, from}, hi[2] = {to, to};
+        attend_tile<DK, DV, 16, true>(qfrag, kat, vat, kb, kb < from || kb + 15 > to, lo, hi, a.keep, sl, m, l, o, lane);
         __syncwarp();
         load(i + ST);
     }
@@ -737,14 +747,15 @@ int attn_query_tile(int heads, int kv_heads) { return std::max(1, 64 / (heads / 
 // Threads of a row's preparation: one block, or several of 256.
 static void prep_shape(const AttnArgs &a, bool queries, int rows, dim3 *grid, dim3 *block) {
     const int threads = ((queries ? a.heads * a.maps : 0) + a.kv_heads * (a.maps + 1)) * head_lanes(a.DK);
-    *block = dim3((unsigned)std::min(256, (threads + 31) / 32 * 32)), *grid = dim3((unsigned)rows, a.qk_norm == QK_NORM_ALL ? 1u : (threads + block->x - 1) / block->x);
+    *block = dim3((unsigned)std::min(256, (threads + 31) / 32 * 32)), *grid = dim3((unsigned)rows, a.wide() ? 1u : (threads + block->x - 1) / block->x);
 }
 
 template <class AT>
 static int32_t rows_attention(const StepDesc &d, const AttnArgs &a, cudaStream_t st) {
     dim3 grid, block;
     prep_shape(a, a.prepared(), d.rows, &grid, &block);
-    attn_prep_kernel<AT><<<grid, block, 0, st>>>(a, d.seq, d.pos, a.prepared(), 0);
+    if (a.wide()) attn_prep_kernel<AT, true><<<grid, block, 0, st>>>(a, d.seq, d.pos, a.prepared(), 0);
+    else attn_prep_kernel<AT, false><<<grid, block, 0, st>>>(a, d.seq, d.pos, a.prepared(), 0);
     attn_rows_kernel<AT><<<(unsigned)((d.rows * (long long)a.heads + 7) / 8), 256, 0, st>>>(a, d.seq, d.pos, d.rows);
     JGPT_CUDA_TRY(cudaGetLastError());
     return JGPT_OK;
@@ -778,12 +789,25 @@ static int32_t tensor_attention(const StepDesc &d, const AttnArgs &a, int pdl, c
         using T = Tile<DK, DV, MAPS>;
         prep_shape(a, false, d.rows, &cfg.gridDim, &cfg.blockDim);
         cfg.dynamicSmemBytes = 0, cfg.numAttrs = (unsigned)early(0);
-        JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, attn_prep_kernel<__nv_bfloat16>, a, d.seq, d.pos, 0, pdl));
-        static thread_local int set_for = -1;
-        if (int32_t rc = opt_in(attn_tile_kernel<DK, DV, MAPS>, T::smem, set_for)) return rc;
-        cfg.gridDim = dim3((unsigned)d.n_tiles, (unsigned)a.kv_heads, (unsigned)((d.qt * grp + T::ROWS - 1) / T::ROWS)), cfg.blockDim = dim3(160);
-        cfg.dynamicSmemBytes = T::smem, cfg.numAttrs = (unsigned)early(0);
-        JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, attn_tile_kernel<DK, DV, MAPS>, a, d.segs, d.tiles, d.qt, pdl));
+        JGPT_CUDA_TRY(a.wide() ? cudaLaunchKernelEx(&cfg, attn_prep_kernel<__nv_bfloat16, true>, a, d.seq, d.pos, 0, pdl)
+                               : cudaLaunchKernelEx(&cfg, attn_prep_kernel<__nv_bfloat16, false>, a, d.seq, d.pos, 0, pdl));
+        auto tiles = [&](auto kern, int &set_for) -> int32_t {
+            if (int32_t rc = opt_in(kern, T::smem, set_for)) return rc;
+            cfg.gridDim = dim3((unsigned)d.n_tiles, (unsigned)a.kv_heads, (unsigned)((d.qt * grp + T::ROWS - 1) / T::ROWS)), cfg.blockDim = dim3(160);
+            cfg.dynamicSmemBytes = T::smem, cfg.numAttrs = (unsigned)early(0);
+            JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, kern, a, d.segs, d.tiles, d.qt, pdl));
+            return JGPT_OK;
+        };
+        static thread_local int plain_for = -1, window_for = -1;
+        if constexpr (MAPS == 1) {
+            if (a.window > 0) {
+                if (int32_t rc = tiles(attn_tile_kernel<DK, DV, MAPS, true>, window_for)) return rc;
+            } else if (int32_t rc = tiles(attn_tile_kernel<DK, DV, MAPS, false>, plain_for)) {
+                return rc;
+            }
+        } else if (int32_t rc = tiles(attn_tile_kernel<DK, DV, MAPS, false>, plain_for)) {
+            return rc;
+        }
     }
     if (d.n_singles) {
         static thread_local int set_for = -1;

@@ -532,7 +532,7 @@ __global__ void __launch_bounds__(128, DK <= 192 ? 3 : 1) latent_tile_kernel(con
         const bool masked = kb + kTileKeys - 1 > p0 - en.key0 || kb < vis_lo;
         auto kat = [&](int r, int c) { return ks + r * LK + c * 8; };
         auto vat = [&](int r, int c) { return ks + kTileKeys * LK + r * LV + c * 8; };
-        attend_tile<DK, DV, kTileKeys>(qfrag, kat, vat, kb, masked, lo, hi, 0, sl, m, l, o, lane);
+        attend_tile<DK, DV, kTileKeys, false>(qfrag, kat, vat, kb, masked, lo, hi, 0, sl, m, l, o, lane);
         __syncthreads();
     }
 #pragma unroll

@@ -71,8 +71,8 @@ __device__ __forceinline__ void store8(float *p, const float (&v)[8]) {
 
 // 16 rows x KT keys of one warp against staged K and V rows: scores, online softmax, P.V.  kat / vat (row, chunk): address of the
 // chunk-th 8 elements of a row.  lo / hi: visible key range of this thread's rows g and g + 8 (inclusive),
-// keys before `keep` are seen as well; kb: first key of the tile.
-template <int DK, int DV, int KT, class QFrag, class KAt, class VAt>
+// with KEEP keys before `keep` are seen as well; kb: first key of the tile.
+template <int DK, int DV, int KT, bool KEEP, class QFrag, class KAt, class VAt>
 __device__ __forceinline__ void attend_tile(const QFrag &qfrag, const KAt &kat, const VAt &vat, int kb, bool masked, const int (&lo)[2],
                                             const int (&hi)[2], int keep, float scale_log2, float (&m)[2], float (&l)[2], float (&o)[DV / 8][4], int lane) {
     constexpr int NT = KT / 8;
@@ -100,7 +100,7 @@ __device__ __forceinline__ void attend_tile(const QFrag &qfrag, const KAt &kat, 
 #pragma unroll
         for (int e = 0; e < 4; e++) {
             const int key = kb + j * 8 + t2 + (e & 1), r = e >> 1;
-            s[j][e] = (!masked || ((key >= lo[r] || key < keep) && key <= hi[r])) ? s[j][e] * scale_log2 : -INFINITY;
+            s[j][e] = (!masked || ((key >= lo[r] || (KEEP && key < keep)) && key <= hi[r])) ? s[j][e] * scale_log2 : -INFINITY;
             mx[r] = fmaxf(mx[r], s[j][e]);
         }
     float f[2];

@@ -316,7 +316,7 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
             if (s.rot_dims) TRY(find_rotation(d, s, &b.rot));
             JGPT_REQUIRE(s.qk_norm >= 0 && s.qk_norm <= JGPT_QK_NORM_UNIT && (s.qk_norm != JGPT_QK_NORM_ALL || b.maps == 1), JGPT_ERR_UNSUPPORTED,
                          "layer %d: norm %d of queries and keys, %d maps", index, s.qk_norm, b.maps);
-            JGPT_REQUIRE(s.window >= 0 && s.keep >= 0 && !(s.window && s.chunk) && (s.window || !s.keep) && s.sink >= 0 && s.sink <= JGPT_SINK_ZERO &&
+            JGPT_REQUIRE(s.window >= 0 && s.keep >= 0 && !(s.window && (s.chunk || b.maps > 1)) && (s.window || !s.keep) && s.sink >= 0 && s.sink <= JGPT_SINK_ZERO &&
                              (!s.sink || b.maps == 1),
                          JGPT_ERR_INVALID_ARGUMENT, "layer %d: window %d with %d kept, chunk %d, sink %d, %d maps", index, s.window, s.keep, s.chunk, s.sink, b.maps);
             if (s.qk_norm == JGPT_QK_NORM_HEAD || s.qk_norm == JGPT_QK_NORM_ALL) {

@@ -170,7 +170,8 @@ struct AttnArgs {
     int ldo, out_off;
     int sm_count;
     int *status;
-    __host__ __device__ bool prepared() const { return qk_norm || cs; }  // heads are normed or rotated on their way
+    __host__ __device__ bool prepared() const { return qk_norm || cs; }
+    bool wide() const { return qk_norm == QK_NORM_ALL || v_first; }  // a row's preparation needs more than its own heads  // heads are normed or rotated on their way
     __host__ __device__ int page_head() const { return kBlockTokens * (page_row(maps * DK) + page_row(DV)); }
 };
 int32_t launch_attention(bool f32, const StepDesc &d, const AttnArgs &a, int pdl, cudaStream_t st);

@@ -1,4 +1,4 @@
-"""Prefill and decode throughput of the layered designs (Nefipel, Zusepel, Somopel; random weights) beside the fixed-block GPT model at
+"""Prefill and decode throughput of the layered designs (Lipelix, Nefipel, Zusepel, Somopel; random weights) beside the fixed-block GPT model at
 equal width, depth, feed-forward parameters and vocabulary: ``bench.py --workload decoder``."""
 from __future__ import annotations
 
@@ -75,7 +75,9 @@ def _random_model(ctx, cfg, shapes, max_rows, seed=0):
             return x - 4
         if n.endswith(".correction"):
             return 0.005 * x
-        if n.endswith((".q.b", ".k.b", ".v.b", ".lq1", ".lk1", ".lq2", ".lk2")):
+        if n.endswith((".shift", ".vmix")):
+            return 0.3 + 0.1 * np.tanh(x)
+        if n.endswith((".a.b", ".rg1.b", ".rg2.b", ".q.b", ".k.b", ".v.b", ".lq1", ".lk1", ".lq2", ".lk2")):
             return 0.1 * x
         return x / np.sqrt(s[1]) if len(s) == 2 else 1 + 0.1 * x
     model = D.DecoderModel(ctx, registry.describe(cfg, shapes.__getitem__), "bfloat16", max_rows)
@@ -159,6 +161,36 @@ def random_nefipel(ctx, width, max_rows):
     return _random_model(ctx, cfg, shapes, max_rows)
 
 
+def lipelix_config(width):
+    """Attention over everything, attention in a window of 512 with 16 kept tokens (heads of 128 in groups of four), generalised
+    delta rule with heads of 128; the gates of the results are taken off the feed-forward parts, so a layer is as large as Zusepel's."""
+    h, mlp = width // 128, {"kind": "dense", "ff": width * 25 // 8}
+    att = {"heads": h, "kv_heads": max(h // 4, 1), "dim": 128, "vdim": 128, "rot": {"base": 10000.0, "dims": 128}, "scale": 128 ** -0.5, "v_mix": True}
+    block = [("attention", att), ("attention_2", {**att, "mask": {"size": 512, "keep_first": 16}}), ("general_delta", {"heads": h, "dim": 128})]
+    return {"architecture": "Lipelix", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "embedding": {"scale": 8.0},
+            "layers": [{"type": t, "mixer": m, "mlp": mlp} for t, m in block * (LAYERS // 3)]}
+
+
+def random_lipelix(ctx, width, max_rows, rank=64):
+    cfg = lipelix_config(width)
+    shapes = {"embed": (VOCAB, width), "head": (VOCAB, width), "final.norm": (width,)}
+    for i, e in enumerate(cfg["layers"]):
+        p, m, ff = f"l{i}.", e["mixer"], e["mlp"]["ff"]
+        new = {n: (width,) for n in ("norm1", "norm1b", "norm2", "norm2b", "shift", "rg1.b", "rg2.b")}
+        new.update({"rg1": (width, width), "rg2": (width, width), "mlp.up": (ff, width), "mlp.down": (width, ff)})
+        H, d = m["heads"], m["dim"]
+        if e["type"] == "general_delta":
+            new.update({f"mix.{s}": (H * d, width) for s in "rkvga"})
+            new.update({"mix.a.b": (H * d,), "mix.w0": (H * d,), "mix.norm": (H * d,), "mix.w1": (rank, width), "mix.w2": (H * d, rank), "mix.o": (width, H * d)})
+        else:
+            G, v = m["kv_heads"], m["vdim"]
+            new.update({"mix.q": (H * d, width), "mix.k": (G * d, width), "mix.v": (G * v, width), "mix.o": (width, H * v), "mix.vmix": (1,)})
+            if e["type"] == "attention":
+                new.update({"mix.q.norm": (H * d,), "mix.k.norm": (G * d,), "mix.sink": (H,)})
+        shapes.update({p + n: s for n, s in new.items()})
+    return _random_model(ctx, cfg, shapes, max_rows)
+
+
 def random_gpt(ctx, width, max_rows):
     """The fixed-block model of the same width, depth, feed-forward size and vocabulary (head size 16, its tuned case)."""
     ff, L = width * 11 // 4, LAYERS
@@ -217,12 +249,12 @@ def _prefill(ctx, model, batch, seq_len, repeats):
     return float(np.median(best))
 
 
-def run_decoder(ctx, widths=(1024, 2048), batches=(1, 16, 64), prompts=((1, 2048), (8, 1024)), ctx_len=1500, steps=24, repeats=5, models=("nefipel", "zusepel", "somopel", "gpt")):
+def run_decoder(ctx, widths=(1024, 2048), batches=(1, 16, 64), prompts=((1, 2048), (8, 1024)), ctx_len=1500, steps=24, repeats=5, models=("lipelix", "nefipel", "zusepel", "somopel", "gpt")):
     out = {"workload": f"{LAYERS} layers, vocabulary {VOCAB}, random weights; prefill = prompts of one call, decode at context {ctx_len}+",
            "timing": "prefill: CUDA events around the call; decode: host clock around a step that reads its ids back; medians", "sizes": []}
     for w in widths:
         row = {"width": w}
-        for name, make in (("nefipel", random_nefipel), ("zusepel", random_zusepel), ("somopel", random_somopel), ("gpt", random_gpt)):
+        for name, make in (("lipelix", random_lipelix), ("nefipel", random_nefipel), ("zusepel", random_zusepel), ("somopel", random_somopel), ("gpt", random_gpt)):
             if name not in models:
                 continue
             m = make(ctx, w, 8192)

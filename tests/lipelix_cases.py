@@ -52,6 +52,7 @@ def weights(cfg, seed=0, rank=6):
             n = m["heads"] * m["dim"]
             for k in "rkvga":
                 lin(q + k, n, w)
+            W[q + "r"] = 0.7 * (W[q + "r"] + W[q + "k"])  # a first token's output is (r . k) v brought to unit size: r . k stays away from 0
             vec(q + "a.b", n, 0.0, 0.7), vec(q + "w0", n, -1.0, 1.5), vec(q + "norm", n)
             lin(q + "w1", rank, w), lin(q + "w2", n, rank, 2.0), lin(q + "o", w, n)
         else:
