@@ -18,8 +18,9 @@ namespace jgpt {
 namespace mix {
 
 // First key of the chunk or window of a position; with a window the keys before a.keep are seen as well.
+template <bool WINDOW = true>
 __host__ __device__ __forceinline__ int first_visible(int pos, const AttnArgs &a) {
-    if (a.window > 0) return pos >= a.window ? pos - a.window + 1 : 0;
+    if (WINDOW && a.window > 0) return pos >= a.window ? pos - a.window + 1 : 0;
     return a.chunk > 0 ? pos / a.chunk * a.chunk : 0;
 }
 // Keys in front of the window that are visited on their own: none, or [0, keep) when the window's first page lies behind them.
@@ -29,35 +30,32 @@ __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)
 
 // What happens to a query or key head (map) behind its projection: norm, rotation.
 struct HeadPrep {
-    const float *w;  // weights of the norm, null: 1
+    const float *w;  // null: no norm
     const float2 *cs;
-    int dim, half, interleaved, norm;
+    int dim, half, interleaved, whole;
     float eps, inv;  // inv: of the whole row
 };
 // head: which of the row's (its weights, when the whole row has some); inv: 1 / root mean square of the row, when that is what the norm takes
+template <bool WHOLE>
 __device__ __forceinline__ HeadPrep head_prep(const AttnArgs &a, bool key, int row, int head, float inv) {
     const float *w = key ? a.k_norm : a.q_norm;
-    return HeadPrep{w + (a.qk_norm == QK_NORM_ALL ? head * a.DK : 0), a.cs + (size_t)row * a.half, a.dim, a.half, a.interleaved, a.qk_norm, a.eps, inv};
+    const bool whole = WHOLE && a.whole_rows;
+    return HeadPrep{w + (whole ? head * a.DK : 0), a.cs + (size_t)row * a.half, a.dim, a.half, a.interleaved, whole, a.eps, inv};
 }
-__device__ __forceinline__ float head_weight(const HeadPrep &h, int j) { return h.norm == QK_NORM_UNIT ? 1.f : __ldg(h.w + j); }
 // The head lies in 8-element pieces in `lanes` neighbouring lanes (a power of two; every lane of the warp takes part); src: its
 // start in memory.
 template <class AT>
 __device__ __forceinline__ void prepare_head(float (&x)[8], const AT *src, int piece, int lanes, const HeadPrep &h) {
     const int j0 = piece * 8;
     float inv = 1.f;
-    if (h.norm == QK_NORM_ALL) {
-        inv = h.inv;
-#pragma unroll
-        for (int e = 0; e < 8; e++) x[e] = j0 + e < h.dim ? x[e] * inv * __ldg(h.w + j0 + e) : 0.f;
-    } else if (h.norm) {
+    if (h.w) {
         float ss = 0.f;
 #pragma unroll
         for (int e = 0; e < 8; e++) ss += x[e] * x[e];
         for (int off = lanes >> 1; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
-        inv = 1.f / sqrtf(ss / (float)h.dim + h.eps);
+        inv = h.whole ? h.inv : 1.f / sqrtf(ss / (float)h.dim + h.eps);
 #pragma unroll
-        for (int e = 0; e < 8; e++) x[e] = j0 + e < h.dim ? x[e] * inv * head_weight(h, j0 + e) : 0.f;
+        for (int e = 0; e < 8; e++) x[e] = j0 + e < h.dim ? x[e] * inv * __ldg(h.w + j0 + e) : 0.f;
     }
     if (!h.half) return;
     if (h.interleaved) {
@@ -85,7 +83,7 @@ __device__ __forceinline__ void prepare_head(float (&x)[8], const AT *src, int p
             const int j = j0 + e, p = j < h.half ? j + h.half : j - h.half;
             if (j >= 2 * h.half) continue;
             const float2 t = h.cs[(j < h.half ? j : p)];
-            const float y = act_load(src + p) * inv * (h.norm ? head_weight(h, p) : 1.f);
+            const float y = act_load(src + p) * inv * (h.w ? __ldg(h.w + p) : 1.f);
             x[e] = j < h.half ? x[e] * t.x - y * t.y : x[e] * t.x + y * t.y;
         }
         __syncwarp();  // whoever writes the head back does so after this
@@ -115,35 +113,29 @@ __device__ __forceinline__ float2 row_rms(const AT *proj, const AttnArgs &a, flo
     return make_float2(1.f / sqrtf(ss.x / (float)(a.heads * a.dim) + a.eps), 1.f / sqrtf(ss.y / (float)(a.kv_heads * a.dim) + a.eps));
 }
 
-// Eight values of a key head from column c on, mixed with another layer's (whose heads may be cut differently).
+// Values of a key head from column c on, mixed with another layer's, whose heads may be cut differently.
+__device__ __forceinline__ bool values_line_up(const AttnArgs &a, int c) { return !a.v_first || (a.vdim_first == a.vdim && c + 8 <= a.DV_first); }
 template <class AT>
-__device__ __forceinline__ void load_values(const AttnArgs &a, int row, int g, int c, float (&x)[8]) {
+__device__ __forceinline__ void load_values(const AttnArgs &a, int row, int g, int c, float (&x)[8]) {  // eight that line up
     load8(reinterpret_cast<const AT *>(a.proj) + (size_t)row * a.ldp + a.v_off + g * a.DV + c, x);
     if (!a.v_first) return;
-    const AT *first = reinterpret_cast<const AT *>(a.v_first) + (size_t)row * a.ld_first;
-    const float keep = 1.f - a.v_share;
-    if (a.vdim_first == a.vdim && c + 8 <= a.DV_first) {
-        float y[8];
-        load8(first + g * a.DV_first + c, y);
+    float y[8];
+    load8(reinterpret_cast<const AT *>(a.v_first) + (size_t)row * a.ld_first + g * a.DV_first + c, y);
 #pragma unroll
-        for (int e = 0; e < 8; e++) x[e] = fmaf(a.v_share, y[e], keep * x[e]);
-        return;
-    }
-    AT mixed[8];
-    const AT *own = reinterpret_cast<const AT *>(a.proj) + (size_t)row * a.ldp + a.v_off + g * a.DV + c;
-#pragma unroll 1
-    for (int e = 0; e < 8; e++) {
-        const int i = g * a.vdim + c + e;
-        act_store(mixed + e, c + e < a.vdim ? fmaf(a.v_share, act_load(first + i / a.vdim_first * a.DV_first + i % a.vdim_first), keep * act_load(own + e)) : 0.f);
-    }
-#pragma unroll
-    for (int e = 0; e < 8; e++) x[e] = act_load(mixed + e);
+    for (int e = 0; e < 8; e++) x[e] = fmaf(a.v_share, y[e], (1.f - a.v_share) * x[e]);
+}
+template <class AT>
+__device__ __forceinline__ float load_value(const AttnArgs &a, int row, int g, int c) {
+    if (c >= a.vdim) return 0.f;
+    const int i = g * a.vdim + c;
+    const float x = act_load(reinterpret_cast<const AT *>(a.proj) + (size_t)row * a.ldp + a.v_off + g * a.DV + c);
+    return fmaf(a.v_share, act_load(reinterpret_cast<const AT *>(a.v_first) + (size_t)row * a.ld_first + i / a.vdim_first * a.DV_first + i % a.vdim_first), (1.f - a.v_share) * x);
 }
 
 // A block (or several, in y) per row: its query maps (with `queries`, in place), key maps and values (into the page), a vector per
 // head_lanes(DK) lanes.  WIDE: norms over the whole row, by the one block that has it, and mixed values.
 template <class AT, bool WIDE>
-__global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a, const int *__restrict__ seq, const int *__restrict__ pos, int queries, int pdl) {
+__global__ void __launch_bounds__(256, sizeof(AT) == 2 ? (WIDE ? 6 : 8) : 1) attn_prep_kernel(const AttnArgs a, const int *__restrict__ seq, const int *__restrict__ pos, int queries, int pdl) {
     __shared__ float2 red[8];
     if (pdl & 2) griddep_launch_dependents();
     const int lanes = head_lanes(a.DK), nq = queries ? a.heads * a.maps : 0, nk = a.kv_heads * a.maps, nv = nq + nk + a.kv_heads;
@@ -152,7 +144,7 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a, const 
     if (pdl & 1) griddep_wait();
     AT *proj = reinterpret_cast<AT *>(a.proj) + (size_t)r * a.ldp;
     float2 inv = make_float2(1.f, 1.f);
-    if (WIDE && a.qk_norm == QK_NORM_ALL) {
+    if (WIDE && a.whole_rows) {
         inv = row_rms(proj, a, red);
         if (threadIdx.x == 0) a.row_inv[r] = inv;
     }
@@ -167,6 +159,11 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a, const 
 #pragma unroll 1
             for (int c = piece; c < a.DV / 8; c += lanes) {
                 float x[8];
+                if (WIDE && !values_line_up(a, c * 8)) {
+#pragma unroll 1
+                    for (int e = 0; e < 8; e++) act_store(dst + page_chunk(a.DV, row, c) * 8 + e, load_value<AT>(a, r, g, c * 8 + e));
+                    continue;
+                }
                 if (WIDE) load_values<AT>(a, r, g, c * 8, x);
                 else load8(proj + a.v_off + g * a.DV + c * 8, x);
                 store8(dst + page_chunk(a.DV, row, c) * 8, x);
@@ -181,7 +178,7 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a, const 
 #pragma unroll
             for (int e = 0; e < 8; e++) x[e] = 0.f;
         }
-        if (a.prepared()) prepare_head(x, src, piece, lanes, head_prep(a, !query, r, head, query ? inv.x : inv.y));
+        if (a.prepared()) prepare_head(x, src, piece, lanes, head_prep<WIDE>(a, !query, r, head, query ? inv.x : inv.y));
         if (load && query) store8(proj + a.q_off + i * a.DK + piece * 8, x);
         else if (load && phys >= 0) store8(page + row * page_row(kw) + page_chunk(kw, row, (i - nq) % a.maps * (a.DK / 8) + piece) * 8, x);
         if (!WIDE) break;
@@ -289,8 +286,8 @@ struct Tile {
     static constexpr size_t smem = (ring > hand ? ring : hand) + (size_t)64 * LQ * 2;
 };
 
-// WINDOW: a window with kept tokens.
-template <int DK, int DV, int MAPS, bool WINDOW>
+// EXTRA: windows with kept tokens, sinks, norms over whole rows.
+template <int DK, int DV, int MAPS, bool EXTRA>
 __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_kernel(const AttnArgs a, const Seg *__restrict__ segs, const int2 *__restrict__ tiles, int qt, int pdl) {
     using T = Tile<DK, DV, MAPS>;
     using P = typename T::P;
@@ -310,7 +307,7 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
     if (r0 >= rows) return;
     const int p0 = sg.pos0 + tile.y, b0 = p0 + r0 / grp, p1 = p0 + (min(rows, r0 + ROWS) - 1) / grp;  // positions: of the tile, of the block's rows
     // keys in tiles: the kept ones when they lie apart, then those from the first one that the block's first row sees
-    const int win = first_visible(b0, a) / kBlockTokens * kBlockTokens, kept = WINDOW ? kept_apart(win, a) : 0, first = WINDOW && a.keep && !kept ? 0 : win;
+    const int win = first_visible<EXTRA>(b0, a) / kBlockTokens * kBlockTokens, kept = EXTRA ? kept_apart(win, a) : 0, first = EXTRA && a.keep && !kept ? 0 : win;
     const int n_kept = (kept + KT - 1) / KT, n_tiles = n_kept + (p1 - first) / KT + 1;
     auto tile_key = [&](int it) { return it < n_kept ? it * KT : first + (it - n_kept) * KT; };
     if (tid == 0) {
@@ -367,10 +364,10 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
             if (a.prepared()) {
                 int row, h;
                 const __nv_bfloat16 *src = source(v, row, h);
-                if (!src) row = row_base, h = kvh * grp;
+                if (!src) row = row_base, h = 0;
                 float x[8];
                 load8(reinterpret_cast<const __nv_bfloat16 *>(&raw[n]), x);
-                prepare_head(x, src ? src : proj, piece, LANES, head_prep(a, false, row, h, a.qk_norm == QK_NORM_ALL ? a.row_inv[row].x : 1.f));
+                prepare_head(x, src ? src : proj, piece, LANES, head_prep<EXTRA>(a, false, row, h, EXTRA && a.whole_rows ? a.row_inv[row].x : 1.f));
                 store8(reinterpret_cast<__nv_bfloat16 *>(&raw[n]), x);
             }
             if (piece * 8 < DK) *reinterpret_cast<uint4 *>(qs + (v % MAPS * ROWS + v / MAPS) * LQ + piece * 8) = raw[n];
@@ -383,7 +380,7 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
         const int r = r0 + warp * 16 + g + 8 * e;
         rt[e] = r < rows ? r : -1;
         hi[e] = p0 + (r < rows ? r : r0) / grp;
-        lo[e] = first_visible(hi[e], a);
+        lo[e] = first_visible<EXTRA>(hi[e], a);
     }
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[DV / 8][4];
 #pragma unroll
@@ -394,10 +391,10 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
         ldmatrix_x4(f, qs + (size_t)(map * ROWS + warp * 16 + (lane & 15)) * LQ + kk * 16 + (lane >> 4) * 8);
     };
     const float sl = a.scale * 1.4426950408889634f;
-    const int vis_lo = first_visible(p1, a);
+    const int vis_lo = first_visible<EXTRA>(p1, a);
     for (int it = 0; it < n_tiles; it++) {
         const int s = it % ST, kb = tile_key(it);
-        const bool apart = WINDOW && it < n_kept;
+        const bool apart = EXTRA && it < n_kept;
         if (!__all_sync(0xffffffffu, mbar_wait_bounded(&full[s], (it / ST) & 1, a.status, s_abort))) break;
         __nv_bfloat16 *stage = ring + s * T::stage_elems;
         if (kb + KT > p1 + 1) {  // every warp clears what it is going to read
@@ -408,7 +405,7 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
         }
         auto kat = [&](int r, int c) { return P::k(stage + (r >> 4) * P::ELEMS, r & 15, map * (DK / 8) + c); };
         auto vat = [&](int r, int c) { return P::v(stage + (r >> 4) * P::ELEMS, r & 15, c); };
-        if (WINDOW) {
+        if (EXTRA) {
             const int from[2] = {apart ? 0 : lo[0], apart ? 0 : lo[1]}, to[2] = {apart ? kept - 1 : hi[0], apart ? kept - 1 : hi[1]};
             attend_tile<DK, DV, KT, true>(qfrag, kat, vat, kb, apart || kb + KT - 1 > b0 || kb < vis_lo, from, to, a.keep, sl, m, l, o, lane);
         } else {
@@ -423,7 +420,7 @@ __global__ void __launch_bounds__(160, (Tile<DK, DV, MAPS>::BLOCKS)) attn_tile_k
         l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
         l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
         f[e] = l[e] > 0.f ? 1.f / l[e] : 0.f;
-        if (MAPS == 1 && a.sink && rt[e] >= 0) {  // its share: relative to the larger of the two scores
+        if (EXTRA && a.sink && rt[e] >= 0) {  // its share: relative to the larger of the two scores
             const float sk = a.sink[kvh * grp + rt[e] % grp] * 1.4426950408889634f, mn = fmaxf(m[e], sk), w = fast_exp2(m[e] - mn);
             f[e] = w / (l[e] * w + fast_exp2(sk - mn));
         }
@@ -553,7 +550,7 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
     const __nv_bfloat16 *proj = reinterpret_cast<const __nv_bfloat16 *>(a.proj) + (size_t)row * a.ldp;
     {
         float2 inv = make_float2(1.f, 1.f);
-        if (a.qk_norm == QK_NORM_ALL) {
+        if (a.whole_rows) {
             if (fused) {
                 inv = row_rms(proj, a, red);
             } else {
@@ -574,7 +571,7 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
 #pragma unroll
                 for (int e = 0; e < 8; e++) x[e] = 0.f;
             }
-            if (a.prepared()) prepare_head(x, src, piece, lanes, head_prep(a, key, row, key ? kvh : min(h0 + v, a.heads - 1), key ? inv.y : inv.x));
+            if (a.prepared()) prepare_head(x, src, piece, lanes, head_prep<true>(a, key, row, key ? kvh : min(h0 + v, a.heads - 1), key ? inv.y : inv.x));
             if (!load) continue;
             if (key) {
                 const int c = (v - nq) * (dk / 8) + piece;
@@ -586,10 +583,15 @@ __global__ void __launch_bounds__(128) attn_single_kernel(const AttnArgs a, cons
         }
         if (append)
             for (int c = tid; c < CV; c += 128) {
-                float x[8];
-                load_values<__nv_bfloat16>(a, row, kvh, c * 8, x);
-                store8(own + DK + c * 8, x);
-                if (phys >= 0) store8(P::v(page, r, c), x);
+                if (values_line_up(a, c * 8)) {
+                    float x[8];
+                    load_values<__nv_bfloat16>(a, row, kvh, c * 8, x);
+                    store8(own + DK + c * 8, x);
+                } else {
+#pragma unroll 1
+                    for (int e = 0; e < 8; e++) act_store(own + DK + c * 8 + e, load_value<__nv_bfloat16>(a, row, kvh, c * 8 + e));
+                }
+                if (phys >= 0) *reinterpret_cast<uint4 *>(P::v(page, r, c)) = *reinterpret_cast<const uint4 *>(own + DK + c * 8);
             }
         __syncthreads();
     }
@@ -798,10 +800,10 @@ static int32_t tensor_attention(const StepDesc &d, const AttnArgs &a, int pdl, c
             JGPT_CUDA_TRY(cudaLaunchKernelEx(&cfg, kern, a, d.segs, d.tiles, d.qt, pdl));
             return JGPT_OK;
         };
-        static thread_local int plain_for = -1, window_for = -1;
+        static thread_local int plain_for = -1, extra_for = -1;
         if constexpr (MAPS == 1) {
-            if (a.window > 0) {
-                if (int32_t rc = tiles(attn_tile_kernel<DK, DV, MAPS, true>, window_for)) return rc;
+            if (a.extra()) {
+                if (int32_t rc = tiles(attn_tile_kernel<DK, DV, MAPS, true>, extra_for)) return rc;
             } else if (int32_t rc = tiles(attn_tile_kernel<DK, DV, MAPS, false>, plain_for)) {
                 return rc;
             }

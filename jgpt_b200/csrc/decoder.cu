@@ -319,10 +319,14 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
             JGPT_REQUIRE(s.window >= 0 && s.keep >= 0 && !(s.window && (s.chunk || b.maps > 1)) && (s.window || !s.keep) && s.sink >= 0 && s.sink <= JGPT_SINK_ZERO &&
                              (!s.sink || b.maps == 1),
                          JGPT_ERR_INVALID_ARGUMENT, "layer %d: window %d with %d kept, chunk %d, sink %d, %d maps", index, s.window, s.keep, s.chunk, s.sink, b.maps);
-            if (s.qk_norm == JGPT_QK_NORM_HEAD || s.qk_norm == JGPT_QK_NORM_ALL) {
+            if (s.qk_norm) {
                 const bool all = s.qk_norm == JGPT_QK_NORM_ALL;
                 TRY(dalloc(d, (void **)&b.q_norm, sizeof(float) * (uint64_t)(all ? s.heads * b.DK : s.dim)));
                 TRY(dalloc(d, (void **)&b.k_norm, sizeof(float) * (uint64_t)(all ? s.kv_heads * b.DK : s.dim)));
+                if (s.qk_norm == JGPT_QK_NORM_UNIT) {
+                    const std::vector<float> ones((size_t)s.dim, 1.f);
+                    for (float *p : {b.q_norm, b.k_norm}) TRY(put_floats(d, p, ones.data(), 1, s.dim, Grouping()));
+                }
             }
             if (s.sink) TRY(dalloc(d, (void **)&b.sink, sizeof(float) * (uint64_t)s.heads));  // zeros
             if (s.v_mix) {
@@ -456,6 +460,7 @@ static int32_t plan_layer(Decoder *d, DLayer &y, const jgpt_layer_spec &ls, int 
     y.n_up = y.ffp + (gated ? d->ldw : 0);
     bool biased = gated;
     for (const DBranch &b : y.br) biased = biased || (b.s.kind == JGPT_MIX_ATTENTION && b.s.qkv_bias);
+    biased = biased || y.tanh_to;  // columns beside those with an activation
     if (biased) TRY(dalloc(d, (void **)&y.bias_in, sizeof(float) * (uint64_t)y.n_in));
     if (y.ff && y.ff_kind == JGPT_FF_MOE) TRY(plan_moe(d, y, ls.moe, index));
     if (d->s.norm_both) {
@@ -606,7 +611,7 @@ static uint64_t needed_roles(const DBranch &b) {
     uint64_t n = bit(JGPT_W_Q) | bit(JGPT_W_K) | bit(JGPT_W_V) | bit(JGPT_W_O);
     if (s.kind == JGPT_MIX_ATTENTION)
         return n | (s.gate ? bit(JGPT_W_G) : 0) | (s.qkv_bias ? bit(JGPT_W_Q_BIAS) | bit(JGPT_W_K_BIAS) | bit(JGPT_W_V_BIAS) : 0) |
-               (b.q_norm ? bit(JGPT_W_Q_NORM) | bit(JGPT_W_K_NORM) : 0) | (s.sink == JGPT_SINK_LEARNED ? bit(JGPT_W_SINK) : 0) |
+               (s.qk_norm == JGPT_QK_NORM_HEAD || s.qk_norm == JGPT_QK_NORM_ALL ? bit(JGPT_W_Q_NORM) | bit(JGPT_W_K_NORM) : 0) | (s.sink == JGPT_SINK_LEARNED ? bit(JGPT_W_SINK) : 0) |
                (b.v_first ? bit(JGPT_W_VMIX) : 0) |
                (s.maps > 1 ? bit(JGPT_W_LQ1) | bit(JGPT_W_LK1) | bit(JGPT_W_LQ2) | bit(JGPT_W_LK2) : 0);
     n |= bit(JGPT_W_A1) | bit(JGPT_W_A2) | bit(JGPT_W_DECAY_BIAS) | bit(JGPT_W_HEAD_NORM);
@@ -1069,7 +1074,7 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
             in.bias = y.bias_in;
             if (gated_result && d->s.token_shift) in.seg_n = y.n_mix, in.a_seg = (long long)mix_stride, in.a_cap = 1;
             if (y.tanh_to) in.act = nt::ACT_TANH, in.act_from = y.tanh_from, in.act_to = y.tanh_to;
-            TRY(product(d, &in, 1, y.tanh_to ? nt::EPI_ACT : nt::EPI_STORE, pdl));
+            TRY(product(d, &in, 1, y.tanh_to ? nt::EPI_ACT_SOME : nt::EPI_STORE, pdl));
         }
         for (DBranch &b : y.br) {
             if (b.s.kind == JGPT_MIX_ATTENTION) {
@@ -1079,7 +1084,7 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
                 a.gate = b.s.gate, a.chunk = b.s.chunk, a.scale = b.s.score_scale, a.out_scale = b.s.out_scale;
                 a.q_norm = b.q_norm, a.k_norm = b.k_norm, a.eps = eps, a.interleaved = b.s.rot_interleaved;
                 if (b.rot >= 0) a.cs = d->rots[(size_t)b.rot].out, a.half = b.s.rot_dims / 2;
-                a.qk_norm = b.s.qk_norm, a.row_inv = d->row_inv, a.window = b.s.window, a.keep = b.s.keep, a.sink = b.sink;
+                a.whole_rows = b.s.qk_norm == JGPT_QK_NORM_ALL, a.row_inv = d->row_inv, a.window = b.s.window, a.keep = b.s.keep, a.sink = b.sink;
                 if (const DBranch *f = b.v_first)
                     a.v_first = reinterpret_cast<uint8_t *>(d->proj_first) + (size_t)f->v * eb, a.ld_first = d->v_first_ld, a.vdim_first = f->s.vdim, a.DV_first = f->DV,
                     a.v_share = b.v_share;
@@ -1118,8 +1123,8 @@ static int32_t enqueue_layers(Decoder *d, Pool *p, const mix::StepDesc &sd, cons
                 const int n_act = one ? y.n_up : y.ffp;
                 nt::Problem in{d->h, y.w_gu, d->act, nullptr, R, one ? y.n_up : 2 * y.ffp, ldw, ldw, ldw, n_act, 1.f};
                 set_activation(y, in);
-                in.act_to = one ? y.ffp : in.act_to, in.bias = y.bias_up;
-                TRY(product(d, &in, 1, one ? nt::EPI_ACT : nt::EPI_GATE, pdl));
+                in.act_to = y.ffp, in.bias = y.bias_up;
+                TRY(product(d, &in, 1, !one ? nt::EPI_GATE : gated_result ? nt::EPI_ACT_SOME : nt::EPI_ACT, pdl));
                 nt::Problem down{d->act, y.w_down, d->y, nullptr, R, ldw, y.ffp, n_act, y.ffp, ldw, 1.f};
                 TRY(product(d, &down, 1, nt::EPI_STORE, pdl));
                 next.y = d->y, next.post = y.post2;

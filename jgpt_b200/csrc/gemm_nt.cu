@@ -200,10 +200,9 @@ __global__ void __launch_bounds__(256) gemm_nt_small_kernel(const SmallArgs args
         } else if (m < M && n < n_end) {
             const size_t at = (size_t)m * P.ldc + n + cn;
             if (EPI == EPI_STORE) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(P.bias ? sum[i] + P.bias[n] : sum[i]);
-            if (EPI == EPI_ACT) {
-                const float v = P.bias ? sum[i] + P.bias[n] : sum[i];
-                reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(n >= P.act_from && n < P.act_to ? activate<true>(P.act, P.p0, P.p1, v) : v);
-            }
+            if (EPI == EPI_ACT) reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(activate<true>(P.act, P.p0, P.p1, sum[i]));
+            if (EPI == EPI_ACT_SOME)
+                reinterpret_cast<__nv_bfloat16 *>(P.C)[at] = __float2bfloat16(n >= P.act_from && n < P.act_to ? activate<true>(P.act, P.p0, P.p1, sum[i]) : sum[i] + P.bias[n]);
             if (EPI == EPI_ADD_F32) reinterpret_cast<float *>(P.C)[at] = P.res_scale * P.res[at] + (P.colscale ? P.colscale[n] * sum[i] : sum[i]);
             if (EPI == EPI_SCALE_F32) reinterpret_cast<float *>(P.C)[at] = sum[i] * P.scale;
         }
@@ -286,6 +285,7 @@ static int32_t complete(const Problem *p, int n, Epilogue epi, Problem (&q)[2]) 
         q[i] = p[i];
         if (q[i].seg_n <= 0) q[i].seg_n = q[i].N;
         if (!q[i].res) q[i].res = reinterpret_cast<const float *>(q[i].C);
+        JGPT_REQUIRE(epi != EPI_ACT_SOME || q[i].bias, JGPT_ERR_INVALID_ARGUMENT, "columns without an activation need a bias");
         JGPT_REQUIRE(!q[i].grp.tiles || (i == 0 && (epi == EPI_STORE || epi == EPI_ACT) && q[i].segments() == 1 && q[i].grp.max_tiles > 0),
                      JGPT_ERR_INVALID_ARGUMENT, "rows in groups: the first product of a launch, one segment, stored or activated");
     }
@@ -313,6 +313,7 @@ int32_t launch_bf16(const Ctx *ctx, const Problem *problems, int n, Epilogue epi
         case EPI_SCALE_F32: return small_dispatch<EPI_SCALE_F32>(ctx, p, n, pdl, st);
         case EPI_GATE: return small_dispatch<EPI_GATE>(ctx, p, n, pdl, st);
         case EPI_ACT: return small_dispatch<EPI_ACT>(ctx, p, n, pdl, st);
+        case EPI_ACT_SOME: return small_dispatch<EPI_ACT_SOME>(ctx, p, n, pdl, st);
     }
     return fail(JGPT_ERR_INVALID_ARGUMENT, "unknown epilogue");
 }
@@ -375,10 +376,8 @@ __global__ void __launch_bounds__(256) gemm_nt_f32_kernel(const Problem P0, cons
                 if (n >= n_end) continue;
                 const size_t at = (size_t)m * P.ldc + n + cn;
                 if (EPI == EPI_STORE) C[at] = P.bias ? acc[i][j] + P.bias[n] : acc[i][j];
-                if (EPI == EPI_ACT) {
-                    const float v = P.bias ? acc[i][j] + P.bias[n] : acc[i][j];
-                    C[at] = n >= P.act_from && n < P.act_to ? activate<false>(P.act, P.p0, P.p1, v) : v;
-                }
+                if (EPI == EPI_ACT) C[at] = activate<false>(P.act, P.p0, P.p1, acc[i][j]);
+                if (EPI == EPI_ACT_SOME) C[at] = n >= P.act_from && n < P.act_to ? activate<false>(P.act, P.p0, P.p1, acc[i][j]) : acc[i][j] + P.bias[n];
                 if (EPI == EPI_ADD_F32) C[at] = P.res_scale * P.res[at] + (P.colscale ? P.colscale[n] * acc[i][j] : acc[i][j]);
                 if (EPI == EPI_SCALE_F32) C[at] = acc[i][j] * P.scale;
             }
@@ -403,6 +402,7 @@ int32_t launch_f32(const Problem *problems, int n, Epilogue epi, cudaStream_t st
         case EPI_SCALE_F32: gemm_nt_f32_kernel<EPI_SCALE_F32><<<grid, 256, 0, st>>>(p[0], q); break;
         case EPI_GATE: gemm_nt_f32_kernel<EPI_GATE><<<grid, 256, 0, st>>>(p[0], q); break;
         case EPI_ACT: gemm_nt_f32_kernel<EPI_ACT><<<grid, 256, 0, st>>>(p[0], q); break;
+        case EPI_ACT_SOME: gemm_nt_f32_kernel<EPI_ACT_SOME><<<grid, 256, 0, st>>>(p[0], q); break;
     }
     JGPT_CUDA_TRY(cudaGetLastError());
     return JGPT_OK;

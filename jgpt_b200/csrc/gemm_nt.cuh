@@ -15,7 +15,8 @@ enum Epilogue : int {
     EPI_ADD_F32 = 1,   // C (fp32) = residual factor * residual + column factor * sum; every element is read and written by one thread
     EPI_SCALE_F32 = 2, // C (fp32) = sum * scale
     EPI_GATE = 3,      // W rows alternate in groups of 16: 16 of the gate, 16 of the linear part; C [M, N / 2] = act(gate) * linear
-    EPI_ACT = 4,       // C (activation type) = act(sum + bias), the function picked per product, for all columns or a range of them
+    EPI_ACT = 4,       // C (activation type) = act(sum), the function picked per product
+    EPI_ACT_SOME = 5,  // the same for columns [act_from, act_to); the others get the bias (which is set) alone
 };
 enum Activation : int { ACT_NONE = 0, ACT_TANH = 1, ACT_XIELU = 2, ACT_GELU = 3, ACT_RELU = 4, ACT_RELU2 = 5 };
 
@@ -49,8 +50,8 @@ struct Problem {
     const float *res = nullptr, *colscale = nullptr;  // EPI_ADD_F32: residual [M, ldc] (null: C itself), factor per column (null: 1)
     int act = ACT_NONE;                               // EPI_ACT
     float p0 = 0.f, p1 = 0.f;                         // its parameters
-    int act_from = 0, act_to = 1 << 30;               // its columns; the others get the bias alone
-    const float *bias = nullptr;                      // EPI_STORE, EPI_ACT: per column
+    int act_from = 0, act_to = 0;                     // EPI_ACT_SOME
+    const float *bias = nullptr;                      // EPI_STORE, EPI_ACT_SOME: per column
     float res_scale = 1.f;                            // EPI_ADD_F32
     RowGroups grp;                                    // tiles set: rows in groups (EPI_STORE, EPI_ACT; one segment)
     int segments() const { return seg_n > 0 ? (N + seg_n - 1) / seg_n : 1; }

@@ -75,6 +75,16 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<const uint32_t *>(&v);
 }
 
+// bias: of v[0], on a 16-byte boundary; of n columns.
+__device__ __forceinline__ void add_bias(float (&v)[32], const float *bias, int n) {
+#pragma unroll
+    for (int q = 0; q < 32; q += 4)
+        if (q < n) {  // multiples of 8 here
+            const float4 b = __ldg(reinterpret_cast<const float4 *>(bias + q));
+            v[q] += b.x, v[q + 1] += b.y, v[q + 2] += b.z, v[q + 3] += b.w;
+        }
+}
+
 template <int BN, int EPI, int ROWS>
 __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __grid_constant__ CUtensorMap amap, const __grid_constant__ CUtensorMap wmap,
                                                                        const UmmaArgs a) {
@@ -175,19 +185,23 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
                 float v[32];
                 load_acc32(acc, quarter, c0, v);
                 if (m >= m_end) continue;
-                if (EPI == EPI_STORE || EPI == EPI_ACT) {
+                if (EPI == EPI_STORE || EPI == EPI_ACT || EPI == EPI_ACT_SOME) {
                     __nv_bfloat16 *c = reinterpret_cast<__nv_bfloat16 *>(a.C) + (size_t)m * a.ldc + n0 + c0 + cn;
                     const int n1 = n0 + c0;
-                    if (a.bias) {
+                    if (EPI == EPI_ACT_SOME) {
+                        if (n1 >= a.act_to || n1 + 32 <= a.act_from) {
+                            add_bias(v, a.bias + n1, n_end - n1);
+                        } else if (n1 >= a.act_from && n1 + 32 <= a.act_to && a.act == ACT_RELU2) {
 #pragma unroll
-                        for (int q = 0; q < 32; q++)
-                            if (n1 + q < n_end) v[q] += __ldg(a.bias + n1 + q);
-                    }
-                    if (EPI == EPI_ACT && (n1 < a.act_from || n1 + 32 > a.act_to)) {
-                        if (n1 + 32 > a.act_from && n1 < a.act_to) {
+                            for (int q = 0; q < 32; q++) v[q] = fmaxf(v[q], 0.f), v[q] *= v[q];
+                        } else {
+                            float w[32];
+#pragma unroll
+                            for (int q = 0; q < 32; q++) w[q] = activate<true>(a.act, a.p0, a.p1, v[q]);
+                            add_bias(v, a.bias + n1, n_end - n1);
 #pragma unroll
                             for (int q = 0; q < 32; q++)
-                                if (n1 + q >= a.act_from && n1 + q < a.act_to) v[q] = activate<true>(a.act, a.p0, a.p1, v[q]);
+                                if (n1 + q >= a.act_from && n1 + q < a.act_to) v[q] = w[q];
                         }
                     } else if (EPI == EPI_ACT && a.act == ACT_XIELU) {
 #pragma unroll
@@ -202,6 +216,7 @@ __global__ void __launch_bounds__(kUmmaThreads, 1) gemm_nt_umma_kernel(const __g
 #pragma unroll
                         for (int q = 0; q < 32; q++) v[q] = activate<true>(a.act, a.p0, a.p1, v[q]);
                     }
+                    if (EPI == EPI_STORE && a.bias) add_bias(v, a.bias + n1, n_end - n1);
 #pragma unroll
                     for (int q = 0; q < 4; q++)
                         if (n0 + c0 + 8 * q < n_end)  // N and seg_n are multiples of 8 here
@@ -327,7 +342,7 @@ int32_t launch_bf16_umma(const Ctx *ctx, const Problem &p, Epilogue epi, int pdl
                  JGPT_ERR_INVALID_ARGUMENT, "operand rows must start on 16-byte boundaries");
     JGPT_REQUIRE((epi != EPI_STORE || (p.N % 8 == 0 && p.ldc % 8 == 0)) && (epi != EPI_GATE || ((p.act == ACT_GELU || p.act == ACT_RELU) && p.N % 32 == 0 && p.ldc % 8 == 0)),
                  JGPT_ERR_INVALID_ARGUMENT, "output columns %d, stride %d", p.N, p.ldc);
-    JGPT_REQUIRE((epi != EPI_ACT || (p.N % 8 == 0 && p.ldc % 8 == 0)) &&
+    JGPT_REQUIRE(((epi != EPI_ACT && epi != EPI_ACT_SOME) || (p.N % 8 == 0 && p.ldc % 8 == 0)) &&
                      (p.segments() == 1 || (p.seg_n % 8 == 0 && p.c_seg % 8 == 0 && p.a_seg % 8 == 0 && epi != EPI_GATE)),
                  JGPT_ERR_INVALID_ARGUMENT, "segments of %d columns, shifts %lld / %d", p.seg_n, p.a_seg, p.c_seg);
     if (p.grp.tiles) {
@@ -336,6 +351,7 @@ int32_t launch_bf16_umma(const Ctx *ctx, const Problem &p, Epilogue epi, int pdl
     }
     switch (epi) {
         case EPI_ACT: return umma_pick<EPI_ACT>(ctx, p, pdl, st);
+        case EPI_ACT_SOME: return umma_pick<EPI_ACT_SOME>(ctx, p, pdl, st);
         case EPI_STORE: return umma_pick<EPI_STORE>(ctx, p, pdl, st);
         case EPI_ADD_F32: return umma_pick<EPI_ADD_F32>(ctx, p, pdl, st);
         case EPI_SCALE_F32: return umma_pick<EPI_SCALE_F32>(ctx, p, pdl, st);

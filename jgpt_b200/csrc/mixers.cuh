@@ -142,7 +142,6 @@ int32_t launch_moe_gather(const RouteArgs &a, const void *h, void *out, int ld, 
 // pieces, so that a page comes in as one bulk copy and eight rows are read without bank conflicts.
 __host__ __device__ constexpr int page_row(int D) { return D % 64 == 0 ? D : D + 8; }
 __host__ __device__ constexpr int page_chunk(int D, int row, int chunk) { return D % 64 == 0 ? chunk ^ (row & 7) : chunk; }
-enum QkNorm : int { QK_NORM_NONE = 0, QK_NORM_HEAD = 1, QK_NORM_ALL = 2, QK_NORM_UNIT = 3 };  // per head with weights; over the whole row; per head without
 enum HeadGate : int { GATE_NONE = 0, GATE_HEAD = 1, GATE_ELEMENT = 2 };
 struct AttnArgs {
     void *proj;         // [rows, ldp] projections of the layer
@@ -152,8 +151,8 @@ struct AttnArgs {
     int window, keep;   // a query sees the last `window` positions and the first `keep` (window 0: as chunk says)
     int chunk;          // a query sees the keys of its own chunk of this many positions (0: all earlier positions)
     float scale, out_scale;
-    int qk_norm;        // QkNorm
-    const float *q_norm, *k_norm;  // its weights: [dim], or padded [heads * DK] for whole rows
+    const float *q_norm, *k_norm;  // weights [dim] of the RMS norm of every query and key head (map); null: none
+    int whole_rows;     // the norm is that of all heads' rows at once, its weights padded [heads * DK]
     float2 *row_inv;    // [rows] 1 / root mean square of the query and key rows, written in steps with prompts
     float eps;
     const float *sink;  // [heads] score without a value; null: none
@@ -170,8 +169,9 @@ struct AttnArgs {
     int ldo, out_off;
     int sm_count;
     int *status;
-    __host__ __device__ bool prepared() const { return qk_norm || cs; }
-    bool wide() const { return qk_norm == QK_NORM_ALL || v_first; }  // a row's preparation needs more than its own heads  // heads are normed or rotated on their way
+    __host__ __device__ bool prepared() const { return q_norm || cs; }
+    bool extra() const { return window > 0 || sink || whole_rows; }  // one map
+    bool wide() const { return whole_rows || v_first; }  // a row's preparation needs more than its own heads  // heads are normed or rotated on their way
     __host__ __device__ int page_head() const { return kBlockTokens * (page_row(maps * DK) + page_row(DV)); }
 };
 int32_t launch_attention(bool f32, const StepDesc &d, const AttnArgs &a, int pdl, cudaStream_t st);
